@@ -23,7 +23,7 @@ import zlib
 import numpy as np
 import torch
 
-from ..models.qwen3 import ForwardMeta
+from ..models.qwen3 import ForwardMeta, RaggedBatch
 
 BUCKETS = [1, 2, 4, 8, 16, 24, 32, 48, 64, 96, 128, 192, 256, 384, 512, 768, 1024]
 
@@ -39,8 +39,9 @@ class DecodeRunner:
         self.n_moe = engine.model.num_moe_layers if cfg.is_moe else 0
         self.topk = cfg.moe_topk
         R, MB = max_rows, self.max_blocks
-        # host mirrors (pinned) — int32 pack: tokens | positions | seq_lens | block_table ; int64 pack: slots | seeds
-        self.h_i32 = torch.zeros(3 * R + R * MB, dtype=torch.int32).pin_memory()
+        # host mirrors (pinned) — int32 pack: tokens | positions | seq_lens | block_table | previous tokens | state slots ;
+        # int64 pack: slots | seeds
+        self.h_i32 = torch.zeros(5 * R + R * MB, dtype=torch.int32).pin_memory()
         self.h_i64 = torch.zeros(2 * R, dtype=torch.int64).pin_memory()
         self.h_f32 = torch.ones(R, dtype=torch.float32).pin_memory()
         self.h_u8 = torch.zeros(R, dtype=torch.uint8).pin_memory()
@@ -55,7 +56,10 @@ class DecodeRunner:
         self.tok_np = self.np_i32[0:R]
         self.pos_np = self.np_i32[R:2 * R]
         self.len_np = self.np_i32[2 * R:3 * R]
-        self.bt_np = self.np_i32[3 * R:].reshape(R, MB)
+        self.bt_np = self.np_i32[3 * R:3 * R + R * MB].reshape(R, MB)
+        self.prev_np = self.np_i32[3 * R + R * MB:4 * R + R * MB]
+        self.state_np = self.np_i32[4 * R + R * MB:]
+        self.state_np[:] = -1
         self.slot_np = self.np_i64[0:R]
         self.seed_np = self.np_i64[R:2 * R]
         self.slot_np[:] = -1
@@ -87,6 +91,8 @@ class DecodeRunner:
         self._err = ops._k().C.error_flag(self.d_i32)      # device error flag: raised (71) when a step samples an id outside the vocabulary
         self.last_logits = None               # [B, V] logits of the last eager step (for top-k log-probs read by the host)
         self.graphs: dict[int, tuple] = {}
+        self.graph_logits: dict[int, torch.Tensor] = {}     # logits of the graphs captured for `feed`
+        self._capturing_feed = False
         self.launches_per_graph: dict[int, int] = {}
         self.pool = None
 
@@ -108,6 +114,7 @@ class DecodeRunner:
         self.rows[row] = None
         self.len_np[row] = 0
         self.slot_np[row] = -1
+        self.state_np[row] = -1
         self.free_rows.append(row)
         req.row = None
         while self.high > 0 and self.rows[self.high - 1] is None:
@@ -130,6 +137,7 @@ class DecodeRunner:
             self.np_f32[hole], self.np_u8[hole] = self.np_f32[src], self.np_u8[src]
             self.len_np[src] = 0
             self.slot_np[src] = -1
+            self.state_np[src] = -1
             self.free_rows.append(src)
             self.free_rows.sort(reverse=True)
             while self.high > 0 and self.rows[self.high - 1] is None:
@@ -144,6 +152,18 @@ class DecodeRunner:
 
     def bucket_needed(self) -> int:
         return self._bucket(max(self.high, 1))
+
+    def _block_table(self, B: int) -> torch.Tensor:
+        R, MB = self.max_rows, self.max_blocks
+        return self.d_i32[3 * R:3 * R + R * MB].view(R, MB)[:B]
+
+    def _prev(self, B: int) -> torch.Tensor:
+        at = 3 * self.max_rows + self.max_rows * self.max_blocks
+        return self.d_i32[at:at + B]
+
+    def _state_slots(self, B: int) -> torch.Tensor:
+        at = 4 * self.max_rows + self.max_rows * self.max_blocks
+        return self.d_i32[at:at + B]
 
     def _forward(self, B: int, record: bool):
         e = self.e
@@ -162,12 +182,19 @@ class DecodeRunner:
         tokens = self.d_i32[0:B]
         meta = ForwardMeta(
             positions=self.d_i32[R:R + B], cu_seqlens=None, max_seqlen=1, kv_cache=e.kv.layers,
-            block_table=self.d_i32[3 * R:].view(R, MB)[:B], seq_lens=self.d_i32[2 * R:2 * R + B],
+            block_table=self._block_table(B), seq_lens=self.d_i32[2 * R:2 * R + B],
             slot_mapping=self.d_i64[0:B], record_topk=[] if record else None)
+        if e.ragged:
+            meta.prev_tokens, meta.state_slots = self._prev(B), self._state_slots(B)
+            meta.states = e.states.layers if e.states is not None else {}
+            meta.ragged = RaggedBatch()
         hidden = e.model(tokens, meta)
         hidden = e.ps.sp_gather(hidden)
         logits = e.model.logits(hidden)
-        if not torch.cuda.is_current_stream_capturing():
+        if torch.cuda.is_current_stream_capturing():
+            if self._capturing_feed:
+                self.graph_logits[B] = logits       # lives in the graph's pool; rewritten by every replay
+        else:
             self.last_logits = logits               # eager steps only (requests that want the k most likely tokens run eagerly)
         from .. import ops
 
@@ -179,23 +206,17 @@ class DecodeRunner:
 
     def _advance(self, B: int, k: int, record: bool):
         """Device-side hand-over between two replays of one multi-step call (rows with length 0 are padding)."""
-        R, MB = self.max_rows, self.max_blocks
+        R = self.max_rows
         from .. import ops
 
         C = ops._k().C
         C.decode_advance(self.o_tok[:B], self.o_lp[:B], self.o_routed[:B] if record else None, self.hist_tok[k, :B], self.hist_lp[k, :B],
                          self.hist_routed[k, :B] if record else None, self.d_i32[0:B], self.d_i32[R:R + B], self.d_i32[2 * R:2 * R + B],
-                         self.d_i32[3 * R:].view(R, MB)[:B], self.e.block_size, self.d_i64[0:B], self.d_i64[R:R + B],
-                         self.e.cfg.vocab_size, self._err)
+                         self._block_table(B), self.e.block_size, self.d_i64[0:B], self.d_i64[R:R + B],
+                         self.e.cfg.vocab_size, self._err, self._prev(B))
 
-    def step(self, reqs: list, step_no: int, min_bucket: int = 0, steps: int = 1):
-        """Run `steps` decode steps for the attached requests (every request must own cache blocks for `steps` more
-        tokens).  Returns (tokens, logprobs, routed | None) as numpy views indexed [row] for one step and [step, row] for
-        several."""
-        e = self.e
-        bs = e.block_size
-        if len(self.free_rows) and (self.high - len(reqs)) > max(8, len(reqs) // 4):
-            self.compact()
+    def _set_rows(self, reqs: list):
+        bs = self.e.block_size
         for r in reqs:
             row = r.row
             n = len(r.input_ids) + len(r.output_ids)
@@ -204,10 +225,54 @@ class DecodeRunner:
                 self.bt_np[row, r.bt_len:len(r.blocks)] = r.blocks[r.bt_len:]
                 r.bt_len = len(r.blocks)
             self.tok_np[row] = r.output_ids[-1] if r.output_ids else r.input_ids[-1]
+            if self.e.ragged:
+                before = r.output_ids[-2] if len(r.output_ids) > 1 else (r.input_ids[-1] if r.output_ids else
+                                                                        (r.input_ids[-2] if n > 1 else -1))
+                self.prev_np[row] = before
+                self.state_np[row] = r.state_slot
             self.pos_np[row] = pos
             self.len_np[row] = n
             self.slot_np[row] = r.blocks[pos // bs] * bs + pos % bs
             self.seed_np[row] = (r.seed * 1000003 + n) & 0x7FFFFFFFFFFFFFFF
+
+    def feed(self, reqs: list) -> torch.Tensor:
+        """One decode step whose tokens are given (the last input token of every request): logits [len(reqs), vocab].  The
+        requests hold rows for this step only; all other rows are padding."""
+        assert self.high == 0, "feeding and generating do not share a step"
+        for r in reqs:
+            self.attach(r)
+        try:
+            self._set_rows(reqs)
+            B = self._bucket(self.high)
+            self.d_i32.copy_(self.h_i32, non_blocking=True)
+            self.d_i64.copy_(self.h_i64, non_blocking=True)
+            self.d_f32.copy_(self.h_f32, non_blocking=True)
+            self.d_u8.copy_(self.h_u8, non_blocking=True)
+            key = (B, False, "feed")
+            if self.use_graph:
+                if key not in self.graphs:
+                    self._capture(key)
+                self.graphs[key].replay()
+                logits = self.graph_logits[B]
+            else:
+                self._forward(B, False)
+                logits = self.last_logits
+            rows = torch.tensor([r.row for r in reqs], dtype=torch.int64, device=self.dev)
+            out = logits.index_select(0, rows)
+            torch.cuda.current_stream().synchronize()      # the host mirrors are written again by the next step
+            return out
+        finally:
+            for r in reqs:
+                self.detach(r)
+
+    def step(self, reqs: list, step_no: int, min_bucket: int = 0, steps: int = 1):
+        """Run `steps` decode steps for the attached requests (every request must own cache blocks for `steps` more
+        tokens).  Returns (tokens, logprobs, routed | None) as numpy views indexed [row] for one step and [step, row] for
+        several."""
+        e = self.e
+        if len(self.free_rows) and (self.high - len(reqs)) > max(8, len(reqs) // 4):
+            self.compact()
+        self._set_rows(reqs)
         B = min(max(self._bucket(max(self.high, 1)), int(min_bucket)), self.max_rows)
         record = self.n_moe > 0 and any(r.return_routed_experts for r in reqs)
         self.d_i32.copy_(self.h_i32, non_blocking=True)
@@ -289,16 +354,25 @@ class DecodeRunner:
     def _capture(self, key):
         from .. import ops
 
-        B, record = key
+        B, record = key[:2]
         if self.e.lockstep_group is None:
             # eager warm-up with the same shapes (initialises per-kernel attributes and the allocator pool); lockstep
-            # engines must not run an extra forward here because their peers would not match its collectives
+            # engines must not run an extra forward here because their peers would not match its collectives.  Writing the
+            # rows' keys and values twice is harmless, stepping a recurrent state twice is not: the warm-up runs without slots
+            slots = self._state_slots(self.max_rows)
+            saved = slots.clone()
+            slots.fill_(-1)
             self._forward(B, record)
+            slots.copy_(saved)
             torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
         n0 = ops._k().launch_count()
-        with torch.cuda.graph(g, pool=self.pool):
-            self._forward(B, record)
+        self._capturing_feed = len(key) > 2
+        try:
+            with torch.cuda.graph(g, pool=self.pool):
+                self._forward(B, record)
+        finally:
+            self._capturing_feed = False
         self.launches_per_graph[key] = ops._k().launch_count() - n0
         if self.pool is None:
             self.pool = g.pool()
@@ -328,4 +402,5 @@ class DecodeRunner:
 
     def reset_graphs(self):
         self.graphs.clear()
+        self.graph_logits.clear()
         self.pool = None

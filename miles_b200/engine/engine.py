@@ -16,6 +16,7 @@ weight hand-over is then a pointer swap and `update_weights` is a version bump.
 from __future__ import annotations
 
 import itertools
+import math
 import threading
 import time
 import zlib
@@ -27,10 +28,10 @@ import numpy as np
 import torch
 
 from ..models.config import ModelConfig
-from ..models.qwen3 import ForwardMeta, Qwen3Model, build_model
+from ..models.qwen3 import SHORT_Q, ForwardMeta, Qwen3Model, RaggedBatch, build_model
 from ..parallel.state import ParallelState
 from ..types import encode_routed_experts
-from .kv_cache import KVCache, make_allocator
+from .kv_cache import KVCache, StateCache, make_allocator
 from .sampler import SamplingParams, sample
 
 
@@ -67,6 +68,7 @@ class Request:
     prefill_pos: int = 0           # tokens whose KV is in place (cached prefix + chunks already run); < len(all_ids) while prefilling
     chunk: tuple = (0, 0)          # token range [start, end) the next prefill step computes
     cached_tokens: int = 0         # prompt tokens whose KV was shared instead of recomputed
+    state_slot: int = -1           # slot of its recurrent state (models with one), held while the request has blocks
 
     @property
     def all_ids(self) -> list[int]:
@@ -121,7 +123,7 @@ class Engine:
                  seed: int = 0, use_cuda_graph: bool = True, record_routing: bool | None = None,
                  share_prompt_kv: bool = True, decode_steps_per_sync: int = 8, decode_steps_idle: int = 32,
                  prefix_cache: bool = True,
-                 chunked_prefill_size: int | None = None):
+                 chunked_prefill_size: int | None = None, mixed_batches: bool = False):
         self.cfg = cfg
         self.ps = ps or ParallelState.single()
         self.device = torch.device(device)
@@ -147,6 +149,10 @@ class Engine:
         self._agreed_steps = 1
         self.use_cuda_graph = use_cuda_graph and self.device.type == "cuda"
         hkv = cfg.num_kv_heads // self.ps.tp_size
+        # models may keep other rows than K and V per token, and fp32 state per sequence
+        rows = self.model.kv_rows() if hasattr(self.model, "kv_rows") else None
+        states = self.model.state_shapes() if hasattr(self.model, "state_shapes") else {}
+        self.ragged = bool(getattr(self.model, "ragged_batches", False))
         if num_blocks is None:
             if self.device.type == "cuda":
                 # blocks the caching allocator holds but no tensor uses (temporaries of the trainer's set-up) count as
@@ -155,19 +161,26 @@ class Engine:
                 free, total = torch.cuda.mem_get_info(self.device)
                 budget = int(free - (1.0 - mem_fraction_static) * total)
                 budget = max(budget, 1 << 30)
-                num_blocks = KVCache.blocks_for_budget(budget, len(self.model.layers), self.block_size, hkv, cfg.head_dim, dtype)
+                # recurrent states come out of the same budget as the paged cache
+                budget -= 4 * max_running_requests * sum(math.prod(s) for s in states.values())
+                num_blocks = KVCache.blocks_for_budget(max(budget, 1 << 28), len(self.model.layers), self.block_size, hkv, cfg.head_dim, dtype, rows)
             else:
                 num_blocks = 512
         lo, hi = self.model.layer_range
         self.kv = KVCache(hi - lo, num_blocks, self.block_size, hkv, cfg.head_dim, dtype, self.device,
-                          layer_ids=list(range(lo, hi)))
+                          layer_ids=list(range(lo, hi)), rows=rows)
+        self.states = StateCache(states, max_running_requests, self.device) if states else None
+        # a step may carry pieces of prompts and one token of every running request together (ragged models only)
+        self.mixed_batches = bool(mixed_batches) and self.ragged
         self.allocator = make_allocator(num_blocks)
         self.stateless = not getattr(self.model, "supports_kv_cache", True)
         # full KV blocks of finished prefills and finished requests stay in a block-granular radix tree: a later prompt that
         # starts with the same tokens (the next turn of a conversation, another sample of a prompt) computes only the rest
         from .prefix_cache import PrefixCache
 
-        self.prefix_cache = PrefixCache(self.allocator, self.block_size) if (prefix_cache and not self.stateless) else None
+        # (a recurrent state exists only where its sequence stands, not at the block boundaries of a shared prefix)
+        use_prefix = prefix_cache and not self.stateless and self.states is None
+        self.prefix_cache = PrefixCache(self.allocator, self.block_size) if use_prefix else None
         # prompts longer than this many new tokens are prefilled in pieces, one per step, each attending to the KV of the
         # pieces before it through the paged cache (None: a prompt is always one piece)
         self.chunked_prefill_size = int(chunked_prefill_size) if chunked_prefill_size else None
@@ -235,6 +248,7 @@ class Engine:
     # ---- prefill / decode disaggregation: a request's KV leaves this engine or arrives from another -------------------------
     def export_kv(self, rid: str) -> torch.Tensor:
         """KV of a finished `keep_kv` request as one tensor [layers, 2, tokens, kv heads, head dim] (a gather over its slots)."""
+        self._refuse_kv_handover()
         with self.lock:
             blocks, n = self.held_kv[rid]
             slots = self._slot_tensor(blocks, n)
@@ -242,6 +256,10 @@ class Engine:
             out = [torch.stack([self.kv.layers[l][0].flatten(0, 1).index_select(0, slots),
                                 self.kv.layers[l][1].flatten(0, 1).index_select(0, slots)]) for l in layers]
             return torch.stack(out)
+
+    def _refuse_kv_handover(self):
+        if self.ragged:
+            raise NotImplementedError("prefill / decode disaggregation hands over K and V tensors; this model caches latents and states")
 
     def _slot_tensor(self, blocks: list[int], n: int) -> torch.Tensor:
         """Flat cache slots of positions 0 … n − 1 of a request with these blocks (built with tensor ops, not a Python loop)."""
@@ -264,6 +282,7 @@ class Engine:
         Raises when the cache cannot take the prompt now (the caller retries or routes elsewhere)."""
         sp = sampling_params if isinstance(sampling_params, SamplingParams) else SamplingParams.from_dict(sampling_params)
         assert not self.stateless, "engines that re-score the whole sequence keep no KV to receive"
+        self._refuse_kv_handover()
         with self.lock:
             n = len(input_ids)
             assert kv.shape[2] == n and kv.shape[0] == len(self.kv.layers), (tuple(kv.shape), n, len(self.kv.layers))
@@ -363,6 +382,8 @@ class Engine:
                 self.prefix_cache.reset()
             self.held_kv.clear()
             self.allocator.reset()
+            if self.states is not None:
+                self.states.reset()
             return True
 
     def _cacheable(self, r: "Request") -> bool:
@@ -424,7 +445,10 @@ class Engine:
                 named = rd.update_to(int(leaf.lstrip("v"))).items()
             else:
                 named = hf_io.load_hf_dir(model_path).items()
-            load_named_into_model(self.model, named, self.cfg, self.ps)
+            loaded = load_named_into_model(self.model, named, self.cfg, self.ps)
+            missing = sorted({n for n, _ in self.model.named_parameters()} - loaded)
+            if self.ragged and missing:
+                raise ValueError(f"{model_path} lacks the tensors of {missing[:8]}")
             self._invalidate_prefix_cache()
             if weight_version is not None:
                 self.weight_version = int(weight_version)
@@ -467,6 +491,9 @@ class Engine:
                 self.kv.free()
                 self.held_kv.clear()
                 self.allocator.reset()
+                if self.states is not None:
+                    self.states.free()
+                    self.states.reset()
             if "cuda_graph" in tags:
                 self._graphs.clear()
                 if self.runner is not None:
@@ -487,6 +514,8 @@ class Engine:
                 self._weights_host = None
             if "kv_cache" in tags and not self.kv.allocated:
                 self.kv.allocate()
+                if self.states is not None:
+                    self.states.allocate()
 
     def health(self) -> dict:
         return {"status": "ok", "running": len(self.running), "waiting": len(self.waiting), "prefilling": len(self.prefilling),
@@ -547,10 +576,16 @@ class Engine:
             else:
                 self.allocator.release(r.blocks)
             r.blocks = []
+        self._release_state(r)
         self.requests.pop(r.rid, None)
         r.done.set()
         if r.on_done is not None:
             r.on_done(r)
+
+    def _release_state(self, r: Request):
+        if r.state_slot >= 0:
+            self.states.release(r.state_slot)
+            r.state_slot = -1
 
     def _retract(self, r: Request):
         """Give the blocks back; the request restarts from a prefill of prompt+output."""
@@ -559,6 +594,7 @@ class Engine:
             r.cache_nodes = []
         if r.blocks:
             self.allocator.release(r.blocks)
+        self._release_state(r)
         r.blocks, r.num_cached, r.prefill_pos = [], 0, 0
         if r in self.prefilling:
             self.prefilling.remove(r)
@@ -582,7 +618,11 @@ class Engine:
             t0 = time.perf_counter()
             batch = self._schedule_prefill()
             if batch:
+                if self.mixed_batches and self.running and self._ensure_decode_blocks(1):
+                    self._join_decodes(batch)
                 self._run_prefill(batch)
+                if self.mixed_batches:
+                    self.running = [r for r in self.running if not r.finished]
                 self.stats["prefill_s"] = self.stats.get("prefill_s", 0.0) + time.perf_counter() - t0
             elif self.running:
                 k = self._decode_lookahead()
@@ -755,6 +795,8 @@ class Engine:
             # keep headroom so running requests can still grow by one block each
             if (need - shared - len(hit)) + len(self.running) > self._free_blocks() and (self.running or batch):
                 break
+            if self.states is not None and self.states.num_free == 0:
+                break
             blocks = self._alloc_blocks(need - shared - len(hit))
             if blocks is None:
                 if not self.running and not batch and not self.prefilling:
@@ -763,6 +805,8 @@ class Engine:
                     continue
                 break
             self.waiting.popleft()
+            if self.states is not None:
+                r.state_slot = self.states.alloc()
             if lead is not None:
                 self.allocator.share(lead.blocks[:shared])
                 r.blocks = lead.blocks[:shared] + blocks
@@ -783,6 +827,15 @@ class Engine:
                     leaders[key] = r                   # only a prompt that completes in this batch can lend its KV
             batch.append(r)
         return batch
+
+    def _join_decodes(self, batch: list[Request]):
+        """One token of every running request rides along with the scheduled prompt pieces."""
+        for r in self.running:
+            r.chunk = (r.num_tokens - 1, r.num_tokens)
+            batch.append(r)
+        self.stats["decode_tokens"] += len(self.running)
+        self.stats["prefill_tokens"] -= len(self.running)
+        self.stats["mixed_steps"] = self.stats.get("mixed_steps", 0) + 1
 
     def _decode_lookahead(self) -> int:
         """Decode steps the next round trip may take: the configured count, bounded by what every running request may still
@@ -869,50 +922,13 @@ class Engine:
         Followers (identical tokens) take their leader's prompt KV — shared full blocks, a copy of the partial last block —
         and its last-position logits.  Requests whose prompt is complete after this step sample their first token."""
         lead_reqs = [r for r in batch if r.leader is None]
-        toks, pos, slots, cu = [], [], [], [0]
-        for r in lead_reqs:
-            a, b = r.chunk
-            ids = r.all_ids
-            toks += ids[a:b]
-            pos += list(range(a, b))
-            slots += self._slots(r, a, b)
-            cu.append(cu[-1] + (b - a))
         dev = self.device
         record = [] if any(r.return_routed_experts for r in batch) else None
-        whole = all(r.chunk[0] == 0 for r in lead_reqs)
-        if whole or self.stateless:
-            meta = ForwardMeta(
-                positions=torch.tensor(pos, dtype=torch.int32, device=dev),
-                cu_seqlens=torch.tensor(cu, dtype=torch.int32, device=dev),
-                max_seqlen=max((r.chunk[1] for r in lead_reqs), default=0),
-                kv_cache=None if self.stateless else self.kv.layers,
-                slot_mapping=None if self.stateless else torch.tensor(slots, dtype=torch.int64, device=dev),
-                record_topk=record, lora_slots=self._lora_slots(len(toks)))
-        else:
-            # keys of request i: positions [0, end_i) read from its blocks; queries: its new tokens [start_i, end_i)
-            gather = []
-            cu_k = [0]
-            for r in lead_reqs:
-                gather += self._slots(r, 0, r.chunk[1])
-                cu_k.append(cu_k[-1] + r.chunk[1])
-            meta = ForwardMeta(
-                positions=torch.tensor(pos, dtype=torch.int32, device=dev), cu_seqlens=None,
-                max_seqlen=max((r.chunk[1] - r.chunk[0] for r in lead_reqs), default=0),
-                kv_cache=self.kv.layers, block_table=self._block_table(lead_reqs),
-                seq_lens=torch.tensor([r.chunk[1] for r in lead_reqs], dtype=torch.int32, device=dev),
-                q_lens=torch.tensor([r.chunk[1] - r.chunk[0] for r in lead_reqs], dtype=torch.int32, device=dev),
-                slot_mapping=torch.tensor(slots, dtype=torch.int64, device=dev),
-                record_topk=record, lora_slots=self._lora_slots(len(toks)))
-            meta.extend = {"cu_q": torch.tensor(cu, dtype=torch.int32, device=dev), "cu_k": torch.tensor(cu_k, dtype=torch.int32, device=dev),
-                           "kv_slots": torch.tensor(gather, dtype=torch.int64, device=dev),
-                           "max_k": max((r.chunk[1] for r in lead_reqs), default=0)}
-            self.stats["extend_tokens"] = self.stats.get("extend_tokens", 0) + len(toks)
-        self.stats["h2d_bytes"] = self.stats.get("h2d_bytes", 0) + 4 * len(toks) * 2 + 4 * len(cu) + 8 * len(slots)
-        hidden = self._dumped_forward(torch.tensor(toks, dtype=torch.int32, device=dev), meta)
+        hidden, cu, lead_reqs = self._forward_pieces(lead_reqs, record)
         if not batch:
             return
         hidden = self.ps.sp_gather(hidden)
-        self.stats["prefill_tokens"] += len(toks)
+        self.stats["prefill_tokens"] += cu[-1]
         span = {id(r): (a, b) for r, a, b in zip(lead_reqs, cu[:-1], cu[1:])}
         for r, a, b in zip(lead_reqs, cu[:-1], cu[1:]):
             if r.logprob_start_len >= 0 and r.input_logprobs is None and r.retractions == 0:
@@ -984,10 +1000,140 @@ class Engine:
                 if self.runner is not None:
                     self.runner.attach(r)
 
+    def _forward_pieces(self, reqs: list[Request], record=None):
+        """One forward over the new tokens [start, end) = `chunk` of every request.  Returns (hidden states, offsets, the requests
+        in the order their tokens were packed)."""
+        if self.ragged:
+            # long pieces first (see RaggedBatch); the order of a batch means nothing to its requests
+            reqs = sorted(reqs, key=lambda r: r.chunk[1] - r.chunk[0] <= SHORT_Q)
+        toks, pos, slots, cu = [], [], [], [0]
+        for r in reqs:
+            a, b = r.chunk
+            ids = r.all_ids
+            toks += ids[a:b]
+            pos += list(range(a, b))
+            slots += self._slots(r, a, b)
+            cu.append(cu[-1] + (b - a))
+        dev = self.device
+        self.stats["h2d_bytes"] = self.stats.get("h2d_bytes", 0) + 4 * len(toks) * 2 + 4 * len(cu) + 8 * len(slots)
+        whole = all(r.chunk[0] == 0 for r in reqs)
+        if self.ragged:
+            meta = self._ragged_meta(reqs, toks, pos, slots, cu)
+        elif whole or self.stateless:
+            meta = ForwardMeta(
+                positions=torch.tensor(pos, dtype=torch.int32, device=dev),
+                cu_seqlens=torch.tensor(cu, dtype=torch.int32, device=dev),
+                max_seqlen=max((r.chunk[1] for r in reqs), default=0),
+                kv_cache=None if self.stateless else self.kv.layers,
+                slot_mapping=None if self.stateless else torch.tensor(slots, dtype=torch.int64, device=dev),
+                record_topk=record, lora_slots=self._lora_slots(len(toks)))
+        else:
+            # keys of request i: positions [0, end_i) read from its blocks; queries: its new tokens [start_i, end_i)
+            gather = []
+            cu_k = [0]
+            for r in reqs:
+                gather += self._slots(r, 0, r.chunk[1])
+                cu_k.append(cu_k[-1] + r.chunk[1])
+            meta = ForwardMeta(
+                positions=torch.tensor(pos, dtype=torch.int32, device=dev), cu_seqlens=None,
+                max_seqlen=max((r.chunk[1] - r.chunk[0] for r in reqs), default=0),
+                kv_cache=self.kv.layers, block_table=self._block_table(reqs),
+                seq_lens=torch.tensor([r.chunk[1] for r in reqs], dtype=torch.int32, device=dev),
+                q_lens=torch.tensor([r.chunk[1] - r.chunk[0] for r in reqs], dtype=torch.int32, device=dev),
+                slot_mapping=torch.tensor(slots, dtype=torch.int64, device=dev),
+                record_topk=record, lora_slots=self._lora_slots(len(toks)))
+            meta.extend = {"cu_q": torch.tensor(cu, dtype=torch.int32, device=dev), "cu_k": torch.tensor(cu_k, dtype=torch.int32, device=dev),
+                           "kv_slots": torch.tensor(gather, dtype=torch.int64, device=dev),
+                           "max_k": max((r.chunk[1] for r in reqs), default=0)}
+            self.stats["extend_tokens"] = self.stats.get("extend_tokens", 0) + len(toks)
+        meta.record_residual = self.record_residual
+        return self._dumped_forward(torch.tensor(toks, dtype=torch.int32, device=dev), meta), cu, reqs
+
+    record_residual: list | None = None      # set to a list: forwards append the residual stream after every layer (ragged models)
+
+    def _ragged_meta(self, reqs: list[Request], toks, pos, slots, cu) -> ForwardMeta:
+        dev = self.device
+        q_lens = [r.chunk[1] - r.chunk[0] for r in reqs]
+        n_long = sum(n > SHORT_Q for n in q_lens)
+        prev, seq = [], []
+        for b, r in enumerate(reqs):
+            a, e = r.chunk
+            if e > a:
+                prev += [r.all_ids[a - 1] if a > 0 else -1] + toks[cu[b]:cu[b + 1] - 1]
+                seq += [b] * (e - a)
+        i32 = dict(dtype=torch.int32, device=dev)
+        return ForwardMeta(
+            positions=torch.tensor(pos, **i32), max_seqlen=max(q_lens, default=0), kv_cache=self.kv.layers, block_table=self._block_table(reqs),
+            seq_lens=torch.tensor([r.chunk[1] for r in reqs], **i32), q_lens=torch.tensor(q_lens, **i32),
+            slot_mapping=torch.tensor(slots, dtype=torch.int64, device=dev), prev_tokens=torch.tensor(prev, **i32),
+            state_slots=torch.tensor([r.state_slot for r in reqs], **i32), states=self.states.layers if self.states is not None else {},
+            ragged=RaggedBatch(cu_q=torch.tensor(cu, **i32), token_seq=torch.tensor(seq, **i32), q_lens=q_lens,
+                               seq_lens=[r.chunk[1] for r in reqs], n_long=n_long, t_long=cu[n_long]))
+
+    # ---- feeding given tokens (no sampling) --------------------------------------------------------------------------
+    def open_request(self, rid: str) -> Request:
+        """A request that is fed token by token or piece by piece (`feed`) instead of generating."""
+        with self.lock:
+            if rid in self.requests:
+                raise ValueError(f"request {rid!r} is already live")
+            if len(self.requests) >= self.max_running or (self.states is not None and self.states.num_free == 0):
+                raise RuntimeError(f"no slot for request {rid!r}: {len(self.requests)} live")
+            r = Request(rid=rid, input_ids=[], sampling=SamplingParams())
+            if self.states is not None:
+                r.state_slot = self.states.alloc()
+            self.requests[rid] = r
+            return r
+
+    def close_request(self, rid: str):
+        """Give back the blocks and the state slot of a fed request."""
+        with self.lock:
+            self._finish(self.requests[rid], {"type": "abort", "message": "closed"})
+
+    @torch.no_grad()
+    def feed(self, entries: "list[tuple[Request, list[int], list[int]]]") -> torch.Tensor:
+        """One step: append each entry's tokens to its request and run all of them as one batch from the cache and state that
+        earlier steps left.  `entries`: (request, tokens, places among these tokens whose logits are wanted); returns the wanted
+        logits [n, vocab] fp32 in the order of the entries.  A batch of single tokens of started sequences takes the decode path
+        (static buffers, CUDA graphs where the engine has them); any other goes through the packed prefill path."""
+        with self.lock, self.ps.no_sequence_parallel():
+            assert self.lockstep_group is None and not self.stateless, "feeding needs a cache and a single-rank engine"
+            if len({id(r) for r, _, _ in entries}) != len(entries):
+                raise ValueError("a request appears twice in one batch")
+            for r, toks, want in entries:
+                if not toks or any(not 0 <= t < self.cfg.vocab_size for t in toks) or any(not 0 <= w < len(toks) for w in want):
+                    raise ValueError(f"request {r.rid!r}: tokens or wanted places out of range")
+                if len(r.input_ids) + len(toks) > self.max_context_len:
+                    raise ValueError(f"request {r.rid!r}: {len(r.input_ids) + len(toks)} tokens exceed the context limit {self.max_context_len}")
+            for r, toks, _ in entries:
+                r.chunk = (len(r.input_ids), len(r.input_ids) + len(toks))
+                r.input_ids += toks
+                need = self._blocks_needed(r.num_tokens) - len(r.blocks)
+                if need > 0:
+                    blocks = self._alloc_blocks(need)
+                    if blocks is None:
+                        raise RuntimeError(f"request {r.rid!r}: the cache pool has no room for {len(toks)} more tokens")
+                    r.blocks += blocks
+            reqs = [r for r, _, _ in entries]
+            self._step_count += 1
+            if self.runner is not None and all(len(t) == 1 and r.chunk[0] > 0 for r, t, _ in entries):
+                logits = self.runner.feed(reqs)
+                rows = [i for i, (_, _, w) in enumerate(entries) for _ in w]
+                out = logits[torch.tensor(rows, dtype=torch.int64, device=self.device)] if rows else logits[:0]
+            else:
+                hidden, cu, order = self._forward_pieces(reqs)
+                start = {id(r): cu[i] for i, r in enumerate(order)}
+                rows = [start[id(r)] + w for r, _, ws in entries for w in ws]
+                out = self.model.logits(hidden[torch.tensor(rows, dtype=torch.int64, device=self.device)]) if rows else hidden.new_zeros(0, self.cfg.vocab_size)
+            for r in reqs:
+                r.num_cached = r.prefill_pos = r.num_tokens
+            return out.float()
+
     def _copy_tail_blocks(self, followers: list[Request]):
         """Followers own their last (partial) prompt block: copy the leader's partial block into it, all followers and
-        all layers' K and V in one indexed copy per tensor."""
+        all layers' K and V in one indexed copy per tensor; and the leader's recurrent state into their slots."""
         bs = self.block_size
+        if self.states is not None:
+            self.states.copy([r.leader.state_slot for r in followers], [r.state_slot for r in followers])
         src, dst = [], []
         for r in followers:
             n = r.num_tokens
@@ -998,9 +1144,9 @@ class Engine:
             return
         s_idx = torch.tensor(src, dtype=torch.int64, device=self.device)
         d_idx = torch.tensor(dst, dtype=torch.int64, device=self.device)
-        for kc, vc in self.kv.layers.values():
-            kc[d_idx] = kc[s_idx]
-            vc[d_idx] = vc[s_idx]
+        for tensors in self.kv.layers.values():
+            for t in tensors:
+                t[d_idx] = t[s_idx]
 
     def _run_decode(self):
         if self.stateless:
@@ -1020,6 +1166,14 @@ class Engine:
         pos = [r.num_tokens - 1 for r in reqs]
         slots = [self._slots(r, p, p + 1)[0] for r, p in zip(reqs, pos)]
         record = [] if any(r.return_routed_experts for r in reqs) else None
+        if self.ragged:
+            for r in reqs:
+                r.chunk = (r.num_tokens - 1, r.num_tokens)
+            hidden, _, _ = self._forward_pieces(reqs)
+            self.stats["decode_tokens"] += len(reqs)
+            self._sample_and_append(reqs, self.model.logits(hidden))
+            self.running = [r for r in reqs if not r.finished]
+            return
         meta = ForwardMeta(
             positions=torch.tensor(pos, dtype=torch.int32, device=dev), cu_seqlens=None, max_seqlen=1,
             kv_cache=self.kv.layers, block_table=self._block_table(reqs),

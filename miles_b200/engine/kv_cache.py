@@ -7,6 +7,8 @@ is external to it; sizing follows its `--sglang-mem-fraction-static` knob.
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 
@@ -56,39 +58,87 @@ def make_allocator(num_blocks: int):
 
 
 class KVCache:
-    """Per-layer K and V tensors of shape [num_blocks, block_size, Hkv, D]."""
+    """Paged tensors per layer, each [num_blocks, block_size, *row]: K and V rows (Hkv, D) by default, or what a model's
+    `kv_rows()` lists per layer (one latent row; nothing for a layer that keeps no tokens or reads another layer's)."""
 
     def __init__(self, num_layers: int, num_blocks: int, block_size: int, num_kv_heads: int, head_dim: int,
-                 dtype, device, layer_ids: list[int] | None = None):
+                 dtype, device, layer_ids: list[int] | None = None, rows: "dict[int, tuple] | None" = None):
         self.num_blocks, self.block_size = num_blocks, block_size
-        self.shape = (num_blocks, block_size, num_kv_heads, head_dim)
         self.dtype, self.device = dtype, device
-        self.layer_ids = layer_ids if layer_ids is not None else list(range(num_layers))
-        self.layers: dict[int, tuple[torch.Tensor, torch.Tensor]] = {}
+        if rows is None:
+            ids = layer_ids if layer_ids is not None else list(range(num_layers))
+            rows = {l: ((num_kv_heads, head_dim), (num_kv_heads, head_dim)) for l in ids}
+        self.rows = rows
+        self.layer_ids = list(rows)
+        self.layers: dict[int, tuple[torch.Tensor, ...]] = {}
+        self.live = False
         self.allocate()
 
     def allocate(self):
-        for l in self.layer_ids:
-            self.layers[l] = (torch.zeros(self.shape, dtype=self.dtype, device=self.device),
-                              torch.zeros(self.shape, dtype=self.dtype, device=self.device))
+        for l, shapes in self.rows.items():
+            self.layers[l] = tuple(torch.zeros((self.num_blocks, self.block_size, *s), dtype=self.dtype, device=self.device) for s in shapes)
+        self.live = True
 
     def free(self):
         """Release the cache memory (engine `release_memory_occupation(tags=['kv_cache'])`)."""
         self.layers = {}
+        self.live = False
         if torch.cuda.is_available():
             torch.cuda.empty_cache()
 
     @property
     def allocated(self) -> bool:
-        return bool(self.layers)
+        return self.live
 
     def bytes(self) -> int:
-        n = 1
-        for s in self.shape:
-            n *= s
-        return 2 * n * len(self.layer_ids) * torch.empty((), dtype=self.dtype).element_size()
+        return self.num_blocks * self.bytes_per_block(self.rows, self.block_size, self.dtype)
 
     @staticmethod
-    def blocks_for_budget(bytes_budget: int, num_layers: int, block_size: int, num_kv_heads: int, head_dim: int, dtype) -> int:
-        per = 2 * num_layers * block_size * num_kv_heads * head_dim * torch.empty((), dtype=dtype).element_size()
-        return max(1, bytes_budget // per)
+    def bytes_per_block(rows: "dict[int, tuple]", block_size: int, dtype) -> int:
+        return block_size * sum(math.prod(s) for shapes in rows.values() for s in shapes) * torch.empty((), dtype=dtype).element_size()
+
+    @staticmethod
+    def blocks_for_budget(bytes_budget: int, num_layers: int, block_size: int, num_kv_heads: int, head_dim: int, dtype,
+                          rows: "dict[int, tuple] | None" = None) -> int:
+        if rows is None:
+            rows = {l: ((num_kv_heads, head_dim), (num_kv_heads, head_dim)) for l in range(num_layers)}
+        return max(1, bytes_budget // max(1, KVCache.bytes_per_block(rows, block_size, dtype)))
+
+
+class StateCache:
+    """Per-sequence fp32 state of recurrent layers: one [slots, *shape] tensor per layer and a free list of slots.  A sequence
+    holds one slot from its admission to its end; the kernels start a sequence from zero state at position 0, so a slot that is
+    used again needs no clearing."""
+
+    def __init__(self, shapes: dict[int, tuple], num_slots: int, device):
+        self.shapes, self.num_slots, self.device = shapes, num_slots, device
+        self.layers: dict[int, torch.Tensor] = {}
+        self.allocate()
+        self.reset()
+
+    def allocate(self):
+        self.layers = {l: torch.zeros((self.num_slots, *s), dtype=torch.float32, device=self.device) for l, s in self.shapes.items()}
+
+    def free(self):
+        self.layers = {}
+
+    @property
+    def num_free(self) -> int:
+        return len(self.free_slots)
+
+    def alloc(self) -> int:
+        return self.free_slots.pop()
+
+    def release(self, slot: int):
+        assert 0 <= slot < self.num_slots and slot not in self.free_slots
+        self.free_slots.append(slot)
+
+    def reset(self):
+        self.free_slots = list(range(self.num_slots - 1, -1, -1))
+
+    def copy(self, src: list[int], dst: list[int]):
+        """The states of slots `src` into slots `dst`, every layer."""
+        s = torch.tensor(src, dtype=torch.int64, device=self.device)
+        d = torch.tensor(dst, dtype=torch.int64, device=self.device)
+        for t in self.layers.values():
+            t.index_copy_(0, d, t.index_select(0, s))

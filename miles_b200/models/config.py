@@ -112,6 +112,8 @@ class ModelConfig:
             path = os.path.join(cfg, "config.json") if os.path.isdir(cfg) else cfg
             with open(path) as f:
                 cfg = json.load(f)
+        if cfg.get("architecture") in ARCHITECTURES:
+            return ARCHITECTURES[cfg["architecture"]](cfg)
         mt = cfg.get("model_type", "qwen3")
         heads = cfg["num_attention_heads"]
         head_dim = cfg.get("head_dim") or cfg["hidden_size"] // heads
@@ -150,6 +152,15 @@ class ModelConfig:
         return asdict(self)
 
 
+def _nopelorn(cfg: dict) -> ModelConfig:
+    from .nopelorn import from_config
+
+    return from_config(cfg)
+
+
+# designs whose config.json names an "architecture" of its own → reader of that file
+ARCHITECTURES = {"Nopelorn": _nopelorn}
+
 PRESETS: dict[str, ModelConfig] = {
     # CPU plumbing model of the tiny GRPO run
     "tiny": ModelConfig(),
@@ -183,7 +194,9 @@ PRESETS: dict[str, ModelConfig] = {
 
 def get_config(name_or_path: str) -> ModelConfig:
     if name_or_path not in PRESETS and not os.path.exists(name_or_path):
-        from . import families  # noqa: F401  (registers the presets of the other model families)
+        from . import families, nopelorn  # noqa: F401  (register the presets of the other model families)
+
+        PRESETS.update(nopelorn.PRESETS)
     if name_or_path in PRESETS:
         return PRESETS[name_or_path]
     if os.path.exists(name_or_path):

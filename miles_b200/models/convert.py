@@ -21,6 +21,10 @@ from .config import ModelConfig
 def to_hf(name: str, tensor: torch.Tensor, cfg: ModelConfig, *, expert_offset: int = 0, _plain: bool = False
           ) -> list[tuple[str, torch.Tensor]]:
     """Convert one *full* (un-sharded along TP) tensor of this package's layout into HF tensors."""
+    if getattr(cfg, "family", "qwen3") == "nopelorn":
+        from . import nopelorn
+
+        return nopelorn.to_checkpoint(name, tensor, cfg)
     if not _plain and getattr(cfg, "family", "qwen3") != "qwen3":
         from . import bridges           # latent / linear attention, shared experts, … of the other families
 
@@ -75,6 +79,10 @@ def to_hf(name: str, tensor: torch.Tensor, cfg: ModelConfig, *, expert_offset: i
 
 def hf_state_to_ours(hf: dict[str, torch.Tensor], cfg: ModelConfig, _plain: bool = False) -> dict[str, torch.Tensor]:
     """Assemble full tensors of this package's layout from an HF state dict."""
+    if getattr(cfg, "family", "qwen3") == "nopelorn":
+        from . import nopelorn
+
+        return nopelorn.from_checkpoint(hf, cfg)
     if not _plain and getattr(cfg, "family", "qwen3") != "qwen3":
         from . import bridges
 
@@ -161,18 +169,25 @@ def unshard_tp(name: str, parts: list[torch.Tensor], cfg: ModelConfig) -> torch.
 
 
 def load_named_into_model(model, named_tensors: Iterable[tuple[str, torch.Tensor]], cfg: ModelConfig, ps):
-    """Copy tensors into a model. Accepts this package's names (shard or full) or HF names (full)."""
+    """Copy tensors into a model. Accepts this package's names (shard or full) or HF names (full).  Returns the names loaded."""
     named = list(named_tensors)
     params = dict(model.named_parameters_global() if hasattr(model, "named_parameters_global") else model.named_parameters())
-    if named and (named[0][0].startswith("model.") or named[0][0].startswith("lm_head")):
+    if getattr(cfg, "family", "qwen3") == "nopelorn":
+        from . import nopelorn
+
+        if nopelorn.is_checkpoint(n for n, _ in named):
+            named = list(nopelorn.from_checkpoint(dict(named), cfg).items())
+    elif named and (named[0][0].startswith("model.") or named[0][0].startswith("lm_head")):
         from ..weight_update.quant_export import dequantize_named, is_quantized_stream
 
         if is_quantized_stream(named):              # fp8 / mxfp8 / nvfp4 / int4 export formats decode on arrival
             named = dequantize_named(named, next(iter(params.values())).dtype)
         named = list(hf_state_to_ours(dict(named), cfg).items())
+    loaded = set()
     for n, t in named:
         if n not in params:
             continue
+        loaded.add(n)
         p = params[n]
         if tuple(t.shape) != tuple(p.shape):
             t = shard_for_rank(n, t, cfg, ps)
@@ -183,6 +198,7 @@ def load_named_into_model(model, named_tensors: Iterable[tuple[str, torch.Tensor
             copy_into(p, t)
         elif t.data_ptr() != p.data.data_ptr():
             p.data.copy_(t)
+    return loaded
 
 
 # ---- Megatron ⇄ ours -------------------------------------------------------------------------

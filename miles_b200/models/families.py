@@ -584,6 +584,10 @@ def provider(cfg, ps, dtype, device, seed=0):
 
 def build_family_model(cfg: FamilyConfig, ps=None, dtype=torch.bfloat16, device="cpu", seed: int = 0):
     ps = ps or ParallelState.single()
+    if getattr(cfg, "layer_specs", ()):
+        from .layered import LayeredModel             # sizes given layer by layer
+
+        return LayeredModel(cfg, ps, dtype=dtype, device=device, seed=seed)
     layer_range = None
     if ps.pp_size > 1:
         per = math.ceil(cfg.num_layers / ps.pp_size)

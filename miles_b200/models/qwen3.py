@@ -47,6 +47,30 @@ class ForwardMeta:
     # prefill that continues cached KV (a prefix-cache hit, a later piece of a chunked prompt): packed offsets of the new
     # tokens (cu_q) and of every request's keys (cu_k), flat cache slots of those keys (kv_slots), longest key sequence (max_k)
     extend: "dict | None" = None
+    # models with per-sequence state and ragged batches (layered.py)
+    ragged: "RaggedBatch | None" = None
+    prev_tokens: torch.Tensor | None = None    # int32 [T] token before each new token, −1 for a sequence's first
+    state_slots: torch.Tensor | None = None    # int32 [B] recurrent-state slot per sequence (−1: padding row)
+    states: "dict[int, torch.Tensor] | None" = None      # layer → [slots, ...] fp32 states
+    record_residual: "list[torch.Tensor] | None" = None  # filled with the residual stream after every layer when not None
+
+
+@dataclass
+class RaggedBatch:
+    """New tokens of several sequences packed one after another, any number each; sequence b's new tokens are the LAST
+    q_lens[b] of its seq_lens[b] positions.  Sequences with more than `SHORT_Q` new tokens come first (`n_long` of them,
+    `t_long` tokens).  A decode step (one token per row, static buffers) has no offsets: token i belongs to row i."""
+
+    cu_q: torch.Tensor | None = None           # int32 [B + 1] offsets of the new tokens
+    token_seq: torch.Tensor | None = None      # int32 [T] sequence of each new token
+    q_lens: "list[int] | None" = None          # the same on the host
+    seq_lens: "list[int] | None" = None
+    n_long: int = 0
+    t_long: int = 0
+    scratch: dict = field(default_factory=dict)   # what the layers of one forward share (key ranges per window)
+
+
+SHORT_Q = 8      # a piece of at most this many tokens attends to the cached latents directly (see layered.py)
 
 
 class _Init:

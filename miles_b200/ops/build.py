@@ -8,6 +8,7 @@ stays in the tree (git-ignored) and is what `miles_b200.ops.cuda` loads at run t
 from __future__ import annotations
 
 import glob
+import hashlib
 import os
 
 HERE = os.path.dirname(os.path.abspath(__file__))
@@ -26,11 +27,74 @@ def sources() -> list[str]:
     return sorted(glob.glob(os.path.join(CSRC, "*.cu")) + glob.glob(os.path.join(CSRC, "*.cpp")))
 
 
+# What serving a layer-by-layer decoder (models/layered.py) takes: dense projections, its mixers, sampling.  A checkout without a
+# full build compiles only these (`build_serve`), into an extension of its own with the same interface.
+SERVE_SUFFIX = "_serve"
+SERVE_SOURCES = ["counter.cpp", "bindings.cpp", "bindings_more.cpp", "bindings_misc.cpp", "bindings_mixers.cpp", "gemm.cu", "gemm_small.cu",
+                 "gemv.cu", "misc.cu", "attention_tc.cu", "mixers.cu", "latent_attn.cu", "linear_state.cu"]
+
+
+def source_stamp() -> str:
+    """Hash of every source, header and flag: what a built extension was made from."""
+    h = hashlib.sha256(" ".join(NVCC_FLAGS).encode())
+    for path in sorted(glob.glob(os.path.join(CSRC, "*"))):
+        with open(path, "rb") as f:
+            h.update(os.path.basename(path).encode() + b"\0" + f.read())
+    return h.hexdigest()
+
+
+def _is_current(so: str) -> bool:
+    try:
+        with open(so + ".stamp") as f:
+            return os.path.exists(so) and f.read() == source_stamp()
+    except OSError:
+        return False
+
+
+def _write_stamp(so: str):
+    with open(so + ".stamp", "w") as f:
+        f.write(source_stamp())
+
+
 DEBUG_SUFFIX = "_debug"                       # the build with device-side index checks (csrc/debug.cuh)
 
 
 def debug_requested() -> bool:
     return os.environ.get("MILES_DEBUG_KERNELS", "0") == "1"
+
+
+def serve_so_path() -> str:
+    return os.path.join(BUILD_DIR + SERVE_SUFFIX, EXT_NAME + SERVE_SUFFIX + ".so")
+
+
+def build_serve(verbose: bool = False) -> str:
+    """Make sure an extension that can serve layer-by-layer decoders is built from the sources as they are: an up-to-date full
+    build if there is one, else the serving subset.  Returns its path; `load()` then picks the same one."""
+    if _is_current(so_path(False)):
+        return so_path(False)
+    so = serve_so_path()
+    if not _is_current(so):
+        from torch.utils import cpp_extension
+
+        _toolchain_env()
+        os.makedirs(os.path.dirname(so), exist_ok=True)
+        cpp_extension.load(
+            name=EXT_NAME + SERVE_SUFFIX, sources=[os.path.join(CSRC, f) for f in SERVE_SOURCES],
+            extra_cflags=["-O3", "-std=c++17", "-DMB_SERVE_SUBSET"], extra_cuda_cflags=NVCC_FLAGS, extra_include_paths=[CSRC],
+            build_directory=os.path.dirname(so), verbose=verbose, with_cuda=True)
+        _write_stamp(so)
+    return so
+
+
+def _toolchain_env():
+    # link against the system libstdc++.so (the same one libtorch uses); a toolchain that links it statically
+    # gives the extension a second, uninitialised copy of the iostream state
+    if os.path.exists("/usr/bin/g++"):
+        os.environ["CXX"] = "/usr/bin/g++"
+        os.environ["CC"] = "/usr/bin/gcc"
+    os.environ.setdefault("MAX_JOBS", str(os.cpu_count() or 8))
+    # torch adds its own -gencode list unless it finds one in the flags; ours targets sm_100a only
+    os.environ.setdefault("TORCH_CUDA_ARCH_LIST", "10.0a")
 
 
 def so_path(debug: bool | None = None) -> str:
@@ -46,27 +110,18 @@ def build(verbose: bool = False, debug: bool = False):
     if debug:
         d = BUILD_DIR + DEBUG_SUFFIX
         os.makedirs(d, exist_ok=True)
-        os.environ.setdefault("MAX_JOBS", str(os.cpu_count() or 8))
-        os.environ.setdefault("TORCH_CUDA_ARCH_LIST", "10.0a")
-        if os.path.exists("/usr/bin/g++"):
-            os.environ["CXX"] = "/usr/bin/g++"
-            os.environ["CC"] = "/usr/bin/gcc"
+        _toolchain_env()
         return cpp_extension.load(
             name=EXT_NAME + DEBUG_SUFFIX, sources=sources(), extra_cflags=["-O3", "-std=c++17"],
             extra_cuda_cflags=NVCC_FLAGS + ["-DMILES_DEBUG_BOUNDS"], extra_include_paths=[CSRC], build_directory=d, verbose=verbose,
             with_cuda=True, is_python_module=True)
     os.makedirs(BUILD_DIR, exist_ok=True)
-    # link against the system libstdc++.so (the same one libtorch uses); a toolchain that links it statically
-    # gives the extension a second, uninitialised copy of the iostream state
-    if os.path.exists("/usr/bin/g++"):
-        os.environ["CXX"] = "/usr/bin/g++"
-        os.environ["CC"] = "/usr/bin/gcc"
-    os.environ.setdefault("MAX_JOBS", str(os.cpu_count() or 8))
-    # torch adds its own -gencode list unless it finds one in the flags; ours targets sm_100a only
-    os.environ.setdefault("TORCH_CUDA_ARCH_LIST", "10.0a")
-    return cpp_extension.load(
+    _toolchain_env()
+    mod = cpp_extension.load(
         name=EXT_NAME, sources=sources(), extra_cflags=["-O3", "-std=c++17"], extra_cuda_cflags=NVCC_FLAGS,
         extra_include_paths=[CSRC], build_directory=BUILD_DIR, verbose=verbose, with_cuda=True)
+    _write_stamp(so_path(False))
+    return mod
 
 
 def load():
@@ -76,12 +131,14 @@ def load():
     import torch  # noqa: F401  (libtorch symbols must be loaded first)
 
     debug = debug_requested()
-    path = so_path(debug)
+    path, suffix = so_path(debug), DEBUG_SUFFIX if debug else ""
+    if not debug and not _is_current(path) and _is_current(serve_so_path()):
+        path, suffix = serve_so_path(), SERVE_SUFFIX
     if not os.path.exists(path):
         raise ImportError(
             f"{path} not found: build the CUDA extension with `python -m miles_b200.ops.build` "
             "(or `python -c 'import __graft_entry__ as g; g.build()'`)")
-    spec = importlib.util.spec_from_file_location(EXT_NAME + (DEBUG_SUFFIX if debug else ""), path)
+    spec = importlib.util.spec_from_file_location(EXT_NAME + suffix, path)
     mod = importlib.util.module_from_spec(spec)
     spec.loader.exec_module(mod)
     return mod

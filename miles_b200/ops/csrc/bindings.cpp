@@ -113,6 +113,7 @@ void gemm_grouped_wgrad(const at::Tensor& dY, const at::Tensor& X, at::Tensor& d
         "mb_gemm_bf16_grouped_wgrad");
 }
 
+#ifndef MB_SERVE_SUBSET
 void rmsnorm_fwd(const at::Tensor& x, const c10::optional<at::Tensor>& residual, const at::Tensor& w, at::Tensor& y,
                  const c10::optional<at::Tensor>& res_out, const c10::optional<at::Tensor>& rstd, double eps) {
   c10::cuda::CUDAGuard g(x.device());
@@ -225,6 +226,7 @@ void adamw(at::Tensor& master, const at::Tensor& grad, at::Tensor& m, at::Tensor
                  master.numel(), lr, b1, b2, eps, wd, step, cur_stream()),
         "mb_adamw");
 }
+#endif  // MB_SERVE_SUBSET
 
 }  // namespace
 
@@ -244,6 +246,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("moe_gemv", &moe_gemv);
   m.def("gemm_small_grouped", &gemm_small_grouped);
   m.def("gemm_grouped_wgrad", &gemm_grouped_wgrad);
+#ifndef MB_SERVE_SUBSET      // the training and grouped-query kernels of elementwise.cu
   m.def("rmsnorm_fwd", &rmsnorm_fwd);
   m.def("rmsnorm_bwd", &rmsnorm_bwd);
   m.def("swiglu_fwd", &swiglu_fwd);
@@ -254,5 +257,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("qk_norm_rope_cache", &qk_norm_rope_cache);
   m.def("kv_cache_write", &kv_cache_write);
   m.def("adamw", &adamw);
+#endif
   register_more(m);
 }

@@ -25,7 +25,7 @@ inline void check(int rc, const char* what) {
 void decode_advance(const at::Tensor& o_tok, const at::Tensor& o_lp, const c10::optional<at::Tensor>& o_routed, at::Tensor& h_tok,
                     at::Tensor& h_lp, const c10::optional<at::Tensor>& h_routed, at::Tensor& tok, at::Tensor& pos, at::Tensor& len,
                     const at::Tensor& block_table, int64_t block_size, at::Tensor& slot, at::Tensor& seed, int64_t vocab,
-                    at::Tensor& error_flag) {
+                    at::Tensor& error_flag, const c10::optional<at::Tensor>& prev) {
   c10::cuda::CUDAGuard g(o_tok.device());
   const int64_t B = tok.numel();
   const bool rec = o_routed.has_value() && o_routed->defined() && h_routed.has_value() && h_routed->defined();
@@ -35,7 +35,8 @@ void decode_advance(const at::Tensor& o_tok, const at::Tensor& o_lp, const c10::
                           h_lp.data_ptr<float>(), rec ? h_routed->data_ptr<int>() : nullptr, per, tok.data_ptr<int>(), pos.data_ptr<int>(),
                           len.data_ptr<int>(), block_table.data_ptr<int>(), block_table.size(1), block_size,
                           reinterpret_cast<long long*>(slot.data_ptr<int64_t>()), reinterpret_cast<long long*>(seed.data_ptr<int64_t>()), B,
-                          static_cast<int>(vocab), error_flag.data_ptr<int>(), cur_stream()),
+                          static_cast<int>(vocab), error_flag.data_ptr<int>(),
+                          prev.has_value() && prev->defined() ? prev->data_ptr<int>() : nullptr, cur_stream()),
         "mb_decode_advance");
 }
 
@@ -91,6 +92,7 @@ void logit_grad(const at::Tensor& logits, const at::Tensor& targets, const at::T
         "mb_logit_grad");
 }
 
+#ifndef MB_SERVE_SUBSET
 std::vector<at::Tensor> mxfp8_quant(const at::Tensor& x) {
   c10::cuda::CUDAGuard g(x.device());
   auto q = at::empty(x.sizes(), x.options().dtype(at::kFloat8_e4m3fn));
@@ -142,14 +144,19 @@ at::Tensor nvfp4_qdq(const at::Tensor& x, const at::Tensor& global_amax, bool fo
   return y;
 }
 
+#endif  // MB_SERVE_SUBSET
+
 }  // namespace
 
 void register_misc(pybind11::module& m) {
-  m.def("decode_advance", &decode_advance);
+  m.def("decode_advance", &decode_advance, py::arg("o_tok"), py::arg("o_lp"), py::arg("o_routed"), py::arg("h_tok"), py::arg("h_lp"),
+        py::arg("h_routed"), py::arg("tok"), py::arg("pos"), py::arg("len"), py::arg("block_table"), py::arg("block_size"), py::arg("slot"),
+        py::arg("seed"), py::arg("vocab"), py::arg("error_flag"), py::arg("prev") = py::none());
   m.def("sample_logprob", &sample_logprob);
   m.def("logit_stats", &logit_stats);
   m.def("logit_stats_finish", &logit_stats_finish);
   m.def("logit_grad", &logit_grad);
+#ifndef MB_SERVE_SUBSET
   m.def("mxfp8_quant", &mxfp8_quant);
   m.def("fp8_block_quant", &fp8_block_quant);
   m.def("int4_fake_quant", &int4_fake_quant);
@@ -172,4 +179,5 @@ void register_misc(pybind11::module& m) {
     if (mb_paged_bounds_read(r, clear) == 0) out.push_back({2, r[0], r[1], r[2], r[3]});
     return out;
   });
+#endif
 }

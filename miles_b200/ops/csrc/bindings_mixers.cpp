@@ -1,0 +1,111 @@
+// Bindings of mixers.cu, latent_attn.cu and linear_state.cu (layer-by-layer decoders).
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/extension.h>
+
+#include "launch.h"
+
+namespace {
+
+using OptTensor = c10::optional<at::Tensor>;
+
+inline cudaStream_t cur_stream() {
+  (void)cudaGetLastError();
+  mb_count_launch(1);
+  return at::cuda::getCurrentCUDAStream().stream();
+}
+inline const void* cptr(const OptTensor& t) { return t.has_value() && t->defined() ? t->data_ptr() : nullptr; }
+inline void* mptr(const OptTensor& t) { return t.has_value() && t->defined() ? t->data_ptr() : nullptr; }
+inline const int* iptr(const OptTensor& t) { return t.has_value() && t->defined() ? t->data_ptr<int>() : nullptr; }
+inline const long long* lptr(const at::Tensor& t) { return reinterpret_cast<const long long*>(t.data_ptr<int64_t>()); }
+inline int f32(const at::Tensor& t) { return t.scalar_type() == at::kFloat; }
+inline void check(int rc, const char* what) {
+  if (rc == 0) return;
+  char buf[256];
+  snprintf(buf, sizeof(buf), "%s failed with code %d (%s)", what, rc,
+           rc > 0 && rc < 1000 ? cudaGetErrorString(static_cast<cudaError_t>(rc)) : "launcher: sizes out of the kernel's range");
+  throw std::runtime_error(buf);
+}
+inline MbLatent layout(const std::vector<int64_t>& v) {
+  TORCH_CHECK(v.size() == 7, "latent layout has 7 sizes");
+  return MbLatent{static_cast<int>(v[0]), static_cast<int>(v[1]), static_cast<int>(v[2]), static_cast<int>(v[3]),
+                  static_cast<int>(v[4]), static_cast<int>(v[5]), static_cast<int>(v[6])};
+}
+
+void bigram_embedding(const at::Tensor& tok, const OptTensor& prev, const at::Tensor& embed, const OptTensor& table, int64_t buckets,
+                      int64_t mul_prev, int64_t mul_cur, at::Tensor& x, at::Tensor& xb) {
+  c10::cuda::CUDAGuard g(embed.device());
+  check(mb_bigram_embedding(tok.data_ptr<int>(), iptr(prev), embed.data_ptr(), cptr(table), buckets, mul_prev, mul_cur, x.data_ptr<float>(),
+                            xb.data_ptr(), tok.numel(), embed.size(1), f32(embed), cur_stream()),
+        "mb_bigram_embedding");
+}
+
+void output_norm(at::Tensor& x, const at::Tensor& y, const at::Tensor& nw, const at::Tensor& ls, const OptTensor& fw, at::Tensor& xb,
+                 double eps) {
+  c10::cuda::CUDAGuard g(x.device());
+  check(mb_output_norm(x.data_ptr<float>(), y.data_ptr(), nw.data_ptr(), ls.data_ptr(), cptr(fw), xb.data_ptr(), x.size(0), x.size(1), eps, f32(y),
+                       cur_stream()),
+        "mb_output_norm");
+}
+
+void clamped_glu(const at::Tensor& in, at::Tensor& out, double limit, double alpha) {
+  c10::cuda::CUDAGuard g(in.device());
+  check(mb_clamped_glu(in.data_ptr(), out.data_ptr(), out.size(0), out.size(1), limit, alpha, f32(in), cur_stream()), "mb_clamped_glu");
+}
+
+void gated_norm(const at::Tensor& o, const at::Tensor& w, const at::Tensor& gate, at::Tensor& out, double eps) {
+  c10::cuda::CUDAGuard g(o.device());
+  check(mb_gated_norm(o.data_ptr(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), o.size(0), o.size(1), eps, f32(o), cur_stream()),
+        "mb_gated_norm");
+}
+
+void latent_prep(const at::Tensor& proj, const at::Tensor& positions, const at::Tensor& slots, const at::Tensor& freq, double magnitude,
+                 const OptTensor& kv_norm, double eps, at::Tensor& cache, const OptTensor& q_abs, const OptTensor& q_full, int64_t t_long,
+                 int64_t q_nope, int64_t q_width, const std::vector<int64_t>& lay) {
+  c10::cuda::CUDAGuard g(proj.device());
+  check(mb_latent_prep(proj.data_ptr(), proj.stride(0), positions.data_ptr<int>(), lptr(slots), freq.data_ptr<double>(), magnitude, cptr(kv_norm),
+                       eps, cache.data_ptr(), mptr(q_abs), mptr(q_full), proj.size(0), t_long, q_nope, q_width, layout(lay), f32(proj),
+                       cur_stream()),
+        "mb_latent_prep");
+}
+
+// x [T, H, K] (any strides of T and H), w [H, N, K] (w_nk) or [H, K, N], y [T, H, N] (any strides of T and H)
+void head_linear(const at::Tensor& x, const at::Tensor& w, bool w_nk, at::Tensor& y) {
+  c10::cuda::CUDAGuard g(x.device());
+  TORCH_CHECK(x.stride(2) == 1 && y.stride(2) == 1 && w.is_contiguous(), "head_linear: innermost dimension must be contiguous");
+  check(mb_head_linear(x.data_ptr(), x.stride(0), x.stride(1), w.data_ptr(), w_nk, y.data_ptr(), y.stride(0), y.stride(1), x.size(0), x.size(1),
+                       y.size(2), x.size(2), f32(x), cur_stream()),
+        "mb_head_linear");
+}
+
+void latent_attend(const at::Tensor& q, const at::Tensor& cache, const at::Tensor& block_table, const OptTensor& token_seq,
+                   const at::Tensor& positions, const at::Tensor& slots, const OptTensor& sink, at::Tensor& out, double scale, int64_t window,
+                   const std::vector<int64_t>& lay) {
+  c10::cuda::CUDAGuard g(q.device());
+  check(mb_latent_attend(q.data_ptr(), cache.data_ptr(), block_table.data_ptr<int>(), block_table.size(1), cache.size(1), iptr(token_seq),
+                         positions.data_ptr<int>(), lptr(slots), cptr(sink), out.data_ptr(), q.size(0), scale, window, layout(lay), f32(q),
+                         cur_stream()),
+        "mb_latent_attend");
+}
+
+void linear_state(const at::Tensor& proj, const at::Tensor& decay, at::Tensor& state, const at::Tensor& slots, const OptTensor& cu_q,
+                  const at::Tensor& positions, at::Tensor& out) {
+  c10::cuda::CUDAGuard g(proj.device());
+  check(mb_linear_state(proj.data_ptr(), proj.stride(0), decay.data_ptr<float>(), state.data_ptr<float>(), slots.data_ptr<int>(), iptr(cu_q),
+                        positions.data_ptr<int>(), out.data_ptr(), slots.numel(), state.size(1), state.size(2), state.size(3), f32(proj),
+                        cur_stream()),
+        "mb_linear_state");
+}
+
+}  // namespace
+
+void register_mixers(pybind11::module& m) {
+  m.def("bigram_embedding", &bigram_embedding);
+  m.def("output_norm", &output_norm);
+  m.def("clamped_glu", &clamped_glu);
+  m.def("gated_norm", &gated_norm);
+  m.def("latent_prep", &latent_prep);
+  m.def("head_linear", &head_linear);
+  m.def("latent_attend", &latent_attend);
+  m.def("linear_state", &linear_state);
+}

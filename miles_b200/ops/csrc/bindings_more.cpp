@@ -43,6 +43,7 @@ void install_crash_handler() {
 }
 
 // ---- attention ---------------------------------------------------------------------------------
+#ifndef MB_SERVE_SUBSET
 void flash_fwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, at::Tensor& o, const c10::optional<at::Tensor>& lse,
                const at::Tensor& cu_seqlens, int64_t max_seqlen, double scale, bool causal) {
   c10::cuda::CUDAGuard g(q.device());
@@ -52,6 +53,8 @@ void flash_fwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, at
                      cur_stream()),
         "mb_flash_fwd");
 }
+
+#endif  // MB_SERVE_SUBSET
 
 void flash_fwd_tc(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, at::Tensor& o, const c10::optional<at::Tensor>& lse,
                   const at::Tensor& cu_seqlens, int64_t max_seqlen, double scale, bool causal, at::Tensor& err,
@@ -65,6 +68,7 @@ void flash_fwd_tc(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v,
         "mb_flash_fwd_tc");
 }
 
+#ifndef MB_SERVE_SUBSET
 void flash_bwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& o, const at::Tensor& dout,
                const at::Tensor& lse, at::Tensor& delta, at::Tensor& dq, at::Tensor& dk, at::Tensor& dv, const at::Tensor& cu_seqlens,
                int64_t max_seqlen, double scale, bool causal) {
@@ -102,6 +106,7 @@ void paged_decode(const at::Tensor& q, const at::Tensor& kc, const at::Tensor& v
                         scale, num_splits, cur_stream()),
         "mb_paged_decode");
 }
+#endif  // MB_SERVE_SUBSET
 
 }  // namespace
 
@@ -109,17 +114,21 @@ void register_moe(pybind11::module& m);    // bindings_moe.cpp
 void register_misc(pybind11::module& m);   // bindings_misc.cpp
 void register_fabric(pybind11::module& m); // bindings_fabric.cpp
 void register_extra(pybind11::module& m);  // bindings_extra.cpp
+void register_mixers(pybind11::module& m); // bindings_mixers.cpp
 
 void register_more(pybind11::module& m) {
   m.def("install_crash_handler", &install_crash_handler);
-  m.def("flash_fwd", &flash_fwd);
   m.def("flash_fwd_tc", &flash_fwd_tc);
   m.def("flash_fwd_tc_ctas_per_sm", []() { return mb_flash_fwd_tc_ctas_per_sm(); });
+  register_misc(m);
+  register_mixers(m);
+#ifndef MB_SERVE_SUBSET
+  m.def("flash_fwd", &flash_fwd);
   m.def("flash_bwd", &flash_bwd);
   m.def("flash_bwd_tc", &flash_bwd_tc);
   m.def("paged_decode", &paged_decode);
   register_moe(m);
-  register_misc(m);
   register_fabric(m);
   register_extra(m);
+#endif
 }

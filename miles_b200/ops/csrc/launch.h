@@ -128,7 +128,7 @@ int mb_sample_logprob_split(const float* logits, const float* temperature, const
                             long long* tokens, float* logprobs, int B, int V, int parts, float* ws, int* counters, cudaStream_t s);
 int mb_decode_advance(const long long* o_tok, const float* o_lp, const int* o_routed, long long* h_tok, float* h_lp, int* h_routed,
                       int routed_per_row, int* tok, int* pos, int* len, const int* block_table, int max_blocks, int block_size,
-                      long long* slot, long long* seed, int B, int vocab, int* error_flag, cudaStream_t s);
+                      long long* slot, long long* seed, int B, int vocab, int* error_flag, int* prev, cudaStream_t s);
 int mb_sample_logprob(const float* logits, const float* temperature, const uint8_t* greedy, const long long* seeds, long long step,
                       long long* tokens, float* logprobs, int B, int V, cudaStream_t s);
 int mb_logit_stats(const float* logits, long long ld, const long long* targets, float* stats, long long R, int Vc, int v0,
@@ -204,6 +204,30 @@ int mb_sparse_attention_fwd(const void* q, const void* k, const void* v, const i
 int mb_multi_copy(const long long* table, const long long* prefix, int n, long long total_chunks, cudaStream_t s);
 int mb_multi_copy2d(const long long* table, const long long* prefix, int n, long long total_items, int qdq, cudaStream_t s);
 int mb_multi_mxfp8(const long long* table, const long long* prefix, int n, long long total_chunks, int qdq, cudaStream_t s);
+
+// ---- mixers.cu (layer-by-layer decoders; f32: tensors of the model's dtype are float instead of bf16) ----
+int mb_bigram_embedding(const int* tok, const int* prev, const void* embed, const void* table, long long buckets, long long mul_prev,
+                        long long mul_cur, float* x, void* xb, int T, int D, int f32, cudaStream_t s);
+int mb_output_norm(float* x, const void* y, const void* nw, const void* ls, const void* fw, void* xb, int T, int D, float eps, int f32,
+                   cudaStream_t s);
+int mb_clamped_glu(const void* in, void* out, long long T, int F, float limit, float alpha, int f32, cudaStream_t s);
+int mb_gated_norm(const void* o, const void* w, const void* gate, long long gate_ld, void* out, int T, int C, float eps, int f32,
+                  cudaStream_t s);
+// ---- latent_attn.cu ----
+typedef struct {
+  int heads, dim, rot, vdim, rank, rank_p, pitch;   // a cached row: [rank, 0 … rank_p, rot, 0 … pitch)
+} MbLatent;
+int mb_latent_prep(const void* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
+                   const void* kv_norm, float eps, void* cache, void* q_abs, void* q_full, int T, int t_long, int q_nope, int q_width,
+                   MbLatent L, int f32, cudaStream_t s);
+int mb_head_linear(const void* x, long long x_t, long long x_h, const void* w, int w_nk, void* y, long long y_t, long long y_h, int T,
+                   int H, int N, int K, int f32, cudaStream_t s);
+int mb_latent_attend(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size, const int* token_seq,
+                     const int* positions, const long long* slots, const void* sink, void* out, int T, float scale, int window, MbLatent L,
+                     int f32, cudaStream_t s);
+// ---- linear_state.cu ----
+int mb_linear_state(const void* proj, long long ld, const float* decay, float* state, const int* state_slots, const int* cu_q,
+                    const int* positions, void* out, int B, int H, int dk, int dv, int f32, cudaStream_t s);
 
 // ---- gemm_comm.cu ----
 int mb_ag_gemm(const long long* xg_ptrs, const void* W, void* Y, int* block_counters, int rows_per_rank, int N, int K, int rank,

@@ -260,7 +260,7 @@ __global__ void decode_advance_kernel(const long long* __restrict__ o_tok, const
                                       int routed_per_row, int* __restrict__ tok, int* __restrict__ pos, int* __restrict__ len,
                                       const int* __restrict__ block_table, int max_blocks, int block_size,
                                       long long* __restrict__ slot, long long* __restrict__ seed, int B, int vocab,
-                                      int* __restrict__ error_flag) {
+                                      int* __restrict__ error_flag, int* __restrict__ prev) {
   pdl_trigger();
   pdl_wait();
   const int r = blockIdx.x * blockDim.x + threadIdx.x;
@@ -274,6 +274,7 @@ __global__ void decode_advance_kernel(const long long* __restrict__ o_tok, const
   h_lp[r] = o_lp[r];
   if (h_routed != nullptr)
     for (int i = 0; i < routed_per_row; ++i) h_routed[static_cast<long long>(r) * routed_per_row + i] = o_routed[static_cast<long long>(r) * routed_per_row + i];
+  if (prev != nullptr) prev[r] = tok[r];
   tok[r] = static_cast<int>(t);
   if (len[r] > 0) {
     const int p = pos[r] + 1;
@@ -292,11 +293,11 @@ using namespace mb;
 
 extern "C" int mb_decode_advance(const long long* o_tok, const float* o_lp, const int* o_routed, long long* h_tok, float* h_lp,
                                  int* h_routed, int routed_per_row, int* tok, int* pos, int* len, const int* block_table, int max_blocks,
-                                 int block_size, long long* slot, long long* seed, int B, int vocab, int* error_flag, cudaStream_t s) {
+                                 int block_size, long long* slot, long long* seed, int B, int vocab, int* error_flag, int* prev, cudaStream_t s) {
   if (B == 0) return 0;
   return static_cast<int>(launch_pdl(decode_advance_kernel, dim3((B + 127) / 128), dim3(128), 0, s, o_tok, o_lp, o_routed, h_tok, h_lp,
                                      h_routed, routed_per_row, tok, pos, len, block_table, max_blocks, block_size, slot, seed, B, vocab,
-                                     error_flag));
+                                     error_flag, prev));
 }
 
 extern "C" int mb_sample_logprob(const float* logits, const float* temperature, const uint8_t* greedy, const long long* seeds,

@@ -66,7 +66,10 @@ def gemm_nt(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None, *
     a, b = _c(a), _c(b)
     M, K = a.shape
     N = b.shape[0]
-    assert b.shape[1] == K and a.dtype == BF16 and b.dtype == BF16 and K % 8 == 0, (a.shape, b.shape, a.dtype)
+    assert b.shape[1] == K and a.dtype == BF16 and b.dtype == BF16, (a.shape, b.shape, a.dtype)
+    if K % 8:                     # TMA rows are multiples of 16 bytes: odd inner sizes are padded with zeros
+        pad = (0, -K % 8)
+        a, b, K = torch.nn.functional.pad(a, pad), torch.nn.functional.pad(b, pad), K + pad[1]
     if out is None:
         out = torch.empty(M, N, dtype=out_dtype or BF16, device=a.device)
     if M and N:
