@@ -88,6 +88,41 @@ void latent_attend(const at::Tensor& q, const at::Tensor& cache, const at::Tenso
         "mb_latent_attend");
 }
 
+void latent_gather(const at::Tensor& cache, const at::Tensor& block_table, const at::Tensor& cu_k, const at::Tensor& base, at::Tensor& out) {
+  c10::cuda::CUDAGuard g(cache.device());
+  check(mb_latent_gather(cache.data_ptr(), block_table.data_ptr<int>(), block_table.size(1), cache.size(1), cu_k.data_ptr<int>(),
+                         base.data_ptr<int>(), out.data_ptr(), base.numel(), out.size(0), cache.size(2), cur_stream()),
+        "mb_latent_gather");
+}
+
+void head_linear_mma(const at::Tensor& x, const at::Tensor& w, bool w_nk, at::Tensor& y) {
+  c10::cuda::CUDAGuard g(x.device());
+  TORCH_CHECK(x.stride(2) == 1 && y.stride(2) == 1 && w.is_contiguous(), "head_linear_mma: innermost dimension must be contiguous");
+  check(mb_head_linear_mma(x.data_ptr(), x.stride(0), x.stride(1), w.data_ptr(), w_nk, y.data_ptr(), y.stride(0), y.stride(1), x.size(0),
+                           x.size(1), y.size(2), x.size(2), cur_stream()),
+        "mb_head_linear_mma");
+}
+
+void latent_decode(const at::Tensor& q, const at::Tensor& cache, const at::Tensor& block_table, const OptTensor& token_seq,
+                   const at::Tensor& positions, const at::Tensor& slots, const OptTensor& sink, at::Tensor& part_o, at::Tensor& part_ml,
+                   at::Tensor& out, double scale, int64_t window, int64_t splits, const std::vector<int64_t>& lay) {
+  c10::cuda::CUDAGuard g(q.device());
+  mb_count_launch(1);
+  check(mb_latent_decode(q.data_ptr(), cache.data_ptr(), block_table.data_ptr<int>(), block_table.size(1), cache.size(1), iptr(token_seq),
+                         positions.data_ptr<int>(), lptr(slots), cptr(sink), part_o.data_ptr<float>(), part_ml.data_ptr<float>(), out.data_ptr(),
+                         q.size(0), scale, window, splits, cache.size(0), layout(lay), cur_stream()),
+        "mb_latent_decode");
+}
+
+void latent_prefill(const at::Tensor& q, const at::Tensor& kv, const at::Tensor& lat, at::Tensor& o, const OptTensor& sink, const at::Tensor& cu_q,
+                    const at::Tensor& cu_k, int64_t n_seq, int64_t max_q, double scale, int64_t window, const std::vector<int64_t>& lay,
+                    at::Tensor& err) {
+  c10::cuda::CUDAGuard g(q.device());
+  check(mb_latent_prefill(q.data_ptr(), kv.data_ptr(), lat.data_ptr(), o.data_ptr(), cptr(sink), cu_q.data_ptr<int>(), cu_k.data_ptr<int>(), n_seq,
+                          max_q, q.size(0), lat.size(0), scale, window, layout(lay), err.data_ptr<int>(), cur_stream()),
+        "mb_latent_prefill");
+}
+
 void linear_state(const at::Tensor& proj, const at::Tensor& decay, at::Tensor& state, const at::Tensor& slots, const OptTensor& cu_q,
                   const at::Tensor& positions, at::Tensor& out) {
   c10::cuda::CUDAGuard g(proj.device());
@@ -107,5 +142,9 @@ void register_mixers(pybind11::module& m) {
   m.def("latent_prep", &latent_prep);
   m.def("head_linear", &head_linear);
   m.def("latent_attend", &latent_attend);
+  m.def("latent_gather", &latent_gather);
+  m.def("head_linear_mma", &head_linear_mma);
+  m.def("latent_decode", &latent_decode);
+  m.def("latent_prefill", &latent_prefill);
   m.def("linear_state", &linear_state);
 }

@@ -225,6 +225,17 @@ int mb_head_linear(const void* x, long long x_t, long long x_h, const void* w, i
 int mb_latent_attend(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                      const int* positions, const long long* slots, const void* sink, void* out, int T, float scale, int window, MbLatent L,
                      int f32, cudaStream_t s);
+// ---- latent_decode.cu (bf16 tensor cores) ----
+int mb_latent_gather(const void* cache, const int* block_table, int max_blocks, int block_size, const int* cu_k, const int* base, void* out,
+                     int n_seq, int total, int pitch, cudaStream_t s);
+int mb_head_linear_mma(const void* x, long long x_t, long long x_h, const void* w, int w_nk, void* y, long long y_t, long long y_h, int T,
+                       int H, int N, int K, cudaStream_t s);
+int mb_latent_decode(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size, const int* token_seq,
+                     const int* positions, const long long* slots, const void* sink, float* part_o, float* part_ml, void* out, int T,
+                     float scale, int window, int splits, int num_blocks, MbLatent L, cudaStream_t s);
+// ---- attention_latent_tc.cu (tcgen05) ----
+int mb_latent_prefill(const void* q, const void* kv, const void* lat, void* o, const void* sink, const int* cu_q, const int* cu_k, int n_seq,
+                      int max_q, int t_long, int tk, float scale, int window, MbLatent L, int* error_flag, cudaStream_t s);
 // ---- linear_state.cu ----
 int mb_linear_state(const void* proj, long long ld, const float* decay, float* state, const int* state_slots, const int* cu_q,
                     const int* positions, void* out, int B, int H, int dk, int dv, int f32, cudaStream_t s);

@@ -7,7 +7,7 @@ from __future__ import annotations
 
 import torch
 
-from .cuda import C, gemm_nt
+from .cuda import BF16, C
 
 
 def _c(x):
@@ -51,21 +51,69 @@ def linear_state(proj, H, dk, dv, decay, state, meta):
     return out
 
 
+# bf16 sizes the tensor-core kernels take; anything else runs the any-size kernels of latent_attn.cu
+def _mma_ok(lay, dt) -> bool:
+    return dt == BF16 and lay.dim % 8 == 0 and lay.vdim % 8 == 0 and lay.rank % 8 == 0 and lay.rot % 8 == 0 and lay.rank_p <= 512 and lay.pitch <= 640
+
+
+def _prefill_ok(lay, dt, scale) -> bool:
+    return _mma_ok(lay, dt) and lay.dim <= 128 and lay.rot <= 64 and lay.vdim <= 128 and scale > 0
+
+
+def _key_ranges(meta, window: int):
+    """Keys the long pieces of a batch can see: packed offsets [n + 1] and first position per sequence (device), and their number."""
+    rg = meta.ragged
+    if window not in rg.scratch:
+        base = [max(0, s - q - window + 1) if window else 0 for s, q in zip(rg.seq_lens[: rg.n_long], rg.q_lens)]
+        cu = [0]
+        for s, b in zip(rg.seq_lens, base):
+            cu.append(cu[-1] + s - b)
+        t = torch.tensor(cu + base, dtype=torch.int32).to(meta.positions.device)
+        rg.scratch[window] = (t[: len(cu)], t[len(cu):], cu[-1], max(rg.q_lens[: rg.n_long]))
+    return rg.scratch[window]
+
+
+def _head_linear(x, w, w_nk, y, fast):
+    (C.head_linear_mma if fast else C.head_linear)(x, w, w_nk, y)
+
+
 def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps):
-    T, H = proj.shape[0], lay.heads
+    T, H, rg = proj.shape[0], lay.heads, meta.ragged
     sizes = [H, lay.dim, lay.rot, lay.vdim, lay.rank, lay.rank_p, lay.pitch]
     dt, dev = proj.dtype, proj.device
-    t_long = 0
-    q_abs = torch.empty(T - t_long, H, lay.pitch, dtype=dt, device=dev)
-    C.latent_prep(proj, meta.positions, meta.slot_mapping, freq, float(magnitude), kv_norm, float(eps), cache, q_abs, None, t_long, 0, 0, sizes)
-    w_uk = w_ukv[: H * lay.dim].view(H, lay.dim, lay.rank)
-    w_uv = w_ukv[H * lay.dim:].view(H, lay.vdim, lay.rank)
+    fast = _mma_ok(lay, dt)
+    t_long = rg.t_long if _prefill_ok(lay, dt, scale) else 0
+    n_short = T - t_long
+    q_nope = (lay.dim + 63) // 64 * 64
+    q_abs = torch.empty(n_short, H, lay.pitch, dtype=dt, device=dev)
+    q_full = torch.empty(t_long, H, q_nope + 64, dtype=dt, device=dev)
+    C.latent_prep(proj, meta.positions, meta.slot_mapping, freq, float(magnitude), kv_norm, float(eps), cache, q_abs, q_full, t_long, q_nope,
+                  q_nope + 64, sizes)
     out = torch.empty(T, H, lay.vdim, dtype=dt, device=dev)
-    q_nope = proj[t_long:, : lay.q_rows].unflatten(1, (H, lay.dim + lay.rot))[..., : lay.dim]
-    C.head_linear(q_nope, w_uk, False, q_abs[..., : lay.rank])
-    o_lat = torch.empty(T - t_long, H, lay.rank, dtype=dt, device=dev)
-    seq = meta.ragged.token_seq
-    C.latent_attend(q_abs, cache, meta.block_table, seq[t_long:] if seq is not None else None, meta.positions[t_long:], meta.slot_mapping[t_long:],
-                    sink, o_lat, float(scale), int(window), sizes)
-    C.head_linear(o_lat, w_uv, True, out[t_long:])
+    if n_short:
+        w_uk, w_uv = w_ukv[: H * lay.dim].view(H, lay.dim, lay.rank), w_ukv[H * lay.dim:].view(H, lay.vdim, lay.rank)
+        qn = proj[t_long:, : lay.q_rows].unflatten(1, (H, lay.dim + lay.rot))[..., : lay.dim]
+        aligned = fast and proj.stride(0) % 8 == 0
+        _head_linear(qn, w_uk, False, q_abs[..., : lay.rank], aligned)
+        o_lat = torch.empty(n_short, H, lay.rank, dtype=dt, device=dev)
+        seq = rg.token_seq[t_long:] if rg.token_seq is not None else None
+        pos, slots = meta.positions[t_long:], meta.slot_mapping[t_long:]
+        if fast:
+            # enough (token, head group, split) CTAs for the 148 SMs, one resident per SM
+            groups = n_short * -(-H // (32 if H > 16 else 16))
+            splits = max(1, min(16, 296 // groups, -(-(window or 4096) // 64)))
+            part_o = torch.empty(n_short * H * splits * lay.rank_p, dtype=torch.float32, device=dev)
+            part_ml = torch.empty(n_short * H * splits * 2, dtype=torch.float32, device=dev)
+            C.latent_decode(q_abs, cache, meta.block_table, seq, pos, slots, sink, part_o, part_ml, o_lat, float(scale), int(window), splits, sizes)
+        else:
+            C.latent_attend(q_abs, cache, meta.block_table, seq, pos, slots, sink, o_lat, float(scale), int(window), sizes)
+        _head_linear(o_lat, w_uv, True, out[t_long:], fast)
+    if t_long:
+        cu_k, base, total, max_q = _key_ranges(meta, window)
+        lat = torch.empty(total, lay.pitch, dtype=dt, device=dev)
+        C.latent_gather(cache, meta.block_table, cu_k, base, lat)
+        N = H * (lay.dim + lay.vdim)
+        kv = torch.empty(total, N, dtype=dt, device=dev)
+        C.gemm(lat, w_ukv, kv, total, N, lay.rank, lay.pitch, lay.rank, N, False, False, False, None, 0)
+        C.latent_prefill(q_full, kv, lat, out, sink, rg.cu_q, cu_k, rg.n_long, max_q, float(scale), int(window), sizes, C.error_flag(proj))
     return out.view(T, H * lay.vdim)
