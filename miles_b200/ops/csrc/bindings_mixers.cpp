@@ -132,6 +132,17 @@ void linear_state(const at::Tensor& proj, const at::Tensor& decay, at::Tensor& s
         "mb_linear_state");
 }
 
+void linear_chunk(const at::Tensor& proj, const at::Tensor& decay, at::Tensor& state, const at::Tensor& slots, const at::Tensor& positions,
+                  const at::Tensor& segs, const at::Tensor& seq_segs, const OptTensor& seg_state, at::Tensor& out) {
+  c10::cuda::CUDAGuard g(proj.device());
+  const bool multi = seg_state.has_value() && seg_state->defined();
+  if (multi) mb_count_launch(2);
+  check(mb_linear_chunk(proj.data_ptr(), proj.stride(0), decay.data_ptr<float>(), state.data_ptr<float>(), slots.data_ptr<int>(),
+                        positions.data_ptr<int>(), segs.data_ptr<int>(), seq_segs.data_ptr<int>(), multi ? seg_state->data_ptr<float>() : nullptr,
+                        out.data_ptr(), seq_segs.numel() - 1, segs.size(0), state.size(1), state.size(2), state.size(3), cur_stream()),
+        "mb_linear_chunk");
+}
+
 }  // namespace
 
 void register_mixers(pybind11::module& m) {
@@ -147,4 +158,5 @@ void register_mixers(pybind11::module& m) {
   m.def("latent_decode", &latent_decode);
   m.def("latent_prefill", &latent_prefill);
   m.def("linear_state", &linear_state);
+  m.def("linear_chunk", &linear_chunk);
 }

@@ -239,6 +239,9 @@ int mb_latent_prefill(const void* q, const void* kv, const void* lat, void* o, c
 // ---- linear_state.cu ----
 int mb_linear_state(const void* proj, long long ld, const float* decay, float* state, const int* state_slots, const int* cu_q,
                     const int* positions, void* out, int B, int H, int dk, int dv, int f32, cudaStream_t s);
+// ---- linear_chunk.cu (bf16 tensor cores) ----
+int mb_linear_chunk(const void* proj, long long ld, const float* decay, float* state, const int* slots, const int* positions, const int* segs,
+                    const int* seq_segs, float* seg_state, void* out, int n_seq, int n_seg, int H, int dk, int dv, cudaStream_t s);
 
 // ---- gemm_comm.cu ----
 int mb_ag_gemm(const long long* xg_ptrs, const void* W, void* Y, int* block_counters, int rows_per_rank, int N, int K, int rank,

@@ -47,8 +47,35 @@ def gated_norm(o, w, gate, eps):
 
 def linear_state(proj, H, dk, dv, decay, state, meta):
     out = torch.empty(proj.shape[0], H * dv, dtype=proj.dtype, device=proj.device)
-    C.linear_state(proj, decay, state, meta.state_slots, meta.ragged.cu_q, meta.positions, out)
+    rg, slots, cu_q = meta.ragged, meta.state_slots, meta.ragged.cu_q
+    if rg.n_long and proj.dtype == BF16 and dk % 8 == 0 and dv % 8 == 0 and dk <= 128 and dv <= 128 and proj.stride(0) % 8 == 0:
+        # long pieces in chunks on the tensor cores, the short ones behind them token by token
+        segs, seq_segs, multi = _segments(meta, H)
+        seg_state = torch.empty(segs.shape[0], H, dk, dv, dtype=torch.float32, device=proj.device) if multi else None
+        C.linear_chunk(proj, decay, state, slots, meta.positions, segs, seq_segs, seg_state, out)
+        if slots.numel() == rg.n_long:
+            return out
+        slots, cu_q = slots[rg.n_long:], cu_q[rg.n_long:]
+    C.linear_state(proj, decay, state, slots, cu_q, meta.positions, out)
     return out
+
+
+def _segments(meta, H: int):
+    """Cut the long pieces of a batch into segments of whole 64-token chunks, about four (segment, head) CTAs per SM.  Returns
+    ([n, 4] (sequence, first token, end, last of its sequence), offsets per sequence, any sequence cut)."""
+    rg = meta.ragged
+    size = min(2048, max(128, -(-rg.t_long * H // (4 * 148 * 64)) * 64))
+    key = ("segments", size)
+    if key not in rg.scratch:
+        segs, cu, t = [], [0], 0
+        for b, n in enumerate(rg.q_lens[: rg.n_long]):
+            for a in range(0, n, size):
+                segs += [b, t + a, t + min(n, a + size), int(a + size >= n)]
+            t += n
+            cu.append(len(segs) // 4)
+        d = torch.tensor(segs + cu, dtype=torch.int32).to(meta.positions.device)
+        rg.scratch[key] = (d[: len(segs)].view(-1, 4), d[len(segs):], len(segs) // 4 > rg.n_long)
+    return rg.scratch[key]
 
 
 # bf16 sizes the tensor-core kernels take; anything else runs the any-size kernels of latent_attn.cu
