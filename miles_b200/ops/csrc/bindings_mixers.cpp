@@ -48,6 +48,14 @@ void output_norm(at::Tensor& x, const at::Tensor& y, const at::Tensor& nw, const
         "mb_output_norm");
 }
 
+void gemv_output_norm(const at::Tensor& x, const at::Tensor& y, const at::Tensor& nw, const at::Tensor& ls, double eps, const at::Tensor& w,
+                      at::Tensor& out, at::Tensor& x_out, bool static_w) {
+  c10::cuda::CUDAGuard g(x.device());
+  check(mb_gemv_output_norm(x.data_ptr<float>(), y.data_ptr(), nw.data_ptr(), ls.data_ptr(), eps, w.data_ptr(), out.data_ptr(), out.stride(0),
+                            x_out.data_ptr<float>(), x.size(0), w.size(0), x.size(1), static_w, cur_stream()),
+        "mb_gemv_output_norm");
+}
+
 void clamped_glu(const at::Tensor& in, at::Tensor& out, double limit, double alpha) {
   c10::cuda::CUDAGuard g(in.device());
   check(mb_clamped_glu(in.data_ptr(), out.data_ptr(), out.size(0), out.size(1), limit, alpha, f32(in), cur_stream()), "mb_clamped_glu");
@@ -148,6 +156,7 @@ void linear_chunk(const at::Tensor& proj, const at::Tensor& decay, at::Tensor& s
 void register_mixers(pybind11::module& m) {
   m.def("bigram_embedding", &bigram_embedding);
   m.def("output_norm", &output_norm);
+  m.def("gemv_output_norm", &gemv_output_norm);
   m.def("clamped_glu", &clamped_glu);
   m.def("gated_norm", &gated_norm);
   m.def("latent_prep", &latent_prep);

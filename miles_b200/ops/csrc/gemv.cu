@@ -164,6 +164,50 @@ __device__ __forceinline__ void stage_rows(uint8_t* xs, int rows, int valid, int
   }
 }
 
+// Output-norm form: x' = x + y / rms(y) · norm_w · scale_w with an fp32 residual x (block 0 writes x' to x_out, another buffer: every
+// CTA reads x); the staged value is bf16(x').
+__device__ __forceinline__ void stage_rows_output_norm(uint8_t* xs, int rows, int valid, int K, const bf16* __restrict__ y,
+                                                       const float* __restrict__ x, const bf16* __restrict__ norm_w,
+                                                       const bf16* __restrict__ scale_w, float eps, float* x_out) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int nv = K / 8, stride = staged_stride(K);
+  for (int r = warp; r < rows; r += kWarps) {
+    uint8_t* row = xs + r * stride;
+    if (r >= valid) {
+      for (int v = lane; v < nv; v += 32) *reinterpret_cast<uint4*>(row + v * 16) = make_uint4(0, 0, 0, 0);
+      continue;
+    }
+    const bf16* yr = y + static_cast<long long>(r) * K;
+    const float* xr = x + static_cast<long long>(r) * K;
+    float ss = 0.f;
+#pragma unroll 4
+    for (int v = lane; v < nv; v += 32) ss += sumsq8(*reinterpret_cast<const uint4*>(yr + v * 8));
+    const float rstd = __fdiv_rn(1.f, __fsqrt_rn(__fdiv_rn(warp_sum(ss), static_cast<float>(K)) + eps));
+#pragma unroll 2
+    for (int v = lane; v < nv; v += 32) {
+      const uint4 yv = *reinterpret_cast<const uint4*>(yr + v * 8), nv4 = *reinterpret_cast<const uint4*>(norm_w + v * 8),
+                  sv = *reinterpret_cast<const uint4*>(scale_w + v * 8);
+      float4 xa = *reinterpret_cast<const float4*>(xr + v * 8), xb = *reinterpret_cast<const float4*>(xr + v * 8 + 4);
+      const float2 y0 = unpack2(yv.x), y1 = unpack2(yv.y), y2 = unpack2(yv.z), y3 = unpack2(yv.w);
+      const float2 n0 = unpack2(nv4.x), n1 = unpack2(nv4.y), n2 = unpack2(nv4.z), n3 = unpack2(nv4.w);
+      const float2 s0 = unpack2(sv.x), s1 = unpack2(sv.y), s2 = unpack2(sv.z), s3 = unpack2(sv.w);
+      xa.x += y0.x * rstd * n0.x * s0.x;
+      xa.y += y0.y * rstd * n0.y * s0.y;
+      xa.z += y1.x * rstd * n1.x * s1.x;
+      xa.w += y1.y * rstd * n1.y * s1.y;
+      xb.x += y2.x * rstd * n2.x * s2.x;
+      xb.y += y2.y * rstd * n2.y * s2.y;
+      xb.z += y3.x * rstd * n3.x * s3.x;
+      xb.w += y3.y * rstd * n3.y * s3.y;
+      if (blockIdx.x == 0) {
+        *reinterpret_cast<float4*>(x_out + static_cast<long long>(r) * K + v * 8) = xa;
+        *reinterpret_cast<float4*>(x_out + static_cast<long long>(r) * K + v * 8 + 4) = xb;
+      }
+      *reinterpret_cast<uint4*>(row + v * 16) = make_uint4(pack2(xa.x, xa.y), pack2(xa.z, xa.w), pack2(xb.x, xb.y), pack2(xb.z, xb.w));
+    }
+  }
+}
+
 // Plain copy of rows [0, valid) of a [*, K] bf16 matrix into shared memory with cp.async (every piece in flight at once, no
 // registers); rows [valid, rows) are zeroed.  The caller commits the group and waits for it before the CTA barrier.
 __device__ __forceinline__ void stage_rows_async(uint8_t* xs, int rows, int valid, int K, const bf16* __restrict__ x) {
@@ -190,13 +234,19 @@ struct GemvParams {
   int out_fp32;
   bf16* res_out;          // [M, K] or null: bf16(x + residual), written by block 0
   bf16* xn_out;           // [M, K] or null: the normalised activations, written by block 0
+  const float* x32;       // output-norm form: fp32 residual, layer scale, and where the new residual goes
+  const bf16* scale_w;
+  float* x32_out;
   int M, N, K;
   int static_w;           // W is not written by a kernel that may still run: its first loads go before the dependency wait
 };
 
+enum GemvMode { kPlain = 0, kAddNorm = 1, kOutputNorm = 2 };
+
 // NT: groups of 8 tokens (1 or 2); S: ring stages.  One CTA = 16 output rows; its 8 warps take the 32-wide k chunks round-robin.
-template <int NT, bool NORM, int S>
+template <int NT, int MODE, int S>
 __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
+  constexpr bool NORM = MODE == kAddNorm;
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float red[kWarps][NT][16][8];
   __shared__ float rstd_s[NT * 8];
@@ -225,6 +275,8 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   if (p.static_w) pdl_wait();          // static weights: their first loads are already in flight
   if (NORM) {
     stage_rows<true>(xs, NT * 8, p.M, p.K, p.x, p.residual, p.norm_w, p.eps, p.res_out, rstd_s);
+  } else if (MODE == kOutputNorm) {
+    stage_rows_output_norm(xs, NT * 8, p.M, p.K, p.x, p.x32, p.norm_w, p.scale_w, p.eps, p.x32_out);
   } else {
     stage_rows_async(xs, NT * 8, p.M, p.K, p.x);
     cp_commit();
@@ -555,16 +607,16 @@ static cudaError_t set_smem(K kernel, int bytes) {
 static constexpr int kDenseStages = 4;
 static constexpr int kMaxSmem = 200 * 1024;
 
-template <int NT, bool NORM>
+template <int NT, int MODE>
 static cudaError_t launch_gemv(const GemvParams& p, cudaStream_t s) {
   const int bytes = kDenseStages * 2 * kThreads * 16 + NT * 8 * staged_stride(p.K);
   static int configured = 0;
   if (configured < bytes) {
-    cudaError_t e = set_smem(gemv_kernel<NT, NORM, kDenseStages>, kMaxSmem);
+    cudaError_t e = set_smem(gemv_kernel<NT, MODE, kDenseStages>, kMaxSmem);
     if (e != cudaSuccess) return e;
     configured = kMaxSmem;
   }
-  return launch_pdl(gemv_kernel<NT, NORM, kDenseStages>, dim3((p.N + 15) / 16), dim3(kThreads), bytes, s, p);
+  return launch_pdl(gemv_kernel<NT, MODE, kDenseStages>, dim3((p.N + 15) / 16), dim3(kThreads), bytes, s, p);
 }
 
 }  // namespace gv
@@ -595,9 +647,30 @@ extern "C" int mb_gemv(const void* x, const void* residual, const void* norm_w, 
   p.xn_out = reinterpret_cast<bf16*>(xn_out);
   p.M = M; p.N = N; p.K = K; p.static_w = static_w;
   cudaError_t e;
-  if (norm_w != nullptr) e = nt == 1 ? launch_gemv<1, true>(p, s) : launch_gemv<2, true>(p, s);
-  else e = nt == 1 ? launch_gemv<1, false>(p, s) : launch_gemv<2, false>(p, s);
+  if (norm_w != nullptr) e = nt == 1 ? launch_gemv<1, kAddNorm>(p, s) : launch_gemv<2, kAddNorm>(p, s);
+  else e = nt == 1 ? launch_gemv<1, kPlain>(p, s) : launch_gemv<2, kPlain>(p, s);
   return static_cast<int>(e);
+}
+
+// out[M, N] = x' · Wᵀ with x' = x + y / rms(y) · norm_w · scale_w (x, x_out fp32 and distinct); same limits as mb_gemv.
+extern "C" int mb_gemv_output_norm(const float* x, const void* y, const void* norm_w, const void* scale_w, float eps, const void* W, void* out,
+                                   long long ldo, float* x_out, int M, int N, int K, int static_w, cudaStream_t s) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M > 16 || K % 32 || K <= 0) return -1;
+  const int nt = M <= 8 ? 1 : 2;
+  if (kDenseStages * 2 * kThreads * 16 + nt * 8 * staged_stride(K) > kMaxSmem) return -2;
+  GemvParams p{};
+  p.x = reinterpret_cast<const bf16*>(y);
+  p.x32 = x;
+  p.x32_out = x_out;
+  p.norm_w = reinterpret_cast<const bf16*>(norm_w);
+  p.scale_w = reinterpret_cast<const bf16*>(scale_w);
+  p.eps = eps;
+  p.W = reinterpret_cast<const bf16*>(W);
+  p.y = out;
+  p.ldy = ldo;
+  p.M = M; p.N = N; p.K = K; p.static_w = static_w;
+  return static_cast<int>(nt == 1 ? launch_gemv<1, kOutputNorm>(p, s) : launch_gemv<2, kOutputNorm>(p, s));
 }
 
 // MoE FFN for T ≤ 8 tokens (T·k ≤ 64): act [T·k, F] scratch, out [T, H].  H and F multiples of 32, H a multiple of 16.

@@ -213,6 +213,9 @@ int mb_output_norm(float* x, const void* y, const void* nw, const void* ls, cons
 int mb_clamped_glu(const void* in, void* out, long long T, int F, float limit, float alpha, int f32, cudaStream_t s);
 int mb_gated_norm(const void* o, const void* w, const void* gate, long long gate_ld, void* out, int T, int C, float eps, int f32,
                   cudaStream_t s);
+// gemv.cu: output norm + layer scale + fp32 residual in front of a projection of ≤ 16 rows
+int mb_gemv_output_norm(const float* x, const void* y, const void* norm_w, const void* scale_w, float eps, const void* W, void* out,
+                        long long ldo, float* x_out, int M, int N, int K, int static_w, cudaStream_t s);
 // ---- latent_attn.cu ----
 typedef struct {
   int heads, dim, rot, vdim, rank, rank_p, pitch;   // a cached row: [rank, 0 … rank_p, rot, 0 … pitch)

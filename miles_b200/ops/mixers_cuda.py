@@ -5,9 +5,11 @@ without TF32 for the dense projections, as `ops.linear` does for float32).
 """
 from __future__ import annotations
 
+import os
+
 import torch
 
-from .cuda import BF16, C
+from .cuda import BF16, C, GEMV_MAX_N, gemv_ok
 
 
 def _c(x):
@@ -29,8 +31,19 @@ def output_norm_residual(x, y, nw, ls, eps, final_w=None):
     return x, xb
 
 
+# rows up to which the output norm runs inside the projection that follows it (every CTA of that projection repeats the norm)
+FUSED_NORM_M = int(os.environ.get("MILES_OUTPUT_NORM_GEMV_M", "4"))
+
+
 def few_row_projection(y, w) -> bool:
-    return False
+    return y.shape[0] <= FUSED_NORM_M and w.shape[0] <= GEMV_MAX_N and gemv_ok(y, w)
+
+
+def output_norm_linear(x, y, nw, ls, eps, w):
+    out = torch.empty(y.shape[0], w.shape[0], dtype=y.dtype, device=y.device)
+    x_new = torch.empty_like(x)
+    C.gemv_output_norm(x, _c(y), nw, ls, float(eps), w, out, x_new, bool(w.is_leaf and w.requires_grad))
+    return out, x_new
 
 
 def clamped_glu(h, limit, alpha):
