@@ -64,6 +64,11 @@ def parse():
     p.add_argument("--no-weight-sync-probe", action="store_true",
                    help="skip the untimed measurement of a weight sync into an engine that holds its own copy of the weights")
     p.add_argument("--quiet", action="store_true")
+    p.add_argument("--layered", action="store_true",
+                   help="instead of the headline workload: prefill, decode and kernel rooflines of a layer-by-layer decoder beside a "
+                        "grouped-query model of equal size (one GPU, JSON lines; --layers, default 12)")
+    p.add_argument("--layered-model", default="nopelorn-4B-shape")
+    p.add_argument("--layered-baseline", default="qwen3-4B")
     return p.parse_args()
 
 
@@ -179,6 +184,10 @@ def main():
     a = parse()
     if a.impl == "reference":
         return reference_arm(a)
+    if a.layered:
+        from miles_b200.engine.bench_layered import main as layered
+
+        return layered(a)
 
     import torch
     import torch.distributed as dist

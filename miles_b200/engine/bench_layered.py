@@ -1,0 +1,282 @@
+"""Prefill and decode of a layer-by-layer decoder beside the closest grouped-query model of equal width, depth and feed-forward.
+
+    python bench.py --layered [--layered-model nopelorn-4B-shape] [--layered-baseline qwen3-4B] [--layers N]
+
+Random weights, synthetic tokens.  `throughput`: whole models through the engine (device-timed forwards and decode graphs).
+`kernels`: the mixers' kernels one by one at the same sizes with their distance from the measured roofline, next to the kernels
+of the grouped-query model that do the like work.  L2 is flushed between timed kernel launches; model forwards move far more
+bytes than L2 holds.
+"""
+from __future__ import annotations
+
+import json
+import os
+
+import torch
+
+ROOT = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+
+
+def peaks() -> tuple[float, float, str]:
+    """(bytes/s, bf16 FLOP/s, which): the measured copy bandwidth and GEMM rate of this machine if recorded, else fallbacks."""
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            d = json.load(f)
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12, "measured"
+    except (OSError, KeyError):
+        return 6.65e12, 1.59e15, "fallback"
+
+
+class _Timer:
+    def __init__(self):
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def ms(self, fn, iters: int = 10, warmup: int = 3) -> float:
+        for _ in range(warmup):
+            fn()
+        total = 0.0
+        for _ in range(iters):
+            self.flush.zero_()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            total += e0.elapsed_time(e1)
+        return total / iters
+
+
+@torch.no_grad()
+def throughput(cfg, prefill=((1, 8192), (8, 1024)), decode=((1, 2048), (8, 2048), (64, 2048)), iters: int = 5) -> dict:
+    """Tokens/s of prefill batches (sequences × length) and decode steps (rows × context), device-timed."""
+    g = torch.Generator().manual_seed(0)
+    rows = max([n for n, _ in prefill] + [n for n, _ in decode])
+    ctx = max([l for _, l in prefill] + [l + 64 for _, l in decode])
+    ctx_tokens = max([n * l for n, l in prefill] + [n * (l + 64) for n, l in decode])
+    from .engine import Engine
+
+    eng = Engine(cfg, device="cuda:0", dtype=torch.bfloat16, num_blocks=ctx_tokens // 64 + 2 * rows, block_size=64, max_running_requests=rows,
+                 max_context_len=ctx, prefix_cache=False)
+    out: dict = {"model": cfg.name, "layers": cfg.num_layers, "params": cfg.num_params(), "prefill": [], "decode": []}
+
+    def opened(n, length):
+        reqs = []
+        for i in range(n):
+            r = eng.open_request(f"b{i}")
+            r.input_ids = torch.randint(3, cfg.vocab_size, (length,), generator=g).tolist()
+            r.blocks = eng._alloc_blocks(eng._blocks_needed(length + 32))
+            reqs.append(r)
+        return reqs
+
+    for n, length in prefill:
+        reqs = opened(n, length)
+        for r in reqs:
+            r.chunk = (0, length)
+        ev = []
+        for i in range(iters + 2):
+            # the inputs of a step go to the device before the clock starts: this is the model's own time
+            hook = _TimedForward(eng.model)
+            eng._forward_pieces(reqs)
+            hook.close()
+            ev.append(hook)
+        torch.cuda.synchronize()
+        ms = sorted(h.elapsed() for h in ev[2:])[iters // 2]
+        out["prefill"].append({"sequences": n, "length": length, "ms": ms, "tokens_per_s": n * length / ms * 1e3})
+        for r in reqs:
+            eng.close_request(r.rid)
+    for n, ctx_len in decode:
+        reqs = opened(n, ctx_len)
+        for i in range(0, n, 8):
+            for r in reqs[i:i + 8]:
+                r.chunk = (0, ctx_len)
+            eng._forward_pieces(reqs[i:i + 8])
+        run = eng.runner
+        for r in reqs:
+            run.attach(r)
+        run._set_rows(reqs)
+        run.d_i32.copy_(run.h_i32)
+        run.d_i64.copy_(run.h_i64)
+        key = (run._bucket(run.high), False)
+        run._capture(key)
+        for _ in range(3):
+            run.graphs[key].replay()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(20):
+            run.graphs[key].replay()
+        e1.record()
+        torch.cuda.synchronize()
+        ms = e0.elapsed_time(e1) / 20
+        out["decode"].append({"rows": n, "context": ctx_len, "ms": ms, "tokens_per_s": n / ms * 1e3, "launches": run.launches_per_graph[key]})
+        for r in reqs:
+            eng.close_request(r.rid)
+        run.reset_graphs()
+    return out
+
+
+class _TimedForward:
+    """CUDA events around one call of a model's forward."""
+
+    def __init__(self, model):
+        self.e0, self.e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        self.h = [model.register_forward_pre_hook(lambda *_: self.e0.record()), model.register_forward_hook(lambda *_: self.e1.record())]
+
+    def close(self):
+        for h in self.h:
+            h.remove()
+
+    def elapsed(self) -> float:
+        return self.e0.elapsed_time(self.e1)
+
+
+def _ragged(lens, bs: int = 64):
+    """A batch of (first position, new tokens) pieces on a fresh block table (device tensors), and the blocks it needs."""
+    from ..models.qwen3 import SHORT_Q, ForwardMeta, RaggedBatch
+
+    pos, slots, seq, cu, nb = [], [], [], [0], 0
+    bt = torch.zeros(len(lens), max(-(-(s + n) // bs) for s, n in lens), dtype=torch.int32)
+    for b, (s, n) in enumerate(lens):
+        k = -(-(s + n) // bs)
+        bt[b, :k] = torch.arange(nb, nb + k)
+        pos += range(s, s + n)
+        slots += [(nb + p // bs) * bs + p % bs for p in range(s, s + n)]
+        seq += [b] * n
+        cu.append(cu[-1] + n)
+        nb += k
+    n_long = sum(n > SHORT_Q for _, n in lens)
+    i32 = dict(dtype=torch.int32, device="cuda")
+    return ForwardMeta(
+        positions=torch.tensor(pos, **i32), block_table=bt.cuda(), slot_mapping=torch.tensor(slots, device="cuda"),
+        state_slots=torch.arange(len(lens), **i32),
+        ragged=RaggedBatch(cu_q=torch.tensor(cu, **i32) if n_long else None, token_seq=torch.tensor(seq, **i32) if n_long else None,
+                           q_lens=[n for _, n in lens], seq_lens=[s + n for s, n in lens], n_long=n_long, t_long=cu[n_long])), nb
+
+
+@torch.no_grad()
+def kernels(cfg, base) -> list[dict]:
+    """Device time and fraction of the roofline of each kernel: max(bytes ÷ copy bandwidth, FLOPs ÷ GEMM rate) ÷ time."""
+    from ..models.layered import LatentSpec, LinearStateSpec
+    from ..ops import cuda as K
+    from ..ops import mixers as MX
+    from ..ops import mixers_cuda as MC
+
+    bw, fl, which = peaks()
+    tm = _Timer()
+    rows: list[dict] = []
+
+    def add(name, like, shape, fn, nbytes, flops=0.0):
+        ms = tm.ms(fn)
+        ideal = max(nbytes / bw, flops / fl) * 1e3
+        rows.append({"kernel": name, "like": like, "shape": shape, "us": round(ms * 1e3, 1), "GB/s": round(nbytes / ms / 1e6),
+                     "TFLOP/s": round(flops / ms / 1e9, 1), "of_roofline": round(ideal / ms, 3), "peaks": which})
+
+    def t(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, device="cuda").to(dtype)
+
+    D = cfg.hidden_size
+    lat = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, LatentSpec))
+    lin = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, LinearStateSpec))
+    ff = next(s.mlp.ff for s in cfg.layer_specs if s.mlp is not None)
+    lay = MX.LatentLayout(lat.heads, lat.dim, lat.rot_dim, lat.vdim, lat.kv_rank)
+    sizes = [lay.heads, lay.dim, lay.rot, lay.vdim, lay.rank, lay.rank_p, lay.pitch]
+    H, sink, err = lat.heads, t(lat.heads), K.C.error_flag(torch.empty(0, device="cuda"))
+    for n, length in ((1, 8192), (8, 1024)):
+        T = n * length
+        m, nb = _ragged([(0, length)] * n)
+        cu_k, _, total, max_q = MC._key_ranges(m, lat.window)
+        qn = (lat.dim + 63) // 64 * 64
+        q, kv, lt, o = t(T, H, qn + 64), t(total, H * (lat.dim + lat.vdim)), t(total, lay.pitch), t(T, H, lat.vdim)
+        w = lat.window or length
+        pairs = n * sum(min(i + 1, w) for i in range(length))
+        add("latent_prefill (tcgen05, window, sink)", "flash_fwd_tc", f"{n}x{length} window {w}",
+            lambda: K.C.latent_prefill(q, kv, lt, o, sink, m.ragged.cu_q, cu_k, n, max_q, lat.scale, lat.window, sizes, err),
+            2 * (q.numel() + kv.numel() + total * lat.rot_dim + o.numel()), 2.0 * pairs * H * (lat.dim + lat.rot_dim + lat.vdim))
+        hq, hk, d = base.num_heads, base.num_kv_heads, base.head_dim
+        q2, k2, v2 = t(T, hq, d), t(T, hk, d), t(T, hk, d)
+        cu = m.ragged.cu_q
+        add("flash_fwd_tc", "", f"{n}x{length}", lambda: K.attention_varlen(q2, k2, v2, cu, length), 2 * (2 * q2.numel() + 2 * k2.numel()),
+            2.0 * n * length * (length + 1) / 2 * hq * 2 * d)
+        proj, dec = t(T, lin.heads * 2 * (lin.dim + lin.vdim)), torch.tensor(lin.decay, device="cuda")
+        st = torch.zeros(n, lin.heads, lin.dim, lin.vdim, device="cuda")
+        C = 64
+        add("linear_chunk (segments + scan + outputs)", "flash_fwd_tc", f"{n}x{length}",
+            lambda: MC.linear_state(proj, lin.heads, lin.dim, lin.vdim, dec, st, m), 2 * T * lin.heads * (2 * lin.dim + 2 * lin.vdim) + 8 * st.numel(),
+            2.0 * T * lin.heads * ((C + 1) / 2 * (lin.dim + lin.vdim) + 2 * lin.dim * lin.vdim))
+        del q, kv, lt, o, q2, k2, v2, proj, st
+    for B, ctx in ((1, 4096), (8, 4096), (64, 4096)):
+        m, nb = _ragged([(ctx - 1, 1)] * B)
+        cache = t(nb, 64, lay.pitch)
+        qa, ol = t(B, H, lay.pitch), t(B, H, lay.rank)
+        w = min(lat.window or ctx, ctx)
+        groups = B * -(-H // (32 if H > 16 else 16))
+        splits = MC.decode_splits(groups, w)
+        po, pm = torch.empty(B * H * splits * lay.rank_p, device="cuda"), torch.empty(B * H * splits * 2, device="cuda")
+        add("latent_decode + merge", "paged_decode", f"{B} rows, window {w}",
+            lambda: K.C.latent_decode(qa, cache, m.block_table, None, m.positions, m.slot_mapping, sink, po, pm, ol, lat.scale, lat.window, splits, sizes),
+            2 * B * (w * (lay.rank + lay.rot) + H * (lay.pitch + lay.rank)), 2.0 * B * w * H * (2 * lay.rank + lay.rot))
+        kc, vc = t(nb, 64, base.num_kv_heads, base.head_dim), t(nb, 64, base.num_kv_heads, base.head_dim)
+        q2 = t(B, base.num_heads, base.head_dim)
+        L = torch.full((B,), w, dtype=torch.int32, device="cuda")
+        add("paged_decode + merge", "", f"{B} rows, context {w}", lambda: K.paged_attention(q2, kc, vc, m.block_table, L),
+            2 * B * (w * 2 * base.num_kv_heads * base.head_dim + 2 * base.num_heads * base.head_dim), 4.0 * B * w * base.num_heads * base.head_dim)
+        wu = t(H, lat.dim, lat.kv_rank)
+        qn, wv, ov = t(B, H, lat.dim), t(H, lat.vdim, lat.kv_rank), t(B, H, lat.vdim)
+        add("head_linear (key up-projection into q)", "gemv", f"{B} rows", lambda: K.C.head_linear_mma(qn, wu, False, qa[..., :lay.rank]),
+            2 * (wu.numel() + qn.numel() + B * H * lay.rank), 2.0 * B * wu.numel())
+        add("head_linear (value up-projection)", "gemv", f"{B} rows", lambda: K.C.head_linear_mma(ol, wv, True, ov),
+            2 * (wv.numel() + ol.numel() + ov.numel()), 2.0 * B * wv.numel())
+        wo = torch.nn.Parameter(t(H * lat.vdim, lat.kv_rank))
+        xo = t(B, lat.kv_rank)
+        add("gemv / gemm of as many weight bytes", "", f"{B} rows", lambda: K.gemm_nt(xo, wo.data), 2 * (wo.numel() + xo.numel() + B * wo.shape[0]),
+            2.0 * B * wo.numel())
+        proj, dec = t(B, lin.heads * 2 * (lin.dim + lin.vdim)), torch.tensor(lin.decay, device="cuda")
+        st = torch.zeros(B, lin.heads, lin.dim, lin.vdim, device="cuda")
+        add("linear_state step", "paged_decode", f"{B} rows", lambda: MC.linear_state(proj, lin.heads, lin.dim, lin.vdim, dec, st, m),
+            8 * st.numel() + 2 * B * lin.heads * (2 * lin.dim + 2 * lin.vdim))
+        del cache, kc, vc, st
+    for T in (8, 8192):
+        x, y, v = t(T, D, dtype=torch.float32), t(T, D), t(D)
+        add("output_norm (fp32 residual)", "add_rmsnorm", f"{T} rows", lambda: MC.output_norm_residual(x, y, v, v, 1e-6), T * D * 12)
+        r2 = t(T, D)
+        add("add_rmsnorm", "", f"{T} rows", lambda: K.add_rmsnorm(y, r2, v, 1e-6), T * D * 8)
+        h = t(T, 2 * ff)
+        add("clamped_glu", "swiglu", f"{T} rows", lambda: MC.clamped_glu(h, 7.0, 1.702), 6 * T * ff)
+        add("swiglu", "", f"{T} rows", lambda: K.swiglu(h), 6 * T * ff)
+        o, gt = t(T, lin.heads * lin.vdim), t(T, lin.heads * lin.vdim)
+        gw = t(lin.heads * lin.vdim)
+        add("gated_norm", "add_rmsnorm", f"{T} rows", lambda: MC.gated_norm(o, gw, gt, 1e-6), 6 * o.numel())
+        m, nb = _ragged([(0, T)] if T > 8 else [(4000, 1)] * T)
+        cache = t(nb, 64, lay.pitch)
+        proj = t(T, lay.q_rows + lay.rank + lay.rot)
+        freq = torch.tensor(lat.rotary.table()[0], dtype=torch.float64, device="cuda")
+        kn = t(lay.rank)
+        tl = m.ragged.t_long
+        qa, qf = t(T - tl, H, lay.pitch), t(tl, H, (lat.dim + 63) // 64 * 64 + 64)
+        add("latent_prep (rotate, norm, cache)", "qk_norm_rope_cache", f"{T} rows",
+            lambda: K.C.latent_prep(proj, m.positions, m.slot_mapping, freq, 1.0, kn, 1e-6, cache, qa, qf, tl, (lat.dim + 63) // 64 * 64,
+                                    (lat.dim + 63) // 64 * 64 + 64, sizes),
+            2 * T * (lay.rank + 2 * lay.rot + lay.pitch + H * (lay.rot * 2 if T <= 8 else lay.dim * 2 + lay.rot * 2)))
+        q2, k2, v2 = t(T, base.num_heads, base.head_dim), t(T, base.num_kv_heads, base.head_dim), t(T, base.num_kv_heads, base.head_dim)
+        qw = t(base.head_dim)
+        kc, vc = t(nb, 64, base.num_kv_heads, base.head_dim), t(nb, 64, base.num_kv_heads, base.head_dim)
+        add("qk_norm_rope_cache", "", f"{T} rows", lambda: K.qk_norm_rope_cache(q2, k2, v2, qw, qw, m.positions, 1e6, 1e-6, kc, vc, m.slot_mapping),
+            2 * (2 * q2.numel() + 5 * k2.numel()))
+    return rows
+
+
+def main(a) -> int:
+    from ..models.config import get_config
+    from ..ops import cuda as K
+
+    torch.cuda.set_device(0)
+    cfg, base = get_config(a.layered_model), get_config(a.layered_baseline)
+    n = a.layers or 12
+    cfg = cfg.with_(num_layers=n, layer_specs=cfg.layer_specs[:n])
+    base = base.with_(num_layers=n)
+    for c in (cfg, base):
+        print(json.dumps(throughput(c)), flush=True)
+        torch.cuda.empty_cache()
+    for r in kernels(cfg, base):
+        print(json.dumps(r), flush=True)
+    print(json.dumps({"kernel_error_flag": K.check_error_flag()}))
+    return 0

@@ -100,6 +100,11 @@ def _prefill_ok(lay, dt, scale) -> bool:
     return _mma_ok(lay, dt) and lay.dim <= 128 and lay.rot <= 64 and lay.vdim <= 128 and scale > 0
 
 
+def decode_splits(groups: int, window: int) -> int:
+    """Key splits of latent_decode: enough (token, head group, split) CTAs for the 148 SMs (one resident per SM), whole key tiles."""
+    return max(1, min(16, 148 // groups, -(-(window or 4096) // 64)))
+
+
 def _key_ranges(meta, window: int):
     """Keys the long pieces of a batch can see: packed offsets [n + 1] and first position per sequence (device), and their number."""
     rg = meta.ragged
@@ -139,9 +144,8 @@ def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sin
         seq = rg.token_seq[t_long:] if rg.token_seq is not None else None
         pos, slots = meta.positions[t_long:], meta.slot_mapping[t_long:]
         if fast:
-            # enough (token, head group, split) CTAs for the 148 SMs, one resident per SM
             groups = n_short * -(-H // (32 if H > 16 else 16))
-            splits = max(1, min(16, 296 // groups, -(-(window or 4096) // 64)))
+            splits = decode_splits(groups, window)
             part_o = torch.empty(n_short * H * splits * lay.rank_p, dtype=torch.float32, device=dev)
             part_ml = torch.empty(n_short * H * splits * 2, dtype=torch.float32, device=dev)
             C.latent_decode(q_abs, cache, meta.block_table, seq, pos, slots, sink, part_o, part_ml, o_lat, float(scale), int(window), splits, sizes)
