@@ -9,11 +9,12 @@
 namespace mb {
 namespace mx {
 
-// One CTA per token.  Rotates the rotated part of every query head (interleaved pairs, angles in double precision, so that a
-// position of any size costs no accuracy), RMS-norms the new latent, rotates the shared key part and writes the cache row.
+// Two CTAs per token: one rotates the rotated part of every query head (interleaved pairs, angles in double precision, so that a
+// position of any size costs no accuracy); the other RMS-norms the new latent, rotates the shared key part and writes the cache row.
 // Tokens before `t_long` get a full query [H][q_width] = [unrotated | 0 … q_nope | rotated | 0 … q_width) for the expanded
 // form; later ones the rotated part and the padding of an absorbed query [H][pitch] (head_linear fills [0, rank)).
-template <typename T>
+// VEC: rows and head parts start on 16-byte boundaries and are whole 16-byte pieces.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ proj, long long ld, const int* __restrict__ positions,
                                                           const long long* __restrict__ slots, const double* __restrict__ freq,
                                                           float magnitude, const T* __restrict__ kv_norm, float eps,
@@ -21,10 +22,11 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
                                                           int q_nope, int q_width, MbLatent L) {
   extern __shared__ float cs[];          // [rot/2] cosines, [rot/2] sines
   __shared__ float sh[8];
+  constexpr int V = VEC ? 16 / static_cast<int>(sizeof(T)) : 2;      // values per piece (a piece is whole pairs)
   pdl_trigger();
   pdl_wait();
   const long long t = blockIdx.x;
-  const int half = L.rot / 2;
+  const int half = L.rot / 2, dq = L.dim + L.rot;
   const T* p = proj + t * ld;
   const double pos = positions[t];
   for (int i = threadIdx.x; i < half; i += 256) {
@@ -42,37 +44,47 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
       cs[half + i] = s * magnitude;
     }
   }
-  __syncthreads();
-  const int dq = L.dim + L.rot;
-  if (t < t_long) {
-    T* q = q_full + t * static_cast<long long>(L.heads) * q_width;
-    for (int i = threadIdx.x; i < L.heads * q_width; i += 256) {
-      const int h = i / q_width, c = i - h * q_width;
-      float v = 0.f;
-      if (c < L.dim) {
-        v = to_f(p[h * dq + c]);
-      } else if (c >= q_nope && c < q_nope + L.rot) {
-        const int r = c - q_nope, k = r >> 1;
-        const float a = to_f(p[h * dq + L.dim + 2 * k]), b = to_f(p[h * dq + L.dim + 2 * k + 1]);
-        v = (r & 1) ? b * cs[k] + a * cs[half + k] : a * cs[k] - b * cs[half + k];
-      }
-      q[i] = from_f<T>(v);
+  auto rotate = [&](float (&f)[V], int k) {      // V values, the first one the even half of pair k
+#pragma unroll
+    for (int j = 0; j < V; j += 2) {
+      const float u = f[j], v = f[j + 1], c = cs[k + j / 2], s = cs[half + k + j / 2];
+      f[j] = u * c - v * s;
+      f[j + 1] = v * c + u * s;
     }
-  } else {
-    T* q = q_abs + (t - t_long) * static_cast<long long>(L.heads) * L.pitch;
-    const int w = L.pitch - L.rank;
-    for (int i = threadIdx.x; i < L.heads * w; i += 256) {
-      const int h = i / w, c = L.rank + (i - h * w);
-      float v = 0.f;
-      if (c >= L.rank_p && c < L.rank_p + L.rot) {
-        const int r = c - L.rank_p, k = r >> 1;
-        const float a = to_f(p[h * dq + L.dim + 2 * k]), b = to_f(p[h * dq + L.dim + 2 * k + 1]);
-        v = (r & 1) ? b * cs[k] + a * cs[half + k] : a * cs[k] - b * cs[half + k];
+  };
+  if (blockIdx.y == 0) {
+    const bool full = t < t_long;
+    T* q = full ? q_full + t * static_cast<long long>(L.heads) * q_width : q_abs + (t - t_long) * static_cast<long long>(L.heads) * L.pitch;
+    const int width = full ? q_width : L.pitch, rot_at = full ? q_nope : L.rank_p, filled = full ? L.dim : L.rank;
+    if (full) {
+      const int n = L.dim / V, rest = L.dim - n * V;
+#pragma unroll 4
+      for (int i = threadIdx.x; i < L.heads * n; i += 256) {
+        const int h = i / n, c = (i - h * n) * V;
+        float f[V];
+        load_n<V>(p + h * dq + c, f);
+        store_n<V>(q + h * width + c, f);
       }
-      q[h * L.pitch + c] = from_f<T>(v);
+      if (rest)
+        for (int h = threadIdx.x; h < L.heads; h += 256) q[h * width + L.dim - 1] = p[h * dq + L.dim - 1];
     }
+    __syncthreads();
+    const int n = L.rot / V;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < L.heads * n; i += 256) {
+      const int h = i / n, c = (i - h * n) * V;
+      float f[V];
+      load_n<V>(p + h * dq + L.dim + c, f);
+      rotate(f, c / 2);
+      store_n<V>(q + h * width + rot_at + c, f);
+    }
+    const int gap = rot_at - filled, tail = width - rot_at - L.rot;
+    for (int i = threadIdx.x; i < L.heads * (gap + tail); i += 256) {
+      const int h = i / (gap + tail), c = i - h * (gap + tail);
+      q[h * width + (c < gap ? filled + c : rot_at + L.rot + c - gap)] = from_f<T>(0.f);
+    }
+    return;
   }
-  if (kv_norm == nullptr) return;
   const long long slot = slots[t];
   if (slot < 0) return;
   const T* kv = p + static_cast<long long>(L.heads) * dq;
@@ -81,7 +93,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
     const float v = to_f(kv[i]);
     ss += v * v;
   }
-  const float rstd = rsqrt_exact(__fdiv_rn(block_sum<256>(ss, sh), static_cast<float>(L.rank)) + eps);
+  const float rstd = rsqrt_exact(__fdiv_rn(block_sum<256>(ss, sh), static_cast<float>(L.rank)) + eps);      // (also orders cs)
   T* row = cache + slot * L.pitch;
   for (int i = threadIdx.x; i < L.pitch; i += 256) {
     float v = 0.f;
@@ -189,9 +201,13 @@ template <typename T>
 static int prep(const T* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
                 const T* kv_norm, float eps, T* cache, T* q_abs, T* q_full, int n, int t_long, int q_nope, int q_width, MbLatent L,
                 cudaStream_t s) {
-  if (L.rot > 4096) return -3;
-  return static_cast<int>(launch_pdl(latent_prep_kernel<T>, dim3(n), dim3(256), L.rot * sizeof(float), s, proj, ld, positions, slots, freq,
-                                     magnitude, kv_norm, eps, cache, q_abs, q_full, t_long, q_nope, q_width, L));
+  if (L.rot > 4096 || L.rot % 2) return -3;
+  const int v = 16 / static_cast<int>(sizeof(T));
+  const bool vec = ld % v == 0 && L.dim % v == 0 && L.rot % v == 0 && q_nope % v == 0 && q_width % v == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0;
+  const dim3 grid(n, kv_norm != nullptr ? 2 : 1);
+  auto kern = vec ? latent_prep_kernel<T, true> : latent_prep_kernel<T, false>;
+  return static_cast<int>(launch_pdl(kern, grid, dim3(256), L.rot * sizeof(float), s, proj, ld, positions, slots, freq, magnitude, kv_norm, eps,
+                                     cache, q_abs, q_full, t_long, q_nope, q_width, L));
 }
 
 template <typename T>

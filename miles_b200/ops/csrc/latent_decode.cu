@@ -148,20 +148,20 @@ __global__ void __launch_bounds__(128) head_linear_mma_kernel(const bf16* __rest
       }
 }
 
-// grid (splits, head groups of 16·MT, tokens), 256 threads.  Warp = (head tile, column group): scores of its head tile for its share
+// grid (splits, head groups of 16·MT, tokens), 512 threads.  Warp = (head tile, column group): scores of its head tile for its share
 // of the 64 keys of a tile, then its share of the latent columns of P·C.
 template <int MT>
 struct Dec {
-  static constexpr int TK = 64, NG = 8 / MT, HT = 16 * MT;
-  static constexpr int NT16 = 32 / NG;                                  // latent columns per warp in 16s (rank ≤ 512)
+  static constexpr int TK = 64, NG = 16 / MT, HT = 16 * MT, KH = NG / 4;      // 4 groups of 16 keys × KH row parts
+  static constexpr int NT16 = (32 + NG - 1) / NG;                       // latent columns per warp in 16s (rank ≤ 512)
   static constexpr int SP = TK + 4, PP = TK + 8;
   static size_t bytes(int pitch) {
-    return static_cast<size_t>(HT + 2 * TK) * (pitch + 8) * 2 + HT * SP * 4 + 2 * HT * PP * 2 + HT * 4;
+    return static_cast<size_t>(HT + 2 * TK) * (pitch + 8) * 2 + KH * HT * SP * 4 + 2 * HT * PP * 2 + HT * 4;
   }
 };
 
 template <int MT>
-__global__ void __launch_bounds__(256) latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
+__global__ void __launch_bounds__(512) latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
                                                             const int* __restrict__ block_table, int max_blocks, int block_size,
                                                             const int* __restrict__ token_seq, const int* __restrict__ positions,
                                                             const long long* __restrict__ slots, float* __restrict__ part_o,
@@ -174,7 +174,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const bf16* __restri
   bf16* sq = reinterpret_cast<bf16*>(smem);                             // [HT][rp]
   bf16* sk = sq + HT * rp;                                              // [2][TK][rp]
   float* ss = reinterpret_cast<float*>(sk + 2 * TK * rp);               // [HT][SP] scores
-  bf16* sph = reinterpret_cast<bf16*>(ss + HT * G::SP);                 // [HT][PP] P_hi, then P_lo
+  bf16* sph = reinterpret_cast<bf16*>(ss + G::KH * HT * G::SP);                 // [HT][PP] P_hi, then P_lo
   bf16* spl = sph + HT * G::PP;
   float* sa = reinterpret_cast<float*>(spl + HT * G::PP);               // [HT] rescale factors of the current tile
   pdl_trigger();
@@ -192,22 +192,28 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const bf16* __restri
   const int n_tiles = k_end > k_begin ? (k_end - k_begin + TK - 1) / TK : 0;
   const int* bt = block_table + static_cast<long long>(token_seq != nullptr ? token_seq[t] : t) * max_blocks;
   const int pieces = L.pitch / 8;
+  // lane j < 4 of a warp looks up the page of its j-th row of a tile, one tile before the tile is copied
+  auto lookup = [&](int i) -> long long {
+    if (lane >= TK / 16) return -1;
+    const int key = k_begin + i * TK + warp + lane * 16;
+    if (key >= k_end) return -1;
+    const long long blk = bt[key / block_size];
+    return blk >= 0 && blk < num_blocks ? blk * block_size + key % block_size : -1;      // an entry outside the pool reads as zeros
+  };
+  long long next = n_tiles > 0 ? lookup(0) : -1;
   auto load_tile = [&](int i, int st) {
-    const int k0 = k_begin + i * TK;
-    for (int r = warp; r < TK; r += 8) {
-      const int key = k0 + r;
-      bool ok = key < k_end;
-      const int kk = ok ? key : k_begin;
-      long long blk = bt[kk / block_size];
-      if (blk < 0 || blk >= num_blocks) { ok = false; blk = 0; }        // a table entry outside the pool reads as zeros
-      const bf16* src = cache + (blk * block_size + kk % block_size) * L.pitch;
-      bf16* dst = sk + (st * TK + r) * rp;
-      for (int c = lane; c < pieces; c += 32) cp16(dst + c * 8, src + c * 8, ok);
+#pragma unroll
+    for (int j = 0; j < TK / 16; ++j) {
+      const long long slot = __shfl_sync(0xffffffffu, next, j);
+      const bf16* src = cache + (slot >= 0 ? slot : 0) * L.pitch;
+      bf16* dst = sk + (st * TK + warp + j * 16) * rp;
+      for (int c = lane; c < pieces; c += 32) cp16(dst + c * 8, src + c * 8, slot >= 0);
     }
     cp_commit();
+    if (i + 1 < n_tiles) next = lookup(i + 1);
   };
   if (n_tiles > 0) {
-    for (int i = threadIdx.x; i < HT * pieces; i += 256) {
+    for (int i = threadIdx.x; i < HT * pieces; i += 512) {
       const int r = i / pieces, c = i - r * pieces;
       const bool ok = h0 + r < L.heads;
       cp16(sq + r * rp + c * 8, ok ? q + (t * L.heads + h0 + r) * L.pitch + c * 8 : q, ok);
@@ -220,8 +226,8 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const bf16* __restri
   for (int i = 0; i < G::NT16; ++i)
 #pragma unroll
     for (int j = 0; j < 2; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
-  // softmax state of row `srow`, held by its 4 (MT 2: 8) consecutive threads
-  constexpr int TPR = 256 / HT, KPT = TK / TPR;
+  // softmax state of row `srow`, held by its 32 (MT 2: 16) consecutive threads
+  constexpr int TPR = 512 / HT, KPT = TK / TPR;
   const int srow = threadIdx.x / TPR, sub = threadIdx.x % TPR;
   float m_run = -INFINITY, l_run = 0.f;
   const float sl2 = scale * kLog2e;
@@ -236,31 +242,25 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const bf16* __restri
     __syncthreads();
     const bf16* tk = sk + st * TK * rp;
     // scores: head tile mt × keys [ng·TK/NG, …)
-    constexpr int NK8 = TK / NG / 8;                                    // 8-key tiles of this warp: 1 (MT 1) or 2 (MT 2)
-    float s[NK8][4];
-#pragma unroll
-    for (int n = 0; n < NK8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
-    for (int ks = 0; ks < L.pitch / 16; ++ks) {
-      uint32_t a[4];
+    // scores: 16 keys and a part (1/KH) of the row per warp — query fragments are the larger half of the shared-memory reads, and wide
+    // key groups re-read them less often; the parts are added up in the softmax
+    constexpr int KH = G::KH;
+    const int kg = ng / KH, kh = ng % KH;
+    float s[2][4] = {};
+    const int steps = L.pitch / 16, per_h = (steps + KH - 1) / KH;
+#pragma unroll 6
+    for (int ks = kh * per_h; ks < min(steps, (kh + 1) * per_h); ++ks) {
+      uint32_t a[4], b[4];
       ldsm4(s_addr(sq + (mt * 16 + (lane & 15)) * rp + ks * 16 + (lane >> 4) * 8), a);
-      if constexpr (NK8 == 2) {
-        uint32_t b[4];
-        ldsm4(s_addr(tk + (ng * 16 + (lane & 7) + ((lane >> 4) << 3)) * rp + ks * 16 + ((lane >> 3) & 1) * 8), b);
-        mma(s[0], a, b[0], b[1]);
-        mma(s[1], a, b[2], b[3]);
-      } else {
-        uint32_t b0, b1;
-        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
-                     : "=r"(b0), "=r"(b1)
-                     : "r"(s_addr(tk + (ng * 8 + (lane & 7)) * rp + ks * 16 + ((lane >> 3) & 1) * 8)));
-        mma(s[0], a, b0, b1);
-      }
+      ldsm4(s_addr(tk + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * rp + ks * 16 + ((lane >> 3) & 1) * 8), b);
+      mma(s[0], a, b[0], b[1]);
+      mma(s[1], a, b[2], b[3]);
     }
 #pragma unroll
-    for (int n = 0; n < NK8; ++n) {
-      const int c = ng * (TK / NG) + n * 8 + (lane & 3) * 2, r = mt * 16 + (lane >> 2);
-      *reinterpret_cast<float2*>(ss + r * G::SP + c) = make_float2(s[n][0], s[n][1]);
-      *reinterpret_cast<float2*>(ss + (r + 8) * G::SP + c) = make_float2(s[n][2], s[n][3]);
+    for (int n = 0; n < 2; ++n) {
+      float* dst = ss + kh * HT * G::SP + (mt * 16 + (lane >> 2)) * G::SP + kg * 16 + n * 8 + (lane & 3) * 2;
+      *reinterpret_cast<float2*>(dst) = make_float2(s[n][0], s[n][1]);
+      *reinterpret_cast<float2*>(dst + 8 * G::SP) = make_float2(s[n][2], s[n][3]);
     }
     __syncthreads();
     {
@@ -269,7 +269,10 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const bf16* __restri
 #pragma unroll
       for (int j = 0; j < KPT; ++j) {
         const int c = j * TPR + sub;
-        v[j] = key0 + c < k_end ? ss[srow * G::SP + c] * sl2 : -INFINITY;
+        float x = ss[srow * G::SP + c];
+#pragma unroll
+        for (int k = 1; k < KH; ++k) x += ss[(k * HT + srow) * G::SP + c];
+        v[j] = key0 + c < k_end ? x * sl2 : -INFINITY;
         mx = fmaxf(mx, v[j]);
       }
 #pragma unroll
@@ -350,19 +353,27 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
   pdl_trigger();
   pdl_wait();
   const long long th = static_cast<long long>(blockIdx.y) * L.heads + blockIdx.x;
-  const float* ml = part_ml + th * num_splits * 2;
+  const int lane = threadIdx.x & 31;
+  // lane = split: maximum, weight and denominator by warp reductions (every warp the same)
+  const float2 ml = lane < num_splits ? *reinterpret_cast<const float2*>(part_ml + (th * num_splits + lane) * 2) : make_float2(-INFINITY, 0.f);
   const float sk = sink != nullptr ? __bfloat162float(sink[blockIdx.x]) * kLog2e : -INFINITY;
-  float mm = sk;
-  for (int s = 0; s < num_splits; ++s) mm = fmaxf(mm, ml[2 * s]);
-  float den = sink != nullptr ? exp2f(sk - mm) : 0.f;
-  for (int s = 0; s < num_splits; ++s)
-    if (ml[2 * s] != -INFINITY) den += ml[2 * s + 1] * exp2f(ml[2 * s] - mm);
-  const float inv = den > 0.f ? __fdiv_rn(1.f, den) : 0.f;
-  for (int c = threadIdx.x; c < L.rank; c += 128) {
+  float mm = fmaxf(ml.x, sk);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, o));
+  const float w = ml.x == -INFINITY ? 0.f : exp2f(ml.x - mm);
+  const float den = mx::warp_sum(ml.y * w) + (sink != nullptr ? exp2f(sk - mm) : 0.f);
+  const float f = den > 0.f ? __fdiv_rn(w, den) : 0.f;
+  const float* po = part_o + th * num_splits * L.rank_p;
+  for (int c0 = 0; c0 < L.rank; c0 += 128) {
+    const int c = c0 + threadIdx.x;
     float r = 0.f;
-    for (int s = 0; s < num_splits; ++s)
-      if (ml[2 * s] != -INFINITY) r += part_o[(th * num_splits + s) * L.rank_p + c] * exp2f(ml[2 * s] - mm);
-    out[th * L.rank + c] = __float2bfloat16(r * inv);
+#pragma unroll 8
+    for (int s = 0; s < num_splits; ++s) {
+      const float fs = __shfl_sync(0xffffffffu, f, s);
+      const float v = c < L.rank ? po[s * L.rank_p + c] : 0.f;
+      r = fs > 0.f ? fmaf(fs, v, r) : r;            // an empty split wrote nothing
+    }
+    if (c < L.rank) out[th * L.rank + c] = __float2bfloat16(r);
   }
 }
 
@@ -375,7 +386,7 @@ static cudaError_t decode(dim3 grid, cudaStream_t s, const bf16* q, const bf16* 
     if (e != cudaSuccess) return e;
     once = true;
   }
-  return launch_pdl(latent_decode_kernel<MT>, grid, dim3(256), Dec<MT>::bytes(L.pitch), s, q, cache, bt, mbk, bs, seq, pos, slots, po, pml, scale,
+  return launch_pdl(latent_decode_kernel<MT>, grid, dim3(512), Dec<MT>::bytes(L.pitch), s, q, cache, bt, mbk, bs, seq, pos, slots, po, pml, scale,
                     window, splits, nb, L);
 }
 
@@ -416,7 +427,7 @@ extern "C" int mb_latent_decode(const void* q, const void* cache, const int* blo
                                 const int* positions, const long long* slots, const void* sink, float* part_o, float* part_ml, void* out,
                                 int T, float scale, int window, int splits, int num_blocks, MbLatent L, cudaStream_t s) {
   if (T <= 0) return 0;
-  if (L.rank_p > 512 || T > 65535 || splits < 1) return -3;
+  if (L.rank_p > 512 || T > 65535 || splits < 1 || splits > 32) return -3;
   const int mt = L.heads > 16 && Dec<2>::bytes(L.pitch) <= 227 * 1024 ? 2 : 1;
   if (Dec<1>::bytes(L.pitch) > 227 * 1024) return -3;
   const dim3 grid(splits, (L.heads + 16 * mt - 1) / (16 * mt), T);

@@ -55,6 +55,15 @@ __device__ __forceinline__ float ipow(float lam, int m) {
   return r;
 }
 
+// silu of two values with one reciprocal: 1/a = b · 1/(ab).  Arguments below −40 count as −40 in the exponential (the result is
+// zero to 15 digits either way), which keeps the product finite.
+__device__ __forceinline__ void silu2(float& x, float& y) {
+  const float a = 1.f + __expf(fminf(-x, 40.f)), b = 1.f + __expf(fminf(-y, 40.f));
+  const float r = __fdividef(1.f, a * b);
+  x *= r * b;
+  y *= r * a;
+}
+
 struct Args {
   const bf16* proj;          // [T, ld]: q [H, dk], k [H, dk], v [H, dv] side by side
   long long ld;
@@ -68,8 +77,8 @@ struct Args {
   int H, dk, dv;
 };
 
-// grid (heads, segments), 512 threads
-template <bool OUT>
+// grid (heads, segments), 512 threads.  KD, VD: dk and dv when known at compile time, 0 otherwise.
+template <bool OUT, int KD, int VD>
 __global__ void __launch_bounds__(kThreads) linear_chunk_kernel(Args a) {
   extern __shared__ __align__(128) uint8_t smem[];
   bf16* tile = reinterpret_cast<bf16*>(smem);        // [2][q | k | v][C][P]
@@ -87,7 +96,7 @@ __global__ void __launch_bounds__(kThreads) linear_chunk_kernel(Args a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
   const float lam = a.decay[h];
   if (threadIdx.x <= C) pw[threadIdx.x] = ipow(lam, threadIdx.x);
-  const int dk = a.dk, dv = a.dv, kdk = (dk + 15) / 16, kdv = (dv + 15) / 16;
+  const int dk = KD ? KD : a.dk, dv = VD ? VD : a.dv, kdk = (dk + 15) / 16, kdv = (dv + 15) / 16;
   const long long HK = static_cast<long long>(a.H) * dk;
   const bf16* src[3] = {a.proj + h * dk, a.proj + HK + h * dk, a.proj + 2 * HK + h * dv};
   // columns [width, 16·⌈width/16⌉) of the tiles are zero for good
@@ -138,38 +147,40 @@ __global__ void __launch_bounds__(kThreads) linear_chunk_kernel(Args a) {
     }
   const int mt = warp >> 2, cq = warp & 3;           // scores and outputs: warp = (16 tokens, quarter of the keys / of dv)
   const int chunks = (t1 - t0 + C - 1) / C;
+  auto activate = [&](int st) {
+    each([&](int which, int r, int col) {
+      bf16* p = tile + (st * 3 + which) * kTile + r * P + col;
+      float f[8];
+      mx::load_n<8>(p, f);
+#pragma unroll
+      for (int j = 0; j < 8; j += 2) silu2(f[j], f[j + 1]);
+      mx::store_n<8>(p, f);
+    });
+  };
+  auto publish_state = [&]() {
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int r = rt * 16 + half * 8 + g, c = ch * 64 + n * 8 + t4 * 2;
+        uint32_t hi, lo;
+        split2(s[n][half * 2], s[n][half * 2 + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(s_hi + r * P + c) = hi;
+        *reinterpret_cast<uint32_t*>(s_lo + r * P + c) = lo;
+      }
+  };
+  // Two barriers per chunk: [scores and Sᵀq] | [P·v, state update, state published, next chunk activated].  The activation of one
+  // warp overlaps the products of another; the copy of chunk i + 2 runs from the first barrier to the end of the second phase.
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  activate(0);
+  if (OUT) publish_state();
   for (int ci = 0; ci < chunks; ++ci) {
     const int st = ci & 1, n_tok = min(C, t1 - t0 - ci * C);
     bf16* tq = tile + st * 3 * kTile;
     bf16* tk = tq + kTile;
     bf16* tv = tk + kTile;
-    if (ci + 1 < chunks) {
-      load(ci + 1, st ^ 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    each([&](int which, int r, int col) {
-      bf16* p = tq + which * kTile + r * P + col;
-      float f[8];
-      mx::load_n<8>(p, f);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) f[j] = mx::silu_t<bf16>(f[j]);
-      mx::store_n<8>(p, f);
-    });
-    if (OUT) {
-#pragma unroll
-      for (int n = 0; n < 8; ++n)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int r = rt * 16 + half * 8 + g, c = ch * 64 + n * 8 + t4 * 2;
-          uint32_t hi, lo;
-          split2(s[n][half * 2], s[n][half * 2 + 1], hi, lo);
-          *reinterpret_cast<uint32_t*>(s_hi + r * P + c) = hi;
-          *reinterpret_cast<uint32_t*>(s_lo + r * P + c) = lo;
-        }
-    }
     __syncthreads();
+    if (ci + 1 < chunks) load(ci + 1, st ^ 1);
     float o[4][4];
 #pragma unroll
     for (int n = 0; n < 4; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -268,7 +279,11 @@ __global__ void __launch_bounds__(kThreads) linear_chunk_kernel(Args a) {
         }
       }
     }
-    __syncthreads();
+    if (ci + 1 < chunks) {
+      if (OUT) publish_state();
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+      activate(st ^ 1);
+    }
   }
   float* dst = OUT ? (last ? slot_p : nullptr) : seg_p;
   if (dst == nullptr || (OUT && slot < 0)) return;
@@ -330,21 +345,24 @@ extern "C" int mb_linear_chunk(const void* proj, long long ld, const float* deca
                                cudaStream_t s) {
   if (n_seg <= 0) return 0;
   if (dk % 8 || dv % 8 || dk > 128 || dv > 128 || ld % 8 || n_seg > 65535) return -3;
-  static bool once = false;
-  if (!once) {
-    cudaError_t e = cudaFuncSetAttribute(linear_chunk_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kSmem));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_chunk_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kSmem));
+  const bool big = dk == 128 && dv == 128;
+  auto outputs = big ? linear_chunk_kernel<true, 128, 128> : linear_chunk_kernel<true, 0, 0>;
+  auto sums = big ? linear_chunk_kernel<false, 128, 128> : linear_chunk_kernel<false, 0, 0>;
+  static bool once[2] = {false, false};
+  if (!once[big]) {
+    cudaError_t e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kSmem));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(sums, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kSmem));
     if (e != cudaSuccess) return static_cast<int>(e);
-    once = true;
+    once[big] = true;
   }
   Args a{reinterpret_cast<const bf16*>(proj), ld, decay, state, slots, positions, segs, seg_state, reinterpret_cast<bf16*>(out), H, dk, dv};
   cudaError_t e = cudaSuccess;
   if (seg_state != nullptr) {
-    e = launch_pdl(linear_chunk_kernel<false>, dim3(H, n_seg), dim3(kThreads), kSmem, s, a);
+    e = launch_pdl(sums, dim3(H, n_seg), dim3(kThreads), kSmem, s, a);
     if (e == cudaSuccess)
       e = launch_pdl(linear_scan_kernel, dim3((dk * dv + 1023) / 1024, H, n_seq), dim3(256), 0, s, static_cast<const float*>(state), slots,
                      positions, decay, segs, seq_segs, seg_state, H, dk * dv);
   }
-  if (e == cudaSuccess) e = launch_pdl(linear_chunk_kernel<true>, dim3(H, n_seg), dim3(kThreads), kSmem, s, a);
+  if (e == cudaSuccess) e = launch_pdl(outputs, dim3(H, n_seg), dim3(kThreads), kSmem, s, a);
   return static_cast<int>(e);
 }

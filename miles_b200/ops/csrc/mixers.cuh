@@ -39,14 +39,15 @@ __device__ __forceinline__ float rsqrt_exact(float x) { return __fdiv_rn(1.f, __
 
 // N consecutive values ↔ floats (N·sizeof(T) bytes, 16-byte aligned pieces)
 template <int N> __device__ __forceinline__ void load_n(const float* p, float (&f)[N]) {
+  if constexpr (N % 4 == 0) {
 #pragma unroll
-  for (int i = 0; i < N; i += 4) {
-    if constexpr (N >= 4) {
+    for (int i = 0; i < N; i += 4) {
       const float4 v = *reinterpret_cast<const float4*>(p + i);
       f[i] = v.x; f[i + 1] = v.y; f[i + 2] = v.z; f[i + 3] = v.w;
-    } else {
-      f[i] = p[i];
     }
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) f[i] = p[i];
   }
 }
 template <int N> __device__ __forceinline__ void load_n(const bf16* p, float (&f)[N]) {
@@ -64,10 +65,12 @@ template <int N> __device__ __forceinline__ void load_n(const bf16* p, float (&f
   }
 }
 template <int N> __device__ __forceinline__ void store_n(float* p, const float (&f)[N]) {
+  if constexpr (N % 4 == 0) {
 #pragma unroll
-  for (int i = 0; i < N; i += 4) {
-    if constexpr (N >= 4) *reinterpret_cast<float4*>(p + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
-    else p[i] = f[i];
+    for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) p[i] = f[i];
   }
 }
 template <int N> __device__ __forceinline__ void store_n(bf16* p, const float (&f)[N]) {

@@ -74,14 +74,18 @@ def linear_state(proj, H, dk, dv, decay, state, meta):
 
 
 def _segments(meta, H: int):
-    """Cut the long pieces of a batch into segments of whole 64-token chunks, about four (segment, head) CTAs per SM.  Returns
-    ([n, 4] (sequence, first token, end, last of its sequence), offsets per sequence, any sequence cut)."""
+    """Cut the long pieces of a batch into segments of whole 64-token chunks so that the (segment, head) CTAs, one per SM at a time,
+    finish in the fewest chunk times (a CTA's start counts as one and a half).  Returns ([n, 4] (sequence, first token, end, last of its sequence), offsets per sequence, any sequence cut)."""
     rg = meta.ragged
-    size = min(2048, max(128, -(-rg.t_long * H // (4 * 148 * 64)) * 64))
-    key = ("segments", size)
+    key = ("segments", H)
     if key not in rg.scratch:
+        lens = rg.q_lens[: rg.n_long]
+        whole = -(-max(lens) // 64)                     # chunks of the longest piece; any cut costs a pass over keys and values more
+        best = min((-(-sum(-(-n // (64 * c)) for n in lens) * H // 148) * (min(c, whole) + 1.5) * (1.0 if c >= whole else 1.7), c)
+                   for c in {*range(2, 33), whole})
+        size = 64 * best[1]
         segs, cu, t = [], [0], 0
-        for b, n in enumerate(rg.q_lens[: rg.n_long]):
+        for b, n in enumerate(lens):
             for a in range(0, n, size):
                 segs += [b, t + a, t + min(n, a + size), int(a + size >= n)]
             t += n
