@@ -988,7 +988,7 @@ class Engine:
         for r in finished_batch:
             r.num_cached = r.num_tokens
             r.prefill_pos = r.num_tokens
-        if followers or len(done) != len(finished_batch):
+        if self.ragged or followers or len(done) != len(finished_batch):      # (ragged batches are packed in another order)
             rows = torch.tensor([lead_row[id(r.leader if r.leader is not None else r)] for r in finished_batch], dtype=torch.int64, device=dev)
             logits = logits[rows]
         for r in batch:
