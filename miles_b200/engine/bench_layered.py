@@ -208,11 +208,10 @@ def kernels(cfg, base) -> list[dict]:
         cache = t(nb, 64, lay.pitch)
         qa, ol = t(B, H, lay.pitch), t(B, H, lay.rank)
         w = min(lat.window or ctx, ctx)
-        groups = B * -(-H // (32 if H > 16 else 16))
-        splits = MC.decode_splits(groups, w)
+        splits = MC.decode_splits(B, H, w, 64)
         po, pm = torch.empty(B * H * splits * lay.rank_p, device="cuda"), torch.empty(B * H * splits * 2, device="cuda")
         add("latent_decode + merge", "paged_decode", f"{B} rows, window {w}",
-            lambda: K.C.latent_decode(qa, cache, m.block_table, None, m.positions, m.slot_mapping, sink, po, pm, ol, lat.scale, lat.window, splits, sizes),
+            lambda: K.C.latent_decode(qa, cache, m.block_table, None, m.positions, m.slot_mapping, sink, po, pm, ol, lat.scale, lat.window, splits, sizes, err),
             2 * B * (w * (lay.rank + lay.rot) + H * (lay.pitch + lay.rank)), 2.0 * B * w * H * (2 * lay.rank + lay.rot))
         kc, vc = t(nb, 64, base.num_kv_heads, base.head_dim), t(nb, 64, base.num_kv_heads, base.head_dim)
         q2 = t(B, base.num_heads, base.head_dim)

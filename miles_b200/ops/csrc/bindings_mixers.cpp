@@ -113,12 +113,12 @@ void head_linear_mma(const at::Tensor& x, const at::Tensor& w, bool w_nk, at::Te
 
 void latent_decode(const at::Tensor& q, const at::Tensor& cache, const at::Tensor& block_table, const OptTensor& token_seq,
                    const at::Tensor& positions, const at::Tensor& slots, const OptTensor& sink, at::Tensor& part_o, at::Tensor& part_ml,
-                   at::Tensor& out, double scale, int64_t window, int64_t splits, const std::vector<int64_t>& lay) {
+                   at::Tensor& out, double scale, int64_t window, int64_t splits, const std::vector<int64_t>& lay, at::Tensor& err) {
   c10::cuda::CUDAGuard g(q.device());
   mb_count_launch(1);
   check(mb_latent_decode(q.data_ptr(), cache.data_ptr(), block_table.data_ptr<int>(), block_table.size(1), cache.size(1), iptr(token_seq),
                          positions.data_ptr<int>(), lptr(slots), cptr(sink), part_o.data_ptr<float>(), part_ml.data_ptr<float>(), out.data_ptr(),
-                         q.size(0), scale, window, splits, cache.size(0), layout(lay), cur_stream()),
+                         q.size(0), scale, window, splits, cache.size(0), layout(lay), err.data_ptr<int>(), cur_stream()),
         "mb_latent_decode");
 }
 

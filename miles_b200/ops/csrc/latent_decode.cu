@@ -422,20 +422,28 @@ extern "C" int mb_head_linear_mma(const void* x, long long x_t, long long x_h, c
   return static_cast<int>(e);
 }
 
-// part_o [T, H, splits, rank_p] and part_ml [T, H, splits, 2] fp32 scratch; bf16, rank ≤ 512, pitch ≤ 640
+// part_o [T, H, splits, rank_p] and part_ml [T, H, splits, 2] fp32 scratch; bf16, rank ≤ 512, pitch ≤ 640.  Pages of a multiple of 64
+// tokens go through the tcgen05 kernel (latent_decode_tc.cu), others through the mma.sync kernel above.
 extern "C" int mb_latent_decode(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                                 const int* positions, const long long* slots, const void* sink, float* part_o, float* part_ml, void* out,
-                                int T, float scale, int window, int splits, int num_blocks, MbLatent L, cudaStream_t s) {
+                                int T, float scale, int window, int splits, int num_blocks, MbLatent L, int* error_flag, cudaStream_t s) {
   if (T <= 0) return 0;
-  if (L.rank_p > 512 || T > 65535 || splits < 1 || splits > 32) return -3;
-  const int mt = L.heads > 16 && Dec<2>::bytes(L.pitch) <= 227 * 1024 ? 2 : 1;
-  if (Dec<1>::bytes(L.pitch) > 227 * 1024) return -3;
-  const dim3 grid(splits, (L.heads + 16 * mt - 1) / (16 * mt), T);
-  auto Q = reinterpret_cast<const bf16*>(q);
-  auto KC = reinterpret_cast<const bf16*>(cache);
-  cudaError_t e = mt == 2 ? decode<2>(grid, s, Q, KC, block_table, max_blocks, block_size, token_seq, positions, slots, part_o, part_ml, scale, window, splits, num_blocks, L)
-                          : decode<1>(grid, s, Q, KC, block_table, max_blocks, block_size, token_seq, positions, slots, part_o, part_ml, scale, window, splits, num_blocks, L);
-  if (e != cudaSuccess) return static_cast<int>(e);
+  if (L.rank_p > 512 || L.pitch > 640 || T > 65535 || splits < 1 || splits > 32) return -3;
+  if (block_size % 64 == 0) {
+    const int rc = mb_latent_decode_tc(q, cache, block_table, max_blocks, block_size, token_seq, positions, slots, part_o, part_ml, T, scale,
+                                       window, splits, num_blocks, L, error_flag, s);
+    if (rc) return rc;
+  } else {
+    const int mt = L.heads > 16 && Dec<2>::bytes(L.pitch) <= 227 * 1024 ? 2 : 1;
+    if (Dec<1>::bytes(L.pitch) > 227 * 1024) return -3;
+    const dim3 grid(splits, (L.heads + 16 * mt - 1) / (16 * mt), T);
+    auto Q = reinterpret_cast<const bf16*>(q);
+    auto KC = reinterpret_cast<const bf16*>(cache);
+    const cudaError_t e =
+        mt == 2 ? decode<2>(grid, s, Q, KC, block_table, max_blocks, block_size, token_seq, positions, slots, part_o, part_ml, scale, window, splits, num_blocks, L)
+                : decode<1>(grid, s, Q, KC, block_table, max_blocks, block_size, token_seq, positions, slots, part_o, part_ml, scale, window, splits, num_blocks, L);
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
   return static_cast<int>(launch_pdl(latent_merge_kernel, dim3(L.heads, T), dim3(128), 0, s, static_cast<const float*>(part_o),
                                      static_cast<const float*>(part_ml), reinterpret_cast<const bf16*>(sink), reinterpret_cast<bf16*>(out), splits, L));
 }

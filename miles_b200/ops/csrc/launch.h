@@ -235,7 +235,11 @@ int mb_head_linear_mma(const void* x, long long x_t, long long x_h, const void* 
                        int H, int N, int K, cudaStream_t s);
 int mb_latent_decode(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                      const int* positions, const long long* slots, const void* sink, float* part_o, float* part_ml, void* out, int T,
-                     float scale, int window, int splits, int num_blocks, MbLatent L, cudaStream_t s);
+                     float scale, int window, int splits, int num_blocks, MbLatent L, int* error_flag, cudaStream_t s);
+// ---- latent_decode_tc.cu (tcgen05; the split part of mb_latent_decode for pages of a multiple of 64 tokens) ----
+int mb_latent_decode_tc(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size, const int* token_seq,
+                        const int* positions, const long long* slots, float* part_o, float* part_ml, int T, float scale, int window,
+                        int splits, int num_blocks, MbLatent L, int* error_flag, cudaStream_t s);
 // ---- attention_latent_tc.cu (tcgen05) ----
 int mb_latent_prefill(const void* q, const void* kv, const void* lat, void* o, const void* sink, const int* cu_q, const int* cu_k, int n_seq,
                       int max_q, int t_long, int tk, float scale, int window, MbLatent L, int* error_flag, cudaStream_t s);

@@ -104,9 +104,10 @@ def _prefill_ok(lay, dt, scale) -> bool:
     return _mma_ok(lay, dt) and lay.dim <= 128 and lay.rot <= 64 and lay.vdim <= 128 and scale > 0
 
 
-def decode_splits(groups: int, window: int) -> int:
+def decode_splits(tokens: int, heads: int, window: int, block_size: int) -> int:
     """Key splits of latent_decode: enough (token, head group, split) CTAs for the 148 SMs (one resident per SM), whole key tiles."""
-    return max(1, min(16, 148 // groups, -(-(window or 4096) // 64)))
+    tile, group = (128, 32) if block_size % 64 == 0 else (64, 32 if heads > 16 else 16)
+    return max(1, min(32, 148 // (tokens * -(-heads // group)), -(-(window or 4096) // tile)))
 
 
 def _key_ranges(meta, window: int):
@@ -148,11 +149,11 @@ def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sin
         seq = rg.token_seq[t_long:] if rg.token_seq is not None else None
         pos, slots = meta.positions[t_long:], meta.slot_mapping[t_long:]
         if fast:
-            groups = n_short * -(-H // (32 if H > 16 else 16))
-            splits = decode_splits(groups, window)
+            splits = decode_splits(n_short, H, window, cache.shape[1])
             part_o = torch.empty(n_short * H * splits * lay.rank_p, dtype=torch.float32, device=dev)
             part_ml = torch.empty(n_short * H * splits * 2, dtype=torch.float32, device=dev)
-            C.latent_decode(q_abs, cache, meta.block_table, seq, pos, slots, sink, part_o, part_ml, o_lat, float(scale), int(window), splits, sizes)
+            C.latent_decode(q_abs, cache, meta.block_table, seq, pos, slots, sink, part_o, part_ml, o_lat, float(scale), int(window), splits, sizes,
+                            C.error_flag(proj))
         else:
             C.latent_attend(q_abs, cache, meta.block_table, seq, pos, slots, sink, o_lat, float(scale), int(window), sizes)
         _head_linear(o_lat, w_uv, True, out[t_long:], fast)
