@@ -270,8 +270,7 @@ def main(a) -> int:
     torch.cuda.set_device(0)
     cfg, base = get_config(a.layered_model), get_config(a.layered_baseline)
     n = a.layers or 12
-    cfg = cfg.with_(num_layers=n, layer_specs=cfg.layer_specs[:n])
-    base = base.with_(num_layers=n)
+    cfg, base = cfg.with_(num_layers=n), base.with_(num_layers=n)
     for c in (cfg, base):
         print(json.dumps(throughput(c)), flush=True)
         torch.cuda.empty_cache()

@@ -342,13 +342,16 @@ def main():
     p.add_argument("--device", default="cuda" if torch.cuda.is_available() else "cpu")
     p.add_argument("--disable-radix-cache", action="store_true", help="do not reuse KV across requests with a common prefix")
     p.add_argument("--chunked-prefill-size", type=int, default=0, help="prefill long prompts in pieces of this many tokens (0: whole)")
+    p.add_argument("--mixed-batches", action="store_true",
+                   help="steps may carry pieces of prompts and one token of every running request together (layer-by-layer decoders)")
     a = p.parse_args()
     cfg = get_config(a.hf_checkpoint or a.model_name)
     dtype = torch.bfloat16 if a.device.startswith("cuda") else torch.float32
     if a.device.startswith("cuda") and torch.device(a.device).index is not None:
         torch.cuda.set_device(torch.device(a.device))      # kernels and allocations of this process default to its own GPU
     eng = Engine(cfg, device=a.device, dtype=dtype, mem_fraction_static=a.mem_fraction_static, max_running_requests=a.max_running_requests,
-                 prefix_cache=not a.disable_radix_cache, chunked_prefill_size=a.chunked_prefill_size or None)
+                 prefix_cache=not a.disable_radix_cache, chunked_prefill_size=a.chunked_prefill_size or None,
+                 mixed_batches=a.mixed_batches)
     if a.hf_checkpoint:
         eng.update_weights_from_disk(a.hf_checkpoint)
     serve(eng, a.host, a.port)

@@ -112,6 +112,11 @@ class LayeredConfig(FamilyConfig):
     layer_specs: tuple = ()
     bigram: BigramSpec | None = None
 
+    def with_(self, **kw) -> "LayeredConfig":
+        if "num_layers" in kw:                     # fewer layers: the first ones
+            kw.setdefault("layer_specs", self.layer_specs[: kw["num_layers"]])
+        return super().with_(**kw)
+
     def num_params(self, active_only: bool = False) -> int:
         n = 2 * self.vocab_size * self.hidden_size + self.hidden_size
         if self.bigram is not None and not active_only:
@@ -269,6 +274,7 @@ class LayeredModel(Qwen3Model):
     def __init__(self, cfg: LayeredConfig, ps=None, dtype=torch.bfloat16, device="cpu", seed: int = 0):
         super().__init__(cfg.with_(num_layers=0), ps, dtype=dtype, device=device, seed=seed, layer_range=(0, 0))
         assert self.ps.tp_size == 1 and self.ps.pp_size == 1 and self.ps.cp_size == 1, "layered models run on one rank"
+        assert len(cfg.layer_specs) == cfg.num_layers, f"{cfg.num_layers} layers, {len(cfg.layer_specs)} described"
         self.cfg = cfg
         gen = _Init(seed)
         self.layer_range = (0, cfg.num_layers)

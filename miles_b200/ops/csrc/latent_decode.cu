@@ -363,17 +363,25 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
   const float w = ml.x == -INFINITY ? 0.f : exp2f(ml.x - mm);
   const float den = mx::warp_sum(ml.y * w) + (sink != nullptr ? exp2f(sk - mm) : 0.f);
   const float f = den > 0.f ? __fdiv_rn(w, den) : 0.f;
+  // four columns per thread (rank_p is a multiple of 16): one round for 512
   const float* po = part_o + th * num_splits * L.rank_p;
-  for (int c0 = 0; c0 < L.rank; c0 += 128) {
-    const int c = c0 + threadIdx.x;
-    float r = 0.f;
-#pragma unroll 8
+  for (int c = threadIdx.x * 4; c - threadIdx.x * 4 < L.rank; c += 512) {
+    float4 r = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
     for (int s = 0; s < num_splits; ++s) {
       const float fs = __shfl_sync(0xffffffffu, f, s);
-      const float v = c < L.rank ? po[s * L.rank_p + c] : 0.f;
-      r = fs > 0.f ? fmaf(fs, v, r) : r;            // an empty split wrote nothing
+      if (fs > 0.f && c < L.rank_p) {               // an empty split wrote nothing
+        const float4 v = *reinterpret_cast<const float4*>(po + s * L.rank_p + c);
+        r.x = fmaf(fs, v.x, r.x);
+        r.y = fmaf(fs, v.y, r.y);
+        r.z = fmaf(fs, v.z, r.z);
+        r.w = fmaf(fs, v.w, r.w);
+      }
     }
-    if (c < L.rank) out[th * L.rank + c] = __float2bfloat16(r);
+    const float o[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (c + j < L.rank) out[th * L.rank + c + j] = __float2bfloat16(o[j]);
   }
 }
 

@@ -106,8 +106,8 @@ def _prefill_ok(lay, dt, scale) -> bool:
 
 def decode_splits(tokens: int, heads: int, window: int, block_size: int) -> int:
     """Key splits of latent_decode: enough (token, head group, split) CTAs for the 148 SMs (one resident per SM), whole key tiles."""
-    tile, group = (128, 32) if block_size % 64 == 0 else (64, 32 if heads > 16 else 16)
-    return max(1, min(32, 148 // (tokens * -(-heads // group)), -(-(window or 4096) // tile)))
+    group = 32 if block_size % 64 == 0 or heads > 16 else 16
+    return max(1, min(32, 148 // (tokens * -(-heads // group)), -(-(window or 4096) // 64)))
 
 
 def _key_ranges(meta, window: int):

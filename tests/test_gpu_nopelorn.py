@@ -274,7 +274,7 @@ def test_odd_inner_sizes_in_the_dense_gemm():
     from miles_b200.ops import cuda as K
 
     g = torch.Generator().manual_seed(0)
-    for M, N, Kd in ((5, 53, 37), (130, 131, 19), (40, 577, 100), (1, 7, 3)):
+    for M, N, Kd in ((5, 53, 37), (130, 131, 19), (40, 577, 100), (1, 7, 3), (5, 53, 64), (40, 577, 264), (20, 1001, 2048), (64, 333, 320)):
         a, b = torch.randn(M, Kd, generator=g).bfloat16().cuda(), torch.randn(N, Kd, generator=g).bfloat16().cuda()
         assert U.rel(K.gemm_nt(a, b), a.double() @ b.double().T) < 0.012
         assert U.rel(K.gemm_nt(a, b, out_dtype=torch.float32), a.double() @ b.double().T) < 1e-4
