@@ -376,7 +376,7 @@ class Engine:
 
     def flush_cache(self) -> bool:
         with self.lock:
-            if self.running or self.prefilling:
+            if self.running or self.prefilling or any(r.blocks for r in self.requests.values()):
                 return False
             if self.prefix_cache is not None:
                 self.prefix_cache.reset()
@@ -1115,7 +1115,7 @@ class Engine:
                     r.blocks += blocks
             reqs = [r for r, _, _ in entries]
             self._step_count += 1
-            if self.runner is not None and all(len(t) == 1 and r.chunk[0] > 0 for r, t, _ in entries):
+            if self.runner is not None and self.runner.high == 0 and all(len(t) == 1 and r.chunk[0] > 0 for r, t, _ in entries):
                 logits = self.runner.feed(reqs)
                 rows = [i for i, (_, _, w) in enumerate(entries) for _ in w]
                 out = logits[torch.tensor(rows, dtype=torch.int64, device=self.device)] if rows else logits[:0]

@@ -176,7 +176,7 @@ def load_named_into_model(model, named_tensors: Iterable[tuple[str, torch.Tensor
         from . import nopelorn
 
         if nopelorn.is_checkpoint(n for n, _ in named):
-            named = list(nopelorn.from_checkpoint(dict(named), cfg).items())
+            return nopelorn.load_into(params, named, cfg)
     elif named and (named[0][0].startswith("model.") or named[0][0].startswith("lm_head")):
         from ..weight_update.quant_export import dequantize_named, is_quantized_stream
 

@@ -77,7 +77,7 @@ _TOP = {"embed": "embed", "bigram": "bigram", "final.norm": "norm", "head": "lm_
 
 
 def is_checkpoint(names) -> bool:
-    return any(re.match(r"l\d+\.(mix|mlp|norm)", n) or n == "final.norm" for n in names)
+    return any(re.match(r"l\d+\.", n) or n in ("final.norm", "head") for n in names)
 
 
 def _stacks(spec: LayerSpec) -> dict[str, list[tuple[str, int]]]:
@@ -106,6 +106,43 @@ def _singles(spec: LayerSpec) -> dict[str, str]:
     if spec.mlp is not None:
         out.update({"norm2": "norm2", "ls2": "ls2", "mlp.w2": "mlp.down"})
     return out
+
+
+def place(name: str, cfg: LayeredConfig) -> tuple[str, int, int | None] | None:
+    """Where a checkpoint tensor goes: (our tensor, first row, rows; None: all of it).  None for a name that is none of the design's."""
+    if name in _TOP:
+        return _TOP[name], 0, None
+    m = re.match(r"l(\d+)\.(.+)", name)
+    if not m or int(m.group(1)) >= cfg.num_layers:
+        return None
+    i, rest = int(m.group(1)), m.group(2)
+    for ours, parts in _stacks(cfg.layer_specs[i]).items():
+        at = 0
+        for n, rows in parts:
+            if n == rest:
+                return f"layers.{i}.{ours}", at, rows
+            at += rows
+    for ours, n in _singles(cfg.layer_specs[i]).items():
+        if n == rest:
+            return f"layers.{i}.{ours}", 0, None
+    return None
+
+
+def load_into(params: dict, named, cfg: LayeredConfig) -> set:
+    """Copy checkpoint tensors (any subset: the parts of a stack may come apart) into the model's parameters.  Returns the
+    parameters of which every row was given."""
+    rows: dict[str, int] = {}
+    for name, t in named:
+        where = place(name, cfg)
+        if where is None:
+            continue
+        ours, at, n = where
+        p = params[ours].data
+        dst = p if n is None else p[at:at + n]
+        assert tuple(t.shape) == tuple(dst.shape), f"{name}: got {tuple(t.shape)}, the configuration says {tuple(dst.shape)}"
+        dst.copy_(t)
+        rows[ours] = rows.get(ours, 0) + dst.shape[0]
+    return {n for n, r in rows.items() if r >= params[n].shape[0]}
 
 
 def from_checkpoint(named: dict[str, torch.Tensor], cfg: LayeredConfig) -> dict[str, torch.Tensor]:

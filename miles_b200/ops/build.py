@@ -31,7 +31,7 @@ def sources() -> list[str]:
 # full build compiles only these (`build_serve`), into an extension of its own with the same interface.
 SERVE_SUFFIX = "_serve"
 SERVE_SOURCES = ["counter.cpp", "bindings.cpp", "bindings_more.cpp", "bindings_misc.cpp", "bindings_mixers.cpp", "gemm.cu", "gemm_small.cu",
-                 "gemv.cu", "misc.cu", "attention_tc.cu", "attention_latent_tc.cu", "mixers.cu", "latent_attn.cu", "latent_decode.cu", "latent_decode_tc.cu", "linear_state.cu",
+                 "gemv.cu", "misc.cu", "attention_latent_tc.cu", "mixers.cu", "latent_attn.cu", "latent_decode.cu", "latent_decode_tc.cu", "linear_state.cu",
                  "linear_chunk.cu"]
 
 

@@ -54,8 +54,6 @@ void flash_fwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, at
         "mb_flash_fwd");
 }
 
-#endif  // MB_SERVE_SUBSET
-
 void flash_fwd_tc(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, at::Tensor& o, const c10::optional<at::Tensor>& lse,
                   const at::Tensor& cu_seqlens, int64_t max_seqlen, double scale, bool causal, at::Tensor& err,
                   const c10::optional<at::Tensor>& cu_seqlens_k) {
@@ -68,7 +66,6 @@ void flash_fwd_tc(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v,
         "mb_flash_fwd_tc");
 }
 
-#ifndef MB_SERVE_SUBSET
 void flash_bwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& o, const at::Tensor& dout,
                const at::Tensor& lse, at::Tensor& delta, at::Tensor& dq, at::Tensor& dk, at::Tensor& dv, const at::Tensor& cu_seqlens,
                int64_t max_seqlen, double scale, bool causal) {
@@ -118,12 +115,12 @@ void register_mixers(pybind11::module& m); // bindings_mixers.cpp
 
 void register_more(pybind11::module& m) {
   m.def("install_crash_handler", &install_crash_handler);
-  m.def("flash_fwd_tc", &flash_fwd_tc);
-  m.def("flash_fwd_tc_ctas_per_sm", []() { return mb_flash_fwd_tc_ctas_per_sm(); });
   register_misc(m);
   register_mixers(m);
 #ifndef MB_SERVE_SUBSET
   m.def("flash_fwd", &flash_fwd);
+  m.def("flash_fwd_tc", &flash_fwd_tc);
+  m.def("flash_fwd_tc_ctas_per_sm", []() { return mb_flash_fwd_tc_ctas_per_sm(); });
   m.def("flash_bwd", &flash_bwd);
   m.def("flash_bwd_tc", &flash_bwd_tc);
   m.def("paged_decode", &paged_decode);

@@ -56,6 +56,23 @@ def test_checkpoint_names_round_trip():
     assert c.num_params() == sum(t.numel() for t in W.values())
 
 
+def test_weights_in_any_portions():
+    """A weight stream may cut a stacked projection anywhere between tensors."""
+    cfg = cases.config_a()
+    W = plain.make_weights(cfg, 12)
+    c = nopelorn.from_config(cfg)
+    from miles_b200.models.convert import load_named_into_model
+    from miles_b200.parallel.state import ParallelState
+
+    model = build_model(c, dtype=torch.float32)
+    whole = hf_state_to_ours(W, c)
+    for name, t in reversed(list(W.items())):
+        load_named_into_model(model, [(name, t)], c, ParallelState.single())
+    for n, p in model.named_parameters():
+        assert torch.equal(p.data, whole[n].float()), n
+    assert load_named_into_model(model, list(whole.items()), c, ParallelState.single()) == set(whole)
+
+
 def test_weights_from_disk(tmp_path):
     from miles_b200.checkpoint.hf_io import save_safetensors
 
