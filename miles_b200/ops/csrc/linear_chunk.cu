@@ -18,6 +18,7 @@ namespace lc {
 using mx::bf16;
 static constexpr int C = 64, P = 136, PP = C + 8, kThreads = 512;      // tokens per chunk, shared row lengths
 static constexpr int kTile = C * P;                                    // elements of a q / k / v tile (≤ 128 wide)
+static constexpr size_t kSmemSums = 6 * kTile * 2 + (C + 1) * 4 + 12;      // without state and scores: two CTAs per SM
 static constexpr size_t kSmem = (6 * kTile + 2 * 128 * P + 2 * C * PP) * 2 + (C + 1) * 4 + 12;
 
 __device__ __forceinline__ uint32_t s_addr(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
@@ -79,14 +80,14 @@ struct Args {
 
 // grid (heads, segments), 512 threads.  KD, VD: dk and dv when known at compile time, 0 otherwise.
 template <bool OUT, int KD, int VD>
-__global__ void __launch_bounds__(kThreads) linear_chunk_kernel(Args a) {
+__global__ void __launch_bounds__(kThreads, OUT ? 1 : 2) linear_chunk_kernel(Args a) {
   extern __shared__ __align__(128) uint8_t smem[];
   bf16* tile = reinterpret_cast<bf16*>(smem);        // [2][q | k | v][C][P]
   bf16* s_hi = tile + 6 * kTile;                     // [128][P]
   bf16* s_lo = s_hi + 128 * P;
   bf16* p_hi = s_lo + 128 * P;                       // [C][PP]
   bf16* p_lo = p_hi + C * PP;
-  float* pw = reinterpret_cast<float*>(p_lo + C * PP);   // λ^0 … λ^C
+  float* pw = reinterpret_cast<float*>(OUT ? p_lo + C * PP : s_hi);   // λ^0 … λ^C
   pdl_trigger();
   pdl_wait();
   const int h = blockIdx.x, seg = blockIdx.y;
@@ -351,14 +352,14 @@ extern "C" int mb_linear_chunk(const void* proj, long long ld, const float* deca
   static bool once[2] = {false, false};
   if (!once[big]) {
     cudaError_t e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kSmem));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(sums, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kSmem));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(sums, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kSmemSums));
     if (e != cudaSuccess) return static_cast<int>(e);
     once[big] = true;
   }
   Args a{reinterpret_cast<const bf16*>(proj), ld, decay, state, slots, positions, segs, seg_state, reinterpret_cast<bf16*>(out), H, dk, dv};
   cudaError_t e = cudaSuccess;
   if (seg_state != nullptr) {
-    e = launch_pdl(sums, dim3(H, n_seg), dim3(kThreads), kSmem, s, a);
+    e = launch_pdl(sums, dim3(H, n_seg), dim3(kThreads), kSmemSums, s, a);
     if (e == cudaSuccess)
       e = launch_pdl(linear_scan_kernel, dim3((dk * dv + 1023) / 1024, H, n_seq), dim3(256), 0, s, static_cast<const float*>(state), slots,
                      positions, decay, segs, seq_segs, seg_state, H, dk * dv);

@@ -73,17 +73,30 @@ def linear_state(proj, H, dk, dv, decay, state, meta):
     return out
 
 
+def _segment_cost(chunks: list[int], c: int, H: int, sms: int = 148) -> float:
+    """Chunk times of segments of c chunks: waves of full segments, the shorter last ones beside or behind the last wave.  A CTA's
+    start counts as one and a half chunks.  (A cut costs its caller a pass over keys and values more.)"""
+    start = 1.5
+    full, rest = sum(n // c for n in chunks) * H, [n % c for n in chunks if n % c]
+    waves = -(-full // sms)
+    time, slots = waves * (c + start), waves * sms - full
+    if rest:
+        if not slots:
+            return time + -(-len(rest) * H // sms) * (max(rest) + start)
+        time = max(time, (waves - 1) * (c + start) + -(-len(rest) * H // slots) * (max(rest) + start))
+    return time
+
+
 def _segments(meta, H: int):
     """Cut the long pieces of a batch into segments of whole 64-token chunks so that the (segment, head) CTAs, one per SM at a time,
-    finish in the fewest chunk times (a CTA's start counts as one and a half).  Returns ([n, 4] (sequence, first token, end, last of its sequence), offsets per sequence, any sequence cut)."""
+    finish in the fewest chunk times.  Returns ([n, 4] (sequence, first token, end, last of its sequence), offsets per sequence, any
+    sequence cut)."""
     rg = meta.ragged
     key = ("segments", H)
     if key not in rg.scratch:
         lens = rg.q_lens[: rg.n_long]
-        whole = -(-max(lens) // 64)                     # chunks of the longest piece; any cut costs a pass over keys and values more
-        best = min((-(-sum(-(-n // (64 * c)) for n in lens) * H // 148) * (min(c, whole) + 1.5) * (1.0 if c >= whole else 1.7), c)
-                   for c in {*range(2, 33), whole})
-        size = 64 * best[1]
+        whole = -(-max(lens) // 64)                     # chunks of the longest piece
+        size = 64 * min((_segment_cost([-(-n // 64) for n in lens], c, H) * (1.0 if c >= whole else 1.4), c) for c in {*range(2, 17), whole})[1]
         segs, cu, t = [], [0], 0
         for b, n in enumerate(lens):
             for a in range(0, n, size):
