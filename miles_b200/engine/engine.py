@@ -164,6 +164,8 @@ class Engine:
                 # recurrent states come out of the same budget as the paged cache
                 budget -= 4 * max_running_requests * sum(math.prod(s) for s in states.values())
                 num_blocks = KVCache.blocks_for_budget(max(budget, 1 << 28), len(self.model.layers), self.block_size, hkv, cfg.head_dim, dtype, rows)
+                if rows is not None:      # a model that keeps few bytes per token, or none, needs no more pages than its requests can fill
+                    num_blocks = min(num_blocks, max_running_requests * (-(-self.max_context_len // self.block_size) + 1))
             else:
                 num_blocks = 512
         lo, hi = self.model.layer_range

@@ -77,6 +77,18 @@ def test_generation(dtype, opts):
         assert e.runner is not None and e.runner.graphs
 
 
+def test_cache_sized_from_device_memory():
+    """No block count given: pages from the memory budget, never more than the requests can fill; all preset layers run."""
+    from miles_b200.engine.engine import Engine
+    from miles_b200.models.config import get_config
+
+    for layers in (4, 1):                        # 1: linear attention only, nothing cached per token
+        e = Engine(get_config("nopelorn-tiny").with_(num_layers=layers), device="cuda:0", max_running_requests=3, max_context_len=256)
+        assert e.kv.num_blocks == 3 * 5
+        out = e.generate([[1, 2, 3] * 20, [7]], {"temperature": 0.0, "max_new_tokens": 40})
+        assert [len(o["output_ids"]) for o in out] == [40, 40]
+
+
 def test_eager_decode_without_graphs():
     cfg = cases.config_a()
     W, toks = plain.make_weights(cfg, 2), U.tokens_for(cfg, 60, 2)

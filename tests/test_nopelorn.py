@@ -173,6 +173,26 @@ def test_greedy_generation(kw):
         assert e.stats.get("mixed_steps", 0) > 0
 
 
+def test_models_with_one_kind_of_layer():
+    """Only latent attention: no state slots, and shared prefixes come from the cache.  Only linear attention: no cached rows."""
+    cfg = plain.make_config([plain.latent_spec(window=19), plain.latent_spec(heads=2, window=50, kv_from=0)])
+    W = plain.make_weights(cfg, 13)
+    e = U.engine_for(cfg, W, **F32)
+    assert e.states is None and e.prefix_cache is not None
+    prompt = U.tokens_for(cfg, 40, 6)
+    for tail in ([], [3, 4, 5]):
+        p = prompt + tail
+        out = e.generate(p, {"temperature": 0.0, "max_new_tokens": 8})
+        assert out["output_ids"] == cases.greedy(cfg, W, p, 8)[0]
+    assert e.stats.get("prefix_cache_hit_tokens", 0) >= 32
+    cfg = plain.make_config([plain.lightning_spec(), plain.lightning_spec(heads=3, dim=4, vdim=20, ff=None)])
+    W = plain.make_weights(cfg, 14)
+    e = U.engine_for(cfg, W, **F32)
+    assert not e.kv.layers and e.kv.allocated and e.prefix_cache is None
+    p = U.tokens_for(cfg, 30, 7)
+    assert e.generate(p, {"temperature": 0.0, "max_new_tokens": 8})["output_ids"] == cases.greedy(cfg, W, p, 8)[0]
+
+
 def test_retraction_restarts_the_state():
     """Too few pages for all: a request loses its pages and slot, starts again from its prompt and output, same tokens."""
     cfg = cases.config_a()
