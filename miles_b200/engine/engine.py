@@ -261,7 +261,7 @@ class Engine:
 
     def _refuse_kv_handover(self):
         if self.ragged:
-            raise NotImplementedError("prefill / decode disaggregation hands over K and V tensors; this model caches latents and states")
+            raise NotImplementedError("prefill / decode disaggregation hands over K and V tensors; this model's layers keep other rows per token")
 
     def _slot_tensor(self, blocks: list[int], n: int) -> torch.Tensor:
         """Flat cache slots of positions 0 … n − 1 of a request with these blocks (built with tensor ops, not a Python loop)."""
@@ -1021,6 +1021,7 @@ class Engine:
         whole = all(r.chunk[0] == 0 for r in reqs)
         if self.ragged:
             meta = self._ragged_meta(reqs, toks, pos, slots, cu)
+            meta.record_topk = record
         elif whole or self.stateless:
             meta = ForwardMeta(
                 positions=torch.tensor(pos, dtype=torch.int32, device=dev),

@@ -54,6 +54,11 @@ class ModelConfig:
     def layer_is_moe(self, layer: int) -> bool:
         return self.is_moe and layer >= self.first_k_dense
 
+    @property
+    def num_moe_layers(self) -> int:
+        """Layers (layer runs, where layers run several times) that record a choice of experts per token."""
+        return sum(self.layer_is_moe(l) for l in range(self.num_layers))
+
     def num_params(self, active_only: bool = False) -> int:
         h = self.hidden_size
         attn = h * self.qkv_size + self.q_size * h + (2 * self.head_dim if self.qk_norm else 0)
@@ -112,8 +117,8 @@ class ModelConfig:
             path = os.path.join(cfg, "config.json") if os.path.isdir(cfg) else cfg
             with open(path) as f:
                 cfg = json.load(f)
-        if cfg.get("architecture") in ARCHITECTURES:
-            return ARCHITECTURES[cfg["architecture"]](cfg)
+        if (design := _architecture(cfg)) is not None:
+            return design.from_config(cfg)
         mt = cfg.get("model_type", "qwen3")
         heads = cfg["num_attention_heads"]
         head_dim = cfg.get("head_dim") or cfg["hidden_size"] // heads
@@ -152,14 +157,14 @@ class ModelConfig:
         return asdict(self)
 
 
-def _nopelorn(cfg: dict) -> ModelConfig:
-    from .nopelorn import from_config
+def _architecture(cfg: dict):
+    """The design whose config.json names an "architecture" of its own (None: a Hugging Face configuration)."""
+    if "architecture" not in cfg:
+        return None
+    from .designs import DESIGNS
 
-    return from_config(cfg)
+    return next((d for d in DESIGNS.values() if d.ARCHITECTURE == cfg["architecture"]), None)
 
-
-# designs whose config.json names an "architecture" of its own → reader of that file
-ARCHITECTURES = {"Nopelorn": _nopelorn}
 
 PRESETS: dict[str, ModelConfig] = {
     # CPU plumbing model of the tiny GRPO run
@@ -194,9 +199,10 @@ PRESETS: dict[str, ModelConfig] = {
 
 def get_config(name_or_path: str) -> ModelConfig:
     if name_or_path not in PRESETS and not os.path.exists(name_or_path):
-        from . import families, nopelorn  # noqa: F401  (register the presets of the other model families)
+        from . import designs, families  # noqa: F401  (register the presets of the other model families)
 
-        PRESETS.update(nopelorn.PRESETS)
+        for d in designs.DESIGNS.values():
+            PRESETS.update(d.PRESETS)
     if name_or_path in PRESETS:
         return PRESETS[name_or_path]
     if os.path.exists(name_or_path):

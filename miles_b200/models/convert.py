@@ -21,10 +21,10 @@ from .config import ModelConfig
 def to_hf(name: str, tensor: torch.Tensor, cfg: ModelConfig, *, expert_offset: int = 0, _plain: bool = False
           ) -> list[tuple[str, torch.Tensor]]:
     """Convert one *full* (un-sharded along TP) tensor of this package's layout into HF tensors."""
-    if getattr(cfg, "family", "qwen3") == "nopelorn":
-        from . import nopelorn
+    if getattr(cfg, "layer_specs", ()):
+        from . import designs           # layers listed one by one: the design's own names
 
-        return nopelorn.to_checkpoint(name, tensor, cfg)
+        return designs.to_checkpoint(name, tensor, cfg)
     if not _plain and getattr(cfg, "family", "qwen3") != "qwen3":
         from . import bridges           # latent / linear attention, shared experts, … of the other families
 
@@ -79,10 +79,10 @@ def to_hf(name: str, tensor: torch.Tensor, cfg: ModelConfig, *, expert_offset: i
 
 def hf_state_to_ours(hf: dict[str, torch.Tensor], cfg: ModelConfig, _plain: bool = False) -> dict[str, torch.Tensor]:
     """Assemble full tensors of this package's layout from an HF state dict."""
-    if getattr(cfg, "family", "qwen3") == "nopelorn":
-        from . import nopelorn
+    if getattr(cfg, "layer_specs", ()):
+        from . import designs
 
-        return nopelorn.from_checkpoint(hf, cfg)
+        return designs.from_checkpoint(hf, cfg)
     if not _plain and getattr(cfg, "family", "qwen3") != "qwen3":
         from . import bridges
 
@@ -172,11 +172,11 @@ def load_named_into_model(model, named_tensors: Iterable[tuple[str, torch.Tensor
     """Copy tensors into a model. Accepts this package's names (shard or full) or HF names (full).  Returns the names loaded."""
     named = list(named_tensors)
     params = dict(model.named_parameters_global() if hasattr(model, "named_parameters_global") else model.named_parameters())
-    if getattr(cfg, "family", "qwen3") == "nopelorn":
-        from . import nopelorn
+    if getattr(cfg, "layer_specs", ()):
+        from . import designs
 
-        if nopelorn.is_checkpoint(n for n, _ in named):
-            return nopelorn.load_into(params, named, cfg)
+        if designs.is_checkpoint((n for n, _ in named), cfg):
+            return designs.load_into(params, named, cfg)
     elif named and (named[0][0].startswith("model.") or named[0][0].startswith("lm_head")):
         from ..weight_update.quant_export import dequantize_named, is_quantized_stream
 

@@ -6,16 +6,23 @@ latent ranks or state sizes are a `LayeredConfig`: a tuple of `LayerSpec`s over 
     LatentMixer        latent attention over a paged cache of latents: sliding window, per-head softmax sink, interleaved
                        rotary with optional YaRN frequencies, layers that read another layer's latents (`kv_from`)
     LinearStateMixer   linear attention with a constant decay per head: fp32 state per sequence, gated norm over all heads
+    AttentionMixer     grouped-query attention over a paged cache of keys and values: sliding window that keeps the first tokens,
+                       per-head softmax sink, RMS norm over a token's whole query (key) projection, interleaved rotary
     ClampedGLU         gate and up projections with clamped pre-activations
-    LayeredModel       hashed-bigram embedding, norms on the sublayers' OUTPUTS with a layer scale, fp32 residual stream
+    RoutedExperts      clamped experts, the `top` largest of biased fp32 logits, weights by a softmax over the chosen ones
+    LayeredModel       hashed-bigram embedding, fp32 residual stream, layers in one of two arrangements (`LayeredConfig.block`):
+                       "output_norm"  mixer, then feed-forward, norms on the sublayers' OUTPUTS with a layer scale
+                       "parallel"     one norm in front; mixer and feed-forward read it side by side and are added together
+                       A range of layers may run several times with the same weights (`LoopSpec`), each pass on its own cache.
 
 The blocks run in the engine only (paged latents, state slots; no autograd).  What the design keeps in 32 bits — rotary
 angles, scores and softmax, norms, the residual sum, recurrent state and decays — is 32-bit in the kernels; matrix products
 and activations use the model's dtype (bfloat16, or float32 throughout).
 
 A forward pass takes a ragged batch: any number of new tokens per sequence (`ForwardMeta.ragged`), with sequences that bring
-at most `SHORT_Q` tokens last.  Long pieces expand the latents of their window to per-head keys and values; short ones (decode
-steps among them) attend to the latents directly with the key up-projection absorbed into the query.
+at most `SHORT_Q` tokens last.  Latent attention expands the latents of a long piece's window to per-head keys and values; short pieces (decode steps
+among them) attend to the latents directly with the key up-projection absorbed into the query.  Grouped-query attention runs long
+pieces as query tiles over the cached pages and short ones token by token.
 """
 from __future__ import annotations
 
@@ -40,12 +47,19 @@ class YarnScaling:
 
 
 @dataclass(frozen=True)
+class LinearScaling:
+    """Positions count `factor` times slower."""
+
+    factor: float
+
+
+@dataclass(frozen=True)
 class Rotary:
     """Rotary embedding of `dims` dimensions in interleaved pairs (2i, 2i + 1)."""
 
     base: float
     dims: int
-    scaling: YarnScaling | None = None
+    scaling: YarnScaling | LinearScaling | None = None
 
     def table(self) -> tuple[list[float], float]:
         """(angular frequency of every pair, factor on cosine and sine)."""
@@ -54,6 +68,8 @@ class Rotary:
         s = self.scaling
         if s is None:
             return freq, 1.0
+        if isinstance(s, LinearScaling):
+            return [f / s.factor for f in freq], 1.0
 
         def pair_of(turns: float) -> float:        # the (real-valued) dimension that turns this often over the original context
             return self.dims * math.log(s.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
@@ -88,6 +104,20 @@ class LinearStateSpec:
 
 
 @dataclass(frozen=True)
+class AttentionSpec:
+    heads: int
+    kv_heads: int
+    dim: int                       # query / key size per head
+    vdim: int
+    scale: float
+    rotary: Rotary | None = None   # rotates the first `rotary.dims` dimensions of queries and keys
+    window: int = 0                # keys a query sees, itself included; 0: all earlier ones
+    keep_first: int = 0            # tokens at the start of a sequence that stay visible whatever the window
+    qk_norm: bool = True           # RMS norm over a token's whole query (key) projection, before the heads are rotated
+    sink: bool = True              # a learned extra term in every head's softmax denominator
+
+
+@dataclass(frozen=True)
 class GluSpec:
     ff: int
     limit: float
@@ -95,9 +125,31 @@ class GluSpec:
 
 
 @dataclass(frozen=True)
+class MoeSpec:
+    experts: int
+    top: int
+    expert: GluSpec
+    shared: GluSpec | None = None  # runs for every token and is added
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentSpec | LinearStateSpec
-    mlp: GluSpec | None
+    mixer: LatentSpec | LinearStateSpec | AttentionSpec
+    mlp: GluSpec | MoeSpec | None
+
+    @property
+    def dense(self) -> GluSpec | None:
+        """The feed-forward every token passes (all of it, or the shared expert beside routed ones)."""
+        return self.mlp.shared if isinstance(self.mlp, MoeSpec) else self.mlp
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers start … stop − 1 run `times` times in a row; the embedding output is added before each pass but the first."""
+
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass(frozen=True)
@@ -111,36 +163,62 @@ class BigramSpec:
 class LayeredConfig(FamilyConfig):
     layer_specs: tuple = ()
     bigram: BigramSpec | None = None
+    block: str = "output_norm"         # or "parallel"
+    loop: LoopSpec | None = None
 
     def with_(self, **kw) -> "LayeredConfig":
         if "num_layers" in kw:                     # fewer layers: the first ones
-            kw.setdefault("layer_specs", self.layer_specs[: kw["num_layers"]])
+            n = kw["num_layers"]
+            kw.setdefault("layer_specs", self.layer_specs[:n])
+            if self.loop is not None and self.loop.stop > n:
+                kw.setdefault("loop", LoopSpec(self.loop.start, n, self.loop.times) if self.loop.start < n else None)
         return super().with_(**kw)
 
+    def runs(self) -> list[tuple[int, bool]]:
+        """The layer runs of a forward pass in order: (layer, the embedding output is added before it).  Caches and states belong to
+        runs: run r of this list owns entry r."""
+        if self.loop is None:
+            return [(i, False) for i in range(self.num_layers)]
+        lo, hi, n = self.loop.start, self.loop.stop, self.loop.times
+        return ([(i, False) for i in range(lo)] + [(i, t > 0 and i == lo) for t in range(n) for i in range(lo, hi)]
+                + [(i, False) for i in range(hi, self.num_layers)])
+
+    def layer_is_moe(self, layer: int) -> bool:
+        return isinstance(self.layer_specs[layer].mlp, MoeSpec)
+
+    @property
+    def num_moe_layers(self) -> int:
+        return sum(self.layer_is_moe(l) for l, _ in self.runs())
+
     def num_params(self, active_only: bool = False) -> int:
-        n = 2 * self.vocab_size * self.hidden_size + self.hidden_size
+        """Parameters; `active_only`: those a token meets, each as often as it meets it, without the embedding look-ups."""
+        H = self.hidden_size
+        n = H + self.vocab_size * H * (1 if self.tie_embeddings else 2)
         if self.bigram is not None and not active_only:
-            n += (self.bigram.buckets + 1) * self.hidden_size
-        for s in self.layer_specs:
-            n += sum(math.prod(shape) for shape in mixer_shapes(s.mixer, self.hidden_size).values()) + 2 * self.hidden_size
-            if s.mlp is not None:
-                n += 3 * s.mlp.ff * self.hidden_size + 2 * self.hidden_size
+            n += (self.bigram.buckets + 1) * H
+        for i in [l for l, _ in self.runs()] if active_only else range(self.num_layers):
+            s = self.layer_specs[i]
+            n += sum(math.prod(shape) for shape in layer_shapes(s, self).values())
+            if active_only and isinstance(s.mlp, MoeSpec):
+                n -= (s.mlp.experts - s.mlp.top) * 3 * s.mlp.expert.ff * H
         return n
 
     def flops_per_token(self, seq_len: int, backward: bool = True) -> float:
-        f = 2.0 * (self.num_params(active_only=True) - self.vocab_size * self.hidden_size)
-        for s in self.layer_specs:
-            m = s.mixer
+        f = 2.0 * (self.num_params(active_only=True) - (0 if self.tie_embeddings else self.vocab_size * self.hidden_size))
+        for i, _ in self.runs():
+            m = self.layer_specs[i].mixer
             if isinstance(m, LatentSpec):
                 f += 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim) * min(m.window or seq_len, seq_len / 2.0)
+            elif isinstance(m, AttentionSpec):
+                f += 2.0 * m.heads * (m.dim + m.vdim) * min(m.window + m.keep_first if m.window else seq_len, seq_len / 2.0)
             else:
                 f += 4.0 * m.heads * m.dim * m.vdim
         return f * (3.0 if backward else 1.0)
 
     def to_hf_config(self) -> dict:
-        from .nopelorn import to_config
+        from .designs import DESIGNS
 
-        return to_config(self)
+        return DESIGNS[self.family].to_config(self)
 
 
 def mixer_shapes(m, hidden: int) -> dict[str, tuple]:
@@ -153,14 +231,45 @@ def mixer_shapes(m, hidden: int) -> dict[str, tuple]:
         if m.sink:
             out["sink"] = (m.heads,)
         return out
+    if isinstance(m, AttentionSpec):
+        q, k = m.heads * m.dim, m.kv_heads * m.dim
+        out = {"w_in": (q + k + m.kv_heads * m.vdim, hidden), "wo": (hidden, m.heads * m.vdim)}
+        if m.qk_norm:
+            out.update({"q_norm": (q,), "k_norm": (k,)})
+        if m.sink:
+            out["sink"] = (m.heads,)
+        return out
     return {"w_in": (m.heads * 2 * (m.dim + m.vdim), hidden), "norm": (m.heads * m.vdim,), "wo": (hidden, m.heads * m.vdim)}
 
 
+def layer_shapes(s: LayerSpec, cfg: LayeredConfig) -> dict[str, tuple]:
+    """Parameter shapes of a whole layer.  In the parallel arrangement the mixer and the dense feed-forward share their input and
+    their sum, so their input projections are stacked along the rows and their output projections along the columns."""
+    H = cfg.hidden_size
+    mix = mixer_shapes(s.mixer, H)
+    out: dict[str, tuple] = {"norm1": (H,)}
+    if cfg.block == "parallel":
+        ff = s.dense.ff if s.dense is not None else 0
+        out["w_in"] = (mix.pop("w_in")[0] + 2 * ff, H)
+        out["w_out"] = (H, mix.pop("wo")[1] + ff)
+        if isinstance(s.mlp, MoeSpec):
+            E, F = s.mlp.experts, s.mlp.expert.ff
+            out.update({"mlp.router": (E, H), "mlp.bias": (E,), "mlp.w13": (E, 2 * F, H), "mlp.w2": (E, H, F)})
+    else:
+        out["ls1"] = (H,)
+        if s.mlp is not None:
+            out.update({"norm2": (H,), "ls2": (H,), "mlp.w13": (2 * s.mlp.ff, H), "mlp.w2": (H, s.mlp.ff)})
+    out.update({f"mix.{n}": shape for n, shape in mix.items()})
+    return out
+
+
 class _Mixer(nn.Module):
-    def __init__(self, spec, hidden: int, std: float, dtype, device, gen, tag: str):
+    def __init__(self, spec, hidden: int, std: float, dtype, device, gen, tag: str, without: tuple = ()):
         super().__init__()
         self.spec = spec
         for name, shape in mixer_shapes(spec, hidden).items():
+            if name in without:                    # projections the layer holds, stacked with others
+                continue
             if len(shape) == 2:
                 t = gen(f"{tag}.{name}", shape, std, dtype, device)
             else:
@@ -175,9 +284,9 @@ class LatentMixer(_Mixer):
         self.register_buffer("freq", torch.tensor(freq, dtype=torch.float64, device=self.wo.device), persistent=False)
         self.layout = MX.LatentLayout(spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank)
 
-    def forward(self, proj, meta: ForwardMeta, layer: int, eps: float):
+    def forward(self, proj, meta: ForwardMeta, run: int, eps: float):
         s = self.spec
-        cache = meta.kv_cache[layer if s.kv_from is None else s.kv_from][0]
+        cache = meta.kv_cache[run if s.kv_from is None else s.kv_from][0]
         return MX.latent_attention(proj, self.layout, cache, meta, freq=self.freq, magnitude=self.magnitude, scale=s.scale,
                                    window=s.window, sink=getattr(self, "sink", None), w_ukv=self.w_ukv,
                                    kv_norm=getattr(self, "kv_norm", None), eps=eps)
@@ -189,9 +298,49 @@ class LinearStateMixer(_Mixer):
         assert len(spec.decay) == spec.heads, "one decay per head"
         self.register_buffer("decay", torch.tensor(spec.decay, dtype=torch.float64, device=self.wo.device).float(), persistent=False)
 
-    def forward(self, proj, meta: ForwardMeta, layer: int, eps: float):
+    def forward(self, proj, meta: ForwardMeta, run: int, eps: float):
         s = self.spec
-        return MX.linear_state_attention(proj, s.heads, s.dim, s.vdim, self.decay, meta.states[layer], meta, self.norm, eps)
+        return MX.linear_state_attention(proj, s.heads, s.dim, s.vdim, self.decay, meta.states[run], meta, self.norm, eps)
+
+
+class AttentionMixer(_Mixer):
+    def __init__(self, spec: AttentionSpec, hidden: int, std: float, dtype, device, gen, tag: str, **kw):
+        super().__init__(spec, hidden, std, dtype, device, gen, tag, **kw)
+        assert spec.heads % spec.kv_heads == 0, "query heads come in equal groups"
+        freq = spec.rotary.table()[0] if spec.rotary is not None else []
+        assert 2 * len(freq) <= spec.dim, "the rotation covers at most a whole head"
+        self.register_buffer("freq", torch.tensor(freq, dtype=torch.float64, device=device), persistent=False)
+        self.magnitude = spec.rotary.table()[1] if spec.rotary is not None else 1.0
+        self.layout = MX.AttentionLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim, 2 * len(freq), spec.window, spec.keep_first)
+
+    def forward(self, proj, meta: ForwardMeta, run: int, eps: float, out=None, aside=None):
+        """proj [T, q; k; v (; more)] → [T, heads · vdim], into `out` if given.  `aside` (mixers.Aside): what reads the same
+        projection beside the attention."""
+        s = self.spec
+        kc, vc = meta.kv_cache[run]
+        if out is None:
+            out = torch.empty(proj.shape[0], s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
+        MX.windowed_attention(proj, self.layout, kc, vc, meta, out, freq=self.freq, magnitude=self.magnitude, scale=s.scale,
+                              sink=getattr(self, "sink", None), q_norm=getattr(self, "q_norm", None), k_norm=getattr(self, "k_norm", None),
+                              eps=eps, aside=aside)
+        return out
+
+
+class RoutedExperts(nn.Module):
+    def __init__(self, spec: MoeSpec, hidden: int, std: float, dtype, device, gen, tag: str):
+        super().__init__()
+        self.spec = spec
+        E, F = spec.experts, spec.expert.ff
+        assert 0 < spec.top <= E
+        self.router = nn.Parameter(gen(f"{tag}.router", (E, hidden), std, dtype, device))
+        self.bias = nn.Parameter(torch.zeros(E, dtype=dtype, device=device))
+        self.w13 = nn.Parameter(gen(f"{tag}.w13", (E, 2 * F, hidden), std, dtype, device))
+        self.w2 = nn.Parameter(gen(f"{tag}.w2", (E, hidden, F), std, dtype, device))
+
+    def forward(self, h, weights, index):
+        """What the chosen experts of every token add (`mixers.Addend`)."""
+        e = self.spec.expert
+        return MX.routed_experts(h, self.w13, self.w2, weights, index, e.limit, e.alpha)
 
 
 class ClampedGLU(nn.Module):
@@ -241,7 +390,12 @@ class _Stream:
         return MX.output_norm_residual(self.x.clone(), y, nw, ls, self.eps)[0]
 
 
+MIXERS = {LatentSpec: LatentMixer, LinearStateSpec: LinearStateMixer, AttentionSpec: AttentionMixer}
+
+
 class LayeredLayer(nn.Module):
+    """The "output_norm" arrangement."""
+
     def __init__(self, spec: LayerSpec, cfg: LayeredConfig, dtype, device, gen, layer: int):
         super().__init__()
         self.layer, self.eps = layer, cfg.rms_eps
@@ -250,7 +404,8 @@ class LayeredLayer(nn.Module):
         def vec():
             return nn.Parameter(torch.ones(H, dtype=dtype, device=device))
 
-        kind = LatentMixer if isinstance(spec.mixer, LatentSpec) else LinearStateMixer
+        assert not isinstance(spec.mlp, MoeSpec), "routed experts run in the parallel arrangement"
+        kind = MIXERS[type(spec.mixer)]
         self.norm1, self.ls1 = vec(), vec()
         self.mix = kind(spec.mixer, H, std, dtype, device, gen, f"L{layer}.mix")
         self.mlp = None
@@ -258,11 +413,96 @@ class LayeredLayer(nn.Module):
             self.norm2, self.ls2 = vec(), vec()
             self.mlp = ClampedGLU(spec.mlp, H, std, dtype, device, gen, f"L{layer}.mlp")
 
-    def forward(self, st: _Stream, meta: ForwardMeta):
-        o = self.mix(st.project(self.mix.w_in), meta, self.layer, self.eps)
+    def forward(self, st: _Stream, meta: ForwardMeta, run: int):
+        o = self.mix(st.project(self.mix.w_in), meta, run, self.eps)
         st.add(ops.linear(o, self.mix.wo), self.norm1, self.ls1)
         if self.mlp is not None:
             st.add(self.mlp(st.project(self.mlp.w13)), self.norm2, self.ls2)
+
+
+class _SumStream:
+    """The fp32 residual of the parallel arrangement and the sublayer outputs that have not been added to it yet.
+
+    `project` adds them (and, before a later pass of a loop, the embedding output), norms the sum and multiplies it by the layer's
+    input projection and its router: one kernel for a handful of rows; a kernel for sum and norm and the products otherwise."""
+
+    def __init__(self, x, _copy, eps: float):
+        self.x, self.first, self.eps = x, x, eps
+        self.pending: list = []
+        self.inject = False                        # the embedding output is due before the next layer
+
+    def _sum_into(self):
+        """Where the next sum goes: never over the embedding output."""
+        if not self.pending and not self.inject:
+            return None
+        return torch.empty_like(self.x) if self.x is self.first else self.x
+
+    def project(self, nw, w, router=None, bias=None, want_normed: bool = False):
+        """(normed residual or None, its product with `w`, fp32 router logits or None)"""
+        extra = self.first if self.inject else None
+        if MX.few_row_sum(self.x, self.pending, w):
+            h, proj, logits, self.x = MX.sum_norm_linear(self.x, self.pending, extra, nw, self.eps, w, router, bias, want_normed)
+        else:
+            to = self._sum_into()
+            h = MX.sum_norm(self.x, to, self.pending, extra, nw, self.eps)
+            self.x = self.x if to is None else to
+            proj, logits = MX.projections(h, w, router, bias)
+        self.pending, self.inject = [], False
+        return h, proj, logits
+
+    def finish(self, final_w):
+        return MX.sum_norm(self.x, None, self.pending, None, final_w, self.eps)
+
+    def value(self):
+        """The residual with everything added (debugging and tests)."""
+        x = torch.empty_like(self.x)
+        if not self.pending:
+            return x.copy_(self.x)
+        MX.sum_norm(self.x, x, self.pending, None, None, self.eps)
+        return x
+
+
+class ParallelLayer(nn.Module):
+    """The "parallel" arrangement: x + mixer(norm(x)) + feed-forward(norm(x)).
+
+    One input projection feeds queries, keys, values and the dense feed-forward; one output projection multiplies the concatenation
+    of the heads' outputs and the dense activations, so their sum is part of the product.  Routed experts run beside it."""
+
+    def __init__(self, spec: LayerSpec, cfg: LayeredConfig, dtype, device, gen, layer: int):
+        super().__init__()
+        self.layer, self.eps, self.dense = layer, cfg.rms_eps, spec.dense
+        H, std, tag = cfg.hidden_size, cfg.init_std, f"L{layer}"
+        assert isinstance(spec.mixer, AttentionSpec), "the parallel arrangement is built for attention mixers"
+        shapes = layer_shapes(spec, cfg)
+        self.norm1 = nn.Parameter(torch.ones(H, dtype=dtype, device=device))
+        self.w_in = nn.Parameter(gen(f"{tag}.w_in", shapes["w_in"], std, dtype, device))
+        self.w_out = nn.Parameter(gen(f"{tag}.w_out", shapes["w_out"], std, dtype, device))
+        self.mix = MIXERS[type(spec.mixer)](spec.mixer, H, std, dtype, device, gen, f"{tag}.mix", without=("w_in", "wo"))
+        self.mlp = RoutedExperts(spec.mlp, H, std, dtype, device, gen, f"{tag}.mlp") if isinstance(spec.mlp, MoeSpec) else None
+        self.at_dense = mixer_shapes(spec.mixer, H)["w_in"][0]      # first row of the dense feed-forward in the projection
+        self.mix_out = spec.mixer.heads * spec.mixer.vdim
+
+    def forward(self, st: _SumStream, meta: ForwardMeta, run: int):
+        moe = self.mlp
+        h, proj, logits = st.project(self.norm1, self.w_in, *((moe.router, moe.bias, True) if moe is not None else ()))
+        both = torch.empty(proj.shape[0], self.w_out.shape[1], dtype=proj.dtype, device=proj.device)
+        aside = MX.Aside(logits=logits, top=moe.spec.top if moe is not None else 0)
+        if self.dense is not None:
+            aside.glu_in, aside.glu_out = proj[:, self.at_dense:], both[:, self.mix_out:]
+            aside.limit, aside.alpha = self.dense.limit, self.dense.alpha
+        self.mix(proj, meta, run, self.eps, out=both[:, : self.mix_out], aside=aside)
+        st.pending = [MX.Addend(ops.linear(both, self.w_out))]
+        if moe is not None:
+            if meta.record_topk is not None:
+                meta.record_topk.append(_as_recorded(aside.index, meta.record_width))
+            st.pending.append(moe(h, aside.weights, aside.index))
+
+
+def _as_recorded(index, width: int):
+    """Expert ids of one layer in the width the engine records (−1: no such choice)."""
+    if index.shape[1] == width:
+        return index
+    return torch.nn.functional.pad(index, (0, width - index.shape[1]), value=-1)
 
 
 class LayeredModel(Qwen3Model):
@@ -279,37 +519,58 @@ class LayeredModel(Qwen3Model):
         gen = _Init(seed)
         self.layer_range = (0, cfg.num_layers)
         self.has_embed = self.has_head = True
+        assert cfg.block in BLOCKS, f"unknown arrangement of layers '{cfg.block}'"
         for i, s in enumerate(cfg.layer_specs):
             m = s.mixer
             if isinstance(m, LatentSpec) and m.kv_from is not None:
                 src = cfg.layer_specs[m.kv_from].mixer
                 assert m.kv_from < i and isinstance(src, LatentSpec) and src.kv_from is None and (src.kv_rank, src.rot_dim) == (
                     m.kv_rank, m.rot_dim), f"layer {i} cannot read the latents of layer {m.kv_from}"
-        self.layers = nn.ModuleList(LayeredLayer(s, cfg, dtype, device, gen, l) for l, s in enumerate(cfg.layer_specs))
+        if cfg.loop is not None:
+            assert 0 <= cfg.loop.start < cfg.loop.stop <= cfg.num_layers and cfg.loop.times > 0, f"{cfg.loop} of {cfg.num_layers} layers"
+            assert cfg.block == "parallel", "loops are built for the parallel arrangement"
+        kind = BLOCKS[cfg.block][0]
+        self.layers = nn.ModuleList(kind(s, cfg, dtype, device, gen, l) for l, s in enumerate(cfg.layer_specs))
+        self.runs = cfg.runs()
         self.bigram = None
         if cfg.bigram is not None:
             self.bigram = nn.Parameter(gen("bigram", (cfg.bigram.buckets + 1, cfg.hidden_size), cfg.init_std, dtype, device))
-        self.num_moe_layers = 0
+        self.num_moe_layers = cfg.num_moe_layers
 
     # ---- what the engine keeps per token and per sequence ------------------------------------------------------------
+    def _run_mixers(self):
+        return [(r, self.layers[l].mix) for r, (l, _) in enumerate(self.runs)]
+
     def kv_rows(self) -> dict[int, tuple]:
-        """Cache row shapes per token of every layer that writes one."""
-        return {l.layer: ((l.mix.layout.pitch,),) for l in self.layers if isinstance(l.mix, LatentMixer) and l.mix.spec.kv_from is None}
+        """Cache row shapes per token of every layer run that writes one."""
+        rows: dict[int, tuple] = {}
+        for r, m in self._run_mixers():
+            if isinstance(m, LatentMixer) and m.spec.kv_from is None:
+                rows[r] = ((m.layout.pitch,),)
+            elif isinstance(m, AttentionMixer):
+                rows[r] = ((m.spec.kv_heads, m.spec.dim), (m.spec.kv_heads, m.spec.vdim))
+        return rows
 
     def state_shapes(self) -> dict[int, tuple]:
-        """fp32 state per sequence of every recurrent layer."""
-        return {l.layer: (l.mix.spec.heads, l.mix.spec.dim, l.mix.spec.vdim) for l in self.layers if isinstance(l.mix, LinearStateMixer)}
+        """fp32 state per sequence of every recurrent layer run."""
+        return {r: (m.spec.heads, m.spec.dim, m.spec.vdim) for r, m in self._run_mixers() if isinstance(m, LinearStateMixer)}
 
     def forward(self, tokens, meta: ForwardMeta, hidden_in=None, inputs_embeds=None):
         if torch.is_grad_enabled():
             raise NotImplementedError("layered models run in the engine only: no backward pass is built for their mixers")
         assert meta.ragged is not None, "layered models take ragged engine batches"
         big = self.cfg.bigram
-        x, xb = MX.bigram_embedding(tokens, meta.prev_tokens, self.embed, self.bigram,
-                                    (big.buckets, big.mul_prev, big.mul_cur) if big is not None else None)
-        st = _Stream(x, xb, self.cfg.rms_eps)
-        for layer in self.layers:
-            layer(st, meta)
+        st = BLOCKS[self.cfg.block][1](*MX.bigram_embedding(tokens, meta.prev_tokens, self.embed, self.bigram,
+                                                            (big.buckets, big.mul_prev, big.mul_cur) if big is not None else None,
+                                                            want_copy=self.cfg.block == "output_norm"), self.cfg.rms_eps)
+        meta.record_width = self.cfg.moe_topk
+        for run, (l, inject) in enumerate(self.runs):
+            st.inject = inject
+            self.layers[l](st, meta, run)
             if meta.record_residual is not None:
                 meta.record_residual.append(st.value())
         return st.finish(self.norm)
+
+
+# arrangement → (layer, stream of residual and pending outputs)
+BLOCKS = {"output_norm": (LayeredLayer, _Stream), "parallel": (ParallelLayer, _SumStream)}

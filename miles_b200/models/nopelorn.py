@@ -7,10 +7,6 @@ of one input are stacked (`mix.w_in`, `mix.w_ukv`, `mlp.w13`).
 """
 from __future__ import annotations
 
-import re
-
-import torch
-
 from .layered import (BigramSpec, GluSpec, LatentSpec, LayeredConfig, LayerSpec, LinearStateSpec, Rotary, YarnScaling)
 
 ARCHITECTURE = "Nopelorn"
@@ -73,105 +69,32 @@ def to_config(cfg: LayeredConfig) -> dict:
 
 # ---- tensor names -----------------------------------------------------------------------------------------------------
 
-_TOP = {"embed": "embed", "bigram": "bigram", "final.norm": "norm", "head": "lm_head"}
+def tensors(cfg: LayeredConfig) -> dict:
+    from .designs import Place, rows_of
 
-
-def is_checkpoint(names) -> bool:
-    return any(re.match(r"l\d+\.", n) or n in ("final.norm", "head") for n in names)
-
-
-def _stacks(spec: LayerSpec) -> dict[str, list[tuple[str, int]]]:
-    """Our stacked tensor → the checkpoint tensors it holds, in order, with their row counts."""
-    m = spec.mixer
-    if isinstance(m, LatentSpec):
-        w_in = [("mix.q", m.heads * (m.dim + m.rot_dim))] + ([("mix.dkv", m.kv_rank + m.rot_dim)] if m.kv_from is None else [])
-        out = {"mix.w_in": w_in, "mix.w_ukv": [("mix.uk", m.heads * m.dim), ("mix.uv", m.heads * m.vdim)]}
-    else:
-        out = {"mix.w_in": [("mix.q", m.heads * m.dim), ("mix.k", m.heads * m.dim), ("mix.v", m.heads * m.vdim), ("mix.g", m.heads * m.vdim)]}
-    if spec.mlp is not None:
-        out["mlp.w13"] = [("mlp.gate", spec.mlp.ff), ("mlp.up", spec.mlp.ff)]
-    return out
-
-
-def _singles(spec: LayerSpec) -> dict[str, str]:
-    m = spec.mixer
-    out = {"norm1": "norm1", "ls1": "ls1", "mix.wo": "mix.o"}
-    if isinstance(m, LatentSpec):
-        if m.kv_from is None:
-            out["mix.kv_norm"] = "mix.dkv.norm"
-        if m.sink:
-            out["mix.sink"] = "mix.sink"
-    else:
-        out["mix.norm"] = "mix.norm"
-    if spec.mlp is not None:
-        out.update({"norm2": "norm2", "ls2": "ls2", "mlp.w2": "mlp.down"})
-    return out
-
-
-def place(name: str, cfg: LayeredConfig) -> tuple[str, int, int | None] | None:
-    """Where a checkpoint tensor goes: (our tensor, first row, rows; None: all of it).  None for a name that is none of the design's."""
-    if name in _TOP:
-        return _TOP[name], 0, None
-    m = re.match(r"l(\d+)\.(.+)", name)
-    if not m or int(m.group(1)) >= cfg.num_layers:
-        return None
-    i, rest = int(m.group(1)), m.group(2)
-    for ours, parts in _stacks(cfg.layer_specs[i]).items():
-        at = 0
-        for n, rows in parts:
-            if n == rest:
-                return f"layers.{i}.{ours}", at, rows
-            at += rows
-    for ours, n in _singles(cfg.layer_specs[i]).items():
-        if n == rest:
-            return f"layers.{i}.{ours}", 0, None
-    return None
-
-
-def load_into(params: dict, named, cfg: LayeredConfig) -> set:
-    """Copy checkpoint tensors (any subset: the parts of a stack may come apart) into the model's parameters.  Returns the
-    parameters of which every row was given."""
-    rows: dict[str, int] = {}
-    for name, t in named:
-        where = place(name, cfg)
-        if where is None:
-            continue
-        ours, at, n = where
-        p = params[ours].data
-        dst = p if n is None else p[at:at + n]
-        assert tuple(t.shape) == tuple(dst.shape), f"{name}: got {tuple(t.shape)}, the configuration says {tuple(dst.shape)}"
-        dst.copy_(t)
-        rows[ours] = rows.get(ours, 0) + dst.shape[0]
-    return {n for n, r in rows.items() if r >= params[n].shape[0]}
-
-
-def from_checkpoint(named: dict[str, torch.Tensor], cfg: LayeredConfig) -> dict[str, torch.Tensor]:
-    out = {ours: named[n] for n, ours in _TOP.items() if n in named}
+    out = {"embed": Place("embed"), "final.norm": Place("norm"), "head": Place("lm_head")}
+    if cfg.bigram is not None:
+        out["bigram"] = Place("bigram")
     for i, s in enumerate(cfg.layer_specs):
-        for ours, parts in _stacks(s).items():
-            if all(f"l{i}.{n}" in named for n, _ in parts):
-                ts = [named[f"l{i}.{n}"] for n, _ in parts]
-                for t, (n, rows) in zip(ts, parts):
-                    assert t.shape[0] == rows, f"l{i}.{n}: {t.shape[0]} rows, the configuration says {rows}"
-                out[f"layers.{i}.{ours}"] = torch.cat(ts, 0)
-        for ours, n in _singles(s).items():
-            if f"l{i}.{n}" in named:
-                out[f"layers.{i}.{ours}"] = named[f"l{i}.{n}"]
+        m, l, p = s.mixer, f"l{i}", f"layers.{i}"
+        single = {"norm1": "norm1", "ls1": "ls1", "mix.o": "mix.wo"}
+        if isinstance(m, LatentSpec):
+            out.update(rows_of(f"{p}.mix.w_in", [(f"{l}.mix.q", m.heads * (m.dim + m.rot_dim))]
+                               + ([(f"{l}.mix.dkv", m.kv_rank + m.rot_dim)] if m.kv_from is None else [])))
+            out.update(rows_of(f"{p}.mix.w_ukv", [(f"{l}.mix.uk", m.heads * m.dim), (f"{l}.mix.uv", m.heads * m.vdim)]))
+            if m.kv_from is None:
+                single["mix.dkv.norm"] = "mix.kv_norm"
+            if m.sink:
+                single["mix.sink"] = "mix.sink"
+        else:
+            out.update(rows_of(f"{p}.mix.w_in", [(f"{l}.mix.q", m.heads * m.dim), (f"{l}.mix.k", m.heads * m.dim),
+                                                 (f"{l}.mix.v", m.heads * m.vdim), (f"{l}.mix.g", m.heads * m.vdim)]))
+            single["mix.norm"] = "mix.norm"
+        if s.mlp is not None:
+            out.update(rows_of(f"{p}.mlp.w13", [(f"{l}.mlp.gate", s.mlp.ff), (f"{l}.mlp.up", s.mlp.ff)]))
+            single.update({"norm2": "norm2", "ls2": "ls2", "mlp.down": "mlp.w2"})
+        out.update({f"{l}.{theirs}": Place(f"{p}.{ours}") for theirs, ours in single.items()})
     return out
-
-
-def to_checkpoint(name: str, tensor: torch.Tensor, cfg: LayeredConfig) -> list[tuple[str, torch.Tensor]]:
-    """One tensor of ours → the checkpoint's tensors."""
-    inv = {v: k for k, v in _TOP.items()}
-    if name in inv:
-        return [(inv[name], tensor)]
-    m = re.match(r"layers\.(\d+)\.(.+)", name)
-    i, rest = int(m.group(1)), m.group(2)
-    stacks = _stacks(cfg.layer_specs[i])
-    if rest in stacks:
-        parts = stacks[rest]
-        return [(f"l{i}.{n}", t) for (n, _), t in zip(parts, tensor.split([r for _, r in parts], 0))]
-    return [(f"l{i}.{_singles(cfg.layer_specs[i])[rest]}", tensor)]
 
 
 _ROT = dict(base=20000.0, dims=16, scaling=YarnScaling(4.0, 256, 24.0, 1.5))

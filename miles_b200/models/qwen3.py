@@ -42,6 +42,7 @@ class ForwardMeta:
     # routing replay / recording
     replay_topk: torch.Tensor | None = None  # int32 [T, L_moe, k] recorded indices (-1 rows → fallthrough)
     record_topk: "list[torch.Tensor] | None" = None  # filled with int32 [T,k] per MoE layer when not None
+    record_width: int = 0                    # k of those records where layers differ in it (narrower layers pad with −1)
     recompute: bool = False                  # activation checkpoint each layer
     lora_slots: torch.Tensor | None = None   # int64 [T] adapter slot per token (None → slot 0; -1 → base model only)
     # prefill that continues cached KV (a prefix-cache hit, a later piece of a chunked prompt): packed offsets of the new
@@ -52,7 +53,7 @@ class ForwardMeta:
     prev_tokens: torch.Tensor | None = None    # int32 [T] token before each new token, −1 for a sequence's first
     state_slots: torch.Tensor | None = None    # int32 [B] recurrent-state slot per sequence (−1: padding row)
     states: "dict[int, torch.Tensor] | None" = None      # layer → [slots, ...] fp32 states
-    record_residual: "list[torch.Tensor] | None" = None  # filled with the residual stream after every layer when not None
+    record_residual: "list[torch.Tensor] | None" = None  # filled with the residual stream after every layer run when not None
 
 
 @dataclass

@@ -105,3 +105,78 @@ def linear_state(proj, H, dk, dv, decay, state, meta):
 def gated_norm(o, w, gate, eps):
     of = o.float()
     return (of * torch.rsqrt(of.square().mean(-1, keepdim=True) + eps) * w.float() * torch.sigmoid(gate.float())).to(o.dtype)
+
+
+def sum_norm(x, to, addends, extra, nw, eps):
+    s = x.clone()
+    for a in addends:
+        s += a.y.float()
+    if extra is not None:
+        s += extra
+    if to is not None:
+        to.copy_(s)
+    if nw is None:
+        return None
+    return (s * torch.rsqrt(s.square().mean(-1, keepdim=True) + eps) * nw.float()).to(nw.dtype)
+
+
+def projections(h, w, w2=None, b2=None):
+    logits = None
+    if w2 is not None:
+        logits = h.float() @ w2.float().T + b2.float()
+    return h @ w.T, logits
+
+
+def topk_softmax(logits, k):
+    top = logits.float().topk(k, -1)
+    return torch.softmax(top.values, -1), top.indices.int()
+
+
+def routed_experts(h, w13, w2, weights, index, limit, alpha):
+    out = torch.zeros(h.shape, dtype=torch.float32)
+    for e in range(w13.shape[0]):
+        t, j = torch.where(index == e)
+        if t.numel():
+            y = clamped_glu(h[t] @ w13[e].T, limit, alpha) @ w2[e].T
+            out.index_add_(0, t, y.float() * weights[t, j][:, None])
+    return out.to(h.dtype)
+
+
+def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps):
+    T, H, G = proj.shape[0], lay.heads, lay.kv_heads
+    q, k, v = proj[:, : lay.rows].split([H * lay.dim, G * lay.dim, G * lay.vdim], -1)
+
+    def prepared(x, w, heads):
+        x = x.float()
+        if w is not None:
+            x = x * torch.rsqrt(x.square().mean(-1, keepdim=True) + eps) * w.float()
+        x = x.view(T, heads, lay.dim)
+        if lay.rot:
+            x = torch.cat([rotate_pairs(x[..., : lay.rot], meta.positions, freq, magnitude), x[..., lay.rot:]], -1)
+        return x.to(proj.dtype)
+
+    q, k = prepared(q, q_norm, H), prepared(k, k_norm, G)
+    ok = meta.slot_mapping >= 0
+    at = meta.slot_mapping[ok].long()
+    kc.view(-1, G, lay.dim)[at] = k[ok].to(kc.dtype)
+    vc.view(-1, G, lay.vdim)[at] = v.reshape(T, G, lay.vdim)[ok].to(vc.dtype)
+    bs = kc.shape[1]
+    out.zero_()
+    for b, s0, s1 in _sequences(meta, T):
+        if s1 == s0 or int(meta.slot_mapping[s0]) < 0:
+            continue
+        pos = meta.positions[s0:s1].long()
+        keys = torch.arange(int(pos[-1]) + 1)
+        slot = meta.block_table[b, keys // bs].long() * bs + keys % bs
+        kk = kc.view(-1, G, lay.dim)[slot].float().repeat_interleave(H // G, 1)
+        vv = vc.view(-1, G, lay.vdim)[slot].float().repeat_interleave(H // G, 1)
+        sc = torch.einsum("thd,shd->hts", q[s0:s1].float(), kk) * scale
+        seen = keys[None] <= pos[:, None]
+        if lay.window:
+            seen &= (pos[:, None] - keys[None] < lay.window) | (keys[None] < lay.keep)
+        sc = sc.masked_fill(~seen[None], float("-inf"))
+        if sink is not None:
+            sc = torch.cat([sc, sink.float()[:, None, None].expand(H, s1 - s0, 1)], -1)
+        p = torch.softmax(sc, -1)[..., : keys.numel()]
+        out[s0:s1] = torch.einsum("hts,shd->thd", p, vv).reshape(s1 - s0, -1).to(out.dtype)
+    return out

@@ -207,7 +207,7 @@ def create_rollout_components(args, ps: ParallelState, actor=None, tracker=None)
                 box = [router_url, worker_urls]
                 torch.distributed.broadcast_object_list(box, src=0)
                 router_url, worker_urls = box
-        n_moe = sum(cfg.layer_is_moe(l) for l in range(cfg.num_layers))
+        n_moe = cfg.num_moe_layers
         n_prefill = int(getattr(args, "rollout_pd_prefill_engines", 0) or 0)
         if n_prefill > 0:
             # prefill / decode disaggregation: the first engines of the fleet run prompts, the others continue from their KV
