@@ -36,14 +36,15 @@ def main(argv=None) -> int:
     if not torch.cuda.is_available():
         print("trace replay runs the CUDA kernels: no CUDA device found", file=sys.stderr)
         return 2
-    build.build_serve()
     from ..models.config import get_config
+
+    cfg = get_config(a.model)
+    build.build_serve(build.serve_kind(cfg))
     from .engine import Engine
 
     # a true 32-bit run: no TF32 in the dense projections
     torch.backends.cuda.matmul.allow_tf32 = False
     torch.cuda.set_device(0)
-    cfg = get_config(a.model)
     engine = Engine(cfg, device="cuda:0", dtype=getattr(torch, a.dtype), num_blocks=max(1, -(-a.max_tokens // a.block_size)), block_size=a.block_size,
                     max_running_requests=SLOTS, max_context_len=max(a.max_tokens, a.block_size), prefix_cache=False)
     engine.update_weights_from_disk(a.model)

@@ -27,12 +27,25 @@ def sources() -> list[str]:
     return sorted(glob.glob(os.path.join(CSRC, "*.cu")) + glob.glob(os.path.join(CSRC, "*.cpp")))
 
 
-# What serving a layer-by-layer decoder (models/layered.py) takes: dense projections, its mixers, sampling.  A checkout without a
-# full build compiles only these (`build_serve`), into an extension of its own with the same interface.
+# What serving a layer-by-layer decoder (models/layered.py) takes: dense projections, sampling and the mixers its layers have.  A
+# checkout without a full build compiles only these (`build_serve`), into an extension of its own with the same interface.
 SERVE_SUFFIX = "_serve"
 SERVE_SOURCES = ["counter.cpp", "bindings.cpp", "bindings_more.cpp", "bindings_misc.cpp", "bindings_mixers.cpp", "gemm.cu", "gemm_small.cu",
-                 "gemv.cu", "misc.cu", "attention_latent_tc.cu", "mixers.cu", "latent_attn.cu", "latent_decode.cu", "latent_decode_tc.cu", "linear_state.cu",
-                 "linear_chunk.cu"]
+                 "gemv.cu", "misc.cu", "mixers.cu", "paged_attend.cu"]
+SERVE_KINDS = {
+    "latent": ["attention_latent_tc.cu", "latent_attn.cu", "latent_decode.cu", "latent_decode_tc.cu", "linear_state.cu", "linear_chunk.cu"],
+    "attention": ["bindings_moe.cpp", "moe.cu", "attention_window_tc.cu", "window_prep.cu", "window_decode.cu", "experts_any.cu"],
+}
+_serving: str | None = None                   # the serving build this process asked for
+
+
+def serve_kind(cfg) -> str:
+    """Which serving build a layered configuration needs."""
+    from ..models.layered import AttentionSpec
+
+    kinds = {"attention" if isinstance(s.mixer, AttentionSpec) else "latent" for s in cfg.layer_specs}
+    assert len(kinds) == 1, f"no serving build has the mixers of {kinds} together: run a full build"
+    return kinds.pop()
 
 
 def source_stamp() -> str:
@@ -64,26 +77,29 @@ def debug_requested() -> bool:
     return os.environ.get("MILES_DEBUG_KERNELS", "0") == "1"
 
 
-def serve_so_path() -> str:
-    return os.path.join(BUILD_DIR + SERVE_SUFFIX, EXT_NAME + SERVE_SUFFIX + ".so")
+def serve_so_path(kind: str) -> str:
+    name = f"{SERVE_SUFFIX}_{kind}"
+    return os.path.join(BUILD_DIR + name, EXT_NAME + name + ".so")
 
 
-def build_serve(verbose: bool = False) -> str:
-    """Make sure an extension that can serve layer-by-layer decoders is built from the sources as they are: an up-to-date full
-    build if there is one, else the serving subset.  Returns its path; `load()` then picks the same one."""
+def build_serve(kind: str, verbose: bool = False) -> str:
+    """Make sure an extension that can serve layer-by-layer decoders with this kind of mixers is built from the sources as they are:
+    an up-to-date full build if there is one, else the serving subset.  Returns its path; `load()` then picks the same one."""
+    global _serving
     if _is_current(so_path(False)):
         return so_path(False)
-    so = serve_so_path()
+    so = serve_so_path(kind)
     if not _is_current(so):
         from torch.utils import cpp_extension
 
         _toolchain_env()
         os.makedirs(os.path.dirname(so), exist_ok=True)
         cpp_extension.load(
-            name=EXT_NAME + SERVE_SUFFIX, sources=[os.path.join(CSRC, f) for f in SERVE_SOURCES],
-            extra_cflags=["-O3", "-std=c++17", "-DMB_SERVE_SUBSET"], extra_cuda_cflags=NVCC_FLAGS, extra_include_paths=[CSRC],
-            build_directory=os.path.dirname(so), verbose=verbose, with_cuda=True)
+            name=f"{EXT_NAME}{SERVE_SUFFIX}_{kind}", sources=[os.path.join(CSRC, f) for f in SERVE_SOURCES + SERVE_KINDS[kind]],
+            extra_cflags=["-O3", "-std=c++17", "-DMB_SERVE_SUBSET", f"-DMB_SERVE_{kind.upper()}"], extra_cuda_cflags=NVCC_FLAGS,
+            extra_include_paths=[CSRC], build_directory=os.path.dirname(so), verbose=verbose, with_cuda=True)
         _write_stamp(so)
+    _serving = kind
     return so
 
 
@@ -133,8 +149,11 @@ def load():
 
     debug = debug_requested()
     path, suffix = so_path(debug), DEBUG_SUFFIX if debug else ""
-    if not debug and not _is_current(path) and _is_current(serve_so_path()):
-        path, suffix = serve_so_path(), SERVE_SUFFIX
+    if not debug and not _is_current(path):
+        for kind in [_serving] if _serving else SERVE_KINDS:
+            if _is_current(serve_so_path(kind)):
+                path, suffix = serve_so_path(kind), f"{SERVE_SUFFIX}_{kind}"
+                break
     if not os.path.exists(path):
         raise ImportError(
             f"{path} not found: build the CUDA extension with `python -m miles_b200.ops.build` "

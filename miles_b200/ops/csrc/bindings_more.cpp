@@ -117,6 +117,9 @@ void register_more(pybind11::module& m) {
   m.def("install_crash_handler", &install_crash_handler);
   register_misc(m);
   register_mixers(m);
+#if !defined(MB_SERVE_SUBSET) || defined(MB_SERVE_ATTENTION)
+  register_moe(m);
+#endif
 #ifndef MB_SERVE_SUBSET
   m.def("flash_fwd", &flash_fwd);
   m.def("flash_fwd_tc", &flash_fwd_tc);
@@ -124,7 +127,6 @@ void register_more(pybind11::module& m) {
   m.def("flash_bwd", &flash_bwd);
   m.def("flash_bwd_tc", &flash_bwd_tc);
   m.def("paged_decode", &paged_decode);
-  register_moe(m);
   register_fabric(m);
   register_extra(m);
 #endif

@@ -495,26 +495,39 @@ static PFN_encodeTiled get_encode_fn() {
 
 // 2-D bf16 tensor map over a row-major [rows, cols] matrix with leading dimension `ld` (elements);
 // box = [box_rows, box_cols] with 128-byte swizzle (box_cols·2 bytes must be 128).
-int make_tmap_bf16_2d(CUtensorMap* out, const void* base, long long rows, long long cols, long long ld, int box_rows,
-                      int box_cols) {
+static int encode_bf16(CUtensorMap* out, const void* base, int rank, const cuuint64_t* dims, const cuuint64_t* strides, const cuuint32_t* box) {
   PFN_encodeTiled enc = get_encode_fn();
   if (enc == nullptr) return -1;
-  cuuint64_t dims[2] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(rows)};
-  cuuint64_t strides[1] = {static_cast<cuuint64_t>(ld) * 2};
-  cuuint32_t box[2] = {static_cast<cuuint32_t>(box_cols), static_cast<cuuint32_t>(box_rows)};
-  cuuint32_t estr[2] = {1, 1};
-  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
-                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  const cuuint32_t estr[3] = {1, 1, 1};
+  auto encode = [&] {
+    return enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, rank, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  };
+  CUresult r = encode();
   if (r == CUDA_ERROR_INVALID_CONTEXT) {
     // a host thread that has not made a runtime call yet (e.g. an autograd worker) has no context bound:
     // bind the device's primary context and encode again
     cudaFree(nullptr);
-    r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
-            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    r = encode();
   }
   return r == CUDA_SUCCESS ? 0 : static_cast<int>(r);
+}
+
+int make_tmap_bf16_2d(CUtensorMap* out, const void* base, long long rows, long long cols, long long ld, int box_rows,
+                      int box_cols) {
+  const cuuint64_t dims[2] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(rows)};
+  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(ld) * 2};
+  const cuuint32_t box[2] = {static_cast<cuuint32_t>(box_cols), static_cast<cuuint32_t>(box_rows)};
+  return encode_bf16(out, base, 2, dims, strides, box);
+}
+
+// [outer, mid, cols], contiguous
+int make_tmap_bf16_3d(CUtensorMap* out, const void* base, long long outer, long long mid, long long cols, int box_outer, int box_mid,
+                      int box_cols) {
+  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(mid), static_cast<cuuint64_t>(outer)};
+  const cuuint64_t strides[2] = {static_cast<cuuint64_t>(cols) * 2, static_cast<cuuint64_t>(mid * cols) * 2};
+  const cuuint32_t box[3] = {static_cast<cuuint32_t>(box_cols), static_cast<cuuint32_t>(box_mid), static_cast<cuuint32_t>(box_outer)};
+  return encode_bf16(out, base, 3, dims, strides, box);
 }
 
 static int g_num_sms = 0;

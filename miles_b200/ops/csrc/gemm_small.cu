@@ -310,7 +310,7 @@ extern "C" int mb_gemm_small_grouped(const void* X, const void* W, void* C, int 
                                      const int* used_rows, int bt, int* error_flag, cudaStream_t s) {
   using namespace mb;
   if (rows <= 0 || N <= 0) return 0;
-  if (rows % bt || N % sm::BMW) return -1;
+  if (rows % bt) return -1;
   CUtensorMap tw, tx;
   int r = make_tmap_bf16_2d(&tw, W, static_cast<long long>(num_experts) * N, K, K, sm::BMW, sm::BK);
   if (r) return 1000 + r;
@@ -319,6 +319,6 @@ extern "C" int mb_gemm_small_grouped(const void* X, const void* W, void* C, int 
   sm::Params p{};
   p.tokens = rows; p.N = N; p.K = K; p.C = C; p.ldc = N; p.out_fp32 = 0;
   p.tile_expert = tile_expert; p.used_rows = used_rows; p.grouped = 1; p.split_k = 1; p.error_flag = error_flag;
-  const int tiles = (N / sm::BMW) * (rows / bt);
+  const int tiles = ((N + sm::BMW - 1) / sm::BMW) * (rows / bt);      // a tile may reach into the next expert's rows: never stored
   return sm::dispatch(bt, tw, tx, p, tiles, s);
 }

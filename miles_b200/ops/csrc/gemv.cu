@@ -15,11 +15,13 @@
 //     permutation of k.   lane = 4·g + t: A rows g and g+8, k ∈ [32c + 8t, 32c + 8t + 8); B column (token) g, same k.
 //
 //   gemv            y[M, N] = norm?(x (+ residual)) · W[N, K]ᵀ (+ bias)       M ≤ 16; optional fused add + RMSNorm prologue
-//   moe_gemv_up     act[pair, F] = silu(W13[e][:F] x) · (W13[e][F:] x)        per distinct expert of the step, T ≤ 8 tokens
+//   moe_gemv_up     act[pair, F] = silu(W13[e][:F] x) · (W13[e][F:] x), or the clamped form of mixers.cuh
+//                   per distinct expert of the step, T ≤ 8 tokens
 //   moe_gemv_down   out[T, H] = Σ_experts gate_w · W2[e] · act                 accumulated over experts in registers
 #include <cuda_bf16.h>
 
 #include "launch.h"
+#include "mixers.cuh"
 #include "pdl.cuh"
 
 namespace mb {
@@ -208,6 +210,57 @@ __device__ __forceinline__ void stage_rows_output_norm(uint8_t* xs, int rows, in
   }
 }
 
+// Sum-norm form: x' = x + y1 + y2 + extra (fp32 x and extra, every addend optional; block 0 writes x' to x_out, another buffer); the
+// staged value is bf16(x' · norm_w), Σx'² → rstd[row].
+__device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int valid, int K, const float* __restrict__ x,
+                                                    const bf16* __restrict__ y1, const bf16* __restrict__ y2, const float* __restrict__ extra,
+                                                    const bf16* __restrict__ norm_w, float eps, float* x_out, float* rstd) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int nv = K / 8, stride = staged_stride(K);
+  for (int r = warp; r < rows; r += kWarps) {
+    uint8_t* row = xs + r * stride;
+    if (r >= valid) {
+      for (int v = lane; v < nv; v += 32) *reinterpret_cast<uint4*>(row + v * 16) = make_uint4(0, 0, 0, 0);
+      if (lane == 0) rstd[r] = 0.f;
+      continue;
+    }
+    const long long base = static_cast<long long>(r) * K;
+    float ss = 0.f;
+#pragma unroll 2
+    for (int v = lane; v < nv; v += 32) {
+      const long long at = base + v * 8;
+      float f[8];
+      const float4 a = *reinterpret_cast<const float4*>(x + at), b = *reinterpret_cast<const float4*>(x + at + 4);
+      const uint4 zero = make_uint4(0, 0, 0, 0);
+      const uint4 p1 = y1 != nullptr ? *reinterpret_cast<const uint4*>(y1 + at) : zero;
+      const uint4 p2 = y2 != nullptr ? *reinterpret_cast<const uint4*>(y2 + at) : zero;
+      const uint4 nw = *reinterpret_cast<const uint4*>(norm_w + v * 8);
+      f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+      if (extra != nullptr) {
+        const float4 c = *reinterpret_cast<const float4*>(extra + at), d = *reinterpret_cast<const float4*>(extra + at + 4);
+        f[0] += c.x; f[1] += c.y; f[2] += c.z; f[3] += c.w; f[4] += d.x; f[5] += d.y; f[6] += d.z; f[7] += d.w;
+      }
+      const uint32_t w1[4] = {p1.x, p1.y, p1.z, p1.w}, w2[4] = {p2.x, p2.y, p2.z, p2.w}, wn[4] = {nw.x, nw.y, nw.z, nw.w};
+      uint32_t o[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 u = unpack2(w1[i]), q = unpack2(w2[i]), n = unpack2(wn[i]);
+        f[2 * i] += u.x + q.x;
+        f[2 * i + 1] += u.y + q.y;
+        ss += f[2 * i] * f[2 * i] + f[2 * i + 1] * f[2 * i + 1];
+        o[i] = pack2(f[2 * i] * n.x, f[2 * i + 1] * n.y);
+      }
+      if (x_out != nullptr && blockIdx.x == 0) {
+        *reinterpret_cast<float4*>(x_out + at) = make_float4(f[0], f[1], f[2], f[3]);
+        *reinterpret_cast<float4*>(x_out + at + 4) = make_float4(f[4], f[5], f[6], f[7]);
+      }
+      *reinterpret_cast<uint4*>(row + v * 16) = make_uint4(o[0], o[1], o[2], o[3]);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) rstd[r] = __fdiv_rn(1.f, __fsqrt_rn(__fdiv_rn(ss, static_cast<float>(K)) + eps));
+  }
+}
+
 // Plain copy of rows [0, valid) of a [*, K] bf16 matrix into shared memory with cp.async (every piece in flight at once, no
 // registers); rows [valid, rows) are zeroed.  The caller commits the group and waits for it before the CTA barrier.
 __device__ __forceinline__ void stage_rows_async(uint8_t* xs, int rows, int valid, int K, const bf16* __restrict__ x) {
@@ -237,16 +290,23 @@ struct GemvParams {
   const float* x32;       // output-norm form: fp32 residual, layer scale, and where the new residual goes
   const bf16* scale_w;
   float* x32_out;
+  const bf16 *y1, *y2;    // sum-norm form: sublayer outputs and an fp32 addend
+  const float* extra;
+  const bf16* W2;         // a second weight [N2, K] behind the first: fp32 y2out[M, N2] (+ bias2)
+  const bf16* bias2;
+  float* y2out;
+  int N2;
   int M, N, K;
   int static_w;           // W is not written by a kernel that may still run: its first loads go before the dependency wait
 };
 
-enum GemvMode { kPlain = 0, kAddNorm = 1, kOutputNorm = 2 };
+enum GemvMode { kPlain = 0, kAddNorm = 1, kOutputNorm = 2, kSumNorm = 3 };
 
 // NT: groups of 8 tokens (1 or 2); S: ring stages.  One CTA = 16 output rows; its 8 warps take the 32-wide k chunks round-robin.
 template <int NT, int MODE, int S>
 __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   constexpr bool NORM = MODE == kAddNorm;
+  constexpr bool SCALED = NORM || MODE == kSumNorm;      // the staged rows still lack 1 / rms
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float red[kWarps][NT][16][8];
   __shared__ float rstd_s[NT * 8];
@@ -255,10 +315,14 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   uint8_t* xs = smem + S * 2 * kThreads * 16;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
-  const int n0 = blockIdx.x * 16;
-  const int ra = min(n0 + g, p.N - 1), rb = min(n0 + g + 8, p.N - 1);
-  const bf16* wa_ptr = p.W + static_cast<long long>(ra) * p.K + t * 8;
-  const bf16* wb_ptr = p.W + static_cast<long long>(rb) * p.K + t * 8;
+  const int first_blocks = (p.N + 15) / 16;
+  const bool second = static_cast<int>(blockIdx.x) >= first_blocks;      // CTAs of the second weight
+  const int N = second ? p.N2 : p.N;
+  const bf16* W = second ? p.W2 : p.W;
+  const int n0 = (blockIdx.x - (second ? first_blocks : 0)) * 16;
+  const int ra = min(n0 + g, N - 1), rb = min(n0 + g + 8, N - 1);
+  const bf16* wa_ptr = W + static_cast<long long>(ra) * p.K + t * 8;
+  const bf16* wb_ptr = W + static_cast<long long>(rb) * p.K + t * 8;
   const int chunks = p.K / 32;
   const int n_i = chunks > warp ? (chunks - warp + kWarps - 1) / kWarps : 0;   // this warp's chunks: warp, warp + 8, …
   auto issue = [&](int i) {
@@ -277,6 +341,8 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
     stage_rows<true>(xs, NT * 8, p.M, p.K, p.x, p.residual, p.norm_w, p.eps, p.res_out, rstd_s);
   } else if (MODE == kOutputNorm) {
     stage_rows_output_norm(xs, NT * 8, p.M, p.K, p.x, p.x32, p.norm_w, p.scale_w, p.eps, p.x32_out);
+  } else if (MODE == kSumNorm) {
+    stage_rows_sum_norm(xs, NT * 8, p.M, p.K, p.x32, p.y1, p.y2, p.extra, p.norm_w, p.eps, p.x32_out, rstd_s);
   } else {
     stage_rows_async(xs, NT * 8, p.M, p.K, p.x);
     cp_commit();
@@ -308,14 +374,32 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   for (int i = threadIdx.x; i < NT * 128; i += kThreads) {
     const int j = i >> 7, tk = (i >> 4) & 7, row = i & 15;
     const int tok = tk + 8 * j, n = n0 + row;
-    if (tok < p.M && n < p.N) {
+    if (tok < p.M && n < N) {
       float s = 0.f;
 #pragma unroll
       for (int w = 0; w < kWarps; ++w) s += red[w][j][row][tk];
-      if (NORM) s *= rstd_s[tok];
+      if (SCALED) s *= rstd_s[tok];
+      if (second) {
+        if (p.bias2 != nullptr) s += __bfloat162float(p.bias2[n]);
+        p.y2out[static_cast<long long>(tok) * p.N2 + n] = s;
+        continue;
+      }
       if (p.bias != nullptr) s += __bfloat162float(p.bias[n]);
       if (p.out_fp32) reinterpret_cast<float*>(p.y)[tok * p.ldy + n] = s;
       else reinterpret_cast<bf16*>(p.y)[tok * p.ldy + n] = __float2bfloat16(s);
+    }
+  }
+  if (MODE == kSumNorm && p.xn_out != nullptr && blockIdx.x == 0) {
+    const float* xr = p.x32_out != nullptr ? p.x32_out : p.x32;      // this CTA's own writes, or nothing was added
+    for (int i = threadIdx.x; i < p.M * (p.K / 8); i += kThreads) {
+      const int tok = i / (p.K / 8), kv = (i % (p.K / 8)) * 8;
+      const long long at = static_cast<long long>(tok) * p.K + kv;
+      const float4 a = *reinterpret_cast<const float4*>(xr + at), b = *reinterpret_cast<const float4*>(xr + at + 4);
+      const uint4 nw = *reinterpret_cast<const uint4*>(p.norm_w + kv);
+      const float2 n0w = unpack2(nw.x), n1w = unpack2(nw.y), n2w = unpack2(nw.z), n3w = unpack2(nw.w);
+      const float r = rstd_s[tok];
+      *reinterpret_cast<uint4*>(p.xn_out + at) = make_uint4(pack2(a.x * r * n0w.x, a.y * r * n0w.y), pack2(a.z * r * n1w.x, a.w * r * n1w.y),
+                                                            pack2(b.x * r * n2w.x, b.y * r * n2w.y), pack2(b.z * r * n3w.x, b.w * r * n3w.y));
     }
   }
   if (NORM && p.xn_out != nullptr && blockIdx.x == 0) {
@@ -372,7 +456,7 @@ __device__ __forceinline__ int pair_of(unsigned long long mask, int tok, int k) 
 // across its items without a break (the ring keeps filling while the CTA reduces and stores an item).
 __global__ void __launch_bounds__(kThreads) moe_gemv_up_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w13,
                                                                const int* __restrict__ topk_idx, bf16* __restrict__ act, int T, int k,
-                                                               int E, int offset, int H, int F) {
+                                                               int E, int offset, int H, int F, float limit, float alpha) {
   constexpr int S = kMoeStages;
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float red[kWarps][16][8];
@@ -473,7 +557,7 @@ __global__ void __launch_bounds__(kThreads) moe_gemv_up_kernel(const bf16* __res
         // the two halves are rounded to bf16 first, like the stored pre-activation of the general path
         gate = __bfloat162float(__float2bfloat16(gate));
         up = __bfloat162float(__float2bfloat16(up));
-        const float a = gate / (1.f + __expf(-gate)) * up;
+        const float a = alpha != 0.f ? mx::clamped_glu_t<bf16>(gate, up, limit, alpha) : gate / (1.f + __expf(-gate)) * up;
         act[static_cast<long long>(pair) * F + f0 + f] = __float2bfloat16(a);
       }
     }
@@ -616,7 +700,7 @@ static cudaError_t launch_gemv(const GemvParams& p, cudaStream_t s) {
     if (e != cudaSuccess) return e;
     configured = kMaxSmem;
   }
-  return launch_pdl(gemv_kernel<NT, MODE, kDenseStages>, dim3((p.N + 15) / 16), dim3(kThreads), bytes, s, p);
+  return launch_pdl(gemv_kernel<NT, MODE, kDenseStages>, dim3((p.N + 15) / 16 + (p.N2 + 15) / 16), dim3(kThreads), bytes, s, p);
 }
 
 }  // namespace gv
@@ -673,9 +757,39 @@ extern "C" int mb_gemv_output_norm(const float* x, const void* y, const void* no
   return static_cast<int>(nt == 1 ? launch_gemv<1, kOutputNorm>(p, s) : launch_gemv<2, kOutputNorm>(p, s));
 }
 
-// MoE FFN for T ≤ 8 tokens (T·k ≤ 64): act [T·k, F] scratch, out [T, H].  H and F multiples of 32, H a multiple of 16.
+// See launch.h; same limits as mb_gemv.
+extern "C" int mb_gemv_sum_norm(const float* x32, const void* y1, const void* y2, const float* extra, const void* x, const void* norm_w, float eps,
+                                const void* W, void* y, long long ldy, const void* W2, const void* bias2, float* out2, float* x_out, void* xn_out,
+                                int M, int N, int N2, int K, int static_w, cudaStream_t s) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M > 16 || K % 32 || K <= 0) return -1;
+  const int nt = M <= 8 ? 1 : 2;
+  if (kDenseStages * 2 * kThreads * 16 + nt * 8 * staged_stride(K) > kMaxSmem) return -2;
+  GemvParams p{};
+  p.x = reinterpret_cast<const bf16*>(x);
+  p.x32 = x32;
+  p.y1 = reinterpret_cast<const bf16*>(y1);
+  p.y2 = reinterpret_cast<const bf16*>(y2);
+  p.extra = extra;
+  p.norm_w = reinterpret_cast<const bf16*>(norm_w);
+  p.eps = eps;
+  p.W = reinterpret_cast<const bf16*>(W);
+  p.y = y;
+  p.ldy = ldy;
+  p.W2 = reinterpret_cast<const bf16*>(W2);
+  p.bias2 = reinterpret_cast<const bf16*>(bias2);
+  p.y2out = out2;
+  p.N2 = W2 != nullptr ? N2 : 0;
+  p.x32_out = x_out;
+  p.xn_out = reinterpret_cast<bf16*>(xn_out);
+  p.M = M; p.N = N; p.K = K; p.static_w = static_w;
+  if (x32 == nullptr) return static_cast<int>(nt == 1 ? launch_gemv<1, kPlain>(p, s) : launch_gemv<2, kPlain>(p, s));
+  return static_cast<int>(nt == 1 ? launch_gemv<1, kSumNorm>(p, s) : launch_gemv<2, kSumNorm>(p, s));
+}
+
+// MoE FFN for T ≤ 8 tokens (T·k ≤ 64): act [T·k, F] scratch, out [T, H].  alpha ≠ 0: clamped activation, else SwiGLU.  H and F multiples of 32, H a multiple of 16.
 extern "C" int mb_moe_gemv(const void* x, const void* w13, const void* w2, const int* topk_idx, const float* topk_w, void* act, void* out,
-                           int T, int k, int E, int expert_offset, int H, int F, cudaStream_t s) {
+                           int T, int k, int E, int expert_offset, int H, int F, float limit, float alpha, cudaStream_t s) {
   if (T <= 0) return 0;
   if (T > 8 || T * k > kMaxPairs || H % 32 || F % 32) return -1;
   const int ring_bytes = kMoeStages * 2 * kThreads * 16;
@@ -692,7 +806,7 @@ extern "C" int mb_moe_gemv(const void* x, const void* w13, const void* w2, const
   const int max_items = (T * k < E ? T * k : E) * (F / 8);
   const int up_grid = max_items < 2 * 148 ? max_items : 2 * 148;
   cudaError_t e = launch_pdl(moe_gemv_up_kernel, dim3(up_grid), dim3(kThreads), up_bytes, s, reinterpret_cast<const bf16*>(x),
-                             reinterpret_cast<const bf16*>(w13), topk_idx, reinterpret_cast<bf16*>(act), T, k, E, expert_offset, H, F);
+                             reinterpret_cast<const bf16*>(w13), topk_idx, reinterpret_cast<bf16*>(act), T, k, E, expert_offset, H, F, limit, alpha);
   if (e != cudaSuccess) return static_cast<int>(e);
   e = launch_pdl(moe_gemv_down_kernel, dim3(H / 16), dim3(kThreads), down_bytes, s, reinterpret_cast<const bf16*>(act),
                  reinterpret_cast<const bf16*>(w2), topk_idx, topk_w, reinterpret_cast<bf16*>(out), T, k, E, expert_offset, H, F);

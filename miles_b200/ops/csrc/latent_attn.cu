@@ -1,6 +1,6 @@
 // Latent attention over a paged cache of latents (any sizes, bf16 or float): rotation and caching of the new tokens' latents, per-head
-// projections, and attention in the absorbed form — the query carries the key up-projection, so keys are the cached rows
-// themselves and the value up-projection follows on the attended latent.
+// projections.  Attention in the absorbed form — the query carries the key up-projection, so keys are the cached rows
+// themselves and the value up-projection follows on the attended latent — is paged_attend.cu for any size.
 //
 // A cached row is [latent (rank) | 0 … rank_p | rotated key part (rot) | 0 … pitch); rank_p and pitch are multiples of 16.
 // An absorbed query has the same layout per head, so a score is one dot product over a row.
@@ -28,22 +28,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
   const long long t = blockIdx.x;
   const int half = L.rot / 2, dq = L.dim + L.rot;
   const T* p = proj + t * ld;
-  const double pos = positions[t];
-  for (int i = threadIdx.x; i < half; i += 256) {
-    double a = pos * freq[i];
-    a -= rint(a * 0.15915494309189535) * 6.283185307179586;      // one turn off per whole turn: |a| ≤ π
-    if constexpr (is_exact<T>::value) {
-      double s, c;
-      sincos(a, &s, &c);
-      cs[i] = static_cast<float>(c * magnitude);
-      cs[half + i] = static_cast<float>(s * magnitude);
-    } else {
-      float s, c;
-      __sincosf(static_cast<float>(a), &s, &c);
-      cs[i] = c * magnitude;
-      cs[half + i] = s * magnitude;
-    }
-  }
+  rotary_table<T, 256>(cs, positions[t], freq, half, magnitude);
   auto rotate = [&](float (&f)[V], int k) {      // V values, the first one the even half of pair k
 #pragma unroll
     for (int j = 0; j < V; j += 2) {
@@ -126,77 +111,6 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
   y[t * y_t + h * y_h + n] = from_f<T>(s);
 }
 
-// grid (heads, tokens), 128 threads: each warp takes every fourth key with its own running softmax; RL · 32 ≥ rank.
-template <typename T, int RL>
-__global__ void __launch_bounds__(128) latent_attend_kernel(const T* __restrict__ q, const T* __restrict__ cache,
-                                                            const int* __restrict__ block_table, int max_blocks, int block_size,
-                                                            const int* __restrict__ token_seq, const int* __restrict__ positions,
-                                                            const long long* __restrict__ slots, const T* __restrict__ sink,
-                                                            T* __restrict__ out, float scale, int window, MbLatent L) {
-  extern __shared__ float sm[];
-  float* sq = sm;                        // [pitch]
-  float* so = sq + L.pitch;              // [4][rank]
-  __shared__ float s_m[4], s_l[4];
-  pdl_trigger();
-  pdl_wait();
-  const long long t = blockIdx.y;
-  const int h = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  T* o = out + (t * L.heads + h) * L.rank;
-  if (slots[t] < 0) {                    // padding row of a decode batch
-    for (int i = threadIdx.x; i < L.rank; i += 128) o[i] = from_f<T>(0.f);
-    return;
-  }
-  const int pos = positions[t];
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
-  const int* bt = block_table + static_cast<long long>(token_seq != nullptr ? token_seq[t] : t) * max_blocks;
-  for (int i = threadIdx.x; i < L.pitch; i += 128) sq[i] = to_f(q[(t * L.heads + h) * L.pitch + i]);
-  __syncthreads();
-  float m = -INFINITY, l = 0.f, acc[RL];
-#pragma unroll
-  for (int i = 0; i < RL; ++i) acc[i] = 0.f;
-  for (int key = lo + warp; key <= pos; key += 4) {
-    const T* row = cache + (static_cast<long long>(bt[key / block_size]) * block_size + key % block_size) * L.pitch;
-    float v[RL], s = 0.f;
-#pragma unroll
-    for (int i = 0; i < RL; ++i) {
-      const int c = lane + 32 * i;
-      v[i] = c < L.rank ? to_f(row[c]) : 0.f;
-      s = fmaf(v[i], c < L.rank ? sq[c] : 0.f, s);
-    }
-    for (int c = L.rank_p + lane; c < L.pitch; c += 32) s = fmaf(to_f(row[c]), sq[c], s);
-    s = warp_sum(s) * scale;
-    const float mn = fmaxf(m, s);
-    const float a = exp_t<T>(m - mn), p = exp_t<T>(s - mn);
-    m = mn;
-    l = fmaf(l, a, p);
-#pragma unroll
-    for (int i = 0; i < RL; ++i) acc[i] = fmaf(acc[i], a, p * v[i]);
-  }
-#pragma unroll
-  for (int i = 0; i < RL; ++i) {
-    const int c = lane + 32 * i;
-    if (c < L.rank) so[warp * L.rank + c] = acc[i];
-  }
-  if (lane == 0) { s_m[warp] = m; s_l[warp] = l; }
-  __syncthreads();
-  float mm = sink != nullptr ? to_f(sink[h]) : -INFINITY;
-#pragma unroll
-  for (int w = 0; w < 4; ++w) mm = fmaxf(mm, s_m[w]);
-  float f[4], den = sink != nullptr ? exp_t<T>(to_f(sink[h]) - mm) : 0.f;
-#pragma unroll
-  for (int w = 0; w < 4; ++w) {
-    f[w] = s_m[w] == -INFINITY ? 0.f : exp_t<T>(s_m[w] - mm);
-    den = fmaf(s_l[w], f[w], den);
-  }
-  for (int i = threadIdx.x; i < L.rank; i += 128) {
-    float r = 0.f;
-#pragma unroll
-    for (int w = 0; w < 4; ++w) r = fmaf(so[w * L.rank + i], f[w], r);
-    o[i] = from_f<T>(__fdiv_rn(r, den));
-  }
-}
-
 template <typename T>
 static int prep(const T* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
                 const T* kv_norm, float eps, T* cache, T* q_abs, T* q_full, int n, int t_long, int q_nope, int q_width, MbLatent L,
@@ -221,32 +135,6 @@ static int head_linear(const T* x, long long x_t, long long x_h, const T* w, int
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   return 0;
-}
-
-template <typename T, int RL>
-static int attend_rl(const T* q, const T* cache, const int* bt, int mb_, int bs, const int* seq, const int* pos, const long long* slots,
-                     const T* sink, T* out, int n, float scale, int window, MbLatent L, cudaStream_t s) {
-  const size_t bytes = (L.pitch + 4 * L.rank) * sizeof(float);
-  if (bytes > 48 * 1024) return -3;
-  for (int t0 = 0; t0 < n; t0 += 65535) {
-    const long long H = L.heads;
-    const cudaError_t e = launch_pdl(latent_attend_kernel<T, RL>, dim3(L.heads, n - t0 < 65535 ? n - t0 : 65535), dim3(128), bytes, s,
-                                     q + t0 * H * L.pitch, cache, bt, mb_, bs, seq != nullptr ? seq + t0 : seq, pos + t0, slots + t0, sink,
-                                     out + t0 * H * L.rank, scale, window, L);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    if (seq == nullptr && n > 65535) return -3;      // a decode batch (token = row) never gets this large
-  }
-  return 0;
-}
-
-template <typename T>
-static int attend(const T* q, const T* cache, const int* bt, int mb_, int bs, const int* seq, const int* pos, const long long* slots,
-                  const T* sink, T* out, int n, float scale, int window, MbLatent L, cudaStream_t s) {
-  if (L.rank <= 128) return attend_rl<T, 4>(q, cache, bt, mb_, bs, seq, pos, slots, sink, out, n, scale, window, L, s);
-  if (L.rank <= 256) return attend_rl<T, 8>(q, cache, bt, mb_, bs, seq, pos, slots, sink, out, n, scale, window, L, s);
-  if (L.rank <= 512) return attend_rl<T, 16>(q, cache, bt, mb_, bs, seq, pos, slots, sink, out, n, scale, window, L, s);
-  if (L.rank <= 1024) return attend_rl<T, 32>(q, cache, bt, mb_, bs, seq, pos, slots, sink, out, n, scale, window, L, s);
-  return -3;
 }
 
 }  // namespace mx
@@ -275,10 +163,17 @@ extern "C" int mb_head_linear(const void* x, long long x_t, long long x_h, const
                          N, K, s));
 }
 
+// the absorbed form on the any-size kernel: one "key head" whose keys are the cached rows and whose values are their latent part
 extern "C" int mb_latent_attend(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size,
                                 const int* token_seq, const int* positions, const long long* slots, const void* sink, void* out, int T,
                                 float scale, int window, MbLatent L, int f32, cudaStream_t s) {
-  if (T <= 0) return 0;
-  MB_BY_TYPE(attend(reinterpret_cast<const E*>(q), reinterpret_cast<const E*>(cache), block_table, max_blocks, block_size, token_seq, positions,
-                    slots, reinterpret_cast<const E*>(sink), reinterpret_cast<E*>(out), T, scale, window, L, s));
+  MbAttend a{};
+  a.heads = a.group = L.heads;
+  a.dk = L.pitch; a.dv = L.rank;
+  a.q_head = L.pitch; a.q_row = static_cast<long long>(L.heads) * L.pitch;
+  a.k_row = a.v_row = L.pitch;
+  a.o_row = static_cast<long long>(L.heads) * L.rank;
+  a.window = window;
+  a.scale = scale;
+  return mb_paged_attend(q, cache, cache, block_table, max_blocks, block_size, token_seq, positions, slots, sink, out, T, a, f32, s);
 }

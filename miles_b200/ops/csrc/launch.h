@@ -31,7 +31,7 @@ int mb_gemm_small_grouped(const void* X, const void* W, void* C, int rows, int N
 int mb_gemv(const void* x, const void* residual, const void* norm_w, float eps, const void* W, const void* bias, void* y, long long ldy,
             int out_fp32, void* res_out, void* xn_out, int M, int N, int K, int static_w, cudaStream_t s);
 int mb_moe_gemv(const void* x, const void* w13, const void* w2, const int* topk_idx, const float* topk_w, void* act, void* out, int T, int k,
-                int E, int expert_offset, int H, int F, cudaStream_t s);
+                int E, int expert_offset, int H, int F, float limit, float alpha, cudaStream_t s);
 int mb_gemm_bf16_grouped_wgrad(const void* dY, const void* X, void* dW, int M_pad, int N, int K, int num_experts,
                                const int* seg_offsets, int out_fp32, int accumulate, int force_bn, int* error_flag,
                                cudaStream_t stream);
@@ -206,16 +206,77 @@ int mb_multi_copy2d(const long long* table, const long long* prefix, int n, long
 int mb_multi_mxfp8(const long long* table, const long long* prefix, int n, long long total_chunks, int qdq, cudaStream_t s);
 
 // ---- mixers.cu (layer-by-layer decoders; f32: tensors of the model's dtype are float instead of bf16) ----
+// xb (the copy in the model's dtype) may be null
 int mb_bigram_embedding(const int* tok, const int* prev, const void* embed, const void* table, long long buckets, long long mul_prev,
                         long long mul_cur, float* x, void* xb, int T, int D, int f32, cudaStream_t s);
 int mb_output_norm(float* x, const void* y, const void* nw, const void* ls, const void* fw, void* xb, int T, int D, float eps, int f32,
                    cudaStream_t s);
-int mb_clamped_glu(const void* in, void* out, long long T, int F, float limit, float alpha, int f32, cudaStream_t s);
+// rows (optional, device): rows in use
+int mb_clamped_glu(const void* in, long long ld_in, void* out, long long ld_out, long long T, int F, float limit, float alpha, const int* rows,
+                   int f32, cudaStream_t s);
+// s = x + y1 + y2 + Σ_j weights[t, j]·rows[dst[t, j]] + extra → to; h = rmsnorm(s)·nw (every pointer but x may be null)
+typedef struct {
+  const float* x;
+  float* to;
+  const void *y1, *y2, *rows;
+  const float* weights;
+  const int* dst;
+  const float* extra;
+  const void* nw;
+  void* h;
+  int T, D, k;
+  float eps;
+} MbSumNorm;
+int mb_sum_norm(MbSumNorm p, int f32, cudaStream_t s);
 int mb_gated_norm(const void* o, const void* w, const void* gate, long long gate_ld, void* out, int T, int C, float eps, int f32,
                   cudaStream_t s);
 // gemv.cu: output norm + layer scale + fp32 residual in front of a projection of ≤ 16 rows
 int mb_gemv_output_norm(const float* x, const void* y, const void* norm_w, const void* scale_w, float eps, const void* W, void* out,
                         long long ldo, float* x_out, int M, int N, int K, int static_w, cudaStream_t s);
+// gemv.cu: sum of an fp32 residual and up to two sublayer outputs, its norm, and up to two products of it, for ≤ 16 rows.  x32 null: plain
+// products of x [M, K].  W2 [N2, K] gives fp32 y2 (+ bias2).
+int mb_gemv_sum_norm(const float* x32, const void* y1, const void* y2, const float* extra, const void* x, const void* norm_w, float eps,
+                     const void* W, void* y, long long ldy, const void* W2, const void* bias2, float* out2, float* x_out, void* xn_out, int M,
+                     int N, int N2, int K, int static_w, cudaStream_t s);
+// ---- paged_attend.cu ----
+typedef struct {
+  int heads, group, dk, dv;                  // query head h uses key head h / group
+  long long q_row, q_head, k_row, k_head, v_row, v_head, o_row;   // strides in elements: token (slot) and head
+  int window, keep;                          // keys a token sees (0: all), first keys that stay visible
+  float scale;
+} MbAttend;
+int mb_paged_attend(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size,
+                    const int* token_seq, const int* positions, const long long* slots, const void* sink, void* out, int T, MbAttend A,
+                    int f32, cudaStream_t s);
+// ---- window_prep.cu ----
+typedef struct {
+  int heads, kv_heads, dim, vdim, rot, window, keep, q_pitch;   // q_pitch: elements per head of the prepared queries (zero-padded)
+} MbWindow;
+typedef struct {                             // what reads the same projection beside the attention (null: nothing)
+  const float* logits;
+  float* weights;
+  int* index;
+  int experts, top;
+  const void* glu_in;
+  void* glu_out;
+  long long glu_ld_in, glu_ld_out;
+  int ff;
+  float limit, alpha;
+} MbAside;
+int mb_window_prep(const void* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
+                   const void* q_norm, const void* k_norm, float eps, void* kc, void* vc, void* q, int T, MbWindow L, MbAside a, int f32,
+                   cudaStream_t s);
+// ---- window_decode.cu (bf16 tensor cores, splits joined inside a cluster) ----
+int mb_window_decode(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size, const int* token_seq,
+                     const int* positions, const long long* slots, const void* sink, void* out, long long o_row, int T, float scale, int splits,
+                     MbWindow L, cudaStream_t s);
+// ---- attention_window_tc.cu (tcgen05, keys and values straight from the pages) ----
+int mb_window_prefill(const void* q, const void* kc, const void* vc, void* o, long long o_row, const void* sink, const int* cu_q,
+                      const int* positions, const int* block_table, int max_blocks, int block_size, int num_blocks, int n_seq, int max_q,
+                      int t_long, float scale, MbWindow L, int* error_flag, cudaStream_t s);
+// ---- experts_any.cu ----
+int mb_experts_any(const void* x, const void* w13, const void* w2, const int* index, const float* weights, void* act, void* out, int T, int k,
+                   int E, int H, int F, float limit, float alpha, int f32, cudaStream_t s);
 // ---- latent_attn.cu ----
 typedef struct {
   int heads, dim, rot, vdim, rank, rank_p, pitch;   // a cached row: [rank, 0 … rank_p, rot, 0 … pitch)

@@ -1,5 +1,6 @@
 // Row-wise kernels of the layer-by-layer decoders: hashed-bigram embedding, output norm + layer scale + fp32 residual (with the
-// model's final norm fused into the last one), clamped gated activation, gated norm over all heads of a mixer.
+// model's final norm fused into the last one), sum of fp32 residual and sublayer outputs (experts' rows gathered and weighted on the
+// way) with the next norm, clamped gated activation, gated norm over all heads of a mixer.
 // fp32 math; activations in the model's dtype T (bf16, or float for 32-bit runs).
 #include <type_traits>
 
@@ -35,7 +36,7 @@ __global__ void __launch_bounds__(128) bigram_embed_kernel(const int* __restrict
       for (int j = 0; j < V; ++j) a[j] += b[j];
     }
     store_n<V>(x + t * D + i, a);
-    store_n<V>(xb + t * D + i, a);
+    if (xb != nullptr) store_n<V>(xb + t * D + i, a);
   }
 }
 
@@ -84,23 +85,96 @@ __global__ void __launch_bounds__(kRow) output_norm_kernel(float* __restrict__ x
 }
 
 template <typename T, int V>
-__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ in, T* __restrict__ out, long long n_vec, int F, float limit,
-                                                          float alpha) {
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ in, long long ld_in, T* __restrict__ out, long long ld_out,
+                                                          long long n, int F, float limit, float alpha, const int* __restrict__ rows) {
   pdl_trigger();
   pdl_wait();
   const int per = F / V;
-  for (long long v = blockIdx.x * 256ll + threadIdx.x; v < n_vec; v += gridDim.x * 256ll) {
+  if (rows != nullptr) n = min(n, static_cast<long long>(*rows));
+  for (long long v = blockIdx.x * 256ll + threadIdx.x; v < n * per; v += gridDim.x * 256ll) {
     const long long t = v / per;
     const int i = static_cast<int>(v - t * per) * V;
     float g[V], u[V];
-    load_n<V>(in + t * 2 * F + i, g);
-    load_n<V>(in + t * 2 * F + F + i, u);
+    load_n<V>(in + t * ld_in + i, g);
+    load_n<V>(in + t * ld_in + F + i, u);
 #pragma unroll
-    for (int j = 0; j < V; ++j) {
-      const float a = fminf(g[j], limit), b = fminf(fmaxf(u[j], -limit), limit);
-      g[j] = a * sigmoid_t<T>(alpha * a) * (b + 1.f);
+    for (int j = 0; j < V; ++j) g[j] = clamped_glu_t<T>(g[j], u[j], limit, alpha);
+    store_n<V>(out + t * ld_out + i, g);
+  }
+}
+
+// One CTA per token; the sum waits in shared memory for its norm.  Addends: see MbSumNorm.
+static constexpr int kMaxTop = 64;
+template <typename T, int V>
+__global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float sh[kRow / 32], s_w[kMaxTop];
+  __shared__ int s_dst[kMaxTop];
+  pdl_trigger();
+  pdl_wait();
+  const long long t = blockIdx.x, base = t * p.D;
+  const T* y1 = reinterpret_cast<const T*>(p.y1);
+  const T* y2 = reinterpret_cast<const T*>(p.y2);
+  const T* rows = reinterpret_cast<const T*>(p.rows);
+  const T* nw = reinterpret_cast<const T*>(p.nw);
+  T* h = reinterpret_cast<T*>(p.h);
+  const int k = rows != nullptr ? p.k : 0;
+  for (int j = threadIdx.x; j < k; j += kRow) {
+    const int d = p.dst[t * p.k + j];
+    s_dst[j] = d;
+    s_w[j] = d >= 0 ? p.weights[t * p.k + j] : 0.f;
+  }
+  if (k > 0) __syncthreads();
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < p.D; i += kRow * V) {
+    float r[V], a[V];
+    load_n<V>(p.x + base + i, r);
+    if (y1 != nullptr) {
+      load_n<V>(y1 + base + i, a);
+#pragma unroll
+      for (int j = 0; j < V; ++j) r[j] += a[j];
     }
-    store_n<V>(out + t * F + i, g);
+    if (y2 != nullptr) {
+      load_n<V>(y2 + base + i, a);
+#pragma unroll
+      for (int j = 0; j < V; ++j) r[j] += a[j];
+    }
+    if (k > 0) {
+      float m[V];
+#pragma unroll
+      for (int j = 0; j < V; ++j) m[j] = 0.f;
+#pragma unroll 4
+      for (int c = 0; c < k; ++c) {
+        const int d = s_dst[c];
+        if (d < 0) continue;
+        load_n<V>(rows + static_cast<long long>(d) * p.D + i, a);
+        const float w = s_w[c];
+#pragma unroll
+        for (int j = 0; j < V; ++j) m[j] = fmaf(w, a[j], m[j]);
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) r[j] += m[j];
+    }
+    if (p.extra != nullptr) {
+      load_n<V>(p.extra + base + i, a);
+#pragma unroll
+      for (int j = 0; j < V; ++j) r[j] += a[j];
+    }
+    if (p.to != nullptr) store_n<V>(p.to + base + i, r);
+    if (nw == nullptr) continue;
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += r[j] * r[j];
+    store_n<V>(row + i, r);
+  }
+  if (nw == nullptr) return;
+  const float rstd = rsqrt_exact(__fdiv_rn(block_sum<kRow>(ss, sh), static_cast<float>(p.D)) + p.eps);
+  for (int i = threadIdx.x * V; i < p.D; i += kRow * V) {      // every thread reads back what it wrote itself
+    float r[V], w[V];
+    load_n<V>(row + i, r);
+    load_n<V>(nw + i, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) r[j] = r[j] * rstd * w[j];
+    store_n<V>(h + base + i, r);
   }
 }
 
@@ -166,15 +240,33 @@ extern "C" int mb_output_norm(float* x, const void* y, const void* nw, const voi
   });
 }
 
-extern "C" int mb_clamped_glu(const void* in, void* out, long long T, int F, float limit, float alpha, int f32, cudaStream_t s) {
+extern "C" int mb_clamped_glu(const void* in, long long ld_in, void* out, long long ld_out, long long T, int F, float limit, float alpha,
+                              const int* rows, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
-  return dispatch(f32, F % 8 == 0, [&](auto ty, auto v) {
+  const bool vec = F % 8 == 0 && ld_in % 8 == 0 && ld_out % 8 == 0 && (reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+  return dispatch(f32, vec, [&](auto ty, auto v) {
     using E = decltype(ty);
     constexpr int V = decltype(v)::value;
-    const long long n = T * (F / V);
-    const long long blocks = (n + 255) / 256;
+    const long long blocks = (T * (F / V) + 255) / 256;
     return static_cast<int>(launch_pdl(clamped_glu_kernel<E, V>, dim3(static_cast<unsigned>(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0,
-                                       s, reinterpret_cast<const E*>(in), reinterpret_cast<E*>(out), n, F, limit, alpha));
+                                       s, reinterpret_cast<const E*>(in), ld_in, reinterpret_cast<E*>(out), ld_out, T, F, limit, alpha, rows));
+  });
+}
+
+extern "C" int mb_sum_norm(MbSumNorm p, int f32, cudaStream_t s) {
+  if (p.T <= 0) return 0;
+  if (p.rows != nullptr && p.k > kMaxTop) return -3;
+  const int bytes = p.D * static_cast<int>(sizeof(float));
+  if (bytes > 200 * 1024) return -3;
+  return dispatch(f32, p.D % 8 == 0, [&](auto ty, auto v) {
+    auto kern = sum_norm_kernel<decltype(ty), decltype(v)::value>;
+    static int configured = 48 * 1024;                 // one per instantiation
+    if (bytes > configured) {
+      const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      if (e != cudaSuccess) return static_cast<int>(e);
+      configured = 200 * 1024;
+    }
+    return static_cast<int>(launch_pdl(kern, dim3(p.T), dim3(kRow), bytes, s, p));
   });
 }
 

@@ -105,5 +105,64 @@ __device__ __forceinline__ float block_sum(float v, float* sh) {
   return r;
 }
 
+// cs[0 … half) = cosines, cs[half … 2·half) = sines of position · frequency, times `magnitude`; angles in double precision, so that a
+// position of any size costs no accuracy.  The caller's CTA barrier comes after.
+template <typename T, int THREADS>
+__device__ __forceinline__ void rotary_table(float* cs, int position, const double* __restrict__ freq, int half, float magnitude) {
+  const double pos = position;
+  for (int i = threadIdx.x; i < half; i += THREADS) {
+    double a = pos * freq[i];
+    a -= rint(a * 0.15915494309189535) * 6.283185307179586;      // one turn off per whole turn: |a| ≤ π
+    if constexpr (is_exact<T>::value) {
+      double s, c;
+      sincos(a, &s, &c);
+      cs[i] = static_cast<float>(c * magnitude);
+      cs[half + i] = static_cast<float>(s * magnitude);
+    } else {
+      float s, c;
+      __sincosf(static_cast<float>(a), &s, &c);
+      cs[i] = c * magnitude;
+      cs[half + i] = s * magnitude;
+    }
+  }
+}
+
+// gate · sigmoid(alpha · gate) · (up + 1) with gate ≤ limit and |up| ≤ limit
+template <typename T> __device__ __forceinline__ float clamped_glu_t(float gate, float up, float limit, float alpha) {
+  const float a = fminf(gate, limit), b = fminf(fmaxf(up, -limit), limit);
+  return a * sigmoid_t<T>(alpha * a) * (b + 1.f);
+}
+
+// One warp chooses the K largest of E logits (ties: the lower index) and weighs them by a softmax over the chosen ones.  A row of
+// NaNs leaves index −1, weight 0.
+template <typename T>
+__device__ __forceinline__ void topk_softmax_row(const float* __restrict__ z, int E, int K, float* __restrict__ w, int* __restrict__ idx) {
+  const int lane = threadIdx.x & 31;
+  float last = INFINITY, first = 0.f, sum = 0.f;
+  int last_i = -1;
+  for (int j = 0; j < K; ++j) {
+    float bv = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < E; e += 32) {
+      const float v = z[e];
+      if ((v < last || (v == last && e > last_i)) && (v > bv || (v == bv && e < bi))) { bv = v; bi = e; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+    }
+    if (j == 0) first = bv;
+    const bool found = bi != 0x7fffffff;
+    const float p = found ? exp_t<T>(bv - first) : 0.f;
+    sum += p;
+    if (lane == (j & 31)) { idx[j] = found ? bi : -1; w[j] = p; }
+    last = bv;
+    last_i = bi;
+  }
+  for (int j = lane; j < K; j += 32) w[j] = sum > 0.f ? __fdiv_rn(w[j], sum) : 0.f;      // every lane reads back what it wrote
+}
+
 }  // namespace mx
 }  // namespace mb

@@ -1,0 +1,265 @@
+// Decode attention over a paged cache of keys and values with a sliding window that keeps the first tokens, and a softmax sink.
+//
+// One cluster = (token, key head, up to 8 query heads of its group); its CTAs split the keys the token sees, which are numbered
+// without a gap: first the kept ones, then those of the window.  As in paged_decode.cu the heads of the group are rows of
+// mma.sync.m16n8k16 and tiles of 64 keys are gathered from their pages with cp.async, double buffered, 16 keys per warp.  What differs:
+//   * the eight rows that padded the softmax weights carry their second bf16 part, so that P·V sees 16 bits of mantissa for no
+//     extra instruction; the two halves of the accumulator are added at the end;
+//   * the splits are joined through distributed shared memory, the sink enters there: one launch, no partial results in HBM.
+// Heads narrower than DK / DV are padded with zeros in shared memory.
+#include <cooperative_groups.h>
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "launch.h"
+#include "mma_sync.cuh"
+#include "pdl.cuh"
+
+namespace mb {
+namespace wd {
+
+namespace cg = cooperative_groups;
+using namespace mb::ms;
+using bf16 = __nv_bfloat16;
+static constexpr float kLog2e = 1.4426950408889634f;
+static constexpr int TK = 64;
+
+template <int D>
+__device__ __forceinline__ int toff(int row, int chunk) { return row * D + ((chunk ^ (row & 7)) << 3); }
+
+template <int DK, int DV>
+struct Smem {
+  // the warps' outputs take the place of the key tiles, the split's output that of the value tiles
+  static constexpr int q = 0, k = 16 * DK * 2, v = k + 2 * TK * DK * 2, ml = v + 2 * TK * DV * 2, fml = ml + 64 * 4, total = fml + 16 * 4, o = k, f = v;
+  static_assert(4 * 8 * DV * 4 <= 2 * TK * DK * 2, "the key tiles hold the warps' outputs");
+};
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
+                                                            const int* __restrict__ block_table, int max_blocks, int block_size,
+                                                            const int* __restrict__ token_seq, const int* __restrict__ positions,
+                                                            const long long* __restrict__ slots, const bf16* __restrict__ sink,
+                                                            bf16* __restrict__ out, long long o_row, float scale, MbWindow L) {
+  using S = Smem<DK, DV>;
+  extern __shared__ __align__(128) uint8_t smem[];
+  bf16* sQ = reinterpret_cast<bf16*>(smem + S::q);
+  bf16* sK = reinterpret_cast<bf16*>(smem + S::k);
+  bf16* sV = reinterpret_cast<bf16*>(smem + S::v);
+  float* sM = reinterpret_cast<float*>(smem + S::ml);      // [4][8] maxima, then [4][8] sums
+  float* sL = sM + 32;
+  float* sO = reinterpret_cast<float*>(smem + S::o);       // [4][8][DV]
+  float* fO = reinterpret_cast<float*>(smem + S::f);       // [8][DV]: this split's output …
+  float* fM = reinterpret_cast<float*>(smem + S::fml);     // [8] maxima (times scale·log2 e), [8] sums
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.z, split = blockIdx.x, splits = gridDim.x;
+  const int group = L.heads / L.kv_heads, chunks = (group + 7) / 8;
+  const int hk = blockIdx.y / chunks, h0 = hk * group + (blockIdx.y % chunks) * 8;
+  const int rows = min(8, group - (blockIdx.y % chunks) * 8);
+  if (slots[t] < 0) {                    // padding row of a decode batch (the whole cluster leaves)
+    for (int i = split * 128 + threadIdx.x; i < rows * L.vdim; i += splits * 128)
+      out[t * o_row + static_cast<long long>(h0 + i / L.vdim) * L.vdim + i % L.vdim] = __float2bfloat16(0.f);
+    return;
+  }
+  const int pos = positions[t];
+  const int lo = L.window > 0 ? max(0, pos - L.window + 1) : 0, kept = min(L.keep, lo);
+  const int n_keys = kept + pos + 1 - lo;
+  const int per = ((n_keys + splits - 1) / splits + TK - 1) / TK * TK;   // keys per split, whole tiles
+  const int k_begin = min(split * per, n_keys), k_end = min(n_keys, k_begin + per);
+  const int n_tiles = (k_end - k_begin + TK - 1) / TK;
+  const int* bt = block_table + static_cast<long long>(token_seq != nullptr ? token_seq[t] : t) * max_blocks;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr int kq = DK / 8, kv = DV / 8;
+
+  for (int i = threadIdx.x; i < 16 * kq; i += 128) {
+    const int r = i / kq, c = i % kq;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (r < rows && c * 8 < L.dim) v = *reinterpret_cast<const uint4*>(q + (static_cast<long long>(t) * L.heads + h0 + r) * L.q_pitch + c * 8);
+    *reinterpret_cast<uint4*>(sQ + toff<DK>(r, c)) = v;
+  }
+  // a thread copies one 16-byte column of every (128 / columns)-th row: K and V rows of equal width share the page look-up
+  auto load_tile = [&](int tile, int st) {
+    const int i0 = k_begin + tile * TK;
+    auto slot_of = [&](int r, bool& ok) -> long long {
+      const int i = i0 + r;
+      ok = i < k_end;
+      const int ii = ok ? i : k_begin;
+      const int key = ii < kept ? ii : lo + ii - kept;
+      return static_cast<long long>(bt[key / block_size]) * block_size + key % block_size;
+    };
+    if constexpr (DK == DV) {
+#pragma unroll
+      for (int j = 0; j < TK * kq / 128; ++j) {
+        const int r = (threadIdx.x + j * 128) / kq, c = (threadIdx.x + j * 128) % kq;
+        bool ok;
+        const long long slot = slot_of(r, ok);
+        const bool okk = ok && c * 8 < L.dim, okv = ok && c * 8 < L.vdim;
+        cp_async16(sK + st * TK * DK + toff<DK>(r, c), kc + (slot * L.kv_heads + hk) * L.dim + (okk ? c * 8 : 0), okk);
+        cp_async16(sV + st * TK * DV + toff<DV>(r, c), vc + (slot * L.kv_heads + hk) * L.vdim + (okv ? c * 8 : 0), okv);
+      }
+    } else {
+      for (int i = threadIdx.x; i < TK * kq; i += 128) {
+        const int r = i / kq, c = i % kq;
+        bool ok;
+        const long long slot = slot_of(r, ok);
+        ok = ok && c * 8 < L.dim;
+        cp_async16(sK + st * TK * DK + toff<DK>(r, c), kc + (slot * L.kv_heads + hk) * L.dim + (ok ? c * 8 : 0), ok);
+      }
+      for (int i = threadIdx.x; i < TK * kv; i += 128) {
+        const int r = i / kv, c = i % kv;
+        bool ok;
+        const long long slot = slot_of(r, ok);
+        ok = ok && c * 8 < L.vdim;
+        cp_async16(sV + st * TK * DV + toff<DV>(r, c), vc + (slot * L.kv_heads + hk) * L.vdim + (ok ? c * 8 : 0), ok);
+      }
+    }
+    cp_async_commit();
+  };
+  if (n_tiles > 0) load_tile(0, 0);
+  __syncthreads();
+  uint32_t qa[DK / 16][4];               // query fragments stay in registers
+#pragma unroll
+  for (int ks = 0; ks < DK / 16; ++ks) ldsm_x4(s_addr(sQ + toff<DK>(lane & 15, ks * 2 + (lane >> 4))), qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3]);
+  float o_acc[DV / 8][4];
+#pragma unroll
+  for (int i = 0; i < DV / 8; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
+  float m_i = -INFINITY, l_i = 0.f;      // of row lane / 4
+  const float sl2 = scale * kLog2e;
+
+  for (int tile = 0; tile < n_tiles; ++tile) {
+    const int st = tile & 1;
+    if (tile + 1 < n_tiles) {
+      load_tile(tile + 1, st ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const bf16* tK = sK + st * TK * DK;
+    const bf16* tV = sV + st * TK * DV;
+    const int key0 = k_begin + tile * TK + warp * 16;
+    if (key0 < k_end) {
+      float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+      for (int ks = 0; ks < DK / 16; ++ks) {
+        uint32_t b[4];
+        ldsm_x4(s_addr(tK + toff<DK>(warp * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1))), b[0], b[1], b[2], b[3]);
+        mma16816(s[0], qa[ks], b[0], b[1]);
+        mma16816(s[1], qa[ks], b[2], b[3]);
+      }
+      float mx = -INFINITY;
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          s[nt][e] = key0 + nt * 8 + (lane & 3) * 2 + e < k_end ? s[nt][e] * sl2 : -INFINITY;
+          mx = fmaxf(mx, s[nt][e]);
+        }
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+      mx = fmaxf(m_i, fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2)));
+      const float alpha = exp2f(m_i - mx);            // the first key of the tile is seen: mx is finite
+      m_i = mx;
+      uint32_t pa[4];
+      float rs = 0.f;
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) {
+        const float a = exp2f(s[nt][0] - mx), b = exp2f(s[nt][1] - mx);
+        rs += a + b;
+        const uint32_t hi = pack2(a, b);
+        pa[2 * nt] = hi;                                // rows 0–7: the weights' first part, rows 8–15: what rounding took off it
+        pa[2 * nt + 1] = pack2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
+      }
+      l_i = l_i * alpha + rs;
+#pragma unroll
+      for (int i = 0; i < DV / 8; ++i) { o_acc[i][0] *= alpha; o_acc[i][1] *= alpha; o_acc[i][2] *= alpha; o_acc[i][3] *= alpha; }
+#pragma unroll
+      for (int nc = 0; nc < DV / 16; ++nc) {
+        uint32_t b[4];
+        ldsm_x4_t(s_addr(tV + toff<DV>(warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), nc * 2 + (lane >> 4))), b[0], b[1], b[2], b[3]);
+        mma16816(o_acc[2 * nc], pa, b[0], b[1]);
+        mma16816(o_acc[2 * nc + 1], pa, b[2], b[3]);
+      }
+    }
+    __syncthreads();
+  }
+  l_i += __shfl_xor_sync(0xffffffffu, l_i, 1);
+  l_i += __shfl_xor_sync(0xffffffffu, l_i, 2);
+  const int r = lane >> 2;
+  if ((lane & 3) == 0) { sM[warp * 8 + r] = m_i; sL[warp * 8 + r] = l_i; }
+#pragma unroll
+  for (int i = 0; i < DV / 8; ++i)
+    *reinterpret_cast<float2*>(sO + (warp * 8 + r) * DV + i * 8 + (lane & 3) * 2) = make_float2(o_acc[i][0] + o_acc[i][2], o_acc[i][1] + o_acc[i][3]);
+  __syncthreads();
+  for (int i = threadIdx.x; i < rows * DV; i += 128) {
+    const int g = i / DV, d = i % DV;
+    float mm = -INFINITY, ll = 0.f, oo = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) mm = fmaxf(mm, sM[w * 8 + g]);
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float a = sM[w * 8 + g] == -INFINITY ? 0.f : exp2f(sM[w * 8 + g] - mm);
+      ll += sL[w * 8 + g] * a;
+      oo += sO[(w * 8 + g) * DV + d] * a;
+    }
+    fO[g * DV + d] = oo;
+    if (d == 0) { fM[g] = mm; fM[8 + g] = ll; }
+  }
+  // join the splits: every CTA of the cluster finishes its share of the outputs
+  cg::cluster_group cluster = cg::this_cluster();
+  if (splits > 1) cluster.sync();
+  else __syncthreads();
+  for (int i = split * 128 + threadIdx.x; i < rows * DV; i += splits * 128) {
+    const int g = i / DV, d = i % DV;
+    const float sk = sink != nullptr ? __bfloat162float(sink[h0 + g]) * kLog2e : -INFINITY;
+    float mm = sk, ms[8];
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+      ms[c] = c < splits ? cluster.map_shared_rank(fM, c)[g] : -INFINITY;
+      mm = fmaxf(mm, ms[c]);
+    }
+    float den = sink != nullptr ? exp2f(sk - mm) : 0.f, oo = 0.f;
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+      if (ms[c] == -INFINITY) continue;
+      const float a = exp2f(ms[c] - mm);
+      den = fmaf(cluster.map_shared_rank(fM, c)[8 + g], a, den);
+      oo = fmaf(cluster.map_shared_rank(fO, c)[g * DV + d], a, oo);
+    }
+    if (d < L.vdim) out[t * o_row + static_cast<long long>(h0 + g) * L.vdim + d] = __float2bfloat16(__fdiv_rn(oo, den));
+  }
+  if (splits > 1) cluster.sync();        // the shared memory stays until the others have read it
+}
+
+template <int DK, int DV>
+static int launch(const bf16* q, const bf16* kc, const bf16* vc, const int* bt, int max_blocks, int bs, const int* seq, const int* pos,
+                  const long long* slots, const bf16* sink, bf16* out, long long o_row, int T, float scale, int splits, MbWindow L, cudaStream_t s) {
+  static bool once = false;
+  if (!once) {
+    const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<DK, DV>::total);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    once = true;
+  }
+  const int chunks = (L.heads / L.kv_heads + 7) / 8;
+  return static_cast<int>(launch_pdl_cluster(window_decode_kernel<DK, DV>, dim3(splits, L.kv_heads * chunks, T), dim3(128), splits,
+                                             Smem<DK, DV>::total, s, q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, scale, L));
+}
+
+}  // namespace wd
+}  // namespace mb
+
+using namespace mb;
+
+// q [T, heads, q_pitch], kc [pages·block_size, kv_heads, dim], vc [.., kv_heads, vdim], out rows of o_row elements.  dim, vdim multiples of
+// 8 up to 128, splits ∈ 1 … 8, T ≤ 65535.
+extern "C" int mb_window_decode(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size, const int* token_seq,
+                                const int* positions, const long long* slots, const void* sink, void* out, long long o_row, int T, float scale,
+                                int splits, MbWindow L, cudaStream_t s) {
+  if (T <= 0) return 0;
+  if (L.dim % 8 || L.vdim % 8 || L.q_pitch % 8 || L.dim > 128 || L.vdim > 128 || L.heads % L.kv_heads || splits < 1 || splits > 8 || T > 65535) return -3;
+  using wd::bf16;
+  auto Q = reinterpret_cast<const bf16*>(q), K = reinterpret_cast<const bf16*>(kc), V = reinterpret_cast<const bf16*>(vc), SK = reinterpret_cast<const bf16*>(sink);
+  auto O = reinterpret_cast<bf16*>(out);
+  auto f = L.dim <= 64 ? (L.vdim <= 64 ? wd::launch<64, 64> : wd::launch<64, 128>) : (L.vdim <= 64 ? wd::launch<128, 64> : wd::launch<128, 128>);
+  return f(Q, K, V, block_table, max_blocks, block_size, token_seq, positions, slots, SK, O, o_row, T, scale, splits, L, s);
+}

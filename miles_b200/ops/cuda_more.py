@@ -169,7 +169,7 @@ MOE_GEMV_T = min(8, int(os.environ.get("MILES_MOE_GEMV_T", "8")))
 
 def small_moe_bt(n_pairs: int, num_experts: int, w13, w2) -> int:
     """Row granularity for an inference MoE call: 128 (general path) or a decode-sized tile."""
-    if SMALL_MOE_AVG <= 0 or torch.is_grad_enabled() or w13.shape[1] % 128 or w2.shape[1] % 128:
+    if SMALL_MOE_AVG <= 0 or torch.is_grad_enabled() or w13.shape[1] % 8 or w2.shape[1] % 8:
         return 128
     avg = n_pairs / max(num_experts, 1)
     if avg > SMALL_MOE_AVG:
@@ -181,21 +181,47 @@ def moe_max_rows_pad(n_pairs: int, num_experts: int, pad: int) -> int:
     return (n_pairs + num_experts * (pad - 1) + pad - 1) // pad * pad
 
 
-def experts_forward(x_perm, w13, w2, seg, tile, bt: int = 128):
-    """Grouped expert FFN on expert-sorted rows whose segments are padded to `bt`. Returns (h1 pre-activation, y_perm)."""
+def few_token_experts(x, w13, T: int, k: int) -> bool:
+    """A handful of tokens: two matrix-vector kernels, no sort / gather / combine (gemv.cu).  Both keep their activations in shared
+    memory next to a 64 KB weight ring."""
+    return (x.dtype == BF16 and 0 < T <= MOE_GEMV_T and T * k <= 64 and not torch.is_grad_enabled() and x.shape[1] % 32 == 0
+            and w13.shape[1] % 64 == 0 and 65536 + max(8 * (2 * x.shape[1] + 64), T * k * (w13.shape[1] + 64)) <= 200 * 1024)
+
+
+def sort_by_expert(x, idx, E: int, bt: int, expert_offset: int = 0):
+    """Rows of `x` per (token, choice), sorted by expert, every expert's segment padded to `bt` rows: (rows, segment offsets, expert of
+    each row tile, row of each (token, choice))."""
+    T, k = idx.shape
+    max_rows = moe_max_rows(T * k, E) if bt == 128 else moe_max_rows_pad(T * k, E, bt)
+    seg, tile, row_src, dst_row = C.moe_align(_c(idx.to(torch.int32)).view(-1), E, expert_offset, max_rows, None, bt)
+    x_perm = torch.empty(max_rows, x.shape[1], dtype=x.dtype, device=x.device)
+    publish_limit(LIMIT_MOE_PAIRS, T * k)
+    C.moe_gather(_c(x), x_perm, row_src, seg, k)
+    return x_perm, seg, tile, dst_row
+
+
+def experts_forward(x_perm, w13, w2, seg, tile, bt: int = 128, glu=None):
+    """Grouped expert FFN on expert-sorted rows whose segments are padded to `bt`. Returns (h1 pre-activation, y_perm).  `glu`: (limit,
+    alpha) of a clamped activation instead of SwiGLU (inference)."""
     max_rows, H = x_perm.shape
     E, F2, _ = w13.shape
     h1 = torch.empty(max_rows, F2, dtype=x_perm.dtype, device=x_perm.device)
     act = torch.empty(max_rows, F2 // 2, dtype=x_perm.dtype, device=x_perm.device)
     y_perm = torch.empty(max_rows, H, dtype=x_perm.dtype, device=x_perm.device)
+    def activate():
+        if glu is None:
+            C.swiglu_fwd(h1, act, seg[-1:])
+        else:
+            C.clamped_glu(h1, act, glu[0], glu[1], seg[-1:])
+
     if bt != 128:
         C.gemm_small_grouped(x_perm, w13, h1, max_rows, F2, H, E, tile, seg[-1:], bt)
-        C.swiglu_fwd(h1, act, seg[-1:])
+        activate()
         C.gemm_small_grouped(act, w2, y_perm, max_rows, H, F2 // 2, E, tile, seg[-1:], bt)
         return h1, y_perm
     from . import cuda as _cuda
 
-    if _cuda.MXFP8_LINEAR and H % 128 == 0 and F2 % 256 == 0 and max_rows >= 8 * _cuda.MXFP8_MIN_ROWS:
+    if glu is None and _cuda.MXFP8_LINEAR and H % 128 == 0 and F2 % 256 == 0 and max_rows >= 8 * _cuda.MXFP8_MIN_ROWS:
         # --fp8-recipe mxfp8: the expert GEMMs of the forward run block-scaled (activations quantised per call, expert weights
         # once per call); the backward uses the bf16 grouped GEMMs on the unquantised operands (straight-through), like the
         # dense projections of this recipe
@@ -211,22 +237,15 @@ def experts_forward(x_perm, w13, w2, seg, tile, bt: int = 128):
         extra.gemm_mxfp8_grouped(aq, as_, w2q.view(E, H, F), w2s.view(E, H, F // 32), tile, out=y_perm)
         return h1, y_perm
     C.gemm_grouped(x_perm, w13, h1, max_rows, F2, H, E, tile, False, 0)
-    C.swiglu_fwd(h1, act, seg[-1:])
+    activate()
     C.gemm_grouped(act, w2, y_perm, max_rows, H, F2 // 2, E, tile, False, 0)
     return h1, y_perm
 
 
 def _moe_ffn_small(x, w13, w2, topk_w, topk_idx, expert_offset, bt):
     T, H = x.shape
-    E = w13.shape[0]
     k = topk_idx.shape[1]
-    x = _c(x)
-    idx32 = _c(topk_idx.to(torch.int32)).view(-1)
-    max_rows = moe_max_rows_pad(T * k, E, bt)
-    seg, tile, row_src, dst_row = C.moe_align(idx32, E, expert_offset, max_rows, None, bt)
-    x_perm = torch.empty(max_rows, H, dtype=x.dtype, device=x.device)
-    publish_limit(LIMIT_MOE_PAIRS, x.shape[0] * k)
-    C.moe_gather(x, x_perm, row_src, seg, k)
+    x_perm, seg, tile, dst_row = sort_by_expert(x, topk_idx, w13.shape[0], bt, expert_offset)
     _, y_perm = experts_forward(x_perm, _c(w13), _c(w2), seg, tile, bt)
     out = torch.empty(T, H, dtype=x.dtype, device=x.device)
     C.moe_combine(y_perm, _c(topk_w.float()), dst_row, out, k)
@@ -315,11 +334,7 @@ def moe_ffn(x, w13, w2, topk_w, topk_idx, expert_offset: int = 0):
     if x.dtype != BF16:
         return ref.moe_ffn(x, w13, w2, topk_w, topk_idx)
     T, k = topk_idx.shape
-    if (0 < T <= MOE_GEMV_T and T * k <= 64 and not torch.is_grad_enabled() and x.shape[1] % 32 == 0
-            and w13.shape[1] % 64 == 0
-            # both kernels keep their activations in shared memory next to a 64 KB weight ring
-            and 65536 + max(8 * (2 * x.shape[1] + 64), T * k * (w13.shape[1] + 64)) <= 200 * 1024):
-        # a handful of tokens: two matrix-vector kernels, no sort / gather / combine (gemv.cu)
+    if few_token_experts(x, w13, T, k):
         act = torch.empty(T * k, w13.shape[1] // 2, dtype=x.dtype, device=x.device)
         out = torch.empty_like(x)
         C.moe_gemv(_c(x), _c(w13), _c(w2), _c(topk_idx.to(torch.int32)), _c(topk_w.float()), act, out, int(expert_offset))

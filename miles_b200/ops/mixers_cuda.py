@@ -1,4 +1,5 @@
-"""CUDA execution of the ops in `mixers.py` (inference only): the kernels of mixers.cu, latent_attn.cu and linear_state.cu.
+"""CUDA execution of the ops in `mixers.py` (inference only): the kernels of mixers.cu, latent_*.cu, linear_*.cu, window_*.cu,
+attention_*_tc.cu, paged_attend.cu and experts_any.cu.
 
 Tensors are bf16, or float32 throughout (then every product is a true 32-bit one: the kernels' own fp32 loops, and cuBLAS
 without TF32 for the dense projections, as `ops.linear` does for float32).
@@ -9,6 +10,7 @@ import os
 
 import torch
 
+from . import cuda as K
 from .cuda import BF16, C, GEMV_MAX_N, gemv_ok
 
 
@@ -16,10 +18,10 @@ def _c(x):
     return x if x.is_contiguous() else x.contiguous()
 
 
-def bigram_embedding(tokens, prev, embed, table, spec):
+def bigram_embedding(tokens, prev, embed, table, spec, want_copy=True):
     T, D = tokens.numel(), embed.shape[1]
     x = torch.empty(T, D, dtype=torch.float32, device=embed.device)
-    xb = torch.empty(T, D, dtype=embed.dtype, device=embed.device)
+    xb = torch.empty(T, D, dtype=embed.dtype, device=embed.device) if want_copy else None
     buckets, mp, mc = spec if table is not None else (0, 0, 0)
     C.bigram_embedding(tokens.to(torch.int32), prev, embed, table, buckets, mp, mc, x, xb)
     return x, xb
@@ -48,7 +50,7 @@ def output_norm_linear(x, y, nw, ls, eps, w):
 
 def clamped_glu(h, limit, alpha):
     out = torch.empty(h.shape[0], h.shape[1] // 2, dtype=h.dtype, device=h.device)
-    C.clamped_glu(_c(h), out, float(limit), float(alpha))
+    C.clamped_glu(h, out, float(limit), float(alpha))
     return out
 
 
@@ -179,3 +181,118 @@ def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sin
         C.gemm(lat, w_ukv, kv, total, N, lay.rank, lay.pitch, lay.rank, N, False, False, False, None, 0)
         C.latent_prefill(q_full, kv, lat, out, sink, rg.cu_q, cu_k, rg.n_long, max_q, float(scale), int(window), sizes, C.error_flag(proj))
     return out.view(T, H * lay.vdim)
+
+
+# ---- parallel arrangement: sum, norm, projections ---------------------------------------------------------------------
+
+def _split_addends(addends):
+    """(two dense outputs or None, expert-sorted rows or None) for one kernel."""
+    dense = [a.y for a in addends if a.dst is None]
+    rows = [a for a in addends if a.dst is not None]
+    assert len(dense) <= 2 and len(rows) <= 1, "a sum takes two dense outputs and one set of experts' rows"
+    return dense + [None] * (2 - len(dense)), (rows[0] if rows else None)
+
+
+def sum_norm(x, to, addends, extra, nw, eps):
+    (y1, y2), r = _split_addends(addends)
+    h = torch.empty(x.shape, dtype=nw.dtype, device=x.device) if nw is not None else None
+    C.sum_norm(x, to, y1, y2, r.y if r else None, r.weights if r else None, r.dst if r else None, extra, nw, h, float(eps))
+    return h
+
+
+def few_row_sum(x, addends, w) -> bool:
+    return (w.dtype == BF16 and x.shape[0] <= FUSED_NORM_M and w.shape[0] <= GEMV_MAX_N and K._gemv_k_ok(x.shape[0], w.shape[1])
+            and all(a.dst is None for a in addends))
+
+
+def _static(w) -> bool:
+    return bool(w.is_leaf and w.requires_grad)
+
+
+def sum_norm_linear(x, addends, extra, nw, eps, w, w2, b2, want_normed):
+    (y1, y2), _ = _split_addends(addends)
+    T, dev = x.shape[0], x.device
+    proj = torch.empty(T, w.shape[0], dtype=w.dtype, device=dev)
+    logits = torch.empty(T, w2.shape[0], dtype=torch.float32, device=dev) if w2 is not None else None
+    x_new = torch.empty_like(x) if addends or extra is not None else None
+    h = torch.empty(x.shape, dtype=w.dtype, device=dev) if want_normed else None
+    C.gemv_sum_norm(x, y1, y2, extra, None, nw, float(eps), w, proj, w2, b2, logits, x_new, h, _static(w))
+    return h, proj, logits, x if x_new is None else x_new
+
+
+def projections(h, w, w2, b2):
+    if h.dtype != BF16:
+        logits = None if w2 is None else torch.addmm(b2, h, w2.t())
+        return torch.nn.functional.linear(h, w), logits
+    T, E = h.shape[0], w2.shape[0] if w2 is not None else 0
+    if w2 is not None and T <= K.GEMV_M and w.shape[0] <= GEMV_MAX_N and gemv_ok(h, w):
+        proj = torch.empty(T, w.shape[0], dtype=BF16, device=h.device)
+        logits = torch.empty(T, E, dtype=torch.float32, device=h.device)
+        C.gemv_sum_norm(None, None, None, None, h, None, 0.0, w, proj, w2, b2, logits, None, None, _static(w))
+        return proj, logits
+    return K.gemm_nt(h, w), None if w2 is None else K.gemm_nt(h, w2, bias=b2, out_dtype=torch.float32)
+
+
+# ---- windowed grouped-query attention ---------------------------------------------------------------------------------
+
+def _window_ok(lay, dt) -> bool:
+    """Sizes the tensor-core kernels take; anything else runs paged_attend.cu."""
+    return dt == BF16 and lay.dim % 8 == 0 and lay.vdim % 8 == 0 and lay.dim <= 128 and lay.vdim <= 128
+
+
+def window_splits(tokens: int, lay) -> int:
+    """CTAs of a cluster that share the keys of one (token, key head): enough for the SMs, at most one per tile of 64 keys."""
+    ctas = tokens * lay.kv_heads * -(-(lay.heads // lay.kv_heads) // 8)
+    tiles = -(-(lay.window + lay.keep) // 64) if lay.window else 64
+    return max(1, min(8, tiles, 444 // ctas))
+
+
+def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps, aside):
+    T, rg, dt, dev = proj.shape[0], meta.ragged, proj.dtype, proj.device
+    fast = _window_ok(lay, dt) and out.stride(0) % 8 == 0
+    pitch = -(-lay.dim // 64) * 64 if fast else lay.dim
+    sizes = [lay.heads, lay.kv_heads, lay.dim, lay.vdim, lay.rot, lay.window, lay.keep, pitch]
+    q = torch.empty(T, lay.heads, pitch, dtype=dt, device=dev)
+    a = aside
+    logits = a.logits if a is not None else None
+    if logits is not None:
+        a.weights = torch.empty(T, a.top, dtype=torch.float32, device=dev)
+        a.index = torch.empty(T, a.top, dtype=torch.int32, device=dev)
+    C.window_prep(proj, meta.positions, meta.slot_mapping, freq, float(magnitude), q_norm, k_norm, float(eps), kc, vc, q, sizes, logits,
+                  a.weights if logits is not None else None, a.index if logits is not None else None, a.glu_in if a is not None else None,
+                  a.glu_out if a is not None else None, float(a.limit) if a is not None else 0.0, float(a.alpha) if a is not None else 0.0)
+    t_long = rg.t_long if fast and scale > 0 and kc.shape[1] % 8 == 0 and lay.heads // lay.kv_heads <= 128 else 0
+    if t_long:
+        C.window_prefill(q, kc, vc, out, sink, rg.cu_q, meta.positions, meta.block_table, rg.n_long, max(rg.q_lens[: rg.n_long]), t_long,
+                         float(scale), sizes, C.error_flag(proj))
+    if T > t_long:
+        seq = rg.token_seq[t_long:] if rg.token_seq is not None else None
+        args = (q[t_long:], kc, vc, meta.block_table, seq, meta.positions[t_long:], meta.slot_mapping[t_long:], sink, out[t_long:], float(scale))
+        if fast:
+            C.window_decode(*args, window_splits(T - t_long, lay), sizes)
+        else:
+            C.window_attend(*args, sizes)
+
+
+# ---- routed experts ---------------------------------------------------------------------------------------------------
+
+def routed_experts(h, w13, w2, weights, index, limit, alpha):
+    from . import cuda_more as M
+    from .mixers import Addend
+
+    T, k = index.shape
+    E, F2, D = w13.shape
+    glu = (float(limit), float(alpha))
+    if M.few_token_experts(h, w13, T, k):
+        act = torch.empty(T * k, F2 // 2, dtype=BF16, device=h.device)
+        out = torch.empty_like(h)
+        C.moe_gemv(h, w13, w2, index, weights, act, out, 0, *glu)
+        return Addend(out)
+    if h.dtype == BF16 and D % 8 == 0 and F2 % 16 == 0 and k <= 64 and E <= 2048:
+        bt = M.small_moe_bt(T * k, E, w13, w2)
+        x_perm, seg, tile, dst = M.sort_by_expert(h, index, E, bt)
+        return Addend(M.experts_forward(x_perm, w13, w2, seg, tile, bt, glu)[1], weights, dst)
+    act = torch.empty(T * k, F2 // 2, dtype=h.dtype, device=h.device)
+    out = torch.empty_like(h)
+    C.experts_any(h, w13, w2, index, weights, act, out, *glu)
+    return Addend(out)
