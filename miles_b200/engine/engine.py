@@ -788,7 +788,7 @@ class Engine:
             chunkable = piece is not None and lead is None and r.logprob_start_len < 0 and not self.stateless
             if chunkable:
                 take = min(new_tokens, piece, room) if batch else min(new_tokens, piece)
-                if take < new_tokens and take < bs:
+                if batch and take < new_tokens and take < bs:
                     break                              # not worth a piece smaller than a block: next step
             else:
                 take = new_tokens
@@ -1172,8 +1172,9 @@ class Engine:
         if self.ragged:
             for r in reqs:
                 r.chunk = (r.num_tokens - 1, r.num_tokens)
-            hidden, _, _ = self._forward_pieces(reqs)
+            hidden, _, _ = self._forward_pieces(reqs, record)
             self.stats["decode_tokens"] += len(reqs)
+            self._keep_routing(reqs, record)
             self._sample_and_append(reqs, self.model.logits(hidden))
             self.running = [r for r in reqs if not r.finished]
             return
@@ -1189,13 +1190,18 @@ class Engine:
         hidden = self.ps.sp_gather(hidden)
         logits = self.model.logits(hidden)
         self.stats["decode_tokens"] += len(toks)
-        if record is not None:
-            rec = torch.stack(record, dim=1).cpu().numpy().astype(np.int32)
-            for i, r in enumerate(reqs):
-                if r.return_routed_experts:
-                    r.routed.append(rec[i:i + 1])
+        self._keep_routing(reqs, record)
         self._sample_and_append(reqs, logits)
         self.running = [r for r in reqs if not r.finished]
+
+    def _keep_routing(self, reqs: list[Request], record):
+        """The experts a decode step chose (one token per request, in order)."""
+        if not record:
+            return
+        rec = torch.stack(record, dim=1).cpu().numpy().astype(np.int32)
+        for i, r in enumerate(reqs):
+            if r.return_routed_experts:
+                r.routed.append(rec[i:i + 1])
 
     def _run_decode_static(self):
         """CUDA path: static buffers + (optionally) a CUDA graph per batch bucket; see `decode_runner`."""

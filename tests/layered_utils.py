@@ -1,4 +1,4 @@
-"""Helpers of the Nopelorn tests: engines over random weights, feeding schedules, op-level batches on shuffled pages."""
+"""Helpers of the layer-by-layer decoders' tests: engines over random weights, feeding schedules, op-level batches on shuffled pages."""
 from __future__ import annotations
 
 import torch
@@ -6,12 +6,13 @@ import torch
 import plain_nopelorn as plain
 from miles_b200.engine.engine import Engine
 from miles_b200.models import nopelorn
+from miles_b200.models.config import ModelConfig
 from miles_b200.models.convert import load_named_into_model
 from miles_b200.models.qwen3 import SHORT_Q, ForwardMeta, RaggedBatch
 
 
 def engine_for(cfg: dict, weights, device="cpu", dtype=torch.float32, blocks=24, block_size=16, slots=4, context=None, **kw) -> Engine:
-    c = nopelorn.from_config(cfg)
+    c = ModelConfig.from_hf_config(cfg)
     e = Engine(c, device=device, dtype=dtype, num_blocks=blocks, block_size=block_size, max_running_requests=slots,
                max_context_len=context or blocks * block_size, **kw)
     loaded = load_named_into_model(e.model, list(weights.items()), c, e.ps)
@@ -67,11 +68,41 @@ def feed_together(engine: Engine, schedule, sequences) -> dict:
     return {n: torch.cat(r) for n, r in rows.items()}
 
 
-def rel(got: torch.Tensor, want: torch.Tensor) -> float:
-    """Largest error of a row, relative to the rows' root mean square (means taken off)."""
+def random_schedule(lengths: dict, seed: int, together: int = 3) -> list:
+    """Steps for `feed_together`: up to `together` requests at a time, pieces of some beside single tokens of others, now and then one
+    left out."""
+    g = torch.Generator().manual_seed(seed)
+    left, schedule, order = dict(lengths), [], list(lengths)
+    live: list[str] = []
+    while left:
+        while len(live) < together and any(n not in live for n in left):
+            live.append(next(n for n in order if n in left and n not in live))
+        step = []
+        for n in live:
+            if torch.rand((), generator=g) < 0.85:
+                k = int([1, 1, 2, 3, 9, 17, 40][int(torch.randint(0, 7, (), generator=g))])
+                step.append((n, min(k, left[n])))
+        if not step:
+            continue
+        for n, k in step:
+            left[n] -= k
+            if not left[n]:
+                del left[n]
+                live.remove(n)
+        schedule.append(step)
+    return schedule
+
+
+def row_errors(got: torch.Tensor, want: torch.Tensor) -> torch.Tensor:
+    """Every row's error relative to the rows' root mean square (means taken off)."""
     got, want = got.double().cpu(), want.double().cpu()
     d = (got - want) - (got - want).mean(-1, keepdim=True)
-    return float(d.square().mean(-1).sqrt().max() / want.square().mean().sqrt())
+    return d.square().mean(-1).sqrt() / want.square().mean().sqrt()
+
+
+def rel(got: torch.Tensor, want: torch.Tensor) -> float:
+    """Largest of `row_errors`."""
+    return float(row_errors(got, want).max())
 
 
 # ---- op level: several sequences on shuffled pages, any pieces ---------------------------------------------------------------

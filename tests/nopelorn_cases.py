@@ -51,25 +51,7 @@ def mixed_batches(engine_kw, cfg, lengths, tol, seed=3):
     W = plain.make_weights(cfg, seed)
     seqs = {f"r{i}": U.tokens_for(cfg, n, 10 + i) for i, n in enumerate(lengths)}
     e = U.engine_for(cfg, W, **engine_kw)
-    g = torch.Generator().manual_seed(seed)
-    left, schedule, order = {n: len(s) for n, s in seqs.items()}, [], list(seqs)
-    live: list[str] = []
-    while left:
-        while len(live) < 3 and any(n not in live for n in left):
-            live.append(next(n for n in order if n in left and n not in live))
-        step = []
-        for n in live:
-            if torch.rand((), generator=g) < 0.85:
-                k = int([1, 1, 2, 3, 9, 17, 40][int(torch.randint(0, 7, (), generator=g))])
-                step.append((n, min(k, left[n])))
-        if not step:
-            continue
-        for n, k in step:
-            left[n] -= k
-            if not left[n]:
-                del left[n]
-                live.remove(n)
-        schedule.append(step)
+    schedule = U.random_schedule({n: len(s) for n, s in seqs.items()}, seed)
     out = U.feed_together(e, schedule, seqs)
     for n, s in seqs.items():
         want = plain.run(cfg, W, s)
