@@ -66,9 +66,9 @@ def parse():
     p.add_argument("--quiet", action="store_true")
     p.add_argument("--layered", action="store_true",
                    help="instead of the headline workload: prefill, decode and kernel rooflines of a layer-by-layer decoder beside a "
-                        "grouped-query model of equal size (one GPU, JSON lines; --layers, default 12)")
+                        "grouped-query model of equal size (one GPU, JSON lines; --layers, default 12 layer runs)")
     p.add_argument("--layered-model", default="nopelorn-4B-shape")
-    p.add_argument("--layered-baseline", default="qwen3-4B")
+    p.add_argument("--layered-baseline", default=None, help="default: qwen3-4B, or qwen3-30B-A3B for a model with routed experts")
     return p.parse_args()
 
 

@@ -1,6 +1,9 @@
 """Prefill and decode of a layer-by-layer decoder beside the closest grouped-query model of equal width, depth and feed-forward.
 
-    python bench.py --layered [--layered-model nopelorn-4B-shape] [--layered-baseline qwen3-4B] [--layers N]
+    python bench.py --layered [--layered-model nopelorn-4B-shape | ronupel-30B-A3B-shape] [--layered-baseline NAME] [--layers N]
+
+The baseline is qwen3-4B for a dense model and qwen3-30B-A3B for one with routed experts, with as many layers as the layered model has
+layer runs.
 
 Random weights, synthetic tokens.  `throughput`: whole models through the engine (device-timed forwards and decode graphs).
 `kernels`: the mixers' kernels one by one at the same sizes with their distance from the measured roofline, next to the kernels
@@ -152,27 +155,34 @@ def _ragged(lens, bs: int = 64):
                            q_lens=[n for _, n in lens], seq_lens=[s + n for s, n in lens], n_long=n_long, t_long=cu[n_long])), nb
 
 
+class _Rows:
+    """Timed kernels: device time and fraction of the roofline, max(bytes ÷ copy bandwidth, FLOPs ÷ GEMM rate) ÷ time."""
+
+    def __init__(self):
+        self.bw, self.fl, self.which = peaks()
+        self.tm = _Timer()
+        self.rows: list[dict] = []
+
+    def add(self, name, like, shape, fn, nbytes, flops=0.0):
+        ms = self.tm.ms(fn)
+        ideal = max(nbytes / self.bw, flops / self.fl) * 1e3
+        self.rows.append({"kernel": name, "like": like, "shape": shape, "us": round(ms * 1e3, 1), "GB/s": round(nbytes / ms / 1e6),
+                          "TFLOP/s": round(flops / ms / 1e9, 1), "of_roofline": round(ideal / ms, 3), "peaks": self.which})
+
+
+def _randn(*shape, dtype=torch.bfloat16):
+    return torch.randn(*shape, device="cuda").to(dtype)
+
+
 @torch.no_grad()
-def kernels(cfg, base) -> list[dict]:
-    """Device time and fraction of the roofline of each kernel: max(bytes ÷ copy bandwidth, FLOPs ÷ GEMM rate) ÷ time."""
+def latent_kernels(cfg, base) -> list[dict]:
     from ..models.layered import LatentSpec, LinearStateSpec
     from ..ops import cuda as K
     from ..ops import mixers as MX
     from ..ops import mixers_cuda as MC
 
-    bw, fl, which = peaks()
-    tm = _Timer()
-    rows: list[dict] = []
-
-    def add(name, like, shape, fn, nbytes, flops=0.0):
-        ms = tm.ms(fn)
-        ideal = max(nbytes / bw, flops / fl) * 1e3
-        rows.append({"kernel": name, "like": like, "shape": shape, "us": round(ms * 1e3, 1), "GB/s": round(nbytes / ms / 1e6),
-                     "TFLOP/s": round(flops / ms / 1e9, 1), "of_roofline": round(ideal / ms, 3), "peaks": which})
-
-    def t(*shape, dtype=torch.bfloat16):
-        return torch.randn(*shape, device="cuda").to(dtype)
-
+    out = _Rows()
+    add, t, rows = out.add, _randn, out.rows
     D = cfg.hidden_size
     lat = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, LatentSpec))
     lin = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, LinearStateSpec))
@@ -263,18 +273,124 @@ def kernels(cfg, base) -> list[dict]:
     return rows
 
 
+@torch.no_grad()
+def attention_kernels(cfg, base) -> list[dict]:
+    """Windowed grouped-query attention, routed clamped experts and the fused sums beside the grouped-query mixture's kernels."""
+    from dataclasses import replace
+
+    from ..ops import cuda as K
+    from ..ops import mixers as MX
+    from ..ops import mixers_cuda as MC
+
+    out = _Rows()
+    add, t = out.add, _randn
+    spec = cfg.layer_specs[0]
+    m, f, D = spec.mixer, spec.mlp, cfg.hidden_size
+    lay = MX.AttentionLayout(m.heads, m.kv_heads, m.dim, m.vdim, m.rotary.dims, m.window, m.keep_first)
+    hq, hk, d = base.num_heads, base.num_kv_heads, base.head_dim
+    H, G, err, sink = m.heads, m.kv_heads, K.C.error_flag(torch.empty(0, device="cuda")), t(m.heads)
+
+    def sizes(l):
+        return [l.heads, l.kv_heads, l.dim, l.vdim, l.rot, l.window, l.keep, -(-l.dim // 64) * 64]
+
+    for n, length in ((1, 8192), (8, 1024), (1, 1024)):
+        T = n * length
+        meta, nb = _ragged([(0, length)] * n)
+        q, kc, vc, o = t(T, H, -(-m.dim // 64) * 64), t(nb, 64, G, m.dim), t(nb, 64, G, m.vdim), t(T, H * m.vdim)
+        for l in (lay, replace(lay, window=0, keep=0)):
+            if l.window >= length:
+                continue
+            pairs = n * sum(min(i + 1, l.window + min(l.keep, max(0, i + 1 - l.window))) if l.window else i + 1 for i in range(length))
+            add("window_prefill (tcgen05, pages, sink)", "flash_fwd_tc", f"{n}x{length} window {l.window} + {l.keep}",
+                lambda: K.C.window_prefill(q, kc, vc, o, sink, meta.ragged.cu_q, meta.positions, meta.block_table, n, length, T, m.scale, sizes(l), err),
+                2 * (q.numel() + kc.numel() + vc.numel() + o.numel()), 2.0 * pairs * H * (m.dim + m.vdim))
+        q2, k2, v2 = t(T, hq, d), t(T, hk, d), t(T, hk, d)
+        add("flash_fwd_tc", "", f"{n}x{length}", lambda: K.attention_varlen(q2, k2, v2, meta.ragged.cu_q, length), 2 * (2 * q2.numel() + 2 * k2.numel()),
+            2.0 * n * length * (length + 1) / 2 * hq * 2 * d)
+    del q, kc, vc, o, q2, k2, v2
+    for B, ctx in ((1, 4096), (8, 4096), (64, 4096)):
+        meta, nb = _ragged([(ctx - 1, 1)] * B)
+        kc, vc, o = t(nb, 64, G, m.dim), t(nb, 64, G, m.vdim), t(B, H * m.vdim)
+        q = t(B, H, -(-m.dim // 64) * 64)
+        n_keys = m.window + m.keep_first
+        add("window_decode (cluster splits, sink)", "paged_decode", f"{B} rows, {n_keys} keys",
+            lambda: K.C.window_decode(q, kc, vc, meta.block_table, None, meta.positions, meta.slot_mapping, sink, o, m.scale,
+                                      MC.window_splits(B, lay), sizes(lay)),
+            2 * B * (n_keys * G * (m.dim + m.vdim) + H * (m.dim + m.vdim)), 2.0 * B * n_keys * H * (m.dim + m.vdim))
+        kb, vb, q2 = t(nb, 64, hk, d), t(nb, 64, hk, d), t(B, hq, d)
+        L = torch.full((B,), n_keys, dtype=torch.int32, device="cuda")
+        add("paged_decode + merge", "", f"{B} rows, {n_keys} keys", lambda: K.paged_attention(q2, kb, vb, meta.block_table, L),
+            2 * B * (n_keys * 2 * hk * d + 2 * hq * d), 4.0 * B * n_keys * hq * d)
+        del kc, vc, kb, vb
+    freq = torch.tensor(m.rotary.table()[0], dtype=torch.float64, device="cuda")
+    qn, kn, nw, w_in = t(H * m.dim), t(G * m.dim), t(D), torch.nn.Parameter(t(lay.rows + 2 * f.shared.ff, D))
+    router, bias, w_out = torch.nn.Parameter(t(f.experts, D)), t(f.experts), torch.nn.Parameter(t(D, H * m.vdim + f.shared.ff))
+    wqkv, wo = torch.nn.Parameter(t(base.qkv_size, D)), torch.nn.Parameter(t(D, base.q_size))
+    for T in (8, 8192):
+        meta, nb = _ragged([(0, T)] if T > 8 else [(4000, 1)] * T)
+        kc, vc = t(nb, 64, G, m.dim), t(nb, 64, G, m.vdim)
+        proj, q, both = t(T, w_in.shape[0]), t(T, H, -(-m.dim // 64) * 64), t(T, w_out.shape[1])
+        logits, w, idx = t(T, f.experts, dtype=torch.float32), torch.empty(T, f.top, device="cuda"), torch.empty(T, f.top, dtype=torch.int32, device="cuda")
+        add("window_prep (norm, rotate, cache, experts, glu)", "qk_norm_rope_cache", f"{T} rows",
+            lambda: K.C.window_prep(proj, meta.positions, meta.slot_mapping, freq, 1.0, qn, kn, 1e-6, kc, vc, q, sizes(lay), logits, w, idx,
+                                    proj[:, lay.rows:], both[:, H * m.vdim:], 7.0, 1.702),
+            2 * T * (2 * lay.rows + 3 * f.shared.ff) + 4 * T * f.experts)
+        q2, k2, v2, qw = t(T, hq, d), t(T, hk, d), t(T, hk, d), t(d)
+        kb, vb = t(nb, 64, hk, d), t(nb, 64, hk, d)
+        add("qk_norm_rope_cache", "", f"{T} rows", lambda: K.qk_norm_rope_cache(q2, k2, v2, qw, qw, meta.positions, 1e6, 1e-6, kb, vb, meta.slot_mapping),
+            2 * (2 * q2.numel() + 5 * k2.numel()))
+        add("router_topk", "", f"{T} rows", lambda: K.router_topk(logits, f.top), 4 * T * f.experts)
+        x, to, y, r2 = t(T, D, dtype=torch.float32), t(T, D, dtype=torch.float32), t(T, D), t(T, D)
+        add("sum_norm (fp32 residual, one addend)", "add_rmsnorm", f"{T} rows", lambda: MC.sum_norm(x, to, [MX.Addend(y)], None, nw, 1e-6), T * D * 12)
+        add("add_rmsnorm", "", f"{T} rows", lambda: K.add_rmsnorm(y, r2, nw, 1e-6), T * D * 8)
+        if T > 8:
+            bt = 128
+            xp, seg, tile, dst = K.sort_by_expert(y, torch.rand(T, f.experts, device="cuda").topk(f.top).indices.int(), f.experts, bt)
+            a = MX.Addend(t(*xp.shape), w.uniform_(), dst)
+            add("sum_norm (one addend, experts' rows)", "moe_combine + add_rmsnorm", f"{T} rows",
+                lambda: MC.sum_norm(x, to, [MX.Addend(y), a], None, nw, 1e-6), T * D * (12 + 2 * f.top))
+            add("moe_combine + add_rmsnorm", "", f"{T} rows",
+                lambda: (K.C.moe_combine(a.y, a.weights, dst, r2, f.top), K.add_rmsnorm(y, r2, nw, 1e-6)), T * D * (2 * f.top + 2 + 8))
+    for T in (1, 4):
+        x, y, y2, r2 = t(T, D, dtype=torch.float32), t(T, D), t(T, D), t(T, D)
+        add("sum_norm_linear (+ router)", "add_rmsnorm_linear", f"{T} rows",
+            lambda: MC.sum_norm_linear(x, [MX.Addend(y), MX.Addend(y2)], None, nw, 1e-6, w_in, router, bias, True),
+            2 * (w_in.numel() + router.numel()))
+        add("add_rmsnorm_linear", "", f"{T} rows", lambda: K.add_rmsnorm_linear(y, r2, nw, 1e-6, wqkv), 2 * wqkv.numel())
+    for T in (1, 8, 64, 8192):
+        h = t(T, D)
+        w13, w2 = t(f.experts, 2 * f.expert.ff, D), t(f.experts, D, f.expert.ff)
+        idx = torch.rand(T, f.experts, device="cuda").topk(f.top).indices.int()
+        w = torch.rand(T, f.top, device="cuda")
+        used = idx.unique().numel()
+        nbytes, flops = 2.0 * used * 3 * D * f.expert.ff + 4 * T * D, 6.0 * T * f.top * D * f.expert.ff
+        add("routed_experts (clamped; sum left to sum_norm)" if T > 8 else "routed_experts (clamped)", "moe_ffn", f"{T} rows, {used} experts",
+            lambda: MC.routed_experts(h, w13, w2, w, idx, f.expert.limit, f.expert.alpha), nbytes, flops)
+        add("moe_ffn", "", f"{T} rows, {used} experts", lambda: K.moe_ffn(h, w13, w2, w, idx), nbytes, flops)
+        both = t(T, w_out.shape[1])
+        add("output projection (heads and shared expert)", "wo", f"{T} rows", lambda: K.linear(both, w_out), 2.0 * (w_out.numel() + both.numel() + T * D),
+            2.0 * T * w_out.numel())
+        ob = t(T, wo.shape[1])
+        add("wo", "", f"{T} rows", lambda: K.linear(ob, wo), 2.0 * (wo.numel() + ob.numel() + T * D), 2.0 * T * wo.numel())
+    return out.rows
+
+
 def main(a) -> int:
     from ..models.config import get_config
+    from ..ops import build
     from ..ops import cuda as K
 
     torch.cuda.set_device(0)
-    cfg, base = get_config(a.layered_model), get_config(a.layered_baseline)
-    n = a.layers or 12
-    cfg, base = cfg.with_(num_layers=n), base.with_(num_layers=n)
+    cfg = get_config(a.layered_model)
+    moe = cfg.num_moe_layers > 0
+    base = get_config(a.layered_baseline or ("qwen3-30B-A3B" if moe else "qwen3-4B"))
+    cfg = cfg.with_(num_layers=a.layers or (8 if moe else 12))
+    base = base.with_(num_layers=len(cfg.runs()))
     for c in (cfg, base):
         print(json.dumps(throughput(c)), flush=True)
         torch.cuda.empty_cache()
-    for r in kernels(cfg, base):
+    kinds = {"attention": attention_kernels, "latent": latent_kernels}
+    for r in kinds[build.serve_kind(cfg)](cfg, base):
         print(json.dumps(r), flush=True)
     print(json.dumps({"kernel_error_flag": K.check_error_flag()}))
     return 0
