@@ -133,33 +133,56 @@ template <typename T> __device__ __forceinline__ float clamped_glu_t(float gate,
   return a * sigmoid_t<T>(alpha * a) * (b + 1.f);
 }
 
+// A float's bits in an order that integers compare: larger float, larger key.  NaN: 0, below everything.
+__device__ __forceinline__ uint32_t order_key(float v) {
+  const uint32_t b = __float_as_uint(v);
+  if ((b & 0x7fffffffu) > 0x7f800000u) return 0u;
+  if (b == 0x80000000u) return 0x80000000u;                // −0 is 0
+  return (b & 0x80000000u) ? ~b : b | 0x80000000u;
+}
+__device__ __forceinline__ float key_value(uint32_t k) { return __uint_as_float((k & 0x80000000u) ? k & 0x7fffffffu : ~k); }
+
 // One warp chooses the K largest of E logits (ties: the lower index) and weighs them by a softmax over the chosen ones.  A row of
-// NaNs leaves index −1, weight 0.
+// NaNs leaves index −1, weight 0.  Up to 32 · kLocal logits stay in registers; more are read again for every choice.
 template <typename T>
 __device__ __forceinline__ void topk_softmax_row(const float* __restrict__ z, int E, int K, float* __restrict__ w, int* __restrict__ idx) {
+  constexpr int kLocal = 8;
   const int lane = threadIdx.x & 31;
-  float last = INFINITY, first = 0.f, sum = 0.f;
-  int last_i = -1;
-  for (int j = 0; j < K; ++j) {
-    float bv = -INFINITY;
-    int bi = 0x7fffffff;
-    for (int e = lane; e < E; e += 32) {
-      const float v = z[e];
-      if ((v < last || (v == last && e > last_i)) && (v > bv || (v == bv && e < bi))) { bv = v; bi = e; }
-    }
+  const bool local = E <= 32 * kLocal;
+  uint32_t key[kLocal];
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+  for (int i = 0; i < kLocal; ++i) key[i] = i * 32 + lane < E ? order_key(z[i * 32 + lane]) : 0u;
+  uint32_t last = 0xffffffffu;
+  int last_i = -1;
+  float first = 0.f, sum = 0.f;
+  for (int j = 0; j < K; ++j) {
+    uint32_t bk = 0u;
+    int bi = 0x7fffffff;
+    if (local) {
+#pragma unroll
+      for (int i = 0; i < kLocal; ++i)
+        if (key[i] > bk) { bk = key[i]; bi = i * 32 + lane; }      // ascending index: ties keep the lower one
+    } else {
+      for (int e = lane; e < E; e += 32) {
+        const uint32_t k = order_key(z[e]);
+        if ((k < last || (k == last && e > last_i)) && k > bk) { bk = k; bi = e; }
+      }
     }
-    if (j == 0) first = bv;
-    const bool found = bi != 0x7fffffff;
-    const float p = found ? exp_t<T>(bv - first) : 0.f;
+    const uint32_t top = __reduce_max_sync(0xffffffffu, bk);
+    const int at = __reduce_min_sync(0xffffffffu, bk == top ? bi : 0x7fffffff);
+    const bool found = top != 0u;
+    const float v = key_value(top);
+    if (j == 0) first = v;
+    const float p = found ? exp_t<T>(v - first) : 0.f;
     sum += p;
-    if (lane == (j & 31)) { idx[j] = found ? bi : -1; w[j] = p; }
-    last = bv;
-    last_i = bi;
+    if (lane == (j & 31)) { idx[j] = found ? at : -1; w[j] = p; }
+    if (local && (at & 31) == lane) {
+#pragma unroll
+      for (int i = 0; i < kLocal; ++i)
+        if (i * 32 + lane == at) key[i] = 0u;
+    }
+    last = top;
+    last_i = at;
   }
   for (int j = lane; j < K; j += 32) w[j] = sum > 0.f ? __fdiv_rn(w[j], sum) : 0.f;      // every lane reads back what it wrote
 }
