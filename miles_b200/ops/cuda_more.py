@@ -208,6 +208,7 @@ def experts_forward(x_perm, w13, w2, seg, tile, bt: int = 128, glu=None):
     h1 = torch.empty(max_rows, F2, dtype=x_perm.dtype, device=x_perm.device)
     act = torch.empty(max_rows, F2 // 2, dtype=x_perm.dtype, device=x_perm.device)
     y_perm = torch.empty(max_rows, H, dtype=x_perm.dtype, device=x_perm.device)
+
     def activate():
         if glu is None:
             C.swiglu_fwd(h1, act, seg[-1:])
