@@ -332,8 +332,8 @@ def attention_kernels(cfg, base) -> list[dict]:
         proj, q, both = t(T, w_in.shape[0]), t(T, H, -(-m.dim // 64) * 64), t(T, w_out.shape[1])
         logits, w, idx = t(T, f.experts, dtype=torch.float32), torch.empty(T, f.top, device="cuda"), torch.empty(T, f.top, dtype=torch.int32, device="cuda")
         add("window_prep (norm, rotate, cache, experts, glu)", "qk_norm_rope_cache", f"{T} rows",
-            lambda: K.C.window_prep(proj, meta.positions, meta.slot_mapping, freq, 1.0, qn, kn, 1e-6, kc, vc, q, sizes(lay), logits, w, idx,
-                                    proj[:, lay.rows:], both[:, H * m.vdim:], 7.0, 1.702),
+            lambda: K.C.window_prep(proj, meta.positions, meta.slot_mapping, freq, 1.0, qn, kn, 1e-6, kc, vc, q, sizes(lay),
+                                    [logits, w, idx, proj[:, lay.rows:], both[:, H * m.vdim:], None], [7.0, 1.702, 1.0, 1.0], [0, 1, 1]),
             2 * T * (2 * lay.rows + 3 * f.shared.ff) + 4 * T * f.experts)
         q2, k2, v2, qw = t(T, hq, d), t(T, hk, d), t(T, hk, d), t(d)
         kb, vb = t(nb, 64, hk, d), t(nb, 64, hk, d)

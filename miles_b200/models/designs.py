@@ -106,6 +106,6 @@ def rows_of(param: str, parts) -> dict[str, Place]:
     return out
 
 
-from . import nopelorn, ronupel  # noqa: E402  (they use Place and rows_of)
+from . import nopelorn, ronupel, vozirax  # noqa: E402  (they use Place and rows_of)
 
-DESIGNS = {"nopelorn": nopelorn, "ronupel": ronupel}
+DESIGNS = {"nopelorn": nopelorn, "ronupel": ronupel, "vozirax": vozirax}

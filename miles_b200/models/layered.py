@@ -8,11 +8,17 @@ latent ranks or state sizes are a `LayeredConfig`: a tuple of `LayerSpec`s over 
     LinearStateMixer   linear attention with a constant decay per head: fp32 state per sequence, gated norm over all heads
     AttentionMixer     grouped-query attention over a paged cache of keys and values: sliding window that keeps the first tokens,
                        per-head softmax sink, RMS norm over a token's whole query (key) projection, interleaved rotary
-    ClampedGLU         gate and up projections with clamped pre-activations
-    RoutedExperts      clamped experts, the `top` largest of biased fp32 logits, weights by a softmax over the chosen ones
-    LayeredModel       hashed-bigram embedding, fp32 residual stream, layers in one of two arrangements (`LayeredConfig.block`):
+    DifferentialMixer  two softmax maps per head over the same values, the second subtracted with a learned weight; norms per head and
+                       map, a query temperature that grows with the position, a gate per head; may read another layer's keys and values
+    SsmMixer           state-space layer with a scalar decay per head and token: short convolution, fp32 state, gate, norm in parts
+    ClampedGLU         gate and up projections with clamped pre-activations (a limit of infinity: plain silu(gate) · up)
+    RoutedExperts      clamped gated experts or ungated ones with a squared relu; chosen by the `top` largest of biased fp32 logits
+                       with weights by their softmax, or by corrected sigmoid scores among the best groups (`Routing`)
+    LayeredModel       hashed-bigram embedding and / or sinusoidal positions, fp32 residual stream, layers in one of three arrangements
+                       (`LayeredConfig.block`):
                        "output_norm"  mixer, then feed-forward, norms on the sublayers' OUTPUTS with a layer scale
                        "parallel"     one norm in front; mixer and feed-forward read it side by side and are added together
+                       "two_norms"    mixer and feed-forward side by side, each behind a norm and before a layer scale of its own
                        A range of layers may run several times with the same weights (`LoopSpec`), each pass on its own cache.
 
 The blocks run in the engine only (paged latents, state slots; no autograd).  What the design keeps in 32 bits — rotary
@@ -118,23 +124,72 @@ class AttentionSpec:
 
 
 @dataclass(frozen=True)
+class QueryTemperature:
+    """Queries at position p count 1 + coef · ln(⌊(p + 1) / every⌋ + 1) times."""
+
+    coef: float
+    every: float
+
+
+@dataclass(frozen=True)
+class DifferentialSpec:
+    heads: int
+    kv_heads: int
+    dim: int                       # query / key size of one of a head's two maps
+    vdim: int
+    scale: float
+    diff: float                    # what the weight of the second map starts from; outputs count 1 − diff times
+    temperature: QueryTemperature | None = None
+    kv_from: int | None = None     # layer whose cached keys and values this layer reads instead of writing its own
+
+
+@dataclass(frozen=True)
+class SsmSpec:
+    heads: int
+    vdim: int
+    state: int
+    groups: int                    # heads of a group share B and C
+    conv: int                      # columns of the causal convolution
+    norm_groups: int = 1           # parts of the output that are normed by themselves
+
+
+@dataclass(frozen=True)
 class GluSpec:
     ff: int
-    limit: float
+    limit: float = math.inf
     alpha: float = 1.702
+    shift: float = 1.0             # added to the up projection
+
+
+def plain_glu(ff: int) -> GluSpec:
+    """silu(gate) · up"""
+    return GluSpec(ff, math.inf, 1.0, 0.0)
+
+
+@dataclass(frozen=True)
+class ReluSquareSpec:
+    """No gate: down(relu(up)²)."""
+
+    ff: int
 
 
 @dataclass(frozen=True)
 class MoeSpec:
     experts: int
     top: int
-    expert: GluSpec
+    expert: GluSpec | ReluSquareSpec
     shared: GluSpec | None = None  # runs for every token and is added
+    routing: MX.Routing | None = None    # None: softmax over the chosen logits (with a bias per expert)
+
+    @property
+    def up_rows(self) -> int:
+        """Rows of an expert's input projection."""
+        return self.expert.ff * (2 if isinstance(self.expert, GluSpec) else 1)
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentSpec | LinearStateSpec | AttentionSpec
+    mixer: LatentSpec | LinearStateSpec | AttentionSpec | DifferentialSpec | SsmSpec
     mlp: GluSpec | MoeSpec | None
 
     @property
@@ -163,8 +218,11 @@ class BigramSpec:
 class LayeredConfig(FamilyConfig):
     layer_specs: tuple = ()
     bigram: BigramSpec | None = None
-    block: str = "output_norm"         # or "parallel"
+    block: str = "output_norm"         # or "parallel", "two_norms"
     loop: LoopSpec | None = None
+    norm_shift: float = 0.0            # what norm weights are added to ("two_norms")
+    position_base: float = 0.0         # sinusoidal position vectors are added to the embedding (0: none)
+    logit_scale: float = 1.0
 
     def with_(self, **kw) -> "LayeredConfig":
         if "num_layers" in kw:                     # fewer layers: the first ones
@@ -200,7 +258,7 @@ class LayeredConfig(FamilyConfig):
             s = self.layer_specs[i]
             n += sum(math.prod(shape) for shape in layer_shapes(s, self).values())
             if active_only and isinstance(s.mlp, MoeSpec):
-                n -= (s.mlp.experts - s.mlp.top) * 3 * s.mlp.expert.ff * H
+                n -= (s.mlp.experts - s.mlp.top) * (s.mlp.up_rows + s.mlp.expert.ff) * H
         return n
 
     def flops_per_token(self, seq_len: int, backward: bool = True) -> float:
@@ -211,6 +269,10 @@ class LayeredConfig(FamilyConfig):
                 f += 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim) * min(m.window or seq_len, seq_len / 2.0)
             elif isinstance(m, AttentionSpec):
                 f += 2.0 * m.heads * (m.dim + m.vdim) * min(m.window + m.keep_first if m.window else seq_len, seq_len / 2.0)
+            elif isinstance(m, DifferentialSpec):
+                f += 4.0 * m.heads * (m.dim + m.vdim) * seq_len / 2.0
+            elif isinstance(m, SsmSpec):
+                f += 4.0 * m.heads * m.state * m.vdim
             else:
                 f += 4.0 * m.heads * m.dim * m.vdim
         return f * (3.0 if backward else 1.0)
@@ -239,7 +301,24 @@ def mixer_shapes(m, hidden: int) -> dict[str, tuple]:
         if m.sink:
             out["sink"] = (m.heads,)
         return out
+    if isinstance(m, DifferentialSpec):
+        kv = 0 if m.kv_from is not None else m.kv_heads * (2 * m.dim + m.vdim)
+        out = {"w_in": (m.heads * 2 * m.dim + kv + m.heads, hidden), "q_norm": (m.dim,), "lvec": (4, m.dim), "wo": (hidden, m.heads * m.vdim)}
+        if m.kv_from is None:
+            out["k_norm"] = (m.dim,)
+        return out
+    if isinstance(m, SsmSpec):
+        inner = m.heads * m.vdim
+        ch = inner + 2 * m.groups * m.state
+        return {"w_in": (inner + ch + m.heads, hidden), "conv": (ch, m.conv), "conv_b": (ch,), "dt_bias": (m.heads,), "A_log": (m.heads,),
+                "D": (m.heads,), "norm": (inner,), "wo": (hidden, inner)}
     return {"w_in": (m.heads * 2 * (m.dim + m.vdim), hidden), "norm": (m.heads * m.vdim,), "wo": (hidden, m.heads * m.vdim)}
+
+
+def expert_shapes(f: MoeSpec, hidden: int) -> dict[str, tuple]:
+    """Parameter shapes of a layer's routed experts (their input projections are `w13` also where there is no gate)."""
+    E = f.experts
+    return {"router": (E, hidden), "bias" if f.routing is None else "correction": (E,), "w13": (E, f.up_rows, hidden), "w2": (E, hidden, f.expert.ff)}
 
 
 def layer_shapes(s: LayerSpec, cfg: LayeredConfig) -> dict[str, tuple]:
@@ -253,8 +332,13 @@ def layer_shapes(s: LayerSpec, cfg: LayeredConfig) -> dict[str, tuple]:
         out["w_in"] = (mix.pop("w_in")[0] + 2 * ff, H)
         out["w_out"] = (H, mix.pop("wo")[1] + ff)
         if isinstance(s.mlp, MoeSpec):
-            E, F = s.mlp.experts, s.mlp.expert.ff
-            out.update({"mlp.router": (E, H), "mlp.bias": (E,), "mlp.w13": (E, 2 * F, H), "mlp.w2": (E, H, F)})
+            out.update({f"mlp.{n}": shape for n, shape in expert_shapes(s.mlp, H).items()})
+    elif cfg.block == "two_norms":
+        out["ls1"] = (H,)
+        if s.mlp is not None:
+            out.update({"norm2": (H,), "ls2": (H,)})
+            out.update({f"mlp.{n}": shape for n, shape in expert_shapes(s.mlp, H).items()} if isinstance(s.mlp, MoeSpec) else
+                       {"mlp.w13": (2 * s.mlp.ff, H), "mlp.w2": (H, s.mlp.ff)})
     else:
         out["ls1"] = (H,)
         if s.mlp is not None:
@@ -273,7 +357,7 @@ class _Mixer(nn.Module):
             if len(shape) == 2:
                 t = gen(f"{tag}.{name}", shape, std, dtype, device)
             else:
-                t = (torch.zeros if name == "sink" else torch.ones)(shape, dtype=dtype, device=device)
+                t = (torch.ones if name.endswith("norm") or name == "D" else torch.zeros)(shape, dtype=dtype, device=device)
             setattr(self, name, nn.Parameter(t))
 
 
@@ -326,21 +410,55 @@ class AttentionMixer(_Mixer):
         return out
 
 
+class DifferentialMixer(_Mixer):
+    def __init__(self, spec: DifferentialSpec, hidden: int, std: float, dtype, device, gen, tag: str, **kw):
+        super().__init__(spec, hidden, std, dtype, device, gen, tag, **kw)
+        assert spec.heads % spec.kv_heads == 0, "query heads come in equal groups"
+        self.layout = MX.DifferentialLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.kv_from is None)
+
+    def forward(self, proj, meta: ForwardMeta, run: int, eps: float, aside=None):
+        """proj [T, q (; k; v); gates] → [T, heads · vdim].  `aside` (mixers.Aside): what runs beside the preparation."""
+        s, t = self.spec, self.spec.temperature
+        kc, vc = meta.kv_cache[run if s.kv_from is None else s.kv_from]
+        return MX.differential_attention(proj, self.layout, kc, vc, meta, scale=s.scale, diff=s.diff, temperature=(t.coef, t.every) if t else None,
+                                         lvec=self.lvec, q_norm=self.q_norm, k_norm=getattr(self, "k_norm", None), eps=eps, aside=aside)
+
+    def finish(self, o, eps: float):
+        return ops.linear(o, self.wo)
+
+
+class SsmMixer(_Mixer):
+    def __init__(self, spec: SsmSpec, hidden: int, std: float, dtype, device, gen, tag: str, **kw):
+        super().__init__(spec, hidden, std, dtype, device, gen, tag, **kw)
+        assert spec.heads % spec.groups == 0 and spec.heads * spec.vdim % spec.norm_groups == 0, "equal groups of heads, equal parts of a norm"
+        self.layout = MX.SsmLayout(spec.heads, spec.vdim, spec.state, spec.groups, spec.conv)
+
+    def forward(self, proj, meta: ForwardMeta, run: int, eps: float, aside=None):
+        """proj [T, z; x; B; C; dt] → gated outputs [T, heads · vdim], before their norm."""
+        return MX.state_space(proj, self.layout, self.conv, self.conv_b, self.dt_bias, self.A_log, self.D, meta.states[run],
+                              meta.states.get((run, "conv")), meta, aside=aside)
+
+    def finish(self, o, eps: float):
+        return MX.part_norm_linear(o, self.norm, self.spec.norm_groups, eps, self.wo)
+
+
 class RoutedExperts(nn.Module):
     def __init__(self, spec: MoeSpec, hidden: int, std: float, dtype, device, gen, tag: str):
         super().__init__()
         self.spec = spec
-        E, F = spec.experts, spec.expert.ff
-        assert 0 < spec.top <= E
-        self.router = nn.Parameter(gen(f"{tag}.router", (E, hidden), std, dtype, device))
-        self.bias = nn.Parameter(torch.zeros(E, dtype=dtype, device=device))
-        self.w13 = nn.Parameter(gen(f"{tag}.w13", (E, 2 * F, hidden), std, dtype, device))
-        self.w2 = nn.Parameter(gen(f"{tag}.w2", (E, hidden, F), std, dtype, device))
+        assert 0 < spec.top <= spec.experts
+        r = spec.routing
+        assert r is None or (spec.experts % r.groups == 0 and 0 < r.keep <= r.groups), "experts come in equal groups"
+        for name, shape in expert_shapes(spec, hidden).items():
+            t = gen(f"{tag}.{name}", shape, std, dtype, device) if len(shape) > 1 else torch.zeros(shape, dtype=dtype, device=device)
+            setattr(self, name, nn.Parameter(t))
 
     def forward(self, h, weights, index):
         """What the chosen experts of every token add (`mixers.Addend`)."""
         e = self.spec.expert
-        return MX.routed_experts(h, self.w13, self.w2, weights, index, e.limit, e.alpha)
+        if isinstance(e, ReluSquareSpec):
+            return MX.routed_experts(h, self.w13, self.w2, weights, index, ungated=True)
+        return MX.routed_experts(h, self.w13, self.w2, weights, index, e.limit, e.alpha, e.shift)
 
 
 class ClampedGLU(nn.Module):
@@ -351,7 +469,7 @@ class ClampedGLU(nn.Module):
         self.w2 = nn.Parameter(gen(f"{tag}.w2", (hidden, spec.ff), std, dtype, device))
 
     def forward(self, proj):
-        return ops.linear(MX.clamped_glu(proj, self.spec.limit, self.spec.alpha), self.w2)
+        return ops.linear(MX.clamped_glu(proj, self.spec.limit, self.spec.alpha, self.spec.shift), self.w2)
 
 
 class _Stream:
@@ -360,8 +478,8 @@ class _Stream:
     `project` adds the pending output (norm, layer scale, residual sum) and multiplies the new residual by a weight: one kernel
     for a handful of rows, a norm kernel and a GEMM otherwise."""
 
-    def __init__(self, x, xb, eps: float):
-        self.x, self.xb, self.eps, self.pending = x, xb, eps, None
+    def __init__(self, x, xb, cfg: "LayeredConfig"):
+        self.x, self.xb, self.eps, self.pending = x, xb, cfg.rms_eps, None
 
     def project(self, w):
         if self.pending is None:
@@ -390,7 +508,8 @@ class _Stream:
         return MX.output_norm_residual(self.x.clone(), y, nw, ls, self.eps)[0]
 
 
-MIXERS = {LatentSpec: LatentMixer, LinearStateSpec: LinearStateMixer, AttentionSpec: AttentionMixer}
+MIXERS = {LatentSpec: LatentMixer, LinearStateSpec: LinearStateMixer, AttentionSpec: AttentionMixer, DifferentialSpec: DifferentialMixer,
+          SsmSpec: SsmMixer}
 
 
 class LayeredLayer(nn.Module):
@@ -426,8 +545,9 @@ class _SumStream:
     `project` adds them (and, before a later pass of a loop, the embedding output), norms the sum and multiplies it by the layer's
     input projection and its router: one kernel for a handful of rows; a kernel for sum and norm and the products otherwise."""
 
-    def __init__(self, x, _copy, eps: float):
-        self.x, self.first, self.eps = x, x, eps
+    def __init__(self, x, _copy, cfg: "LayeredConfig"):
+        self.x, self.first, self.eps = x, x, cfg.rms_eps
+        self.shift, self.gain = cfg.norm_shift, cfg.logit_scale
         self.pending: list = []
         self.inject = False                        # the embedding output is due before the next layer
 
@@ -451,7 +571,8 @@ class _SumStream:
         return h, proj, logits
 
     def finish(self, final_w):
-        return MX.sum_norm(self.x, None, self.pending, None, final_w, self.eps)
+        # the logits' scale is part of the final norm: whatever multiplies these rows by the head sees it
+        return MX.sum_norm(self.x, None, self.pending, None, final_w, self.eps, shift=self.shift, gain=self.gain)
 
     def value(self):
         """The residual with everything added (debugging and tests)."""
@@ -460,6 +581,70 @@ class _SumStream:
             return x.copy_(self.x)
         MX.sum_norm(self.x, x, self.pending, None, None, self.eps)
         return x
+
+
+class _TwoNormStream(_SumStream):
+    """The same for the "two_norms" arrangement: sublayer outputs have scales, and the sum is normed by two weights (one root mean
+    square), the second for the feed-forward's input projection or router."""
+
+    def project(self, nw, w, nw2=None, w2=None, routes: bool = False):
+        """(product of the residual normed by `nw` with `w`, product of the one normed by `nw2` with `w2` — fp32 logits where it routes,
+        the normed rows of those logits)"""
+        if MX.few_row_sum(self.x, self.pending, w) and (w2 is None or MX.few_row_sum(self.x, self.pending, w2)):
+            proj, second, h2, self.x = MX.sum_two_norms_linear(self.x, self.pending, nw, w, nw2, w2, self.eps, self.shift, routes)
+        else:
+            to = self._sum_into()
+            h, h2 = MX.sum_norm(self.x, to, self.pending, None, nw, self.eps, shift=self.shift, nw2=nw2, two=True)
+            self.x = self.x if to is None else to
+            proj = MX.product(h, w)
+            second = None if w2 is None else MX.product(h2, w2, fp32=routes)
+        self.pending = []
+        return proj, second, h2 if routes else None
+
+
+class TwoNormLayer(nn.Module):
+    """The "two_norms" arrangement: x + ls1 · mixer(norm1(x)) + ls2 · feed-forward(norm2(x))."""
+
+    def __init__(self, spec: LayerSpec, cfg: LayeredConfig, dtype, device, gen, layer: int):
+        super().__init__()
+        self.layer, self.eps, self.spec = layer, cfg.rms_eps, spec
+        H, std, tag = cfg.hidden_size, cfg.init_std, f"L{layer}"
+        assert isinstance(spec.mixer, (DifferentialSpec, SsmSpec)), "mixers of the two-norm arrangement take an aside and finish their own output"
+        assert spec.dense is None or not isinstance(spec.mlp, MoeSpec), "no shared expert in the two-norm arrangement"
+
+        def vec(value):
+            return nn.Parameter(torch.full((H,), value, dtype=dtype, device=device))
+
+        self.norm1, self.ls1 = vec(1.0 - cfg.norm_shift), vec(1.0)
+        self.mix = MIXERS[type(spec.mixer)](spec.mixer, H, std, dtype, device, gen, f"{tag}.mix")
+        self.mlp = None
+        if spec.mlp is not None:
+            self.norm2, self.ls2 = vec(1.0 - cfg.norm_shift), vec(1.0)
+            self.mlp = (RoutedExperts if isinstance(spec.mlp, MoeSpec) else ClampedGLU)(spec.mlp, H, std, dtype, device, gen, f"{tag}.mlp")
+
+    def forward(self, st: _TwoNormStream, meta: ForwardMeta, run: int):
+        mlp, f = self.mlp, self.spec.mlp
+        moe = isinstance(f, MoeSpec)
+        if mlp is None:
+            proj, second, h2 = st.project(self.norm1, self.mix.w_in)
+        else:
+            proj, second, h2 = st.project(self.norm1, self.mix.w_in, self.norm2, mlp.router if moe else mlp.w13, moe)
+        aside = MX.Aside()
+        if moe:
+            aside.logits, aside.top, aside.routing, aside.correction = second, f.top, f.routing, getattr(mlp, "correction", None)
+        elif mlp is not None:
+            aside.glu_in, aside.glu_out = second, torch.empty(proj.shape[0], f.ff, dtype=proj.dtype, device=proj.device)
+            aside.limit, aside.alpha, aside.shift = f.limit, f.alpha, f.shift
+        o = self.mix(proj, meta, run, self.eps, aside=aside)
+        st.pending = [MX.Addend(self.mix.finish(o, self.eps), scale=self.ls1)]
+        if moe:
+            if meta.record_topk is not None:
+                meta.record_topk.append(_as_recorded(aside.index, meta.record_width))
+            a = mlp(h2, aside.weights, aside.index)
+            a.scale = self.ls2
+            st.pending.append(a)
+        elif mlp is not None:
+            st.pending.append(MX.Addend(ops.linear(aside.glu_out, mlp.w2), scale=self.ls2))
 
 
 class ParallelLayer(nn.Module):
@@ -473,6 +658,7 @@ class ParallelLayer(nn.Module):
         self.layer, self.eps, self.dense = layer, cfg.rms_eps, spec.dense
         H, std, tag = cfg.hidden_size, cfg.init_std, f"L{layer}"
         assert isinstance(spec.mixer, AttentionSpec), "the parallel arrangement is built for attention mixers"
+        assert spec.mlp is None or (isinstance(spec.mlp, MoeSpec) and spec.mlp.routing is None) or spec.dense is not None
         shapes = layer_shapes(spec, cfg)
         self.norm1 = nn.Parameter(torch.ones(H, dtype=dtype, device=device))
         self.w_in = nn.Parameter(gen(f"{tag}.w_in", shapes["w_in"], std, dtype, device))
@@ -489,7 +675,7 @@ class ParallelLayer(nn.Module):
         aside = MX.Aside(logits=logits, top=moe.spec.top if moe is not None else 0)
         if self.dense is not None:
             aside.glu_in, aside.glu_out = proj[:, self.at_dense:], both[:, self.mix_out:]
-            aside.limit, aside.alpha = self.dense.limit, self.dense.alpha
+            aside.limit, aside.alpha, aside.shift = self.dense.limit, self.dense.alpha, self.dense.shift
         self.mix(proj, meta, run, self.eps, out=both[:, : self.mix_out], aside=aside)
         st.pending = [MX.Addend(ops.linear(both, self.w_out))]
         if moe is not None:
@@ -526,6 +712,12 @@ class LayeredModel(Qwen3Model):
                 src = cfg.layer_specs[m.kv_from].mixer
                 assert m.kv_from < i and isinstance(src, LatentSpec) and src.kv_from is None and (src.kv_rank, src.rot_dim) == (
                     m.kv_rank, m.rot_dim), f"layer {i} cannot read the latents of layer {m.kv_from}"
+            if isinstance(m, DifferentialSpec) and m.kv_from is not None:
+                src = cfg.layer_specs[m.kv_from].mixer
+                assert m.kv_from < i and isinstance(src, DifferentialSpec) and src.kv_from is None and (src.kv_heads, src.dim, src.vdim) == (
+                    m.kv_heads, m.dim, m.vdim), f"layer {i} cannot read the keys and values of layer {m.kv_from}"
+        assert cfg.norm_shift == 0.0 or cfg.block == "two_norms", "norm weights stored around another value: two-norm arrangement only"
+        assert cfg.logit_scale == 1.0 or cfg.block != "output_norm", "a logit scale is part of the final norm of the summing streams"
         if cfg.loop is not None:
             assert 0 <= cfg.loop.start < cfg.loop.stop <= cfg.num_layers and cfg.loop.times > 0, f"{cfg.loop} of {cfg.num_layers} layers"
             assert cfg.block == "parallel", "loops are built for the parallel arrangement"
@@ -536,6 +728,12 @@ class LayeredModel(Qwen3Model):
         if cfg.bigram is not None:
             self.bigram = nn.Parameter(gen("bigram", (cfg.bigram.buckets + 1, cfg.hidden_size), cfg.init_std, dtype, device))
         self.num_moe_layers = cfg.num_moe_layers
+        if cfg.norm_shift:
+            with torch.no_grad():
+                self.norm.fill_(1.0 - cfg.norm_shift)
+        H = cfg.hidden_size
+        freq = [cfg.position_base ** (-2.0 * i / H) for i in range((H + 1) // 2)] if cfg.position_base else []
+        self.register_buffer("position_freq", torch.tensor(freq, dtype=torch.float64, device=device) if freq else None, persistent=False)
 
     # ---- what the engine keeps per token and per sequence ------------------------------------------------------------
     def _run_mixers(self):
@@ -549,11 +747,21 @@ class LayeredModel(Qwen3Model):
                 rows[r] = ((m.layout.pitch,),)
             elif isinstance(m, AttentionMixer):
                 rows[r] = ((m.spec.kv_heads, m.spec.dim), (m.spec.kv_heads, m.spec.vdim))
+            elif isinstance(m, DifferentialMixer) and m.spec.kv_from is None:
+                rows[r] = ((m.spec.kv_heads, 2 * m.spec.dim), (m.spec.kv_heads, m.spec.vdim))      # a key row holds both maps
         return rows
 
-    def state_shapes(self) -> dict[int, tuple]:
-        """fp32 state per sequence of every recurrent layer run."""
-        return {r: (m.spec.heads, m.spec.dim, m.spec.vdim) for r, m in self._run_mixers() if isinstance(m, LinearStateMixer)}
+    def state_shapes(self) -> dict:
+        """fp32 state per sequence of every recurrent layer run; under (run, "conv") the last inputs of its convolution."""
+        out: dict = {}
+        for r, m in self._run_mixers():
+            if isinstance(m, LinearStateMixer):
+                out[r] = (m.spec.heads, m.spec.dim, m.spec.vdim)
+            elif isinstance(m, SsmMixer):
+                out[r] = (m.spec.heads, m.spec.state, m.spec.vdim)
+                if m.spec.conv > 1:
+                    out[(r, "conv")] = (m.spec.conv, m.layout.channels)
+        return out
 
     def forward(self, tokens, meta: ForwardMeta, hidden_in=None, inputs_embeds=None):
         if torch.is_grad_enabled():
@@ -562,7 +770,8 @@ class LayeredModel(Qwen3Model):
         big = self.cfg.bigram
         st = BLOCKS[self.cfg.block][1](*MX.bigram_embedding(tokens, meta.prev_tokens, self.embed, self.bigram,
                                                             (big.buckets, big.mul_prev, big.mul_cur) if big is not None else None,
-                                                            want_copy=self.cfg.block == "output_norm"), self.cfg.rms_eps)
+                                                            want_copy=self.cfg.block == "output_norm", positions=meta.positions,
+                                                            freq=self.position_freq), self.cfg)
         meta.record_width = self.cfg.moe_topk
         for run, (l, inject) in enumerate(self.runs):
             st.inject = inject
@@ -573,4 +782,4 @@ class LayeredModel(Qwen3Model):
 
 
 # arrangement → (layer, stream of residual and pending outputs)
-BLOCKS = {"output_norm": (LayeredLayer, _Stream), "parallel": (ParallelLayer, _SumStream)}
+BLOCKS = {"output_norm": (LayeredLayer, _Stream), "parallel": (ParallelLayer, _SumStream), "two_norms": (TwoNormLayer, _TwoNormStream)}

@@ -32,18 +32,22 @@ def sources() -> list[str]:
 SERVE_SUFFIX = "_serve"
 SERVE_SOURCES = ["counter.cpp", "bindings.cpp", "bindings_more.cpp", "bindings_misc.cpp", "bindings_mixers.cpp", "gemm.cu", "gemm_small.cu",
                  "gemv.cu", "misc.cu", "mixers.cu", "paged_attend.cu"]
+_EXPERTS = ["bindings_moe.cpp", "moe.cu", "experts_any.cu"]
+_WINDOW = ["attention_window_tc.cu", "window_decode.cu"]
 SERVE_KINDS = {
     "latent": ["attention_latent_tc.cu", "latent_attn.cu", "latent_decode.cu", "latent_decode_tc.cu", "linear_state.cu", "linear_chunk.cu"],
-    "attention": ["bindings_moe.cpp", "moe.cu", "attention_window_tc.cu", "window_prep.cu", "window_decode.cu", "experts_any.cu"],
+    "attention": [*_EXPERTS, *_WINDOW, "window_prep.cu"],
+    "hybrid": [*_EXPERTS, *_WINDOW, "diff_prep.cu", "ssm_state.cu", "ssm_chunk.cu"],
 }
 _serving: str | None = None                   # the serving build this process asked for
 
 
 def serve_kind(cfg) -> str:
     """Which serving build a layered configuration needs."""
-    from ..models.layered import AttentionSpec
+    from ..models.layered import AttentionSpec, DifferentialSpec, SsmSpec
 
-    kinds = {"attention" if isinstance(s.mixer, AttentionSpec) else "latent" for s in cfg.layer_specs}
+    of = {AttentionSpec: "attention", DifferentialSpec: "hybrid", SsmSpec: "hybrid"}
+    kinds = {of.get(type(s.mixer), "latent") for s in cfg.layer_specs}
     assert len(kinds) == 1, f"no serving build has the mixers of {kinds} together: run a full build"
     return kinds.pop()
 

@@ -9,6 +9,8 @@
 //   * keys and values come straight from their pages: a tile of 64 positions is one box of a page of ≥ 64 tokens (or several boxes
 //     of smaller pages).  What a box reads past a head's own columns meets zero query columns or is never stored; rows of a page behind
 //     the sequence's end are masked;
+//   * differential attention (MbDiff): heads 2h and 2h + 1 are neighbouring rows; their threads exchange the two maps' outputs, and the
+//     difference is normed and gated on its way out;
 //   * the key tiles of a query tile are those of the kept first tokens and those of the window; what lies between is skipped.
 #include "launch.h"
 #include "ptx.cuh"
@@ -38,6 +40,7 @@ struct Params {
   int dim, vdim;
   float scale;
   int window, keep;            // window 0: all earlier keys
+  MbDiff diff;
   int* error_flag;
 };
 
@@ -265,7 +268,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     if (!ok) {
       *abort_flag = 1;
       atomicExch(p.error_flag, 83);
-    } else if (!*abort_flag) {
+    }
+    if (__all_sync(0xffffffffu, ok && !*abort_flag)) {      // the whole warp or none of it: the loads and exchanges below are collective
       tc_fence_after();
       // O / (l + exp(sink)), both relative to the larger of the running maximum and the sink
       float inv = 0.f;
@@ -278,22 +282,72 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
           inv = __fdiv_rn(1.f, l_run);
         }
       }
-      __nv_bfloat16* orow = p.o + static_cast<long long>(q_start + t0 + tok) * p.o_row + static_cast<long long>(head) * p.vdim;
-#pragma unroll 1
-      for (int c = 0; c < NV * 2; ++c) {
-        uint32_t o[32];
-        tmem_ld_32x32(tmem_o + lane_off + c * 32, o);
-        tmem_ld_wait();
-        if (valid) {
+      if (p.diff.lam != nullptr) {
+        // both rows of a head hold o = a1 − lam·a2 after the exchange; the even one stores the first half of every 32 columns, the odd
+        // one the second
+        const float lam = *p.diff.lam;
+        const bool odd = row & 1;
+        auto difference = [&](uint32_t (&o)[32]) {
 #pragma unroll
-          for (int i = 0; i < 32; i += 8) {
-            if (c * 32 + i < p.vdim) {         // vdim is a multiple of 8
-              uint4 v;
-              v.x = pack_bf16x2(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
-              v.y = pack_bf16x2(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
-              v.z = pack_bf16x2(__uint_as_float(o[i + 4]) * inv, __uint_as_float(o[i + 5]) * inv);
-              v.w = pack_bf16x2(__uint_as_float(o[i + 6]) * inv, __uint_as_float(o[i + 7]) * inv);
-              *reinterpret_cast<uint4*>(orow + c * 32 + i) = v;
+          for (int i = 0; i < 32; ++i) {
+            const float a = __uint_as_float(o[i]) * inv, other = __shfl_xor_sync(0xffffffffu, a, 1);
+            o[i] = __float_as_uint(odd ? fmaf(-lam, a, other) : fmaf(-lam, other, a));
+          }
+        };
+        float ss = 0.f;
+#pragma unroll 1
+        for (int c = 0; c < NV * 2; ++c) {
+          uint32_t o[32];
+          tmem_ld_32x32(tmem_o + lane_off + c * 32, o);
+          tmem_ld_wait();
+          difference(o);
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i < p.vdim) ss = fmaf(__uint_as_float(o[i]), __uint_as_float(o[i]), ss);
+        }
+        float f = 0.f;
+        if (valid) {
+          const float g = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.diff.gate)[static_cast<long long>(q_start + t0 + tok) * p.diff.gate_ld + head / 2]);
+          f = __fdiv_rn(p.diff.gain, __fsqrt_rn(__fdiv_rn(ss, static_cast<float>(p.vdim)) + p.diff.eps)) * __fdividef(1.f, 1.f + __expf(-g));
+        }
+        __nv_bfloat16* orow = p.o + static_cast<long long>(q_start + t0 + tok) * p.o_row + static_cast<long long>(head / 2) * p.vdim;
+#pragma unroll 1
+        for (int c = 0; c < NV * 2; ++c) {
+          uint32_t o[32];
+          tmem_ld_32x32(tmem_o + lane_off + c * 32, o);
+          tmem_ld_wait();
+          difference(o);
+          if (valid) {
+#pragma unroll
+            for (int i = 0; i < 16; i += 8) {
+              const int col = c * 32 + (odd ? 16 : 0) + i;
+              uint32_t w[4];
+#pragma unroll
+              for (int k = 0; k < 4; ++k)
+                w[k] = odd ? pack_bf16x2(__uint_as_float(o[16 + i + 2 * k]) * f, __uint_as_float(o[16 + i + 2 * k + 1]) * f)
+                           : pack_bf16x2(__uint_as_float(o[i + 2 * k]) * f, __uint_as_float(o[i + 2 * k + 1]) * f);
+              if (col < p.vdim) *reinterpret_cast<uint4*>(orow + col) = make_uint4(w[0], w[1], w[2], w[3]);
+            }
+          }
+        }
+      } else {
+        __nv_bfloat16* orow = p.o + static_cast<long long>(q_start + t0 + tok) * p.o_row + static_cast<long long>(head) * p.vdim;
+#pragma unroll 1
+        for (int c = 0; c < NV * 2; ++c) {
+          uint32_t o[32];
+          tmem_ld_32x32(tmem_o + lane_off + c * 32, o);
+          tmem_ld_wait();
+          if (valid) {
+#pragma unroll
+            for (int i = 0; i < 32; i += 8) {
+              if (c * 32 + i < p.vdim) {         // vdim is a multiple of 8
+                uint4 v;
+                v.x = pack_bf16x2(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
+                v.y = pack_bf16x2(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
+                v.z = pack_bf16x2(__uint_as_float(o[i + 4]) * inv, __uint_as_float(o[i + 5]) * inv);
+                v.w = pack_bf16x2(__uint_as_float(o[i + 6]) * inv, __uint_as_float(o[i + 7]) * inv);
+                *reinterpret_cast<uint4*>(orow + c * 32 + i) = v;
+              }
             }
           }
         }
@@ -333,11 +387,11 @@ using namespace mb;
 // o_row elements (a multiple of 8).  dim, vdim multiples of 8 up to 128, block_size a multiple of 8, up to 128 query heads per key head, scale > 0.
 extern "C" int mb_window_prefill(const void* q, const void* kc, const void* vc, void* o, long long o_row, const void* sink, const int* cu_q,
                                  const int* positions, const int* block_table, int max_blocks, int block_size, int num_blocks, int n_seq, int max_q,
-                                 int t_long, float scale, MbWindow L, int* error_flag, cudaStream_t s) {
+                                 int t_long, float scale, MbWindow L, MbDiff d, int* error_flag, cudaStream_t s) {
   if (n_seq <= 0 || t_long <= 0) return 0;
   const int group = L.heads / L.kv_heads, na = (L.dim + 63) / 64, nv = (L.vdim + 63) / 64;
   if (L.dim % 8 || L.vdim % 8 || L.dim > 128 || L.vdim > 128 || L.q_pitch != na * 64 || L.heads % L.kv_heads || group > 128 || block_size % 8 ||
-      o_row % 8 || !(scale > 0.f))
+      o_row % 8 || !(scale > 0.f) || (d.lam != nullptr && (sink != nullptr || group % 2)))
     return -3;
   int box = 64;
   while (block_size % box) box /= 2;
@@ -351,7 +405,7 @@ extern "C" int mb_window_prefill(const void* q, const void* kc, const void* vc, 
   rc = make_tmap_bf16_2d(&tv, vc, rows, vw, vw, box, 64);
   if (rc) return 3000 + rc;
   fw::Params p{reinterpret_cast<__nv_bfloat16*>(o), o_row, reinterpret_cast<const __nv_bfloat16*>(sink), cu_q, positions, block_table, max_blocks,
-               block_size, box, group, tokens, L.dim, L.vdim, scale, L.window, L.keep, error_flag};
+               block_size, box, group, tokens, L.dim, L.vdim, scale, L.window, L.keep, d, error_flag};
   if (na == 1) return nv == 1 ? fw::launch<1, 1>(tq, tk, tv, p, max_q, L.kv_heads, n_seq, s) : fw::launch<1, 2>(tq, tk, tv, p, max_q, L.kv_heads, n_seq, s);
   return nv == 1 ? fw::launch<2, 1>(tq, tk, tv, p, max_q, L.kv_heads, n_seq, s) : fw::launch<2, 2>(tq, tk, tv, p, max_q, L.kv_heads, n_seq, s);
 }

@@ -77,12 +77,12 @@ void gemv(const at::Tensor& x, const c10::optional<at::Tensor>& residual, const 
 }
 
 void moe_gemv(const at::Tensor& x, const at::Tensor& w13, const at::Tensor& w2, const at::Tensor& topk_idx, const at::Tensor& topk_w,
-              at::Tensor& act, at::Tensor& out, int64_t expert_offset, double limit, double alpha) {
+              at::Tensor& act, at::Tensor& out, int64_t expert_offset, double limit, double alpha, double shift, bool ungated) {
   c10::cuda::CUDAGuard g(x.device());
-  const int64_t T = x.size(0), H = x.size(1), k = topk_idx.size(1), E = w13.size(0), F = w13.size(1) / 2;
+  const int64_t T = x.size(0), H = x.size(1), k = topk_idx.size(1), E = w13.size(0), F = w13.size(1) / (ungated ? 1 : 2);
   mb_count_launch(1);
   check(mb_moe_gemv(x.data_ptr(), w13.data_ptr(), w2.data_ptr(), topk_idx.data_ptr<int>(), topk_w.data_ptr<float>(), act.data_ptr(),
-                    out.data_ptr(), T, k, E, expert_offset, H, F, limit, alpha, cur_stream()),
+                    out.data_ptr(), T, k, E, expert_offset, H, F, limit, alpha, shift, ungated, cur_stream()),
         "mb_moe_gemv");
 }
 
@@ -244,7 +244,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_small", &gemm_small);
   m.def("gemv", &gemv);
   m.def("moe_gemv", &moe_gemv, py::arg("x"), py::arg("w13"), py::arg("w2"), py::arg("topk_idx"), py::arg("topk_w"), py::arg("act"), py::arg("out"),
-        py::arg("expert_offset"), py::arg("limit") = 0.0, py::arg("alpha") = 0.0);
+        py::arg("expert_offset"), py::arg("limit") = 0.0, py::arg("alpha") = 0.0, py::arg("shift") = 1.0, py::arg("ungated") = false);
   m.def("gemm_small_grouped", &gemm_small_grouped);
   m.def("gemm_grouped_wgrad", &gemm_grouped_wgrad);
 #ifndef MB_SERVE_SUBSET      // the training and grouped-query kernels of elementwise.cu

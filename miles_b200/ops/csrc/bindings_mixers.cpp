@@ -1,4 +1,5 @@
-// Bindings of the layer-by-layer decoders' kernels: mixers.cu, latent_*.cu, linear_*.cu, window_*.cu, paged_attend.cu, experts_any.cu.
+// Bindings of the layer-by-layer decoders' kernels: mixers.cu, latent_*.cu, linear_*.cu, window_*.cu, paged_attend.cu, experts_any.cu,
+// diff_prep.cu, ssm_*.cu.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
@@ -10,6 +11,12 @@
 #define MB_HAS_LATENT
 #endif
 #if !defined(MB_SERVE_SUBSET) || defined(MB_SERVE_ATTENTION)
+#define MB_HAS_WINDOW
+#endif
+#if !defined(MB_SERVE_SUBSET) || defined(MB_SERVE_HYBRID)
+#define MB_HAS_HYBRID
+#endif
+#if defined(MB_HAS_WINDOW) || defined(MB_HAS_HYBRID)
 #define MB_HAS_ATTENTION
 #endif
 
@@ -37,10 +44,12 @@ inline void check(int rc, const char* what) {
   throw std::runtime_error(buf);
 }
 void bigram_embedding(const at::Tensor& tok, const OptTensor& prev, const at::Tensor& embed, const OptTensor& table, int64_t buckets,
-                      int64_t mul_prev, int64_t mul_cur, at::Tensor& x, const OptTensor& xb) {
+                      int64_t mul_prev, int64_t mul_cur, const OptTensor& positions, const OptTensor& freq, at::Tensor& x, const OptTensor& xb) {
   c10::cuda::CUDAGuard g(embed.device());
-  check(mb_bigram_embedding(tok.data_ptr<int>(), iptr(prev), embed.data_ptr(), cptr(table), buckets, mul_prev, mul_cur, x.data_ptr<float>(),
-                            mptr(xb), tok.numel(), embed.size(1), f32(embed), cur_stream()),
+  const double* f = freq.has_value() && freq->defined() ? freq->data_ptr<double>() : nullptr;
+  TORCH_CHECK(f == nullptr || freq->numel() * 2 >= embed.size(1), "bigram_embedding: a frequency per pair of channels");
+  check(mb_bigram_embedding(tok.data_ptr<int>(), iptr(prev), embed.data_ptr(), cptr(table), buckets, mul_prev, mul_cur, iptr(positions), f,
+                            x.data_ptr<float>(), mptr(xb), tok.numel(), embed.size(1), f32(embed), cur_stream()),
         "mb_bigram_embedding");
 }
 
@@ -61,50 +70,97 @@ void gemv_output_norm(const at::Tensor& x, const at::Tensor& y, const at::Tensor
 }
 
 // rows of `in` [gate, up] and of `out` may be strided; rows (optional): device count of the rows in use
-void clamped_glu(const at::Tensor& in, at::Tensor& out, double limit, double alpha, const OptTensor& rows) {
+void clamped_glu(const at::Tensor& in, at::Tensor& out, double limit, double alpha, const OptTensor& rows, double shift) {
   c10::cuda::CUDAGuard g(in.device());
   TORCH_CHECK(in.stride(1) == 1 && out.stride(1) == 1 && in.size(1) >= 2 * out.size(1), "clamped_glu: rows of [gate, up]");
-  check(mb_clamped_glu(in.data_ptr(), in.stride(0), out.data_ptr(), out.stride(0), out.size(0), out.size(1), limit, alpha, iptr(rows), f32(in),
+  check(mb_clamped_glu(in.data_ptr(), in.stride(0), out.data_ptr(), out.stride(0), out.size(0), out.size(1), limit, alpha, shift, iptr(rows), f32(in),
                        cur_stream()),
         "mb_clamped_glu");
 }
 
-void sum_norm(const at::Tensor& x, const OptTensor& to, const OptTensor& y1, const OptTensor& y2, const OptTensor& rows, const OptTensor& weights,
-              const OptTensor& dst, const OptTensor& extra, const OptTensor& nw, const OptTensor& h, double eps) {
+void relu_square(at::Tensor& x, const OptTensor& rows) {
+  c10::cuda::CUDAGuard g(x.device());
+  TORCH_CHECK(x.is_contiguous(), "relu_square: contiguous rows");
+  check(mb_relu_square(x.data_ptr(), x.size(0), x.size(1), iptr(rows), f32(x), cur_stream()), "mb_relu_square");
+}
+
+void part_norm(const at::Tensor& x, const at::Tensor& w, at::Tensor& out, int64_t parts, double eps) {
+  c10::cuda::CUDAGuard g(x.device());
+  TORCH_CHECK(x.is_contiguous() && out.is_contiguous() && w.numel() == x.size(1), "part_norm: contiguous rows, a weight per channel");
+  check(mb_part_norm(x.data_ptr(), w.data_ptr(), out.data_ptr(), x.size(0), x.size(1), parts, eps, f32(x), cur_stream()), "mb_part_norm");
+}
+
+// every addend may have a scale (s1 of y1; s2 of y2 or of the experts' rows)
+void sum_norm(const at::Tensor& x, const OptTensor& to, const OptTensor& y1, const OptTensor& s1, const OptTensor& y2, const OptTensor& s2,
+              const OptTensor& rows, const OptTensor& weights, const OptTensor& dst, const OptTensor& extra, const OptTensor& nw, const OptTensor& h,
+              const OptTensor& nw2, const OptTensor& h2, double eps, double shift, double gain) {
   c10::cuda::CUDAGuard g(x.device());
   MbSumNorm p{};
   p.x = x.data_ptr<float>();
   p.to = fmut(to);
   p.y1 = cptr(y1);
   p.y2 = cptr(y2);
+  p.s1 = cptr(s1);
+  p.s2 = cptr(s2);
   p.rows = cptr(rows);
   p.weights = fptr(weights);
   p.dst = iptr(dst);
   p.extra = fptr(extra);
   p.nw = cptr(nw);
   p.h = mptr(h);
+  p.nw2 = cptr(nw2);
+  p.h2 = mptr(h2);
   p.T = x.size(0);
   p.D = x.size(1);
   p.k = p.weights != nullptr ? weights->size(1) : 0;
   p.eps = eps;
-  for (const OptTensor* t : {&y1, &y2, &rows, &nw})
+  p.shift = shift;
+  p.gain = gain;
+  for (const OptTensor* t : {&y1, &y2, &rows, &nw, &nw2, &s1, &s2})
     TORCH_CHECK(!t->has_value() || !(*t)->defined() || (*t)->is_contiguous(), "sum_norm: contiguous rows");
+  TORCH_CHECK(p.s2 == nullptr || p.y2 == nullptr || p.rows == nullptr, "sum_norm: one addend per scale");
   int is32 = 0;
   for (const OptTensor* t : {&nw, &y1, &y2, &rows})
     if (t->has_value() && (*t)->defined()) is32 = f32(**t);
   check(mb_sum_norm(p, is32, cur_stream()), "mb_sum_norm");
 }
 
-// x32 (with y1, y2, extra, norm_w) or plain rows x; W [N, K] → y, W2 [N2, K] → fp32 y2out
-void gemv_sum_norm(const OptTensor& x32, const OptTensor& y1, const OptTensor& y2, const OptTensor& extra, const OptTensor& x, const OptTensor& norm_w,
-                   double eps, const at::Tensor& W, at::Tensor& y, const OptTensor& W2, const OptTensor& bias2, const OptTensor& y2out,
-                   const OptTensor& x_out, const OptTensor& xn_out, bool static_w) {
+// x32 (with y1·s1, y2·s2, extra, norm_w) or plain rows x; W [N, K] → y, W2 [N2, K] → y2out (float or bf16; its rows by norm_w2 if given)
+void gemv_sum_norm(const OptTensor& x32, const OptTensor& y1, const OptTensor& s1, const OptTensor& y2, const OptTensor& s2, const OptTensor& extra,
+                   const OptTensor& x, const OptTensor& norm_w, const OptTensor& norm_w2, double eps, double shift, const at::Tensor& W, at::Tensor& y,
+                   const OptTensor& W2, const OptTensor& bias2, const OptTensor& y2out, const OptTensor& x_out, const OptTensor& xn_out, bool static_w) {
   c10::cuda::CUDAGuard g(W.device());
   const bool two = W2.has_value() && W2->defined();
-  check(mb_gemv_sum_norm(fptr(x32), cptr(y1), cptr(y2), fptr(extra), cptr(x), cptr(norm_w), eps, W.data_ptr(), y.data_ptr(), y.stride(0), cptr(W2),
-                         cptr(bias2), fmut(y2out), fmut(x_out), mptr(xn_out), y.size(0), W.size(0), two ? W2->size(0) : 0, W.size(1), static_w,
-                         cur_stream()),
-        "mb_gemv_sum_norm");
+  MbGemvSum a{};
+  a.x32 = fptr(x32);
+  a.y1 = cptr(y1);
+  a.s1 = cptr(s1);
+  a.y2 = cptr(y2);
+  a.s2 = cptr(s2);
+  a.extra = fptr(extra);
+  a.x = cptr(x);
+  a.norm_w = cptr(norm_w);
+  a.norm_w2 = cptr(norm_w2);
+  a.eps = eps;
+  a.shift = shift;
+  a.W = W.data_ptr();
+  a.y = y.data_ptr();
+  a.ldy = y.stride(0);
+  a.W2 = cptr(W2);
+  a.bias2 = cptr(bias2);
+  if (two) {
+    a.out2 = mptr(y2out);
+    a.ld2 = y2out->stride(0);
+    a.out2_fp32 = f32(*y2out);
+    a.N2 = W2->size(0);
+  }
+  a.x_out = fmut(x_out);
+  a.xn_out = mptr(xn_out);
+  a.M = y.size(0);
+  a.N = W.size(0);
+  a.K = W.size(1);
+  a.static_w = static_w;
+  check(mb_gemv_sum_norm(a, cur_stream()), "mb_gemv_sum_norm");
 }
 
 void gated_norm(const at::Tensor& o, const at::Tensor& w, const at::Tensor& gate, at::Tensor& out, double eps) {
@@ -206,47 +262,74 @@ void linear_chunk(const at::Tensor& proj, const at::Tensor& decay, at::Tensor& s
 #endif  // MB_HAS_LATENT
 
 #ifdef MB_HAS_ATTENTION
+// {logits, weights, index, glu_in, glu_out, correction (each or None)}, {limit, alpha, up shift, weights' scale}, {grouped, groups, keep}
+inline MbAside aside(const std::vector<OptTensor>& t, const std::vector<double>& f, const std::vector<int64_t>& n) {
+  TORCH_CHECK(t.size() == 6 && f.size() == 4 && n.size() == 3, "an aside has 6 tensors, 4 numbers and 3 counts");
+  MbAside a{};
+  if (t[0].has_value() && t[0]->defined()) {
+    a.logits = t[0]->data_ptr<float>();
+    a.weights = fmut(t[1]);
+    a.index = t[2]->data_ptr<int>();
+    a.experts = t[0]->size(1);
+    a.top = t[2]->size(1);
+    TORCH_CHECK(t[0]->is_contiguous(), "an aside's logits are contiguous");
+  }
+  if (t[3].has_value() && t[3]->defined()) {
+    a.glu_in = t[3]->data_ptr();
+    a.glu_out = mptr(t[4]);
+    a.glu_ld_in = t[3]->stride(0);
+    a.glu_ld_out = t[4]->stride(0);
+    a.ff = t[4]->size(1);
+  }
+  a.correction = cptr(t[5]);
+  a.limit = f[0];
+  a.alpha = f[1];
+  a.shift = f[2];
+  a.scale = f[3];
+  a.grouped = n[0];
+  a.groups = n[1];
+  a.keep = n[2];
+  return a;
+}
+
+// (weight of the second map, gate rows, gain, eps), or nothing
+inline MbDiff difference(const OptTensor& lam, const OptTensor& gate, double gain, double eps) {
+  MbDiff d{};
+  d.lam = fptr(lam);
+  if (d.lam == nullptr) return d;
+  TORCH_CHECK(gate.has_value() && gate->stride(1) == 1, "differential attention has gates, one per head");
+  d.gate = gate->data_ptr();
+  d.gate_ld = gate->stride(0);
+  d.gain = gain;
+  d.eps = eps;
+  return d;
+}
+
 inline MbWindow window(const std::vector<int64_t>& v) {
   TORCH_CHECK(v.size() == 8, "a windowed attention layout has 8 sizes");
   return MbWindow{static_cast<int>(v[0]), static_cast<int>(v[1]), static_cast<int>(v[2]), static_cast<int>(v[3]),
                   static_cast<int>(v[4]), static_cast<int>(v[5]), static_cast<int>(v[6]), static_cast<int>(v[7])};
 }
 
+#ifdef MB_HAS_WINDOW
 void window_prep(const at::Tensor& proj, const at::Tensor& positions, const at::Tensor& slots, const at::Tensor& freq, double magnitude,
                  const OptTensor& q_norm, const OptTensor& k_norm, double eps, at::Tensor& kc, at::Tensor& vc, at::Tensor& q,
-                 const std::vector<int64_t>& lay, const OptTensor& logits, const OptTensor& weights, const OptTensor& index, const OptTensor& glu_in,
-                 const OptTensor& glu_out, double limit, double alpha) {
+                 const std::vector<int64_t>& lay, const std::vector<OptTensor>& at, const std::vector<double>& af, const std::vector<int64_t>& an) {
   c10::cuda::CUDAGuard g(proj.device());
-  MbAside a{};
-  if (logits.has_value() && logits->defined()) {
-    a.logits = logits->data_ptr<float>();
-    a.weights = fmut(weights);
-    a.index = index->data_ptr<int>();
-    a.experts = logits->size(1);
-    a.top = index->size(1);
-    TORCH_CHECK(logits->is_contiguous(), "window_prep: contiguous logits");
-  }
-  if (glu_in.has_value() && glu_in->defined()) {
-    a.glu_in = glu_in->data_ptr();
-    a.glu_out = mptr(glu_out);
-    a.glu_ld_in = glu_in->stride(0);
-    a.glu_ld_out = glu_out->stride(0);
-    a.ff = glu_out->size(1);
-    a.limit = limit;
-    a.alpha = alpha;
-  }
   check(mb_window_prep(proj.data_ptr(), proj.stride(0), positions.data_ptr<int>(), lptr(slots), freq.data_ptr<double>(), magnitude, cptr(q_norm),
-                       cptr(k_norm), eps, kc.data_ptr(), vc.data_ptr(), q.data_ptr(), proj.size(0), window(lay), a, f32(proj), cur_stream()),
+                       cptr(k_norm), eps, kc.data_ptr(), vc.data_ptr(), q.data_ptr(), proj.size(0), window(lay), aside(at, af, an), f32(proj),
+                       cur_stream()),
         "mb_window_prep");
 }
+#endif
 
 void window_decode(const at::Tensor& q, const at::Tensor& kc, const at::Tensor& vc, const at::Tensor& block_table, const OptTensor& token_seq,
                    const at::Tensor& positions, const at::Tensor& slots, const OptTensor& sink, at::Tensor& out, double scale, int64_t splits,
-                   const std::vector<int64_t>& lay) {
+                   const std::vector<int64_t>& lay, const OptTensor& lam, const OptTensor& gate, double gain, double eps) {
   c10::cuda::CUDAGuard g(q.device());
   check(mb_window_decode(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), block_table.data_ptr<int>(), block_table.size(1), kc.size(1), iptr(token_seq),
                          positions.data_ptr<int>(), lptr(slots), cptr(sink), out.data_ptr(), out.stride(0), q.size(0), scale, splits, window(lay),
-                         cur_stream()),
+                         difference(lam, gate, gain, eps), cur_stream()),
         "mb_window_decode");
 }
 
@@ -271,29 +354,108 @@ void window_attend(const at::Tensor& q, const at::Tensor& kc, const at::Tensor& 
   a.keep = L.keep;
   a.scale = scale;
   check(mb_paged_attend(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), block_table.data_ptr<int>(), block_table.size(1), kc.size(1), iptr(token_seq),
-                        positions.data_ptr<int>(), lptr(slots), cptr(sink), out.data_ptr(), q.size(0), a, f32(q), cur_stream()),
+                        positions.data_ptr<int>(), lptr(slots), cptr(sink), out.data_ptr(), q.size(0), a, f32(q), f32(out), cur_stream()),
         "mb_paged_attend");
 }
 
 void window_prefill(const at::Tensor& q, const at::Tensor& kc, const at::Tensor& vc, at::Tensor& out, const OptTensor& sink, const at::Tensor& cu_q,
                     const at::Tensor& positions, const at::Tensor& block_table, int64_t n_seq, int64_t max_q, int64_t t_long, double scale,
-                    const std::vector<int64_t>& lay, at::Tensor& err) {
+                    const std::vector<int64_t>& lay, at::Tensor& err, const OptTensor& lam, const OptTensor& gate, double gain, double eps) {
   c10::cuda::CUDAGuard g(q.device());
   check(mb_window_prefill(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), out.data_ptr(), out.stride(0), cptr(sink), cu_q.data_ptr<int>(),
                           positions.data_ptr<int>(), block_table.data_ptr<int>(), block_table.size(1), kc.size(1), kc.size(0), n_seq, max_q, t_long,
-                          scale, window(lay), err.data_ptr<int>(), cur_stream()),
+                          scale, window(lay), difference(lam, gate, gain, eps), err.data_ptr<int>(), cur_stream()),
         "mb_window_prefill");
 }
 
 void experts_any(const at::Tensor& x, const at::Tensor& w13, const at::Tensor& w2, const at::Tensor& index, const at::Tensor& weights, at::Tensor& act,
-                 at::Tensor& out, double limit, double alpha) {
+                 at::Tensor& out, double limit, double alpha, double shift) {
   c10::cuda::CUDAGuard g(x.device());
   mb_count_launch(1);
   check(mb_experts_any(x.data_ptr(), w13.data_ptr(), w2.data_ptr(), index.data_ptr<int>(), weights.data_ptr<float>(), act.data_ptr(), out.data_ptr(),
-                       x.size(0), index.size(1), w13.size(0), x.size(1), w2.size(2), limit, alpha, f32(x), cur_stream()),
+                       x.size(0), index.size(1), w13.size(0), x.size(1), w2.size(2), limit, alpha, shift, f32(x), cur_stream()),
         "mb_experts_any");
 }
 #endif  // MB_HAS_ATTENTION
+
+#ifdef MB_HAS_HYBRID
+// sizes: heads, key heads (0: another layer's keys and values), one map's size, value size, elements per prepared query row
+void diff_prep(const at::Tensor& proj, const at::Tensor& positions, const at::Tensor& slots, const at::Tensor& q_norm, const OptTensor& k_norm,
+               const at::Tensor& lvec, at::Tensor& lam, const OptTensor& kc, const OptTensor& vc, at::Tensor& q, const std::vector<int64_t>& sizes,
+               double eps, double temp_coef, double temp_every, double diff, const std::vector<OptTensor>& at, const std::vector<double>& af,
+               const std::vector<int64_t>& an) {
+  c10::cuda::CUDAGuard g(proj.device());
+  TORCH_CHECK(sizes.size() == 5 && lvec.is_contiguous(), "diff_prep: 5 sizes, stacked vectors");
+  const MbDiffPrep L{static_cast<int>(sizes[0]), static_cast<int>(sizes[1]), static_cast<int>(sizes[2]), static_cast<int>(sizes[3]),
+                     static_cast<int>(sizes[4]), static_cast<float>(eps), static_cast<float>(temp_coef), temp_every, static_cast<float>(diff)};
+  check(mb_diff_prep(proj.data_ptr(), proj.stride(0), positions.data_ptr<int>(), lptr(slots), q_norm.data_ptr(), cptr(k_norm), lvec.data_ptr(),
+                     lam.data_ptr<float>(), mptr(kc), mptr(vc), q.data_ptr(), proj.size(0), L, aside(at, af, an), f32(proj), cur_stream()),
+        "mb_diff_prep");
+}
+
+void diff_combine(const at::Tensor& a, at::Tensor& out, int64_t heads, int64_t vdim, const OptTensor& lam, const OptTensor& gate, double gain, double eps) {
+  c10::cuda::CUDAGuard g(a.device());
+  check(mb_diff_combine(a.data_ptr<float>(), out.data_ptr(), out.stride(0), out.size(0), heads, vdim, difference(lam, gate, gain, eps), f32(out),
+                        cur_stream()),
+        "mb_diff_combine");
+}
+
+// sizes: heads, value size, state size, groups, taps; t: conv weight, conv bias, dt_bias, A_log, D, state, ring (or None), slots, positions
+inline MbSsm ssm(const std::vector<int64_t>& sizes, const std::vector<OptTensor>& t) {
+  TORCH_CHECK(sizes.size() == 5 && t.size() == 9, "a state-space mixer has 5 sizes and 9 tensors");
+  MbSsm m{};
+  m.H = sizes[0];
+  m.V = sizes[1];
+  m.N = sizes[2];
+  m.G = sizes[3];
+  m.taps = sizes[4];
+  m.conv_w = cptr(t[0]);
+  m.conv_b = cptr(t[1]);
+  m.dt_bias = cptr(t[2]);
+  m.A_log = cptr(t[3]);
+  m.D = cptr(t[4]);
+  m.state = fmut(t[5]);
+  m.ring = fmut(t[6]);
+  m.slots = iptr(t[7]);
+  m.positions = iptr(t[8]);
+  return m;
+}
+
+void ssm_conv(const at::Tensor& proj, const std::vector<int64_t>& sizes, const std::vector<OptTensor>& t, const OptTensor& tiles, const OptTensor& cu_q,
+              at::Tensor& xbc, at::Tensor& dt, at::Tensor& la, const std::vector<OptTensor>& at, const std::vector<double>& af,
+              const std::vector<int64_t>& an) {
+  c10::cuda::CUDAGuard g(proj.device());
+  const bool given = tiles.has_value() && tiles->defined();
+  check(mb_ssm_conv(proj.data_ptr(), proj.stride(0), ssm(sizes, t), iptr(tiles), iptr(cu_q), given ? tiles->size(0) : proj.size(0), xbc.data_ptr(),
+                    dt.data_ptr<float>(), la.data_ptr<float>(), proj.size(0), aside(at, af, an), f32(proj), cur_stream()),
+        "mb_ssm_conv");
+}
+
+void ssm_step(const at::Tensor& proj, const std::vector<int64_t>& sizes, const std::vector<OptTensor>& t, at::Tensor& out,
+              const std::vector<OptTensor>& at, const std::vector<double>& af, const std::vector<int64_t>& an) {
+  c10::cuda::CUDAGuard g(proj.device());
+  check(mb_ssm_step(proj.data_ptr(), proj.stride(0), ssm(sizes, t), out.data_ptr(), proj.size(0), aside(at, af, an), f32(proj), cur_stream()),
+        "mb_ssm_step");
+}
+
+void ssm_seq(const at::Tensor& proj, const at::Tensor& xbc, const at::Tensor& dt, const at::Tensor& la, const std::vector<int64_t>& sizes,
+             const std::vector<OptTensor>& t, const OptTensor& cu_q, at::Tensor& out) {
+  c10::cuda::CUDAGuard g(proj.device());
+  check(mb_ssm_seq(proj.data_ptr(), proj.stride(0), xbc.data_ptr(), dt.data_ptr<float>(), la.data_ptr<float>(), ssm(sizes, t), iptr(cu_q),
+                   out.data_ptr(), t[7]->numel(), f32(proj), cur_stream()),
+        "mb_ssm_seq");
+}
+
+void ssm_chunk(const at::Tensor& proj, const at::Tensor& xbc, const at::Tensor& dt, const at::Tensor& la, const std::vector<int64_t>& sizes,
+               const std::vector<OptTensor>& t, const at::Tensor& segs, const at::Tensor& seq_segs, const OptTensor& seg_state, const OptTensor& seg_decay,
+               at::Tensor& out) {
+  c10::cuda::CUDAGuard g(proj.device());
+  if (fptr(seg_state) != nullptr) mb_count_launch(2);
+  check(mb_ssm_chunk(proj.data_ptr(), proj.stride(0), xbc.data_ptr(), dt.data_ptr<float>(), la.data_ptr<float>(), ssm(sizes, t), segs.data_ptr<int>(),
+                     seq_segs.data_ptr<int>(), fmut(seg_state), fmut(seg_decay), out.data_ptr(), seq_segs.numel() - 1, segs.size(0), cur_stream()),
+        "mb_ssm_chunk");
+}
+#endif  // MB_HAS_HYBRID
 
 }  // namespace
 
@@ -302,10 +464,12 @@ void register_mixers(pybind11::module& m) {
   m.def("output_norm", &output_norm);
   m.def("gemv_output_norm", &gemv_output_norm);
   m.def("clamped_glu", &clamped_glu, pybind11::arg("in"), pybind11::arg("out"), pybind11::arg("limit"), pybind11::arg("alpha"),
-        pybind11::arg("rows") = pybind11::none());
+        pybind11::arg("rows") = pybind11::none(), pybind11::arg("shift") = 1.0);
   m.def("sum_norm", &sum_norm);
   m.def("gemv_sum_norm", &gemv_sum_norm);
   m.def("gated_norm", &gated_norm);
+  m.def("relu_square", &relu_square, pybind11::arg("x"), pybind11::arg("rows") = pybind11::none());
+  m.def("part_norm", &part_norm);
 #ifdef MB_HAS_LATENT
   m.def("latent_prep", &latent_prep);
   m.def("head_linear", &head_linear);
@@ -317,11 +481,27 @@ void register_mixers(pybind11::module& m) {
   m.def("linear_state", &linear_state);
   m.def("linear_chunk", &linear_chunk);
 #endif
-#ifdef MB_HAS_ATTENTION
+#ifdef MB_HAS_WINDOW
   m.def("window_prep", &window_prep);
-  m.def("window_decode", &window_decode);
+#endif
+#ifdef MB_HAS_HYBRID
+  m.def("diff_prep", &diff_prep);
+  m.def("diff_combine", &diff_combine);
+  m.def("ssm_conv", &ssm_conv);
+  m.def("ssm_step", &ssm_step);
+  m.def("ssm_seq", &ssm_seq);
+  m.def("ssm_chunk", &ssm_chunk);
+  m.def("ssm_heads_per_cta", &mb_ssm_heads_per_cta);
+#endif
+#ifdef MB_HAS_ATTENTION
+  m.def("window_decode", &window_decode, pybind11::arg("q"), pybind11::arg("kc"), pybind11::arg("vc"), pybind11::arg("block_table"), pybind11::arg("token_seq"), pybind11::arg("positions"),
+        pybind11::arg("slots"), pybind11::arg("sink"), pybind11::arg("out"), pybind11::arg("scale"), pybind11::arg("splits"), pybind11::arg("lay"),
+        pybind11::arg("lam") = pybind11::none(), pybind11::arg("gate") = pybind11::none(), pybind11::arg("gain") = 0.0, pybind11::arg("eps") = 0.0);
   m.def("window_attend", &window_attend);
-  m.def("window_prefill", &window_prefill);
-  m.def("experts_any", &experts_any);
+  m.def("window_prefill", &window_prefill, pybind11::arg("q"), pybind11::arg("kc"), pybind11::arg("vc"), pybind11::arg("out"), pybind11::arg("sink"), pybind11::arg("cu_q"), pybind11::arg("positions"),
+        pybind11::arg("block_table"), pybind11::arg("n_seq"), pybind11::arg("max_q"), pybind11::arg("t_long"), pybind11::arg("scale"), pybind11::arg("lay"), pybind11::arg("err"),
+        pybind11::arg("lam") = pybind11::none(), pybind11::arg("gate") = pybind11::none(), pybind11::arg("gain") = 0.0, pybind11::arg("eps") = 0.0);
+  m.def("experts_any", &experts_any, pybind11::arg("x"), pybind11::arg("w13"), pybind11::arg("w2"), pybind11::arg("index"), pybind11::arg("weights"),
+        pybind11::arg("act"), pybind11::arg("out"), pybind11::arg("limit"), pybind11::arg("alpha"), pybind11::arg("shift") = 1.0);
 #endif
 }

@@ -1,4 +1,4 @@
-// Routed clamped experts of any size (bf16 or float) without sorting: one row of activations per (token, choice), then one output row
+// Routed experts (clamped gated ones, or ungated ones with the square of relu) of any size (bf16 or float) without sorting: one row of activations per (token, choice), then one output row
 // per token.  The form of 32-bit runs and of sizes the tensor-core kernels do not take; every weight row is read by one warp.
 #include "mixers.cuh"
 
@@ -7,10 +7,11 @@ namespace mx {
 
 static constexpr int kExp = 256;
 
-// act[pair, f] = clamped_glu(W13[e][f]·x, W13[e][F + f]·x).  grid (pairs, feature blocks of 8 warps)
+// act[pair, f] = clamped_glu(W13[e][f]·x, W13[e][F + f]·x), or with alpha = 0 relu(W13[e][f]·x)² of [E, F, H] experts.  grid (pairs, feature blocks of 8 warps)
 template <typename T>
 __global__ void __launch_bounds__(kExp) experts_up_kernel(const T* __restrict__ x, const T* __restrict__ w13, const int* __restrict__ index,
-                                                          T* __restrict__ act, int k, int E, int H, int F, float limit, float alpha) {
+                                                          T* __restrict__ act, int k, int E, int H, int F, float limit, float alpha,
+                                                          float shift) {
   extern __shared__ float xs[];
   pdl_trigger();
   pdl_wait();
@@ -21,16 +22,17 @@ __global__ void __launch_bounds__(kExp) experts_up_kernel(const T* __restrict__ 
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int f = blockIdx.y * (kExp / 32) + warp; f < F; f += gridDim.y * (kExp / 32)) {
-    const T* g = w13 + (static_cast<long long>(e) * 2 * F + f) * H;
-    const T* u = g + static_cast<long long>(F) * H;
+    const bool gated = alpha != 0.f;
+    const T* g = w13 + (static_cast<long long>(e) * (gated ? 2 : 1) * F + f) * H;
+    const T* u = gated ? g + static_cast<long long>(F) * H : g;
     float a = 0.f, b = 0.f;
     for (int i = lane; i < H; i += 32) {
       a = fmaf(to_f(g[i]), xs[i], a);
-      b = fmaf(to_f(u[i]), xs[i], b);
+      if (gated) b = fmaf(to_f(u[i]), xs[i], b);
     }
     a = warp_sum(a);
     b = warp_sum(b);
-    if (lane == 0) act[pair * F + f] = from_f<T>(clamped_glu_t<T>(a, b, limit, alpha));
+    if (lane == 0) act[pair * F + f] = from_f<T>(gated ? clamped_glu_t<T>(a, b, limit, alpha, shift) : relu_square(a));
   }
 }
 
@@ -64,9 +66,9 @@ __global__ void __launch_bounds__(kExp) experts_down_kernel(const T* __restrict_
 using namespace mb;
 using namespace mb::mx;
 
-// x [T, H], w13 [E, 2F, H], w2 [E, H, F], index / weights [T, k]; act [T·k, F] scratch, out [T, H]
+// x [T, H], w13 [E, 2F, H] (alpha 0: [E, F, H]), w2 [E, H, F], index / weights [T, k]; act [T·k, F] scratch, out [T, H]
 extern "C" int mb_experts_any(const void* x, const void* w13, const void* w2, const int* index, const float* weights, void* act, void* out, int T,
-                              int k, int E, int H, int F, float limit, float alpha, int f32, cudaStream_t s) {
+                              int k, int E, int H, int F, float limit, float alpha, float shift, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
   if (H > 12288 || k <= 0) return -3;
   auto run = [&](auto ty) {
@@ -74,7 +76,7 @@ extern "C" int mb_experts_any(const void* x, const void* w13, const void* w2, co
     const int fb = (F + 7) / 8 < 64 ? (F + 7) / 8 : 64, hb = (H + 7) / 8 < 64 ? (H + 7) / 8 : 64;
     cudaError_t e = launch_pdl(experts_up_kernel<P>, dim3(static_cast<unsigned>(T) * k, fb), dim3(kExp), H * sizeof(float), s,
                                reinterpret_cast<const P*>(x), reinterpret_cast<const P*>(w13), index, reinterpret_cast<P*>(act), k, E, H, F, limit,
-                               alpha);
+                               alpha, shift);
     if (e == cudaSuccess)
       e = launch_pdl(experts_down_kernel<P>, dim3(T, hb), dim3(kExp), 0, s, reinterpret_cast<const P*>(act), reinterpret_cast<const P*>(w2), index,
                      weights, reinterpret_cast<P*>(out), k, E, H, F);

@@ -15,7 +15,7 @@
 //     permutation of k.   lane = 4·g + t: A rows g and g+8, k ∈ [32c + 8t, 32c + 8t + 8); B column (token) g, same k.
 //
 //   gemv            y[M, N] = norm?(x (+ residual)) · W[N, K]ᵀ (+ bias)       M ≤ 16; optional fused add + RMSNorm prologue
-//   moe_gemv_up     act[pair, F] = silu(W13[e][:F] x) · (W13[e][F:] x), or the clamped form of mixers.cuh
+//   moe_gemv_up     act[pair, F] = silu(W13[e][:F] x) · (W13[e][F:] x), or the clamped form of mixers.cuh, or relu(W1[e] x)²
 //                   per distinct expert of the step, T ≤ 8 tokens
 //   moe_gemv_down   out[T, H] = Σ_experts gate_w · W2[e] · act                 accumulated over experts in registers
 #include <cuda_bf16.h>
@@ -210,11 +210,12 @@ __device__ __forceinline__ void stage_rows_output_norm(uint8_t* xs, int rows, in
   }
 }
 
-// Sum-norm form: x' = x + y1 + y2 + extra (fp32 x and extra, every addend optional; block 0 writes x' to x_out, another buffer); the
-// staged value is bf16(x' · norm_w), Σx'² → rstd[row].
+// Sum-norm form: x' = x + y1·s1 + y2·s2 + extra (fp32 x and extra, every addend and scale optional; block 0 writes x' to x_out, another
+// buffer); the staged value is bf16(x' · (norm_w + shift)), Σx'² → rstd[row].
 __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int valid, int K, const float* __restrict__ x,
-                                                    const bf16* __restrict__ y1, const bf16* __restrict__ y2, const float* __restrict__ extra,
-                                                    const bf16* __restrict__ norm_w, float eps, float* x_out, float* rstd) {
+                                                    const bf16* __restrict__ y1, const bf16* __restrict__ s1, const bf16* __restrict__ y2,
+                                                    const bf16* __restrict__ s2, const float* __restrict__ extra,
+                                                    const bf16* __restrict__ norm_w, float eps, float shift, float* x_out, float* rstd) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nv = K / 8, stride = staged_stride(K);
   for (int r = warp; r < rows; r += kWarps) {
@@ -231,9 +232,11 @@ __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int v
       const long long at = base + v * 8;
       float f[8];
       const float4 a = *reinterpret_cast<const float4*>(x + at), b = *reinterpret_cast<const float4*>(x + at + 4);
-      const uint4 zero = make_uint4(0, 0, 0, 0);
+      const uint4 zero = make_uint4(0, 0, 0, 0), one = make_uint4(0x3f803f80u, 0x3f803f80u, 0x3f803f80u, 0x3f803f80u);
       const uint4 p1 = y1 != nullptr ? *reinterpret_cast<const uint4*>(y1 + at) : zero;
       const uint4 p2 = y2 != nullptr ? *reinterpret_cast<const uint4*>(y2 + at) : zero;
+      const uint4 q1 = s1 != nullptr ? *reinterpret_cast<const uint4*>(s1 + v * 8) : one;
+      const uint4 q2 = s2 != nullptr ? *reinterpret_cast<const uint4*>(s2 + v * 8) : one;
       const uint4 nw = *reinterpret_cast<const uint4*>(norm_w + v * 8);
       f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
       if (extra != nullptr) {
@@ -241,14 +244,15 @@ __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int v
         f[0] += c.x; f[1] += c.y; f[2] += c.z; f[3] += c.w; f[4] += d.x; f[5] += d.y; f[6] += d.z; f[7] += d.w;
       }
       const uint32_t w1[4] = {p1.x, p1.y, p1.z, p1.w}, w2[4] = {p2.x, p2.y, p2.z, p2.w}, wn[4] = {nw.x, nw.y, nw.z, nw.w};
+      const uint32_t l1[4] = {q1.x, q1.y, q1.z, q1.w}, l2[4] = {q2.x, q2.y, q2.z, q2.w};
       uint32_t o[4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float2 u = unpack2(w1[i]), q = unpack2(w2[i]), n = unpack2(wn[i]);
-        f[2 * i] += u.x + q.x;
-        f[2 * i + 1] += u.y + q.y;
+        const float2 u = unpack2(w1[i]), q = unpack2(w2[i]), n = unpack2(wn[i]), c = unpack2(l1[i]), d = unpack2(l2[i]);
+        f[2 * i] += u.x * c.x + q.x * d.x;
+        f[2 * i + 1] += u.y * c.y + q.y * d.y;
         ss += f[2 * i] * f[2 * i] + f[2 * i + 1] * f[2 * i + 1];
-        o[i] = pack2(f[2 * i] * n.x, f[2 * i + 1] * n.y);
+        o[i] = pack2(f[2 * i] * (n.x + shift), f[2 * i + 1] * (n.y + shift));
       }
       if (x_out != nullptr && blockIdx.x == 0) {
         *reinterpret_cast<float4*>(x_out + at) = make_float4(f[0], f[1], f[2], f[3]);
@@ -290,11 +294,15 @@ struct GemvParams {
   const float* x32;       // output-norm form: fp32 residual, layer scale, and where the new residual goes
   const bf16* scale_w;
   float* x32_out;
-  const bf16 *y1, *y2;    // sum-norm form: sublayer outputs and an fp32 addend
+  const bf16 *y1, *s1, *y2, *s2;   // sum-norm form: sublayer outputs with their scales, an fp32 addend, what norm weights count from
   const float* extra;
-  const bf16* W2;         // a second weight [N2, K] behind the first: fp32 y2out[M, N2] (+ bias2)
+  float shift;
+  const bf16* norm_w2;    // norm weight of the second product's rows (null: the first one's)
+  const bf16* W2;         // a second weight [N2, K] behind the first: y2out[M, N2] (+ bias2), fp32 or bf16
   const bf16* bias2;
-  float* y2out;
+  void* y2out;
+  long long ld2;
+  int out2_fp32;
   int N2;
   int M, N, K;
   int static_w;           // W is not written by a kernel that may still run: its first loads go before the dependency wait
@@ -342,7 +350,8 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   } else if (MODE == kOutputNorm) {
     stage_rows_output_norm(xs, NT * 8, p.M, p.K, p.x, p.x32, p.norm_w, p.scale_w, p.eps, p.x32_out);
   } else if (MODE == kSumNorm) {
-    stage_rows_sum_norm(xs, NT * 8, p.M, p.K, p.x32, p.y1, p.y2, p.extra, p.norm_w, p.eps, p.x32_out, rstd_s);
+    stage_rows_sum_norm(xs, NT * 8, p.M, p.K, p.x32, p.y1, p.s1, p.y2, p.s2, p.extra, second && p.norm_w2 != nullptr ? p.norm_w2 : p.norm_w, p.eps,
+                        p.shift, p.x32_out, rstd_s);
   } else {
     stage_rows_async(xs, NT * 8, p.M, p.K, p.x);
     cp_commit();
@@ -381,7 +390,8 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
       if (SCALED) s *= rstd_s[tok];
       if (second) {
         if (p.bias2 != nullptr) s += __bfloat162float(p.bias2[n]);
-        p.y2out[static_cast<long long>(tok) * p.N2 + n] = s;
+        if (p.out2_fp32) reinterpret_cast<float*>(p.y2out)[tok * p.ld2 + n] = s;
+        else reinterpret_cast<bf16*>(p.y2out)[tok * p.ld2 + n] = __float2bfloat16(s);
         continue;
       }
       if (p.bias != nullptr) s += __bfloat162float(p.bias[n]);
@@ -395,8 +405,10 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
       const int tok = i / (p.K / 8), kv = (i % (p.K / 8)) * 8;
       const long long at = static_cast<long long>(tok) * p.K + kv;
       const float4 a = *reinterpret_cast<const float4*>(xr + at), b = *reinterpret_cast<const float4*>(xr + at + 4);
-      const uint4 nw = *reinterpret_cast<const uint4*>(p.norm_w + kv);
-      const float2 n0w = unpack2(nw.x), n1w = unpack2(nw.y), n2w = unpack2(nw.z), n3w = unpack2(nw.w);
+      const uint4 nw = *reinterpret_cast<const uint4*>((p.norm_w2 != nullptr ? p.norm_w2 : p.norm_w) + kv);
+      float2 n0w = unpack2(nw.x), n1w = unpack2(nw.y), n2w = unpack2(nw.z), n3w = unpack2(nw.w);
+      n0w.x += p.shift; n0w.y += p.shift; n1w.x += p.shift; n1w.y += p.shift;
+      n2w.x += p.shift; n2w.y += p.shift; n3w.x += p.shift; n3w.y += p.shift;
       const float r = rstd_s[tok];
       *reinterpret_cast<uint4*>(p.xn_out + at) = make_uint4(pack2(a.x * r * n0w.x, a.y * r * n0w.y), pack2(a.z * r * n1w.x, a.w * r * n1w.y),
                                                             pack2(b.x * r * n2w.x, b.y * r * n2w.y), pack2(b.z * r * n3w.x, b.w * r * n3w.y));
@@ -451,13 +463,14 @@ __device__ __forceinline__ int pair_of(unsigned long long mask, int tok, int k) 
   return m ? tok * k + __ffsll(static_cast<long long>(m)) - 1 : -1;
 }
 
-// Persistent grid over (distinct expert, block of 8 features): an item computes gate rows f0..f0+7 and up rows F+f0..F+f0+7
-// of the expert for all tokens and stores silu(gate) · up for the tokens routed to it.  A warp's weight stream runs
+// Persistent grid over (distinct expert, block of features).  GATED: 8 features, gate rows f0..f0+7 and up rows F+f0..F+f0+7 of the expert
+// for all tokens, silu(gate) · up (or its clamped form) stored for the tokens routed to it.  Otherwise 16 rows of a [F, H] expert, relu(·)².  A warp's weight stream runs
 // across its items without a break (the ring keeps filling while the CTA reduces and stores an item).
+template <bool GATED>
 __global__ void __launch_bounds__(kThreads) moe_gemv_up_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w13,
                                                                const int* __restrict__ topk_idx, bf16* __restrict__ act, int T, int k,
-                                                               int E, int offset, int H, int F, float limit, float alpha) {
-  constexpr int S = kMoeStages;
+                                                               int E, int offset, int H, int F, float limit, float alpha, float shift) {
+  constexpr int S = kMoeStages, kFeat = GATED ? 8 : 16;
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float red[kWarps][16][8];
   __shared__ int slot_e[kMaxPairs];
@@ -499,7 +512,7 @@ __global__ void __launch_bounds__(kThreads) moe_gemv_up_kernel(const bf16* __res
   cp_commit();
   cp_wait<0>();
   __syncthreads();
-  const int nfb = F / 8;
+  const int nfb = F / kFeat;
   const int n_items = n_slots_s * nfb;
   const int n_mine = n_items > static_cast<int>(blockIdx.x) ? (n_items - blockIdx.x + gridDim.x - 1) / gridDim.x : 0;
   const int chunks = H / 32;
@@ -508,11 +521,11 @@ __global__ void __launch_bounds__(kThreads) moe_gemv_up_kernel(const bf16* __res
   const int stride = staged_stride(H);
   // the copies are issued in stream order, so the (item, chunk) cursor advances incrementally: no division per copy
   int i_u = 0, i_item = blockIdx.x;
-  const long long up_off = static_cast<long long>(F) * H;
+  const long long up_off = static_cast<long long>(GATED ? F : 8) * H;
   const bf16* i_base = nullptr;
   auto set_item = [&]() {
     if (i_item < n_items)
-      i_base = w13 + static_cast<long long>(slot_e[i_item / nfb]) * 2 * F * H + static_cast<long long>((i_item % nfb) * 8 + g) * H + t * 8;
+      i_base = w13 + static_cast<long long>(slot_e[i_item / nfb]) * (GATED ? 2 : 1) * F * H + static_cast<long long>((i_item % nfb) * kFeat + g) * H + t * 8;
   };
   set_item();
   auto issue = [&](int q) {
@@ -529,7 +542,7 @@ __global__ void __launch_bounds__(kThreads) moe_gemv_up_kernel(const bf16* __res
   int q = 0;
   for (int j = 0; j < n_mine; ++j) {
     const int item = blockIdx.x + j * gridDim.x;
-    const int s = item / nfb, f0 = (item % nfb) * 8;
+    const int s = item / nfb, f0 = (item % nfb) * kFeat;
     float c[4] = {};
     for (int u = 0; u < cpw; ++u, ++q) {
       cp_wait<S - 1>();
@@ -544,20 +557,22 @@ __global__ void __launch_bounds__(kThreads) moe_gemv_up_kernel(const bf16* __res
     red[warp][g + 8][2 * t] = c[2];
     red[warp][g + 8][2 * t + 1] = c[3];
     __syncthreads();
-    if (threadIdx.x < 64) {
-      const int f = threadIdx.x & 7, tok = threadIdx.x >> 3;
+    if (threadIdx.x < 8 * kFeat) {
+      const int f = threadIdx.x & (kFeat - 1), tok = threadIdx.x / kFeat;
       const int pair = tok < T ? pair_of(slot_mask[s], tok, k) : -1;
       if (pair >= 0) {
         float gate = 0.f, up = 0.f;
 #pragma unroll
         for (int w = 0; w < kWarps; ++w) {
           gate += red[w][f][tok];
-          up += red[w][f + 8][tok];
+          if (GATED) up += red[w][f + 8][tok];
         }
-        // the two halves are rounded to bf16 first, like the stored pre-activation of the general path
+        // the sums are rounded to bf16 first, like the stored pre-activation of the general path
         gate = __bfloat162float(__float2bfloat16(gate));
         up = __bfloat162float(__float2bfloat16(up));
-        const float a = alpha != 0.f ? mx::clamped_glu_t<bf16>(gate, up, limit, alpha) : gate / (1.f + __expf(-gate)) * up;
+        float a;
+        if (!GATED) a = mx::relu_square(gate);
+        else a = alpha != 0.f ? mx::clamped_glu_t<bf16>(gate, up, limit, alpha, shift) : gate / (1.f + __expf(-gate)) * up;
         act[static_cast<long long>(pair) * F + f0 + f] = __float2bfloat16(a);
       }
     }
@@ -758,38 +773,42 @@ extern "C" int mb_gemv_output_norm(const float* x, const void* y, const void* no
 }
 
 // See launch.h; same limits as mb_gemv.
-extern "C" int mb_gemv_sum_norm(const float* x32, const void* y1, const void* y2, const float* extra, const void* x, const void* norm_w, float eps,
-                                const void* W, void* y, long long ldy, const void* W2, const void* bias2, float* out2, float* x_out, void* xn_out,
-                                int M, int N, int N2, int K, int static_w, cudaStream_t s) {
-  if (M <= 0 || N <= 0) return 0;
-  if (M > 16 || K % 32 || K <= 0) return -1;
-  const int nt = M <= 8 ? 1 : 2;
-  if (kDenseStages * 2 * kThreads * 16 + nt * 8 * staged_stride(K) > kMaxSmem) return -2;
+extern "C" int mb_gemv_sum_norm(MbGemvSum a, cudaStream_t s) {
+  if (a.M <= 0 || a.N <= 0) return 0;
+  if (a.M > 16 || a.K % 32 || a.K <= 0) return -1;
+  const int nt = a.M <= 8 ? 1 : 2;
+  if (kDenseStages * 2 * kThreads * 16 + nt * 8 * staged_stride(a.K) > kMaxSmem) return -2;
+  auto b = [](const void* p) { return reinterpret_cast<const bf16*>(p); };
   GemvParams p{};
-  p.x = reinterpret_cast<const bf16*>(x);
-  p.x32 = x32;
-  p.y1 = reinterpret_cast<const bf16*>(y1);
-  p.y2 = reinterpret_cast<const bf16*>(y2);
-  p.extra = extra;
-  p.norm_w = reinterpret_cast<const bf16*>(norm_w);
-  p.eps = eps;
-  p.W = reinterpret_cast<const bf16*>(W);
-  p.y = y;
-  p.ldy = ldy;
-  p.W2 = reinterpret_cast<const bf16*>(W2);
-  p.bias2 = reinterpret_cast<const bf16*>(bias2);
-  p.y2out = out2;
-  p.N2 = W2 != nullptr ? N2 : 0;
-  p.x32_out = x_out;
-  p.xn_out = reinterpret_cast<bf16*>(xn_out);
-  p.M = M; p.N = N; p.K = K; p.static_w = static_w;
-  if (x32 == nullptr) return static_cast<int>(nt == 1 ? launch_gemv<1, kPlain>(p, s) : launch_gemv<2, kPlain>(p, s));
+  p.x = b(a.x);
+  p.x32 = a.x32;
+  p.y1 = b(a.y1); p.s1 = b(a.s1);
+  p.y2 = b(a.y2); p.s2 = b(a.s2);
+  p.extra = a.extra;
+  p.norm_w = b(a.norm_w);
+  p.norm_w2 = b(a.norm_w2);
+  p.eps = a.eps;
+  p.shift = a.shift;
+  p.W = b(a.W);
+  p.y = a.y;
+  p.ldy = a.ldy;
+  p.W2 = b(a.W2);
+  p.bias2 = b(a.bias2);
+  p.y2out = a.out2;
+  p.ld2 = a.ld2;
+  p.out2_fp32 = a.out2_fp32;
+  p.N2 = a.W2 != nullptr ? a.N2 : 0;
+  p.x32_out = a.x_out;
+  p.xn_out = reinterpret_cast<bf16*>(a.xn_out);
+  p.M = a.M; p.N = a.N; p.K = a.K; p.static_w = a.static_w;
+  if (a.x32 == nullptr) return static_cast<int>(nt == 1 ? launch_gemv<1, kPlain>(p, s) : launch_gemv<2, kPlain>(p, s));
   return static_cast<int>(nt == 1 ? launch_gemv<1, kSumNorm>(p, s) : launch_gemv<2, kSumNorm>(p, s));
 }
 
-// MoE FFN for T ≤ 8 tokens (T·k ≤ 64): act [T·k, F] scratch, out [T, H].  alpha ≠ 0: clamped activation, else SwiGLU.  H and F multiples of 32, H a multiple of 16.
+// MoE FFN for T ≤ 8 tokens (T·k ≤ 64): act [T·k, F] scratch, out [T, H].  alpha ≠ 0: clamped activation, else SwiGLU; ungated:
+// w13 is [E, F, H], the activation relu(·)².  H and F multiples of 32, H a multiple of 16.
 extern "C" int mb_moe_gemv(const void* x, const void* w13, const void* w2, const int* topk_idx, const float* topk_w, void* act, void* out,
-                           int T, int k, int E, int expert_offset, int H, int F, float limit, float alpha, cudaStream_t s) {
+                           int T, int k, int E, int expert_offset, int H, int F, float limit, float alpha, float shift, int ungated, cudaStream_t s) {
   if (T <= 0) return 0;
   if (T > 8 || T * k > kMaxPairs || H % 32 || F % 32) return -1;
   const int ring_bytes = kMoeStages * 2 * kThreads * 16;
@@ -798,15 +817,17 @@ extern "C" int mb_moe_gemv(const void* x, const void* w13, const void* w2, const
   if (up_bytes > kMaxSmem || down_bytes > kMaxSmem) return -2;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = set_smem(moe_gemv_up_kernel, kMaxSmem);
+    cudaError_t e = set_smem(moe_gemv_up_kernel<true>, kMaxSmem);
+    if (e == cudaSuccess) e = set_smem(moe_gemv_up_kernel<false>, kMaxSmem);
     if (e == cudaSuccess) e = set_smem(moe_gemv_down_kernel, kMaxSmem);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
-  const int max_items = (T * k < E ? T * k : E) * (F / 8);
+  const int max_items = (T * k < E ? T * k : E) * (F / (ungated ? 16 : 8));
   const int up_grid = max_items < 2 * 148 ? max_items : 2 * 148;
-  cudaError_t e = launch_pdl(moe_gemv_up_kernel, dim3(up_grid), dim3(kThreads), up_bytes, s, reinterpret_cast<const bf16*>(x),
-                             reinterpret_cast<const bf16*>(w13), topk_idx, reinterpret_cast<bf16*>(act), T, k, E, expert_offset, H, F, limit, alpha);
+  cudaError_t e = launch_pdl(ungated ? moe_gemv_up_kernel<false> : moe_gemv_up_kernel<true>, dim3(up_grid), dim3(kThreads), up_bytes, s, reinterpret_cast<const bf16*>(x),
+                             reinterpret_cast<const bf16*>(w13), topk_idx, reinterpret_cast<bf16*>(act), T, k, E, expert_offset, H, F, limit, alpha,
+                             shift);
   if (e != cudaSuccess) return static_cast<int>(e);
   e = launch_pdl(moe_gemv_down_kernel, dim3(H / 16), dim3(kThreads), down_bytes, s, reinterpret_cast<const bf16*>(act),
                  reinterpret_cast<const bf16*>(w2), topk_idx, topk_w, reinterpret_cast<bf16*>(out), T, k, E, expert_offset, H, F);

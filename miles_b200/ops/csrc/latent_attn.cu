@@ -175,5 +175,5 @@ extern "C" int mb_latent_attend(const void* q, const void* cache, const int* blo
   a.o_row = static_cast<long long>(L.heads) * L.rank;
   a.window = window;
   a.scale = scale;
-  return mb_paged_attend(q, cache, cache, block_table, max_blocks, block_size, token_seq, positions, slots, sink, out, T, a, f32, s);
+  return mb_paged_attend(q, cache, cache, block_table, max_blocks, block_size, token_seq, positions, slots, sink, out, T, a, f32, 0, s);
 }

@@ -31,7 +31,7 @@ int mb_gemm_small_grouped(const void* X, const void* W, void* C, int rows, int N
 int mb_gemv(const void* x, const void* residual, const void* norm_w, float eps, const void* W, const void* bias, void* y, long long ldy,
             int out_fp32, void* res_out, void* xn_out, int M, int N, int K, int static_w, cudaStream_t s);
 int mb_moe_gemv(const void* x, const void* w13, const void* w2, const int* topk_idx, const float* topk_w, void* act, void* out, int T, int k,
-                int E, int expert_offset, int H, int F, float limit, float alpha, cudaStream_t s);
+                int E, int expert_offset, int H, int F, float limit, float alpha, float shift, int ungated, cudaStream_t s);
 int mb_gemm_bf16_grouped_wgrad(const void* dY, const void* X, void* dW, int M_pad, int N, int K, int num_experts,
                                const int* seg_offsets, int out_fp32, int accumulate, int force_bn, int* error_flag,
                                cudaStream_t stream);
@@ -206,15 +206,20 @@ int mb_multi_copy2d(const long long* table, const long long* prefix, int n, long
 int mb_multi_mxfp8(const long long* table, const long long* prefix, int n, long long total_chunks, int qdq, cudaStream_t s);
 
 // ---- mixers.cu (layer-by-layer decoders; f32: tensors of the model's dtype are float instead of bf16) ----
-// xb (the copy in the model's dtype) may be null
+// xb (the copy in the model's dtype) may be null; freq [D / 2 up] (optional): sines and cosines of positions · freq are added
 int mb_bigram_embedding(const int* tok, const int* prev, const void* embed, const void* table, long long buckets, long long mul_prev,
-                        long long mul_cur, float* x, void* xb, int T, int D, int f32, cudaStream_t s);
+                        long long mul_cur, const int* positions, const double* freq, float* x, void* xb, int T, int D, int f32, cudaStream_t s);
 int mb_output_norm(float* x, const void* y, const void* nw, const void* ls, const void* fw, void* xb, int T, int D, float eps, int f32,
                    cudaStream_t s);
 // rows (optional, device): rows in use
-int mb_clamped_glu(const void* in, long long ld_in, void* out, long long ld_out, long long T, int F, float limit, float alpha, const int* rows,
-                   int f32, cudaStream_t s);
-// s = x + y1 + y2 + Σ_j weights[t, j]·rows[dst[t, j]] + extra → to; h = rmsnorm(s)·nw (every pointer but x may be null)
+int mb_clamped_glu(const void* in, long long ld_in, void* out, long long ld_out, long long T, int F, float limit, float alpha, float shift,
+                   const int* rows, int f32, cudaStream_t s);
+// x ← max(x, 0)² (n values a row, rows of them or as many as the device count says)
+int mb_relu_square(void* x, long long T, int n, const int* rows, int f32, cudaStream_t s);
+// out = x / rms(x) · w, each of `parts` equal parts of a row by its own root mean square
+int mb_part_norm(const void* x, const void* w, void* out, int T, int C, int parts, float eps, int f32, cudaStream_t s);
+// s = x + y1·s1 + y2·s2 + s2·Σ_j weights[t, j]·rows[dst[t, j]] + extra → to; h = rmsnorm(s)·(nw + shift)·gain, h2 the same with nw2 (every
+// pointer but x may be null; a null scale is 1; at most one of y2 and rows where s2 is given)
 typedef struct {
   const float* x;
   float* to;
@@ -222,10 +227,11 @@ typedef struct {
   const float* weights;
   const int* dst;
   const float* extra;
-  const void* nw;
-  void* h;
+  const void *s1, *s2;
+  const void *nw, *nw2;
+  void *h, *h2;
   int T, D, k;
-  float eps;
+  float eps, shift, gain;
 } MbSumNorm;
 int mb_sum_norm(MbSumNorm p, int f32, cudaStream_t s);
 int mb_gated_norm(const void* o, const void* w, const void* gate, long long gate_ld, void* out, int T, int C, float eps, int f32,
@@ -233,11 +239,28 @@ int mb_gated_norm(const void* o, const void* w, const void* gate, long long gate
 // gemv.cu: output norm + layer scale + fp32 residual in front of a projection of ≤ 16 rows
 int mb_gemv_output_norm(const float* x, const void* y, const void* norm_w, const void* scale_w, float eps, const void* W, void* out,
                         long long ldo, float* x_out, int M, int N, int K, int static_w, cudaStream_t s);
-// gemv.cu: sum of an fp32 residual and up to two sublayer outputs, its norm, and up to two products of it, for ≤ 16 rows.  x32 null: plain
-// products of x [M, K].  W2 [N2, K] gives fp32 y2 (+ bias2).
-int mb_gemv_sum_norm(const float* x32, const void* y1, const void* y2, const float* extra, const void* x, const void* norm_w, float eps,
-                     const void* W, void* y, long long ldy, const void* W2, const void* bias2, float* out2, float* x_out, void* xn_out, int M,
-                     int N, int N2, int K, int static_w, cudaStream_t s);
+// gemv.cu: sum of an fp32 residual and up to two sublayer outputs (each times a scale vector, if given), its norm, and up to two products of
+// it, for ≤ 16 rows.  x32 null: plain products of x [M, K].  W2 [N2, K] gives out2 (+ bias2), fp32 or bf16; with norm_w2 its rows are the sum
+// normed by that weight.  Norm weights count from `shift`.  xn_out: the normed sum (by norm_w2 if there is one).
+typedef struct {
+  const float* x32;
+  const void *y1, *s1, *y2, *s2;
+  const float* extra;
+  const void* x;
+  const void *norm_w, *norm_w2;
+  float eps, shift;
+  const void* W;
+  void* y;
+  long long ldy;
+  const void *W2, *bias2;
+  void* out2;
+  long long ld2;
+  int out2_fp32;
+  float* x_out;
+  void* xn_out;
+  int M, N, N2, K, static_w;
+} MbGemvSum;
+int mb_gemv_sum_norm(MbGemvSum a, cudaStream_t s);
 // ---- paged_attend.cu ----
 typedef struct {
   int heads, group, dk, dv;                  // query head h uses key head h / group
@@ -245,9 +268,10 @@ typedef struct {
   int window, keep;                          // keys a token sees (0: all), first keys that stay visible
   float scale;
 } MbAttend;
+// out_f32: rows of floats whatever the dtype of the rest
 int mb_paged_attend(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size,
                     const int* token_seq, const int* positions, const long long* slots, const void* sink, void* out, int T, MbAttend A,
-                    int f32, cudaStream_t s);
+                    int f32, int out_f32, cudaStream_t s);
 // ---- window_prep.cu ----
 typedef struct {
   int heads, kv_heads, dim, vdim, rot, window, keep, q_pitch;   // q_pitch: elements per head of the prepared queries (zero-padded)
@@ -261,22 +285,74 @@ typedef struct {                             // what reads the same projection b
   void* glu_out;
   long long glu_ld_in, glu_ld_out;
   int ff;
-  float limit, alpha;
+  float limit, alpha, shift;
+  // grouped: choice by sigmoid scores plus `correction` (or null) among the `keep` best groups, weights from the scores times `scale`;
+  // else the largest logits, weights by their softmax
+  int grouped, groups, keep;
+  float scale;
+  const void* correction;
 } MbAside;
 int mb_window_prep(const void* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
                    const void* q_norm, const void* k_norm, float eps, void* kc, void* vc, void* q, int T, MbWindow L, MbAside a, int f32,
                    cudaStream_t s);
+// ---- diff_prep.cu (differential attention: two score maps per head over the same values) ----
+// Query heads 2h and 2h + 1 are the maps of head h; a key head is [map 1 | map 2], a query row has zeros in the other map's half, so that
+// the attention kernels see heads = 2·(query heads) of dim = 2·(map size).  What is left of a pair of outputs a1, a2:
+// o = a1 − lam·a2, o / rms(o) · gain · sigmoid(gate of the head).
+typedef struct {
+  const float* lam;                          // device scalar; null: ordinary attention
+  const void* gate;                          // [T, heads / 2] rows of gate_ld, before the sigmoid
+  long long gate_ld;
+  float gain, eps;
+} MbDiff;
+typedef struct {
+  int heads, kv_heads, dim, vdim, q_pitch;   // heads, dim: of the design (one map's size); kv_heads 0: keys and values of another layer
+  float eps, temp_coef;                      // queries times 1 + coef · ln(⌊(position + 1) / every⌋ + 1)
+  double temp_every;
+  float diff;
+} MbDiffPrep;
+// lvec: lq1, lk1, lq2, lk2 [4, dim]; lam ← exp(lq1·lk1) − exp(lq2·lk2) + diff
+int mb_diff_prep(const void* proj, long long ld, const int* positions, const long long* slots, const void* q_norm, const void* k_norm,
+                 const void* lvec, float* lam, void* kc, void* vc, void* q, int T, MbDiffPrep L, MbAside a, int f32, cudaStream_t s);
+// a [T, 2·heads, vdim] floats → out [T, heads·vdim] rows of o_row
+int mb_diff_combine(const float* a, void* out, long long o_row, int T, int heads, int vdim, MbDiff d, int f32, cudaStream_t s);
+// ---- ssm_*.cu (state-space mixer: S ← exp(−exp(A_log)·dt)·S + dt·B xᵀ, y = Sᵀ C + D·x) ----
+// A row of the projection is [z: H·V | x: H·V | B: G·N | C: G·N | dt: H]; x, B and C pass a causal convolution of `taps` columns and silu.
+typedef struct {
+  int H, V, N, G, taps;
+  const void *conv_w, *conv_b;               // [H·V + 2·G·N, taps], [H·V + 2·G·N]
+  const void *dt_bias, *A_log, *D;           // [H]
+  float* state;                              // [slots, H, N, V]
+  float* ring;                               // [slots, taps, channels]: the inputs of the last positions, by position mod taps (null: taps 1)
+  const int* slots;                          // per sequence
+  const int* positions;                      // per token
+} MbSsm;
+// Convolution, step sizes and log decays of any pieces.  tiles [n][4]: first token, end (32 tokens but for a piece's last tile), sequence, 1 for a
+// piece's first tile; null: one token per sequence.  xbc [T, channels], dt and la [T, H].
+int mb_ssm_conv(const void* proj, long long ld, MbSsm m, const int* tiles, const int* cu_q, int n_tiles, void* xbc, float* dt, float* la, int T,
+                MbAside a, int f32, cudaStream_t s);
+// One token per sequence: convolution, state, gate in one kernel; out [T, H·V] = y · silu(z).  V % 4 == 0.
+int mb_ssm_step(const void* proj, long long ld, MbSsm m, void* out, int B, MbAside a, int f32, cudaStream_t s);
+// Any pieces token by token (cu_q null: one token per sequence), from what mb_ssm_conv left.
+int mb_ssm_seq(const void* proj, long long ld, const void* xbc, const float* dt, const float* la, MbSsm m, const int* cu_q, void* out, int B,
+               int f32, cudaStream_t s);
+// Long pieces in chunks on tensor cores (bf16; N, V multiples of 8 up to 128).  segs, seq_segs as in mb_linear_chunk; seg_state [n_seg, H, N, V]
+// and seg_decay [n_seg, H] scratch, null when every sequence is one segment.
+int mb_ssm_chunk(const void* proj, long long ld, const void* xbc, const float* dt, const float* la, MbSsm m, const int* segs, const int* seq_segs,
+                 float* seg_state, float* seg_decay, void* out, int n_seq, int n_seg, cudaStream_t s);
+int mb_ssm_heads_per_cta(int H, int V, int G);
 // ---- window_decode.cu (bf16 tensor cores, splits joined inside a cluster) ----
 int mb_window_decode(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                      const int* positions, const long long* slots, const void* sink, void* out, long long o_row, int T, float scale, int splits,
-                     MbWindow L, cudaStream_t s);
+                     MbWindow L, MbDiff d, cudaStream_t s);
 // ---- attention_window_tc.cu (tcgen05, keys and values straight from the pages) ----
 int mb_window_prefill(const void* q, const void* kc, const void* vc, void* o, long long o_row, const void* sink, const int* cu_q,
                       const int* positions, const int* block_table, int max_blocks, int block_size, int num_blocks, int n_seq, int max_q,
-                      int t_long, float scale, MbWindow L, int* error_flag, cudaStream_t s);
+                      int t_long, float scale, MbWindow L, MbDiff d, int* error_flag, cudaStream_t s);
 // ---- experts_any.cu ----
+// alpha 0: w13 is [E, F, H] (no gate), the activation the square of relu
 int mb_experts_any(const void* x, const void* w13, const void* w2, const int* index, const float* weights, void* act, void* out, int T, int k,
-                   int E, int H, int F, float limit, float alpha, int f32, cudaStream_t s);
+                   int E, int H, int F, float limit, float alpha, float shift, int f32, cudaStream_t s);
 // ---- latent_attn.cu ----
 typedef struct {
   int heads, dim, rot, vdim, rank, rank_p, pitch;   // a cached row: [rank, 0 … rank_p, rot, 0 … pitch)

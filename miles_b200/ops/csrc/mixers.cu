@@ -11,12 +11,13 @@ namespace mx {
 
 static constexpr int kRow = 256;
 
-// x[t] = embed[tok] + table[(prev·mul_prev + tok·mul_cur) mod buckets]; the last row of the table for a sequence's first token
+// x[t] = embed[tok] + table[(prev·mul_prev + tok·mul_cur) mod buckets] (the last row of the table for a sequence's first token) + sines and
+// cosines of position · freq (pairs of neighbours share a frequency; angles in double precision, reduced by whole turns)
 template <typename T, int V>
 __global__ void __launch_bounds__(128) bigram_embed_kernel(const int* __restrict__ tok, const int* __restrict__ prev,
                                                            const T* __restrict__ embed, const T* __restrict__ table, long long buckets,
-                                                           long long mul_prev, long long mul_cur, float* __restrict__ x,
-                                                           T* __restrict__ xb, int D) {
+                                                           long long mul_prev, long long mul_cur, const int* __restrict__ positions,
+                                                           const double* __restrict__ freq, float* __restrict__ x, T* __restrict__ xb, int D) {
   pdl_trigger();
   pdl_wait();
   const long long t = blockIdx.x;
@@ -34,6 +35,16 @@ __global__ void __launch_bounds__(128) bigram_embed_kernel(const int* __restrict
       load_n<V>(table + row * D + i, b);
 #pragma unroll
       for (int j = 0; j < V; ++j) a[j] += b[j];
+    }
+    if (freq != nullptr) {
+      const double pos = positions[t];
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        double ang = pos * freq[(i + j) >> 1];
+        ang -= rint(ang * 0.15915494309189535) * 6.283185307179586;
+        if constexpr (is_exact<T>::value) a[j] += static_cast<float>(((i + j) & 1) ? cos(ang) : sin(ang));
+        else a[j] += ((i + j) & 1) ? __cosf(static_cast<float>(ang)) : __sinf(static_cast<float>(ang));
+      }
     }
     store_n<V>(x + t * D + i, a);
     if (xb != nullptr) store_n<V>(xb + t * D + i, a);
@@ -86,7 +97,8 @@ __global__ void __launch_bounds__(kRow) output_norm_kernel(float* __restrict__ x
 
 template <typename T, int V>
 __global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ in, long long ld_in, T* __restrict__ out, long long ld_out,
-                                                          long long n, int F, float limit, float alpha, const int* __restrict__ rows) {
+                                                          long long n, int F, float limit, float alpha, float shift,
+                                                          const int* __restrict__ rows) {
   pdl_trigger();
   pdl_wait();
   const int per = F / V;
@@ -98,8 +110,23 @@ __global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ 
     load_n<V>(in + t * ld_in + i, g);
     load_n<V>(in + t * ld_in + F + i, u);
 #pragma unroll
-    for (int j = 0; j < V; ++j) g[j] = clamped_glu_t<T>(g[j], u[j], limit, alpha);
+    for (int j = 0; j < V; ++j) g[j] = clamped_glu_t<T>(g[j], u[j], limit, alpha, shift);
     store_n<V>(out + t * ld_out + i, g);
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) relu_square_kernel(T* __restrict__ x, long long T_, int n, const int* __restrict__ rows) {
+  pdl_trigger();
+  pdl_wait();
+  if (rows != nullptr) T_ = min(T_, static_cast<long long>(*rows));
+  const long long total = T_ * n;
+  for (long long i = (blockIdx.x * 256ll + threadIdx.x) * V; i < total; i += gridDim.x * 256ll * V) {
+    float a[V];
+    load_n<V>(x + i, a);
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] = relu_square(a[j]);
+    store_n<V>(x + i, a);
   }
 }
 
@@ -116,8 +143,12 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
   const T* y1 = reinterpret_cast<const T*>(p.y1);
   const T* y2 = reinterpret_cast<const T*>(p.y2);
   const T* rows = reinterpret_cast<const T*>(p.rows);
+  const T* s1 = reinterpret_cast<const T*>(p.s1);
+  const T* s2 = reinterpret_cast<const T*>(p.s2);
   const T* nw = reinterpret_cast<const T*>(p.nw);
+  const T* nw2 = reinterpret_cast<const T*>(p.nw2);
   T* h = reinterpret_cast<T*>(p.h);
+  T* h2 = reinterpret_cast<T*>(p.h2);
   const int k = rows != nullptr ? p.k : 0;
   for (int j = threadIdx.x; j < k; j += kRow) {
     const int d = p.dst[t * p.k + j];
@@ -127,17 +158,21 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
   if (k > 0) __syncthreads();
   float ss = 0.f;
   for (int i = threadIdx.x * V; i < p.D; i += kRow * V) {
-    float r[V], a[V];
+    float r[V], a[V], c1[V], c2[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) c1[j] = c2[j] = 1.f;
+    if (s1 != nullptr) load_n<V>(s1 + i, c1);
+    if (s2 != nullptr) load_n<V>(s2 + i, c2);
     load_n<V>(p.x + base + i, r);
     if (y1 != nullptr) {
       load_n<V>(y1 + base + i, a);
 #pragma unroll
-      for (int j = 0; j < V; ++j) r[j] += a[j];
+      for (int j = 0; j < V; ++j) r[j] += a[j] * c1[j];
     }
     if (y2 != nullptr) {
       load_n<V>(y2 + base + i, a);
 #pragma unroll
-      for (int j = 0; j < V; ++j) r[j] += a[j];
+      for (int j = 0; j < V; ++j) r[j] += a[j] * c2[j];
     }
     if (k > 0) {
       float m[V];
@@ -153,7 +188,7 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
         for (int j = 0; j < V; ++j) m[j] = fmaf(w, a[j], m[j]);
       }
 #pragma unroll
-      for (int j = 0; j < V; ++j) r[j] += m[j];
+      for (int j = 0; j < V; ++j) r[j] += m[j] * c2[j];
     }
     if (p.extra != nullptr) {
       load_n<V>(p.extra + base + i, a);
@@ -173,8 +208,64 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
     load_n<V>(row + i, r);
     load_n<V>(nw + i, w);
 #pragma unroll
-    for (int j = 0; j < V; ++j) r[j] = r[j] * rstd * w[j];
-    store_n<V>(h + base + i, r);
+    for (int j = 0; j < V; ++j) {
+      r[j] *= rstd;
+      w[j] = r[j] * (w[j] + p.shift) * p.gain;
+    }
+    store_n<V>(h + base + i, w);
+    if (nw2 == nullptr) continue;
+    load_n<V>(nw2 + i, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) w[j] = r[j] * (w[j] + p.shift) * p.gain;
+    store_n<V>(h2 + base + i, w);
+  }
+}
+
+// out = x / rms(x) · w for every one of `parts` equal parts of a row; grid (rows, parts)
+template <typename T, int V>
+__global__ void __launch_bounds__(kRow) part_norm_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict__ out, int n, int parts,
+                                                         float eps) {
+  __shared__ float sh[kRow / 32];
+  constexpr int kHold = 4;                 // vectors per thread that stay in registers between the two passes
+  pdl_trigger();
+  pdl_wait();
+  const long long base = (static_cast<long long>(blockIdx.x) * parts + blockIdx.y) * n;
+  const T* pw = w + static_cast<long long>(blockIdx.y) * n;
+  float a[kHold][V], ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < kHold; ++u) {
+    const int i = (threadIdx.x + u * kRow) * V;
+    if (i < n) {
+      load_n<V>(x + base + i, a[u]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += a[u][j] * a[u][j];
+    }
+  }
+  for (int i = (threadIdx.x + kHold * kRow) * V; i < n; i += kRow * V) {
+    float b[V];
+    load_n<V>(x + base + i, b);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += b[j] * b[j];
+  }
+  const float rstd = rsqrt_exact(__fdiv_rn(block_sum<kRow>(ss, sh), static_cast<float>(n)) + eps);
+#pragma unroll
+  for (int u = 0; u < kHold; ++u) {
+    const int i = (threadIdx.x + u * kRow) * V;
+    if (i < n) {
+      float b[V];
+      load_n<V>(pw + i, b);
+#pragma unroll
+      for (int j = 0; j < V; ++j) b[j] *= a[u][j] * rstd;
+      store_n<V>(out + base + i, b);
+    }
+  }
+  for (int i = (threadIdx.x + kHold * kRow) * V; i < n; i += kRow * V) {
+    float b[V], c[V];
+    load_n<V>(x + base + i, b);
+    load_n<V>(pw + i, c);
+#pragma unroll
+    for (int j = 0; j < V; ++j) b[j] *= rstd * c[j];
+    store_n<V>(out + base + i, b);
   }
 }
 
@@ -219,13 +310,14 @@ using namespace mb;
 using namespace mb::mx;
 
 extern "C" int mb_bigram_embedding(const int* tok, const int* prev, const void* embed, const void* table, long long buckets,
-                                   long long mul_prev, long long mul_cur, float* x, void* xb, int T, int D, int f32, cudaStream_t s) {
+                                   long long mul_prev, long long mul_cur, const int* positions, const double* freq, float* x, void* xb, int T, int D,
+                                   int f32, cudaStream_t s) {
   if (T <= 0) return 0;
   return dispatch(f32, D % 8 == 0, [&](auto ty, auto v) {
     using E = decltype(ty);
     return static_cast<int>(launch_pdl(bigram_embed_kernel<E, decltype(v)::value>, dim3(T), dim3(128), 0, s, tok, prev,
-                                       reinterpret_cast<const E*>(embed), reinterpret_cast<const E*>(table), buckets, mul_prev, mul_cur, x,
-                                       reinterpret_cast<E*>(xb), D));
+                                       reinterpret_cast<const E*>(embed), reinterpret_cast<const E*>(table), buckets, mul_prev, mul_cur,
+                                       positions, freq, x, reinterpret_cast<E*>(xb), D));
   });
 }
 
@@ -241,7 +333,7 @@ extern "C" int mb_output_norm(float* x, const void* y, const void* nw, const voi
 }
 
 extern "C" int mb_clamped_glu(const void* in, long long ld_in, void* out, long long ld_out, long long T, int F, float limit, float alpha,
-                              const int* rows, int f32, cudaStream_t s) {
+                              float shift, const int* rows, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
   const bool vec = F % 8 == 0 && ld_in % 8 == 0 && ld_out % 8 == 0 && (reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
   return dispatch(f32, vec, [&](auto ty, auto v) {
@@ -249,7 +341,29 @@ extern "C" int mb_clamped_glu(const void* in, long long ld_in, void* out, long l
     constexpr int V = decltype(v)::value;
     const long long blocks = (T * (F / V) + 255) / 256;
     return static_cast<int>(launch_pdl(clamped_glu_kernel<E, V>, dim3(static_cast<unsigned>(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0,
-                                       s, reinterpret_cast<const E*>(in), ld_in, reinterpret_cast<E*>(out), ld_out, T, F, limit, alpha, rows));
+                                       s, reinterpret_cast<const E*>(in), ld_in, reinterpret_cast<E*>(out), ld_out, T, F, limit, alpha, shift, rows));
+  });
+}
+
+extern "C" int mb_relu_square(void* x, long long T, int n, const int* rows, int f32, cudaStream_t s) {
+  if (T <= 0) return 0;
+  return dispatch(f32, n % 8 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0, [&](auto ty, auto v) {
+    using E = decltype(ty);
+    constexpr int V = decltype(v)::value;
+    const long long blocks = (T * n / V + 255) / 256;
+    return static_cast<int>(launch_pdl(relu_square_kernel<E, V>, dim3(static_cast<unsigned>(blocks < 148 * 16 ? blocks + 1 : 148 * 16)), dim3(256), 0, s,
+                                       reinterpret_cast<E*>(x), T, n, rows));
+  });
+}
+
+extern "C" int mb_part_norm(const void* x, const void* w, void* out, int T, int C, int parts, float eps, int f32, cudaStream_t s) {
+  if (T <= 0) return 0;
+  if (parts <= 0 || C % parts || parts > 65535) return -3;
+  const int n = C / parts;
+  return dispatch(f32, n % 8 == 0, [&](auto ty, auto v) {
+    using E = decltype(ty);
+    return static_cast<int>(launch_pdl(part_norm_kernel<E, decltype(v)::value>, dim3(T, parts), dim3(kRow), 0, s, reinterpret_cast<const E*>(x),
+                                       reinterpret_cast<const E*>(w), reinterpret_cast<E*>(out), n, parts, eps));
   });
 }
 

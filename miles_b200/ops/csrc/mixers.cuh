@@ -127,11 +127,12 @@ __device__ __forceinline__ void rotary_table(float* cs, int position, const doub
   }
 }
 
-// gate · sigmoid(alpha · gate) · (up + 1) with gate ≤ limit and |up| ≤ limit
-template <typename T> __device__ __forceinline__ float clamped_glu_t(float gate, float up, float limit, float alpha) {
+// gate · sigmoid(alpha · gate) · (up + shift) with gate ≤ limit and |up| ≤ limit (limit ∞, alpha 1, shift 0: silu(gate) · up)
+template <typename T> __device__ __forceinline__ float clamped_glu_t(float gate, float up, float limit, float alpha, float shift) {
   const float a = fminf(gate, limit), b = fminf(fmaxf(up, -limit), limit);
-  return a * sigmoid_t<T>(alpha * a) * (b + 1.f);
+  return a * sigmoid_t<T>(alpha * a) * (b + shift);
 }
+__device__ __forceinline__ float relu_square(float v) { v = fmaxf(v, 0.f); return v * v; }
 
 // A float's bits in an order that integers compare: larger float, larger key.  NaN: 0, below everything.
 __device__ __forceinline__ uint32_t order_key(float v) {
@@ -185,6 +186,147 @@ __device__ __forceinline__ void topk_softmax_row(const float* __restrict__ z, in
     last_i = at;
   }
   for (int j = lane; j < K; j += 32) w[j] = sum > 0.f ? __fdiv_rn(w[j], sum) : 0.f;      // every lane reads back what it wrote
+}
+
+// One warp chooses the K largest of E choice scores σ(z) + correction among the experts of the `keep` best of `groups` equal groups of
+// neighbours (a group is worth the sum of its two largest choice scores), ties to the lower index, and weighs the chosen ones by their
+// σ(z) over the sum of those, times `scale`.  Index −1 with weight 0 where nothing is left to choose (NaNs).  groups ≤ 256.
+template <typename T>
+__device__ __forceinline__ void topk_grouped_row(const float* __restrict__ z, const T* __restrict__ correction, int E, int K, int groups, int keep,
+                                                 float scale, float* __restrict__ w, int* __restrict__ idx) {
+  constexpr int kLocal = 8;                      // keys (and groups) per lane that stay in registers
+  const int lane = threadIdx.x & 31, size = E / groups;
+  const bool local = E <= 32 * kLocal;
+  auto key_of = [&](int e) -> uint32_t { return order_key(sigmoid_t<T>(z[e]) + (correction != nullptr ? to_f(correction[e]) : 0.f)); };
+  uint32_t key[kLocal], open[kLocal];            // open: bit g of the groups whose experts can be chosen
+#pragma unroll
+  for (int i = 0; i < kLocal; ++i) {
+    key[i] = local && i * 32 + lane < E ? key_of(i * 32 + lane) : 0u;
+    open[i] = 0xffffffffu;
+  }
+  if (keep < groups) {
+    uint32_t worth[kLocal];                      // of group i·32 + lane
+#pragma unroll
+    for (int i = 0; i < kLocal; ++i) { worth[i] = 0u; open[i] = 0u; }
+    for (int g = 0; g < groups; ++g) {
+      uint32_t b1 = 0u, b2 = 0u;                 // the lane's two largest of the group
+      auto see = [&](uint32_t k) {
+        if (k > b1) { b2 = b1; b1 = k; }
+        else if (k > b2) b2 = k;
+      };
+      if (local) {
+#pragma unroll
+        for (int i = 0; i < kLocal; ++i) {
+          const int e = i * 32 + lane;
+          if (e >= g * size && e < (g + 1) * size) see(key[i]);
+        }
+      } else {
+        for (int e = g * size + lane; e < (g + 1) * size; e += 32) see(key_of(e));
+      }
+      const uint32_t top = __reduce_max_sync(0xffffffffu, b1);
+      const int owner = __ffs(__ballot_sync(0xffffffffu, b1 == top)) - 1;
+      const uint32_t second = __reduce_max_sync(0xffffffffu, lane == owner ? b2 : b1);
+      const uint32_t v = top == 0u ? 0u : order_key(key_value(top) + (second != 0u ? key_value(second) : 0.f));
+#pragma unroll
+      for (int i = 0; i < kLocal; ++i)
+        if (i * 32 + lane == g) worth[i] = v;
+    }
+    for (int j = 0; j < keep; ++j) {
+      uint32_t bk = 0u;
+      int bi = 0x7fffffff;
+#pragma unroll
+      for (int i = 0; i < kLocal; ++i)
+        if (worth[i] > bk) { bk = worth[i]; bi = i * 32 + lane; }
+      const uint32_t top = __reduce_max_sync(0xffffffffu, bk);
+      if (top == 0u) break;
+      const int at = __reduce_min_sync(0xffffffffu, bk == top ? bi : 0x7fffffff);
+#pragma unroll
+      for (int i = 0; i < kLocal; ++i) {
+        if (i * 32 + lane == at) worth[i] = 0u;
+        if ((at >> 5) == i) open[i] |= 1u << (at & 31);
+      }
+    }
+  }
+  auto is_open = [&](int e) -> bool {
+    const int g = e / size;
+    bool r = false;
+#pragma unroll
+    for (int i = 0; i < kLocal; ++i)
+      if ((g >> 5) == i) r = (open[i] >> (g & 31)) & 1u;
+    return r;
+  };
+  if (keep < groups && local) {
+#pragma unroll
+    for (int i = 0; i < kLocal; ++i)
+      if (i * 32 + lane < E && !is_open(i * 32 + lane)) key[i] = 0u;
+  }
+  uint32_t last = 0xffffffffu;
+  int last_i = -1;
+  float sum = 0.f;
+  for (int j = 0; j < K; ++j) {
+    uint32_t bk = 0u;
+    int bi = 0x7fffffff;
+    if (local) {
+#pragma unroll
+      for (int i = 0; i < kLocal; ++i)
+        if (key[i] > bk) { bk = key[i]; bi = i * 32 + lane; }
+    } else {
+      for (int e = lane; e < E; e += 32) {
+        const uint32_t k = is_open(e) ? key_of(e) : 0u;
+        if ((k < last || (k == last && e > last_i)) && k > bk) { bk = k; bi = e; }
+      }
+    }
+    const uint32_t top = __reduce_max_sync(0xffffffffu, bk);
+    const int at = __reduce_min_sync(0xffffffffu, bk == top ? bi : 0x7fffffff);
+    const bool found = top != 0u;
+    const float s = found ? sigmoid_t<T>(z[at]) : 0.f;
+    sum += s;
+    if (lane == (j & 31)) { idx[j] = found ? at : -1; w[j] = s; }
+    if (local && found && (at & 31) == lane) {
+#pragma unroll
+      for (int i = 0; i < kLocal; ++i)
+        if (i * 32 + lane == at) key[i] = 0u;
+    }
+    last = top;
+    last_i = at;
+  }
+  for (int j = lane; j < K; j += 32) w[j] = __fdiv_rn(w[j], sum + 1e-20f) * scale;      // every lane reads back what it wrote
+}
+
+// What runs beside a mixer's preparation for token t, by a CTA of THREADS threads: its choice of experts and the activation of its
+// dense feed-forward (see MbAside).
+template <typename T, bool VEC, int THREADS>
+__device__ __forceinline__ void aside_row(const MbAside& a, long long t) {
+  if (a.logits != nullptr && threadIdx.x < 32) {
+    if (a.grouped)
+      topk_grouped_row<T>(a.logits + t * a.experts, reinterpret_cast<const T*>(a.correction), a.experts, a.top, a.groups, a.keep, a.scale,
+                          a.weights + t * a.top, a.index + t * a.top);
+    else
+      topk_softmax_row<T>(a.logits + t * a.experts, a.experts, a.top, a.weights + t * a.top, a.index + t * a.top);
+  }
+  if (a.glu_in == nullptr) return;
+  const T* in = reinterpret_cast<const T*>(a.glu_in) + t * a.glu_ld_in;
+  T* out = reinterpret_cast<T*>(a.glu_out) + t * a.glu_ld_out;
+  constexpr int V = VEC ? 16 / static_cast<int>(sizeof(T)) : 1;
+  for (int i = threadIdx.x * V; i < a.ff; i += THREADS * V) {
+    float g[V], u[V];
+    load_n<V>(in + i, g);
+    load_n<V>(in + a.ff + i, u);
+#pragma unroll
+    for (int j = 0; j < V; ++j) g[j] = clamped_glu_t<T>(g[j], u[j], a.limit, a.alpha, a.shift);
+    store_n<V>(out + i, g);
+  }
+}
+// 16-byte accesses fit the feed-forward of an aside
+template <typename T>
+inline bool aside_vec(const MbAside& a) {
+  constexpr int v = 16 / static_cast<int>(sizeof(T));
+  return a.glu_in == nullptr || (a.ff % v == 0 && a.glu_ld_in % v == 0 && a.glu_ld_out % v == 0 &&
+                                 (reinterpret_cast<uintptr_t>(a.glu_in) | reinterpret_cast<uintptr_t>(a.glu_out)) % 16 == 0);
+}
+inline bool aside_on(const MbAside& a) { return a.logits != nullptr || a.glu_in != nullptr; }
+inline bool aside_ok(const MbAside& a) {
+  return a.logits == nullptr || !a.grouped || (a.groups > 0 && a.groups <= 256 && a.experts % a.groups == 0 && a.keep > 0);
 }
 
 }  // namespace mx

@@ -9,12 +9,12 @@ namespace mb {
 namespace mx {
 
 // grid (heads, tokens), 128 threads: each warp takes every fourth key with its own running softmax; RL · 32 ≥ dv.
-template <typename T, int RL>
+template <typename T, typename O, int RL>
 __global__ void __launch_bounds__(128) paged_attend_kernel(const T* __restrict__ q, const T* __restrict__ kc, const T* __restrict__ vc,
                                                            const int* __restrict__ block_table, int max_blocks, int block_size,
                                                            const int* __restrict__ token_seq, const int* __restrict__ positions,
                                                            const long long* __restrict__ slots, const T* __restrict__ sink,
-                                                           T* __restrict__ out, MbAttend A) {
+                                                           O* __restrict__ out, MbAttend A) {
   extern __shared__ float sm[];
   float* sq = sm;                        // [dk]
   float* so = sq + A.dk;                 // [4][dv]
@@ -24,9 +24,9 @@ __global__ void __launch_bounds__(128) paged_attend_kernel(const T* __restrict__
   const long long t = blockIdx.y;
   const int h = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  T* o = out + t * A.o_row + static_cast<long long>(h) * A.dv;
+  O* o = out + t * A.o_row + static_cast<long long>(h) * A.dv;
   if (slots[t] < 0) {                    // padding row of a decode batch
-    for (int i = threadIdx.x; i < A.dv; i += 128) o[i] = from_f<T>(0.f);
+    for (int i = threadIdx.x; i < A.dv; i += 128) o[i] = from_f<O>(0.f);
     return;
   }
   const int pos = positions[t];
@@ -79,18 +79,18 @@ __global__ void __launch_bounds__(128) paged_attend_kernel(const T* __restrict__
     float r = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) r = fmaf(so[w * A.dv + i], f[w], r);
-    o[i] = from_f<T>(__fdiv_rn(r, den));
+    o[i] = from_f<O>(__fdiv_rn(r, den));
   }
 }
 
-template <typename T, int RL>
+template <typename T, typename O, int RL>
 static int attend_rl(const T* q, const T* kc, const T* vc, const int* bt, int mb_, int bs, const int* seq, const int* pos, const long long* slots,
-                     const T* sink, T* out, int n, MbAttend A, cudaStream_t s) {
+                     const T* sink, O* out, int n, MbAttend A, cudaStream_t s) {
   const size_t bytes = (A.dk + 4 * A.dv) * sizeof(float);
   if (bytes > 48 * 1024) return -3;
   if (seq == nullptr && n > 65535) return -3;      // a decode batch (token = row) never gets this large
   for (int t0 = 0; t0 < n; t0 += 65535) {
-    const cudaError_t e = launch_pdl(paged_attend_kernel<T, RL>, dim3(A.heads, n - t0 < 65535 ? n - t0 : 65535), dim3(128), bytes, s,
+    const cudaError_t e = launch_pdl(paged_attend_kernel<T, O, RL>, dim3(A.heads, n - t0 < 65535 ? n - t0 : 65535), dim3(128), bytes, s,
                                      q + t0 * A.q_row, kc, vc, bt, mb_, bs, seq != nullptr ? seq + t0 : seq, pos + t0, slots + t0, sink,
                                      out + t0 * A.o_row, A);
     if (e != cudaSuccess) return static_cast<int>(e);
@@ -98,13 +98,13 @@ static int attend_rl(const T* q, const T* kc, const T* vc, const int* bt, int mb
   return 0;
 }
 
-template <typename T>
+template <typename T, typename O>
 static int attend(const T* q, const T* kc, const T* vc, const int* bt, int mb_, int bs, const int* seq, const int* pos, const long long* slots,
-                  const T* sink, T* out, int n, MbAttend A, cudaStream_t s) {
-  if (A.dv <= 128) return attend_rl<T, 4>(q, kc, vc, bt, mb_, bs, seq, pos, slots, sink, out, n, A, s);
-  if (A.dv <= 256) return attend_rl<T, 8>(q, kc, vc, bt, mb_, bs, seq, pos, slots, sink, out, n, A, s);
-  if (A.dv <= 512) return attend_rl<T, 16>(q, kc, vc, bt, mb_, bs, seq, pos, slots, sink, out, n, A, s);
-  if (A.dv <= 1024) return attend_rl<T, 32>(q, kc, vc, bt, mb_, bs, seq, pos, slots, sink, out, n, A, s);
+                  const T* sink, O* out, int n, MbAttend A, cudaStream_t s) {
+  if (A.dv <= 128) return attend_rl<T, O, 4>(q, kc, vc, bt, mb_, bs, seq, pos, slots, sink, out, n, A, s);
+  if (A.dv <= 256) return attend_rl<T, O, 8>(q, kc, vc, bt, mb_, bs, seq, pos, slots, sink, out, n, A, s);
+  if (A.dv <= 512) return attend_rl<T, O, 16>(q, kc, vc, bt, mb_, bs, seq, pos, slots, sink, out, n, A, s);
+  if (A.dv <= 1024) return attend_rl<T, O, 32>(q, kc, vc, bt, mb_, bs, seq, pos, slots, sink, out, n, A, s);
   return -3;
 }
 
@@ -116,13 +116,15 @@ using namespace mb::mx;
 
 extern "C" int mb_paged_attend(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size,
                                const int* token_seq, const int* positions, const long long* slots, const void* sink, void* out, int T,
-                               MbAttend A, int f32, cudaStream_t s) {
+                               MbAttend A, int f32, int out_f32, cudaStream_t s) {
   if (T <= 0) return 0;
   if (A.heads <= 0 || A.group <= 0 || A.heads % A.group) return -3;
-  auto run = [&](auto ty) {
+  auto run = [&](auto ty, auto to) {
     using E = decltype(ty);
-    return attend(reinterpret_cast<const E*>(q), reinterpret_cast<const E*>(kc), reinterpret_cast<const E*>(vc), block_table, max_blocks,
-                  block_size, token_seq, positions, slots, reinterpret_cast<const E*>(sink), reinterpret_cast<E*>(out), T, A, s);
+    using O = decltype(to);
+    return attend<E, O>(reinterpret_cast<const E*>(q), reinterpret_cast<const E*>(kc), reinterpret_cast<const E*>(vc), block_table, max_blocks,
+                  block_size, token_seq, positions, slots, reinterpret_cast<const E*>(sink), reinterpret_cast<O*>(out), T, A, s);
   };
-  return f32 ? run(float{}) : run(bf16{});
+  if (f32) return run(float{}, float{});
+  return out_f32 ? run(bf16{}, float{}) : run(bf16{}, bf16{});
 }

@@ -5,7 +5,8 @@
 // mma.sync.m16n8k16 and tiles of 64 keys are gathered from their pages with cp.async, double buffered, 16 keys per warp.  What differs:
 //   * the eight rows that padded the softmax weights carry their second bf16 part, so that P·V sees 16 bits of mantissa for no
 //     extra instruction; the two halves of the accumulator are added at the end;
-//   * the splits are joined through distributed shared memory, the sink enters there: one launch, no partial results in HBM.
+//   * the splits are joined through distributed shared memory, the sink enters there: one launch, no partial results in HBM;
+//   * differential attention (MbDiff): heads 2h and 2h + 1 are neighbours among the rows; a warp joins both, subtracts, norms and gates.
 // Heads narrower than DK / DV are padded with zeros in shared memory.
 #include <cooperative_groups.h>
 #include <cuda_bf16.h>
@@ -40,7 +41,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
                                                             const int* __restrict__ block_table, int max_blocks, int block_size,
                                                             const int* __restrict__ token_seq, const int* __restrict__ positions,
                                                             const long long* __restrict__ slots, const bf16* __restrict__ sink,
-                                                            bf16* __restrict__ out, long long o_row, float scale, MbWindow L) {
+                                                            bf16* __restrict__ out, long long o_row, float scale, MbWindow L, MbDiff D) {
   using S = Smem<DK, DV>;
   extern __shared__ __align__(128) uint8_t smem[];
   bf16* sQ = reinterpret_cast<bf16*>(smem + S::q);
@@ -57,9 +58,11 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
   const int group = L.heads / L.kv_heads, chunks = (group + 7) / 8;
   const int hk = blockIdx.y / chunks, h0 = hk * group + (blockIdx.y % chunks) * 8;
   const int rows = min(8, group - (blockIdx.y % chunks) * 8);
+  const bool diff = D.lam != nullptr;
   if (slots[t] < 0) {                    // padding row of a decode batch (the whole cluster leaves)
-    for (int i = split * 128 + threadIdx.x; i < rows * L.vdim; i += splits * 128)
-      out[t * o_row + static_cast<long long>(h0 + i / L.vdim) * L.vdim + i % L.vdim] = __float2bfloat16(0.f);
+    const int heads = diff ? rows / 2 : rows, first = diff ? h0 / 2 : h0;
+    for (int i = split * 128 + threadIdx.x; i < heads * L.vdim; i += splits * 128)
+      out[t * o_row + static_cast<long long>(first + i / L.vdim) * L.vdim + i % L.vdim] = __float2bfloat16(0.f);
     return;
   }
   const int pos = positions[t];
@@ -209,7 +212,52 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
   cg::cluster_group cluster = cg::this_cluster();
   if (splits > 1) cluster.sync();
   else __syncthreads();
-  for (int i = split * 128 + threadIdx.x; i < rows * DV; i += splits * 128) {
+  if (diff) {                            // a warp per head: both maps, their difference, its norm and gate
+    const float lam = *D.lam;
+    for (int hp = split * 4 + warp; hp < rows / 2; hp += splits * 4) {
+      const int head = h0 / 2 + hp;
+      const float gate = __bfloat162float(reinterpret_cast<const bf16*>(D.gate)[t * D.gate_ld + head]);
+      float v[DV / 32], ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < DV / 32; ++j) v[j] = 0.f;
+#pragma unroll
+      for (int map = 0; map < 2; ++map) {
+        const int g = 2 * hp + map;
+        float mm = -INFINITY, ms[8], den = 0.f, w[8];
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          ms[c] = c < splits ? cluster.map_shared_rank(fM, c)[g] : -INFINITY;
+          mm = fmaxf(mm, ms[c]);
+        }
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          w[c] = 0.f;
+          if (ms[c] == -INFINITY) continue;
+          w[c] = exp2f(ms[c] - mm);
+          den = fmaf(cluster.map_shared_rank(fM, c)[8 + g], w[c], den);
+        }
+        const float f = __fdiv_rn(map ? -lam : 1.f, den);
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          if (w[c] == 0.f) continue;
+          const float* o = cluster.map_shared_rank(fO, c) + g * DV;
+#pragma unroll
+          for (int j = 0; j < DV / 32; ++j) v[j] = fmaf(o[lane + 32 * j], w[c] * f, v[j]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < DV / 32; ++j)
+        if (lane + 32 * j < L.vdim) ss = fmaf(v[j], v[j], ss);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float rstd = __fdiv_rn(1.f, __fsqrt_rn(__fdiv_rn(ss, static_cast<float>(L.vdim)) + D.eps));
+      const float f = rstd * D.gain * __fdividef(1.f, 1.f + __expf(-gate));
+#pragma unroll
+      for (int j = 0; j < DV / 32; ++j)
+        if (lane + 32 * j < L.vdim) out[t * o_row + static_cast<long long>(head) * L.vdim + lane + 32 * j] = __float2bfloat16(v[j] * f);
+    }
+  }
+  for (int i = split * 128 + threadIdx.x; !diff && i < rows * DV; i += splits * 128) {
     const int g = i / DV, d = i % DV;
     const float sk = sink != nullptr ? __bfloat162float(sink[h0 + g]) * kLog2e : -INFINITY;
     float mm = sk, ms[8];
@@ -233,7 +281,8 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
 
 template <int DK, int DV>
 static int launch(const bf16* q, const bf16* kc, const bf16* vc, const int* bt, int max_blocks, int bs, const int* seq, const int* pos,
-                  const long long* slots, const bf16* sink, bf16* out, long long o_row, int T, float scale, int splits, MbWindow L, cudaStream_t s) {
+                  const long long* slots, const bf16* sink, bf16* out, long long o_row, int T, float scale, int splits, MbWindow L, MbDiff d,
+                  cudaStream_t s) {
   static bool once = false;
   if (!once) {
     const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<DK, DV>::total);
@@ -242,7 +291,7 @@ static int launch(const bf16* q, const bf16* kc, const bf16* vc, const int* bt, 
   }
   const int chunks = (L.heads / L.kv_heads + 7) / 8;
   return static_cast<int>(launch_pdl_cluster(window_decode_kernel<DK, DV>, dim3(splits, L.kv_heads * chunks, T), dim3(128), splits,
-                                             Smem<DK, DV>::total, s, q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, scale, L));
+                                             Smem<DK, DV>::total, s, q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, scale, L, d));
 }
 
 }  // namespace wd
@@ -254,12 +303,13 @@ using namespace mb;
 // 8 up to 128, splits ∈ 1 … 8, T ≤ 65535.
 extern "C" int mb_window_decode(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                                 const int* positions, const long long* slots, const void* sink, void* out, long long o_row, int T, float scale,
-                                int splits, MbWindow L, cudaStream_t s) {
+                                int splits, MbWindow L, MbDiff d, cudaStream_t s) {
   if (T <= 0) return 0;
   if (L.dim % 8 || L.vdim % 8 || L.q_pitch % 8 || L.dim > 128 || L.vdim > 128 || L.heads % L.kv_heads || splits < 1 || splits > 8 || T > 65535) return -3;
+  if (d.lam != nullptr && (sink != nullptr || (L.heads / L.kv_heads) % 2)) return -3;
   using wd::bf16;
   auto Q = reinterpret_cast<const bf16*>(q), K = reinterpret_cast<const bf16*>(kc), V = reinterpret_cast<const bf16*>(vc), SK = reinterpret_cast<const bf16*>(sink);
   auto O = reinterpret_cast<bf16*>(out);
   auto f = L.dim <= 64 ? (L.vdim <= 64 ? wd::launch<64, 64> : wd::launch<64, 128>) : (L.vdim <= 64 ? wd::launch<128, 64> : wd::launch<128, 128>);
-  return f(Q, K, V, block_table, max_blocks, block_size, token_seq, positions, slots, SK, O, o_row, T, scale, splits, L, s);
+  return f(Q, K, V, block_table, max_blocks, block_size, token_seq, positions, slots, SK, O, o_row, T, scale, splits, L, d, s);
 }

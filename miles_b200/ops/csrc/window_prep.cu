@@ -81,20 +81,7 @@ __global__ void __launch_bounds__(kPrep) window_prep_kernel(const T* __restrict_
   const T* p = proj + t * ld;
   const int nq = L.heads * L.dim, nk = L.kv_heads * L.dim, nv = L.kv_heads * L.vdim;
   if (blockIdx.y == 2) {
-    if (a.logits != nullptr && threadIdx.x < 32)
-      topk_softmax_row<T>(a.logits + t * a.experts, a.experts, a.top, a.weights + t * a.top, a.index + t * a.top);
-    if (a.glu_in == nullptr) return;
-    const T* in = reinterpret_cast<const T*>(a.glu_in) + t * a.glu_ld_in;
-    T* out = reinterpret_cast<T*>(a.glu_out) + t * a.glu_ld_out;
-    constexpr int V = VEC ? 16 / static_cast<int>(sizeof(T)) : 1;
-    for (int i = threadIdx.x * V; i < a.ff; i += kPrep * V) {
-      float g[V], u[V];
-      load_n<V>(in + i, g);
-      load_n<V>(in + a.ff + i, u);
-#pragma unroll
-      for (int j = 0; j < V; ++j) g[j] = clamped_glu_t<T>(g[j], u[j], a.limit, a.alpha);
-      store_n<V>(out + i, g);
-    }
+    aside_row<T, VEC, kPrep>(a, t);
     return;
   }
   const bool keys = blockIdx.y == 1;
@@ -125,12 +112,9 @@ template <typename T>
 static int prep(const T* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
                 const T* q_norm, const T* k_norm, float eps, T* kc, T* vc, T* q, int n, MbWindow L, MbAside a, cudaStream_t s) {
   const int v = 16 / static_cast<int>(sizeof(T));
-  bool vec = ld % v == 0 && L.dim % v == 0 && L.vdim % v == 0 && L.rot % v == 0 && L.q_pitch % v == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0;
-  if (a.glu_in != nullptr)
-    vec = vec && a.ff % v == 0 && a.glu_ld_in % v == 0 && a.glu_ld_out % v == 0 &&
-          (reinterpret_cast<uintptr_t>(a.glu_in) | reinterpret_cast<uintptr_t>(a.glu_out)) % 16 == 0;
+  const bool vec = ld % v == 0 && L.dim % v == 0 && L.vdim % v == 0 && L.rot % v == 0 && L.q_pitch % v == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0 && aside_vec<T>(a);
   auto kern = vec ? window_prep_kernel<T, true> : window_prep_kernel<T, false>;
-  return static_cast<int>(launch_pdl(kern, dim3(n, a.logits != nullptr || a.glu_in != nullptr ? 3 : 2), dim3(kPrep), L.rot * sizeof(float), s, proj,
+  return static_cast<int>(launch_pdl(kern, dim3(n, aside_on(a) ? 3 : 2), dim3(kPrep), L.rot * sizeof(float), s, proj,
                                      ld, positions, slots, freq, magnitude, q_norm, k_norm, eps, kc, vc, q, L, a));
 }
 
@@ -144,7 +128,7 @@ extern "C" int mb_window_prep(const void* proj, long long ld, const int* positio
                               float magnitude, const void* q_norm, const void* k_norm, float eps, void* kc, void* vc, void* q, int T,
                               MbWindow L, MbAside a, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
-  if (L.rot > 4096 || L.rot % 2 || L.rot > L.dim || L.heads % L.kv_heads) return -3;
+  if (L.rot > 4096 || L.rot % 2 || L.rot > L.dim || L.heads % L.kv_heads || !aside_ok(a)) return -3;
   auto run = [&](auto ty) {
     using E = decltype(ty);
     return prep(reinterpret_cast<const E*>(proj), ld, positions, slots, freq, magnitude, reinterpret_cast<const E*>(q_norm),

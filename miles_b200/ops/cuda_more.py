@@ -181,11 +181,13 @@ def moe_max_rows_pad(n_pairs: int, num_experts: int, pad: int) -> int:
     return (n_pairs + num_experts * (pad - 1) + pad - 1) // pad * pad
 
 
-def few_token_experts(x, w13, T: int, k: int) -> bool:
+def few_token_experts(x, w13, T: int, k: int, ungated: bool = False) -> bool:
     """A handful of tokens: two matrix-vector kernels, no sort / gather / combine (gemv.cu).  Both keep their activations in shared
-    memory next to a 64 KB weight ring."""
+    memory next to a 64 KB weight ring.  `ungated`: w13 has no gate rows."""
+    F = w13.shape[1] if ungated else w13.shape[1] // 2
     return (x.dtype == BF16 and 0 < T <= MOE_GEMV_T and T * k <= 64 and not torch.is_grad_enabled() and x.shape[1] % 32 == 0
-            and w13.shape[1] % 64 == 0 and 65536 + max(8 * (2 * x.shape[1] + 64), T * k * (w13.shape[1] + 64)) <= 200 * 1024)
+            and F % 32 == 0 and (ungated or w13.shape[1] % 64 == 0)
+            and 65536 + max(8 * (2 * x.shape[1] + 64), T * k * (2 * F + 64)) <= 200 * 1024)
 
 
 def sort_by_expert(x, idx, E: int, bt: int, expert_offset: int = 0):
@@ -202,23 +204,26 @@ def sort_by_expert(x, idx, E: int, bt: int, expert_offset: int = 0):
 
 def experts_forward(x_perm, w13, w2, seg, tile, bt: int = 128, glu=None):
     """Grouped expert FFN on expert-sorted rows whose segments are padded to `bt`. Returns (h1 pre-activation, y_perm).  `glu`: (limit,
-    alpha) of a clamped activation instead of SwiGLU (inference)."""
+    alpha, shift) of a clamped activation instead of SwiGLU, or "relu2" for experts without a gate (inference)."""
     max_rows, H = x_perm.shape
     E, F2, _ = w13.shape
+    F = w2.shape[2]
     h1 = torch.empty(max_rows, F2, dtype=x_perm.dtype, device=x_perm.device)
-    act = torch.empty(max_rows, F2 // 2, dtype=x_perm.dtype, device=x_perm.device)
+    act = h1 if glu == "relu2" else torch.empty(max_rows, F, dtype=x_perm.dtype, device=x_perm.device)      # squared in place
     y_perm = torch.empty(max_rows, H, dtype=x_perm.dtype, device=x_perm.device)
 
     def activate():
         if glu is None:
             C.swiglu_fwd(h1, act, seg[-1:])
+        elif glu == "relu2":
+            C.relu_square(h1, seg[-1:])
         else:
-            C.clamped_glu(h1, act, glu[0], glu[1], seg[-1:])
+            C.clamped_glu(h1, act, glu[0], glu[1], seg[-1:], glu[2])
 
     if bt != 128:
         C.gemm_small_grouped(x_perm, w13, h1, max_rows, F2, H, E, tile, seg[-1:], bt)
         activate()
-        C.gemm_small_grouped(act, w2, y_perm, max_rows, H, F2 // 2, E, tile, seg[-1:], bt)
+        C.gemm_small_grouped(act, w2, y_perm, max_rows, H, F, E, tile, seg[-1:], bt)
         return h1, y_perm
     from . import cuda as _cuda
 
@@ -228,7 +233,6 @@ def experts_forward(x_perm, w13, w2, seg, tile, bt: int = 128, glu=None):
         # dense projections of this recipe
         from . import extra
 
-        F = F2 // 2
         xq, xs = mxfp8_quant(x_perm)
         wq, ws = mxfp8_quant(w13.reshape(E * F2, H))
         extra.gemm_mxfp8_grouped(xq, xs, wq.view(E, F2, H), ws.view(E, F2, H // 32), tile, out=h1)
@@ -239,7 +243,7 @@ def experts_forward(x_perm, w13, w2, seg, tile, bt: int = 128, glu=None):
         return h1, y_perm
     C.gemm_grouped(x_perm, w13, h1, max_rows, F2, H, E, tile, False, 0)
     activate()
-    C.gemm_grouped(act, w2, y_perm, max_rows, H, F2 // 2, E, tile, False, 0)
+    C.gemm_grouped(act, w2, y_perm, max_rows, H, F, E, tile, False, 0)
     return h1, y_perm
 
 

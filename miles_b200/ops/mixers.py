@@ -65,6 +65,61 @@ class AttentionLayout:
         return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
 
 
+@dataclass(frozen=True)
+class DifferentialLayout:
+    """Sizes of one differential-attention layer.  The cache keeps [kv_heads, 2·dim] keys (both maps side by side) and [kv_heads, vdim]
+    values per token; `writes`: the layer has keys and values of its own."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    writes: bool = True
+
+    @property
+    def q_rows(self) -> int:
+        return self.heads * 2 * self.dim
+
+    @property
+    def gate_at(self) -> int:
+        return self.q_rows + (self.kv_heads * (2 * self.dim + self.vdim) if self.writes else 0)
+
+    @property
+    def paired(self) -> AttentionLayout:
+        """The grouped-query layer it is to the attention kernels: every map a query head over whole key rows."""
+        return AttentionLayout(2 * self.heads, self.kv_heads, 2 * self.dim, self.vdim, 0, 0, 0)
+
+
+@dataclass(frozen=True)
+class SsmLayout:
+    """Sizes of one state-space layer; a row of its projection is [z | x | B | C | dt]."""
+
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    taps: int
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        """x, B and C: what passes the convolution."""
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass(frozen=True)
+class Routing:
+    """Choice of experts by sigmoid scores: corrected scores compete inside the `keep` best of `groups` groups of neighbours (a group is
+    worth its two largest); weights are the chosen ones' uncorrected scores over their sum, times `scale`."""
+
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+
+
 @dataclass
 class Addend:
     """A sublayer's output on its way into the residual: rows `y` [T, D], or (with `dst`) the expert-sorted rows `y` whose sum
@@ -73,12 +128,14 @@ class Addend:
     y: torch.Tensor
     weights: torch.Tensor | None = None
     dst: torch.Tensor | None = None
+    scale: torch.Tensor | None = None      # a factor per channel
 
 
 @dataclass
 class Aside:
-    """Work on the same projection that runs beside an attention layer's preparation: the choice of experts from `logits`
-    (→ `weights`, `index`) and the activation of a dense feed-forward (`glu_in` [T, ≥ 2F] → `glu_out` [T, F], both may be strided)."""
+    """Work that runs beside a mixer's preparation: the choice of experts from `logits` (→ `weights`, `index`; by `routing` and
+    `correction` if given, else by a softmax over the largest) and the activation of a dense feed-forward (`glu_in` [T, ≥ 2F] →
+    `glu_out` [T, F], both may be strided)."""
 
     logits: torch.Tensor | None = None
     top: int = 0
@@ -88,14 +145,18 @@ class Aside:
     glu_out: torch.Tensor | None = None
     limit: float = 0.0
     alpha: float = 0.0
+    shift: float = 1.0
+    routing: Routing | None = None
+    correction: torch.Tensor | None = None
 
 
-def bigram_embedding(tokens, prev, embed, table=None, spec=None, want_copy=True):
+def bigram_embedding(tokens, prev, embed, table=None, spec=None, want_copy=True, positions=None, freq=None):
     """(fp32 residual, copy in the model's dtype or None): embed[token] + table[(prev·m_prev + token·m_cur) mod buckets]; a sequence's first
-    token (prev < 0) takes the table's last row.  spec = (buckets, m_prev, m_cur)."""
+    token (prev < 0) takes the table's last row.  spec = (buckets, m_prev, m_cur).  `freq` (one per pair of channels): the sine and the
+    cosine of position · freq are added to the pair."""
     if embed.is_cuda:
-        return _k().bigram_embedding(tokens, prev, embed, table, spec, want_copy)
-    return ref.bigram_embedding(tokens, prev, embed, table, spec)
+        return _k().bigram_embedding(tokens, prev, embed, table, spec, want_copy, positions, freq)
+    return ref.bigram_embedding(tokens, prev, embed, table, spec, positions, freq)
 
 
 def output_norm_residual(x, y, nw, ls, eps, final_w=None):
@@ -114,11 +175,11 @@ def output_norm_linear(x, y, nw, ls, eps, w):
     return _k().output_norm_linear(x, y, nw, ls, eps, w)
 
 
-def clamped_glu(h, limit, alpha):
-    """h = [gate; up] → g·sigmoid(alpha·g)·(u + 1), g = min(gate, limit), u = clamp(up, ±limit)."""
+def clamped_glu(h, limit, alpha, shift=1.0):
+    """h = [gate; up] → g·sigmoid(alpha·g)·(u + shift), g = min(gate, limit), u = clamp(up, ±limit)."""
     if h.is_cuda:
-        return _k().clamped_glu(h, limit, alpha)
-    return ref.clamped_glu(h, limit, alpha)
+        return _k().clamped_glu(h, limit, alpha, shift)
+    return ref.clamped_glu(h, limit, alpha, shift)
 
 
 def latent_attention(proj, lay: LatentLayout, cache, meta, *, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps):
@@ -139,11 +200,11 @@ def linear_state_attention(proj, heads, dk, dv, decay, state, meta, norm_w, eps)
     return ref.gated_norm(ref.linear_state(proj, heads, dk, dv, decay, state, meta), norm_w, gate, eps)
 
 
-def sum_norm(x, to, addends, extra, nw, eps):
-    """s = x + Σ addends (+ extra), fp32, written to `to` if given; returns rmsnorm(s)·nw in the model's dtype (None without `nw`)."""
-    if x.is_cuda:
-        return _k().sum_norm(x, to, addends, extra, nw, eps)
-    return ref.sum_norm(x, to, addends, extra, nw, eps)
+def sum_norm(x, to, addends, extra, nw, eps, shift=0.0, gain=1.0, nw2=None, two=False):
+    """s = x + Σ addends (+ extra), fp32, written to `to` if given; returns rmsnorm(s)·(nw + shift)·gain in the model's dtype (None without
+    `nw`); with `two` a pair, the second by `nw2` (None without)."""
+    h = (_k() if x.is_cuda else ref).sum_norm(x, to, addends, extra, nw, eps, shift, gain, nw2)
+    return h if two else h[0]
 
 
 def few_row_sum(x, addends, w) -> bool:
@@ -153,6 +214,20 @@ def few_row_sum(x, addends, w) -> bool:
 def sum_norm_linear(x, addends, extra, nw, eps, w, w2=None, b2=None, want_normed=False):
     """`sum_norm` and `projections` in one kernel (where `few_row_sum` holds).  Returns (normed or None, product, logits, sum)."""
     return _k().sum_norm_linear(x, addends, extra, nw, eps, w, w2, b2, want_normed)
+
+
+def sum_two_norms_linear(x, addends, nw, w, nw2, w2, eps, shift, routes):
+    """Sum, two norms of it and the product of each with its weight in one kernel (where `few_row_sum` holds for both weights; `w2` may be
+    None).  Returns (first product, second product — fp32 where it `routes`, the rows normed by `nw2` there, sum)."""
+    return _k().sum_two_norms_linear(x, addends, nw, w, nw2, w2, eps, shift, routes)
+
+
+def product(h, w, fp32=False):
+    """h·wᵀ in the model's dtype or fp32; rows may be padded to whole 16-byte pieces."""
+    if h.is_cuda:
+        return _k().product(h, w, fp32)
+    y = h @ w.T
+    return y.float() if fp32 else y
 
 
 def projections(h, w, w2=None, b2=None):
@@ -168,16 +243,40 @@ def windowed_attention(proj, lay: AttentionLayout, kc, vc, meta, out, *, freq, m
     `keep` ones.  `aside` is done on the way."""
     if proj.is_cuda:
         return _k().windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps, aside)
-    if aside is not None:
-        if aside.logits is not None:
-            aside.weights, aside.index = ref.topk_softmax(aside.logits, aside.top)
-        if aside.glu_in is not None:
-            aside.glu_out.copy_(ref.clamped_glu(aside.glu_in[:, : 2 * aside.glu_out.shape[1]], aside.limit, aside.alpha))
+    ref.aside(aside)
     return ref.windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps)
 
 
-def routed_experts(h, w13, w2, weights, index, limit, alpha) -> Addend:
-    """Σ_j weights[t, j] · W2[e]·clamped_glu(W13[e]·h[t]) with e = index[t, j], as an addend."""
+def differential_attention(proj, lay: DifferentialLayout, kc, vc, meta, *, scale, diff, temperature, lvec, q_norm, k_norm, eps, aside=None):
+    """proj [T, q (; k; v); gates] → [T, heads·vdim].  Norms queries and keys per head and map, multiplies queries by the temperature
+    (coef, every) of their position, caches keys and values (with `k_norm`; else they are another layer's); every token attends to all
+    cached tokens up to itself with both maps of every head: o = a1 − λ·a2 with λ = exp(l₀·l₁) − exp(l₂·l₃) + diff (rows of `lvec`),
+    normed over the head, times (1 − diff) · sigmoid(gate of the head).  `aside` is done on the way."""
+    if proj.is_cuda:
+        return _k().differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lvec, q_norm, k_norm, eps, aside)
+    ref.aside(aside)
+    return ref.differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lvec, q_norm, k_norm, eps)
+
+
+def state_space(proj, lay: SsmLayout, conv, conv_b, dt_bias, A_log, D, state, ring, meta, aside=None):
+    """proj [T, z; x; B; C; dt] → [T, heads·vdim] = y·silu(z): causal convolution and silu on x, B, C; dt ← softplus(dt + dt_bias); per head
+    S ← exp(−exp(A_log)·dt)·S + dt·B xᵀ, y = Sᵀ C + D·x.  `state` [slots, heads, state, vdim] and `ring` [slots, taps, channels] (the
+    convolution's inputs by position mod taps; None without look-back), fp32, are read (nothing before position 0) and written.  `aside` is done on the way."""
+    if proj.is_cuda:
+        return _k().state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta, aside)
+    ref.aside(aside)
+    return ref.state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta)
+
+
+def part_norm_linear(x, nw, parts, eps, w):
+    """(every one of `parts` equal parts of a row over its own root mean square, times nw)·wᵀ"""
+    if x.is_cuda:
+        return _k().part_norm_linear(x, nw, parts, eps, w)
+    return ref.part_norm(x, nw, parts, eps) @ w.T
+
+
+def routed_experts(h, w13, w2, weights, index, limit=0.0, alpha=0.0, shift=1.0, ungated=False) -> Addend:
+    """Σ_j weights[t, j] · W2[e]·act(W13[e]·h[t]) with e = index[t, j], as an addend; act: `clamped_glu`, or relu(·)² without a gate."""
     if h.is_cuda:
-        return _k().routed_experts(h, w13, w2, weights, index, limit, alpha)
-    return Addend(ref.routed_experts(h, w13, w2, weights, index, limit, alpha))
+        return _k().routed_experts(h, w13, w2, weights, index, limit, alpha, shift, ungated)
+    return Addend(ref.routed_experts(h, w13, w2, weights, index, limit, alpha, shift, ungated))

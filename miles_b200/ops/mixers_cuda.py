@@ -1,5 +1,5 @@
 """CUDA execution of the ops in `mixers.py` (inference only): the kernels of mixers.cu, latent_*.cu, linear_*.cu, window_*.cu,
-attention_*_tc.cu, paged_attend.cu and experts_any.cu.
+diff_prep.cu, ssm_*.cu, attention_*_tc.cu, paged_attend.cu and experts_any.cu.
 
 Tensors are bf16, or float32 throughout (then every product is a true 32-bit one: the kernels' own fp32 loops, and cuBLAS
 without TF32 for the dense projections, as `ops.linear` does for float32).
@@ -18,12 +18,12 @@ def _c(x):
     return x if x.is_contiguous() else x.contiguous()
 
 
-def bigram_embedding(tokens, prev, embed, table, spec, want_copy=True):
+def bigram_embedding(tokens, prev, embed, table, spec, want_copy=True, positions=None, freq=None):
     T, D = tokens.numel(), embed.shape[1]
     x = torch.empty(T, D, dtype=torch.float32, device=embed.device)
     xb = torch.empty(T, D, dtype=embed.dtype, device=embed.device) if want_copy else None
     buckets, mp, mc = spec if table is not None else (0, 0, 0)
-    C.bigram_embedding(tokens.to(torch.int32), prev, embed, table, buckets, mp, mc, x, xb)
+    C.bigram_embedding(tokens.to(torch.int32), prev, embed, table, buckets, mp, mc, positions if freq is not None else None, freq, x, xb)
     return x, xb
 
 
@@ -48,9 +48,9 @@ def output_norm_linear(x, y, nw, ls, eps, w):
     return out, x_new
 
 
-def clamped_glu(h, limit, alpha):
+def clamped_glu(h, limit, alpha, shift=1.0):
     out = torch.empty(h.shape[0], h.shape[1] // 2, dtype=h.dtype, device=h.device)
-    C.clamped_glu(h, out, float(limit), float(alpha))
+    C.clamped_glu(h, out, float(limit), float(alpha), shift=float(shift))
     return out
 
 
@@ -193,11 +193,20 @@ def _split_addends(addends):
     return dense + [None] * (2 - len(dense)), (rows[0] if rows else None)
 
 
-def sum_norm(x, to, addends, extra, nw, eps):
+def sum_norm(x, to, addends, extra, nw, eps, shift=0.0, gain=1.0, nw2=None):
     (y1, y2), r = _split_addends(addends)
-    h = torch.empty(x.shape, dtype=nw.dtype, device=x.device) if nw is not None else None
-    C.sum_norm(x, to, y1, y2, r.y if r else None, r.weights if r else None, r.dst if r else None, extra, nw, h, float(eps))
-    return h
+    h, h2 = (torch.empty(x.shape, dtype=w.dtype, device=x.device) if w is not None else None for w in (nw, nw2))
+    s1, s2 = _scales(addends)
+    C.sum_norm(x, to, y1, s1, y2, s2, r.y if r else None, r.weights if r else None, r.dst if r else None, extra, nw, h, nw2, h2, float(eps),
+               float(shift), float(gain))
+    return h, h2
+
+
+def _scales(addends):
+    """Scales of the first dense output and of what comes with it (another dense output, else experts' rows)."""
+    dense, rows = [a.scale for a in addends if a.dst is None], [a.scale for a in addends if a.dst is not None]
+    second = dense[1:] + rows
+    return dense[0] if dense else None, second[0] if second else None
 
 
 def few_row_sum(x, addends, w) -> bool:
@@ -216,8 +225,37 @@ def sum_norm_linear(x, addends, extra, nw, eps, w, w2, b2, want_normed):
     logits = torch.empty(T, w2.shape[0], dtype=torch.float32, device=dev) if w2 is not None else None
     x_new = torch.empty_like(x) if addends or extra is not None else None
     h = torch.empty(x.shape, dtype=w.dtype, device=dev) if want_normed else None
-    C.gemv_sum_norm(x, y1, y2, extra, None, nw, float(eps), w, proj, w2, b2, logits, x_new, h, _static(w))
+    C.gemv_sum_norm(x, y1, None, y2, None, extra, None, nw, None, float(eps), 0.0, w, proj, w2, b2, logits, x_new, h, _static(w))
     return h, proj, logits, x if x_new is None else x_new
+
+
+def _rows(T: int, n: int, dtype, device):
+    """[T, n] in rows of whole 16-byte pieces, so that kernels behind a projection of any width can use them."""
+    piece = 16 // torch.empty(0, dtype=dtype).element_size()
+    return torch.empty(T, -(-n // piece) * piece, dtype=dtype, device=device)[:, :n]
+
+
+def sum_two_norms_linear(x, addends, nw, w, nw2, w2, eps, shift, routes):
+    (y1, y2), _ = _split_addends(addends)
+    s1, s2 = _scales(addends)
+    T, dev = x.shape[0], x.device
+    proj = _rows(T, w.shape[0], w.dtype, dev)
+    second = None
+    if w2 is not None:
+        second = torch.empty(T, w2.shape[0], dtype=torch.float32, device=dev) if routes else _rows(T, w2.shape[0], w.dtype, dev)
+    x_new = torch.empty_like(x) if addends else None
+    h2 = torch.empty(x.shape, dtype=w.dtype, device=dev) if routes else None
+    C.gemv_sum_norm(x, y1, s1, y2, s2, None, None, nw, nw2, float(eps), float(shift), w, proj, w2, None, second, x_new, h2,
+                    _static(w) and (w2 is None or _static(w2)))
+    return proj, second, h2, x if x_new is None else x_new
+
+
+def product(h, w, fp32):
+    if h.dtype != BF16:
+        return torch.nn.functional.linear(h, w)
+    if fp32:
+        return K.gemm_nt(h, w, out_dtype=torch.float32)
+    return K.gemm_nt(h, w, _rows(h.shape[0], w.shape[0], BF16, h.device))
 
 
 def projections(h, w, w2, b2):
@@ -228,7 +266,7 @@ def projections(h, w, w2, b2):
     if w2 is not None and T <= K.GEMV_M and w.shape[0] <= GEMV_MAX_N and gemv_ok(h, w):
         proj = torch.empty(T, w.shape[0], dtype=BF16, device=h.device)
         logits = torch.empty(T, E, dtype=torch.float32, device=h.device)
-        C.gemv_sum_norm(None, None, None, None, h, None, 0.0, w, proj, w2, b2, logits, None, None, _static(w))
+        C.gemv_sum_norm(None, None, None, None, None, None, h, None, None, 0.0, 0.0, w, proj, w2, b2, logits, None, None, _static(w))
         return proj, logits
     return K.gemm_nt(h, w), None if w2 is None else K.gemm_nt(h, w2, bias=b2, out_dtype=torch.float32)
 
@@ -253,46 +291,137 @@ def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sin
     pitch = -(-lay.dim // 64) * 64 if fast else lay.dim
     sizes = [lay.heads, lay.kv_heads, lay.dim, lay.vdim, lay.rot, lay.window, lay.keep, pitch]
     q = torch.empty(T, lay.heads, pitch, dtype=dt, device=dev)
-    a = aside
-    logits = a.logits if a is not None else None
-    if logits is not None:
-        a.weights = torch.empty(T, a.top, dtype=torch.float32, device=dev)
-        a.index = torch.empty(T, a.top, dtype=torch.int32, device=dev)
-    C.window_prep(proj, meta.positions, meta.slot_mapping, freq, float(magnitude), q_norm, k_norm, float(eps), kc, vc, q, sizes, logits,
-                  a.weights if logits is not None else None, a.index if logits is not None else None, a.glu_in if a is not None else None,
-                  a.glu_out if a is not None else None, float(a.limit) if a is not None else 0.0, float(a.alpha) if a is not None else 0.0)
+    C.window_prep(proj, meta.positions, meta.slot_mapping, freq, float(magnitude), q_norm, k_norm, float(eps), kc, vc, q, sizes, *_aside(aside, T))
+    _paged_attention(q, lay, kc, vc, meta, out, scale, sink, sizes, fast)
+
+
+def _aside(a, T: int):
+    """The arguments of a kernel that does an `Aside` on the way; allocates what it chooses."""
+    if a is None:
+        return [None] * 6, [0.0] * 4, [0] * 3
+    if a.logits is not None:
+        a.weights = torch.empty(T, a.top, dtype=torch.float32, device=a.logits.device)
+        a.index = torch.empty(T, a.top, dtype=torch.int32, device=a.logits.device)
+    r = a.routing
+    return ([a.logits, a.weights if a.logits is not None else None, a.index if a.logits is not None else None, a.glu_in, a.glu_out, a.correction],
+            [float(a.limit), float(a.alpha), float(a.shift), float(r.scale) if r else 1.0], [1, r.groups, r.keep] if r else [0, 1, 1])
+
+
+def _paged_attention(q, lay, kc, vc, meta, out, scale, sink, sizes, fast, difference=()):
+    """Prepared queries over the paged cache: long pieces as query tiles, short ones token by token.  `difference`: (weight of the second map,
+    gates, gain, eps) of differential attention."""
+    T, rg = q.shape[0], meta.ragged
     t_long = rg.t_long if fast and scale > 0 and kc.shape[1] % 8 == 0 and lay.heads // lay.kv_heads <= 128 else 0
     if t_long:
         C.window_prefill(q, kc, vc, out, sink, rg.cu_q, meta.positions, meta.block_table, rg.n_long, max(rg.q_lens[: rg.n_long]), t_long,
-                         float(scale), sizes, C.error_flag(proj))
+                         float(scale), sizes, C.error_flag(q), *difference)
     if T > t_long:
         seq = rg.token_seq[t_long:] if rg.token_seq is not None else None
-        args = (q[t_long:], kc, vc, meta.block_table, seq, meta.positions[t_long:], meta.slot_mapping[t_long:], sink, out[t_long:], float(scale))
+        where = (kc, vc, meta.block_table, seq, meta.positions[t_long:], meta.slot_mapping[t_long:], sink)
+        if difference:
+            difference = (difference[0], difference[1][t_long:], *difference[2:])
         if fast:
-            C.window_decode(*args, window_splits(T - t_long, lay), sizes)
+            C.window_decode(q[t_long:], *where, out[t_long:], float(scale), window_splits(T - t_long, lay), sizes, *difference)
+        elif difference:
+            both = torch.empty(T - t_long, lay.heads * lay.vdim, dtype=torch.float32, device=q.device)
+            C.window_attend(q[t_long:], *where, both, float(scale), sizes)
+            C.diff_combine(both, out[t_long:], lay.heads // 2, lay.vdim, *difference)
         else:
-            C.window_attend(*args, sizes)
+            C.window_attend(q[t_long:], *where, out[t_long:], float(scale), sizes)
+
+
+def differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lvec, q_norm, k_norm, eps, aside):
+    T, dt, dev, pair = proj.shape[0], proj.dtype, proj.device, lay.paired
+    out = torch.empty(T, lay.heads * lay.vdim, dtype=dt, device=dev)
+    fast = _window_ok(pair, dt)
+    pitch = -(-pair.dim // 64) * 64 if fast else pair.dim
+    sizes = [pair.heads, pair.kv_heads, pair.dim, pair.vdim, 0, 0, 0, pitch]
+    q = torch.empty(T, pair.heads, pitch, dtype=dt, device=dev)
+    lam = torch.empty(1, dtype=torch.float32, device=dev)
+    coef, every = temperature or (0.0, 1.0)
+    C.diff_prep(proj, meta.positions, meta.slot_mapping, q_norm, k_norm, lvec, lam, kc if lay.writes else None, vc if lay.writes else None, q,
+                [lay.heads, lay.kv_heads if lay.writes else 0, lay.dim, lay.vdim, pitch], float(eps), float(coef), float(every), float(diff),
+                *_aside(aside, T))
+    gates = proj[:, lay.gate_at: lay.gate_at + lay.heads]
+    _paged_attention(q, pair, kc, vc, meta, out, scale, None, sizes, fast, (lam, gates, 1.0 - diff, float(eps)))
+    return out
+
+
+# ---- state-space mixer ------------------------------------------------------------------------------------------------
+
+CONV_TILE = 32           # tokens of a convolution tile (ssm_state.cu)
+
+
+def _conv_tiles(meta):
+    """[n, 4] (first token, end, sequence, first tile of its piece) over all pieces of a packed batch."""
+    rg = meta.ragged
+    if "conv_tiles" not in rg.scratch:
+        tiles, t = [], 0
+        for b, n in enumerate(rg.q_lens):
+            for a in range(0, n, CONV_TILE):
+                tiles += [t + a, t + min(n, a + CONV_TILE), b, int(a == 0)]
+            t += n
+        rg.scratch["conv_tiles"] = torch.tensor(tiles, dtype=torch.int32).to(meta.positions.device).view(-1, 4)
+    return rg.scratch["conv_tiles"]
+
+
+def state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta, aside):
+    T, dt, dev, rg = proj.shape[0], proj.dtype, proj.device, meta.ragged
+    sizes = [lay.heads, lay.vdim, lay.state, lay.groups, lay.taps]
+    out = torch.empty(T, lay.inner, dtype=dt, device=dev)
+    a = _aside(aside, T)
+
+    def tensors(slots, positions):
+        return [conv, conv_b, dt_bias, A_log, D, state, ring, slots, positions]
+
+    slots, cu_q = meta.state_slots, rg.cu_q
+    if cu_q is None and lay.vdim % 4 == 0 and lay.vdim <= 1024 and lay.state <= 4096:
+        C.ssm_step(proj, sizes, tensors(slots, meta.positions), out, *a)
+        return out
+    xbc = torch.empty(T, lay.channels, dtype=dt, device=dev)
+    step, decay = (torch.empty(T, lay.heads, dtype=torch.float32, device=dev) for _ in range(2))
+    C.ssm_conv(proj, sizes, tensors(slots, meta.positions), _conv_tiles(meta) if cu_q is not None else None, cu_q, xbc, step, decay, *a)
+    if rg.n_long and dt == BF16 and lay.state % 8 == 0 and lay.vdim % 8 == 0 and lay.state <= 128 and lay.vdim <= 128 and proj.stride(0) % 2 == 0:
+        # long pieces in chunks on the tensor cores, the short ones behind them token by token
+        segs, seq_segs, multi = _segments(meta, lay.heads // C.ssm_heads_per_cta(lay.heads, lay.vdim, lay.groups))
+        seg_state = torch.empty(segs.shape[0], lay.heads, lay.state, lay.vdim, dtype=torch.float32, device=dev) if multi else None
+        seg_decay = torch.empty(segs.shape[0], lay.heads, dtype=torch.float32, device=dev) if multi else None
+        C.ssm_chunk(proj, xbc, step, decay, sizes, tensors(slots, meta.positions), segs, seq_segs, seg_state, seg_decay, out)
+        if slots.numel() == rg.n_long:
+            return out
+        slots, cu_q = slots[rg.n_long:], cu_q[rg.n_long:]
+    C.ssm_seq(proj, xbc, step, decay, sizes, tensors(slots, meta.positions), cu_q, out)
+    return out
+
+
+def part_norm_linear(x, nw, parts, eps, w):
+    if parts == 1 and w.shape[0] <= GEMV_MAX_N and gemv_ok(x, w):
+        return K.add_rmsnorm_linear(x, None, nw, eps, w)[0]        # a handful of rows: the norm inside the product
+    h = torch.empty_like(x)
+    C.part_norm(x, nw, h, parts, float(eps))
+    return K.linear(h, w)
 
 
 # ---- routed experts ---------------------------------------------------------------------------------------------------
 
-def routed_experts(h, w13, w2, weights, index, limit, alpha):
+def routed_experts(h, w13, w2, weights, index, limit, alpha, shift=1.0, ungated=False):
     from . import cuda_more as M
     from .mixers import Addend
 
     T, k = index.shape
-    E, F2, D = w13.shape
-    glu = (float(limit), float(alpha))
-    if M.few_token_experts(h, w13, T, k):
-        act = torch.empty(T * k, F2 // 2, dtype=BF16, device=h.device)
+    E, rows, D = w13.shape
+    F = w2.shape[2]
+    glu = (0.0, 0.0, 0.0) if ungated else (float(limit), float(alpha), float(shift))
+    if M.few_token_experts(h, w13, T, k, ungated):
+        act = torch.empty(T * k, F, dtype=BF16, device=h.device)
         out = torch.empty_like(h)
-        C.moe_gemv(h, w13, w2, index, weights, act, out, 0, *glu)
+        C.moe_gemv(h, w13, w2, index, weights, act, out, 0, *glu, ungated)
         return Addend(out)
-    if h.dtype == BF16 and D % 8 == 0 and F2 % 16 == 0 and k <= 64 and E <= 2048:
+    if h.dtype == BF16 and D % 8 == 0 and F % 8 == 0 and k <= 64 and E <= 2048:
         bt = M.small_moe_bt(T * k, E, w13, w2)
         x_perm, seg, tile, dst = M.sort_by_expert(h, index, E, bt)
-        return Addend(M.experts_forward(x_perm, w13, w2, seg, tile, bt, glu)[1], weights, dst)
-    act = torch.empty(T * k, F2 // 2, dtype=h.dtype, device=h.device)
+        return Addend(M.experts_forward(x_perm, w13, w2, seg, tile, bt, "relu2" if ungated else glu)[1], weights, dst)
+    act = torch.empty(T * k, F, dtype=h.dtype, device=h.device)
     out = torch.empty_like(h)
     C.experts_any(h, w13, w2, index, weights, act, out, *glu)
     return Addend(out)

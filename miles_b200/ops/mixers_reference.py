@@ -13,12 +13,15 @@ def _sequences(meta, T: int):
     return [(b, cu[b], cu[b + 1]) for b in range(len(cu) - 1)]
 
 
-def bigram_embedding(tokens, prev, embed, table, spec):
+def bigram_embedding(tokens, prev, embed, table, spec, positions=None, freq=None):
     x = embed[tokens.long()].float()
     if table is not None:
         buckets, mp, mc = spec
         row = (prev.long() * mp + tokens.long() * mc) % buckets
         x = x + table[torch.where(prev < 0, torch.full_like(row, buckets), row)].float()
+    if freq is not None:
+        ang = positions.double()[:, None] * freq[None]
+        x = x + torch.stack([ang.sin(), ang.cos()], -1).flatten(1)[:, : x.shape[1]].float()
     return x, x.to(embed.dtype)
 
 
@@ -30,10 +33,19 @@ def output_norm_residual(x, y, nw, ls, eps, final_w=None):
     return x, (x * torch.rsqrt(x.square().mean(-1, keepdim=True) + eps) * final_w.float()).to(y.dtype)
 
 
-def clamped_glu(h, limit, alpha):
+def clamped_glu(h, limit, alpha, shift=1.0):
     g, u = h.float().chunk(2, -1)
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
-    return (g * torch.sigmoid(alpha * g) * (u + 1)).to(h.dtype)
+    return (g * torch.sigmoid(alpha * g) * (u + shift)).to(h.dtype)
+
+
+def aside(a):
+    if a is None:
+        return
+    if a.logits is not None:
+        a.weights, a.index = topk_softmax(a.logits, a.top) if a.routing is None else topk_grouped(a.logits, a.correction, a.top, a.routing)
+    if a.glu_in is not None:
+        a.glu_out.copy_(clamped_glu(a.glu_in[:, : 2 * a.glu_out.shape[1]], a.limit, a.alpha, a.shift))
 
 
 def rotate_pairs(x, positions, freq, magnitude):
@@ -107,17 +119,16 @@ def gated_norm(o, w, gate, eps):
     return (of * torch.rsqrt(of.square().mean(-1, keepdim=True) + eps) * w.float() * torch.sigmoid(gate.float())).to(o.dtype)
 
 
-def sum_norm(x, to, addends, extra, nw, eps):
+def sum_norm(x, to, addends, extra, nw, eps, shift=0.0, gain=1.0, nw2=None):
     s = x.clone()
     for a in addends:
-        s += a.y.float()
+        s += a.y.float() if a.scale is None else a.y.float() * a.scale.float()
     if extra is not None:
         s += extra
     if to is not None:
         to.copy_(s)
-    if nw is None:
-        return None
-    return (s * torch.rsqrt(s.square().mean(-1, keepdim=True) + eps) * nw.float()).to(nw.dtype)
+    n = s * torch.rsqrt(s.square().mean(-1, keepdim=True) + eps)
+    return tuple(None if w is None else (n * (w.float() + shift) * gain).to(w.dtype) for w in (nw, nw2))
 
 
 def projections(h, w, w2=None, b2=None):
@@ -132,12 +143,25 @@ def topk_softmax(logits, k):
     return torch.softmax(top.values, -1), top.indices.int()
 
 
-def routed_experts(h, w13, w2, weights, index, limit, alpha):
+def topk_grouped(logits, correction, k, r):
+    s = torch.sigmoid(logits.float())
+    c = s if correction is None else s + correction.float()
+    T, E = c.shape
+    by_group = c.view(T, r.groups, -1)
+    worth = by_group.topk(min(2, by_group.shape[-1]), -1).values.sum(-1)
+    closed = torch.ones(T, r.groups, dtype=torch.bool).scatter(1, worth.topk(r.keep, -1).indices, False)
+    idx = by_group.masked_fill(closed[..., None], float("-inf")).view(T, E).topk(k, -1).indices
+    w = s.gather(1, idx)
+    return w / (w.sum(-1, keepdim=True) + 1e-20) * r.scale, idx.int()
+
+
+def routed_experts(h, w13, w2, weights, index, limit=0.0, alpha=0.0, shift=1.0, ungated=False):
     out = torch.zeros(h.shape, dtype=torch.float32)
     for e in range(w13.shape[0]):
         t, j = torch.where(index == e)
         if t.numel():
-            y = clamped_glu(h[t] @ w13[e].T, limit, alpha) @ w2[e].T
+            up = h[t] @ w13[e].T
+            y = (up.float().relu().square().to(h.dtype) if ungated else clamped_glu(up, limit, alpha, shift)) @ w2[e].T
             out.index_add_(0, t, y.float() * weights[t, j][:, None])
     return out.to(h.dtype)
 
@@ -180,3 +204,74 @@ def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sin
         p = torch.softmax(sc, -1)[..., : keys.numel()]
         out[s0:s1] = torch.einsum("hts,shd->thd", p, vv).reshape(s1 - s0, -1).to(out.dtype)
     return out
+
+
+def differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lvec, q_norm, k_norm, eps):
+    T, H, G, d = proj.shape[0], lay.heads, lay.kv_heads, lay.dim
+
+    def normed(rows, heads, w):
+        x = rows.float().reshape(T, heads, 2, d)
+        return x * torch.rsqrt(x.square().mean(-1, keepdim=True) + eps) * w.float()
+
+    q = normed(proj[:, : lay.q_rows], H, q_norm)
+    if temperature is not None:
+        coef, every = temperature
+        q = q * (1 + coef * torch.log(torch.floor((meta.positions.double() + 1) / every) + 1)).float()[:, None, None, None]
+    q = q.to(proj.dtype).float()
+    bs = kc.shape[1]
+    if k_norm is not None:
+        k, v = proj[:, lay.q_rows: lay.gate_at].split([G * 2 * d, G * lay.vdim], -1)
+        ok = meta.slot_mapping >= 0
+        at = meta.slot_mapping[ok].long()
+        kc.view(-1, G, 2 * d)[at] = normed(k, G, k_norm).flatten(2)[ok].to(kc.dtype)
+        vc.view(-1, G, lay.vdim)[at] = v.reshape(T, G, lay.vdim)[ok].to(vc.dtype)
+    l = lvec.float()
+    lam = torch.exp((l[0] * l[1]).sum()) - torch.exp((l[2] * l[3]).sum()) + diff
+    out = torch.zeros(T, H, lay.vdim)
+    for b, s0, s1 in _sequences(meta, T):
+        if s1 == s0 or int(meta.slot_mapping[s0]) < 0:
+            continue
+        pos = meta.positions[s0:s1].long()
+        keys = torch.arange(int(pos[-1]) + 1)
+        slot = meta.block_table[b, keys // bs].long() * bs + keys % bs
+        kk = kc.view(-1, G, 2, d)[slot].float().repeat_interleave(H // G, 1)
+        vv = vc.view(-1, G, lay.vdim)[slot].float().repeat_interleave(H // G, 1)
+        sc = torch.einsum("thmd,shmd->mhts", q[s0:s1], kk) * scale
+        p = torch.softmax(sc.masked_fill(keys[None] > pos[:, None], float("-inf")), -1)
+        out[s0:s1] = torch.einsum("hts,shd->thd", p[0] - lam * p[1], vv)
+    out = out * torch.rsqrt(out.square().mean(-1, keepdim=True) + eps) * (1 - diff)
+    gate = proj[:, lay.gate_at: lay.gate_at + H].float()
+    return (out * torch.sigmoid(gate)[..., None]).reshape(T, H * lay.vdim).to(proj.dtype)
+
+
+def state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta):
+    T, H, V, N, G, taps = proj.shape[0], lay.heads, lay.vdim, lay.state, lay.groups, lay.taps
+    z, xbc, dt = proj[:, : lay.inner + lay.channels + H].split([lay.inner, lay.channels, H], -1)
+    dt = torch.nn.functional.softplus(dt.float() + dt_bias.float(), threshold=1e9)
+    decay = torch.exp(-torch.exp(A_log.float()) * dt)
+    out = torch.zeros(T, H, V)
+    for b, s0, s1 in _sequences(meta, T):
+        slot = int(meta.state_slots[b])
+        if slot < 0 or s1 == s0:
+            continue
+        p0 = int(meta.positions[s0])
+        before = [ring[slot, p % taps] if p >= 0 else torch.zeros(lay.channels) for p in range(p0 - taps + 1, p0)]
+        rows = torch.cat([torch.stack(before), xbc[s0:s1].float()]) if before else xbc[s0:s1].float()
+        act = conv_b.float() + sum(rows[k: k + s1 - s0] * conv[:, k].float() for k in range(taps))
+        x, B, C = torch.nn.functional.silu(act).to(proj.dtype).float().split([lay.inner, G * N, G * N], -1)
+        if ring is not None:
+            for t in range(max(s0, s1 - taps + 1), s1):
+                ring[slot, (p0 + t - s0) % taps] = xbc[t].float()
+        x = x.view(-1, H, V)
+        B, C = (y.reshape(-1, G, N).repeat_interleave(H // G, 1) for y in (B, C))
+        S = state[slot].clone() if p0 > 0 else torch.zeros_like(state[slot])
+        for i, t in enumerate(range(s0, s1)):
+            S = S * decay[t][:, None, None] + (dt[t][:, None] * B[i])[:, :, None] * x[i][:, None, :]
+            out[t] = torch.einsum("hnv,hn->hv", S, C[i]) + D.float()[:, None] * x[i]
+        state[slot] = S
+    return (out.reshape(T, lay.inner) * torch.nn.functional.silu(z.float())).to(proj.dtype)
+
+
+def part_norm(x, w, parts, eps):
+    p = x.float().unflatten(-1, (parts, -1))
+    return ((p * torch.rsqrt(p.square().mean(-1, keepdim=True) + eps)).flatten(-2) * w.float()).to(x.dtype)
