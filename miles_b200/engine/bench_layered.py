@@ -1,6 +1,8 @@
 """Prefill and decode of a layer-by-layer decoder beside the closest grouped-query model of equal width, depth and feed-forward.
 
-    python bench.py --layered [--layered-model nopelorn-4B-shape | ronupel-30B-A3B-shape] [--layered-baseline NAME] [--layers N]
+    python bench.py --layered [--layered-model NAME] [--layered-baseline NAME] [--layers N]
+
+NAME: nopelorn-4B-shape, ronupel-30B-A3B-shape or vozirax-30B-A3B-shape.
 
 The baseline is qwen3-4B for a dense model and qwen3-30B-A3B for one with routed experts, with as many layers as the layered model has
 layer runs.
@@ -375,6 +377,142 @@ def attention_kernels(cfg, base) -> list[dict]:
     return out.rows
 
 
+@torch.no_grad()
+def hybrid_kernels(cfg, base) -> list[dict]:
+    """Differential attention, the state-space mixer, ungated experts and the sums with two norms beside the grouped-query mixture's kernels
+    (and beside linear attention with as large a state)."""
+    from ..models.layered import DifferentialSpec, MoeSpec, SsmSpec
+    from ..ops import cuda as K
+    from ..ops import mixers as MX
+    from ..ops import mixers_cuda as MC
+
+    out = _Rows()
+    add, t = out.add, _randn
+    D = cfg.hidden_size
+    m = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, DifferentialSpec))
+    c = next(s.mixer for s in cfg.layer_specs if isinstance(s.mixer, SsmSpec))
+    f = next(s.mlp for s in cfg.layer_specs if isinstance(s.mlp, MoeSpec))
+    lay, ss = MX.DifferentialLayout(m.heads, m.kv_heads, m.dim, m.vdim), MX.SsmLayout(c.heads, c.vdim, c.state, c.groups, c.conv)
+    pair, H, G = lay.paired, m.heads, m.kv_heads
+    hq, hk, d = base.num_heads, base.num_kv_heads, base.head_dim
+    pitch = -(-pair.dim // 64) * 64
+    sizes = [pair.heads, pair.kv_heads, pair.dim, pair.vdim, 0, 0, 0, pitch]
+    lam, qn, lvec = torch.full((1,), 0.6, device="cuda"), t(m.dim), t(4, m.dim)
+
+    def diff(gates):
+        return lam, gates, 0.2, 1e-6
+
+    conv, conv_b, vec, Dv = t(ss.channels, c.conv), t(ss.channels), t(c.heads), t(c.heads)
+    lin_h, lin_d = c.heads * c.vdim // c.state, c.state              # linear attention with a state of the same size
+    for n, length in ((1, 8192), (8, 1024), (1, 1024)):
+        T = n * length
+        meta, nb = _ragged([(0, length)] * n)
+        q, kc, vc, o, gates = t(T, 2 * H, pitch), t(nb, 64, G, pair.dim), t(nb, 64, G, m.vdim), t(T, H * m.vdim), t(T, H)
+        pairs = n * length * (length + 1) / 2
+        add("differential prefill (two maps, norm, gate)", "flash_fwd_tc", f"{n}x{length}",
+            lambda: MC._paged_attention(q, pair, kc, vc, meta, o, m.scale, None, sizes, True, diff(gates)),
+            2 * (T * 2 * H * m.dim + kc.numel() + vc.numel() + o.numel()), 4.0 * pairs * H * (m.dim + m.vdim))
+        q2, k2, v2 = t(T, hq, d), t(T, hk, d), t(T, hk, d)
+        add("flash_fwd_tc", "", f"{n}x{length}", lambda: K.attention_varlen(q2, k2, v2, meta.ragged.cu_q, length), 2 * (2 * q2.numel() + 2 * k2.numel()),
+            4.0 * pairs * hq * d)
+        del q, kc, vc, o, q2, k2, v2
+        proj, xbc = t(T, ss.inner + ss.channels + c.heads), t(T, ss.channels)
+        step, decay = torch.rand(T, c.heads, device="cuda") * 0.1, -torch.rand(T, c.heads, device="cuda") * 0.1
+        state, ring = torch.zeros(n, c.heads, c.state, c.vdim, device="cuda"), torch.zeros(n, c.conv, ss.channels, device="cuda")
+        w = [conv, conv_b, vec, vec, Dv, state, ring, meta.state_slots, meta.positions]
+        segs, seq_segs, multi = MC._segments(meta, c.heads // K.C.ssm_heads_per_cta(c.heads, c.vdim, c.groups))
+        seg_state = torch.empty(segs.shape[0], c.heads, c.state, c.vdim, device="cuda") if multi else None
+        seg_decay = torch.empty(segs.shape[0], c.heads, device="cuda") if multi else None
+        y, S, C = t(T, ss.inner), [c.heads, c.vdim, c.state, c.groups, c.conv], 64
+        add("ssm_chunk (segments + scan + outputs, gate)", "linear_chunk", f"{n}x{length}",
+            lambda: K.C.ssm_chunk(proj, xbc, step, decay, S, w, segs, seq_segs, seg_state, seg_decay, y),
+            2 * T * (2 * ss.inner + ss.channels) + 8 * T * c.heads + 8 * state.numel(),
+            2.0 * T * ((C + 1) / 2 * (c.groups * c.state + c.heads * c.vdim) + 2 * c.heads * c.state * c.vdim))
+        lin = t(T, lin_h * 4 * lin_d)
+        dec, lst = torch.rand(lin_h, device="cuda"), torch.zeros(n, lin_h, lin_d, lin_d, device="cuda")
+        add("linear_chunk (segments + scan + outputs)", "", f"{n}x{length}", lambda: MC.linear_state(lin, lin_h, lin_d, lin_d, dec, lst, meta),
+            2 * T * lin_h * 4 * lin_d + 8 * lst.numel(), 2.0 * T * lin_h * ((C + 1) / 2 * 2 * lin_d + 2 * lin_d * lin_d))
+        tiles = MC._conv_tiles(meta, c.conv)
+        add("ssm_conv (convolution, step sizes)", "swiglu", f"{n}x{length}",
+            lambda: K.C.ssm_conv(proj, S, w, tiles, meta.ragged.cu_q, xbc, step, decay, *MC._aside(None, T)), 4 * T * ss.channels + 10 * T * c.heads)
+        h = t(T, 2 * ss.channels)
+        add("swiglu", "", f"{n}x{length}", lambda: K.swiglu(h), 6 * T * ss.channels)
+        del proj, xbc, lin, h
+    for B, ctx in ((1, 4096), (8, 4096), (64, 4096)):
+        meta, nb = _ragged([(ctx - 1, 1)] * B)
+        kc, vc, o, gates, q = t(nb, 64, G, pair.dim), t(nb, 64, G, m.vdim), t(B, H * m.vdim), t(B, H), t(B, 2 * H, pitch)
+        add("differential decode (two maps, norm, gate)", "paged_decode", f"{B} rows, {ctx} keys",
+            lambda: MC._paged_attention(q, pair, kc, vc, meta, o, m.scale, None, sizes, True, diff(gates)),
+            2 * B * (ctx * G * (pair.dim + m.vdim) + H * (2 * m.dim + m.vdim)), 4.0 * B * ctx * H * (m.dim + m.vdim))
+        kb, vb, q2 = t(nb, 64, hk, d), t(nb, 64, hk, d), t(B, hq, d)
+        L = torch.full((B,), ctx, dtype=torch.int32, device="cuda")
+        add("paged_decode + merge", "", f"{B} rows, {ctx} keys", lambda: K.paged_attention(q2, kb, vb, meta.block_table, L),
+            2 * B * (ctx * 2 * hk * d + 2 * hq * d), 4.0 * B * ctx * hq * d)
+        del kc, vc, kb, vb
+        proj, y = t(B, ss.inner + ss.channels + c.heads), t(B, ss.inner)
+        state, ring = torch.zeros(B, c.heads, c.state, c.vdim, device="cuda"), torch.zeros(B, c.conv, ss.channels, device="cuda")
+        w = [conv, conv_b, vec, vec, Dv, state, ring, meta.state_slots, meta.positions]
+        S = [c.heads, c.vdim, c.state, c.groups, c.conv]
+        add("ssm_step (convolution, state, gate)", "linear_state step", f"{B} rows", lambda: K.C.ssm_step(proj, S, w, y, *MC._aside(None, B)),
+            8 * state.numel() + 4 * ring.numel() + 2 * B * (2 * ss.inner + ss.channels))
+        lin, dec = t(B, lin_h * 4 * lin_d), torch.rand(lin_h, device="cuda")
+        lst = torch.zeros(B, lin_h, lin_d, lin_d, device="cuda")
+        add("linear_state step", "", f"{B} rows", lambda: MC.linear_state(lin, lin_h, lin_d, lin_d, dec, lst, meta), 8 * lst.numel() + 2 * B * lin_h * 4 * lin_d)
+    nw, corr, z = t(D), t(f.experts), t(ss.inner)
+    w_in = torch.nn.Parameter(t(ss.inner + ss.channels + c.heads, D))
+    router, wo = torch.nn.Parameter(t(f.experts, D)), torch.nn.Parameter(t(D, ss.inner))
+    wqkv = torch.nn.Parameter(t(base.qkv_size, D))
+    for T in (8, 8192):
+        meta, nb = _ragged([(0, T)] if T > 8 else [(4000, 1)] * T)
+        kc, vc, q = t(nb, 64, G, pair.dim), t(nb, 64, G, m.vdim), t(T, 2 * H, pitch)
+        proj, logits = t(T, lay.gate_at + H), t(T, f.experts, dtype=torch.float32)
+        a = MX.Aside(logits=logits, top=f.top, routing=f.routing, correction=corr)
+        add("diff_prep (norms, temperature, cache, experts)", "qk_norm_rope_cache", f"{T} rows",
+            lambda: K.C.diff_prep(proj, meta.positions, meta.slot_mapping, qn, qn, lvec, lam, kc, vc, q, [H, G, m.dim, m.vdim, pitch], 1e-6, 0.1, 8192.0,
+                                  0.8, *MC._aside(a, T)),
+            2 * T * (2 * lay.gate_at + 2 * H * m.dim) + 4 * T * f.experts)
+        q2, k2, v2, qw = t(T, hq, d), t(T, hk, d), t(T, hk, d), t(d)
+        kb, vb = t(nb, 64, hk, d), t(nb, 64, hk, d)
+        add("qk_norm_rope_cache", "", f"{T} rows", lambda: K.qk_norm_rope_cache(q2, k2, v2, qw, qw, meta.positions, 1e6, 1e-6, kb, vb, meta.slot_mapping),
+            2 * (2 * q2.numel() + 5 * k2.numel()))
+        add("router_topk", "", f"{T} rows", lambda: K.router_topk(logits, f.top), 4 * T * f.experts)
+        y, y2 = t(T, ss.inner), t(T, ss.inner)
+        add("part_norm (state-space output)", "add_rmsnorm", f"{T} rows", lambda: K.C.part_norm(y, z, y2, c.norm_groups, 1e-6), 4 * y.numel())
+        x, to, o, r2 = t(T, D, dtype=torch.float32), t(T, D, dtype=torch.float32), t(T, D), t(T, D)
+        add("sum_norm (one scaled addend, two norms)", "add_rmsnorm", f"{T} rows",
+            lambda: MC.sum_norm(x, to, [MX.Addend(o, scale=nw)], None, nw, 1e-6, 1.0, 1.0, nw), T * D * 14)
+        add("add_rmsnorm", "", f"{T} rows", lambda: K.add_rmsnorm(o, r2, nw, 1e-6), T * D * 8)
+        if T > 8:
+            xp, seg, tile, dst = K.sort_by_expert(o, torch.rand(T, f.experts, device="cuda").topk(f.top).indices.int(), f.experts, 128)
+            e = MX.Addend(t(*xp.shape), torch.rand(T, f.top, device="cuda"), dst, nw)
+            add("sum_norm (addend, experts' rows, two norms)", "moe_combine + add_rmsnorm", f"{T} rows",
+                lambda: MC.sum_norm(x, to, [MX.Addend(o, scale=nw), e], None, nw, 1e-6, 1.0, 1.0, nw), T * D * (14 + 2 * f.top))
+            add("moe_combine + add_rmsnorm", "", f"{T} rows",
+                lambda: (K.C.moe_combine(e.y, e.weights, dst, r2, f.top), K.add_rmsnorm(o, r2, nw, 1e-6)), T * D * (2 * f.top + 2 + 8))
+    for T in (1, 4):
+        x, o, o2, r2 = t(T, D, dtype=torch.float32), t(T, D), t(T, D), t(T, D)
+        add("sum_two_norms_linear (+ router)", "add_rmsnorm_linear", f"{T} rows",
+            lambda: MC.sum_two_norms_linear(x, [MX.Addend(o, scale=nw), MX.Addend(o2, scale=nw)], nw, w_in, nw, router, 1e-6, 1.0, True),
+            2 * (w_in.numel() + router.numel()))
+        add("add_rmsnorm_linear", "", f"{T} rows", lambda: K.add_rmsnorm_linear(o, r2, nw, 1e-6, wqkv), 2 * wqkv.numel())
+        y = t(T, ss.inner)
+        add("part_norm_linear (norm inside the output projection)", "add_rmsnorm_linear", f"{T} rows",
+            lambda: MC.part_norm_linear(y, z, c.norm_groups, 1e-6, wo), 2 * wo.numel())
+    for T in (1, 8, 64, 8192):
+        h = t(T, D)
+        w1, w2 = t(f.experts, f.up_rows, D), t(f.experts, D, f.expert.ff)
+        Fb = base.moe_ffn_hidden_size
+        b13, b2 = t(f.experts, 2 * Fb, D), t(f.experts, D, Fb)
+        idx = torch.rand(T, f.experts, device="cuda").topk(f.top).indices.int()
+        w = torch.rand(T, f.top, device="cuda")
+        used = idx.unique().numel()
+        nbytes, flops = 2.0 * used * 2 * D * f.expert.ff + 4 * T * D, 4.0 * T * f.top * D * f.expert.ff
+        add("routed_experts (squared relu; sum left to sum_norm)" if T > 8 else "routed_experts (squared relu)", "moe_ffn", f"{T} rows, {used} experts",
+            lambda: MC.routed_experts(h, w1, w2, w, idx, 0.0, 0.0, 0.0, True), nbytes, flops)
+        add("moe_ffn", "", f"{T} rows, {used} experts", lambda: K.moe_ffn(h, b13, b2, w, idx), 2.0 * used * 3 * D * Fb + 4 * T * D, 6.0 * T * f.top * D * Fb)
+    return out.rows
+
+
 def main(a) -> int:
     from ..models.config import get_config
     from ..ops import build
@@ -389,7 +527,7 @@ def main(a) -> int:
     for c in (cfg, base):
         print(json.dumps(throughput(c)), flush=True)
         torch.cuda.empty_cache()
-    kinds = {"attention": attention_kernels, "latent": latent_kernels}
+    kinds = {"attention": attention_kernels, "latent": latent_kernels, "hybrid": hybrid_kernels}
     for r in kinds[build.serve_kind(cfg)](cfg, base):
         print(json.dumps(r), flush=True)
     print(json.dumps({"kernel_error_flag": K.check_error_flag()}))

@@ -55,7 +55,7 @@ __device__ __forceinline__ void norm_rows(const T* __restrict__ x, const T* __re
   }
 }
 
-template <typename T, bool VEC>
+template <typename T, bool VEC, bool GROUPED>
 __global__ void __launch_bounds__(kDiff) diff_prep_kernel(const T* __restrict__ proj, long long ld, const int* __restrict__ positions,
                                                           const long long* __restrict__ slots, const T* __restrict__ q_norm,
                                                           const T* __restrict__ k_norm, const T* __restrict__ lvec, float* __restrict__ lam,
@@ -67,7 +67,7 @@ __global__ void __launch_bounds__(kDiff) diff_prep_kernel(const T* __restrict__ 
   const T* p = proj + t * ld;
   const int nq = L.heads * 2 * L.dim, nk = L.kv_heads * 2 * L.dim, nv = L.kv_heads * L.vdim;
   if (blockIdx.y == (L.kv_heads > 0 ? 2 : 1)) {
-    aside_row<T, VEC, kDiff>(a, t);
+    aside_row<T, VEC, kDiff, GROUPED>(a, t);
     return;
   }
   if (blockIdx.y == 0) {
@@ -147,7 +147,8 @@ extern "C" int mb_diff_prep(const void* proj, long long ld, const int* positions
     constexpr int v = 16 / static_cast<int>(sizeof(E));
     const bool vec = ld % v == 0 && L.dim % v == 0 && L.dim <= 32 * v && L.vdim % v == 0 && L.q_pitch % v == 0 &&
                      (reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q)) % 16 == 0 && aside_vec<E>(a);
-    auto kern = vec ? diff_prep_kernel<E, true> : diff_prep_kernel<E, false>;
+    auto kern = a.grouped ? (vec ? diff_prep_kernel<E, true, true> : diff_prep_kernel<E, false, true>)
+                          : (vec ? diff_prep_kernel<E, true, false> : diff_prep_kernel<E, false, false>);
     return static_cast<int>(launch_pdl(kern, dim3(T, (L.kv_heads > 0 ? 2 : 1) + aside_on(a)), dim3(kDiff), 0, s, reinterpret_cast<const E*>(proj), ld,
                                        positions, slots, reinterpret_cast<const E*>(q_norm), reinterpret_cast<const E*>(k_norm),
                                        reinterpret_cast<const E*>(lvec), lam, reinterpret_cast<E*>(kc), reinterpret_cast<E*>(vc),

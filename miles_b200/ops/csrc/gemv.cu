@@ -212,6 +212,7 @@ __device__ __forceinline__ void stage_rows_output_norm(uint8_t* xs, int rows, in
 
 // Sum-norm form: x' = x + y1·s1 + y2·s2 + extra (fp32 x and extra, every addend and scale optional; block 0 writes x' to x_out, another
 // buffer); the staged value is bf16(x' · (norm_w + shift)), Σx'² → rstd[row].
+template <bool SCALED>
 __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int valid, int K, const float* __restrict__ x,
                                                     const bf16* __restrict__ y1, const bf16* __restrict__ s1, const bf16* __restrict__ y2,
                                                     const bf16* __restrict__ s2, const float* __restrict__ extra,
@@ -235,8 +236,8 @@ __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int v
       const uint4 zero = make_uint4(0, 0, 0, 0), one = make_uint4(0x3f803f80u, 0x3f803f80u, 0x3f803f80u, 0x3f803f80u);
       const uint4 p1 = y1 != nullptr ? *reinterpret_cast<const uint4*>(y1 + at) : zero;
       const uint4 p2 = y2 != nullptr ? *reinterpret_cast<const uint4*>(y2 + at) : zero;
-      const uint4 q1 = s1 != nullptr ? *reinterpret_cast<const uint4*>(s1 + v * 8) : one;
-      const uint4 q2 = s2 != nullptr ? *reinterpret_cast<const uint4*>(s2 + v * 8) : one;
+      const uint4 q1 = SCALED && s1 != nullptr ? *reinterpret_cast<const uint4*>(s1 + v * 8) : one;
+      const uint4 q2 = SCALED && s2 != nullptr ? *reinterpret_cast<const uint4*>(s2 + v * 8) : one;
       const uint4 nw = *reinterpret_cast<const uint4*>(norm_w + v * 8);
       f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
       if (extra != nullptr) {
@@ -249,10 +250,10 @@ __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int v
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float2 u = unpack2(w1[i]), q = unpack2(w2[i]), n = unpack2(wn[i]), c = unpack2(l1[i]), d = unpack2(l2[i]);
-        f[2 * i] += u.x * c.x + q.x * d.x;
-        f[2 * i + 1] += u.y * c.y + q.y * d.y;
+        f[2 * i] += SCALED ? u.x * c.x + q.x * d.x : u.x + q.x;
+        f[2 * i + 1] += SCALED ? u.y * c.y + q.y * d.y : u.y + q.y;
         ss += f[2 * i] * f[2 * i] + f[2 * i + 1] * f[2 * i + 1];
-        o[i] = pack2(f[2 * i] * (n.x + shift), f[2 * i + 1] * (n.y + shift));
+        o[i] = SCALED ? pack2(f[2 * i] * (n.x + shift), f[2 * i + 1] * (n.y + shift)) : pack2(f[2 * i] * n.x, f[2 * i + 1] * n.y);
       }
       if (x_out != nullptr && blockIdx.x == 0) {
         *reinterpret_cast<float4*>(x_out + at) = make_float4(f[0], f[1], f[2], f[3]);
@@ -308,13 +309,14 @@ struct GemvParams {
   int static_w;           // W is not written by a kernel that may still run: its first loads go before the dependency wait
 };
 
-enum GemvMode { kPlain = 0, kAddNorm = 1, kOutputNorm = 2, kSumNorm = 3 };
+enum GemvMode { kPlain = 0, kAddNorm = 1, kOutputNorm = 2, kSumNorm = 3, kScaledSum = 4 };      // kScaledSum: kSumNorm with scales, shifted norm weights, two norms
 
 // NT: groups of 8 tokens (1 or 2); S: ring stages.  One CTA = 16 output rows; its 8 warps take the 32-wide k chunks round-robin.
 template <int NT, int MODE, int S>
 __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   constexpr bool NORM = MODE == kAddNorm;
-  constexpr bool SCALED = NORM || MODE == kSumNorm;      // the staged rows still lack 1 / rms
+  constexpr bool SUM = MODE == kSumNorm || MODE == kScaledSum;
+  constexpr bool SCALED = NORM || SUM;                   // the staged rows still lack 1 / rms
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float red[kWarps][NT][16][8];
   __shared__ float rstd_s[NT * 8];
@@ -349,8 +351,8 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
     stage_rows<true>(xs, NT * 8, p.M, p.K, p.x, p.residual, p.norm_w, p.eps, p.res_out, rstd_s);
   } else if (MODE == kOutputNorm) {
     stage_rows_output_norm(xs, NT * 8, p.M, p.K, p.x, p.x32, p.norm_w, p.scale_w, p.eps, p.x32_out);
-  } else if (MODE == kSumNorm) {
-    stage_rows_sum_norm(xs, NT * 8, p.M, p.K, p.x32, p.y1, p.s1, p.y2, p.s2, p.extra, second && p.norm_w2 != nullptr ? p.norm_w2 : p.norm_w, p.eps,
+  } else if (SUM) {
+    stage_rows_sum_norm<MODE == kScaledSum>(xs, NT * 8, p.M, p.K, p.x32, p.y1, p.s1, p.y2, p.s2, p.extra, second && p.norm_w2 != nullptr ? p.norm_w2 : p.norm_w, p.eps,
                         p.shift, p.x32_out, rstd_s);
   } else {
     stage_rows_async(xs, NT * 8, p.M, p.K, p.x);
@@ -399,7 +401,7 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
       else reinterpret_cast<bf16*>(p.y)[tok * p.ldy + n] = __float2bfloat16(s);
     }
   }
-  if (MODE == kSumNorm && p.xn_out != nullptr && blockIdx.x == 0) {
+  if (SUM && p.xn_out != nullptr && blockIdx.x == 0) {
     const float* xr = p.x32_out != nullptr ? p.x32_out : p.x32;      // this CTA's own writes, or nothing was added
     for (int i = threadIdx.x; i < p.M * (p.K / 8); i += kThreads) {
       const int tok = i / (p.K / 8), kv = (i % (p.K / 8)) * 8;
@@ -802,6 +804,8 @@ extern "C" int mb_gemv_sum_norm(MbGemvSum a, cudaStream_t s) {
   p.xn_out = reinterpret_cast<bf16*>(a.xn_out);
   p.M = a.M; p.N = a.N; p.K = a.K; p.static_w = a.static_w;
   if (a.x32 == nullptr) return static_cast<int>(nt == 1 ? launch_gemv<1, kPlain>(p, s) : launch_gemv<2, kPlain>(p, s));
+  if (p.s1 != nullptr || p.s2 != nullptr || p.norm_w2 != nullptr || p.shift != 0.f)
+    return static_cast<int>(nt == 1 ? launch_gemv<1, kScaledSum>(p, s) : launch_gemv<2, kScaledSum>(p, s));
   return static_cast<int>(nt == 1 ? launch_gemv<1, kSumNorm>(p, s) : launch_gemv<2, kSumNorm>(p, s));
 }
 

@@ -327,8 +327,8 @@ typedef struct {
   const int* slots;                          // per sequence
   const int* positions;                      // per token
 } MbSsm;
-// Convolution, step sizes and log decays of any pieces.  tiles [n][4]: first token, end (32 tokens but for a piece's last tile), sequence, 1 for a
-// piece's first tile; null: one token per sequence.  xbc [T, channels], dt and la [T, H].
+// Convolution, step sizes and log decays of any pieces.  tiles [n][4]: first token, end (at least taps − 1 tokens but for a piece's last tile),
+// sequence, 1 for a piece's first tile; null: one token per sequence.  xbc [T, channels], dt and la [T, H].
 int mb_ssm_conv(const void* proj, long long ld, MbSsm m, const int* tiles, const int* cu_q, int n_tiles, void* xbc, float* dt, float* la, int T,
                 MbAside a, int f32, cudaStream_t s);
 // One token per sequence: convolution, state, gate in one kernel; out [T, H·V] = y · silu(z).  V % 4 == 0.

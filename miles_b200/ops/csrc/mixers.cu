@@ -132,7 +132,8 @@ __global__ void __launch_bounds__(256) relu_square_kernel(T* __restrict__ x, lon
 
 // One CTA per token; the sum waits in shared memory for its norm.  Addends: see MbSumNorm.
 static constexpr int kMaxTop = 64;
-template <typename T, int V>
+// SCALED: with scales of the addends, or a second norm.
+template <typename T, int V, bool SCALED>
 __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
   extern __shared__ __align__(16) float row[];
   __shared__ float sh[kRow / 32], s_w[kMaxTop];
@@ -161,8 +162,8 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
     float r[V], a[V], c1[V], c2[V];
 #pragma unroll
     for (int j = 0; j < V; ++j) c1[j] = c2[j] = 1.f;
-    if (s1 != nullptr) load_n<V>(s1 + i, c1);
-    if (s2 != nullptr) load_n<V>(s2 + i, c2);
+    if (SCALED && s1 != nullptr) load_n<V>(s1 + i, c1);
+    if (SCALED && s2 != nullptr) load_n<V>(s2 + i, c2);
     load_n<V>(p.x + base + i, r);
     if (y1 != nullptr) {
       load_n<V>(y1 + base + i, a);
@@ -213,7 +214,7 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
       w[j] = r[j] * (w[j] + p.shift) * p.gain;
     }
     store_n<V>(h + base + i, w);
-    if (nw2 == nullptr) continue;
+    if (!SCALED || nw2 == nullptr) continue;
     load_n<V>(nw2 + i, w);
 #pragma unroll
     for (int j = 0; j < V; ++j) w[j] = r[j] * (w[j] + p.shift) * p.gain;
@@ -373,10 +374,14 @@ extern "C" int mb_sum_norm(MbSumNorm p, int f32, cudaStream_t s) {
   const int bytes = p.D * static_cast<int>(sizeof(float));
   if (bytes > 200 * 1024) return -3;
   return dispatch(f32, p.D % 8 == 0, [&](auto ty, auto v) {
-    auto kern = sum_norm_kernel<decltype(ty), decltype(v)::value>;
-    static int configured = 48 * 1024;                 // one per instantiation
+    using E = decltype(ty);
+    constexpr int V = decltype(v)::value;
+    const bool scaled = p.s1 != nullptr || p.s2 != nullptr || p.nw2 != nullptr;
+    auto kern = scaled ? sum_norm_kernel<E, V, true> : sum_norm_kernel<E, V, false>;
+    static int configured = 48 * 1024;                 // one per dtype and vector
     if (bytes > configured) {
-      const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      cudaError_t e = cudaFuncSetAttribute(sum_norm_kernel<E, V, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      if (e == cudaSuccess) e = cudaFuncSetAttribute(sum_norm_kernel<E, V, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
       if (e != cudaSuccess) return static_cast<int>(e);
       configured = 200 * 1024;
     }

@@ -294,11 +294,11 @@ __device__ __forceinline__ void topk_grouped_row(const float* __restrict__ z, co
 }
 
 // What runs beside a mixer's preparation for token t, by a CTA of THREADS threads: its choice of experts and the activation of its
-// dense feed-forward (see MbAside).
-template <typename T, bool VEC, int THREADS>
+// dense feed-forward (see MbAside).  GROUPED: the kernel holds the choice among groups instead of the softmax one.
+template <typename T, bool VEC, int THREADS, bool GROUPED>
 __device__ __forceinline__ void aside_row(const MbAside& a, long long t) {
   if (a.logits != nullptr && threadIdx.x < 32) {
-    if (a.grouped)
+    if constexpr (GROUPED)
       topk_grouped_row<T>(a.logits + t * a.experts, reinterpret_cast<const T*>(a.correction), a.experts, a.top, a.groups, a.keep, a.scale,
                           a.weights + t * a.top, a.index + t * a.top);
     else

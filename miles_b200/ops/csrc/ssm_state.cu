@@ -12,7 +12,41 @@
 namespace mb {
 namespace mx {
 
-static constexpr int kConvTile = 32, kConv = 128, kConvTaps = 33;      // tokens per tile, threads, most taps
+static constexpr int kConv = 128, kConvTaps = 33;      // threads, most taps (a tile has at least taps − 1 tokens)
+
+// silu of neighbours; in bf16 two share one reciprocal: 1/a = b · 1/(ab).  Arguments below −40 count as −40 in the exponential (the result
+// is zero to 15 digits either way), which keeps the product finite.
+template <typename T, int V> __device__ __forceinline__ void silu_n(float (&y)[V]) {
+  if constexpr (is_exact<T>::value || V % 2) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = silu_t<T>(y[j]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < V; j += 2) {
+      const float a = 1.f + __expf(fminf(-y[j], 40.f)), b = 1.f + __expf(fminf(-y[j + 1], 40.f));
+      const float r = __fdividef(1.f, a * b);
+      y[j] *= r * b;
+      y[j + 1] *= r * a;
+    }
+  }
+}
+
+// V values as they lie in memory (16 bytes, or one value), and as floats
+template <typename T, int V> struct Raw {
+  uint4 v;
+  __device__ __forceinline__ void load(const T* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void get(float (&f)[V]) const {
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int j = 0; j < V; ++j)
+      f[j] = sizeof(T) == 4 ? __uint_as_float(w[j % 4]) : __uint_as_float((j & 1) ? w[j / 2 % 4] & 0xffff0000u : w[j / 2 % 4] << 16);
+  }
+};
+template <typename T> struct Raw<T, 1> {
+  T v;
+  __device__ __forceinline__ void load(const T* p) { v = *p; }
+  __device__ __forceinline__ void get(float (&f)[1]) const { f[0] = to_f(v); }
+};
 
 template <typename T> __device__ __forceinline__ float softplus_t(float x) {
   if constexpr (is_exact<T>::value) {
@@ -25,7 +59,7 @@ template <typename T> __device__ __forceinline__ float softplus_t(float x) {
 }
 
 // 1-D grid: n_tiles · (channel blocks + 1), then one CTA per token for the aside.  TAPS 0: any number, one load per tap and token.
-template <typename T, int V, int TAPS>
+template <typename T, int V, int TAPS, bool GROUPED>
 __global__ void __launch_bounds__(kConv) ssm_conv_kernel(const T* __restrict__ proj, long long ld, MbSsm m, const int* __restrict__ tiles,
                                                          const int* __restrict__ cu_q, int n_tiles, int blocks, T* __restrict__ xbc,
                                                          float* __restrict__ dt, float* __restrict__ la, MbAside a) {
@@ -33,17 +67,15 @@ __global__ void __launch_bounds__(kConv) ssm_conv_kernel(const T* __restrict__ p
   pdl_wait();
   const int inner = m.H * m.V, CH = inner + 2 * m.G * m.N;
   if (static_cast<int>(blockIdx.x) >= n_tiles * (blocks + 1)) {
-    aside_row<T, V != 1, kConv>(a, blockIdx.x - n_tiles * (blocks + 1));
+    aside_row<T, V != 1, kConv, GROUPED>(a, blockIdx.x - n_tiles * (blocks + 1));
     return;
   }
   const int tile = blockIdx.x / (blocks + 1), cb = blockIdx.x % (blocks + 1);
-  int t0 = tile, t1 = tile + 1, seq = tile, first = 1, begin = tile, end = tile + 1;
+  int t0 = tile, t1 = tile + 1, seq = tile, first = 1;
   if (tiles != nullptr) {
-    t0 = tiles[tile * 4]; t1 = tiles[tile * 4 + 1]; seq = tiles[tile * 4 + 2]; first = tiles[tile * 4 + 3];
-    begin = cu_q[seq]; end = cu_q[seq + 1];
+    const int4 v = reinterpret_cast<const int4*>(tiles)[tile];
+    t0 = v.x; t1 = v.y; seq = v.z; first = v.w;
   }
-  const int slot = m.slots[seq];
-  if (slot < 0) return;                                  // padding row of a decode batch
   if (cb == blocks) {
     const T* bias = reinterpret_cast<const T*>(m.dt_bias);
     const T* al = reinterpret_cast<const T*>(m.A_log);
@@ -59,9 +91,23 @@ __global__ void __launch_bounds__(kConv) ssm_conv_kernel(const T* __restrict__ p
   if (c >= CH) return;
   const T* in = proj + inner + c;
   const T* W = reinterpret_cast<const T*>(m.conv_w) + static_cast<long long>(c) * m.taps;
+  // weights and the first tokens are on their way before anything is known of the sequence
+  constexpr int U = 4;
+  Raw<T, V> packed[TAPS > 0 ? TAPS : 1], cur[U];         // V · TAPS weights side by side
+  if constexpr (TAPS > 0) {
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) packed[k].load(W + k * V);
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (t0 + u < t1) cur[u].load(in + (t0 + u) * ld);
+  }
+  float b[V];
+  load_n<V>(reinterpret_cast<const T*>(m.conv_b) + c, b);
+  const int slot = m.slots[seq], pos0 = m.positions[t0];
+  const int begin = tiles != nullptr ? cu_q[seq] : tile, end = tiles != nullptr ? cu_q[seq + 1] : tile + 1;
+  if (slot < 0) return;                                  // padding row of a decode batch
   float* ring = m.ring != nullptr ? m.ring + static_cast<long long>(slot) * m.taps * CH + c : nullptr;
   const int taps = TAPS ? TAPS : m.taps;
-  const int pos0 = m.positions[t0];
   // the input `back` places before token t (t − back ≥ t0 − taps + 1)
   auto before = [&](int t, int back, float (&f)[V]) {
     if (t - back >= begin) {
@@ -74,36 +120,45 @@ __global__ void __launch_bounds__(kConv) ssm_conv_kernel(const T* __restrict__ p
 #pragma unroll
       for (int j = 0; j < V; ++j) f[j] = 0.f;
   };
-  float b[V];
-  load_n<V>(reinterpret_cast<const T*>(m.conv_b) + c, b);
   auto finish = [&](int t, float (&y)[V]) {
-#pragma unroll
-    for (int j = 0; j < V; ++j) y[j] = silu_t<T>(y[j]);
+    silu_n<T, V>(y);
     store_n<V>(xbc + static_cast<long long>(t) * CH + c, y);
   };
   if constexpr (TAPS > 0) {
     float w[TAPS][V], x[TAPS][V];                        // x[k]: the input taps − 1 − k places back
 #pragma unroll
-    for (int j = 0; j < V; ++j)
-#pragma unroll
-      for (int k = 0; k < TAPS; ++k) w[k][j] = to_f(W[j * TAPS + k]);
-#pragma unroll
     for (int k = 0; k < TAPS - 1; ++k) before(t0, TAPS - 1 - k, x[k]);
-#pragma unroll 4
-    for (int t = t0; t < t1; ++t) {
-      load_n<V>(in + t * ld, x[TAPS - 1]);
-      float y[V];
 #pragma unroll
-      for (int j = 0; j < V; ++j) {
-        y[j] = b[j];
+    for (int k = 0; k < TAPS; ++k) {
+      float f[V];
+      packed[k].get(f);
 #pragma unroll
-        for (int k = 0; k < TAPS; ++k) y[j] = fmaf(w[k][j], x[k][j], y[j]);
+      for (int j = 0; j < V; ++j) w[(k * V + j) % TAPS][(k * V + j) / TAPS] = f[j];
+    }
+    for (int tb = t0; tb < t1; tb += U) {
+      Raw<T, V> next[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (tb + U + u < t1) next[u].load(in + (tb + U + u) * ld);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        if (tb + u < t1) {
+          float y[V];
+          cur[u].get(x[TAPS - 1]);
+#pragma unroll
+          for (int j = 0; j < V; ++j) {
+            y[j] = b[j];
+#pragma unroll
+            for (int k = 0; k < TAPS; ++k) y[j] = fmaf(w[k][j], x[k][j], y[j]);
+          }
+          finish(tb + u, y);
+#pragma unroll
+          for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+            for (int j = 0; j < V; ++j) x[k][j] = x[k + 1][j];
+        }
+        cur[u] = next[u];
       }
-      finish(t, y);
-#pragma unroll
-      for (int k = 0; k < TAPS - 1; ++k)
-#pragma unroll
-        for (int j = 0; j < V; ++j) x[k][j] = x[k + 1][j];
     }
   } else {
     for (int t = t0; t < t1; ++t) {
@@ -204,63 +259,93 @@ __global__ void __launch_bounds__(128) ssm_seq_kernel(const T* __restrict__ proj
 }
 
 static constexpr int kStep = 256;
-// grid (heads (+ 1 with an aside), rows), 256 threads; V % 4 == 0, V ≤ 1024.  A thread owns four columns of every (256 / (V / 4))-th state row.
-template <typename T>
+// grid (heads / HP (+ 1 with an aside), rows), 256 threads; V % 4 == 0, HP · V ≤ 1024.  A CTA takes HP neighbouring heads of a group: they share
+// the convolution of B and C, and enough of the state is on its way.  A thread owns four columns of a head in every (256 / (HP · V / 4))-th
+// state row.
+template <typename T, bool GROUPED, int HP>
 __global__ void __launch_bounds__(kStep) ssm_step_kernel(const T* __restrict__ proj, long long ld, MbSsm m, T* __restrict__ out, MbAside a,
                                                          int aside_vec_ok) {
   extern __shared__ __align__(16) float sm[];
   pdl_trigger();
   pdl_wait();
   const int N = m.N, V = m.V, H = m.H, inner = H * V, CH = inner + 2 * m.G * N, per = H / m.G;
-  const int b = blockIdx.y, h = blockIdx.x;
-  if (h == H) {
-    if (aside_vec_ok) aside_row<T, true, kStep>(a, b);
-    else aside_row<T, false, kStep>(a, b);
+  const int b = blockIdx.y, h0 = blockIdx.x * HP, W = HP * V;
+  if (h0 >= H) {
+    if (aside_vec_ok) aside_row<T, true, kStep, GROUPED>(a, b);
+    else aside_row<T, false, kStep, GROUPED>(a, b);
     return;
   }
   const int slot = m.slots[b];
-  T* o = out + static_cast<long long>(b) * inner + h * V;
+  T* o = out + static_cast<long long>(b) * inner + h0 * V;
   if (slot < 0) {                        // padding row
-    for (int i = threadIdx.x; i < V; i += kStep) o[i] = from_f<T>(0.f);
+    for (int i = threadIdx.x; i < W; i += kStep) o[i] = from_f<T>(0.f);
     return;
   }
-  const int cg = V / 4, rpp = kStep / cg;                // column groups, state rows per pass
-  float* red = sm;                       // [rpp][V]
-  float* sx = red + rpp * V;             // [V | N | N]: x, B, C of this token
-  const int row0 = threadIdx.x / cg, col = (threadIdx.x % cg) * 4;
+  const int cg = W / 4, rpp = kStep / cg;                // column groups, state rows per pass
+  float* red = sm;                       // [rpp][W]
+  float* sx = red + rpp * W;             // [W | N | N]: x, B, C of this token
+  const int row0 = threadIdx.x / cg, col = (threadIdx.x % cg) * 4, mine = HP == 2 && col >= V;      // column among the CTA's, its head
   const bool on = row0 < rpp;
-  float* st = m.state + (static_cast<long long>(slot) * H + h) * N * V;
+  float* st = m.state + (static_cast<long long>(slot) * H + h0 + mine) * N * V + (col - mine * V);
   const int pos = m.positions[b];
   // the state is on its way while the projections of this token are read, convolved and activated
-  constexpr int U = 8;
+  constexpr int U = 8 * HP;
   float4 s[U];
 #pragma unroll
   for (int u = 0; u < U; ++u) {
     const int d = row0 + u * rpp;
-    s[u] = (on && pos > 0 && d < N) ? *reinterpret_cast<const float4*>(st + static_cast<long long>(d) * V + col) : make_float4(0, 0, 0, 0);
+    s[u] = (on && pos > 0 && d < N) ? *reinterpret_cast<const float4*>(st + static_cast<long long>(d) * V) : make_float4(0, 0, 0, 0);
   }
   const T* p = proj + b * ld;
-  const int g = h / per;
+  const int g = h0 / per;
   float* ring = m.ring != nullptr ? m.ring + static_cast<long long>(slot) * m.taps * CH : nullptr;
-  for (int i = threadIdx.x; i < V + 2 * N; i += kStep) {
-    const int c = i < V ? h * V + i : i < V + N ? inner + g * N + i - V : inner + (m.G + g) * N + i - V - N;
-    const T* w = reinterpret_cast<const T*>(m.conv_w) + static_cast<long long>(c) * m.taps;
-    const float x = to_f(p[inner + c]);
-    float y = to_f(reinterpret_cast<const T*>(m.conv_b)[c]);
-#pragma unroll 4
-    for (int k = 0; k < m.taps - 1; ++k) {
-      const int q = pos - (m.taps - 1 - k);
-      if (q >= 0) y = fmaf(to_f(w[k]), ring[static_cast<long long>(q % m.taps) * CH + c], y);
+  const float z0 = threadIdx.x < W ? to_f(p[h0 * V + threadIdx.x]) : 0.f;
+  const T raw_dt = p[inner + CH + h0 + mine], raw_bias = reinterpret_cast<const T*>(m.dt_bias)[h0 + mine],
+          raw_a = reinterpret_cast<const T*>(m.A_log)[h0 + mine];
+  constexpr int R = 2;                                   // channels of a thread that are on their way together
+  auto channel = [&](int i) { return i < W ? h0 * V + i : i < W + N ? inner + g * N + i - W : inner + (m.G + g) * N + i - W - N; };
+  for (int i0 = threadIdx.x; i0 < W + 2 * N; i0 += R * kStep) {
+    float x[R], y[R];
+#pragma unroll
+    for (int u = 0; u < R; ++u) {
+      const int i = i0 + u * kStep;
+      x[u] = y[u] = 0.f;
+      if (i >= W + 2 * N) continue;
+      const int c = channel(i);
+      x[u] = to_f(p[inner + c]);
+      y[u] = fmaf(to_f(reinterpret_cast<const T*>(m.conv_w)[static_cast<long long>(c) * m.taps + m.taps - 1]), x[u],
+                  to_f(reinterpret_cast<const T*>(m.conv_b)[c]));
     }
-    y = fmaf(to_f(w[m.taps - 1]), x, y);
-    sx[i] = to_f(from_f<T>(silu_t<T>(y)));               // as the general path stores it
-    if (ring != nullptr && (i < V || h % per == 0)) ring[static_cast<long long>(pos % m.taps) * CH + c] = x;
+    for (int k0 = 1; k0 < m.taps; k0 += 3) {             // three inputs back at a time, all on their way together
+      float f[R][3], w[R][3];
+#pragma unroll
+      for (int u = 0; u < R; ++u) {
+        const int i = i0 + u * kStep, c = i < W + 2 * N ? channel(i) : 0;
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+          const int q = pos - k0 - k;
+          const bool ok = i < W + 2 * N && k0 + k < m.taps && q >= 0;
+          f[u][k] = ok ? ring[static_cast<long long>(q % m.taps) * CH + c] : 0.f;
+          w[u][k] = ok ? to_f(reinterpret_cast<const T*>(m.conv_w)[static_cast<long long>(c) * m.taps + m.taps - 1 - k0 - k]) : 0.f;
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < R; ++u)
+#pragma unroll
+        for (int k = 0; k < 3; ++k) y[u] = fmaf(w[u][k], f[u][k], y[u]);
+    }
+#pragma unroll
+    for (int u = 0; u < R; ++u) {
+      const int i = i0 + u * kStep;
+      if (i >= W + 2 * N) continue;
+      sx[i] = to_f(from_f<T>(silu_t<T>(y[u])));          // as the general path stores it
+      if (ring != nullptr && (i < W || h0 % per == 0)) ring[static_cast<long long>(pos % m.taps) * CH + channel(i)] = x[u];
+    }
   }
-  const float dt = softplus_t<T>(to_f(p[inner + CH + h]) + to_f(reinterpret_cast<const T*>(m.dt_bias)[h]));
-  const float lam = exp_t<T>(-exp_t<T>(to_f(reinterpret_cast<const T*>(m.A_log)[h])) * dt);
+  const float dt = softplus_t<T>(to_f(raw_dt) + to_f(raw_bias)), lam = exp_t<T>(-exp_t<T>(to_f(raw_a)) * dt);
   __syncthreads();
   if (on) {
-    const float* sB = sx + V;
+    const float* sB = sx + W;
     const float* sC = sB + N;
     float v[4], y[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -270,13 +355,12 @@ __global__ void __launch_bounds__(kStep) ssm_step_kernel(const T* __restrict__ p
 #pragma unroll
         for (int u = 0; u < U; ++u) {
           const int d = d0 + u * rpp;
-          s[u] = (pos > 0 && d < N) ? *reinterpret_cast<const float4*>(st + static_cast<long long>(d) * V + col) : make_float4(0, 0, 0, 0);
+          s[u] = (pos > 0 && d < N) ? *reinterpret_cast<const float4*>(st + static_cast<long long>(d) * V) : make_float4(0, 0, 0, 0);
         }
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const int d = d0 + u * rpp;
         if (d >= N) break;
-        float* at = st + static_cast<long long>(d) * V + col;
         const float k = sB[d], q = sC[d];
         s[u].x = fmaf(lam, s[u].x, k * v[0]);
         s[u].y = fmaf(lam, s[u].y, k * v[1]);
@@ -286,25 +370,25 @@ __global__ void __launch_bounds__(kStep) ssm_step_kernel(const T* __restrict__ p
         y[1] = fmaf(s[u].y, q, y[1]);
         y[2] = fmaf(s[u].z, q, y[2]);
         y[3] = fmaf(s[u].w, q, y[3]);
-        *reinterpret_cast<float4*>(at) = s[u];
+        *reinterpret_cast<float4*>(st + static_cast<long long>(d) * V) = s[u];
       }
     }
-    *reinterpret_cast<float4*>(red + row0 * V + col) = make_float4(y[0], y[1], y[2], y[3]);
+    *reinterpret_cast<float4*>(red + row0 * W + col) = make_float4(y[0], y[1], y[2], y[3]);
   }
   __syncthreads();
-  const float D = to_f(reinterpret_cast<const T*>(m.D)[h]);
-  for (int i = threadIdx.x; i < V; i += kStep) {
-    float r = D * sx[i];
-    for (int w = 0; w < rpp; ++w) r += red[w * V + i];
-    o[i] = from_f<T>(r * silu_t<T>(to_f(p[h * V + i])));
+  for (int i = threadIdx.x; i < W; i += kStep) {
+    float r = to_f(reinterpret_cast<const T*>(m.D)[h0 + i / V]) * sx[i];
+    for (int w = 0; w < rpp; ++w) r += red[w * W + i];
+    o[i] = from_f<T>(r * silu_t<T>(i < kStep ? z0 : to_f(p[h0 * V + i])));
   }
 }
 
-template <typename T, int V>
+template <typename T, int V, bool GROUPED>
 static int conv_taps(const T* proj, long long ld, MbSsm m, const int* tiles, const int* cu_q, int n_tiles, T* xbc, float* dt, float* la, int n_aside,
                      MbAside a, cudaStream_t s) {
   const int CH = m.H * m.V + 2 * m.G * m.N, blocks = (CH + kConv * V - 1) / (kConv * V);
-  auto kern = m.taps == 4 ? ssm_conv_kernel<T, V, 4> : m.taps == 3 ? ssm_conv_kernel<T, V, 3> : m.taps == 2 ? ssm_conv_kernel<T, V, 2> : ssm_conv_kernel<T, V, 0>;
+  auto kern = m.taps == 4 ? ssm_conv_kernel<T, V, 4, GROUPED> : m.taps == 3 ? ssm_conv_kernel<T, V, 3, GROUPED>
+            : m.taps == 2 ? ssm_conv_kernel<T, V, 2, GROUPED> : ssm_conv_kernel<T, V, 0, GROUPED>;
   return static_cast<int>(launch_pdl(kern, dim3(static_cast<unsigned>(n_tiles * (blocks + 1) + n_aside)), dim3(kConv), 0, s, proj, ld, m, tiles, cu_q,
                                      n_tiles, blocks, xbc, dt, la, a));
 }
@@ -330,8 +414,8 @@ extern "C" int mb_ssm_conv(const void* proj, long long ld, MbSsm m, const int* t
     const bool vec = ld % v == 0 && (m.H * m.V) % v == 0 && (m.G * m.N) % v == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0 && aside_vec<E>(a);
     auto P = reinterpret_cast<const E*>(proj);
     auto X = reinterpret_cast<E*>(xbc);
-    return vec ? conv_taps<E, v>(P, ld, m, tiles, cu_q, n_tiles, X, dt, la, n_aside, a, s)
-               : conv_taps<E, 1>(P, ld, m, tiles, cu_q, n_tiles, X, dt, la, n_aside, a, s);
+    auto f = a.grouped ? (vec ? conv_taps<E, v, true> : conv_taps<E, 1, true>) : (vec ? conv_taps<E, v, false> : conv_taps<E, 1, false>);
+    return f(P, ld, m, tiles, cu_q, n_tiles, X, dt, la, n_aside, a, s);
   };
   return f32 ? run(float{}) : run(bf16{});
 }
@@ -339,11 +423,15 @@ extern "C" int mb_ssm_conv(const void* proj, long long ld, MbSsm m, const int* t
 extern "C" int mb_ssm_step(const void* proj, long long ld, MbSsm m, void* out, int B, MbAside a, int f32, cudaStream_t s) {
   if (B <= 0) return 0;
   if (!sizes_ok(m) || m.V % 4 || m.V > 4 * kStep || B > 65535 || !aside_ok(a)) return -3;
-  const size_t bytes = (static_cast<size_t>(kStep / (m.V / 4)) * m.V + m.V + 2 * m.N) * sizeof(float);
+  // two heads per CTA where that leaves CTAs for every SM
+  const int hp = m.V <= 64 && (m.H / m.G) % 2 == 0 && static_cast<long long>(B) * m.H >= 4 * 148 ? 2 : 1, W = hp * m.V;
+  const size_t bytes = (static_cast<size_t>(kStep / (W / 4)) * W + W + 2 * m.N) * sizeof(float);
   if (bytes > 48 * 1024) return -3;
   auto run = [&](auto ty) {
     using E = decltype(ty);
-    return static_cast<int>(launch_pdl(ssm_step_kernel<E>, dim3(m.H + aside_on(a), B), dim3(kStep), bytes, s, reinterpret_cast<const E*>(proj), ld, m,
+    auto kern = hp == 2 ? (a.grouped ? ssm_step_kernel<E, true, 2> : ssm_step_kernel<E, false, 2>)
+                        : (a.grouped ? ssm_step_kernel<E, true, 1> : ssm_step_kernel<E, false, 1>);
+    return static_cast<int>(launch_pdl(kern, dim3(m.H / hp + aside_on(a), B), dim3(kStep), bytes, s, reinterpret_cast<const E*>(proj), ld, m,
                                        reinterpret_cast<E*>(out), a, aside_vec<E>(a) ? 1 : 0));
   };
   return f32 ? run(float{}) : run(bf16{});

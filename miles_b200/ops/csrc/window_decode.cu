@@ -1,10 +1,10 @@
 // Decode attention over a paged cache of keys and values with a sliding window that keeps the first tokens, and a softmax sink.
 //
-// One cluster = (token, key head, up to 8 query heads of its group); its CTAs split the keys the token sees, which are numbered
+// One cluster = (token, key head, up to R = 8 or 16 query heads of its group); its CTAs split the keys the token sees, which are numbered
 // without a gap: first the kept ones, then those of the window.  As in paged_decode.cu the heads of the group are rows of
 // mma.sync.m16n8k16 and tiles of 64 keys are gathered from their pages with cp.async, double buffered, 16 keys per warp.  What differs:
-//   * the eight rows that padded the softmax weights carry their second bf16 part, so that P·V sees 16 bits of mantissa for no
-//     extra instruction; the two halves of the accumulator are added at the end;
+//   * the softmax weights enter P·V as two bf16 parts, 16 bits of mantissa.  R = 8: the eight rows that pad the tile carry the second
+//     part for no extra instruction, and the two halves of the accumulator are added at the end.  R = 16: two products;
 //   * the splits are joined through distributed shared memory, the sink enters there: one launch, no partial results in HBM;
 //   * differential attention (MbDiff): heads 2h and 2h + 1 are neighbours among the rows; a warp joins both, subtracts, norms and gates.
 // Heads narrower than DK / DV are padded with zeros in shared memory.
@@ -29,35 +29,37 @@ static constexpr int TK = 64;
 template <int D>
 __device__ __forceinline__ int toff(int row, int chunk) { return row * D + ((chunk ^ (row & 7)) << 3); }
 
-template <int DK, int DV>
+template <int DK, int DV, int R>
 struct Smem {
-  // the warps' outputs take the place of the key tiles, the split's output that of the value tiles
-  static constexpr int q = 0, k = 16 * DK * 2, v = k + 2 * TK * DK * 2, ml = v + 2 * TK * DV * 2, fml = ml + 64 * 4, total = fml + 16 * 4, o = k, f = v;
-  static_assert(4 * 8 * DV * 4 <= 2 * TK * DK * 2, "the key tiles hold the warps' outputs");
+  // the warps' outputs take the place of the key tiles where they fit, the split's output that of the value tiles
+  static constexpr int q = 0, k = 16 * DK * 2, v = k + 2 * TK * DK * 2, ml = v + 2 * TK * DV * 2, fml = ml + 8 * R * 4, total = fml + 2 * R * 4;
+  static constexpr int o = 4 * R * DV * 4 <= 2 * TK * DK * 2 ? k : v + 2 * TK * DV * 2 + 10 * R * 4, f = v;
+  static constexpr int bytes = o == k ? total : o + 4 * R * DV * 4;
 };
 
-template <int DK, int DV>
+template <int DK, int DV, int R>
 __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
                                                             const int* __restrict__ block_table, int max_blocks, int block_size,
                                                             const int* __restrict__ token_seq, const int* __restrict__ positions,
                                                             const long long* __restrict__ slots, const bf16* __restrict__ sink,
                                                             bf16* __restrict__ out, long long o_row, float scale, MbWindow L, MbDiff D) {
-  using S = Smem<DK, DV>;
+  using S = Smem<DK, DV, R>;
   extern __shared__ __align__(128) uint8_t smem[];
   bf16* sQ = reinterpret_cast<bf16*>(smem + S::q);
   bf16* sK = reinterpret_cast<bf16*>(smem + S::k);
   bf16* sV = reinterpret_cast<bf16*>(smem + S::v);
-  float* sM = reinterpret_cast<float*>(smem + S::ml);      // [4][8] maxima, then [4][8] sums
-  float* sL = sM + 32;
-  float* sO = reinterpret_cast<float*>(smem + S::o);       // [4][8][DV]
-  float* fO = reinterpret_cast<float*>(smem + S::f);       // [8][DV]: this split's output …
-  float* fM = reinterpret_cast<float*>(smem + S::fml);     // [8] maxima (times scale·log2 e), [8] sums
+  float* sM = reinterpret_cast<float*>(smem + S::ml);      // [4][R] maxima, then [4][R] sums
+  float* sL = sM + 4 * R;
+  float* sO = reinterpret_cast<float*>(smem + S::o);       // [4][R][DV]
+  float* fO = reinterpret_cast<float*>(smem + S::f);       // [R][DV]: this split's output …
+  float* fM = reinterpret_cast<float*>(smem + S::fml);     // [R] maxima (times scale·log2 e), [R] sums
+  constexpr int RS = R / 8;                                // rows of a thread: lane / 4 (+ 8)
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.z, split = blockIdx.x, splits = gridDim.x;
-  const int group = L.heads / L.kv_heads, chunks = (group + 7) / 8;
-  const int hk = blockIdx.y / chunks, h0 = hk * group + (blockIdx.y % chunks) * 8;
-  const int rows = min(8, group - (blockIdx.y % chunks) * 8);
+  const int group = L.heads / L.kv_heads, chunks = (group + R - 1) / R;
+  const int hk = blockIdx.y / chunks, h0 = hk * group + (blockIdx.y % chunks) * R;
+  const int rows = min(R, group - (blockIdx.y % chunks) * R);
   const bool diff = D.lam != nullptr;
   if (slots[t] < 0) {                    // padding row of a decode batch (the whole cluster leaves)
     const int heads = diff ? rows / 2 : rows, first = diff ? h0 / 2 : h0;
@@ -127,7 +129,9 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
   float o_acc[DV / 8][4];
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
-  float m_i = -INFINITY, l_i = 0.f;      // of row lane / 4
+  float m_i[RS], l_i[RS];                // of rows lane / 4 (and 8 more)
+#pragma unroll
+  for (int r = 0; r < RS; ++r) { m_i[r] = -INFINITY; l_i[r] = 0.f; }
   const float sl2 = scale * kLog2e;
 
   for (int tile = 0; tile < n_tiles; ++tile) {
@@ -151,62 +155,78 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
         mma16816(s[0], qa[ks], b[0], b[1]);
         mma16816(s[1], qa[ks], b[2], b[3]);
       }
-      float mx = -INFINITY;
+      float alpha[RS];
+      uint32_t pa[RS][4];                               // R = 8: rows 0–7 the weights' first part, rows 8–15 what rounding took off it
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
+      for (int r = 0; r < RS; ++r) {
+        float mx = -INFINITY;
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          s[nt][e] = key0 + nt * 8 + (lane & 3) * 2 + e < k_end ? s[nt][e] * sl2 : -INFINITY;
-          mx = fmaxf(mx, s[nt][e]);
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            s[nt][2 * r + e] = key0 + nt * 8 + (lane & 3) * 2 + e < k_end ? s[nt][2 * r + e] * sl2 : -INFINITY;
+            mx = fmaxf(mx, s[nt][2 * r + e]);
+          }
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(m_i[r], fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2)));
+        alpha[r] = exp2f(m_i[r] - mx);                  // the first key of the tile is seen: mx is finite
+        m_i[r] = mx;
+        float rs = 0.f;
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          const float a = exp2f(s[nt][2 * r] - mx), b = exp2f(s[nt][2 * r + 1] - mx);
+          rs += a + b;
+          const uint32_t hi = pack2(a, b), lo = pack2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
+          if (R == 8) {
+            pa[0][2 * nt] = hi;
+            pa[0][2 * nt + 1] = lo;
+          } else {                                      // pa[0]: first parts of rows lane / 4 and lane / 4 + 8, pa[1]: second parts
+            pa[0][2 * nt + r] = hi;
+            pa[RS - 1][2 * nt + r] = lo;
+          }
         }
-      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-      mx = fmaxf(m_i, fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2)));
-      const float alpha = exp2f(m_i - mx);            // the first key of the tile is seen: mx is finite
-      m_i = mx;
-      uint32_t pa[4];
-      float rs = 0.f;
-#pragma unroll
-      for (int nt = 0; nt < 2; ++nt) {
-        const float a = exp2f(s[nt][0] - mx), b = exp2f(s[nt][1] - mx);
-        rs += a + b;
-        const uint32_t hi = pack2(a, b);
-        pa[2 * nt] = hi;                                // rows 0–7: the weights' first part, rows 8–15: what rounding took off it
-        pa[2 * nt + 1] = pack2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
+        l_i[r] = l_i[r] * alpha[r] + rs;
       }
-      l_i = l_i * alpha + rs;
 #pragma unroll
-      for (int i = 0; i < DV / 8; ++i) { o_acc[i][0] *= alpha; o_acc[i][1] *= alpha; o_acc[i][2] *= alpha; o_acc[i][3] *= alpha; }
+      for (int i = 0; i < DV / 8; ++i) { o_acc[i][0] *= alpha[0]; o_acc[i][1] *= alpha[0]; o_acc[i][2] *= alpha[RS - 1]; o_acc[i][3] *= alpha[RS - 1]; }
 #pragma unroll
       for (int nc = 0; nc < DV / 16; ++nc) {
         uint32_t b[4];
         ldsm_x4_t(s_addr(tV + toff<DV>(warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), nc * 2 + (lane >> 4))), b[0], b[1], b[2], b[3]);
-        mma16816(o_acc[2 * nc], pa, b[0], b[1]);
-        mma16816(o_acc[2 * nc + 1], pa, b[2], b[3]);
+#pragma unroll
+        for (int part = 0; part < RS; ++part) {
+          mma16816(o_acc[2 * nc], pa[part], b[0], b[1]);
+          mma16816(o_acc[2 * nc + 1], pa[part], b[2], b[3]);
+        }
       }
     }
     __syncthreads();
   }
-  l_i += __shfl_xor_sync(0xffffffffu, l_i, 1);
-  l_i += __shfl_xor_sync(0xffffffffu, l_i, 2);
-  const int r = lane >> 2;
-  if ((lane & 3) == 0) { sM[warp * 8 + r] = m_i; sL[warp * 8 + r] = l_i; }
 #pragma unroll
-  for (int i = 0; i < DV / 8; ++i)
-    *reinterpret_cast<float2*>(sO + (warp * 8 + r) * DV + i * 8 + (lane & 3) * 2) = make_float2(o_acc[i][0] + o_acc[i][2], o_acc[i][1] + o_acc[i][3]);
+  for (int k = 0; k < RS; ++k) {
+    l_i[k] += __shfl_xor_sync(0xffffffffu, l_i[k], 1);
+    l_i[k] += __shfl_xor_sync(0xffffffffu, l_i[k], 2);
+    const int r = (lane >> 2) + 8 * k;
+    if ((lane & 3) == 0) { sM[warp * R + r] = m_i[k]; sL[warp * R + r] = l_i[k]; }
+#pragma unroll
+    for (int i = 0; i < DV / 8; ++i)
+      *reinterpret_cast<float2*>(sO + (warp * R + r) * DV + i * 8 + (lane & 3) * 2) =
+          R == 8 ? make_float2(o_acc[i][0] + o_acc[i][2], o_acc[i][1] + o_acc[i][3]) : make_float2(o_acc[i][2 * k], o_acc[i][2 * k + 1]);
+  }
   __syncthreads();
   for (int i = threadIdx.x; i < rows * DV; i += 128) {
     const int g = i / DV, d = i % DV;
     float mm = -INFINITY, ll = 0.f, oo = 0.f;
 #pragma unroll
-    for (int w = 0; w < 4; ++w) mm = fmaxf(mm, sM[w * 8 + g]);
+    for (int w = 0; w < 4; ++w) mm = fmaxf(mm, sM[w * R + g]);
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
-      const float a = sM[w * 8 + g] == -INFINITY ? 0.f : exp2f(sM[w * 8 + g] - mm);
-      ll += sL[w * 8 + g] * a;
-      oo += sO[(w * 8 + g) * DV + d] * a;
+      const float a = sM[w * R + g] == -INFINITY ? 0.f : exp2f(sM[w * R + g] - mm);
+      ll += sL[w * R + g] * a;
+      oo += sO[(w * R + g) * DV + d] * a;
     }
     fO[g * DV + d] = oo;
-    if (d == 0) { fM[g] = mm; fM[8 + g] = ll; }
+    if (d == 0) { fM[g] = mm; fM[R + g] = ll; }
   }
   // join the splits: every CTA of the cluster finishes its share of the outputs
   cg::cluster_group cluster = cg::this_cluster();
@@ -234,7 +254,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
           w[c] = 0.f;
           if (ms[c] == -INFINITY) continue;
           w[c] = exp2f(ms[c] - mm);
-          den = fmaf(cluster.map_shared_rank(fM, c)[8 + g], w[c], den);
+          den = fmaf(cluster.map_shared_rank(fM, c)[R + g], w[c], den);
         }
         const float f = __fdiv_rn(map ? -lam : 1.f, den);
 #pragma unroll
@@ -271,7 +291,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
     for (int c = 0; c < 8; ++c) {
       if (ms[c] == -INFINITY) continue;
       const float a = exp2f(ms[c] - mm);
-      den = fmaf(cluster.map_shared_rank(fM, c)[8 + g], a, den);
+      den = fmaf(cluster.map_shared_rank(fM, c)[R + g], a, den);
       oo = fmaf(cluster.map_shared_rank(fO, c)[g * DV + d], a, oo);
     }
     if (d < L.vdim) out[t * o_row + static_cast<long long>(h0 + g) * L.vdim + d] = __float2bfloat16(__fdiv_rn(oo, den));
@@ -279,19 +299,28 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
   if (splits > 1) cluster.sync();        // the shared memory stays until the others have read it
 }
 
-template <int DK, int DV>
-static int launch(const bf16* q, const bf16* kc, const bf16* vc, const int* bt, int max_blocks, int bs, const int* seq, const int* pos,
+template <int DK, int DV, int R>
+static int launch_rows(const bf16* q, const bf16* kc, const bf16* vc, const int* bt, int max_blocks, int bs, const int* seq, const int* pos,
                   const long long* slots, const bf16* sink, bf16* out, long long o_row, int T, float scale, int splits, MbWindow L, MbDiff d,
                   cudaStream_t s) {
   static bool once = false;
   if (!once) {
-    const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<DK, DV>::total);
+    const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<DK, DV, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<DK, DV, R>::bytes);
     if (e != cudaSuccess) return static_cast<int>(e);
     once = true;
   }
-  const int chunks = (L.heads / L.kv_heads + 7) / 8;
-  return static_cast<int>(launch_pdl_cluster(window_decode_kernel<DK, DV>, dim3(splits, L.kv_heads * chunks, T), dim3(128), splits,
-                                             Smem<DK, DV>::total, s, q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, scale, L, d));
+  const int chunks = (L.heads / L.kv_heads + R - 1) / R;
+  return static_cast<int>(launch_pdl_cluster(window_decode_kernel<DK, DV, R>, dim3(splits, L.kv_heads * chunks, T), dim3(128), splits,
+                                             Smem<DK, DV, R>::bytes, s, q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, scale, L, d));
+}
+
+// groups of more than 8 heads are read once for 16 of them
+template <int DK, int DV>
+static int launch(const bf16* q, const bf16* kc, const bf16* vc, const int* bt, int max_blocks, int bs, const int* seq, const int* pos,
+                  const long long* slots, const bf16* sink, bf16* out, long long o_row, int T, float scale, int splits, MbWindow L, MbDiff d,
+                  cudaStream_t s) {
+  auto f = L.heads / L.kv_heads > 8 ? launch_rows<DK, DV, 16> : launch_rows<DK, DV, 8>;
+  return f(q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, T, scale, splits, L, d, s);
 }
 
 }  // namespace wd

@@ -67,7 +67,7 @@ __device__ __forceinline__ void norm_rotate(const T* __restrict__ x, const T* __
   for (int i = threadIdx.x; i < heads * gap; i += kPrep) y[(i / gap) * pitch + dim + i % gap] = from_f<T>(0.f);
 }
 
-template <typename T, bool VEC>
+template <typename T, bool VEC, bool GROUPED>
 __global__ void __launch_bounds__(kPrep) window_prep_kernel(const T* __restrict__ proj, long long ld, const int* __restrict__ positions,
                                                             const long long* __restrict__ slots, const double* __restrict__ freq,
                                                             float magnitude, const T* __restrict__ q_norm, const T* __restrict__ k_norm,
@@ -81,7 +81,7 @@ __global__ void __launch_bounds__(kPrep) window_prep_kernel(const T* __restrict_
   const T* p = proj + t * ld;
   const int nq = L.heads * L.dim, nk = L.kv_heads * L.dim, nv = L.kv_heads * L.vdim;
   if (blockIdx.y == 2) {
-    aside_row<T, VEC, kPrep>(a, t);
+    aside_row<T, VEC, kPrep, GROUPED>(a, t);
     return;
   }
   const bool keys = blockIdx.y == 1;
@@ -113,7 +113,8 @@ static int prep(const T* proj, long long ld, const int* positions, const long lo
                 const T* q_norm, const T* k_norm, float eps, T* kc, T* vc, T* q, int n, MbWindow L, MbAside a, cudaStream_t s) {
   const int v = 16 / static_cast<int>(sizeof(T));
   const bool vec = ld % v == 0 && L.dim % v == 0 && L.vdim % v == 0 && L.rot % v == 0 && L.q_pitch % v == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0 && aside_vec<T>(a);
-  auto kern = vec ? window_prep_kernel<T, true> : window_prep_kernel<T, false>;
+  auto kern = a.grouped ? (vec ? window_prep_kernel<T, true, true> : window_prep_kernel<T, false, true>)
+                        : (vec ? window_prep_kernel<T, true, false> : window_prep_kernel<T, false, false>);
   return static_cast<int>(launch_pdl(kern, dim3(n, aside_on(a) ? 3 : 2), dim3(kPrep), L.rot * sizeof(float), s, proj,
                                      ld, positions, slots, freq, magnitude, q_norm, k_norm, eps, kc, vc, q, L, a));
 }

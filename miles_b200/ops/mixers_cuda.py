@@ -280,7 +280,8 @@ def _window_ok(lay, dt) -> bool:
 
 def window_splits(tokens: int, lay) -> int:
     """CTAs of a cluster that share the keys of one (token, key head): enough for the SMs, at most one per tile of 64 keys."""
-    ctas = tokens * lay.kv_heads * -(-(lay.heads // lay.kv_heads) // 8)
+    group = lay.heads // lay.kv_heads
+    ctas = tokens * lay.kv_heads * -(-group // (16 if group > 8 else 8))
     tiles = -(-(lay.window + lay.keep) // 64) if lay.window else 64
     return max(1, min(8, tiles, 444 // ctas))
 
@@ -349,20 +350,20 @@ def differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lv
 
 # ---- state-space mixer ------------------------------------------------------------------------------------------------
 
-CONV_TILE = 32           # tokens of a convolution tile (ssm_state.cu)
-
-
-def _conv_tiles(meta):
-    """[n, 4] (first token, end, sequence, first tile of its piece) over all pieces of a packed batch."""
+def _conv_tiles(meta, taps: int):
+    """[n, 4] (first token, end, sequence, first tile of its piece) over all pieces of a packed batch.  A tile has at least as many tokens as the
+    convolution looks back (ssm_state.cu)."""
     rg = meta.ragged
-    if "conv_tiles" not in rg.scratch:
+    T = sum(rg.q_lens)
+    size = max(32 if T > 4096 else 16, taps - 1)
+    if ("conv tiles", size) not in rg.scratch:
         tiles, t = [], 0
         for b, n in enumerate(rg.q_lens):
-            for a in range(0, n, CONV_TILE):
-                tiles += [t + a, t + min(n, a + CONV_TILE), b, int(a == 0)]
+            for a in range(0, n, size):
+                tiles += [t + a, t + min(n, a + size), b, int(a == 0)]
             t += n
-        rg.scratch["conv_tiles"] = torch.tensor(tiles, dtype=torch.int32).to(meta.positions.device).view(-1, 4)
-    return rg.scratch["conv_tiles"]
+        rg.scratch["conv tiles", size] = torch.tensor(tiles, dtype=torch.int32).to(meta.positions.device).view(-1, 4)
+    return rg.scratch["conv tiles", size]
 
 
 def state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta, aside):
@@ -380,7 +381,7 @@ def state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta, a
         return out
     xbc = torch.empty(T, lay.channels, dtype=dt, device=dev)
     step, decay = (torch.empty(T, lay.heads, dtype=torch.float32, device=dev) for _ in range(2))
-    C.ssm_conv(proj, sizes, tensors(slots, meta.positions), _conv_tiles(meta) if cu_q is not None else None, cu_q, xbc, step, decay, *a)
+    C.ssm_conv(proj, sizes, tensors(slots, meta.positions), _conv_tiles(meta, lay.taps) if cu_q is not None else None, cu_q, xbc, step, decay, *a)
     if rg.n_long and dt == BF16 and lay.state % 8 == 0 and lay.vdim % 8 == 0 and lay.state <= 128 and lay.vdim <= 128 and proj.stride(0) % 2 == 0:
         # long pieces in chunks on the tensor cores, the short ones behind them token by token
         segs, seq_segs, multi = _segments(meta, lay.heads // C.ssm_heads_per_cta(lay.heads, lay.vdim, lay.groups))
