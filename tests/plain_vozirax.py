@@ -212,8 +212,9 @@ def make_config(layers, width=64, vocab=131, eps=1e-5, logit_scale=0.7):
     return {"architecture": "Vozirax", "layers": layers, "logit_scale": logit_scale, "norm": {"eps": eps}, "vocab": vocab, "width": width}
 
 
-def make_weights(cfg, seed=0, gain=1.0):
-    """Random weights of every tensor of the checkpoint (bf16-exact values, so every run sees the same numbers)."""
+def make_weights(cfg, seed=0, gain=1.0, apart=False):
+    """Random weights of every tensor of the checkpoint (bf16-exact values, so every run sees the same numbers).  `apart`: corrections that
+    decide the choice of experts whatever the scores (no close calls for 16-bit runs; the weights of the choice still differ by token)."""
     g = torch.Generator().manual_seed(seed)
     D, out = cfg["width"], {}
 
@@ -263,6 +264,8 @@ def make_weights(cfg, seed=0, gain=1.0):
                 lin(f"{p}mlp.e{e}.down", D, f["expert"]["ff"])
             lin(p + "mlp.router", f["router"]["experts"], D, 2.0)
             vec(p + "mlp.correction", f["router"]["experts"], -0.3, 0.4)   # some choice scores are negative
+            if apart:
+                out[p + "mlp.correction"] = (4.0 * torch.randperm(f["router"]["experts"], generator=g) - 9.0).bfloat16()
     vec("final.norm", D)
     lin("head", cfg["vocab"], D, 2.0)
     return out
