@@ -84,7 +84,7 @@ __global__ void __launch_bounds__(kThreads, OUT ? 1 : 2) ssm_chunk_kernel(Args a
   if (!OUT && last) return;                          // nobody continues from a last segment's own sum
   const int slot = a.m.slots[seq];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
-  const int W = HP * V, kn = (N + 15) / 16, kv = (V + 15) / 16;          // columns of x in a tile; 16-wide steps of N and of a head's V
+  const int W = HP * V, kn = (N + 15) / 16;          // columns of x in a tile; 16-wide steps of N
   const bf16* src[3] = {a.xbc + inner + (G + grp) * N, a.xbc + inner + grp * N, a.xbc + h0 * V};
   // columns [width, 16·⌈width/16⌉) of the tiles are zero for good
   for (int i = threadIdx.x; i < 6 * C; i += kThreads) {

@@ -2,6 +2,7 @@
 from __future__ import annotations
 
 import json
+import os
 
 import pytest
 import torch
@@ -112,6 +113,9 @@ def test_serving_build_of_a_configuration():
 
     assert build.serve_kind(get_config("vozirax-tiny")) == "hybrid"
     assert "window_prep.cu" not in build.SERVE_KINDS["hybrid"] and "ssm_chunk.cu" not in build.SERVE_KINDS["attention"]
+    for kind, files in build.SERVE_KINDS.items():       # a build with experts registers their bindings
+        with open(os.path.join(build.CSRC, "bindings_more.cpp")) as f:
+            assert ("bindings_moe.cpp" in files) == (f"MB_SERVE_{kind.upper()}" in f.read()), kind
 
 
 # ---- mechanisms ---------------------------------------------------------------------------------------------------------------
