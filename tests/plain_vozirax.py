@@ -214,7 +214,7 @@ def make_config(layers, width=64, vocab=131, eps=1e-5, logit_scale=0.7):
 
 def make_weights(cfg, seed=0, gain=1.0, apart=False):
     """Random weights of every tensor of the checkpoint (bf16-exact values, so every run sees the same numbers).  `apart`: corrections that
-    decide the choice of experts whatever the scores (no close calls for 16-bit runs; the weights of the choice still differ by token)."""
+    decide the choice of groups and experts whatever the scores (no close calls for 16-bit runs; the weights of the choice still differ by token)."""
     g = torch.Generator().manual_seed(seed)
     D, out = cfg["width"], {}
 
@@ -265,7 +265,7 @@ def make_weights(cfg, seed=0, gain=1.0, apart=False):
             lin(p + "mlp.router", f["router"]["experts"], D, 2.0)
             vec(p + "mlp.correction", f["router"]["experts"], -0.3, 0.4)   # some choice scores are negative
             if apart:
-                out[p + "mlp.correction"] = (4.0 * torch.randperm(f["router"]["experts"], generator=g) - 9.0).bfloat16()
+                out[p + "mlp.correction"] = (4.0 * 1.9 ** torch.randperm(f["router"]["experts"], generator=g) - 9.0).bfloat16()
     vec("final.norm", D)
     lin("head", cfg["vocab"], D, 2.0)
     return out
