@@ -60,6 +60,16 @@ def read_safetensors_header(path: str) -> tuple[dict, int]:
     return header, 8 + n
 
 
+def tensor_shapes(directory: str) -> dict[str, tuple]:
+    """Name → shape of every tensor in a directory's safetensors files (headers only)."""
+    out: dict[str, tuple] = {}
+    for f in sorted(os.listdir(directory)):
+        if f.endswith(".safetensors"):
+            header, _ = read_safetensors_header(os.path.join(directory, f))
+            out.update({n: tuple(info["shape"]) for n, info in header.items() if n != "__metadata__"})
+    return out
+
+
 def load_safetensors(path: str, names: Iterable[str] | None = None) -> dict[str, torch.Tensor]:
     header, base = read_safetensors_header(path)
     want = set(names) if names is not None else None

@@ -113,11 +113,17 @@ class ModelConfig:
 
     @staticmethod
     def from_hf_config(cfg: dict | str) -> "ModelConfig":
+        folder = None
         if isinstance(cfg, str):
             path = os.path.join(cfg, "config.json") if os.path.isdir(cfg) else cfg
+            folder = os.path.dirname(path)
             with open(path) as f:
                 cfg = json.load(f)
         if (design := _architecture(cfg)) is not None:
+            if folder is not None and getattr(design, "SIZES_FROM_TENSORS", False):
+                from ..checkpoint.hf_io import tensor_shapes
+
+                return design.from_config(cfg, tensor_shapes(folder))
             return design.from_config(cfg)
         mt = cfg.get("model_type", "qwen3")
         heads = cfg["num_attention_heads"]

@@ -2,7 +2,8 @@
 
 A design module gives `ARCHITECTURE`, `from_config` / `to_config` (config.json ⇄ `LayeredConfig`), `PRESETS`, and
 `tensors(cfg)`: checkpoint tensor name → `Place`, where its values live in this package's (stacked) parameters.  Loading,
-assembling and exporting checkpoints follow from that table.
+assembling and exporting checkpoints follow from that table.  A design whose config.json leaves sizes to the tensors' shapes says so
+with `SIZES_FROM_TENSORS`: its `from_config` then also takes the checkpoint's shapes by name.
 """
 from __future__ import annotations
 
@@ -46,6 +47,8 @@ def param_shapes(cfg: LayeredConfig) -> dict[str, tuple]:
         out["lm_head"] = (V, H)
     if cfg.bigram is not None:
         out["bigram"] = (cfg.bigram.buckets + 1, H)
+    if cfg.token_side:
+        out["side_embed"] = (V, cfg.num_layers * cfg.token_side)
     for i, s in enumerate(cfg.layer_specs):
         out.update({f"layers.{i}.{n}": shape for n, shape in layer_shapes(s, cfg).items()})
     return out
@@ -106,6 +109,6 @@ def rows_of(param: str, parts) -> dict[str, Place]:
     return out
 
 
-from . import nopelorn, ronupel, vozirax  # noqa: E402  (they use Place and rows_of)
+from . import nopelorn, ronupel, senadra, vozirax  # noqa: E402  (they use Place and rows_of)
 
-DESIGNS = {"nopelorn": nopelorn, "ronupel": ronupel, "vozirax": vozirax}
+DESIGNS = {"nopelorn": nopelorn, "ronupel": ronupel, "vozirax": vozirax, "senadra": senadra}

@@ -5,20 +5,27 @@ latent ranks or state sizes are a `LayeredConfig`: a tuple of `LayerSpec`s over 
 
     LatentMixer        latent attention over a paged cache of latents: sliding window, per-head softmax sink, interleaved
                        rotary with optional YaRN frequencies, layers that read another layer's latents (`kv_from`)
+                       queries through a latent of their own, output gate
     LinearStateMixer   linear attention with a constant decay per head: fp32 state per sequence, gated norm over all heads
-    AttentionMixer     grouped-query attention over a paged cache of keys and values: sliding window that keeps the first tokens,
-                       per-head softmax sink, RMS norm over a token's whole query (key) projection, interleaved rotary
+    DeltaMixer         gated delta rule with a decay per key channel: short convolutions, unit queries and keys, fp32 state, gated norm
+                       per head
+    AttentionMixer     grouped-query attention over a paged cache of keys and values: sliding window that keeps the first tokens, or
+                       chunks; per-head softmax sink or distance bias, RMS norm over a token's whole query (key) projection or
+                       over its values, interleaved rotary, output gate; may read another layer's keys and values
     DifferentialMixer  two softmax maps per head over the same values, the second subtracted with a learned weight; norms per head and
                        map, a query temperature that grows with the position, a gate per head; may read another layer's keys and values
     SsmMixer           state-space layer with a scalar decay per head and token: short convolution, fp32 state, gate, norm in parts
     ClampedGLU         gate and up projections with clamped pre-activations (a limit of infinity: plain silu(gate) · up)
+    Xielu              ungated feed-forward with a learned quadratic / exponential activation
+    TokenSide          per-layer token input: a second look-up per token and layer, gated by the residual, normed and added
     RoutedExperts      clamped gated experts or ungated ones with a squared relu; chosen by the `top` largest of biased fp32 logits
                        with weights by their softmax, or by corrected sigmoid scores among the best groups (`Routing`)
-    LayeredModel       hashed-bigram embedding and / or sinusoidal positions, fp32 residual stream, layers in one of three arrangements
+    LayeredModel       hashed-bigram embedding and / or sinusoidal positions, fp32 residual stream, layers in one of four arrangements
                        (`LayeredConfig.block`):
                        "output_norm"  mixer, then feed-forward, norms on the sublayers' OUTPUTS with a layer scale
                        "parallel"     one norm in front; mixer and feed-forward read it side by side and are added together
                        "two_norms"    mixer and feed-forward side by side, each behind a norm and before a layer scale of its own
+                       "pre_norm"     mixer, then feed-forward, then token input, each behind a norm in front and times one factor
                        A range of layers may run several times with the same weights (`LoopSpec`), each pass on its own cache.
 
 The blocks run in the engine only (paged latents, state slots; no autograd).  What the design keeps in 32 bits — rotary
@@ -99,6 +106,21 @@ class LatentSpec:
     window: int = 0                # keys a query sees, itself included; 0: all earlier ones
     sink: bool = True              # a learned extra term in every head's softmax denominator
     kv_from: int | None = None     # layer whose cached latents this layer reads instead of writing its own
+    q_rank: int = 0                # queries come from a normed latent of this size (0: straight from the input)
+    gate: bool = False             # outputs times the sigmoid of a projection of the input
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """Gated delta rule: per head S ← diag(g)·S, S ← S + β k (v − Sᵀk)ᵀ, o = Sᵀq, with a decay g per key channel."""
+
+    heads: int
+    kv_heads: int                  # query / key heads; heads share them in equal groups
+    dim: int
+    vdim: int
+    conv: int                      # columns of the causal convolutions
+    decay_rank: int                # inner size of the decays' two projections
+    gate_rank: int                 # … of the output gate's
 
 
 @dataclass(frozen=True)
@@ -121,6 +143,11 @@ class AttentionSpec:
     keep_first: int = 0            # tokens at the start of a sequence that stay visible whatever the window
     qk_norm: bool = True           # RMS norm over a token's whole query (key) projection, before the heads are rotated
     sink: bool = True              # a learned extra term in every head's softmax denominator
+    chunk: int = 0                 # tokens see their own chunk of this many positions only (0: no chunks)
+    distance_bias: bool = False    # r1 · ln(1 + r2 · distance) per head off the scores
+    value_norm: bool = False       # every head's values over their root mean square
+    gate: bool = False             # outputs times the sigmoid of a projection of the input
+    kv_from: int | None = None     # layer whose cached keys and values this layer reads instead of writing its own
 
 
 @dataclass(frozen=True)
@@ -174,6 +201,13 @@ class ReluSquareSpec:
 
 
 @dataclass(frozen=True)
+class XieluSpec:
+    """No gate: down(xielu(up)), an activation with two learned numbers."""
+
+    ff: int
+
+
+@dataclass(frozen=True)
 class MoeSpec:
     experts: int
     top: int
@@ -189,11 +223,11 @@ class MoeSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentSpec | LinearStateSpec | AttentionSpec | DifferentialSpec | SsmSpec
-    mlp: GluSpec | MoeSpec | None
+    mixer: LatentSpec | LinearStateSpec | AttentionSpec | DifferentialSpec | SsmSpec | DeltaSpec
+    mlp: GluSpec | XieluSpec | MoeSpec | None
 
     @property
-    def dense(self) -> GluSpec | None:
+    def dense(self) -> GluSpec | XieluSpec | None:
         """The feed-forward every token passes (all of it, or the shared expert beside routed ones)."""
         return self.mlp.shared if isinstance(self.mlp, MoeSpec) else self.mlp
 
@@ -218,11 +252,14 @@ class BigramSpec:
 class LayeredConfig(FamilyConfig):
     layer_specs: tuple = ()
     bigram: BigramSpec | None = None
-    block: str = "output_norm"         # or "parallel", "two_norms"
+    block: str = "output_norm"         # or "parallel", "two_norms", "pre_norm"
     loop: LoopSpec | None = None
     norm_shift: float = 0.0            # what norm weights are added to ("two_norms")
     position_base: float = 0.0         # sinusoidal position vectors are added to the embedding (0: none)
     logit_scale: float = 1.0
+    logit_softcap: float = 0.0         # logits ← cap · tanh(logits / cap) (0: as they are)
+    residual_mult: float = 1.0         # factor on what sublayers add ("pre_norm")
+    token_side: int = 0                # size of the per-layer token input (0: none; "pre_norm")
 
     def with_(self, **kw) -> "LayeredConfig":
         if "num_layers" in kw:                     # fewer layers: the first ones
@@ -254,6 +291,8 @@ class LayeredConfig(FamilyConfig):
         n = H + self.vocab_size * H * (1 if self.tie_embeddings else 2)
         if self.bigram is not None and not active_only:
             n += (self.bigram.buckets + 1) * H
+        if not active_only:
+            n += self.vocab_size * self.num_layers * self.token_side
         for i in [l for l, _ in self.runs()] if active_only else range(self.num_layers):
             s = self.layer_specs[i]
             n += sum(math.prod(shape) for shape in layer_shapes(s, self).values())
@@ -268,7 +307,9 @@ class LayeredConfig(FamilyConfig):
             if isinstance(m, LatentSpec):
                 f += 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim) * min(m.window or seq_len, seq_len / 2.0)
             elif isinstance(m, AttentionSpec):
-                f += 2.0 * m.heads * (m.dim + m.vdim) * min(m.window + m.keep_first if m.window else seq_len, seq_len / 2.0)
+                f += 2.0 * m.heads * (m.dim + m.vdim) * min(m.window + m.keep_first if m.window else (m.chunk or seq_len) / 2.0, seq_len / 2.0)
+            elif isinstance(m, DeltaSpec):
+                f += 6.0 * m.heads * m.dim * m.vdim
             elif isinstance(m, DifferentialSpec):
                 f += 4.0 * m.heads * (m.dim + m.vdim) * seq_len / 2.0
             elif isinstance(m, SsmSpec):
@@ -286,16 +327,27 @@ class LayeredConfig(FamilyConfig):
 def mixer_shapes(m, hidden: int) -> dict[str, tuple]:
     """Parameter shapes of a mixer (projections of one input stacked so that each input is multiplied once)."""
     if isinstance(m, LatentSpec):
-        rows = m.heads * (m.dim + m.rot_dim) + (0 if m.kv_from is not None else m.kv_rank + m.rot_dim)
+        rows = ((m.q_rank or m.heads * (m.dim + m.rot_dim)) + (0 if m.kv_from is not None else m.kv_rank + m.rot_dim)
+                + (m.heads * m.vdim if m.gate else 0))
         out = {"w_in": (rows, hidden), "w_ukv": (m.heads * (m.dim + m.vdim), m.kv_rank), "wo": (hidden, m.heads * m.vdim)}
         if m.kv_from is None:
             out["kv_norm"] = (m.kv_rank,)
         if m.sink:
             out["sink"] = (m.heads,)
+        if m.q_rank:
+            out.update({"w_uq": (m.heads * (m.dim + m.rot_dim), m.q_rank), "q_norm": (m.q_rank,)})
         return out
+    if isinstance(m, DeltaSpec):
+        k, v = m.kv_heads * m.dim, m.heads * m.vdim
+        return {"w_in": (2 * k + v + m.decay_rank + m.gate_rank + m.heads, hidden), "conv": (2 * k + v, m.conv),
+                "w_a": (m.heads * m.dim, m.decay_rank), "w_g": (v, m.gate_rank), "A_log": (m.heads,), "dt_bias": (m.heads * m.dim,),
+                "norm": (m.vdim,), "wo": (hidden, v)}
     if isinstance(m, AttentionSpec):
         q, k = m.heads * m.dim, m.kv_heads * m.dim
-        out = {"w_in": (q + k + m.kv_heads * m.vdim, hidden), "wo": (hidden, m.heads * m.vdim)}
+        own = k + m.kv_heads * m.vdim if m.kv_from is None else 0
+        out = {"w_in": (q + own + (m.heads * m.vdim if m.gate else 0), hidden), "wo": (hidden, m.heads * m.vdim)}
+        if m.distance_bias:
+            out.update({"r1": (m.heads,), "r2": (m.heads,)})
         if m.qk_norm:
             out.update({"q_norm": (q,), "k_norm": (k,)})
         if m.sink:
@@ -333,6 +385,12 @@ def layer_shapes(s: LayerSpec, cfg: LayeredConfig) -> dict[str, tuple]:
         out["w_out"] = (H, mix.pop("wo")[1] + ff)
         if isinstance(s.mlp, MoeSpec):
             out.update({f"mlp.{n}": shape for n, shape in expert_shapes(s.mlp, H).items()})
+    elif cfg.block == "pre_norm":
+        if s.mlp is not None:
+            out.update({"norm2": (H,), "mlp.w2": (H, s.mlp.ff)})
+            out.update({"mlp.w13": (s.mlp.ff, H), "mlp.act": (2,)} if isinstance(s.mlp, XieluSpec) else {"mlp.w13": (2 * s.mlp.ff, H)})
+        if cfg.token_side:
+            out.update({"side.gate": (cfg.token_side, H), "side.proj": (H, cfg.token_side), "side.norm": (H,)})
     elif cfg.block == "two_norms":
         out["ls1"] = (H,)
         if s.mlp is not None:
@@ -367,13 +425,17 @@ class LatentMixer(_Mixer):
         freq, self.magnitude = spec.rotary.table()
         self.register_buffer("freq", torch.tensor(freq, dtype=torch.float64, device=self.wo.device), persistent=False)
         self.layout = MX.LatentLayout(spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank)
+        # columns of the projection: queries (or their latent), latents, gate
+        self.gate_at = (spec.q_rank or self.layout.q_rows) + (spec.kv_rank + spec.rot_dim if spec.kv_from is None else 0)
 
     def forward(self, proj, meta: ForwardMeta, run: int, eps: float):
         s = self.spec
         cache = meta.kv_cache[run if s.kv_from is None else s.kv_from][0]
-        return MX.latent_attention(proj, self.layout, cache, meta, freq=self.freq, magnitude=self.magnitude, scale=s.scale,
-                                   window=s.window, sink=getattr(self, "sink", None), w_ukv=self.w_ukv,
-                                   kv_norm=getattr(self, "kv_norm", None), eps=eps)
+        q = MX.part_norm_linear(proj[:, : s.q_rank], self.q_norm, 1, eps, self.w_uq) if s.q_rank else None
+        return MX.latent_attention(proj[:, s.q_rank: self.gate_at], self.layout, cache, meta, freq=self.freq, magnitude=self.magnitude,
+                                   scale=s.scale, window=s.window, sink=getattr(self, "sink", None), w_ukv=self.w_ukv,
+                                   kv_norm=getattr(self, "kv_norm", None), eps=eps, q=q,
+                                   gate=proj[:, self.gate_at: self.gate_at + s.heads * s.vdim] if s.gate else None)
 
 
 class LinearStateMixer(_Mixer):
@@ -387,6 +449,18 @@ class LinearStateMixer(_Mixer):
         return MX.linear_state_attention(proj, s.heads, s.dim, s.vdim, self.decay, meta.states[run], meta, self.norm, eps)
 
 
+class DeltaMixer(_Mixer):
+    def __init__(self, spec: DeltaSpec, *a):
+        super().__init__(spec, *a)
+        assert spec.heads % spec.kv_heads == 0, "heads come in equal groups"
+        self.layout = MX.DeltaLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.conv, spec.decay_rank, spec.gate_rank)
+
+    def forward(self, proj, meta: ForwardMeta, run: int, eps: float):
+        """proj [T, q; k; v; decay latent; gate latent; β] → gated, normed outputs [T, heads · vdim]."""
+        return MX.delta_rule(proj, self.layout, self.conv, self.w_a, self.w_g, self.A_log, self.dt_bias, self.norm, meta.states[run],
+                             meta.states.get((run, "conv")), meta, eps)
+
+
 class AttentionMixer(_Mixer):
     def __init__(self, spec: AttentionSpec, hidden: int, std: float, dtype, device, gen, tag: str, **kw):
         super().__init__(spec, hidden, std, dtype, device, gen, tag, **kw)
@@ -395,18 +469,21 @@ class AttentionMixer(_Mixer):
         assert 2 * len(freq) <= spec.dim, "the rotation covers at most a whole head"
         self.register_buffer("freq", torch.tensor(freq, dtype=torch.float64, device=device), persistent=False)
         self.magnitude = spec.rotary.table()[1] if spec.rotary is not None else 1.0
-        self.layout = MX.AttentionLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim, 2 * len(freq), spec.window, spec.keep_first)
+        assert not (spec.window and spec.chunk), "a window or chunks"
+        self.layout = MX.AttentionLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim, 2 * len(freq), spec.window, spec.keep_first, spec.chunk,
+                                         spec.kv_from is None, spec.value_norm)
 
     def forward(self, proj, meta: ForwardMeta, run: int, eps: float, out=None, aside=None):
-        """proj [T, q; k; v (; more)] → [T, heads · vdim], into `out` if given.  `aside` (mixers.Aside): what reads the same
+        """proj [T, q (; k; v) (; gate; more)] → [T, heads · vdim], into `out` if given.  `aside` (mixers.Aside): what reads the same
         projection beside the attention."""
         s = self.spec
-        kc, vc = meta.kv_cache[run]
+        kc, vc = meta.kv_cache[run if s.kv_from is None else s.kv_from]
         if out is None:
             out = torch.empty(proj.shape[0], s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
         MX.windowed_attention(proj, self.layout, kc, vc, meta, out, freq=self.freq, magnitude=self.magnitude, scale=s.scale,
                               sink=getattr(self, "sink", None), q_norm=getattr(self, "q_norm", None), k_norm=getattr(self, "k_norm", None),
-                              eps=eps, aside=aside)
+                              eps=eps, aside=aside, bias=(self.r1, self.r2) if s.distance_bias else None,
+                              gate=proj[:, self.layout.rows: self.layout.rows + s.heads * s.vdim] if s.gate else None)
         return out
 
 
@@ -472,6 +549,31 @@ class ClampedGLU(nn.Module):
         return ops.linear(MX.clamped_glu(proj, self.spec.limit, self.spec.alpha, self.spec.shift), self.w2)
 
 
+class Xielu(nn.Module):
+    def __init__(self, spec: XieluSpec, hidden: int, std: float, dtype, device, gen, tag: str):
+        super().__init__()
+        self.spec = spec
+        self.w13 = nn.Parameter(gen(f"{tag}.w13", (spec.ff, hidden), std, dtype, device))
+        self.w2 = nn.Parameter(gen(f"{tag}.w2", (hidden, spec.ff), std, dtype, device))
+        self.act = nn.Parameter(torch.zeros(2, dtype=dtype, device=device))
+
+    def forward(self, proj):
+        return ops.linear(MX.xielu(proj, self.act), self.w2)
+
+
+class TokenSide(nn.Module):
+    """y = proj(gelu(gate x) · rows of the layer's part of a token table); the stream norms and adds it."""
+
+    def __init__(self, dim: int, hidden: int, std: float, dtype, device, gen, tag: str):
+        super().__init__()
+        self.gate = nn.Parameter(gen(f"{tag}.gate", (dim, hidden), std, dtype, device))
+        self.proj = nn.Parameter(gen(f"{tag}.proj", (hidden, dim), std, dtype, device))
+        self.norm = nn.Parameter(torch.ones(hidden, dtype=dtype, device=device))
+
+    def forward(self, z, tokens, table, layer: int):
+        return ops.linear(MX.gelu_times_rows(z, tokens, table, layer * self.gate.shape[0]), self.proj)
+
+
 class _Stream:
     """The fp32 residual and a sublayer output that has not been added to it yet.
 
@@ -509,7 +611,8 @@ class _Stream:
 
 
 MIXERS = {LatentSpec: LatentMixer, LinearStateSpec: LinearStateMixer, AttentionSpec: AttentionMixer, DifferentialSpec: DifferentialMixer,
-          SsmSpec: SsmMixer}
+          SsmSpec: SsmMixer, DeltaSpec: DeltaMixer}
+FEED_FORWARDS = {GluSpec: ClampedGLU, XieluSpec: Xielu}
 
 
 class LayeredLayer(nn.Module):
@@ -647,6 +750,68 @@ class TwoNormLayer(nn.Module):
             st.pending.append(MX.Addend(ops.linear(aside.glu_out, mlp.w2), scale=self.ls2))
 
 
+class _PreNormStream:
+    """The fp32 residual of the "pre_norm" arrangement and the sublayer output that has not been added to it yet (with its norm, if it has
+    one).  `project` adds it and multiplies the new residual, normed or as it is, by a weight: one kernel for a handful of rows, a
+    kernel for sum and norm and a product otherwise."""
+
+    def __init__(self, x, _copy, cfg: LayeredConfig):
+        self.x, self.eps, self.mult, self.gain = x, cfg.rms_eps, cfg.residual_mult, cfg.logit_scale
+        self.pending = (None, None)
+
+    def project(self, nw, w):
+        y, yn = self.pending
+        self.pending = (None, None)
+        if MX.few_row_sum(self.x, (), w):
+            out, self.x = MX.residual_linear(self.x, y, yn, self.mult, nw, self.eps, w)
+            return out
+        return MX.product(MX.residual_norm(self.x, y, yn, self.mult, nw, self.eps, w.dtype), w)
+
+    def add(self, y, norm=None):
+        self.pending = (y, norm)
+
+    def finish(self, final_w):
+        return MX.residual_norm(self.x, *self.pending, self.mult, final_w, self.eps, final_w.dtype, gain=self.gain)
+
+    def value(self):
+        """The residual with everything added (debugging and tests)."""
+        x = self.x.clone()
+        if self.pending[0] is not None:
+            MX.residual_norm(x, *self.pending, self.mult, None, self.eps, self.pending[0].dtype)
+        return x
+
+
+class PreNormLayer(nn.Module):
+    """The "pre_norm" arrangement: x + m · mixer(norm1(x)), then + m · feed-forward(norm2(x)), then + m · norm(token input of x)."""
+
+    def __init__(self, spec: LayerSpec, cfg: LayeredConfig, dtype, device, gen, layer: int):
+        super().__init__()
+        self.layer, self.eps = layer, cfg.rms_eps
+        H, std, tag = cfg.hidden_size, cfg.init_std, f"L{layer}"
+        assert spec.mlp is None or type(spec.mlp) in FEED_FORWARDS, "dense feed-forwards in the pre-norm arrangement"
+        assert isinstance(spec.mixer, (LatentSpec, LinearStateSpec, AttentionSpec, DeltaSpec)), "mixers that need no aside"
+
+        def vec():
+            return nn.Parameter(torch.ones(H, dtype=dtype, device=device))
+
+        self.norm1 = vec()
+        self.mix = MIXERS[type(spec.mixer)](spec.mixer, H, std, dtype, device, gen, f"{tag}.mix")
+        self.mlp = self.side = None
+        if spec.mlp is not None:
+            self.norm2 = vec()
+            self.mlp = FEED_FORWARDS[type(spec.mlp)](spec.mlp, H, std, dtype, device, gen, f"{tag}.mlp")
+        if cfg.token_side:
+            self.side = TokenSide(cfg.token_side, H, std, dtype, device, gen, f"{tag}.side")
+
+    def forward(self, st: _PreNormStream, meta: ForwardMeta, run: int):
+        o = self.mix(st.project(self.norm1, self.mix.w_in), meta, run, self.eps)
+        st.add(ops.linear(o, self.mix.wo))
+        if self.mlp is not None:
+            st.add(self.mlp(st.project(self.norm2, self.mlp.w13)))
+        if self.side is not None:
+            st.add(self.side(st.project(None, self.side.gate), *st.token_rows, self.layer), self.side.norm)
+
+
 class ParallelLayer(nn.Module):
     """The "parallel" arrangement: x + mixer(norm(x)) + feed-forward(norm(x)).
 
@@ -712,11 +877,12 @@ class LayeredModel(Qwen3Model):
                 src = cfg.layer_specs[m.kv_from].mixer
                 assert m.kv_from < i and isinstance(src, LatentSpec) and src.kv_from is None and (src.kv_rank, src.rot_dim) == (
                     m.kv_rank, m.rot_dim), f"layer {i} cannot read the latents of layer {m.kv_from}"
-            if isinstance(m, DifferentialSpec) and m.kv_from is not None:
+            if isinstance(m, (DifferentialSpec, AttentionSpec)) and m.kv_from is not None:
                 src = cfg.layer_specs[m.kv_from].mixer
-                assert m.kv_from < i and isinstance(src, DifferentialSpec) and src.kv_from is None and (src.kv_heads, src.dim, src.vdim) == (
+                assert m.kv_from < i and type(src) is type(m) and src.kv_from is None and (src.kv_heads, src.dim, src.vdim) == (
                     m.kv_heads, m.dim, m.vdim), f"layer {i} cannot read the keys and values of layer {m.kv_from}"
         assert cfg.norm_shift == 0.0 or cfg.block == "two_norms", "norm weights stored around another value: two-norm arrangement only"
+        assert (cfg.residual_mult == 1.0 and not cfg.token_side) or cfg.block == "pre_norm", "residual factor, token input: pre-norm arrangement only"
         assert cfg.logit_scale == 1.0 or cfg.block != "output_norm", "a logit scale is part of the final norm of the summing streams"
         if cfg.loop is not None:
             assert 0 <= cfg.loop.start < cfg.loop.stop <= cfg.num_layers and cfg.loop.times > 0, f"{cfg.loop} of {cfg.num_layers} layers"
@@ -727,6 +893,9 @@ class LayeredModel(Qwen3Model):
         self.bigram = None
         if cfg.bigram is not None:
             self.bigram = nn.Parameter(gen("bigram", (cfg.bigram.buckets + 1, cfg.hidden_size), cfg.init_std, dtype, device))
+        self.side_embed = None
+        if cfg.token_side:
+            self.side_embed = nn.Parameter(gen("side_embed", (cfg.vocab_size, cfg.num_layers * cfg.token_side), cfg.init_std, dtype, device))
         self.num_moe_layers = cfg.num_moe_layers
         if cfg.norm_shift:
             with torch.no_grad():
@@ -745,7 +914,7 @@ class LayeredModel(Qwen3Model):
         for r, m in self._run_mixers():
             if isinstance(m, LatentMixer) and m.spec.kv_from is None:
                 rows[r] = ((m.layout.pitch,),)
-            elif isinstance(m, AttentionMixer):
+            elif isinstance(m, AttentionMixer) and m.spec.kv_from is None:
                 rows[r] = ((m.spec.kv_heads, m.spec.dim), (m.spec.kv_heads, m.spec.vdim))
             elif isinstance(m, DifferentialMixer) and m.spec.kv_from is None:
                 rows[r] = ((m.spec.kv_heads, 2 * m.spec.dim), (m.spec.kv_heads, m.spec.vdim))      # a key row holds both maps
@@ -759,8 +928,10 @@ class LayeredModel(Qwen3Model):
                 out[r] = (m.spec.heads, m.spec.dim, m.spec.vdim)
             elif isinstance(m, SsmMixer):
                 out[r] = (m.spec.heads, m.spec.state, m.spec.vdim)
-                if m.spec.conv > 1:
-                    out[(r, "conv")] = (m.spec.conv, m.layout.channels)
+            elif isinstance(m, DeltaMixer):
+                out[r] = (m.spec.heads, m.spec.dim, m.spec.vdim)
+            if isinstance(m, (SsmMixer, DeltaMixer)) and m.spec.conv > 1:
+                out[(r, "conv")] = (m.spec.conv, m.layout.channels)
         return out
 
     def forward(self, tokens, meta: ForwardMeta, hidden_in=None, inputs_embeds=None):
@@ -772,6 +943,7 @@ class LayeredModel(Qwen3Model):
                                                             (big.buckets, big.mul_prev, big.mul_cur) if big is not None else None,
                                                             want_copy=self.cfg.block == "output_norm", positions=meta.positions,
                                                             freq=self.position_freq), self.cfg)
+        st.token_rows = (tokens, self.side_embed)
         meta.record_width = self.cfg.moe_topk
         for run, (l, inject) in enumerate(self.runs):
             st.inject = inject
@@ -780,6 +952,22 @@ class LayeredModel(Qwen3Model):
                 meta.record_residual.append(st.value())
         return st.finish(self.norm)
 
+    def logits(self, hidden):
+        lg = super().logits(hidden)
+        return MX.softcap_(lg, self.cfg.logit_softcap, exact=self.embed.dtype == torch.float32) if self.cfg.logit_softcap else lg
+
+    def log_probs(self, hidden, targets, temperature: float = 1.0, with_entropy: bool = False):
+        if not self.cfg.logit_softcap:
+            return super().log_probs(hidden, targets, temperature, with_entropy)
+        out, entropy = [], []
+        for h, t in zip(hidden.split(512), targets.split(512)):        # a few rows of the whole vocabulary at a time
+            lp = torch.log_softmax(self.logits(h).float() / temperature, -1)
+            out.append(lp.gather(-1, t.long()[:, None]).squeeze(-1))
+            if with_entropy:
+                entropy.append(-(lp.exp() * lp).sum(-1))
+        return torch.cat(out), torch.cat(entropy) if with_entropy else None
+
 
 # arrangement → (layer, stream of residual and pending outputs)
-BLOCKS = {"output_norm": (LayeredLayer, _Stream), "parallel": (ParallelLayer, _SumStream), "two_norms": (TwoNormLayer, _TwoNormStream)}
+BLOCKS = {"output_norm": (LayeredLayer, _Stream), "parallel": (ParallelLayer, _SumStream), "two_norms": (TwoNormLayer, _TwoNormStream),
+          "pre_norm": (PreNormLayer, _PreNormStream)}

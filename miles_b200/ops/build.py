@@ -27,29 +27,34 @@ def sources() -> list[str]:
     return sorted(glob.glob(os.path.join(CSRC, "*.cu")) + glob.glob(os.path.join(CSRC, "*.cpp")))
 
 
-# What serving a layer-by-layer decoder (models/layered.py) takes: dense projections, sampling and the mixers its layers have.  A
+# What serving a layer-by-layer decoder (models/layered.py) takes: dense projections, sampling and the parts its layers need.  A
 # checkout without a full build compiles only these (`build_serve`), into an extension of its own with the same interface.
 SERVE_SUFFIX = "_serve"
 SERVE_SOURCES = ["counter.cpp", "bindings.cpp", "bindings_more.cpp", "bindings_misc.cpp", "bindings_mixers.cpp", "gemm.cu", "gemm_small.cu",
                  "gemv.cu", "misc.cu", "mixers.cu", "paged_attend.cu"]
-_EXPERTS = ["bindings_moe.cpp", "moe.cu", "experts_any.cu"]
-_WINDOW = ["attention_window_tc.cu", "window_decode.cu"]
-SERVE_KINDS = {
-    "latent": ["attention_latent_tc.cu", "latent_attn.cu", "latent_decode.cu", "latent_decode_tc.cu", "linear_state.cu", "linear_chunk.cu"],
-    "attention": [*_EXPERTS, *_WINDOW, "window_prep.cu"],
-    "hybrid": [*_EXPERTS, *_WINDOW, "diff_prep.cu", "ssm_state.cu", "ssm_chunk.cu"],
+SERVE_PARTS = {
+    "latent": ["attention_latent_tc.cu", "latent_attn.cu", "latent_decode.cu", "latent_decode_tc.cu"],
+    "linear": ["linear_state.cu", "linear_chunk.cu"],
+    "attention": ["attention_window_tc.cu", "window_decode.cu"],
+    "prep": ["window_prep.cu"],
+    "differential": ["diff_prep.cu"],
+    "ssm": ["ssm_state.cu", "ssm_chunk.cu"],
+    "delta": ["delta_state.cu"],
+    "experts": ["bindings_moe.cpp", "moe.cu", "experts_any.cu"],
 }
 _serving: str | None = None                   # the serving build this process asked for
 
 
 def serve_kind(cfg) -> str:
-    """Which serving build a layered configuration needs."""
-    from ..models.layered import AttentionSpec, DifferentialSpec, SsmSpec
+    """Which serving build a layered configuration needs: the names of its parts."""
+    from ..models.layered import AttentionSpec, DeltaSpec, DifferentialSpec, LatentSpec, LinearStateSpec, MoeSpec, SsmSpec
 
-    of = {AttentionSpec: "attention", DifferentialSpec: "hybrid", SsmSpec: "hybrid"}
-    kinds = {of.get(type(s.mixer), "latent") for s in cfg.layer_specs}
-    assert len(kinds) == 1, f"no serving build has the mixers of {kinds} together: run a full build"
-    return kinds.pop()
+    of = {LatentSpec: {"latent"}, LinearStateSpec: {"linear"}, AttentionSpec: {"attention", "prep"}, DifferentialSpec: {"attention", "differential"},
+          SsmSpec: {"ssm"}, DeltaSpec: {"delta"}}
+    parts = set().union(*(of[type(s.mixer)] for s in cfg.layer_specs))
+    if any(isinstance(s.mlp, MoeSpec) for s in cfg.layer_specs):
+        parts.add("experts")
+    return "_".join(sorted(parts))
 
 
 def source_stamp() -> str:
@@ -87,7 +92,7 @@ def serve_so_path(kind: str) -> str:
 
 
 def build_serve(kind: str, verbose: bool = False) -> str:
-    """Make sure an extension that can serve layer-by-layer decoders with this kind of mixers is built from the sources as they are:
+    """Make sure an extension that can serve layer-by-layer decoders with these parts (`serve_kind`) is built from the sources as they are:
     an up-to-date full build if there is one, else the serving subset.  Returns its path; `load()` then picks the same one."""
     global _serving
     if _is_current(so_path(False)):
@@ -98,9 +103,10 @@ def build_serve(kind: str, verbose: bool = False) -> str:
 
         _toolchain_env()
         os.makedirs(os.path.dirname(so), exist_ok=True)
+        parts = kind.split("_")
         cpp_extension.load(
-            name=f"{EXT_NAME}{SERVE_SUFFIX}_{kind}", sources=[os.path.join(CSRC, f) for f in SERVE_SOURCES + SERVE_KINDS[kind]],
-            extra_cflags=["-O3", "-std=c++17", "-DMB_SERVE_SUBSET", f"-DMB_SERVE_{kind.upper()}"], extra_cuda_cflags=NVCC_FLAGS,
+            name=f"{EXT_NAME}{SERVE_SUFFIX}_{kind}", sources=[os.path.join(CSRC, f) for f in SERVE_SOURCES + sum((SERVE_PARTS[p] for p in parts), [])],
+            extra_cflags=["-O3", "-std=c++17", "-DMB_SERVE_SUBSET", *(f"-DMB_SERVE_{p.upper()}" for p in parts)], extra_cuda_cflags=NVCC_FLAGS,
             extra_include_paths=[CSRC], build_directory=os.path.dirname(so), verbose=verbose, with_cuda=True)
         _write_stamp(so)
     _serving = kind
@@ -154,7 +160,8 @@ def load():
     debug = debug_requested()
     path, suffix = so_path(debug), DEBUG_SUFFIX if debug else ""
     if not debug and not _is_current(path):
-        for kind in [_serving] if _serving else SERVE_KINDS:
+        built = sorted(glob.glob(BUILD_DIR + SERVE_SUFFIX + "_*"))
+        for kind in [_serving] if _serving else [d[len(BUILD_DIR + SERVE_SUFFIX) + 1:] for d in built]:
             if _is_current(serve_so_path(kind)):
                 path, suffix = serve_so_path(kind), f"{SERVE_SUFFIX}_{kind}"
                 break

@@ -27,6 +27,8 @@ static constexpr float kLog2e = 1.4426950408889634f;
 struct Params {
   __nv_bfloat16* o;            // [tokens, H, vdim]
   const __nv_bfloat16* sink;   // [H] or null
+  const __nv_bfloat16* gate;   // rows of gate_ld, [H·vdim], or null: outputs times its sigmoid
+  long long gate_ld;
   const int* cu_q;
   const int* cu_k;
   int H, dim, vdim, rank_p;
@@ -273,6 +275,15 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             if (c * 32 + i < p.vdim) {         // vdim is a multiple of 8
+              if (p.gate != nullptr) {
+                const uint4 gv = *reinterpret_cast<const uint4*>(p.gate + static_cast<long long>(q_start + q0 + row) * p.gate_ld + h * p.vdim + c * 32 + i);
+                const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+                for (int k = 0; k < 8; ++k) {
+                  const float z = __uint_as_float((k & 1) ? gw[k / 2] & 0xffff0000u : gw[k / 2] << 16);
+                  o[i + k] = __float_as_uint(__uint_as_float(o[i + k]) * __fdividef(1.f, 1.f + __expf(-z)));
+                }
+              }
               uint4 v;
               v.x = pack_bf16x2(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
               v.y = pack_bf16x2(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
@@ -315,11 +326,12 @@ using namespace mb;
 
 // q [t_long, H, (NA + 1)·64] zero-padded queries; kv [Tk, H·dim + H·vdim] expanded keys and values; lat [Tk, pitch] gathered cache rows;
 // o [t_long, H, vdim].  dim, vdim multiples of 8, dim ≤ 128, rot ≤ 64, vdim ≤ 128, scale > 0.
-extern "C" int mb_latent_prefill(const void* q, const void* kv, const void* lat, void* o, const void* sink, const int* cu_q, const int* cu_k,
-                                 int n_seq, int max_q, int t_long, int tk, float scale, int window, MbLatent L, int* error_flag,
+extern "C" int mb_latent_prefill(const void* q, const void* kv, const void* lat, void* o, const void* sink, const void* gate, long long gate_ld,
+                                 const int* cu_q, const int* cu_k, int n_seq, int max_q, int t_long, int tk, float scale, int window, MbLatent L, int* error_flag,
                                  cudaStream_t s) {
   if (n_seq <= 0 || t_long <= 0) return 0;
   if (L.dim % 8 || L.vdim % 8 || L.dim > 128 || L.rot > 64 || L.vdim > 128 || !(scale > 0.f)) return -3;
+  if (gate != nullptr && (gate_ld % 8 || reinterpret_cast<uintptr_t>(gate) % 16)) return -3;
   const int na = (L.dim + 63) / 64, nv = (L.vdim + 63) / 64;
   CUtensorMap tq, tkv, tl;
   const long long qw = static_cast<long long>(L.heads) * (na + 1) * 64, kvw = static_cast<long long>(L.heads) * (L.dim + L.vdim);
@@ -329,7 +341,7 @@ extern "C" int mb_latent_prefill(const void* q, const void* kv, const void* lat,
   if (rc) return 2000 + rc;
   rc = make_tmap_bf16_2d(&tl, lat, tk, L.pitch, L.pitch, fl::BKV, 64);
   if (rc) return 3000 + rc;
-  fl::Params p{reinterpret_cast<__nv_bfloat16*>(o), reinterpret_cast<const __nv_bfloat16*>(sink), cu_q, cu_k, L.heads, L.dim, L.vdim, L.rank_p,
+  fl::Params p{reinterpret_cast<__nv_bfloat16*>(o), reinterpret_cast<const __nv_bfloat16*>(sink), reinterpret_cast<const __nv_bfloat16*>(gate), gate_ld, cu_q, cu_k, L.heads, L.dim, L.vdim, L.rank_p,
                scale, window, error_flag};
   if (na == 1) return nv == 1 ? fl::launch<1, 1>(tq, tkv, tl, p, max_q, n_seq, s) : fl::launch<1, 2>(tq, tkv, tl, p, max_q, n_seq, s);
   return nv == 1 ? fl::launch<2, 1>(tq, tkv, tl, p, max_q, n_seq, s) : fl::launch<2, 2>(tq, tkv, tl, p, max_q, n_seq, s);

@@ -11,7 +11,9 @@
 //     the sequence's end are masked;
 //   * differential attention (MbDiff): heads 2h and 2h + 1 are neighbouring rows; their threads exchange the two maps' outputs, and the
 //     difference is normed and gated on its way out;
-//   * the key tiles of a query tile are those of the kept first tokens and those of the window; what lies between is skipped.
+//   * the key tiles of a query tile are those of the kept first tokens and those of the window, or of its tokens' chunks; what lies
+//     between is skipped;
+//   * BIAS: r1 · ln(1 + r2 · distance) comes off the scores; outputs may pass a gate (MbScores).
 #include "launch.h"
 #include "ptx.cuh"
 
@@ -39,7 +41,8 @@ struct Params {
   int group, tokens;           // query heads per key head, tokens per tile
   int dim, vdim;
   float scale;
-  int window, keep;            // window 0: all earlier keys
+  int window, keep, chunk;     // window 0: all earlier keys, or those of a chunk
+  MbScores x;
   MbDiff diff;
   int* error_flag;
 };
@@ -50,7 +53,7 @@ struct Cfg {
   static constexpr int q = 0, k = kQBytes, v = k + 2 * kKBytes, bars = v + 2 * kVBytes, total = bars + 256;
 };
 
-template <int NA, int NV>
+template <int NA, int NV, bool BIAS>
 __global__ void __launch_bounds__(192, 2)
 window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                       Params p) {
@@ -79,7 +82,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   if (t0 >= L) return;
   const int first_pos = p.positions[q_start] + t0;             // positions of the tile's tokens: first_pos … last_pos
   const int last_pos = first_pos + min(p.tokens, L - t0) - 1;
-  const int win_tile = p.window > 0 ? max(0, first_pos - p.window + 1) / BKV : 0;
+  auto first_key = [&](int pos) { return p.window > 0 ? pos - p.window + 1 : p.chunk > 0 ? pos - pos % p.chunk : 0; };
+  const int win_tile = max(0, first_key(first_pos)) / BKV;
   const int n_keep = p.window > 0 ? min((p.keep + BKV - 1) / BKV, win_tile) : 0;
   const int n_blocks = n_keep + last_pos / BKV + 1 - win_tile;
   auto key_of = [&](int j) { return (j < n_keep ? j : win_tile + j - n_keep) * BKV; };
@@ -184,9 +188,14 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     const bool valid = tok < p.tokens && t0 + tok < L;
     const int pos = valid ? first_pos + tok : -1;                           // a row of nothing sees no key
     const uint32_t lane_off = static_cast<uint32_t>(q4 * 32) << 16;
-    const float sl2 = p.scale * kLog2e;
-    const int lo = p.window > 0 ? pos - p.window + 1 : 0;                   // first key of the row's window
-    const int tile_lo = p.window > 0 ? last_pos - p.window + 1 : 0;         // … of the tile's last token
+    const float sl2 = BIAS ? 1.f : p.scale * kLog2e;                        // with a bias scores are in these units before the maximum
+    const int lo = first_key(pos);                                          // first key of the row's window or chunk
+    const int tile_lo = first_key(last_pos);                                // … of the tile's last token
+    float r1 = 0.f, r2 = 0.f;
+    if (BIAS && valid) {
+      r1 = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.x.r1)[head]);
+      r2 = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.x.r2)[head]);
+    }
     const int keep = p.window > 0 ? p.keep : 0;
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
@@ -206,8 +215,12 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           float v = __uint_as_float(s[c][i]);
+          const int col = kv0 + c * 32 + i;
+          if (BIAS) {
+            v = fmaf(v, p.scale * kLog2e, -r1 * __log2f(fmaf(r2, static_cast<float>(pos - col), 1.f)));
+            s[c][i] = __float_as_uint(v);
+          }
           if (need_mask) {
-            const int col = kv0 + c * 32 + i;
             if (col > pos || (col < lo && col >= keep)) v = -INFINITY;
             s[c][i] = __float_as_uint(v);
           }
@@ -341,6 +354,17 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 #pragma unroll
             for (int i = 0; i < 32; i += 8) {
               if (c * 32 + i < p.vdim) {         // vdim is a multiple of 8
+                if (p.x.gate != nullptr) {
+                  const __nv_bfloat16* gr = reinterpret_cast<const __nv_bfloat16*>(p.x.gate) + (q_start + t0 + tok) * p.x.gate_ld +
+                                            static_cast<long long>(head) * p.vdim + c * 32 + i;
+                  const uint4 gv = *reinterpret_cast<const uint4*>(gr);
+                  const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+                  for (int k = 0; k < 8; ++k) {
+                    const float z = __uint_as_float((k & 1) ? gw[k / 2] & 0xffff0000u : gw[k / 2] << 16);
+                    o[i + k] = __float_as_uint(__uint_as_float(o[i + k]) * __fdividef(1.f, 1.f + __expf(-z)));
+                  }
+                }
                 uint4 v;
                 v.x = pack_bf16x2(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
                 v.y = pack_bf16x2(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
@@ -362,20 +386,26 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   }
 }
 
-template <int NA, int NV>
-static int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const Params& p, int max_q, int kv_heads, int n_seq,
+template <int NA, int NV, bool BIAS>
+static int launch_as(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const Params& p, int max_q, int kv_heads, int n_seq,
                   cudaStream_t s) {
   using G = Cfg<NA, NV>;
   static bool once = false;
   if (!once) {
-    cudaError_t e = cudaFuncSetAttribute(window_prefill_kernel<NA, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::total);
+    cudaError_t e = cudaFuncSetAttribute(window_prefill_kernel<NA, NV, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::total);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(window_prefill_kernel<NA, NV>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+      e = cudaFuncSetAttribute(window_prefill_kernel<NA, NV, BIAS>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
     if (e != cudaSuccess) return static_cast<int>(e);
     once = true;
   }
-  window_prefill_kernel<NA, NV><<<dim3((max_q + p.tokens - 1) / p.tokens, kv_heads, n_seq), 192, G::total, s>>>(tq, tk, tv, p);
+  window_prefill_kernel<NA, NV, BIAS><<<dim3((max_q + p.tokens - 1) / p.tokens, kv_heads, n_seq), 192, G::total, s>>>(tq, tk, tv, p);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <int NA, int NV>
+static int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const Params& p, int max_q, int kv_heads, int n_seq,
+                  cudaStream_t s) {
+  return p.x.r1 != nullptr ? launch_as<NA, NV, true>(tq, tk, tv, p, max_q, kv_heads, n_seq, s) : launch_as<NA, NV, false>(tq, tk, tv, p, max_q, kv_heads, n_seq, s);
 }
 
 }  // namespace fw
@@ -387,11 +417,13 @@ using namespace mb;
 // o_row elements (a multiple of 8).  dim, vdim multiples of 8 up to 128, block_size a multiple of 8, up to 128 query heads per key head, scale > 0.
 extern "C" int mb_window_prefill(const void* q, const void* kc, const void* vc, void* o, long long o_row, const void* sink, const int* cu_q,
                                  const int* positions, const int* block_table, int max_blocks, int block_size, int num_blocks, int n_seq, int max_q,
-                                 int t_long, float scale, MbWindow L, MbDiff d, int* error_flag, cudaStream_t s) {
+                                 int t_long, float scale, MbWindow L, MbDiff d, MbScores x, int* error_flag, cudaStream_t s) {
   if (n_seq <= 0 || t_long <= 0) return 0;
   const int group = L.heads / L.kv_heads, na = (L.dim + 63) / 64, nv = (L.vdim + 63) / 64;
   if (L.dim % 8 || L.vdim % 8 || L.dim > 128 || L.vdim > 128 || L.q_pitch != na * 64 || L.heads % L.kv_heads || group > 128 || block_size % 8 ||
-      o_row % 8 || !(scale > 0.f) || (d.lam != nullptr && (sink != nullptr || group % 2)))
+      o_row % 8 || !(scale > 0.f) || (d.lam != nullptr && (sink != nullptr || group % 2 || x.gate != nullptr)) || (L.chunk > 0 && L.window > 0) ||
+      (x.r1 != nullptr && sink != nullptr) ||
+      (x.gate != nullptr && (x.gate_ld % 8 || reinterpret_cast<uintptr_t>(x.gate) % 16)))
     return -3;
   int box = 64;
   while (block_size % box) box /= 2;
@@ -405,7 +437,7 @@ extern "C" int mb_window_prefill(const void* q, const void* kc, const void* vc, 
   rc = make_tmap_bf16_2d(&tv, vc, rows, vw, vw, box, 64);
   if (rc) return 3000 + rc;
   fw::Params p{reinterpret_cast<__nv_bfloat16*>(o), o_row, reinterpret_cast<const __nv_bfloat16*>(sink), cu_q, positions, block_table, max_blocks,
-               block_size, box, group, tokens, L.dim, L.vdim, scale, L.window, L.keep, d, error_flag};
+               block_size, box, group, tokens, L.dim, L.vdim, scale, L.window, L.keep, L.chunk, x, d, error_flag};
   if (na == 1) return nv == 1 ? fw::launch<1, 1>(tq, tk, tv, p, max_q, L.kv_heads, n_seq, s) : fw::launch<1, 2>(tq, tk, tv, p, max_q, L.kv_heads, n_seq, s);
   return nv == 1 ? fw::launch<2, 1>(tq, tk, tv, p, max_q, L.kv_heads, n_seq, s) : fw::launch<2, 2>(tq, tk, tv, p, max_q, L.kv_heads, n_seq, s);
 }

@@ -117,7 +117,7 @@ void register_more(pybind11::module& m) {
   m.def("install_crash_handler", &install_crash_handler);
   register_misc(m);
   register_mixers(m);
-#if !defined(MB_SERVE_SUBSET) || defined(MB_SERVE_ATTENTION) || defined(MB_SERVE_HYBRID)
+#if !defined(MB_SERVE_SUBSET) || defined(MB_SERVE_EXPERTS)
   register_moe(m);
 #endif
 #ifndef MB_SERVE_SUBSET

@@ -166,17 +166,20 @@ __device__ __forceinline__ void stage_rows(uint8_t* xs, int rows, int valid, int
   }
 }
 
-// Output-norm form: x' = x + y / rms(y) · norm_w · scale_w with an fp32 residual x (block 0 writes x' to x_out, another buffer: every
-// CTA reads x); the staged value is bf16(x').
+// Output-norm form: x' = x + mult · y / rms(y) · norm_w · scale_w with an fp32 residual x (block 0 writes x' to x_out, another buffer:
+// every CTA reads x; scale_w null: 1); the staged value is bf16(x').  NEXT: bf16(x' · next_w), Σx'² → rstd[row].
+template <bool NEXT>
 __device__ __forceinline__ void stage_rows_output_norm(uint8_t* xs, int rows, int valid, int K, const bf16* __restrict__ y,
                                                        const float* __restrict__ x, const bf16* __restrict__ norm_w,
-                                                       const bf16* __restrict__ scale_w, float eps, float* x_out) {
+                                                       const bf16* __restrict__ scale_w, float mult, const bf16* __restrict__ next_w, float eps,
+                                                       float* x_out, float* rstd_next) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nv = K / 8, stride = staged_stride(K);
   for (int r = warp; r < rows; r += kWarps) {
     uint8_t* row = xs + r * stride;
     if (r >= valid) {
       for (int v = lane; v < nv; v += 32) *reinterpret_cast<uint4*>(row + v * 16) = make_uint4(0, 0, 0, 0);
+      if (NEXT && lane == 0) rstd_next[r] = 0.f;
       continue;
     }
     const bf16* yr = y + static_cast<long long>(r) * K;
@@ -184,11 +187,12 @@ __device__ __forceinline__ void stage_rows_output_norm(uint8_t* xs, int rows, in
     float ss = 0.f;
 #pragma unroll 4
     for (int v = lane; v < nv; v += 32) ss += sumsq8(*reinterpret_cast<const uint4*>(yr + v * 8));
-    const float rstd = __fdiv_rn(1.f, __fsqrt_rn(__fdiv_rn(warp_sum(ss), static_cast<float>(K)) + eps));
+    const float rstd = __fdiv_rn(mult, __fsqrt_rn(__fdiv_rn(warp_sum(ss), static_cast<float>(K)) + eps));
+    ss = 0.f;
 #pragma unroll 2
     for (int v = lane; v < nv; v += 32) {
       const uint4 yv = *reinterpret_cast<const uint4*>(yr + v * 8), nv4 = *reinterpret_cast<const uint4*>(norm_w + v * 8),
-                  sv = *reinterpret_cast<const uint4*>(scale_w + v * 8);
+                  sv = scale_w != nullptr ? *reinterpret_cast<const uint4*>(scale_w + v * 8) : make_uint4(0x3f803f80u, 0x3f803f80u, 0x3f803f80u, 0x3f803f80u);
       float4 xa = *reinterpret_cast<const float4*>(xr + v * 8), xb = *reinterpret_cast<const float4*>(xr + v * 8 + 4);
       const float2 y0 = unpack2(yv.x), y1 = unpack2(yv.y), y2 = unpack2(yv.z), y3 = unpack2(yv.w);
       const float2 n0 = unpack2(nv4.x), n1 = unpack2(nv4.y), n2 = unpack2(nv4.z), n3 = unpack2(nv4.w);
@@ -205,18 +209,30 @@ __device__ __forceinline__ void stage_rows_output_norm(uint8_t* xs, int rows, in
         *reinterpret_cast<float4*>(x_out + static_cast<long long>(r) * K + v * 8) = xa;
         *reinterpret_cast<float4*>(x_out + static_cast<long long>(r) * K + v * 8 + 4) = xb;
       }
+      if (NEXT) {
+        const uint4 mv = *reinterpret_cast<const uint4*>(next_w + v * 8);
+        const float2 m0 = unpack2(mv.x), m1 = unpack2(mv.y), m2 = unpack2(mv.z), m3 = unpack2(mv.w);
+        ss += xa.x * xa.x + xa.y * xa.y + xa.z * xa.z + xa.w * xa.w + xb.x * xb.x + xb.y * xb.y + xb.z * xb.z + xb.w * xb.w;
+        xa.x *= m0.x; xa.y *= m0.y; xa.z *= m1.x; xa.w *= m1.y;
+        xb.x *= m2.x; xb.y *= m2.y; xb.z *= m3.x; xb.w *= m3.y;
+      }
       *reinterpret_cast<uint4*>(row + v * 16) = make_uint4(pack2(xa.x, xa.y), pack2(xa.z, xa.w), pack2(xb.x, xb.y), pack2(xb.z, xb.w));
+    }
+    if (NEXT) {
+      ss = warp_sum(ss);
+      if (lane == 0) rstd_next[r] = __fdiv_rn(1.f, __fsqrt_rn(__fdiv_rn(ss, static_cast<float>(K)) + eps));
     }
   }
 }
 
-// Sum-norm form: x' = x + y1·s1 + y2·s2 + extra (fp32 x and extra, every addend and scale optional; block 0 writes x' to x_out, another
-// buffer); the staged value is bf16(x' · (norm_w + shift)), Σx'² → rstd[row].
+// Sum-norm form: x' = x + mult·(y1·s1 + y2·s2) + extra (fp32 x and extra, every addend and scale optional; block 0 writes x' to x_out,
+// another buffer); the staged value is bf16(x' · (norm_w + shift)), Σx'² → rstd[row].  Without norm_w: bf16(x'), rstd[row] = 1.
 template <bool SCALED>
 __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int valid, int K, const float* __restrict__ x,
                                                     const bf16* __restrict__ y1, const bf16* __restrict__ s1, const bf16* __restrict__ y2,
                                                     const bf16* __restrict__ s2, const float* __restrict__ extra,
-                                                    const bf16* __restrict__ norm_w, float eps, float shift, float* x_out, float* rstd) {
+                                                    const bf16* __restrict__ norm_w, float eps, float shift, float mult, float* x_out,
+                                                    float* rstd) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nv = K / 8, stride = staged_stride(K);
   for (int r = warp; r < rows; r += kWarps) {
@@ -238,7 +254,7 @@ __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int v
       const uint4 p2 = y2 != nullptr ? *reinterpret_cast<const uint4*>(y2 + at) : zero;
       const uint4 q1 = SCALED && s1 != nullptr ? *reinterpret_cast<const uint4*>(s1 + v * 8) : one;
       const uint4 q2 = SCALED && s2 != nullptr ? *reinterpret_cast<const uint4*>(s2 + v * 8) : one;
-      const uint4 nw = *reinterpret_cast<const uint4*>(norm_w + v * 8);
+      const uint4 nw = norm_w != nullptr ? *reinterpret_cast<const uint4*>(norm_w + v * 8) : one;
       f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
       if (extra != nullptr) {
         const float4 c = *reinterpret_cast<const float4*>(extra + at), d = *reinterpret_cast<const float4*>(extra + at + 4);
@@ -250,8 +266,8 @@ __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int v
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float2 u = unpack2(w1[i]), q = unpack2(w2[i]), n = unpack2(wn[i]), c = unpack2(l1[i]), d = unpack2(l2[i]);
-        f[2 * i] += SCALED ? u.x * c.x + q.x * d.x : u.x + q.x;
-        f[2 * i + 1] += SCALED ? u.y * c.y + q.y * d.y : u.y + q.y;
+        f[2 * i] += mult * (SCALED ? u.x * c.x + q.x * d.x : u.x + q.x);
+        f[2 * i + 1] += mult * (SCALED ? u.y * c.y + q.y * d.y : u.y + q.y);
         ss += f[2 * i] * f[2 * i] + f[2 * i + 1] * f[2 * i + 1];
         o[i] = SCALED ? pack2(f[2 * i] * (n.x + shift), f[2 * i + 1] * (n.y + shift)) : pack2(f[2 * i] * n.x, f[2 * i + 1] * n.y);
       }
@@ -262,7 +278,7 @@ __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int v
       *reinterpret_cast<uint4*>(row + v * 16) = make_uint4(o[0], o[1], o[2], o[3]);
     }
     ss = warp_sum(ss);
-    if (lane == 0) rstd[r] = __fdiv_rn(1.f, __fsqrt_rn(__fdiv_rn(ss, static_cast<float>(K)) + eps));
+    if (lane == 0) rstd[r] = norm_w != nullptr ? __fdiv_rn(1.f, __fsqrt_rn(__fdiv_rn(ss, static_cast<float>(K)) + eps)) : 1.f;
   }
 }
 
@@ -297,7 +313,7 @@ struct GemvParams {
   float* x32_out;
   const bf16 *y1, *s1, *y2, *s2;   // sum-norm form: sublayer outputs with their scales, an fp32 addend, what norm weights count from
   const float* extra;
-  float shift;
+  float shift, mult;      // mult: factor on the addends
   const bf16* norm_w2;    // norm weight of the second product's rows (null: the first one's)
   const bf16* W2;         // a second weight [N2, K] behind the first: y2out[M, N2] (+ bias2), fp32 or bf16
   const bf16* bias2;
@@ -309,14 +325,15 @@ struct GemvParams {
   int static_w;           // W is not written by a kernel that may still run: its first loads go before the dependency wait
 };
 
-enum GemvMode { kPlain = 0, kAddNorm = 1, kOutputNorm = 2, kSumNorm = 3, kScaledSum = 4 };      // kScaledSum: kSumNorm with scales, shifted norm weights, two norms
+// kScaledSum: kSumNorm with scales, shifted norm weights, two norms; kOutputNormNext: kOutputNorm with the new residual normed by norm_w2
+enum GemvMode { kPlain = 0, kAddNorm = 1, kOutputNorm = 2, kSumNorm = 3, kScaledSum = 4, kOutputNormNext = 5 };
 
 // NT: groups of 8 tokens (1 or 2); S: ring stages.  One CTA = 16 output rows; its 8 warps take the 32-wide k chunks round-robin.
 template <int NT, int MODE, int S>
 __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   constexpr bool NORM = MODE == kAddNorm;
   constexpr bool SUM = MODE == kSumNorm || MODE == kScaledSum;
-  constexpr bool SCALED = NORM || SUM;                   // the staged rows still lack 1 / rms
+  constexpr bool SCALED = NORM || SUM || MODE == kOutputNormNext;                   // the staged rows still lack 1 / rms
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float red[kWarps][NT][16][8];
   __shared__ float rstd_s[NT * 8];
@@ -349,11 +366,11 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   if (p.static_w) pdl_wait();          // static weights: their first loads are already in flight
   if (NORM) {
     stage_rows<true>(xs, NT * 8, p.M, p.K, p.x, p.residual, p.norm_w, p.eps, p.res_out, rstd_s);
-  } else if (MODE == kOutputNorm) {
-    stage_rows_output_norm(xs, NT * 8, p.M, p.K, p.x, p.x32, p.norm_w, p.scale_w, p.eps, p.x32_out);
+  } else if (MODE == kOutputNorm || MODE == kOutputNormNext) {
+    stage_rows_output_norm<MODE == kOutputNormNext>(xs, NT * 8, p.M, p.K, p.x, p.x32, p.norm_w, p.scale_w, p.mult, p.norm_w2, p.eps, p.x32_out, rstd_s);
   } else if (SUM) {
     stage_rows_sum_norm<MODE == kScaledSum>(xs, NT * 8, p.M, p.K, p.x32, p.y1, p.s1, p.y2, p.s2, p.extra, second && p.norm_w2 != nullptr ? p.norm_w2 : p.norm_w, p.eps,
-                        p.shift, p.x32_out, rstd_s);
+                        p.shift, p.mult, p.x32_out, rstd_s);
   } else {
     stage_rows_async(xs, NT * 8, p.M, p.K, p.x);
     cp_commit();
@@ -753,9 +770,11 @@ extern "C" int mb_gemv(const void* x, const void* residual, const void* norm_w, 
   return static_cast<int>(e);
 }
 
-// out[M, N] = x' · Wᵀ with x' = x + y / rms(y) · norm_w · scale_w (x, x_out fp32 and distinct); same limits as mb_gemv.
-extern "C" int mb_gemv_output_norm(const float* x, const void* y, const void* norm_w, const void* scale_w, float eps, const void* W, void* out,
-                                   long long ldo, float* x_out, int M, int N, int K, int static_w, cudaStream_t s) {
+// out[M, N] = x' · Wᵀ with x' = x + mult · y / rms(y) · norm_w · scale_w (x, x_out fp32 and distinct; scale_w null: 1), or, with next_w,
+// (x' / rms(x') · next_w) · Wᵀ; same limits as mb_gemv.
+extern "C" int mb_gemv_output_norm(const float* x, const void* y, const void* norm_w, const void* scale_w, float mult, const void* next_w,
+                                   float eps, const void* W, void* out, long long ldo, float* x_out, int M, int N, int K, int static_w,
+                                   cudaStream_t s) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 16 || K % 32 || K <= 0) return -1;
   const int nt = M <= 8 ? 1 : 2;
@@ -766,11 +785,14 @@ extern "C" int mb_gemv_output_norm(const float* x, const void* y, const void* no
   p.x32_out = x_out;
   p.norm_w = reinterpret_cast<const bf16*>(norm_w);
   p.scale_w = reinterpret_cast<const bf16*>(scale_w);
+  p.mult = mult;
+  p.norm_w2 = reinterpret_cast<const bf16*>(next_w);
   p.eps = eps;
   p.W = reinterpret_cast<const bf16*>(W);
   p.y = out;
   p.ldy = ldo;
   p.M = M; p.N = N; p.K = K; p.static_w = static_w;
+  if (next_w != nullptr) return static_cast<int>(nt == 1 ? launch_gemv<1, kOutputNormNext>(p, s) : launch_gemv<2, kOutputNormNext>(p, s));
   return static_cast<int>(nt == 1 ? launch_gemv<1, kOutputNorm>(p, s) : launch_gemv<2, kOutputNorm>(p, s));
 }
 
@@ -791,6 +813,7 @@ extern "C" int mb_gemv_sum_norm(MbGemvSum a, cudaStream_t s) {
   p.norm_w2 = b(a.norm_w2);
   p.eps = a.eps;
   p.shift = a.shift;
+  p.mult = a.mult;
   p.W = b(a.W);
   p.y = a.y;
   p.ldy = a.ldy;

@@ -15,7 +15,8 @@ namespace mx {
 // form; later ones the rotated part and the padding of an absorbed query [H][pitch] (head_linear fills [0, rank)).
 // VEC: rows and head parts start on 16-byte boundaries and are whole 16-byte pieces.
 template <typename T, bool VEC>
-__global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ proj, long long ld, const int* __restrict__ positions,
+__global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ q_in, long long q_ld, const T* __restrict__ kv_in, long long kv_ld,
+                                                          const int* __restrict__ positions,
                                                           const long long* __restrict__ slots, const double* __restrict__ freq,
                                                           float magnitude, const T* __restrict__ kv_norm, float eps,
                                                           T* __restrict__ cache, T* __restrict__ q_abs, T* __restrict__ q_full, int t_long,
@@ -27,7 +28,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
   pdl_wait();
   const long long t = blockIdx.x;
   const int half = L.rot / 2, dq = L.dim + L.rot;
-  const T* p = proj + t * ld;
+  const T* p = q_in + t * q_ld;
   rotary_table<T, 256>(cs, positions[t], freq, half, magnitude);
   auto rotate = [&](float (&f)[V], int k) {      // V values, the first one the even half of pair k
 #pragma unroll
@@ -72,7 +73,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
   }
   const long long slot = slots[t];
   if (slot < 0) return;
-  const T* kv = p + static_cast<long long>(L.heads) * dq;
+  const T* kv = kv_in + t * kv_ld;
   float ss = 0.f;
   for (int i = threadIdx.x; i < L.rank; i += 256) {
     const float v = to_f(kv[i]);
@@ -96,7 +97,8 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
 // y[t, h, n] = Σ_k x[t, h, k] · w[h](n, k); w [H, N, K] when NK, else [H, K, N].  Any sizes; one output per thread.
 template <typename T, bool NK>
 __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ x, long long x_t, long long x_h, const T* __restrict__ w,
-                                                          T* __restrict__ y, long long y_t, long long y_h, int N, int K) {
+                                                          T* __restrict__ y, long long y_t, long long y_h, int N, int K,
+                                                          const T* __restrict__ gate, long long gate_ld) {
   extern __shared__ float xs[];
   pdl_trigger();
   pdl_wait();
@@ -108,30 +110,31 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
   const T* wh = w + static_cast<long long>(h) * N * K + (NK ? static_cast<long long>(n) * K : n);
   float s = 0.f;
   for (int k = 0; k < K; ++k) s = fmaf(xs[k], to_f(wh[NK ? k : static_cast<long long>(k) * N]), s);
+  if (gate != nullptr) s *= sigmoid_t<T>(to_f(gate[t * gate_ld + h * N + n]));
   y[t * y_t + h * y_h + n] = from_f<T>(s);
 }
 
 template <typename T>
-static int prep(const T* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
+static int prep(const T* q, long long q_ld, const T* kv, long long kv_ld, const int* positions, const long long* slots, const double* freq, float magnitude,
                 const T* kv_norm, float eps, T* cache, T* q_abs, T* q_full, int n, int t_long, int q_nope, int q_width, MbLatent L,
                 cudaStream_t s) {
   if (L.rot > 4096 || L.rot % 2) return -3;
   const int v = 16 / static_cast<int>(sizeof(T));
-  const bool vec = ld % v == 0 && L.dim % v == 0 && L.rot % v == 0 && q_nope % v == 0 && q_width % v == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0;
+  const bool vec = q_ld % v == 0 && L.dim % v == 0 && L.rot % v == 0 && q_nope % v == 0 && q_width % v == 0 && reinterpret_cast<uintptr_t>(q) % 16 == 0;
   const dim3 grid(n, kv_norm != nullptr ? 2 : 1);
   auto kern = vec ? latent_prep_kernel<T, true> : latent_prep_kernel<T, false>;
-  return static_cast<int>(launch_pdl(kern, grid, dim3(256), L.rot * sizeof(float), s, proj, ld, positions, slots, freq, magnitude, kv_norm, eps,
+  return static_cast<int>(launch_pdl(kern, grid, dim3(256), L.rot * sizeof(float), s, q, q_ld, kv, kv_ld, positions, slots, freq, magnitude, kv_norm, eps,
                                      cache, q_abs, q_full, t_long, q_nope, q_width, L));
 }
 
 template <typename T>
 static int head_linear(const T* x, long long x_t, long long x_h, const T* w, int nk, T* y, long long y_t, long long y_h, int n, int H, int N,
-                       int K, cudaStream_t s) {
+                       int K, const T* gate, long long gate_ld, cudaStream_t s) {
   if (K > 8192) return -3;
   for (int t0 = 0; t0 < n; t0 += 65535) {
     const dim3 grid((N + 127) / 128, H, n - t0 < 65535 ? n - t0 : 65535);
-    const cudaError_t e = nk ? launch_pdl(head_linear_kernel<T, true>, grid, dim3(128), K * sizeof(float), s, x + t0 * x_t, x_t, x_h, w, y + t0 * y_t, y_t, y_h, N, K)
-                             : launch_pdl(head_linear_kernel<T, false>, grid, dim3(128), K * sizeof(float), s, x + t0 * x_t, x_t, x_h, w, y + t0 * y_t, y_t, y_h, N, K);
+    const cudaError_t e = launch_pdl(nk ? head_linear_kernel<T, true> : head_linear_kernel<T, false>, grid, dim3(128), K * sizeof(float), s, x + t0 * x_t, x_t,
+                                     x_h, w, y + t0 * y_t, y_t, y_h, N, K, gate != nullptr ? gate + t0 * gate_ld : gate, gate_ld);
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   return 0;
@@ -148,19 +151,19 @@ using namespace mb::mx;
   using E = bf16;                                 \
   return call
 
-extern "C" int mb_latent_prep(const void* proj, long long ld, const int* positions, const long long* slots, const double* freq,
+extern "C" int mb_latent_prep(const void* q, long long q_ld, const void* kv, long long kv_ld, const int* positions, const long long* slots, const double* freq,
                               float magnitude, const void* kv_norm, float eps, void* cache, void* q_abs, void* q_full, int T, int t_long,
                               int q_nope, int q_width, MbLatent L, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
-  MB_BY_TYPE(prep(reinterpret_cast<const E*>(proj), ld, positions, slots, freq, magnitude, reinterpret_cast<const E*>(kv_norm), eps,
+  MB_BY_TYPE(prep(reinterpret_cast<const E*>(q), q_ld, reinterpret_cast<const E*>(kv), kv_ld, positions, slots, freq, magnitude, reinterpret_cast<const E*>(kv_norm), eps,
                   reinterpret_cast<E*>(cache), reinterpret_cast<E*>(q_abs), reinterpret_cast<E*>(q_full), T, t_long, q_nope, q_width, L, s));
 }
 
 extern "C" int mb_head_linear(const void* x, long long x_t, long long x_h, const void* w, int w_nk, void* y, long long y_t, long long y_h,
-                              int T, int H, int N, int K, int f32, cudaStream_t s) {
+                              int T, int H, int N, int K, const void* gate, long long gate_ld, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
   MB_BY_TYPE(head_linear(reinterpret_cast<const E*>(x), x_t, x_h, reinterpret_cast<const E*>(w), w_nk, reinterpret_cast<E*>(y), y_t, y_h, T, H,
-                         N, K, s));
+                         N, K, reinterpret_cast<const E*>(gate), gate_ld, s));
 }
 
 // the absorbed form on the any-size kernel: one "key head" whose keys are the cached rows and whose values are their latent part
@@ -175,5 +178,5 @@ extern "C" int mb_latent_attend(const void* q, const void* cache, const int* blo
   a.o_row = static_cast<long long>(L.heads) * L.rank;
   a.window = window;
   a.scale = scale;
-  return mb_paged_attend(q, cache, cache, block_table, max_blocks, block_size, token_seq, positions, slots, sink, out, T, a, f32, 0, s);
+  return mb_paged_attend(q, cache, cache, block_table, max_blocks, block_size, token_seq, positions, slots, sink, out, T, a, MbScores{}, f32, 0, s);
 }

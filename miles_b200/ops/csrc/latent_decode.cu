@@ -63,7 +63,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* __restri
 template <bool NK, int NW>
 __global__ void __launch_bounds__(128) head_linear_mma_kernel(const bf16* __restrict__ x, long long x_t, long long x_h,
                                                               const bf16* __restrict__ w, bf16* __restrict__ y, long long y_t, long long y_h,
-                                                              int T, int N, int K) {
+                                                              int T, int N, int K, const bf16* __restrict__ gate, long long gate_ld) {
   constexpr int TN = 32 * NW, S = NW == 2 ? 2 : 3, XP = 72, WP = NK ? 72 : TN + 8, WR = NK ? TN : 64;
   __shared__ __align__(16) bf16 sx[S][64 * XP];
   __shared__ __align__(16) bf16 sw[S][WR * WP];
@@ -143,6 +143,11 @@ __global__ void __launch_bounds__(128) head_linear_mma_kernel(const bf16* __rest
         const int t = m * 16 + half * 8 + (lane >> 2), n = n0 + warp * 8 * NW + nw * 8 + (lane & 3) * 2;
         if (t < nt && n < N) {                  // N is even
           bf16* dst = y + (t0 + t) * y_t + h * y_h + n;
+          if (gate != nullptr) {
+            const bf16* g = gate + (t0 + t) * gate_ld + h * N + n;
+            acc[m][nw][half * 2] *= mx::sigmoid_t<bf16>(__bfloat162float(g[0]));
+            acc[m][nw][half * 2 + 1] *= mx::sigmoid_t<bf16>(__bfloat162float(g[1]));
+          }
           *reinterpret_cast<uint32_t*>(dst) = pack2(acc[m][nw][half * 2], acc[m][nw][half * 2 + 1]);
         }
       }
@@ -413,7 +418,7 @@ extern "C" int mb_latent_gather(const void* cache, const int* block_table, int m
 
 // bf16, K % 8 == 0, N % 8 == 0, 16-byte aligned rows of x
 extern "C" int mb_head_linear_mma(const void* x, long long x_t, long long x_h, const void* w, int w_nk, void* y, long long y_t, long long y_h, int T,
-                                  int H, int N, int K, cudaStream_t s) {
+                                  int H, int N, int K, const void* gate, long long gate_ld, cudaStream_t s) {
   if (T <= 0) return 0;
   if (K % 8 || N % 8 || x_t % 8 || x_h % 8 || y_t % 2 || y_h % 2) return -3;
   const int zt = (T + 63) / 64;
@@ -422,11 +427,9 @@ extern "C" int mb_head_linear_mma(const void* x, long long x_t, long long x_h, c
   auto X = reinterpret_cast<const bf16*>(x);
   auto W = reinterpret_cast<const bf16*>(w);
   auto Y = reinterpret_cast<bf16*>(y);
-  cudaError_t e;
-  if (w_nk) e = wide ? launch_pdl(head_linear_mma_kernel<true, 2>, grid, dim3(128), 0, s, X, x_t, x_h, W, Y, y_t, y_h, T, N, K)
-                     : launch_pdl(head_linear_mma_kernel<true, 1>, grid, dim3(128), 0, s, X, x_t, x_h, W, Y, y_t, y_h, T, N, K);
-  else e = wide ? launch_pdl(head_linear_mma_kernel<false, 2>, grid, dim3(128), 0, s, X, x_t, x_h, W, Y, y_t, y_h, T, N, K)
-                : launch_pdl(head_linear_mma_kernel<false, 1>, grid, dim3(128), 0, s, X, x_t, x_h, W, Y, y_t, y_h, T, N, K);
+  auto kern = w_nk ? (wide ? head_linear_mma_kernel<true, 2> : head_linear_mma_kernel<true, 1>)
+                   : (wide ? head_linear_mma_kernel<false, 2> : head_linear_mma_kernel<false, 1>);
+  const cudaError_t e = launch_pdl(kern, grid, dim3(128), 0, s, X, x_t, x_h, W, Y, y_t, y_h, T, N, K, reinterpret_cast<const bf16*>(gate), gate_ld);
   return static_cast<int>(e);
 }
 

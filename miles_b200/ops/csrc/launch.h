@@ -209,17 +209,28 @@ int mb_multi_mxfp8(const long long* table, const long long* prefix, int n, long 
 // xb (the copy in the model's dtype) may be null; freq [D / 2 up] (optional): sines and cosines of positions · freq are added
 int mb_bigram_embedding(const int* tok, const int* prev, const void* embed, const void* table, long long buckets, long long mul_prev,
                         long long mul_cur, const int* positions, const double* freq, float* x, void* xb, int T, int D, int f32, cudaStream_t s);
-int mb_output_norm(float* x, const void* y, const void* nw, const void* ls, const void* fw, void* xb, int T, int D, float eps, int f32,
-                   cudaStream_t s);
+// x += mult · y / rms(y) · nw · ls (ls null: 1); xb = x, or with fw x / rms(x) · fw · gain
+int mb_output_norm(float* x, const void* y, const void* nw, const void* ls, float mult, const void* fw, float gain, void* xb, int T, int D,
+                   float eps, int f32, cudaStream_t s);
+// out = z²·softplus(act[0]) + z/2 for z > 0, (½ + softplus(act[1]))·(exp(z) − 1 − z) + z/2 else (n values)
+int mb_xielu(const void* z, const void* act, void* out, long long n, int f32, cudaStream_t s);
+// out[t, i] = gelu(z[t, i]) · table[tok[t], col + i] (tanh form), n columns
+int mb_gelu_rows(const void* z, long long ld, const int* tok, const void* table, long long table_ld, int col, void* out, int T, int n, int f32,
+                 cudaStream_t s);
+// x ← cap · tanh(x / cap); exact: in double precision
+int mb_softcap(float* x, long long n, float cap, int exact, cudaStream_t s);
+// out = o / rms(o) · w · sigmoid(gate), every head of V channels by itself (w [V], gate [T, H·V] rows of gate_ld)
+int mb_head_gated_norm(const void* o, const void* w, const void* gate, long long gate_ld, void* out, long long T, int H, int V, float eps, int f32,
+                       cudaStream_t s);
 // rows (optional, device): rows in use
 int mb_clamped_glu(const void* in, long long ld_in, void* out, long long ld_out, long long T, int F, float limit, float alpha, float shift,
                    const int* rows, int f32, cudaStream_t s);
 // x ← max(x, 0)² (n values a row, rows of them or as many as the device count says)
 int mb_relu_square(void* x, long long T, int n, const int* rows, int f32, cudaStream_t s);
 // out = x / rms(x) · w, each of `parts` equal parts of a row by its own root mean square
-int mb_part_norm(const void* x, const void* w, void* out, int T, int C, int parts, float eps, int f32, cudaStream_t s);
-// s = x + y1·s1 + y2·s2 + s2·Σ_j weights[t, j]·rows[dst[t, j]] + extra → to; h = rmsnorm(s)·(nw + shift)·gain, h2 the same with nw2 (every
-// pointer but x may be null; a null scale is 1; at most one of y2 and rows where s2 is given)
+int mb_part_norm(const void* x, long long ld, const void* w, void* out, int T, int C, int parts, float eps, int f32, cudaStream_t s);
+// s = x + mult·(y1·s1 + y2·s2 + s2·Σ_j weights[t, j]·rows[dst[t, j]]) + extra → to; h = rmsnorm(s)·(nw + shift)·gain (nw null: s), h2 the
+// same with nw2 (every pointer but x may be null; a null scale is 1; at most one of y2 and rows where s2 is given)
 typedef struct {
   const float* x;
   float* to;
@@ -231,14 +242,14 @@ typedef struct {
   const void *nw, *nw2;
   void *h, *h2;
   int T, D, k;
-  float eps, shift, gain;
+  float eps, shift, gain, mult;
 } MbSumNorm;
 int mb_sum_norm(MbSumNorm p, int f32, cudaStream_t s);
 int mb_gated_norm(const void* o, const void* w, const void* gate, long long gate_ld, void* out, int T, int C, float eps, int f32,
                   cudaStream_t s);
 // gemv.cu: output norm + layer scale + fp32 residual in front of a projection of ≤ 16 rows
-int mb_gemv_output_norm(const float* x, const void* y, const void* norm_w, const void* scale_w, float eps, const void* W, void* out,
-                        long long ldo, float* x_out, int M, int N, int K, int static_w, cudaStream_t s);
+int mb_gemv_output_norm(const float* x, const void* y, const void* norm_w, const void* scale_w, float mult, const void* next_w, float eps,
+                        const void* W, void* out, long long ldo, float* x_out, int M, int N, int K, int static_w, cudaStream_t s);
 // gemv.cu: sum of an fp32 residual and up to two sublayer outputs (each times a scale vector, if given), its norm, and up to two products of
 // it, for ≤ 16 rows.  x32 null: plain products of x [M, K].  W2 [N2, K] gives out2 (+ bias2), fp32 or bf16; with norm_w2 its rows are the sum
 // normed by that weight.  Norm weights count from `shift`.  xn_out: the normed sum (by norm_w2 if there is one).
@@ -248,7 +259,7 @@ typedef struct {
   const float* extra;
   const void* x;
   const void *norm_w, *norm_w2;
-  float eps, shift;
+  float eps, shift, mult;                    // mult: factor on the addends; norm_w null: the sum as it is
   const void* W;
   void* y;
   long long ldy;
@@ -261,20 +272,28 @@ typedef struct {
   int M, N, N2, K, static_w;
 } MbGemvSum;
 int mb_gemv_sum_norm(MbGemvSum a, cudaStream_t s);
+// ---- what attention kernels do to scores and outputs besides scale and softmax (null: nothing) ----
+typedef struct {
+  const void *r1, *r2;                       // [heads]: r1 · ln(1 + r2 · distance) off the scores
+  const void* gate;                          // [T, heads·vdim] rows of gate_ld: outputs times its sigmoid
+  long long gate_ld;
+} MbScores;
 // ---- paged_attend.cu ----
 typedef struct {
   int heads, group, dk, dv;                  // query head h uses key head h / group
   long long q_row, q_head, k_row, k_head, v_row, v_head, o_row;   // strides in elements: token (slot) and head
   int window, keep;                          // keys a token sees (0: all), first keys that stay visible
+  int chunk;                                 // tokens see their own chunk of this many positions (0: no chunks; without a window)
   float scale;
 } MbAttend;
 // out_f32: rows of floats whatever the dtype of the rest
 int mb_paged_attend(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size,
                     const int* token_seq, const int* positions, const long long* slots, const void* sink, void* out, int T, MbAttend A,
-                    int f32, int out_f32, cudaStream_t s);
+                    MbScores x, int f32, int out_f32, cudaStream_t s);
 // ---- window_prep.cu ----
 typedef struct {
   int heads, kv_heads, dim, vdim, rot, window, keep, q_pitch;   // q_pitch: elements per head of the prepared queries (zero-padded)
+  int chunk;                                                    // as in MbAttend
 } MbWindow;
 typedef struct {                             // what reads the same projection beside the attention (null: nothing)
   const float* logits;
@@ -292,9 +311,10 @@ typedef struct {                             // what reads the same projection b
   float scale;
   const void* correction;
 } MbAside;
+// kc, vc null: the layer reads another's keys and values, its projection has none.  v_norm: values over their root mean square per head.
 int mb_window_prep(const void* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
-                   const void* q_norm, const void* k_norm, float eps, void* kc, void* vc, void* q, int T, MbWindow L, MbAside a, int f32,
-                   cudaStream_t s);
+                   const void* q_norm, const void* k_norm, int v_norm, float eps, void* kc, void* vc, void* q, int T, MbWindow L, MbAside a,
+                   int f32, cudaStream_t s);
 // ---- diff_prep.cu (differential attention: two score maps per head over the same values) ----
 // Query heads 2h and 2h + 1 are the maps of head h; a key head is [map 1 | map 2], a query row has zeros in the other map's half, so that
 // the attention kernels see heads = 2·(query heads) of dim = 2·(map size).  What is left of a pair of outputs a1, a2:
@@ -316,6 +336,37 @@ int mb_diff_prep(const void* proj, long long ld, const int* positions, const lon
                  const void* lvec, float* lam, void* kc, void* vc, void* q, int T, MbDiffPrep L, MbAside a, int f32, cudaStream_t s);
 // a [T, 2·heads, vdim] floats → out [T, heads·vdim] rows of o_row
 int mb_diff_combine(const float* a, void* out, long long o_row, int T, int heads, int vdim, MbDiff d, int f32, cudaStream_t s);
+// ---- short_conv.cuh ----
+typedef struct {
+  int at, channels, taps;                    // first column of the inputs in a row of the projection
+  const void *w, *b;                         // [channels, taps], [channels] (null: no bias)
+  float* ring;                               // [slots, taps, channels]: the inputs of the last positions, by position mod taps (null: taps 1)
+  const int* slots;                          // per sequence
+  const int* positions;                      // per token
+} MbConv;
+// ---- delta_*.cu (gated delta rule: S ← diag(g)·S, S ← S + k (β (v − Sᵀk))ᵀ, o = Sᵀq) ----
+// A row of the projection is [q: G·K | k: G·K | v: H·V | … | β: H at column beta_at]; q, k and v pass a causal convolution and silu, then q
+// and k become unit vectors (q over √K on top).  g = exp(−exp(A_log)·softplus(raw + dt_bias)), raw [T, H·K] rows of raw_ld.
+typedef struct {
+  int H, G, K, V, taps, beta_at;
+  const void* conv_w;                        // [2·G·K + H·V, taps]
+  const void *A_log, *dt_bias;               // [H], [H·K]
+  float* state;                              // [slots, H, K, V]
+  float* ring;                               // as in MbConv
+  const int* slots;
+  const int* positions;
+  const void* raw;
+  long long raw_ld;
+} MbDelta;
+// Convolution of any pieces (tiles as in mb_ssm_conv): act [T, channels].
+int mb_delta_conv(const void* proj, long long ld, MbDelta m, const int* tiles, const int* cu_q, int n_tiles, void* act, int f32, cudaStream_t s);
+// Any pieces token by token from the convolution's outputs (cu_q null: one token per sequence); out [T, H·V] = o.
+int mb_delta_seq(const void* proj, long long ld, const void* act, MbDelta m, const int* cu_q, void* out, int B, int f32, cudaStream_t s);
+// One token per sequence in one launch: convolution, state, and o over its root mean square per head, times norm_w [V] and sigmoid(gate).
+// V % 4 == 0, V ≤ 1024, K·V ≤ mb_delta_step_max().
+int mb_delta_step(const void* proj, long long ld, MbDelta m, const void* norm_w, const void* gate, long long gate_ld, float eps, void* out, int B,
+                  int f32, cudaStream_t s);
+int mb_delta_step_max(void);
 // ---- ssm_*.cu (state-space mixer: S ← exp(−exp(A_log)·dt)·S + dt·B xᵀ, y = Sᵀ C + D·x) ----
 // A row of the projection is [z: H·V | x: H·V | B: G·N | C: G·N | dt: H]; x, B and C pass a causal convolution of `taps` columns and silu.
 typedef struct {
@@ -344,11 +395,11 @@ int mb_ssm_heads_per_cta(int H, int V, int G);
 // ---- window_decode.cu (bf16 tensor cores, splits joined inside a cluster) ----
 int mb_window_decode(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                      const int* positions, const long long* slots, const void* sink, void* out, long long o_row, int T, float scale, int splits,
-                     MbWindow L, MbDiff d, cudaStream_t s);
+                     MbWindow L, MbDiff d, MbScores x, cudaStream_t s);
 // ---- attention_window_tc.cu (tcgen05, keys and values straight from the pages) ----
 int mb_window_prefill(const void* q, const void* kc, const void* vc, void* o, long long o_row, const void* sink, const int* cu_q,
                       const int* positions, const int* block_table, int max_blocks, int block_size, int num_blocks, int n_seq, int max_q,
-                      int t_long, float scale, MbWindow L, MbDiff d, int* error_flag, cudaStream_t s);
+                      int t_long, float scale, MbWindow L, MbDiff d, MbScores x, int* error_flag, cudaStream_t s);
 // ---- experts_any.cu ----
 // alpha 0: w13 is [E, F, H] (no gate), the activation the square of relu
 int mb_experts_any(const void* x, const void* w13, const void* w2, const int* index, const float* weights, void* act, void* out, int T, int k,
@@ -357,11 +408,13 @@ int mb_experts_any(const void* x, const void* w13, const void* w2, const int* in
 typedef struct {
   int heads, dim, rot, vdim, rank, rank_p, pitch;   // a cached row: [rank, 0 … rank_p, rot, 0 … pitch)
 } MbLatent;
-int mb_latent_prep(const void* proj, long long ld, const int* positions, const long long* slots, const double* freq, float magnitude,
-                   const void* kv_norm, float eps, void* cache, void* q_abs, void* q_full, int T, int t_long, int q_nope, int q_width,
-                   MbLatent L, int f32, cudaStream_t s);
+// q [T, heads·(dim + rot)] rows of q_ld, kv [T, rank + rot] rows of kv_ld (read with kv_norm)
+int mb_latent_prep(const void* q, long long q_ld, const void* kv, long long kv_ld, const int* positions, const long long* slots, const double* freq,
+                   float magnitude, const void* kv_norm, float eps, void* cache, void* q_abs, void* q_full, int T, int t_long, int q_nope,
+                   int q_width, MbLatent L, int f32, cudaStream_t s);
+// gate (optional): y times the sigmoid of gate[t·gate_ld + h·N + n]
 int mb_head_linear(const void* x, long long x_t, long long x_h, const void* w, int w_nk, void* y, long long y_t, long long y_h, int T,
-                   int H, int N, int K, int f32, cudaStream_t s);
+                   int H, int N, int K, const void* gate, long long gate_ld, int f32, cudaStream_t s);
 int mb_latent_attend(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                      const int* positions, const long long* slots, const void* sink, void* out, int T, float scale, int window, MbLatent L,
                      int f32, cudaStream_t s);
@@ -369,7 +422,7 @@ int mb_latent_attend(const void* q, const void* cache, const int* block_table, i
 int mb_latent_gather(const void* cache, const int* block_table, int max_blocks, int block_size, const int* cu_k, const int* base, void* out,
                      int n_seq, int total, int pitch, cudaStream_t s);
 int mb_head_linear_mma(const void* x, long long x_t, long long x_h, const void* w, int w_nk, void* y, long long y_t, long long y_h, int T,
-                       int H, int N, int K, cudaStream_t s);
+                       int H, int N, int K, const void* gate, long long gate_ld, cudaStream_t s);
 int mb_latent_decode(const void* q, const void* cache, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                      const int* positions, const long long* slots, const void* sink, float* part_o, float* part_ml, void* out, int T,
                      float scale, int window, int splits, int num_blocks, MbLatent L, int* error_flag, cudaStream_t s);
@@ -378,8 +431,9 @@ int mb_latent_decode_tc(const void* q, const void* cache, const int* block_table
                         const int* positions, const long long* slots, float* part_o, float* part_ml, int T, float scale, int window,
                         int splits, int num_blocks, MbLatent L, int* error_flag, cudaStream_t s);
 // ---- attention_latent_tc.cu (tcgen05) ----
-int mb_latent_prefill(const void* q, const void* kv, const void* lat, void* o, const void* sink, const int* cu_q, const int* cu_k, int n_seq,
-                      int max_q, int t_long, int tk, float scale, int window, MbLatent L, int* error_flag, cudaStream_t s);
+int mb_latent_prefill(const void* q, const void* kv, const void* lat, void* o, const void* sink, const void* gate, long long gate_ld, const int* cu_q,
+                      const int* cu_k, int n_seq, int max_q, int t_long, int tk, float scale, int window, MbLatent L, int* error_flag,
+                      cudaStream_t s);
 // ---- linear_state.cu ----
 int mb_linear_state(const void* proj, long long ld, const float* decay, float* state, const int* state_slots, const int* cu_q,
                     const int* positions, void* out, int B, int H, int dk, int dv, int f32, cudaStream_t s);

@@ -1,6 +1,7 @@
 // Row-wise kernels of the layer-by-layer decoders: hashed-bigram embedding, output norm + layer scale + fp32 residual (with the
 // model's final norm fused into the last one), sum of fp32 residual and sublayer outputs (experts' rows gathered and weighted on the
-// way) with the next norm, clamped gated activation, gated norm over all heads of a mixer.
+// way) with the next norm, clamped gated activation, xIELU, gated token rows, gated norm over all heads of a mixer or each by itself,
+// soft cap of logits.
 // fp32 math; activations in the model's dtype T (bf16, or float for 32-bit runs).
 #include <type_traits>
 
@@ -51,11 +52,11 @@ __global__ void __launch_bounds__(128) bigram_embed_kernel(const int* __restrict
   }
 }
 
-// x += y / rms(y) · nw · ls;  xb = x, or x / rms(x) · fw with the model's final norm
+// x += mult · y / rms(y) · nw · ls (ls null: 1);  xb = x, or x / rms(x) · fw · gain (the next norm, or the model's final one)
 template <typename T, int V>
 __global__ void __launch_bounds__(kRow) output_norm_kernel(float* __restrict__ x, const T* __restrict__ y, const T* __restrict__ nw,
-                                                           const T* __restrict__ ls, const T* __restrict__ fw, T* __restrict__ xb, int D,
-                                                           float eps) {
+                                                           const T* __restrict__ ls, float mult, const T* __restrict__ fw, float gain,
+                                                           T* __restrict__ xb, int D, float eps) {
   __shared__ float sh[kRow / 32];
   pdl_trigger();
   pdl_wait();
@@ -67,13 +68,15 @@ __global__ void __launch_bounds__(kRow) output_norm_kernel(float* __restrict__ x
 #pragma unroll
     for (int j = 0; j < V; ++j) ss += a[j] * a[j];
   }
-  const float rstd = rsqrt_exact(__fdiv_rn(block_sum<kRow>(ss, sh), static_cast<float>(D)) + eps);
+  const float rstd = mult * rsqrt_exact(__fdiv_rn(block_sum<kRow>(ss, sh), static_cast<float>(D)) + eps);
   ss = 0.f;
   for (int i = threadIdx.x * V; i < D; i += kRow * V) {
     float a[V], w[V], l[V], r[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) l[j] = 1.f;
     load_n<V>(y + base + i, a);
     load_n<V>(nw + i, w);
-    load_n<V>(ls + i, l);
+    if (ls != nullptr) load_n<V>(ls + i, l);
     load_n<V>(x + base + i, r);
 #pragma unroll
     for (int j = 0; j < V; ++j) {
@@ -90,7 +93,7 @@ __global__ void __launch_bounds__(kRow) output_norm_kernel(float* __restrict__ x
     load_n<V>(fw + i, w);
     load_n<V>(x + base + i, r);
 #pragma unroll
-    for (int j = 0; j < V; ++j) r[j] = r[j] * rs2 * w[j];
+    for (int j = 0; j < V; ++j) r[j] = r[j] * rs2 * w[j] * gain;
     store_n<V>(xb + base + i, r);
   }
 }
@@ -164,6 +167,8 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
     for (int j = 0; j < V; ++j) c1[j] = c2[j] = 1.f;
     if (SCALED && s1 != nullptr) load_n<V>(s1 + i, c1);
     if (SCALED && s2 != nullptr) load_n<V>(s2 + i, c2);
+#pragma unroll
+    for (int j = 0; j < V; ++j) { c1[j] *= p.mult; c2[j] *= p.mult; }
     load_n<V>(p.x + base + i, r);
     if (y1 != nullptr) {
       load_n<V>(y1 + base + i, a);
@@ -197,7 +202,10 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
       for (int j = 0; j < V; ++j) r[j] += a[j];
     }
     if (p.to != nullptr) store_n<V>(p.to + base + i, r);
-    if (nw == nullptr) continue;
+    if (nw == nullptr) {
+      if (h != nullptr) store_n<V>(h + base + i, r);
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < V; ++j) ss += r[j] * r[j];
     store_n<V>(row + i, r);
@@ -222,16 +230,17 @@ __global__ void __launch_bounds__(kRow) sum_norm_kernel(MbSumNorm p) {
   }
 }
 
-// out = x / rms(x) · w for every one of `parts` equal parts of a row; grid (rows, parts)
+// out = x / rms(x) · w for every one of `parts` equal parts of a row (of x: ld elements apart); grid (rows, parts)
 template <typename T, int V>
-__global__ void __launch_bounds__(kRow) part_norm_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict__ out, int n, int parts,
-                                                         float eps) {
+__global__ void __launch_bounds__(kRow) part_norm_kernel(const T* __restrict__ xs, long long ld, const T* __restrict__ w, T* __restrict__ out, int n,
+                                                         int parts, float eps) {
   __shared__ float sh[kRow / 32];
   constexpr int kHold = 4;                 // vectors per thread that stay in registers between the two passes
   pdl_trigger();
   pdl_wait();
   const long long base = (static_cast<long long>(blockIdx.x) * parts + blockIdx.y) * n;
   const T* pw = w + static_cast<long long>(blockIdx.y) * n;
+  const T* x = xs + blockIdx.x * ld + static_cast<long long>(blockIdx.y) * n - base;
   float a[kHold][V], ss = 0.f;
 #pragma unroll
   for (int u = 0; u < kHold; ++u) {
@@ -297,6 +306,96 @@ __global__ void __launch_bounds__(kRow) gated_norm_kernel(const T* __restrict__ 
   }
 }
 
+// out = o / rms(o) · w · sigmoid(gate), every head's V channels by themselves: `lanes` (a power of two up to 32) threads a head
+template <typename T, int N>
+__global__ void __launch_bounds__(256) head_gated_norm_kernel(const T* __restrict__ o, const T* __restrict__ w, const T* __restrict__ gate,
+                                                              long long gate_ld, T* __restrict__ out, long long heads, int H, int V, int lanes,
+                                                              float eps) {
+  pdl_trigger();
+  pdl_wait();
+  const long long hd = (blockIdx.x * 256ll + threadIdx.x) / lanes;      // head of all tokens
+  const int l = threadIdx.x & (lanes - 1);
+  const bool on = hd < heads;
+  const long long base = hd * V;
+  const T* g = gate + (hd / H) * gate_ld + (hd % H) * V;
+  float ss = 0.f, a[N], first[N];
+  for (int i = l * N; on && i < V; i += lanes * N) {
+    load_n<N>(o + base + i, a);
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+      ss += a[j] * a[j];
+      if (i == l * N) first[j] = a[j];
+    }
+  }
+  for (int x = lanes / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+  if (!on) return;
+  const float rstd = rsqrt_exact(__fdiv_rn(ss, static_cast<float>(V)) + eps);
+  for (int i = l * N; i < V; i += lanes * N) {
+    float b[N], c[N];
+    if (i == l * N) {
+#pragma unroll
+      for (int j = 0; j < N; ++j) a[j] = first[j];
+    } else {
+      load_n<N>(o + base + i, a);
+    }
+    load_n<N>(w + i, b);
+    load_n<N>(g + i, c);
+#pragma unroll
+    for (int j = 0; j < N; ++j) a[j] = a[j] * rstd * b[j] * sigmoid_t<T>(c[j]);
+    store_n<N>(out + base + i, a);
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) xielu_kernel(const T* __restrict__ z, const T* __restrict__ act, T* __restrict__ out, long long n) {
+  pdl_trigger();
+  pdl_wait();
+  const float pos = softplus_t<T>(to_f(act[0])), neg = 0.5f + softplus_t<T>(to_f(act[1]));
+  for (long long i = (blockIdx.x * 256ll + threadIdx.x) * V; i < n; i += gridDim.x * 256ll * V) {
+    float a[V];
+    load_n<V>(z + i, a);
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] = fmaf(0.5f, a[j], a[j] > 0.f ? pos * a[j] * a[j] : neg * (expm1f(a[j]) - a[j]));
+    store_n<V>(out + i, a);
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) gelu_rows_kernel(const T* __restrict__ z, long long ld, const int* __restrict__ tok, const T* __restrict__ table,
+                                                        long long table_ld, int col, T* __restrict__ out, long long rows, int n) {
+  pdl_trigger();
+  pdl_wait();
+  const int per = n / V;
+  for (long long v = blockIdx.x * 256ll + threadIdx.x; v < rows * per; v += gridDim.x * 256ll) {
+    const long long t = v / per;
+    const int i = static_cast<int>(v - t * per) * V;
+    float a[V], e[V];
+    load_n<V>(z + t * ld + i, a);
+    load_n<V>(table + tok[t] * table_ld + col + i, e);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {      // ½ (1 + tanh u) = sigmoid(2u)
+      const float u = 0.7978845608028654f * (a[j] + 0.044715f * a[j] * a[j] * a[j]);
+      a[j] = a[j] * sigmoid_t<T>(2.f * u) * e[j];
+    }
+    store_n<V>(out + t * n + i, a);
+  }
+}
+
+template <bool EXACT>
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long long n, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  const float inv = __fdiv_rn(1.f, cap);
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
+    if (EXACT) {
+      x[i] = static_cast<float>(cap * tanh(static_cast<double>(x[i]) / cap));
+    } else {                           // tanh u = 1 − 2 / (exp(2u) + 1), odd: exponentials of −2|u| never overflow
+      const float u = x[i] * inv, e = __expf(-2.f * fabsf(u));
+      x[i] = copysignf(cap * __fdividef(1.f - e, 1.f + e), u);
+    }
+  }
+}
+
 // 16-byte accesses need element counts (and strides) that are whole vectors
 template <typename F>
 static int dispatch(int f32, bool vec, F&& f) {
@@ -322,13 +421,13 @@ extern "C" int mb_bigram_embedding(const int* tok, const int* prev, const void* 
   });
 }
 
-extern "C" int mb_output_norm(float* x, const void* y, const void* nw, const void* ls, const void* fw, void* xb, int T, int D, float eps,
-                              int f32, cudaStream_t s) {
+extern "C" int mb_output_norm(float* x, const void* y, const void* nw, const void* ls, float mult, const void* fw, float gain, void* xb, int T,
+                              int D, float eps, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
   return dispatch(f32, D % 8 == 0, [&](auto ty, auto v) {
     using E = decltype(ty);
     return static_cast<int>(launch_pdl(output_norm_kernel<E, decltype(v)::value>, dim3(T), dim3(kRow), 0, s, x, reinterpret_cast<const E*>(y),
-                                       reinterpret_cast<const E*>(nw), reinterpret_cast<const E*>(ls), reinterpret_cast<const E*>(fw),
+                                       reinterpret_cast<const E*>(nw), reinterpret_cast<const E*>(ls), mult, reinterpret_cast<const E*>(fw), gain,
                                        reinterpret_cast<E*>(xb), D, eps));
   });
 }
@@ -357,14 +456,65 @@ extern "C" int mb_relu_square(void* x, long long T, int n, const int* rows, int 
   });
 }
 
-extern "C" int mb_part_norm(const void* x, const void* w, void* out, int T, int C, int parts, float eps, int f32, cudaStream_t s) {
+static unsigned elementwise_blocks(long long pieces) {
+  const long long blocks = (pieces + 255) / 256;
+  return static_cast<unsigned>(blocks < 148 * 16 ? (blocks > 0 ? blocks : 1) : 148 * 16);
+}
+
+extern "C" int mb_xielu(const void* z, const void* act, void* out, long long n, int f32, cudaStream_t s) {
+  if (n <= 0) return 0;
+  return dispatch(f32, n % 8 == 0 && (reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) % 16 == 0, [&](auto ty, auto v) {
+    using E = decltype(ty);
+    constexpr int V = decltype(v)::value;
+    return static_cast<int>(launch_pdl(xielu_kernel<E, V>, dim3(elementwise_blocks(n / V)), dim3(256), 0, s, reinterpret_cast<const E*>(z),
+                                       reinterpret_cast<const E*>(act), reinterpret_cast<E*>(out), n));
+  });
+}
+
+extern "C" int mb_gelu_rows(const void* z, long long ld, const int* tok, const void* table, long long table_ld, int col, void* out, int T, int n, int f32,
+                            cudaStream_t s) {
+  if (T <= 0 || n <= 0) return 0;
+  const bool vec = n % 8 == 0 && ld % 8 == 0 && table_ld % 8 == 0 && col % 8 == 0 &&
+                   (reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(table)) % 16 == 0;
+  return dispatch(f32, vec, [&](auto ty, auto v) {
+    using E = decltype(ty);
+    constexpr int V = decltype(v)::value;
+    return static_cast<int>(launch_pdl(gelu_rows_kernel<E, V>, dim3(elementwise_blocks(static_cast<long long>(T) * (n / V))), dim3(256), 0, s,
+                                       reinterpret_cast<const E*>(z), ld, tok, reinterpret_cast<const E*>(table), table_ld, col,
+                                       reinterpret_cast<E*>(out), static_cast<long long>(T), n));
+  });
+}
+
+extern "C" int mb_softcap(float* x, long long n, float cap, int exact, cudaStream_t s) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return -3;
+  return static_cast<int>(launch_pdl(exact ? softcap_kernel<true> : softcap_kernel<false>, dim3(elementwise_blocks(n)), dim3(256), 0, s, x, n, cap));
+}
+
+extern "C" int mb_head_gated_norm(const void* o, const void* w, const void* gate, long long gate_ld, void* out, long long T, int H, int V, float eps, int f32,
+                                  cudaStream_t s) {
+  if (T <= 0) return 0;
+  const bool vec = V % 8 == 0 && gate_ld % 8 == 0 && (reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+  return dispatch(f32, vec, [&](auto ty, auto v) {
+    using E = decltype(ty);
+    constexpr int N = decltype(v)::value;
+    int lanes = 1;
+    while (lanes < 32 && lanes * N < V) lanes *= 2;
+    const long long threads = T * H * lanes;
+    return static_cast<int>(launch_pdl(head_gated_norm_kernel<E, N>, dim3(static_cast<unsigned>((threads + 255) / 256)), dim3(256), 0, s,
+                                       reinterpret_cast<const E*>(o), reinterpret_cast<const E*>(w), reinterpret_cast<const E*>(gate), gate_ld,
+                                       reinterpret_cast<E*>(out), T * H, H, V, lanes, eps));
+  });
+}
+
+extern "C" int mb_part_norm(const void* x, long long ld, const void* w, void* out, int T, int C, int parts, float eps, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
   if (parts <= 0 || C % parts || parts > 65535) return -3;
   const int n = C / parts;
-  return dispatch(f32, n % 8 == 0, [&](auto ty, auto v) {
+  return dispatch(f32, n % 8 == 0 && ld % 8 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0, [&](auto ty, auto v) {
     using E = decltype(ty);
     return static_cast<int>(launch_pdl(part_norm_kernel<E, decltype(v)::value>, dim3(T, parts), dim3(kRow), 0, s, reinterpret_cast<const E*>(x),
-                                       reinterpret_cast<const E*>(w), reinterpret_cast<E*>(out), n, parts, eps));
+                                       ld, reinterpret_cast<const E*>(w), reinterpret_cast<E*>(out), n, parts, eps));
   });
 }
 

@@ -37,6 +37,16 @@ template <typename T> __device__ __forceinline__ float sigmoid_t(float x) {
 template <typename T> __device__ __forceinline__ float silu_t(float x) { return x * sigmoid_t<T>(x); }
 __device__ __forceinline__ float rsqrt_exact(float x) { return __fdiv_rn(1.f, __fsqrt_rn(x)); }
 
+template <typename T> __device__ __forceinline__ float softplus_t(float x) {
+  if constexpr (is_exact<T>::value) {
+    const double d = x;
+    return static_cast<float>(d > 0. ? d + log1p(exp(-d)) : log1p(exp(d)));
+  } else {
+    const float e = __expf(-fabsf(x));
+    return fmaxf(x, 0.f) + log1pf(e);
+  }
+}
+
 // N consecutive values ↔ floats (N·sizeof(T) bytes, 16-byte aligned pieces)
 template <int N> __device__ __forceinline__ void load_n(const float* p, float (&f)[N]) {
   if constexpr (N % 4 == 0) {

@@ -6,6 +6,8 @@
 //   * the softmax weights enter P·V as two bf16 parts, 16 bits of mantissa.  R = 8: the eight rows that pad the tile carry the second
 //     part for no extra instruction, and the two halves of the accumulator are added at the end.  R = 16: two products;
 //   * the splits are joined through distributed shared memory, the sink enters there: one launch, no partial results in HBM;
+//   * a token may see its own chunk instead of a window; BIAS: r1 · ln(1 + r2 · distance) comes off the scores; outputs may pass a gate
+//     (MbScores);
 //   * differential attention (MbDiff): heads 2h and 2h + 1 are neighbours among the rows; a warp joins both, subtracts, norms and gates.
 // Heads narrower than DK / DV are padded with zeros in shared memory.
 #include <cooperative_groups.h>
@@ -37,12 +39,12 @@ struct Smem {
   static constexpr int bytes = o == k ? total : o + 4 * R * DV * 4;
 };
 
-template <int DK, int DV, int R>
+template <int DK, int DV, int R, bool BIAS>
 __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
                                                             const int* __restrict__ block_table, int max_blocks, int block_size,
                                                             const int* __restrict__ token_seq, const int* __restrict__ positions,
                                                             const long long* __restrict__ slots, const bf16* __restrict__ sink,
-                                                            bf16* __restrict__ out, long long o_row, float scale, MbWindow L, MbDiff D) {
+                                                            bf16* __restrict__ out, long long o_row, float scale, MbWindow L, MbDiff D, MbScores X) {
   using S = Smem<DK, DV, R>;
   extern __shared__ __align__(128) uint8_t smem[];
   bf16* sQ = reinterpret_cast<bf16*>(smem + S::q);
@@ -68,7 +70,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
     return;
   }
   const int pos = positions[t];
-  const int lo = L.window > 0 ? max(0, pos - L.window + 1) : 0, kept = min(L.keep, lo);
+  const int lo = L.window > 0 ? max(0, pos - L.window + 1) : L.chunk > 0 ? pos - pos % L.chunk : 0, kept = L.window > 0 ? min(L.keep, lo) : 0;
   const int n_keys = kept + pos + 1 - lo;
   const int per = ((n_keys + splits - 1) / splits + TK - 1) / TK * TK;   // keys per split, whole tiles
   const int k_begin = min(split * per, n_keys), k_end = min(n_keys, k_begin + per);
@@ -133,6 +135,13 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
 #pragma unroll
   for (int r = 0; r < RS; ++r) { m_i[r] = -INFINITY; l_i[r] = 0.f; }
   const float sl2 = scale * kLog2e;
+  float r1[RS], r2[RS];
+#pragma unroll
+  for (int r = 0; r < RS; ++r) {
+    const int row = (lane >> 2) + 8 * r;
+    r1[r] = BIAS && row < rows ? __bfloat162float(reinterpret_cast<const bf16*>(X.r1)[h0 + row]) : 0.f;
+    r2[r] = BIAS && row < rows ? __bfloat162float(reinterpret_cast<const bf16*>(X.r2)[h0 + row]) : 0.f;
+  }
 
   for (int tile = 0; tile < n_tiles; ++tile) {
     const int st = tile & 1;
@@ -164,7 +173,9 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            s[nt][2 * r + e] = key0 + nt * 8 + (lane & 3) * 2 + e < k_end ? s[nt][2 * r + e] * sl2 : -INFINITY;
+            const int i = key0 + nt * 8 + (lane & 3) * 2 + e;
+            s[nt][2 * r + e] = i < k_end ? s[nt][2 * r + e] * sl2 : -INFINITY;
+            if (BIAS) s[nt][2 * r + e] -= r1[r] * __log2f(fmaf(r2[r], static_cast<float>(max(pos - (i < kept ? i : lo + i - kept), 0)), 1.f));
             mx = fmaxf(mx, s[nt][2 * r + e]);
           }
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -294,33 +305,39 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const bf16* __restri
       den = fmaf(cluster.map_shared_rank(fM, c)[R + g], a, den);
       oo = fmaf(cluster.map_shared_rank(fO, c)[g * DV + d], a, oo);
     }
-    if (d < L.vdim) out[t * o_row + static_cast<long long>(h0 + g) * L.vdim + d] = __float2bfloat16(__fdiv_rn(oo, den));
+    if (d < L.vdim) {
+      const long long at = static_cast<long long>(h0 + g) * L.vdim + d;
+      float r = __fdiv_rn(oo, den);
+      if (X.gate != nullptr) r *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(reinterpret_cast<const bf16*>(X.gate)[t * X.gate_ld + at])));
+      out[t * o_row + at] = __float2bfloat16(r);
+    }
   }
   if (splits > 1) cluster.sync();        // the shared memory stays until the others have read it
 }
 
-template <int DK, int DV, int R>
+template <int DK, int DV, int R, bool BIAS>
 static int launch_rows(const bf16* q, const bf16* kc, const bf16* vc, const int* bt, int max_blocks, int bs, const int* seq, const int* pos,
                   const long long* slots, const bf16* sink, bf16* out, long long o_row, int T, float scale, int splits, MbWindow L, MbDiff d,
-                  cudaStream_t s) {
+                  MbScores x, cudaStream_t s) {
   static bool once = false;
   if (!once) {
-    const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<DK, DV, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<DK, DV, R>::bytes);
+    const cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<DK, DV, R, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<DK, DV, R>::bytes);
     if (e != cudaSuccess) return static_cast<int>(e);
     once = true;
   }
   const int chunks = (L.heads / L.kv_heads + R - 1) / R;
-  return static_cast<int>(launch_pdl_cluster(window_decode_kernel<DK, DV, R>, dim3(splits, L.kv_heads * chunks, T), dim3(128), splits,
-                                             Smem<DK, DV, R>::bytes, s, q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, scale, L, d));
+  return static_cast<int>(launch_pdl_cluster(window_decode_kernel<DK, DV, R, BIAS>, dim3(splits, L.kv_heads * chunks, T), dim3(128), splits,
+                                             Smem<DK, DV, R>::bytes, s, q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, scale, L, d, x));
 }
 
 // groups of more than 8 heads are read once for 16 of them
 template <int DK, int DV>
 static int launch(const bf16* q, const bf16* kc, const bf16* vc, const int* bt, int max_blocks, int bs, const int* seq, const int* pos,
                   const long long* slots, const bf16* sink, bf16* out, long long o_row, int T, float scale, int splits, MbWindow L, MbDiff d,
-                  cudaStream_t s) {
-  auto f = L.heads / L.kv_heads > 8 ? launch_rows<DK, DV, 16> : launch_rows<DK, DV, 8>;
-  return f(q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, T, scale, splits, L, d, s);
+                  MbScores x, cudaStream_t s) {
+  auto f = x.r1 != nullptr ? (L.heads / L.kv_heads > 8 ? launch_rows<DK, DV, 16, true> : launch_rows<DK, DV, 8, true>)
+                           : (L.heads / L.kv_heads > 8 ? launch_rows<DK, DV, 16, false> : launch_rows<DK, DV, 8, false>);
+  return f(q, kc, vc, bt, max_blocks, bs, seq, pos, slots, sink, out, o_row, T, scale, splits, L, d, x, s);
 }
 
 }  // namespace wd
@@ -332,13 +349,14 @@ using namespace mb;
 // 8 up to 128, splits ∈ 1 … 8, T ≤ 65535.
 extern "C" int mb_window_decode(const void* q, const void* kc, const void* vc, const int* block_table, int max_blocks, int block_size, const int* token_seq,
                                 const int* positions, const long long* slots, const void* sink, void* out, long long o_row, int T, float scale,
-                                int splits, MbWindow L, MbDiff d, cudaStream_t s) {
+                                int splits, MbWindow L, MbDiff d, MbScores x, cudaStream_t s) {
   if (T <= 0) return 0;
   if (L.dim % 8 || L.vdim % 8 || L.q_pitch % 8 || L.dim > 128 || L.vdim > 128 || L.heads % L.kv_heads || splits < 1 || splits > 8 || T > 65535) return -3;
-  if (d.lam != nullptr && (sink != nullptr || (L.heads / L.kv_heads) % 2)) return -3;
+  if (d.lam != nullptr && (sink != nullptr || (L.heads / L.kv_heads) % 2 || x.gate != nullptr)) return -3;
+  if ((L.chunk > 0 && L.window > 0) || (x.r1 != nullptr && sink != nullptr)) return -3;
   using wd::bf16;
   auto Q = reinterpret_cast<const bf16*>(q), K = reinterpret_cast<const bf16*>(kc), V = reinterpret_cast<const bf16*>(vc), SK = reinterpret_cast<const bf16*>(sink);
   auto O = reinterpret_cast<bf16*>(out);
   auto f = L.dim <= 64 ? (L.vdim <= 64 ? wd::launch<64, 64> : wd::launch<64, 128>) : (L.vdim <= 64 ? wd::launch<128, 64> : wd::launch<128, 128>);
-  return f(Q, K, V, block_table, max_blocks, block_size, token_seq, positions, slots, SK, O, o_row, T, scale, splits, L, d, s);
+  return f(Q, K, V, block_table, max_blocks, block_size, token_seq, positions, slots, SK, O, o_row, T, scale, splits, L, d, x, s);
 }

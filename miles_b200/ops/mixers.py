@@ -59,10 +59,43 @@ class AttentionLayout:
     rot: int           # rotated dimensions of a head, the first ones
     window: int        # 0: no window
     keep: int          # first tokens a window keeps
+    chunk: int = 0     # 0: no chunks
+    writes: bool = True            # the layer has keys and values of its own
+    value_norm: bool = False       # they are kept with every head's values over their root mean square
 
     @property
     def rows(self) -> int:
-        return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
+        return self.heads * self.dim + (self.kv_heads * (self.dim + self.vdim) if self.writes else 0)
+
+
+@dataclass(frozen=True)
+class DeltaLayout:
+    """Sizes of one gated-delta-rule layer; a row of its projection is [q | k | v | decay latent | gate latent | β]."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+    decay_rank: int
+    gate_rank: int
+
+    @property
+    def key_rows(self) -> int:
+        return self.kv_heads * self.dim
+
+    @property
+    def channels(self) -> int:
+        """q, k and v: what passes the convolution."""
+        return 2 * self.key_rows + self.heads * self.vdim
+
+    @property
+    def gate_at(self) -> int:
+        return self.channels + self.decay_rank
+
+    @property
+    def beta_at(self) -> int:
+        return self.gate_at + self.gate_rank
 
 
 @dataclass(frozen=True)
@@ -182,12 +215,14 @@ def clamped_glu(h, limit, alpha, shift=1.0):
     return ref.clamped_glu(h, limit, alpha, shift)
 
 
-def latent_attention(proj, lay: LatentLayout, cache, meta, *, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps):
-    """proj [T, q rows (+ rank + rot)] → attention output [T, heads·vdim].  Rotates queries and (with `kv_norm`) norms, rotates
-    and caches the new latents; then every token attends to the cached latents it sees."""
-    if proj.is_cuda:
-        return _k().latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps)
-    return ref.latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps)
+def latent_attention(proj, lay: LatentLayout, cache, meta, *, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps, q=None, gate=None):
+    """proj [T, q rows (+ rank + rot)], or q [T, q rows] and proj [T, (rank + rot)] → attention output [T, heads·vdim], times
+    sigmoid(gate) if given.  Rotates queries and (with `kv_norm`) norms, rotates and caches the new latents; then every token attends
+    to the cached latents it sees."""
+    kv = proj[:, lay.q_rows:] if q is None else proj
+    q = proj[:, : lay.q_rows] if q is None else q
+    f = _k().latent_attention if proj.is_cuda else ref.latent_attention
+    return f(q, kv, lay, cache, meta, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps, gate)
 
 
 def linear_state_attention(proj, heads, dk, dv, decay, state, meta, norm_w, eps):
@@ -237,14 +272,52 @@ def projections(h, w, w2=None, b2=None):
     return ref.projections(h, w, w2, b2)
 
 
-def windowed_attention(proj, lay: AttentionLayout, kc, vc, meta, out, *, freq, magnitude, scale, sink, q_norm, k_norm, eps, aside=None):
-    """proj [T, ≥ q; k; v] → `out` [T, heads·vdim] (may be strided).  Norms queries and keys over the whole projection, rotates them,
-    caches keys and values; then every token attends to the cached tokens it sees: those less than `window` back, and the first
-    `keep` ones.  `aside` is done on the way."""
+def windowed_attention(proj, lay: AttentionLayout, kc, vc, meta, out, *, freq, magnitude, scale, sink, q_norm, k_norm, eps, aside=None, bias=None,
+                       gate=None):
+    """proj [T, ≥ q (; k; v)] → `out` [T, heads·vdim] (may be strided).  Norms queries and keys over the whole projection, rotates them,
+    caches keys and values (those of a layer that has its own); then every token attends to the cached tokens it sees: those less than
+    `window` back, and the first `keep` ones, or those of its own `chunk`.  `bias` (r1, r2 per head): r1·ln(1 + r2·distance) off the
+    scores; `gate` [T, heads·vdim]: outputs times its sigmoid.  `aside` is done on the way."""
     if proj.is_cuda:
-        return _k().windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps, aside)
+        return _k().windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps, aside, bias, gate)
     ref.aside(aside)
-    return ref.windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps)
+    return ref.windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps, bias, gate)
+
+
+def delta_rule(proj, lay: DeltaLayout, conv, w_a, w_g, A_log, dt_bias, norm_w, state, ring, meta, eps):
+    """proj [T, q; k; v; decay latent; gate latent; β] → [T, heads·vdim].  Causal convolution and silu on q, k, v; q and k to unit vectors per
+    head (q over √dim on top); decays g = exp(−exp(A_log)·softplus(w_a·latent + dt_bias)) per head and key channel; per head
+    S ← diag(g)·S, S ← S + k (σ(β)·(v − Sᵀk))ᵀ, o = Sᵀq; every head's o over its root mean square, times norm_w and the sigmoid of w_g·latent.
+    `state` [slots, heads, dim, vdim] and `ring` [slots, taps, channels] (the convolution's inputs by position mod taps; None
+    without look-back), fp32, are read (nothing before position 0) and written."""
+    f = _k().delta_rule if proj.is_cuda else ref.delta_rule
+    return f(proj, lay, conv, w_a, w_g, A_log, dt_bias, norm_w, state, ring, meta, eps)
+
+
+def residual_norm(x, y, yn, mult, nw, eps, dtype, gain=1.0):
+    """x ← x + mult·y, or x + mult·rmsnorm(y)·yn (fp32, in place; y None: x as it is).  Returns rmsnorm(x)·nw·gain in `dtype` (without
+    `nw`: a copy of x)."""
+    return (_k() if x.is_cuda else ref).residual_norm(x, y, yn, mult, nw, eps, dtype, gain)
+
+
+def residual_linear(x, y, yn, mult, nw, eps, w):
+    """`residual_norm` and the product with w in one kernel (where `few_row_sum` holds).  Returns (product, new x)."""
+    return _k().residual_linear(x, y, yn, mult, nw, eps, w)
+
+
+def xielu(z, act):
+    """z²·softplus(act₀) + z/2 for z > 0, (½ + softplus(act₁))·(exp(z) − 1 − z) + z/2 for z ≤ 0."""
+    return (_k() if z.is_cuda else ref).xielu(z, act)
+
+
+def gelu_times_rows(z, tokens, table, col):
+    """gelu(z) (tanh form) times columns [col, col + width) of the tokens' rows of `table`."""
+    return (_k() if z.is_cuda else ref).gelu_times_rows(z, tokens, table, col)
+
+
+def softcap_(logits, cap, exact=False):
+    """logits ← cap·tanh(logits / cap), fp32 in place; `exact`: good to 32 bits."""
+    return (_k() if logits.is_cuda else ref).softcap_(logits, cap, exact)
 
 
 def differential_attention(proj, lay: DifferentialLayout, kc, vc, meta, *, scale, diff, temperature, lvec, q_norm, k_norm, eps, aside=None):

@@ -1,5 +1,5 @@
 """CUDA execution of the ops in `mixers.py` (inference only): the kernels of mixers.cu, latent_*.cu, linear_*.cu, window_*.cu,
-diff_prep.cu, ssm_*.cu, attention_*_tc.cu, paged_attend.cu and experts_any.cu.
+diff_prep.cu, ssm_*.cu, delta_*.cu, attention_*_tc.cu, paged_attend.cu and experts_any.cu.
 
 Tensors are bf16, or float32 throughout (then every product is a true 32-bit one: the kernels' own fp32 loops, and cuBLAS
 without TF32 for the dense projections, as `ops.linear` does for float32).
@@ -138,27 +138,35 @@ def _key_ranges(meta, window: int):
     return rg.scratch[window]
 
 
-def _head_linear(x, w, w_nk, y, fast):
-    (C.head_linear_mma if fast else C.head_linear)(x, w, w_nk, y)
+def _head_linear(x, w, w_nk, y, fast, gate=None):
+    (C.head_linear_mma if fast else C.head_linear)(x, w, w_nk, y, gate)
 
 
-def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps):
-    T, H, rg = proj.shape[0], lay.heads, meta.ragged
+def _whole_rows(x):
+    """Rows that start on 16-byte boundaries: x itself, or a copy in rows of whole 16-byte pieces (None stays None)."""
+    piece = 16 // x.element_size() if x is not None else 1
+    if x is None or (x.stride(0) % piece == 0 and x.data_ptr() % 16 == 0):
+        return x
+    return _rows(x.shape[0], x.shape[1], x.dtype, x.device).copy_(x)
+
+
+def latent_attention(q, kv, lay, cache, meta, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps, gate=None):
+    T, H, rg = q.shape[0], lay.heads, meta.ragged
     sizes = [H, lay.dim, lay.rot, lay.vdim, lay.rank, lay.rank_p, lay.pitch]
-    dt, dev = proj.dtype, proj.device
+    dt, dev = q.dtype, q.device
     fast = _mma_ok(lay, dt)
     t_long = rg.t_long if _prefill_ok(lay, dt, scale) else 0
     n_short = T - t_long
     q_nope = (lay.dim + 63) // 64 * 64
     q_abs = torch.empty(n_short, H, lay.pitch, dtype=dt, device=dev)
     q_full = torch.empty(t_long, H, q_nope + 64, dtype=dt, device=dev)
-    C.latent_prep(proj, meta.positions, meta.slot_mapping, freq, float(magnitude), kv_norm, float(eps), cache, q_abs, q_full, t_long, q_nope,
+    C.latent_prep(q, kv, meta.positions, meta.slot_mapping, freq, float(magnitude), kv_norm, float(eps), cache, q_abs, q_full, t_long, q_nope,
                   q_nope + 64, sizes)
     out = torch.empty(T, H, lay.vdim, dtype=dt, device=dev)
     if n_short:
         w_uk, w_uv = w_ukv[: H * lay.dim].view(H, lay.dim, lay.rank), w_ukv[H * lay.dim:].view(H, lay.vdim, lay.rank)
-        qn = proj[t_long:, : lay.q_rows].unflatten(1, (H, lay.dim + lay.rot))[..., : lay.dim]
-        aligned = fast and proj.stride(0) % 8 == 0
+        qn = q[t_long:].unflatten(1, (H, lay.dim + lay.rot))[..., : lay.dim]
+        aligned = fast and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
         _head_linear(qn, w_uk, False, q_abs[..., : lay.rank], aligned)
         o_lat = torch.empty(n_short, H, lay.rank, dtype=dt, device=dev)
         seq = rg.token_seq[t_long:] if rg.token_seq is not None else None
@@ -168,10 +176,10 @@ def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sin
             part_o = torch.empty(n_short * H * splits * lay.rank_p, dtype=torch.float32, device=dev)
             part_ml = torch.empty(n_short * H * splits * 2, dtype=torch.float32, device=dev)
             C.latent_decode(q_abs, cache, meta.block_table, seq, pos, slots, sink, part_o, part_ml, o_lat, float(scale), int(window), splits, sizes,
-                            C.error_flag(proj))
+                            C.error_flag(q))
         else:
             C.latent_attend(q_abs, cache, meta.block_table, seq, pos, slots, sink, o_lat, float(scale), int(window), sizes)
-        _head_linear(o_lat, w_uv, True, out[t_long:], fast)
+        _head_linear(o_lat, w_uv, True, out[t_long:], fast, gate[t_long:] if gate is not None else None)
     if t_long:
         cu_k, base, total, max_q = _key_ranges(meta, window)
         lat = torch.empty(total, lay.pitch, dtype=dt, device=dev)
@@ -179,7 +187,8 @@ def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sin
         N = H * (lay.dim + lay.vdim)
         kv = torch.empty(total, N, dtype=dt, device=dev)
         C.gemm(lat, w_ukv, kv, total, N, lay.rank, lay.pitch, lay.rank, N, False, False, False, None, 0)
-        C.latent_prefill(q_full, kv, lat, out, sink, rg.cu_q, cu_k, rg.n_long, max_q, float(scale), int(window), sizes, C.error_flag(proj))
+        C.latent_prefill(q_full, kv, lat, out, sink, rg.cu_q, cu_k, rg.n_long, max_q, float(scale), int(window), sizes, C.error_flag(q),
+                         _whole_rows(gate[:t_long]) if gate is not None else None)
     return out.view(T, H * lay.vdim)
 
 
@@ -282,18 +291,19 @@ def window_splits(tokens: int, lay) -> int:
     """CTAs of a cluster that share the keys of one (token, key head): enough for the SMs, at most one per tile of 64 keys."""
     group = lay.heads // lay.kv_heads
     ctas = tokens * lay.kv_heads * -(-group // (16 if group > 8 else 8))
-    tiles = -(-(lay.window + lay.keep) // 64) if lay.window else 64
+    tiles = -(-(lay.window + lay.keep) // 64) if lay.window else -(-lay.chunk // 64) if lay.chunk else 64
     return max(1, min(8, tiles, 444 // ctas))
 
 
-def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps, aside):
+def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps, aside, bias=None, gate=None):
     T, rg, dt, dev = proj.shape[0], meta.ragged, proj.dtype, proj.device
     fast = _window_ok(lay, dt) and out.stride(0) % 8 == 0
     pitch = -(-lay.dim // 64) * 64 if fast else lay.dim
-    sizes = [lay.heads, lay.kv_heads, lay.dim, lay.vdim, lay.rot, lay.window, lay.keep, pitch]
+    sizes = [lay.heads, lay.kv_heads, lay.dim, lay.vdim, lay.rot, lay.window, lay.keep, pitch, lay.chunk]
     q = torch.empty(T, lay.heads, pitch, dtype=dt, device=dev)
-    C.window_prep(proj, meta.positions, meta.slot_mapping, freq, float(magnitude), q_norm, k_norm, float(eps), kc, vc, q, sizes, *_aside(aside, T))
-    _paged_attention(q, lay, kc, vc, meta, out, scale, sink, sizes, fast)
+    C.window_prep(proj, meta.positions, meta.slot_mapping, freq, float(magnitude), q_norm, k_norm, float(eps), kc if lay.writes else None,
+                  vc if lay.writes else None, q, sizes, *_aside(aside, T), lay.value_norm)
+    _paged_attention(q, lay, kc, vc, meta, out, scale, sink, sizes, fast, bias=bias, gate=_whole_rows(gate) if fast else gate)
 
 
 def _aside(a, T: int):
@@ -308,27 +318,29 @@ def _aside(a, T: int):
             [float(a.limit), float(a.alpha), float(a.shift), float(r.scale) if r else 1.0], [1, r.groups, r.keep] if r else [0, 1, 1])
 
 
-def _paged_attention(q, lay, kc, vc, meta, out, scale, sink, sizes, fast, difference=()):
+def _paged_attention(q, lay, kc, vc, meta, out, scale, sink, sizes, fast, difference=(), bias=None, gate=None):
     """Prepared queries over the paged cache: long pieces as query tiles, short ones token by token.  `difference`: (weight of the second map,
-    gates, gain, eps) of differential attention."""
+    gates, gain, eps) of differential attention; `bias` (r1, r2), `gate`: see `windowed_attention`."""
     T, rg = q.shape[0], meta.ragged
+    r1, r2 = bias or (None, None)
     t_long = rg.t_long if fast and scale > 0 and kc.shape[1] % 8 == 0 and lay.heads // lay.kv_heads <= 128 else 0
     if t_long:
         C.window_prefill(q, kc, vc, out, sink, rg.cu_q, meta.positions, meta.block_table, rg.n_long, max(rg.q_lens[: rg.n_long]), t_long,
-                         float(scale), sizes, C.error_flag(q), *difference)
+                         float(scale), sizes, C.error_flag(q), *difference, r1=r1, r2=r2, out_gate=gate)
     if T > t_long:
         seq = rg.token_seq[t_long:] if rg.token_seq is not None else None
         where = (kc, vc, meta.block_table, seq, meta.positions[t_long:], meta.slot_mapping[t_long:], sink)
+        extra = dict(r1=r1, r2=r2, out_gate=gate[t_long:] if gate is not None else None)
         if difference:
             difference = (difference[0], difference[1][t_long:], *difference[2:])
         if fast:
-            C.window_decode(q[t_long:], *where, out[t_long:], float(scale), window_splits(T - t_long, lay), sizes, *difference)
+            C.window_decode(q[t_long:], *where, out[t_long:], float(scale), window_splits(T - t_long, lay), sizes, *difference, **extra)
         elif difference:
             both = torch.empty(T - t_long, lay.heads * lay.vdim, dtype=torch.float32, device=q.device)
             C.window_attend(q[t_long:], *where, both, float(scale), sizes)
             C.diff_combine(both, out[t_long:], lay.heads // 2, lay.vdim, *difference)
         else:
-            C.window_attend(q[t_long:], *where, out[t_long:], float(scale), sizes)
+            C.window_attend(q[t_long:], *where, out[t_long:], float(scale), sizes, **extra)
 
 
 def differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lvec, q_norm, k_norm, eps, aside):
@@ -346,6 +358,48 @@ def differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lv
     gates = proj[:, lay.gate_at: lay.gate_at + lay.heads]
     _paged_attention(q, pair, kc, vc, meta, out, scale, None, sizes, fast, (lam, gates, 1.0 - diff, float(eps)))
     return out
+
+
+# ---- gated delta rule -------------------------------------------------------------------------------------------------
+
+def _low_rank(x, w):
+    """x·wᵀ for rows that are part of a wider projection."""
+    if x.dtype != BF16:
+        return torch.nn.functional.linear(x, w)
+    K_ = x.shape[1]
+    if x.shape[0] > K.GEMV_M and K_ % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
+        out = _rows(x.shape[0], w.shape[0], BF16, x.device)
+        C.gemm(x, w, out, x.shape[0], w.shape[0], K_, x.stride(0), K_, out.stride(0), False, False, False, None, 0)
+        return out
+    return K.gemm_nt(x, w)
+
+
+def delta_rule(proj, lay, conv, w_a, w_g, A_log, dt_bias, norm_w, state, ring, meta, eps):
+    T, dt, dev, rg = proj.shape[0], proj.dtype, proj.device, meta.ragged
+    sizes = [lay.heads, lay.kv_heads, lay.dim, lay.vdim, lay.taps, lay.beta_at]
+    raw, gate = _low_rank(proj[:, lay.channels: lay.gate_at], w_a), _low_rank(proj[:, lay.gate_at: lay.beta_at], w_g)
+    out = torch.empty(T, lay.heads * lay.vdim, dtype=dt, device=dev)
+
+    def tensors(slots, positions, raw):
+        return [conv, A_log, dt_bias, state, ring, slots, positions, raw]
+
+    slots, cu_q = meta.state_slots, rg.cu_q
+    if cu_q is None and _step_ok(lay):
+        C.delta_step(proj, sizes, tensors(slots, meta.positions, raw), norm_w, gate, float(eps), out)
+        return out
+    act = torch.empty(T, lay.channels, dtype=dt, device=dev)
+    C.delta_conv(proj, sizes, tensors(slots, meta.positions, raw), _conv_tiles(meta, lay.taps) if cu_q is not None else None, cu_q, act)
+    C.delta_seq(proj, act, sizes, tensors(slots, meta.positions, raw), cu_q, out)
+    normed = torch.empty_like(out)
+    C.head_gated_norm(out, norm_w, gate, normed, float(eps))
+    return normed
+
+
+def _step_ok(lay) -> bool:
+    if lay.vdim % 4 or lay.vdim > 1024:
+        return False
+    rows = 256 // (lay.vdim // 4)
+    return -(-lay.dim // rows) * rows * lay.vdim <= C.delta_step_max() and (rows * lay.vdim + lay.vdim + 3 * lay.dim) * 4 <= 48 * 1024
 
 
 # ---- state-space mixer ------------------------------------------------------------------------------------------------
@@ -395,10 +449,50 @@ def state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta, a
     return out
 
 
+def residual_norm(x, y, yn, mult, nw, eps, dtype, gain=1.0):
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    if yn is None:
+        C.sum_norm(x, x if y is not None else None, y, None, None, None, None, None, None, None, nw, h, None, None, float(eps), 0.0, float(gain), float(mult))
+    else:
+        C.output_norm(x, _c(y), yn, None, nw, h, float(eps), float(mult), float(gain))
+    return h
+
+
+def residual_linear(x, y, yn, mult, nw, eps, w):
+    out = _rows(x.shape[0], w.shape[0], w.dtype, x.device)
+    if y is None:
+        C.gemv_sum_norm(x, None, None, None, None, None, None, nw, None, float(eps), 0.0, w, out, None, None, None, None, None, _static(w))
+        return out, x
+    x_new = torch.empty_like(x)
+    if yn is None:
+        C.gemv_sum_norm(x, _c(y), None, None, None, None, None, nw, None, float(eps), 0.0, w, out, None, None, None, x_new, None, _static(w), float(mult))
+    else:
+        C.gemv_output_norm(x, _c(y), yn, None, float(eps), w, out, x_new, _static(w), float(mult), nw)
+    return out, x_new
+
+
+def xielu(z, act):
+    z = _c(z)
+    out = torch.empty_like(z)
+    C.xielu(z, act, out)
+    return out
+
+
+def gelu_times_rows(z, tokens, table, col):
+    out = torch.empty(z.shape, dtype=z.dtype, device=z.device)
+    C.gelu_rows(z, tokens.to(torch.int32), table, col, out)
+    return out
+
+
+def softcap_(logits, cap, exact):
+    C.softcap(logits, float(cap), bool(exact))
+    return logits
+
+
 def part_norm_linear(x, nw, parts, eps, w):
     if parts == 1 and w.shape[0] <= GEMV_MAX_N and gemv_ok(x, w):
         return K.add_rmsnorm_linear(x, None, nw, eps, w)[0]        # a handful of rows: the norm inside the product
-    h = torch.empty_like(x)
+    h = torch.empty(x.shape, dtype=x.dtype, device=x.device)
     C.part_norm(x, nw, h, parts, float(eps))
     return K.linear(h, w)
 

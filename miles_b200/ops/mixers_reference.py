@@ -57,13 +57,17 @@ def rotate_pairs(x, positions, freq, magnitude):
     return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2).to(x.dtype)
 
 
-def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps):
-    T, H = proj.shape[0], lay.heads
-    q = proj[:, :lay.q_rows].view(T, H, lay.dim + lay.rot)
+def gated(o, gate):
+    return o if gate is None else o * torch.sigmoid(gate.float())
+
+
+def latent_attention(q, kv, lay, cache, meta, freq, magnitude, scale, window, sink, w_ukv, kv_norm, eps, gate=None):
+    T, H, dtype = q.shape[0], lay.heads, q.dtype
+    q = q.reshape(T, H, lay.dim + lay.rot)
     qn, qr = q[..., :lay.dim].float(), rotate_pairs(q[..., lay.dim:], meta.positions, freq, magnitude).float()
     flat = cache.view(-1, lay.pitch)
     if kv_norm is not None:
-        kv = proj[:, lay.q_rows:].float()
+        kv = kv[:, : lay.rank + lay.rot].float()
         c = kv[:, :lay.rank]
         c = c * torch.rsqrt(c.square().mean(-1, keepdim=True) + eps) * kv_norm.float()
         ok = meta.slot_mapping >= 0
@@ -93,7 +97,7 @@ def latent_attention(proj, lay, cache, meta, freq, magnitude, scale, window, sin
             sc = torch.cat([sc, sink.float()[:, None, None].expand(H, s1 - s0, 1)], -1)
         p = torch.softmax(sc, -1)[..., : keys.numel()]
         out[s0:s1] = torch.einsum("hts,shd->thd", p, v)
-    return out.reshape(T, H * lay.vdim).to(proj.dtype)
+    return gated(out.reshape(T, H * lay.vdim), gate).to(dtype)
 
 
 def linear_state(proj, H, dk, dv, decay, state, meta):
@@ -166,9 +170,9 @@ def routed_experts(h, w13, w2, weights, index, limit=0.0, alpha=0.0, shift=1.0, 
     return out.to(h.dtype)
 
 
-def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps):
+def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sink, q_norm, k_norm, eps, bias=None, gate=None):
     T, H, G = proj.shape[0], lay.heads, lay.kv_heads
-    q, k, v = proj[:, : lay.rows].split([H * lay.dim, G * lay.dim, G * lay.vdim], -1)
+    q = proj[:, : H * lay.dim]
 
     def prepared(x, w, heads):
         x = x.float()
@@ -179,11 +183,16 @@ def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sin
             x = torch.cat([rotate_pairs(x[..., : lay.rot], meta.positions, freq, magnitude), x[..., lay.rot:]], -1)
         return x.to(proj.dtype)
 
-    q, k = prepared(q, q_norm, H), prepared(k, k_norm, G)
-    ok = meta.slot_mapping >= 0
-    at = meta.slot_mapping[ok].long()
-    kc.view(-1, G, lay.dim)[at] = k[ok].to(kc.dtype)
-    vc.view(-1, G, lay.vdim)[at] = v.reshape(T, G, lay.vdim)[ok].to(vc.dtype)
+    q = prepared(q, q_norm, H)
+    if lay.writes:
+        k, v = proj[:, H * lay.dim: lay.rows].split([G * lay.dim, G * lay.vdim], -1)
+        v = v.reshape(T, G, lay.vdim)
+        if lay.value_norm:
+            v = v.float() * torch.rsqrt(v.float().square().mean(-1, keepdim=True) + eps)
+        ok = meta.slot_mapping >= 0
+        at = meta.slot_mapping[ok].long()
+        kc.view(-1, G, lay.dim)[at] = prepared(k, k_norm, G)[ok].to(kc.dtype)
+        vc.view(-1, G, lay.vdim)[at] = v[ok].to(vc.dtype)
     bs = kc.shape[1]
     out.zero_()
     for b, s0, s1 in _sequences(meta, T):
@@ -198,11 +207,17 @@ def windowed_attention(proj, lay, kc, vc, meta, out, freq, magnitude, scale, sin
         seen = keys[None] <= pos[:, None]
         if lay.window:
             seen &= (pos[:, None] - keys[None] < lay.window) | (keys[None] < lay.keep)
+        if lay.chunk:
+            seen &= pos[:, None] // lay.chunk == keys[None] // lay.chunk
+        if bias is not None:
+            r1, r2 = (r.float()[:, None, None] for r in bias)
+            sc = sc - r1 * torch.log1p(r2 * (pos[:, None] - keys[None]).clamp(min=0).float())
         sc = sc.masked_fill(~seen[None], float("-inf"))
         if sink is not None:
             sc = torch.cat([sc, sink.float()[:, None, None].expand(H, s1 - s0, 1)], -1)
         p = torch.softmax(sc, -1)[..., : keys.numel()]
-        out[s0:s1] = torch.einsum("hts,shd->thd", p, vv).reshape(s1 - s0, -1).to(out.dtype)
+        o = torch.einsum("hts,shd->thd", p, vv).reshape(s1 - s0, -1)
+        out[s0:s1] = gated(o, gate[s0:s1] if gate is not None else None).to(out.dtype)
     return out
 
 
@@ -244,6 +259,70 @@ def differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lv
     return (out * torch.sigmoid(gate)[..., None]).reshape(T, H * lay.vdim).to(proj.dtype)
 
 
+def short_conv(x, w, b, ring, slot, p0):
+    """silu of the causal convolution of a piece's rows that starts at position p0, from and to the ring of its last inputs (rounded to
+    the rows' dtype, as floats)."""
+    taps, n = w.shape[1], x.shape[0]
+    before = [ring[slot, p % taps] if p >= 0 else torch.zeros(x.shape[1]) for p in range(p0 - taps + 1, p0)]
+    rows = torch.cat([torch.stack(before), x.float()]) if before else x.float()
+    act = sum(rows[k: k + n] * w[:, k].float() for k in range(taps))
+    if ring is not None:
+        for t in range(max(0, n - taps + 1), n):
+            ring[slot, (p0 + t) % taps] = x[t].float()
+    return torch.nn.functional.silu(act if b is None else act + b.float()).to(x.dtype).float()
+
+
+def delta_rule(proj, lay, conv, w_a, w_g, A_log, dt_bias, norm_w, state, ring, meta, eps):
+    T, H, G, K, V = proj.shape[0], lay.heads, lay.kv_heads, lay.dim, lay.vdim
+    raw = proj[:, lay.channels: lay.gate_at] @ w_a.T
+    logg = -torch.exp(A_log.float())[:, None] * torch.nn.functional.softplus((raw.float() + dt_bias.float()).view(T, H, K), threshold=1e9)
+    gate = proj[:, lay.gate_at: lay.beta_at] @ w_g.T
+    beta = torch.sigmoid(proj[:, lay.beta_at: lay.beta_at + H].float())
+    out = torch.zeros(T, H, V)
+    for b, s0, s1 in _sequences(meta, T):
+        slot = int(meta.state_slots[b])
+        if slot < 0 or s1 == s0:
+            continue
+        p0 = int(meta.positions[s0])
+        q, k, v = short_conv(proj[s0:s1, : lay.channels], conv, None, ring, slot, p0).split([G * K, G * K, H * V], -1)
+        q, k = (x.reshape(-1, G, K) * torch.rsqrt(x.reshape(-1, G, K).square().sum(-1, keepdim=True) + 1e-6) for x in (q, k))
+        q, k = (x.repeat_interleave(H // G, 1) for x in (q * K ** -0.5, k))
+        v = v.reshape(-1, H, V)
+        S = state[slot].clone() if p0 > 0 else torch.zeros_like(state[slot])
+        for i, t in enumerate(range(s0, s1)):
+            S = S * torch.exp(logg[t])[:, :, None]
+            u = beta[t][:, None] * (v[i] - torch.einsum("hkv,hk->hv", S, k[i]))
+            S = S + k[i][:, :, None] * u[:, None, :]
+            out[t] = torch.einsum("hkv,hk->hv", S, q[i])
+        state[slot] = S
+    out = out.to(proj.dtype).float()
+    out = out * torch.rsqrt(out.square().mean(-1, keepdim=True) + eps) * norm_w.float()
+    return (out.reshape(T, H * V) * torch.sigmoid(gate.float())).to(proj.dtype)
+
+
+def residual_norm(x, y, yn, mult, nw, eps, dtype, gain=1.0):
+    if y is not None:
+        yf = y.float()
+        x.add_(mult * (yf if yn is None else yf * torch.rsqrt(yf.square().mean(-1, keepdim=True) + eps) * yn.float()))
+    return (x if nw is None else x * torch.rsqrt(x.square().mean(-1, keepdim=True) + eps) * nw.float() * gain).to(dtype)
+
+
+def xielu(z, act):
+    f = z.float()
+    a, b = torch.nn.functional.softplus(act.float(), threshold=1e9)
+    neg = f.clamp(max=0)
+    return (0.5 * f + torch.where(f > 0, a * f * f, (0.5 + b) * (torch.expm1(neg) - neg))).to(z.dtype)
+
+
+def gelu_times_rows(z, tokens, table, col):
+    e = table[tokens.long(), col: col + z.shape[1]].float()
+    return (torch.nn.functional.gelu(z.float(), approximate="tanh") * e).to(z.dtype)
+
+
+def softcap_(logits, cap, exact=False):
+    return logits.div_(cap).tanh_().mul_(cap)
+
+
 def state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta):
     T, H, V, N, G, taps = proj.shape[0], lay.heads, lay.vdim, lay.state, lay.groups, lay.taps
     z, xbc, dt = proj[:, : lay.inner + lay.channels + H].split([lay.inner, lay.channels, H], -1)
@@ -255,13 +334,7 @@ def state_space(proj, lay, conv, conv_b, dt_bias, A_log, D, state, ring, meta):
         if slot < 0 or s1 == s0:
             continue
         p0 = int(meta.positions[s0])
-        before = [ring[slot, p % taps] if p >= 0 else torch.zeros(lay.channels) for p in range(p0 - taps + 1, p0)]
-        rows = torch.cat([torch.stack(before), xbc[s0:s1].float()]) if before else xbc[s0:s1].float()
-        act = conv_b.float() + sum(rows[k: k + s1 - s0] * conv[:, k].float() for k in range(taps))
-        x, B, C = torch.nn.functional.silu(act).to(proj.dtype).float().split([lay.inner, G * N, G * N], -1)
-        if ring is not None:
-            for t in range(max(s0, s1 - taps + 1), s1):
-                ring[slot, (p0 + t - s0) % taps] = xbc[t].float()
+        x, B, C = short_conv(xbc[s0:s1], conv, conv_b, ring, slot, p0).split([lay.inner, G * N, G * N], -1)
         x = x.view(-1, H, V)
         B, C = (y.reshape(-1, G, N).repeat_interleave(H // G, 1) for y in (B, C))
         S = state[slot].clone() if p0 > 0 else torch.zeros_like(state[slot])

@@ -116,8 +116,8 @@ def test_weights_from_disk(tmp_path):
 def test_serving_build_of_a_configuration():
     from miles_b200.ops import build
 
-    assert build.serve_kind(get_config("ronupel-tiny")) == "attention" and build.serve_kind(get_config("nopelorn-tiny")) == "latent"
-    for kind, files in build.SERVE_KINDS.items():
+    assert build.serve_kind(get_config("ronupel-tiny")) == "attention_experts_prep" and build.serve_kind(get_config("nopelorn-tiny")) == "latent_linear"
+    for kind, files in build.SERVE_PARTS.items():
         assert all(os.path.exists(os.path.join(build.CSRC, f)) for f in build.SERVE_SOURCES + files), kind
 
 

@@ -111,11 +111,11 @@ def test_weights_from_disk(tmp_path):
 def test_serving_build_of_a_configuration():
     from miles_b200.ops import build
 
-    assert build.serve_kind(get_config("vozirax-tiny")) == "hybrid"
-    assert "window_prep.cu" not in build.SERVE_KINDS["hybrid"] and "ssm_chunk.cu" not in build.SERVE_KINDS["attention"]
-    for kind, files in build.SERVE_KINDS.items():       # a build with experts registers their bindings
-        with open(os.path.join(build.CSRC, "bindings_more.cpp")) as f:
-            assert ("bindings_moe.cpp" in files) == (f"MB_SERVE_{kind.upper()}" in f.read()), kind
+    assert build.serve_kind(get_config("vozirax-tiny")) == "attention_differential_experts_ssm"
+    for part, files in build.SERVE_PARTS.items():       # the part with experts registers their bindings, every other one its mixers'
+        registered = "bindings_more.cpp" if "bindings_moe.cpp" in files else "bindings_mixers.cpp"
+        with open(os.path.join(build.CSRC, registered)) as f:
+            assert f"MB_SERVE_{part.upper()})" in f.read() or registered == "bindings_mixers.cpp", part
 
 
 # ---- mechanisms ---------------------------------------------------------------------------------------------------------------
