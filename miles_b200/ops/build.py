@@ -39,7 +39,7 @@ SERVE_PARTS = {
     "prep": ["window_prep.cu"],
     "differential": ["diff_prep.cu"],
     "ssm": ["ssm_state.cu", "ssm_chunk.cu"],
-    "delta": ["delta_state.cu"],
+    "delta": ["delta_state.cu", "delta_chunk.cu"],
     "experts": ["bindings_moe.cpp", "moe.cu", "experts_any.cu"],
 }
 _serving: str | None = None                   # the serving build this process asked for

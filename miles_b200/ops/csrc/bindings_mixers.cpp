@@ -558,6 +558,17 @@ void delta_seq(const at::Tensor& proj, const at::Tensor& act, const std::vector<
         "mb_delta_seq");
 }
 
+void delta_chunk(const at::Tensor& proj, const at::Tensor& act, const std::vector<int64_t>& sizes, const std::vector<OptTensor>& t, const at::Tensor& chunks,
+                 const at::Tensor& parts, at::Tensor& scratch, int64_t warps, at::Tensor& out, at::Tensor& err) {
+  c10::cuda::CUDAGuard g(proj.device());
+  const MbDelta m = delta(sizes, t);
+  TORCH_CHECK(scratch.nbytes() >= static_cast<size_t>(mb_delta_chunk_bytes(m.K, m.V)) * chunks.size(0) * m.H, "delta_chunk: scratch too small");
+  mb_count_launch(1);
+  check(mb_delta_chunk(proj.data_ptr(), proj.stride(0), act.data_ptr(), m, chunks.data_ptr<int>(), parts.data_ptr<int>(), scratch.data_ptr(),
+                       out.data_ptr(), chunks.size(0), parts.size(0), warps, err.data_ptr<int>(), cur_stream()),
+        "mb_delta_chunk");
+}
+
 void delta_step(const at::Tensor& proj, const std::vector<int64_t>& sizes, const std::vector<OptTensor>& t, const at::Tensor& norm_w, const at::Tensor& gate,
                 double eps, at::Tensor& out) {
   c10::cuda::CUDAGuard g(proj.device());
@@ -611,6 +622,8 @@ void register_mixers(pybind11::module& m) {
   m.def("delta_seq", &delta_seq);
   m.def("delta_step", &delta_step);
   m.def("delta_step_max", &mb_delta_step_max);
+  m.def("delta_chunk", &delta_chunk);
+  m.def("delta_chunk_bytes", &mb_delta_chunk_bytes);
 #endif
 #ifdef MB_SERVE_DIFFERENTIAL
   m.def("diff_prep", &diff_prep);

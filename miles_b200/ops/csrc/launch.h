@@ -367,6 +367,12 @@ int mb_delta_seq(const void* proj, long long ld, const void* act, MbDelta m, con
 int mb_delta_step(const void* proj, long long ld, MbDelta m, const void* norm_w, const void* gate, long long gate_ld, float eps, void* out, int B,
                   int f32, cudaStream_t s);
 int mb_delta_step_max(void);
+// Long pieces in chunks of 64 tokens on tensor cores (bf16; K, V multiples of 8 up to 128).  chunks [n_chunks][4]: sequence, first token,
+// end; parts [n_parts][4]: first chunk, chunks, sequence (a part's chunks follow one another; a sequence has one part).  scratch:
+// mb_delta_chunk_bytes(K, V) per chunk and head.  warps (2, 4 or 8): 16 value columns each that a CTA of the second kernel takes.
+long long mb_delta_chunk_bytes(int K, int V);
+int mb_delta_chunk(const void* proj, long long ld, const void* act, MbDelta m, const int* chunks, const int* parts, void* scratch, void* out,
+                   int n_chunks, int n_parts, int warps, int* error_flag, cudaStream_t s);
 // ---- ssm_*.cu (state-space mixer: S ← exp(−exp(A_log)·dt)·S + dt·B xᵀ, y = Sᵀ C + D·x) ----
 // A row of the projection is [z: H·V | x: H·V | B: G·N | C: G·N | dt: H]; x, B and C pass a causal convolution of `taps` columns and silu.
 typedef struct {

@@ -389,10 +389,55 @@ def delta_rule(proj, lay, conv, w_a, w_g, A_log, dt_bias, norm_w, state, ring, m
         return out
     act = torch.empty(T, lay.channels, dtype=dt, device=dev)
     C.delta_conv(proj, sizes, tensors(slots, meta.positions, raw), _conv_tiles(meta, lay.taps) if cu_q is not None else None, cu_q, act)
-    C.delta_seq(proj, act, sizes, tensors(slots, meta.positions, raw), cu_q, out)
+    n = rg.n_long if dt == BF16 and lay.dim % 8 == 0 and lay.vdim % 8 == 0 and lay.dim <= 128 and lay.vdim <= 128 and cu_q is not None else 0
+    if n:                                # long pieces in chunks on the tensor cores, the short ones behind them token by token
+        err = C.error_flag(proj)
+        for chunks, parts in _chunk_rounds(meta, lay):
+            scratch = torch.empty(chunks.shape[0] * lay.heads * C.delta_chunk_bytes(lay.dim, lay.vdim), dtype=torch.uint8, device=dev)
+            C.delta_chunk(proj, act, sizes, tensors(slots, meta.positions, raw), chunks, parts, scratch, scan_warps(parts.shape[0] * lay.heads, lay.vdim),
+                          out, err)
+    if slots.numel() > n:
+        C.delta_seq(proj, act, sizes, tensors(slots[n:], meta.positions, raw), cu_q[n:] if cu_q is not None else None, out)
     normed = torch.empty_like(out)
     C.head_gated_norm(out, norm_w, gate, normed, float(eps))
     return normed
+
+
+DELTA_SCRATCH = int(os.environ.get("MILES_DELTA_SCRATCH_MB", "800")) << 20      # what a round of chunks leaves for its second kernel, at most
+
+
+def _chunk_rounds(meta, lay):
+    """The long pieces of a batch in chunks of 64 tokens, in rounds whose scratch stays within bounds; in each every piece gets its share, and
+    its state passes through its slot.  Returns [(chunks [n, 4], parts [n, 4])] (see mb_delta_chunk)."""
+    rg = meta.ragged
+    key = ("delta", lay.heads, lay.dim, lay.vdim)
+    if key not in rg.scratch:
+        lens = rg.q_lens[: rg.n_long]
+        whole = sum(-(-n // 64) for n in lens)
+        rounds = -(-whole // max(1, min(65535, DELTA_SCRATCH // (lay.heads * C.delta_chunk_bytes(lay.dim, lay.vdim)))))
+        tables = []
+        for r in range(rounds):
+            chunks, parts, t = [], [], 0
+            for b, n in enumerate(lens):
+                per = -(-(-(-n // 64)) // rounds) * 64
+                lo, hi = min(n, r * per), min(n, (r + 1) * per)
+                if lo < hi:
+                    parts += [len(chunks) // 4, -(-(hi - lo) // 64), b, 0]
+                    for a in range(lo, hi, 64):
+                        chunks += [b, t + a, t + min(hi, a + 64), 0]
+                t += n
+            if chunks:
+                d = torch.tensor(chunks + parts, dtype=torch.int32).to(meta.positions.device)
+                tables.append((d[: len(chunks)].view(-1, 4), d[len(chunks):].view(-1, 4)))
+        rg.scratch[key] = tables
+    return rg.scratch[key]
+
+
+def scan_warps(pairs: int, vdim: int, sms: int = 148) -> int:
+    """Warps of a CTA of delta_chunk's second kernel, 16 value columns each: the fewest waves of CTAs (one per SM), each slower the more warps
+    share the SM."""
+    slices = -(-vdim // 16)
+    return min((-(-pairs * -(-slices // w) // sms) * cost, w) for w, cost in ((8, 1.0), (4, 0.6), (2, 0.45)) if w == 2 or w <= slices)[1]
 
 
 def _step_ok(lay) -> bool:

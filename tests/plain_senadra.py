@@ -114,9 +114,10 @@ def keys_values(h, W, p, m, eps):
     return (h @ W[p + "k"].T).unflatten(-1, (m["kv_heads"], m["dim"])), rms((h @ W[p + "v"].T).unflatten(-1, (m["kv_heads"], m["vdim"])), eps)
 
 
-def chunk_mask(T, size):
+def chunk_mask(T, size, off=0):
+    """off: a mistake of so many tokens in where chunks start"""
     i = torch.arange(T)
-    return (i[:, None] >= i) & (i[:, None] // size == i // size)
+    return (i[:, None] >= i) & ((i[:, None] + off) // size == (i + off) // size)
 
 
 def distance_bias(T, r1, r2):
@@ -125,10 +126,10 @@ def distance_bias(T, r1, r2):
     return r1[:, None, None] * torch.log1p(r2[:, None, None] * d)
 
 
-def attend(q, k, v, r1, r2, m):
+def attend(q, k, v, r1, r2, m, off=0):
     """q [T, H, dim], k [T, G, dim], v [T, G, vdim] (normed) → [T, H · vdim]"""
     T, H = len(q), m["heads"]
-    seen, off = chunk_mask(T, m["mask"]["size"]), distance_bias(T, r1, r2)
+    seen, off = chunk_mask(T, m["mask"]["size"], off), distance_bias(T, r1, r2)
     out = []
     for h in range(H):
         g = h // (H // m["kv_heads"])
@@ -187,3 +188,92 @@ def run(cfg, W, tokens, layers=None):
             layers.append(x)
     z = rms(x, eps) * W["final.norm"] @ W["head"].T
     return cfg["logit_softcap"] * torch.tanh(z / cfg["logit_softcap"])
+
+
+# ---- configurations and weights of the tests ---------------------------------------------------------------------------------------
+
+def delta(heads=6, kv_heads=3, dim=24, vdim=40, conv=4, decay_rank=10, gate_rank=7):
+    return {"conv": conv, "decay_rank": decay_rank, "dim": dim, "gate_rank": gate_rank, "heads": heads, "kv_heads": kv_heads, "vdim": vdim}
+
+
+def latent(heads=3, dim=24, rot_dim=16, vdim=40, kv_rank=56, q_rank=48, scale=None, base=700.0):
+    return {"dim": dim, "heads": heads, "kv_rank": kv_rank, "q_rank": q_rank, "rot": {"base": base, "dims": rot_dim}, "rot_dim": rot_dim,
+            "scale": scale if scale is not None else 1.2 / math.sqrt(dim + rot_dim), "vdim": vdim}
+
+
+def attn(heads=6, kv_heads=2, dim=16, vdim=24, size=20, scale=None, kv_from=None):
+    m = {"dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": {"size": size}, "scale": scale if scale is not None else 1.3 / math.sqrt(dim), "vdim": vdim}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return m
+
+
+def layer(mixer, ff=72):
+    kind = "channel_delta" if "conv" in mixer else "latent_attention" if "kv_rank" in mixer else "attention"
+    return {"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def make_config(layers, width=64, vocab=131, eps=1e-5, mult=0.6, softcap=12.0, side=16):
+    return {"architecture": "Senadra", "layers": layers, "logit_softcap": softcap, "norm": {"eps": eps}, "residual_mult": mult,
+            "token_side": {"dim": side}, "vocab": vocab, "width": width}
+
+
+def make_weights(cfg, seed=0, gain=1.0):
+    """Random weights of every tensor of the checkpoint (bf16-exact values, so every run sees the same numbers)."""
+    g = torch.Generator().manual_seed(seed)
+    D, n, out = cfg["width"], cfg["token_side"]["dim"], {}
+
+    def lin(name, o, i, k=1.0):
+        out[name] = (torch.randn(o, i, generator=g) * k * gain / math.sqrt(i)).bfloat16()
+
+    def vec(name, n, mean=0.0, std=0.2, sign=False):
+        t = mean + std * torch.randn(n, generator=g)
+        out[name] = (t.abs() if sign else t).bfloat16()
+
+    lin("embed", cfg["vocab"], D, math.sqrt(D))
+    lin("side.embed", cfg["vocab"], n * len(cfg["layers"]), math.sqrt(n * len(cfg["layers"])))
+    for i, spec in enumerate(cfg["layers"]):
+        m, f, p = spec["mixer"], spec["mlp"], f"l{i}."
+        vec(p + "norm1", D, 1.0)
+        q = p + "mix."
+        if spec["type"] == "channel_delta":
+            for t, rows in (("q", m["kv_heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["heads"] * m["vdim"])):
+                lin(q + t, rows, D, 1.5)
+                lin(q + t + ".conv", rows, m["conv"], 1.3)
+            lin(q + "b", m["heads"], D, 1.5)
+            vec(q + "A_log", m["heads"], -1.5, 1.5)             # heads that forget at once beside heads that remember
+            vec(q + "dt_bias", m["heads"] * m["dim"], -1.5, 1.5)
+            vec(q + "norm", m["vdim"], 1.0)
+            lin(q + "a1", m["decay_rank"], D)
+            lin(q + "a2", m["heads"] * m["dim"], m["decay_rank"])
+            lin(q + "g1", m["gate_rank"], D)
+            lin(q + "g2", m["heads"] * m["vdim"], m["gate_rank"], 1.5)
+        elif spec["type"] == "latent_attention":
+            lin(q + "dq", m["q_rank"], D)
+            vec(q + "dq.norm", m["q_rank"], 1.0)
+            lin(q + "uq", m["heads"] * (m["dim"] + m["rot_dim"]), m["q_rank"], 1.5)
+            lin(q + "dkv", m["kv_rank"] + m["rot_dim"], D, 1.5)
+            vec(q + "dkv.norm", m["kv_rank"], 1.0)
+            lin(q + "uk", m["heads"] * m["dim"], m["kv_rank"])
+            lin(q + "uv", m["heads"] * m["vdim"], m["kv_rank"])
+        else:
+            lin(q + "q", m["heads"] * m["dim"], D, 1.5)
+            if m.get("kv_from") is None:
+                lin(q + "k", m["kv_heads"] * m["dim"], D, 1.5)
+                lin(q + "v", m["kv_heads"] * m["vdim"], D)
+            vec(q + "r1", m["heads"], 0.6, 0.5, True)
+            vec(q + "r2", m["heads"], 0.4, 0.3, True)
+        if spec["type"] != "channel_delta":
+            lin(q + "g", m["heads"] * m["vdim"], D, 1.5)
+        lin(q + "o", D, m["heads"] * m["vdim"])
+        if f is not None:
+            vec(p + "norm2", D, 1.0)
+            lin(p + "mlp.up", f["ff"], D, 1.5)
+            lin(p + "mlp.down", D, f["ff"])
+            vec(p + "mlp.act", 2, 0.3, 0.7)
+        lin(p + "side.gate", n, D, 1.5)
+        lin(p + "side.proj", D, n)
+        vec(p + "side.norm", D, 0.8)
+    vec("final.norm", D, 1.0)
+    lin("head", cfg["vocab"], D, 4.0)
+    return out
