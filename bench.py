@@ -68,7 +68,7 @@ def parse():
                    help="instead of the headline workload: prefill, decode and kernel rooflines of a layer-by-layer decoder beside a "
                         "grouped-query model of equal size (one GPU, JSON lines; --layers, default 12 layer runs)")
     p.add_argument("--layered-model", default="nopelorn-4B-shape")
-    p.add_argument("--layered-baseline", default=None, help="default: qwen3-4B, or qwen3-30B-A3B for a model with routed experts")
+    p.add_argument("--layered-baseline", default=None, help="default: qwen3-4B, qwen3-30B-A3B for a model with routed experts, nopelorn-4B-shape for one with delta-rule layers")
     return p.parse_args()
 
 

@@ -1,11 +1,11 @@
-"""Prefill and decode of a layer-by-layer decoder beside the closest grouped-query model of equal width, depth and feed-forward.
+"""Prefill and decode of a layer-by-layer decoder beside the closest other model of equal width, depth and feed-forward.
 
     python bench.py --layered [--layered-model NAME] [--layered-baseline NAME] [--layers N]
 
-NAME: nopelorn-4B-shape, ronupel-30B-A3B-shape or vozirax-30B-A3B-shape.
+NAME: nopelorn-4B-shape, ronupel-30B-A3B-shape, vozirax-30B-A3B-shape or senadra-4B-shape.
 
 The baseline is qwen3-4B for a dense model and qwen3-30B-A3B for one with routed experts, with as many layers as the layered model has
-layer runs.
+layer runs; nopelorn-4B-shape (latent and linear attention) for a model with delta-rule layers.
 
 Random weights, synthetic tokens.  `throughput`: whole models through the engine (device-timed forwards and decode graphs).
 `kernels`: the mixers' kernels one by one at the same sizes with their distance from the measured roofline, next to the kernels
@@ -513,6 +513,159 @@ def hybrid_kernels(cfg, base) -> list[dict]:
     return out.rows
 
 
+@torch.no_grad()
+def delta_kernels(cfg, base) -> list[dict]:
+    """Gated delta rule, chunked attention with a distance bias, gated latent attention and the pre-norm arrangement's row-wise kernels beside
+    those of a model with latent and linear attention (`base`)."""
+    from ..models.layered import AttentionSpec, DeltaSpec, LatentSpec, LinearStateSpec
+    from ..ops import cuda as K
+    from ..ops import mixers as MX
+    from ..ops import mixers_cuda as MC
+
+    out = _Rows()
+    add, t = out.add, _randn
+    D, ff = cfg.hidden_size, next(s.mlp.ff for s in cfg.layer_specs if s.mlp is not None)
+
+    def first(c, kind):
+        return next(s.mixer for s in c.layer_specs if isinstance(s.mixer, kind))
+
+    m, a, l, lin, wl = first(cfg, DeltaSpec), first(cfg, AttentionSpec), first(cfg, LatentSpec), first(base, LinearStateSpec), first(base, LatentSpec)
+    ds = MX.DeltaLayout(m.heads, m.kv_heads, m.dim, m.vdim, m.conv, m.decay_rank, m.gate_rank)
+    al = MX.AttentionLayout(a.heads, a.kv_heads, a.dim, a.vdim, 0, 0, 0, a.chunk, True, True)
+    pitch = -(-a.dim // 64) * 64
+    asz = [a.heads, a.kv_heads, a.dim, a.vdim, 0, 0, 0, pitch, a.chunk]
+    H, G, err = a.heads, a.kv_heads, K.C.error_flag(torch.empty(0, device="cuda"))
+    r1, r2, sink = torch.rand(H, device="cuda").bfloat16(), torch.rand(H, device="cuda").bfloat16(), t(wl.heads)
+
+    def latent_sizes(s):
+        y = MX.LatentLayout(s.heads, s.dim, s.rot_dim, s.vdim, s.kv_rank)
+        return y, [y.heads, y.dim, y.rot, y.vdim, y.rank, y.rank_p, y.pitch]
+
+    conv, A, dtb, nv = t(ds.channels, m.conv), t(m.heads) - 2, t(m.heads * m.dim) - 2, t(m.vdim)
+    S = [m.heads, m.kv_heads, m.dim, m.vdim, m.conv, ds.beta_at]
+    n_state = m.heads * m.dim * m.vdim
+    for n, length in ((1, 8192), (8, 1024), (1, 1024)):
+        T, shape = n * length, f"{n}x{length}"
+        meta, nb = _ragged([(0, length)] * n)
+        proj, act, raw, gate, y = t(T, ds.beta_at + m.heads), t(T, ds.channels), t(T, m.heads * m.dim), t(T, m.heads * m.vdim), t(T, m.heads * m.vdim)
+        state, ring = torch.zeros(n, m.heads, m.dim, m.vdim, device="cuda"), torch.zeros(n, m.conv, ds.channels, device="cuda")
+        w = [conv, A, dtb, state, ring, meta.state_slots, meta.positions, raw]
+        rounds = MC._chunk_rounds(meta, ds)
+        scratch = torch.empty(max(c.shape[0] for c, _ in rounds) * m.heads * K.C.delta_chunk_bytes(m.dim, m.vdim), dtype=torch.uint8, device="cuda")
+
+        def chunks():
+            for c, p in rounds:
+                K.C.delta_chunk(proj, act, S, w, c, p, scratch, MC.scan_warps(p.shape[0] * m.heads, m.vdim), y, err)
+
+        C = 64
+        # the mathematics in chunks: two triangles of key products, the triangular solve on values and keys, three products with the state
+        flops = 2.0 * T * m.heads * ((C + 1) / 2 * (2 * m.dim + (m.dim + m.vdim) + m.vdim) + 3 * m.dim * m.vdim)
+        add("delta_chunk (decays, triangles, scan)", "linear_chunk", shape, chunks, 2 * T * (ds.channels + m.heads * (m.dim + 1 + m.vdim)) + 8 * state.numel(), flops)
+        lp, dec = t(T, lin.heads * 2 * (lin.dim + lin.vdim)), torch.tensor(lin.decay, device="cuda")
+        ls = torch.zeros(n, lin.heads, lin.dim, lin.vdim, device="cuda")
+        add("linear_chunk (segments + scan + outputs)", "", shape, lambda: MC.linear_state(lp, lin.heads, lin.dim, lin.vdim, dec, ls, meta),
+            2 * T * lin.heads * (2 * lin.dim + 2 * lin.vdim) + 8 * ls.numel(), 2.0 * T * lin.heads * ((C + 1) / 2 * (lin.dim + lin.vdim) + 2 * lin.dim * lin.vdim))
+        tiles = MC._conv_tiles(meta, m.conv)
+        add("delta_conv", "swiglu", shape, lambda: K.C.delta_conv(proj, S, w, tiles, meta.ragged.cu_q, act), 4 * T * ds.channels)
+        h = t(T, 2 * ds.channels)
+        add("swiglu", "", shape, lambda: K.swiglu(h), 6 * T * ds.channels)
+        g2 = torch.empty_like(y)
+        add("head_gated_norm", "gated_norm", shape, lambda: K.C.head_gated_norm(y, nv, gate, g2, 1e-6), 6 * y.numel())
+        gw = t(m.heads * m.vdim)
+        add("gated_norm", "", shape, lambda: K.C.gated_norm(y, gw, gate, g2, 1e-6), 6 * y.numel())
+        del proj, act, raw, scratch, lp, h
+        q, kc, vc, o, og = t(T, H, pitch), t(nb, 64, G, a.dim), t(nb, 64, G, a.vdim), t(T, H * a.vdim), t(T, H * a.vdim)
+        pairs = n * sum(i % a.chunk + 1 for i in range(length))
+        add(f"window_prefill (chunks of {a.chunk}, distance bias, gate)", "flash_fwd_tc", shape,
+            lambda: K.C.window_prefill(q, kc, vc, o, None, meta.ragged.cu_q, meta.positions, meta.block_table, n, length, T, a.scale, asz, err, r1=r1, r2=r2, out_gate=og),
+            2 * (q.numel() + kc.numel() + vc.numel() + 2 * o.numel()), 2.0 * pairs * H * (a.dim + a.vdim))
+        q2, k2, v2 = t(T, H, a.dim), t(T, G, a.dim), t(T, G, a.vdim)
+        add("flash_fwd_tc", "", shape, lambda: K.attention_varlen(q2, k2, v2, meta.ragged.cu_q, length), 2 * (2 * q2.numel() + 2 * k2.numel()),
+            2.0 * n * length * (length + 1) / 2 * H * 2 * a.dim)
+        del q, kc, vc, o, og, q2, k2, v2
+        for name, s, like in (("latent_prefill (all keys, gate)", l, "latent_prefill of the other model"), ("latent_prefill of the other model (window, sink)", wl, "")):
+            y_, sz = latent_sizes(s)
+            cu_k, _, total, max_q = MC._key_ranges(meta, s.window)
+            q, kv, lt, o, og = t(T, s.heads, (s.dim + 63) // 64 * 64 + 64), t(total, s.heads * (s.dim + s.vdim)), t(total, y_.pitch), t(T, s.heads, s.vdim), t(T, s.heads * s.vdim)
+            wn = s.window or length
+            pairs = n * sum(min(i + 1, wn) for i in range(length))
+            add(name, like, shape, lambda: K.C.latent_prefill(q, kv, lt, o, sink if s.sink else None, meta.ragged.cu_q, cu_k, n, max_q, s.scale, s.window, sz, err,
+                                                              og if s.gate else None),
+                2 * (q.numel() + kv.numel() + total * s.rot_dim + o.numel() * (2 if s.gate else 1)), 2.0 * pairs * s.heads * (s.dim + s.rot_dim + s.vdim))
+            del q, kv, lt, o, og
+    for B, ctx in ((1, 4096), (8, 4096), (64, 4096)):
+        shape = f"{B} rows"
+        meta, nb = _ragged([(ctx - 1, 1)] * B)
+        proj, raw, gate, y = t(B, ds.beta_at + m.heads), t(B, m.heads * m.dim), t(B, m.heads * m.vdim), t(B, m.heads * m.vdim)
+        state, ring = torch.zeros(B, m.heads, m.dim, m.vdim, device="cuda"), torch.zeros(B, m.conv, ds.channels, device="cuda")
+        w = [conv, A, dtb, state, ring, meta.state_slots, meta.positions, raw]
+        add("delta_step (convolution, state, gated norm)", "linear_state step", shape, lambda: K.C.delta_step(proj, S, w, nv, gate, 1e-6, y),
+            8 * state.numel() + 4 * ring.numel() + 2 * B * (ds.channels + m.heads * (m.dim + 2 * m.vdim)))
+        lp, dec = t(B, lin.heads * 2 * (lin.dim + lin.vdim)), torch.tensor(lin.decay, device="cuda")
+        ls = torch.zeros(B, lin.heads, lin.dim, lin.vdim, device="cuda")
+        add("linear_state step", "", shape, lambda: MC.linear_state(lp, lin.heads, lin.dim, lin.vdim, dec, ls, meta), 8 * ls.numel() + 2 * B * lin.heads * 2 * (lin.dim + lin.vdim))
+        del state, ring, ls
+        q, kc, vc, o, og = t(B, H, pitch), t(nb, 64, G, a.dim), t(nb, 64, G, a.vdim), t(B, H * a.vdim), t(B, H * a.vdim)
+        keys = (ctx - 1) % a.chunk + 1
+        add("window_decode (chunk, distance bias, gate)", "paged_decode", f"{shape}, {keys} keys",
+            lambda: K.C.window_decode(q, kc, vc, meta.block_table, None, meta.positions, meta.slot_mapping, None, o, a.scale, MC.window_splits(B, al), asz, r1=r1,
+                                      r2=r2, out_gate=og), 2 * B * (keys * G * (a.dim + a.vdim) + H * (a.dim + 2 * a.vdim)), 2.0 * B * keys * H * (a.dim + a.vdim))
+        L, q2 = torch.full((B,), keys, dtype=torch.int32, device="cuda"), t(B, H, a.dim)
+        add("paged_decode + merge", "", f"{shape}, {keys} keys", lambda: K.paged_attention(q2, kc, vc, meta.block_table, L),
+            2 * B * (keys * G * (a.dim + a.vdim) + H * (a.dim + a.vdim)), 2.0 * B * keys * H * (a.dim + a.vdim))
+        del kc, vc
+        for name, s, like in (("latent_decode + merge (all keys)", l, "latent_decode of the other model"), ("latent_decode of the other model (window, sink) + merge", wl, "")):
+            y_, sz = latent_sizes(s)
+            cache, qa, ol = t(nb, 64, y_.pitch), t(B, s.heads, y_.pitch), t(B, s.heads, y_.rank)
+            wn = min(s.window or ctx, ctx)
+            splits = MC.decode_splits(B, s.heads, s.window, 64)
+            po, pm = torch.empty(B * s.heads * splits * y_.rank_p, device="cuda"), torch.empty(B * s.heads * splits * 2, device="cuda")
+            add(name, like, f"{shape}, {wn} keys",
+                lambda: K.C.latent_decode(qa, cache, meta.block_table, None, meta.positions, meta.slot_mapping, sink if s.sink else None, po, pm, ol, s.scale, s.window,
+                                          splits, sz, err),
+                2 * B * (wn * (y_.rank + y_.rot) + s.heads * (y_.pitch + y_.rank)), 2.0 * B * wn * s.heads * (2 * y_.rank + y_.rot))
+            del cache
+        wv, ov, gv = t(l.heads, l.vdim, l.kv_rank), t(B, l.heads, l.vdim), t(B, l.heads * l.vdim)
+        add("head_linear (value up-projection, gate)", "head_linear", shape, lambda: K.C.head_linear_mma(ol, wv, True, ov, gv), 2 * (wv.numel() + ol.numel() + 2 * ov.numel()))
+        add("head_linear", "", shape, lambda: K.C.head_linear_mma(ol, wv, True, ov), 2 * (wv.numel() + ol.numel() + ov.numel()))
+    side, nw = cfg.token_side, t(D)
+    table = t(4096, cfg.num_layers * side)
+    for T in (8, 8192):
+        shape = f"{T} rows"
+        meta, nb = _ragged([(0, T)] if T > 8 else [(4000, 1)] * T)
+        x, y, r2_ = t(T, D, dtype=torch.float32), t(T, D), t(T, D)
+        add("residual_norm (factor, next norm)", "add_rmsnorm", shape, lambda: MC.residual_norm(x, y, None, 0.4, nw, 1e-6, torch.bfloat16), T * D * 12)
+        add("residual_norm (normed addend, next norm)", "add_rmsnorm", shape, lambda: MC.residual_norm(x, y, nw, 0.4, nw, 1e-6, torch.bfloat16), T * D * 12)
+        add("residual_norm (copy for the token input)", "add_rmsnorm", shape, lambda: MC.residual_norm(x, y, None, 0.4, None, 1e-6, torch.bfloat16), T * D * 12)
+        add("add_rmsnorm", "", shape, lambda: K.add_rmsnorm(y, r2_, nw, 1e-6), T * D * 8)
+        h, act2 = t(T, ff), t(2)
+        add("xielu", "swiglu", shape, lambda: MC.xielu(h, act2), 4 * T * ff)
+        h2 = t(T, 2 * ff)
+        add("swiglu", "", shape, lambda: K.swiglu(h2), 6 * T * ff)
+        z, tok = t(T, side), torch.randint(0, 4096, (T,), dtype=torch.int32, device="cuda")
+        add("gelu_rows", "swiglu", shape, lambda: MC.gelu_times_rows(z, tok, table, side), 6 * T * side)
+        h3 = t(T, 2 * side)
+        add("swiglu", "", f"{shape} of {side}", lambda: K.swiglu(h3), 6 * T * side)
+        proj, q = t(T, al.rows + H * a.vdim), t(T, H, pitch)
+        kc, vc = t(nb, 64, G, a.dim), t(nb, 64, G, a.vdim)
+        freq = torch.zeros(0, dtype=torch.float64, device="cuda")
+        add("window_prep (value norm, cache)", "qk_norm_rope_cache", shape,
+            lambda: K.C.window_prep(proj, meta.positions, meta.slot_mapping, freq, 1.0, None, None, 1e-6, kc, vc, q, asz, *MC._aside(None, T), True),
+            2 * T * (al.rows + H * a.dim + G * (a.dim + a.vdim)))
+        q2, k2, v2, qw = t(T, H, a.dim), t(T, G, a.dim), t(T, G, a.vdim), t(a.dim)
+        add("qk_norm_rope_cache", "", shape, lambda: K.qk_norm_rope_cache(q2, k2, v2, qw, qw, meta.positions, 1e6, 1e-6, kc, vc, meta.slot_mapping),
+            2 * (2 * q2.numel() + 5 * k2.numel()))
+    w1 = torch.nn.Parameter(t(ds.beta_at + m.heads, D))
+    for T in (1, 4):
+        x, y, r2_ = t(T, D, dtype=torch.float32), t(T, D), t(T, D)
+        for name, yn, n2 in (("factor, norm", None, nw), ("normed addend, norm", nw, nw), ("factor, no norm", None, None)):
+            add(f"residual_linear ({name})", "add_rmsnorm_linear", f"{T} rows", lambda: MC.residual_linear(x, y, yn, 0.4, n2, 1e-6, w1), 2 * w1.numel())
+        add("add_rmsnorm_linear", "", f"{T} rows", lambda: K.add_rmsnorm_linear(y, r2_, nw, 1e-6, w1), 2 * w1.numel())
+    lg = t(64, cfg.vocab_size, dtype=torch.float32)
+    add("softcap (64 rows of logits)", "swiglu", "64 rows", lambda: MC.softcap_(lg, 30.0, False), 8 * lg.numel())
+    return out.rows
+
+
 def main(a) -> int:
     from ..models.config import get_config
     from ..ops import build
@@ -521,14 +674,15 @@ def main(a) -> int:
     torch.cuda.set_device(0)
     cfg = get_config(a.layered_model)
     moe = cfg.num_moe_layers > 0
-    base = get_config(a.layered_baseline or ("qwen3-30B-A3B" if moe else "qwen3-4B"))
+    parts = build.serve_kind(cfg).split("_")
+    base = get_config(a.layered_baseline or ("qwen3-30B-A3B" if moe else "nopelorn-4B-shape" if "delta" in parts else "qwen3-4B"))
     cfg = cfg.with_(num_layers=a.layers or (8 if moe else 12))
-    base = base.with_(num_layers=len(cfg.runs()))
+    base = base.with_(num_layers=len(cfg.runs()))      # (a layered baseline keeps its first layers)
     for c in (cfg, base):
         print(json.dumps(throughput(c)), flush=True)
         torch.cuda.empty_cache()
-    kinds = {"attention": attention_kernels, "latent": latent_kernels, "hybrid": hybrid_kernels}
-    for r in kinds[build.serve_kind(cfg)](cfg, base):
+    kinds = {"delta": delta_kernels, "ssm": hybrid_kernels, "linear": latent_kernels, "attention": attention_kernels}
+    for r in next(f for part, f in kinds.items() if part in parts)(cfg, base):
         print(json.dumps(r), flush=True)
     print(json.dumps({"kernel_error_flag": K.check_error_flag()}))
     return 0

@@ -565,7 +565,7 @@ void delta_chunk(const at::Tensor& proj, const at::Tensor& act, const std::vecto
   TORCH_CHECK(scratch.nbytes() >= static_cast<size_t>(mb_delta_chunk_bytes(m.K, m.V)) * chunks.size(0) * m.H, "delta_chunk: scratch too small");
   mb_count_launch(1);
   check(mb_delta_chunk(proj.data_ptr(), proj.stride(0), act.data_ptr(), m, chunks.data_ptr<int>(), parts.data_ptr<int>(), scratch.data_ptr(),
-                       out.data_ptr(), chunks.size(0), parts.size(0), warps, err.data_ptr<int>(), cur_stream()),
+                       out.data_ptr(), proj.size(0), chunks.size(0), parts.size(0), warps, err.data_ptr<int>(), cur_stream()),
         "mb_delta_chunk");
 }
 

@@ -17,11 +17,14 @@
 #include "ptx.cuh"
 
 namespace mb {
+
+int make_tmap_bf16_2d(CUtensorMap* out, const void* base, long long rows, long long cols, long long ld, int box_rows, int box_cols);
+
 namespace dc {
 
 using mx::bf16;
 static constexpr int C = 64, kThreads = 512;
-static constexpr int P = 136, LP = 132, AP = 68;      // shared rows: bf16 tiles (≤ 128 wide), floats per channel, floats per token
+static constexpr int P = 136, LP = 132, AP = 72, DP = 20;      // shared rows: bf16 tiles (≤ 128 wide), floats per channel, bf16 per token, floats of a diagonal block
 static constexpr int kTile = C * P;
 static constexpr float kLog2e = 1.4426950408889634f, kFar = -100.f;
 static constexpr int kUPitch = 288;                   // bytes of a row of U (64 floats and padding)
@@ -105,69 +108,131 @@ struct Args {
 struct Shared {
   bf16 q_hi[kTile], q_lo[kTile], k_hi[kTile], k_lo[kTile], c_hi[kTile], c_lo[kTile], v[kTile];
   float L[C * LP];           // log2 of the decays, summed from the start of a token's block
-  float A[C * AP];
+  bf16 a_hi[C * AP], a_lo[C * AP];         // A below its diagonal blocks, their inverses T in these
+  float diagonal[4][16 * DP];              // A inside them
   float D[4][128], before[4][128], after[4][128], between[7][128];
-  float fq[C], fk[C], beta[C];
-  int direct[4];
+  float fq[C], fk[C], beta[C], beta_k[C];
+  int direct[4], next;
+  uint64_t full;             // the inputs of a unit have come
 };
 
-// (row block, column block) of the pairs whose columns take a factor: those with blocks between them, and the diagonal ones
+// Pairs of blocks i: the diagonal ones, those with blocks between them, neighbours.  The first seven have a factor on the columns, between[i].
 __device__ __forceinline__ void pair_of(int i, int& a, int& b) {
-  a = i < 3 ? (i == 0 ? 2 : 3) : i - 3;
-  b = i < 3 ? (i == 2 ? 1 : 0) : i - 3;
+  a = i < 4 ? i : i < 7 ? (i == 4 ? 2 : 3) : i - 6;
+  b = i < 4 ? i : i < 7 ? (i == 6 ? 1 : 0) : i - 7;
 }
 
-// grid (heads, chunks)
-__global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(Args p) {
-  extern __shared__ __align__(128) uint8_t smem[];
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+// 1 / √x: the approximation and one Newton step, good to the last bits
+__device__ __forceinline__ float inv_sqrt(float x) {
+  const float y = rsqrtf(x);
+  return y * fmaf(-0.5f * x, y * y, 1.5f);
+}
+
+// A CTA per SM takes every gridDim.x-th (chunk, head).  The inputs of the next one come by TMA while the products of the last phase run, into
+// tiles that are free by then: boxes of 64 tokens × 64 columns (128-byte swizzle), q and v over q_hi and q_lo, k and what decays come from
+// over c_hi and c_lo.  Rows behind the chunk and columns behind the head are whatever lies there: they count as zeros.
+__global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(const __grid_constant__ CUtensorMap tm_act, const __grid_constant__ CUtensorMap tm_raw,
+                                                                    Args p, int n_units) {
+  extern __shared__ __align__(1024) uint8_t smem[];
   Shared& s = *reinterpret_cast<Shared*>(smem);
-  pdl_trigger();
-  pdl_wait();
-  const int h = blockIdx.x, H = p.m.H, K = p.m.K, V = p.m.V, gq = h / (H / p.m.G), CH = 2 * p.m.G * K + H * V;
-  const int4 ch = reinterpret_cast<const int4*>(p.chunks)[blockIdx.y];
-  const int t0 = ch.y, n_tok = ch.z - ch.y;
+  if (smem_u32(smem) & 1023u) {
+    if (threadIdx.x == 0) atomicExch(p.error_flag, 93);
+    return;
+  }
+  const int H = p.m.H, K = p.m.K, V = p.m.V, per = H / p.m.G, CH = 2 * p.m.G * K + H * V;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int kdk = (K + 15) / 16, kdv = (V + 15) / 16;
-  uint8_t* unit = p.scratch + (static_cast<long long>(blockIdx.y) * H + h) * p.unit.bytes();
   const int KR = p.unit.KR, half = p.unit.half();
-
-  // ---- inputs: q and k as they are (with the factors that make them unit vectors), v, log decays, β
   const float q_scale = __fdiv_rn(1.f, __fsqrt_rn(static_cast<float>(K)));
-  for (int r = warp; r < C; r += kThreads / 32) {
-    const int piece = lane & 15;
-    const bool key = lane >= 16;
-    uint4 x = make_uint4(0, 0, 0, 0);
-    if (r < n_tok && piece * 8 < K) x = *reinterpret_cast<const uint4*>(p.act + static_cast<long long>(t0 + r) * CH + (key ? p.m.G * K : 0) + gq * K + piece * 8);
-    const uint32_t w[4] = {x.x, x.y, x.z, x.w};
-    float ss = 0.f;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) ss += lo16(w[i]) * lo16(w[i]) + hi16(w[i]) * hi16(w[i]);
-#pragma unroll
-    for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const float f = mx::rsqrt_exact(ss + 1e-6f);
-    if (piece == 0) (key ? s.fk : s.fq)[r] = key ? f : f * q_scale;
-    *reinterpret_cast<uint4*>((key ? s.k_hi : s.q_hi) + r * P + piece * 8) = x;
+  const int my_row = tid >> 4, my_c = (tid & 15) * 8;      // 8 channels of rows my_row and my_row + 32
+  if (tid == 0) {
+    mbar_init(&s.full, 1);
+    mbar_fence_init();
   }
-  const float rate = __expf(__bfloat162float(reinterpret_cast<const bf16*>(p.m.A_log)[h]));
-  for (int i = tid; i < C * 16; i += kThreads) {
-    const int r = i >> 4, c = (i & 15) * 8;
-    uint4 x = make_uint4(0, 0, 0, 0);
-    if (r < n_tok && c < V) x = *reinterpret_cast<const uint4*>(p.act + static_cast<long long>(t0 + r) * CH + 2 * p.m.G * K + h * V + c);
-    *reinterpret_cast<uint4*>(s.v + r * P + c) = x;
+  pdl_trigger();
+  pdl_wait();
+  __syncthreads();
+  // what a thread keeps of the next unit: its chunk, its channels' bias, its row's β, the head's rate
+  int4 ch = reinterpret_cast<const int4*>(p.chunks)[blockIdx.x / H];
+  uint4 bias_raw = make_uint4(0, 0, 0, 0);
+  bf16 beta_raw = __float2bfloat16(0.f), a_raw = __float2bfloat16(0.f);
+  uint8_t* in_q = reinterpret_cast<uint8_t*>(s.q_hi);      // [q | v], then [k | raw]: two boxes each
+  uint8_t* in_k = reinterpret_cast<uint8_t*>(s.c_hi);
+  auto fetch = [&](int idx) {
+    const int h = idx % H, gq = h / per;
+    if (tid == 0) {
+      const int na = (K + 63) / 64, nv = (V + 63) / 64;
+      mbar_expect_tx(&s.full, (3 * na + nv) * 8192);
+      for (int i = 0; i < na; ++i) {
+        tma_load_2d(in_q + i * 8192, &tm_act, &s.full, gq * K + i * 64, ch.y);
+        tma_load_2d(in_k + i * 8192, &tm_act, &s.full, (p.m.G + gq) * K + i * 64, ch.y);
+        tma_load_2d(in_k + 16384 + i * 8192, &tm_raw, &s.full, h * K + i * 64, ch.y);
+      }
+      for (int i = 0; i < nv; ++i) tma_load_2d(in_q + 16384 + i * 8192, &tm_act, &s.full, 2 * p.m.G * K + h * V + i * 64, ch.y);
+    }
+    if (my_c < K) bias_raw = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.m.dt_bias) + h * K + my_c);
+    a_raw = reinterpret_cast<const bf16*>(p.m.A_log)[h];
+    if (tid < ch.z - ch.y) beta_raw = p.proj[(ch.y + tid) * p.ld + p.m.beta_at + h];      // (at most 64 tokens)
+  };
+  fetch(blockIdx.x);
+  uint32_t phase = 0;
+  for (int idx = blockIdx.x; idx < n_units; idx += gridDim.x) {
+  const int h = idx % H, gq = h / per, t0_now = ch.y, n_now = ch.z - ch.y, after_idx = idx + gridDim.x;
+  if (after_idx < n_units) ch = reinterpret_cast<const int4*>(p.chunks)[after_idx / H];
+  uint8_t* unit = p.scratch + static_cast<long long>(idx) * p.unit.bytes();
+  if (!mbar_wait(&s.full, phase)) {
+    atomicExch(p.error_flag, 92);
+    return;
+  }
+  phase ^= 1;
+  __syncthreads();
+  // ---- q and k with the factors that make unit vectors of them, v into its place, log decays, β
+  uint4 q_in[2], k_in[2];
+  const float rate = __expf(__bfloat162float(a_raw));
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = my_row + i * 32, at = r * P + my_c;
+    const int from = (my_c >> 6) * 8192 + r * 128 + ((((my_c >> 3) & 7) ^ (r & 7)) << 4);
+    const bool ok = r < n_now && my_c < K;
+    uint4 v = make_uint4(0, 0, 0, 0), x = make_uint4(0, 0, 0, 0);
+    q_in[i] = k_in[i] = v;
+    if (ok) {
+      q_in[i] = *reinterpret_cast<const uint4*>(in_q + from);
+      k_in[i] = *reinterpret_cast<const uint4*>(in_k + from);
+      x = *reinterpret_cast<const uint4*>(in_k + 16384 + from);
+    }
+    if (r < n_now && my_c < V) v = *reinterpret_cast<const uint4*>(in_q + 16384 + from);
+    *reinterpret_cast<uint4*>(s.v + at) = v;
+    const uint32_t qw[4] = {q_in[i].x, q_in[i].y, q_in[i].z, q_in[i].w}, kw[4] = {k_in[i].x, k_in[i].y, k_in[i].z, k_in[i].w};
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      sq += lo16(qw[j]) * lo16(qw[j]) + hi16(qw[j]) * hi16(qw[j]);
+      sk += lo16(kw[j]) * lo16(kw[j]) + hi16(kw[j]) * hi16(kw[j]);
+    }
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) {    // a row's 16 threads are half a warp
+      sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      sk += __shfl_xor_sync(0xffffffffu, sk, o);
+    }
+    if (my_c == 0) {
+      s.fq[r] = inv_sqrt(sq + 1e-6f) * q_scale;
+      s.fk[r] = inv_sqrt(sk + 1e-6f);
+    }
+    const uint32_t xw[4] = {x.x, x.y, x.z, x.w}, bw[4] = {bias_raw.x, bias_raw.y, bias_raw.z, bias_raw.w};
     float l[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) l[j] = 0.f;
-    if (r < n_tok && c < K) {
-      float bias[8];
-      mx::load_n<8>(reinterpret_cast<const bf16*>(p.m.raw) + (t0 + r) * p.m.raw_ld + h * K + c, l);
-      mx::load_n<8>(reinterpret_cast<const bf16*>(p.m.dt_bias) + h * K + c, bias);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) l[j] = -rate * softplus2(l[j] + bias[j]);
-    }
-    mx::store_n<8>(s.L + r * LP + c, l);
+    for (int j = 0; j < 8; ++j)
+      l[j] = ok ? -rate * softplus2((j & 1) ? hi16(xw[j / 2]) + hi16(bw[j / 2]) : lo16(xw[j / 2]) + lo16(bw[j / 2])) : 0.f;
+    mx::store_n<8>(s.L + r * LP + my_c, l);
   }
-  if (tid < C) s.beta[tid] = tid < n_tok ? mx::sigmoid_t<bf16>(__bfloat162float(p.proj[(t0 + tid) * p.ld + p.m.beta_at + h])) : 0.f;
+  if (tid < C) s.beta[tid] = tid < n_now ? mx::sigmoid_t<bf16>(__bfloat162float(beta_raw)) : 0.f;
   if (tid < 4) s.direct[tid] = 0;
+  if (tid == 4) s.next = 0;
   __syncthreads();
   {                                      // running sums inside the blocks: a thread per (block, channel)
     const int b = tid >> 7, c = tid & 127;
@@ -192,22 +257,30 @@ __global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(Args p) {
     s.after[1][tid] = e2(d2 + d3);
     s.after[2][tid] = e2(d3);
     s.after[3][tid] = 1.f;
-    s.between[0][tid] = e2(d1);
-    s.between[1][tid] = e2(d1 + d2);
-    s.between[2][tid] = e2(d2);
-    s.between[3][tid] = e2(fminf(-d0, -kFar));           // blocks beyond are summed directly
-    s.between[4][tid] = e2(fminf(-d1, -kFar));
-    s.between[5][tid] = e2(fminf(-d2, -kFar));
-    s.between[6][tid] = e2(fminf(-d3, -kFar));
+    s.between[0][tid] = e2(fminf(-d0, -kFar));           // blocks beyond are summed directly
+    s.between[1][tid] = e2(fminf(-d1, -kFar));
+    s.between[2][tid] = e2(fminf(-d2, -kFar));
+    s.between[3][tid] = e2(fminf(-d3, -kFar));
+    s.between[4][tid] = e2(d1);
+    s.between[5][tid] = e2(d1 + d2);
+    s.between[6][tid] = e2(d2);
     reinterpret_cast<float*>(unit + p.unit.decay())[tid] = e2(d0 + d1 + d2 + d3);
+  } else if (tid < 128 + C) {
+    s.beta_k[tid - 128] = s.beta[tid - 128] * s.fk[tid - 128];
   }
-  // ---- q and k decayed from the start of their block, k to its end
-  for (int i = tid; i < C * 16; i += kThreads) {
-    const int r = i >> 4, c = (i & 15) * 8, at = r * P + c;
+  __syncthreads();
+  // ---- q and k decayed from the start of their block, k to its end; queries decayed from the chunk's start
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = my_row + i * 32, c = my_c, at = r * P + c;
     float q[8], k[8], l[8], d[8], x[8];
     uint4 hi, lo;
-    mx::load_n<8>(s.q_hi + at, q);
-    mx::load_n<8>(s.k_hi + at, k);
+    const uint32_t qw[4] = {q_in[i].x, q_in[i].y, q_in[i].z, q_in[i].w}, kw[4] = {k_in[i].x, k_in[i].y, k_in[i].z, k_in[i].w};
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      q[j] = (j & 1) ? hi16(qw[j / 2]) : lo16(qw[j / 2]);
+      k[j] = (j & 1) ? hi16(kw[j / 2]) : lo16(kw[j / 2]);
+    }
     mx::load_n<8>(s.L + r * LP + c, l);
     mx::load_n<8>(s.D[r >> 4] + c, d);
 #pragma unroll
@@ -219,6 +292,17 @@ __global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(Args p) {
     split8(x, hi, lo);
     *reinterpret_cast<uint4*>(s.q_hi + at) = hi;
     *reinterpret_cast<uint4*>(s.q_lo + at) = lo;
+    if (c < kdk * 16) {
+      float f[8];
+      mx::load_n<8>(s.before[r >> 4] + c, f);
+      const float scale = s.fq[r];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[j] *= f[j] * scale;
+      split8(x, hi, lo);
+      uint8_t* to = unit + p.unit.q() + r * KR * 2 + (((c >> 3) ^ (r & 7)) << 4);
+      *reinterpret_cast<uint4*>(to) = hi;
+      *reinterpret_cast<uint4*>(to + half) = lo;
+    }
 #pragma unroll
     for (int j = 0; j < 8; ++j) x[j] = k[j] * l[j];
     split8(x, hi, lo);
@@ -229,181 +313,288 @@ __global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(Args p) {
     *reinterpret_cast<uint4*>(s.c_lo + at) = lo;
   }
   __syncthreads();
-  // ---- A and B, a warp per (pair of blocks, 8 columns): 14 units with a factor on the columns, 6 of neighbouring blocks without
-  for (int round = 0; round < (warp < 14 ? 1 : 3); ++round) {
+  // ---- A and B, a warp per pair of blocks; the diagonal blocks of I + A are inverted by the warps that made them
+  if (warp < 10) {
     int a, b;
-    const int n = warp < 14 ? warp & 1 : warp - 14;
-    if (warp < 14) pair_of(warp >> 1, a, b);
-    else { a = round + 1; b = round; }
-    const float* fac = warp < 14 ? s.between[warp >> 1] : nullptr;
-    float kk[4] = {0.f, 0.f, 0.f, 0.f}, qk[4] = {0.f, 0.f, 0.f, 0.f};
+    pair_of(warp, a, b);
+    float kk[2][4] = {}, qk[2][4] = {}, kk1[2][4] = {}, qk1[2][4] = {};      // (the products with low parts have sums of their own)
     if (a == b && s.direct[a]) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int i = a * 16 + g + (e >> 1) * 8, j = a * 16 + n * 8 + t4 * 2 + (e & 1);
-        if (j > i || i >= n_tok) continue;
-        const bf16* qi = p.act + static_cast<long long>(t0 + i) * CH + gq * K;
-        const bf16* ki = qi + p.m.G * K;
-        const bf16* kj = p.act + static_cast<long long>(t0 + j) * CH + p.m.G * K + gq * K;
-        for (int c = 0; c < K; ++c) {
-          const float x = __bfloat162float(kj[c]) * e2(s.L[i * LP + c] - s.L[j * LP + c]);
-          kk[e] = fmaf(__bfloat162float(ki[c]), x, kk[e]);
-          qk[e] = fmaf(__bfloat162float(qi[c]), x, qk[e]);
+#pragma unroll 1
+      for (int x = 0; x < 8; ++x) {
+        const int i = a * 16 + g + (x & 2) * 4, j = a * 16 + (x >> 2) * 8 + t4 * 2 + (x & 1);
+        float sk = 0.f, sq = 0.f;
+        if (j <= i && i < n_now) {
+          const bf16* qi = p.act + static_cast<long long>(t0_now + i) * CH + gq * K;
+          const bf16* ki = qi + p.m.G * K;
+          const bf16* kj = p.act + static_cast<long long>(t0_now + j) * CH + p.m.G * K + gq * K;
+          for (int c = 0; c < K; ++c) {
+            const float w = __bfloat162float(kj[c]) * e2(s.L[i * LP + c] - s.L[j * LP + c]);
+            sk = fmaf(__bfloat162float(ki[c]), w, sk);
+            sq = fmaf(__bfloat162float(qi[c]), w, sq);
+          }
         }
+#pragma unroll
+        for (int y = 0; y < 8; ++y)
+          if (y == x) { kk[y >> 2][y & 3] = sk; qk[y >> 2][y & 3] = sq; }
       }
       __syncwarp();
     } else {
       const int row_a = (a * 16 + (lane & 15)) * P + (lane >> 4) * 8;
-      const uint32_t b_at = smem_u32((lane < 16 ? s.c_hi : s.c_lo) + (b * 16 + n * 8 + (lane & 7)) * P + ((lane >> 3) & 1) * 8);
+      const int row_b = (b * 16 + (lane & 7) + ((lane >> 4) << 3)) * P + ((lane >> 3) & 1) * 8;
+      const float* fac = s.between[min(warp, 6)];
+#pragma unroll 2
       for (int ks = 0; ks < kdk; ++ks) {
-        uint32_t qh[4], ql[4], kh[4], kl[4], c[4];
-        ldsm4(b_at + ks * 32, c);                        // hi: c[0], c[1]; lo: c[2], c[3]
+        uint32_t qh[4], ql[4], kh[4], kl[4], ch[4], cl[4];
+        ldsm4(smem_u32(s.c_hi + row_b + ks * 16), ch);
+        ldsm4(smem_u32(s.c_lo + row_b + ks * 16), cl);
         ldsm4(smem_u32(s.k_hi + row_a + ks * 16), kh);
-        ldsm4(smem_u32(s.k_lo + row_a + ks * 16), kl);
         ldsm4(smem_u32(s.q_hi + row_a + ks * 16), qh);
+        ldsm4(smem_u32(s.k_lo + row_a + ks * 16), kl);
         ldsm4(smem_u32(s.q_lo + row_a + ks * 16), ql);
-        if (fac != nullptr) {
+        if (warp < 7) {
 #pragma unroll
           for (int i = 0; i < 2; ++i) {
             const float2 f = *reinterpret_cast<const float2*>(fac + ks * 16 + i * 8 + t4 * 2);
-            split2((lo16(c[i]) + lo16(c[2 + i])) * f.x, (hi16(c[i]) + hi16(c[2 + i])) * f.y, c[i], c[2 + i]);
+#pragma unroll
+            for (int n = 0; n < 4; n += 2) split2((lo16(ch[n + i]) + lo16(cl[n + i])) * f.x, (hi16(ch[n + i]) + hi16(cl[n + i])) * f.y, ch[n + i], cl[n + i]);
           }
         }
-        mma(kk, kh, c[0], c[1]);
-        mma(qk, qh, c[0], c[1]);
-        mma(kk, kh, c[2], c[3]);
-        mma(qk, qh, c[2], c[3]);
-        mma(kk, kl, c[0], c[1]);
-        mma(qk, ql, c[0], c[1]);
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          mma(kk[n], kh, ch[2 * n], ch[2 * n + 1]);
+          mma(qk[n], qh, ch[2 * n], ch[2 * n + 1]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          mma(kk1[n], kh, cl[2 * n], cl[2 * n + 1]);
+          mma(qk1[n], qh, cl[2 * n], cl[2 * n + 1]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          mma(kk1[n], kl, ch[2 * n], ch[2 * n + 1]);
+          mma(qk1[n], ql, ch[2 * n], ch[2 * n + 1]);
+        }
       }
     }
 #pragma unroll
-    for (int e = 0; e < 4; e += 2) {
-      const int i = a * 16 + g + e * 4, j = b * 16 + n * 8 + t4 * 2;
-      const float f0 = s.fk[j], f1 = s.fk[j + 1], fi = s.fk[i] * s.beta[i], fo = s.fq[i];
-      *reinterpret_cast<float2*>(s.A + i * AP + j) = make_float2(j < i ? kk[e] * fi * f0 : 0.f, j + 1 < i ? kk[e + 1] * fi * f1 : 0.f);
-      uint32_t hi, lo;
-      split2(j <= i ? qk[e] * fo * f0 : 0.f, j + 1 <= i ? qk[e + 1] * fo * f1 : 0.f, hi, lo);
-      uint8_t* at = unit + p.unit.b() + i * 128 + (((j >> 3) ^ (i & 7)) << 4) + (j & 7) * 2;
-      *reinterpret_cast<uint32_t*>(at) = hi;
-      *reinterpret_cast<uint32_t*>(at + 8192) = lo;
-    }
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        const int i = a * 16 + g + e * 4, j = b * 16 + n * 8 + t4 * 2;
+        const float k0 = kk[n][e] + kk1[n][e], k1 = kk[n][e + 1] + kk1[n][e + 1], q0 = qk[n][e] + qk1[n][e], q1 = qk[n][e + 1] + qk1[n][e + 1];
+        const float f0 = s.fk[j], f1 = s.fk[j + 1], fi = s.beta_k[i], fo = s.fq[i];
+        uint32_t hi, lo;
+        if (a == b) {
+          *reinterpret_cast<float2*>(s.diagonal[a] + (i & 15) * DP + (j & 15)) = make_float2(k0 * fi * f0, k1 * fi * f1);      // (read below its diagonal)
+        } else {
+          split2(k0 * fi * f0, k1 * fi * f1, hi, lo);
+          *reinterpret_cast<uint32_t*>(s.a_hi + i * AP + j) = hi;
+          *reinterpret_cast<uint32_t*>(s.a_lo + i * AP + j) = lo;
+        }
+        split2(j <= i ? q0 * fo * f0 : 0.f, j + 1 <= i ? q1 * fo * f1 : 0.f, hi, lo);
+        uint8_t* at = unit + p.unit.b() + i * 128 + (((j >> 3) ^ (i & 7)) << 4) + (j & 7) * 2;
+        *reinterpret_cast<uint32_t*>(at) = hi;
+        *reinterpret_cast<uint32_t*>(at + 8192) = lo;
+      }
   }
-  __syncthreads();
-  if (warp < 4) {
-    // ---- inverses of the diagonal blocks of I + A, over them: a lane per column
+  if (warp < 4) {                        // a lane per column of the inverse
+    __syncwarp();
     const int c = lane & 15;
-    float* blk = s.A + warp * 16 * AP + warp * 16;
+    const float* blk = s.diagonal[warp];
     float x[16];
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
-      float r = i == c ? 1.f : 0.f;
+      float r[4] = {i == c ? 1.f : 0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int j = 0; j < i; ++j) r = fmaf(-blk[i * AP + j], x[j], r);
-      x[i] = r;
+      for (int j = 0; j < i; j += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(blk + i * DP + j);
+        r[0] = fmaf(-a.x, x[j], r[0]);
+        if (j + 1 < i) r[1] = fmaf(-a.y, x[j + 1], r[1]);
+        if (j + 2 < i) r[2] = fmaf(-a.z, x[j + 2], r[2]);
+        if (j + 3 < i) r[3] = fmaf(-a.w, x[j + 3], r[3]);
+      }
+      x[i] = (r[0] + r[1]) + (r[2] + r[3]);
     }
-    __syncwarp();
-    if (lane < 16)
+    if (lane < 16) {
+      const int at = warp * 16 * AP + warp * 16 + c;
 #pragma unroll
-      for (int i = 0; i < 16; ++i) blk[i * AP + c] = x[i];
-  } else {
-    // ---- queries decayed from the chunk's start, keys to its end
-    for (int i = tid - 128; i < 2 * C * 16; i += kThreads - 128) {
-      const int r = (i >> 4) & (C - 1), piece = i & 15, c = piece * 8, at = r * P + c;
-      const bool key = i >= C * 16;
-      if (c >= kdk * 16) continue;
-      float x[8], y[8];
-      mx::load_n<8>((key ? s.c_hi : s.q_hi) + at, x);
-      mx::load_n<8>((key ? s.c_lo : s.q_lo) + at, y);
-      const float* f = (key ? s.after : s.before)[r >> 4] + c;
-      const float scale = key ? s.fk[r] : s.fq[r];
+      for (int i = 0; i < 16; ++i) {
+        const bf16 hi = __float2bfloat16(x[i]);
+        s.a_hi[at + i * AP] = hi;
+        s.a_lo[at + i * AP] = __float2bfloat16(x[i] - __bfloat162float(hi));
+      }
+    }
+  }
+  // ---- keys decayed to the chunk's end: two rows at a time by whichever warp has nothing else to do
+  for (;;) {
+    int turn = 0;
+    if (lane == 0) turn = atomicAdd(&s.next, 1);
+    turn = __shfl_sync(0xffffffffu, turn, 0);
+    if (turn >= C / 2) break;
+    const int r = turn * 2 + (lane >> 4), piece = lane & 15, c = piece * 8, at = r * P + c;
+    if (c < kdk * 16) {
+      float x[8], y[8], f[8];
+      mx::load_n<8>(s.c_hi + at, x);
+      mx::load_n<8>(s.c_lo + at, y);
+      mx::load_n<8>(s.after[r >> 4] + c, f);
+      const float scale = s.fk[r];
 #pragma unroll
       for (int j = 0; j < 8; ++j) x[j] = (x[j] + y[j]) * (f[j] * scale);
       uint4 hi, lo;
       split8(x, hi, lo);
-      uint8_t* to = unit + (key ? p.unit.k() : p.unit.q()) + r * KR * 2 + ((piece ^ (r & 7)) << 4);
+      uint8_t* to = unit + p.unit.k() + r * KR * 2 + ((piece ^ (r & 7)) << 4);
       *reinterpret_cast<uint4*>(to) = hi;
       *reinterpret_cast<uint4*>(to + half) = lo;
     }
   }
+  fence_proxy_async();                   // what was written to the tiles comes before the copies into them
   __syncthreads();
+  if (after_idx < n_units) fetch(after_idx);
   // ---- X = T·[β v | β k e^G] by blocks of tokens, transposed: a warp's 16 columns are the rows of its products
+  const int a_row = (lane & 7) + ((lane >> 4) << 3), a_col = ((lane >> 3) & 1) * 8;
+  const int r_row = (lane & 7) + ((lane >> 4) << 3), r_col = ((lane >> 3) & 1) * 8;
   for (int mt = warp; mt < kdv + kdk; mt += kThreads / 32) {
     const bool is_u = mt < kdv;
     const int c0 = (is_u ? mt : mt - kdv) * 16;
+    uint8_t* w_rows = reinterpret_cast<uint8_t*>(s.L) + (mt - kdv) % 8 * 4096;      // 16 rows of W, hi and lo, on their way out (the decays are not needed any more)
     uint32_t xh[4][4], xl[4][4];
 #pragma unroll
     for (int a = 0; a < 4; ++a) {
-      float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-      // rows of A (or T) are the columns of the second factor
-      auto times = [&](float (&d)[2][4], const uint32_t (&yh)[4], const uint32_t (&yl)[4], int b) {
+      float acc[2][4], acc1[2][4];
+      // rows of A (or T) are the columns of the second factor; the products with low parts have sums of their own
+      auto times = [&](const uint32_t (&yh)[4], const uint32_t (&yl)[4], int b) {
+        uint32_t bh[4], bl[4];
+        const int at = (a * 16 + a_row) * AP + b * 16 + a_col;
+        ldsm4(smem_u32(s.a_hi + at), bh);
+        ldsm4(smem_u32(s.a_lo + at), bl);
+        mma(acc[0], yh, bh[0], bh[1]);
+        mma(acc[1], yh, bh[2], bh[3]);
+        mma(acc1[0], yh, bl[0], bl[1]);
+        mma(acc1[1], yh, bl[2], bl[3]);
+        mma(acc1[0], yl, bh[0], bh[1]);
+        mma(acc1[1], yl, bh[2], bh[3]);
+      };
+      auto clear = [&]() {
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[n][e] = acc1[n][e] = 0.f;
+      };
+      auto sum = [&]() {
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[n][e] += acc1[n][e];
+      };
+      clear();
+#pragma unroll
+      for (int b = 0; b < a; ++b) times(xh[b], xl[b], b);
+      sum();
+      // the block's right-hand side, transposed on its way from shared memory: register 2n + e holds tokens 8n + 2·t4 and the next of column g + 8e
+      const int at = (a * 16 + r_row) * P + c0 + r_col;
+      if (is_u) {
+        uint32_t v[4];
+        ldsm4t(smem_u32(s.v + at), v);
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
-          const float* row = s.A + (a * 16 + n * 8 + g) * AP + b * 16 + t4 * 2;
-          const float2 u = *reinterpret_cast<const float2*>(row), v = *reinterpret_cast<const float2*>(row + 8);
-          uint32_t h0, l0, h1, l1;
-          split2(u.x, u.y, h0, l0);
-          split2(v.x, v.y, h1, l1);
-          mma(d[n], yh, h0, h1);
-          mma(d[n], yh, l0, l1);
-          mma(d[n], yl, h0, h1);
+          const float2 f = *reinterpret_cast<const float2*>(s.beta + a * 16 + n * 8 + t4 * 2);
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            acc[n][e * 2] = fmaf(lo16(v[n * 2 + e]), f.x, -acc[n][e * 2]);
+            acc[n][e * 2 + 1] = fmaf(hi16(v[n * 2 + e]), f.y, -acc[n][e * 2 + 1]);
+          }
         }
-      };
+      } else {
+        uint32_t v[4], w[4];
+        ldsm4t(smem_u32(s.k_hi + at), v);
+        ldsm4t(smem_u32(s.k_lo + at), w);
+        const float from[2] = {s.before[a][c0 + g], s.before[a][c0 + g + 8]};
 #pragma unroll
-      for (int b = 0; b < a; ++b) times(acc, xh[b], xl[b], b);
+        for (int n = 0; n < 2; ++n) {
+          const float2 f = *reinterpret_cast<const float2*>(s.beta_k + a * 16 + n * 8 + t4 * 2);
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int c = c0 + g + (e >> 1) * 8, t = a * 16 + n * 8 + t4 * 2 + (e & 1);
-          float r;
-          if (is_u) r = __bfloat162float(s.v[t * P + c]);
-          else r = (__bfloat162float(s.k_hi[t * P + c]) + __bfloat162float(s.k_lo[t * P + c])) * (s.fk[t] * s.before[a][c]);
-          acc[n][e] = fmaf(r, s.beta[t], -acc[n][e]);
+          for (int e = 0; e < 2; ++e) {
+            acc[n][e * 2] = fmaf(lo16(v[n * 2 + e]) + lo16(w[n * 2 + e]), f.x * from[e], -acc[n][e * 2]);
+            acc[n][e * 2 + 1] = fmaf(hi16(v[n * 2 + e]) + hi16(w[n * 2 + e]), f.y * from[e], -acc[n][e * 2 + 1]);
+          }
         }
+      }
       uint32_t yh[4], yl[4];
       operand(acc[0], acc[1], yh, yl);
-      float x[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-      times(x, yh, yl, a);
-      operand(x[0], x[1], xh[a], xl[a]);
+      clear();
+      times(yh, yl, a);
+      sum();
+      operand(acc[0], acc[1], xh[a], xl[a]);
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int c = c0 + g + e * 8, t = a * 16 + n * 8 + t4 * 2;
           if (is_u) {
-            *reinterpret_cast<float2*>(unit + p.unit.u() + c * kUPitch + t * 4) = make_float2(x[n][e * 2], x[n][e * 2 + 1]);
+            *reinterpret_cast<float2*>(unit + p.unit.u() + c * kUPitch + t * 4) = make_float2(acc[n][e * 2], acc[n][e * 2 + 1]);
           } else {                       // −W: the second kernel adds
-            uint8_t* to = unit + c * 128 + (((t >> 3) ^ (c & 7)) << 4) + (t & 7) * 2;
+            uint8_t* to = w_rows + (g + e * 8) * 128 + (((t >> 3) ^ (c & 7)) << 4) + (t & 7) * 2;
             *reinterpret_cast<uint32_t*>(to) = xh[a][n * 2 + e] ^ 0x80008000u;
-            *reinterpret_cast<uint32_t*>(to + half) = xl[a][n * 2 + e] ^ 0x80008000u;
+            *reinterpret_cast<uint32_t*>(to + 2048) = xl[a][n * 2 + e] ^ 0x80008000u;
           }
         }
     }
+    if (!is_u) {
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int at = (i * 32 + lane) * 16;
+        *reinterpret_cast<uint4*>(unit + c0 * 128 + at) = *reinterpret_cast<const uint4*>(w_rows + at);
+        *reinterpret_cast<uint4*>(unit + half + c0 * 128 + at) = *reinterpret_cast<const uint4*>(w_rows + 2048 + at);
+      }
+      __syncwarp();
+    }
+  }
   }
 }
 
-__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-               ::"r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+// the warps' corners: outputs on their way out, and with two warps per 16 columns the parts they exchange
+__host__ __device__ constexpr int corner_bytes(int ks) { return ks == 2 ? 4096 + 128 : 2048; }
+static size_t scan_bytes(const Unit& u, int nw, int ks) { return static_cast<size_t>(u.u()) + nw * 16 * kUPitch + nw * ks * corner_bytes(ks) + 64; }
+
+// c[2·np], c[2·np + 1] += (ah + al)·(hi + lo) without the product of the low parts; b[np] = the operands of two neighbouring accumulators.  One
+// accumulator comes up again only after all others.
+template <int N>
+__device__ __forceinline__ void products(float (*c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh)[N][4], const uint32_t (&bl)[N][4]) {
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+    mma(c[2 * n], ah, bh[n][0], bh[n][1]);
+    mma(c[2 * n + 1], ah, bh[n][2], bh[n][3]);
+  }
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+    mma(c[2 * n], ah, bl[n][0], bl[n][1]);
+    mma(c[2 * n + 1], ah, bl[n][2], bl[n][3]);
+  }
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+    mma(c[2 * n], al, bh[n][0], bh[n][1]);
+    mma(c[2 * n + 1], al, bh[n][2], bh[n][3]);
+  }
 }
 
-static size_t scan_bytes(const Unit& u, int warps) { return static_cast<size_t>(u.u()) + warps * (16 * kUPitch + 2048) + 64; }
-
-// grid (slices of 16·NW value columns, heads, parts of sequences), 32·NW threads
-template <int NW>
-__global__ void __launch_bounds__(32 * NW, 1) delta_scan_kernel(Args p) {
+// grid (slices of 16·NW value columns, heads, parts of sequences), 32·NW·KS threads.  KS = 2: two warps share 16 value columns, each with half
+// of the channels; they exchange their parts of u and of the outputs.
+template <int NW, int KS>
+__global__ void __launch_bounds__(32 * NW * KS, 1) delta_scan_kernel(Args p) {
   extern __shared__ __align__(128) uint8_t smem[];
+  constexpr int NT = 16 / KS, KT = 8 / KS;               // accumulators (8 channels) and k steps (16 channels) of a warp
   const Unit un = p.unit;
   const int KR = un.KR, half = un.half();
   uint8_t* sU = smem + un.u();
-  uint8_t* stage = sU + NW * 16 * kUPitch;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(stage + NW * 2048);        // W and U | q and B | k and decay
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 3);
+  uint8_t* corners = sU + NW * 16 * kUPitch;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(corners + NW * KS * corner_bytes(KS));        // W, q and U | B, k and decay
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 2);
   const int h = blockIdx.y, H = p.m.H, K = p.m.K, V = p.m.V, kdk = (K + 15) / 16;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int cg = warp % NW, kh = warp / NW, ks0 = kh * KT;
   if (tid == 0) {
-    for (int i = 0; i < 3; ++i) mbar_init(&bars[i], 1);
+    for (int i = 0; i < 2; ++i) mbar_init(&bars[i], 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -411,29 +602,25 @@ __global__ void __launch_bounds__(32 * NW, 1) delta_scan_kernel(Args p) {
   pdl_wait();
   const int4 part = reinterpret_cast<const int4*>(p.parts)[blockIdx.z];
   const int first = part.x, n_chunks = part.y, slot = p.m.slots[part.z];
-  const int c_cta = blockIdx.x * NW * 16, c0 = c_cta + warp * 16;
+  const int c_cta = blockIdx.x * NW * 16, c0 = c_cta + cg * 16;
   const int u_rows = min(NW * 16, un.VP - c_cta);
   const bool active = c0 < un.VP;        // (the last slice may be narrower)
   __syncthreads();
   auto unit_of = [&](int i) { return p.scratch + (static_cast<long long>(first + i) * H + h) * un.bytes(); };
-  auto load_w = [&](int i) {
+  auto load_first = [&](int i) {
     const uint8_t* src = unit_of(i);
-    mbar_expect_tx(&bars[0], 2 * half + u_rows * kUPitch);
-    bulk_load(smem, src, 2 * half, &bars[0]);
+    mbar_expect_tx(&bars[0], 4 * half + u_rows * kUPitch);
+    bulk_load(smem, src, 4 * half, &bars[0]);
     bulk_load(sU, src + un.u() + c_cta * kUPitch, u_rows * kUPitch, &bars[0]);
   };
-  auto load_q = [&](int i) {
-    mbar_expect_tx(&bars[1], 2 * half + 16384);
-    bulk_load(smem + un.q(), unit_of(i) + un.q(), 2 * half + 16384, &bars[1]);
-  };
-  auto load_k = [&](int i) {
-    mbar_expect_tx(&bars[2], 2 * half + 512);
-    bulk_load(smem + un.k(), unit_of(i) + un.k(), 2 * half + 512, &bars[2]);
+  auto load_second = [&](int i) {
+    const uint32_t bytes = un.u() - un.b();
+    mbar_expect_tx(&bars[1], bytes);
+    bulk_load(smem + un.b(), unit_of(i) + un.b(), bytes, &bars[1]);
   };
   if (tid == 0) {
-    load_w(0);
-    load_q(0);
-    load_k(0);
+    load_first(0);
+    load_second(0);
   }
   auto wait = [&](int which, int i) {
     if (*abort_flag) return;
@@ -442,122 +629,117 @@ __global__ void __launch_bounds__(32 * NW, 1) delta_scan_kernel(Args p) {
       atomicExch(p.error_flag, 91);
     }
   };
-  // Sᵀ: rows are the warp's value columns g and g + 8, accumulator n holds channels 8n + 2·t4 and the next
+  // Sᵀ: rows are the warp's value columns g and g + 8, accumulator n holds channels 16·ks0 + 8n + 2·t4 and the next
   float* st = p.m.state + (static_cast<long long>(max(slot, 0)) * H + h) * K * V;
   const int t_first = reinterpret_cast<const int4*>(p.chunks)[first].y;
   const bool fresh = slot < 0 || p.m.positions[t_first] == 0;
-  float S[16][4];
+  float S[NT][4];
 #pragma unroll
-  for (int n = 0; n < 16; ++n)
+  for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int k = n * 8 + t4 * 2 + (e & 1), v = c0 + g + (e >> 1) * 8;
+      const int k = ks0 * 16 + n * 8 + t4 * 2 + (e & 1), v = c0 + g + (e >> 1) * 8;
       S[n][e] = (!fresh && k < K && v < V) ? st[static_cast<long long>(k) * V + v] : 0.f;
     }
   const uint32_t w_base = smem_u32(smem), q_base = w_base + un.q(), b_base = w_base + un.b(), k_base = w_base + un.k();
   const int l7 = lane & 7, l8 = (lane >> 3) & 1, l16 = lane >> 4;
+  uint8_t* mine = corners + warp * corner_bytes(KS);
+  uint8_t* other = corners + (warp < NW ? warp + NW : warp - NW) * corner_bytes(KS);
+  auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(cg + 1) : "memory"); };
+  // accumulators [n0, n0 + N) of a warp in its corner and back: a lane's float4s, 32 lanes side by side
+  auto put = [&](const float (*x)[4], int n0, int N) {
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+      if (n < N) *reinterpret_cast<float4*>(mine + (n * 32 + lane) * 16) = make_float4(x[n0 + n][0], x[n0 + n][1], x[n0 + n][2], x[n0 + n][3]);
+  };
+  auto take = [&](float (*x)[4], int n0, int N) {
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+      if (n < N) {
+        const float4 v = *reinterpret_cast<const float4*>(other + (n * 32 + lane) * 16);
+        x[n0 + n][0] += v.x; x[n0 + n][1] += v.y; x[n0 + n][2] += v.z; x[n0 + n][3] += v.w;
+      }
+  };
   for (int ci = 0; ci < n_chunks; ++ci) {
     const int4 ch = reinterpret_cast<const int4*>(p.chunks)[first + ci];
     uint32_t uh[4][4], ul[4][4];
+    float o[8][4];
+#pragma unroll
+    for (int n = 0; n < 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
     wait(0, ci);
-    {                                    // u = U − W S
+    {                                    // u = U − W S, o = q S
       float u[8][4];
 #pragma unroll
       for (int n = 0; n < 8; ++n)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const float2 x = active ? *reinterpret_cast<const float2*>(sU + (warp * 16 + g + e * 8) * kUPitch + (n * 8 + t4 * 2) * 4) : make_float2(0.f, 0.f);
+          float2 x = make_float2(0.f, 0.f);
+          if (active && kh == 0) x = *reinterpret_cast<const float2*>(sU + (cg * 16 + g + e * 8) * kUPitch + (n * 8 + t4 * 2) * 4);
           u[n][e * 2] = x.x;
           u[n][e * 2 + 1] = x.y;
         }
 #pragma unroll
-      for (int ks = 0; ks < 8; ++ks) {
-        if (ks >= kdk) break;
-        uint32_t sh[4], sl[4];
-        operand(S[2 * ks], S[2 * ks + 1], sh, sl);
-        const int row = ks * 16 + l7 + l8 * 8;
+      for (int i = 0; i < KT; ++i) {
+        if (ks0 + i >= kdk) break;
+        uint32_t sh[4], sl[4], bh[4][4], bl[4][4];
+        operand(S[2 * i], S[2 * i + 1], sh, sl);
 #pragma unroll
         for (int np = 0; np < 4; ++np) {
-          uint32_t bh[4], bl[4];
+          const int row = (ks0 + i) * 16 + l7 + l8 * 8;
           const uint32_t at = w_base + row * 128 + (((np * 2 + l16) ^ (row & 7)) << 4);
-          ldsm4t(at, bh);
-          ldsm4t(at + half, bl);
-          mma(u[2 * np], sh, bh[0], bh[1]);
-          mma(u[2 * np + 1], sh, bh[2], bh[3]);
-          mma(u[2 * np], sh, bl[0], bl[1]);
-          mma(u[2 * np + 1], sh, bl[2], bl[3]);
-          mma(u[2 * np], sl, bh[0], bh[1]);
-          mma(u[2 * np + 1], sl, bh[2], bh[3]);
+          ldsm4t(at, bh[np]);
+          ldsm4t(at + half, bl[np]);
         }
+        products<4>(u, sh, sl, bh, bl);
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {
+          const int row = np * 16 + l7 + l16 * 8;
+          const uint32_t at = q_base + row * KR * 2 + ((((ks0 + i) * 2 + l8) ^ (row & 7)) << 4);
+          ldsm4(at, bh[np]);
+          ldsm4(at + half, bl[np]);
+        }
+        products<4>(o, sh, sl, bh, bl);
+      }
+      if (KS == 2) {
+        put(u, 0, 8);
+        pair_sync();
+        take(u, 0, 8);
       }
 #pragma unroll
       for (int ks = 0; ks < 4; ++ks) operand(u[2 * ks], u[2 * ks + 1], uh[ks], ul[ks]);
     }
     __syncthreads();
-    if (tid == 0 && ci + 1 < n_chunks && !*abort_flag) load_w(ci + 1);
+    if (tid == 0 && ci + 1 < n_chunks && !*abort_flag) load_first(ci + 1);
     wait(1, ci);
-    {                                    // outputs
-      float o[8][4];
+    // o += B u, by blocks of 16 tokens; of two warps one takes the last row of blocks
 #pragma unroll
-      for (int n = 0; n < 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    for (int ks = 0; ks < 4; ++ks) {
+      uint32_t bh[4][4], bl[4][4];
 #pragma unroll
-      for (int ks = 0; ks < 8; ++ks) {
-        if (ks >= kdk) break;
-        uint32_t sh[4], sl[4];
-        operand(S[2 * ks], S[2 * ks + 1], sh, sl);
+      for (int np = 0; np < 4; ++np) {
+        if (np < ks || (KS == 2 && (np == 3) != (kh == 1))) continue;
+        const int row = np * 16 + l7 + l16 * 8;
+        const uint32_t at = b_base + row * 128 + (((ks * 2 + l8) ^ (row & 7)) << 4);
+        ldsm4(at, bh[np]);
+        ldsm4(at + 8192, bl[np]);
+      }
+#pragma unroll
+      for (int term = 0; term < 3; ++term)
 #pragma unroll
         for (int np = 0; np < 4; ++np) {
-          uint32_t bh[4], bl[4];
-          const int row = np * 16 + l7 + l16 * 8;
-          const uint32_t at = q_base + row * KR * 2 + (((ks * 2 + l8) ^ (row & 7)) << 4);
-          ldsm4(at, bh);
-          ldsm4(at + half, bl);
-          mma(o[2 * np], sh, bh[0], bh[1]);
-          mma(o[2 * np + 1], sh, bh[2], bh[3]);
-          mma(o[2 * np], sh, bl[0], bl[1]);
-          mma(o[2 * np + 1], sh, bl[2], bl[3]);
-          mma(o[2 * np], sl, bh[0], bh[1]);
-          mma(o[2 * np + 1], sl, bh[2], bh[3]);
+          if (np < ks || (KS == 2 && (np == 3) != (kh == 1))) continue;
+          mma(o[2 * np], term == 2 ? ul[ks] : uh[ks], term == 1 ? bl[np][0] : bh[np][0], term == 1 ? bl[np][1] : bh[np][1]);
+          mma(o[2 * np + 1], term == 2 ? ul[ks] : uh[ks], term == 1 ? bl[np][2] : bh[np][2], term == 1 ? bl[np][3] : bh[np][3]);
         }
-      }
-#pragma unroll
-      for (int np = 0; np < 4; ++np)
-#pragma unroll
-        for (int ks = 0; ks <= np; ++ks) {
-          uint32_t bh[4], bl[4];
-          const int row = np * 16 + l7 + l16 * 8;
-          const uint32_t at = b_base + row * 128 + (((ks * 2 + l8) ^ (row & 7)) << 4);
-          ldsm4(at, bh);
-          ldsm4(at + 8192, bl);
-          mma(o[2 * np], uh[ks], bh[0], bh[1]);
-          mma(o[2 * np + 1], uh[ks], bh[2], bh[3]);
-          mma(o[2 * np], uh[ks], bl[0], bl[1]);
-          mma(o[2 * np + 1], uh[ks], bl[2], bl[3]);
-          mma(o[2 * np], ul[ks], bh[0], bh[1]);
-          mma(o[2 * np + 1], ul[ks], bh[2], bh[3]);
-        }
-      // rows of 16 columns per token in the warp's own corner of shared memory, then 16-byte stores
-      uint8_t* mine = stage + warp * 2048;
-#pragma unroll
-      for (int np = 0; np < 4; ++np)
-        stsm4t(smem_u32(mine + ((np * 2 + l16) * 8 + l7) * 32 + l8 * 16), pack2(o[2 * np][0], o[2 * np][1]), pack2(o[2 * np][2], o[2 * np][3]),
-               pack2(o[2 * np + 1][0], o[2 * np + 1][1]), pack2(o[2 * np + 1][2], o[2 * np + 1][3]));
-      __syncwarp();
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int r = (i * 32 + lane) >> 1, c = c0 + (lane & 1) * 8;
-        if (active && ch.y + r < ch.z && c < V)
-          *reinterpret_cast<uint4*>(p.out + static_cast<long long>(ch.y + r) * H * V + h * V + c) = *reinterpret_cast<const uint4*>(mine + r * 32 + (lane & 1) * 16);
-      }
     }
-    __syncthreads();
-    if (tid == 0 && ci + 1 < n_chunks && !*abort_flag) load_q(ci + 1);
-    wait(2, ci);
+    if (KS == 2) {                       // each finishes half of the tokens
+      if (kh == 0) put(o, 4, 4);
+      else put(o, 0, 4);
+    }
     {                                    // S ← decay · S + Σ k uᵀ
-      const float* dec = reinterpret_cast<const float*>(smem + un.decay());
+      const float* dec = reinterpret_cast<const float*>(smem + un.decay()) + ks0 * 16;
 #pragma unroll
-      for (int n = 0; n < 16; ++n) {
-        if (n >= 2 * kdk) break;
+      for (int n = 0; n < NT; ++n) {
         const float2 d = *reinterpret_cast<const float2*>(dec + n * 8 + t4 * 2);
         S[n][0] *= d.x; S[n][1] *= d.y; S[n][2] *= d.x; S[n][3] *= d.y;
       }
@@ -565,43 +747,64 @@ __global__ void __launch_bounds__(32 * NW, 1) delta_scan_kernel(Args p) {
       for (int ks = 0; ks < 4; ++ks) {
         const int row = ks * 16 + l7 + l8 * 8;
 #pragma unroll
-        for (int np = 0; np < 8; ++np) {
-          if (np >= kdk) break;
-          uint32_t bh[4], bl[4];
-          const uint32_t at = k_base + row * KR * 2 + (((np * 2 + l16) ^ (row & 7)) << 4);
-          ldsm4t(at, bh);
-          ldsm4t(at + half, bl);
-          mma(S[2 * np], uh[ks], bh[0], bh[1]);
-          mma(S[2 * np + 1], uh[ks], bh[2], bh[3]);
-          mma(S[2 * np], uh[ks], bl[0], bl[1]);
-          mma(S[2 * np + 1], uh[ks], bl[2], bl[3]);
-          mma(S[2 * np], ul[ks], bh[0], bh[1]);
-          mma(S[2 * np + 1], ul[ks], bh[2], bh[3]);
+        for (int n4 = 0; n4 < KT; n4 += 4) {
+          if (ks0 + n4 >= kdk) break;
+          uint32_t bh[4][4], bl[4][4];
+#pragma unroll
+          for (int np = 0; np < 4; ++np) {               // (columns behind K: whatever lies there stays in accumulators that nobody reads)
+            const int piece = min((ks0 + n4 + np) * 2 + l16, KR / 8 - 1);
+            const uint32_t at = k_base + row * KR * 2 + ((piece ^ (row & 7)) << 4);
+            ldsm4t(at, bh[np]);
+            ldsm4t(at + half, bl[np]);
+          }
+          products<4>(S + 2 * n4, uh[ks], ul[ks], bh, bl);
         }
       }
     }
     __syncthreads();
-    if (tid == 0 && ci + 1 < n_chunks && !*abort_flag) load_k(ci + 1);
+    if (tid == 0 && ci + 1 < n_chunks && !*abort_flag) load_second(ci + 1);
+    if (KS == 2) {
+      if (kh == 0) take(o, 0, 4);
+      else take(o, 4, 4);
+      pair_sync();
+    }
+    // rows of 16 columns per token in the warp's own corner of shared memory, then 16-byte stores
+#pragma unroll
+    for (int np = 0; np < 4; ++np) {
+      if (KS == 2 && (np >> 1) != kh) continue;
+      stsm4t(smem_u32(mine + ((np * 2 + l16) * 8 + l7) * 32 + l8 * 16), pack2(o[2 * np][0], o[2 * np][1]), pack2(o[2 * np][2], o[2 * np][3]),
+             pack2(o[2 * np + 1][0], o[2 * np + 1][1]), pack2(o[2 * np + 1][2], o[2 * np + 1][3]));
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      if (KS == 2 && (i >> 1) != kh) continue;
+      const int r = (i * 32 + lane) >> 1, c = c0 + (lane & 1) * 8;
+      if (active && ch.y + r < ch.z && c < V)
+        *reinterpret_cast<uint4*>(p.out + static_cast<long long>(ch.y + r) * H * V + h * V + c) = *reinterpret_cast<const uint4*>(mine + r * 32 + (lane & 1) * 16);
+    }
+    __syncwarp();
   }
   if (slot < 0 || *abort_flag) return;
 #pragma unroll
-  for (int n = 0; n < 16; ++n)
+  for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int k = n * 8 + t4 * 2 + (e & 1), v = c0 + g + (e >> 1) * 8;
+      const int k = ks0 * 16 + n * 8 + t4 * 2 + (e & 1), v = c0 + g + (e >> 1) * 8;
       if (k < K && v < V) st[static_cast<long long>(k) * V + v] = S[n][e];
     }
 }
 
-template <int NW>
+template <int NW, int KS>
 static cudaError_t scan(const Args& a, int n_parts, cudaStream_t s) {
   static bool once = false;
   if (!once) {
-    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(scan_bytes(Unit{128, 128}, NW)));
+    const cudaError_t e =
+        cudaFuncSetAttribute(delta_scan_kernel<NW, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(scan_bytes(Unit{128, 128}, NW, KS)));
     if (e != cudaSuccess) return e;
     once = true;
   }
-  return launch_pdl(delta_scan_kernel<NW>, dim3((a.unit.VP / 16 + NW - 1) / NW, a.m.H, n_parts), dim3(32 * NW), scan_bytes(a.unit, NW), s, a);
+  return launch_pdl(delta_scan_kernel<NW, KS>, dim3((a.unit.VP / 16 + NW - 1) / NW, a.m.H, n_parts), dim3(32 * NW * KS), scan_bytes(a.unit, NW, KS), s, a);
 }
 
 static Unit unit_of(int K, int V) { return Unit{(K + 63) / 64 * 64, (V + 15) / 16 * 16}; }
@@ -615,7 +818,7 @@ using namespace mb::dc;
 extern "C" long long mb_delta_chunk_bytes(int K, int V) { return unit_of(K, V).bytes(); }
 
 extern "C" int mb_delta_chunk(const void* proj, long long ld, const void* act, MbDelta m, const int* chunks, const int* parts, void* scratch, void* out,
-                              int n_chunks, int n_parts, int warps, int* error_flag, cudaStream_t s) {
+                              int T, int n_chunks, int n_parts, int warps, int* error_flag, cudaStream_t s) {
   if (n_chunks <= 0 || n_parts <= 0) return 0;
   if (m.K % 8 || m.V % 8 || m.K > 128 || m.V > 128 || m.K <= 0 || m.V <= 0 || m.G <= 0 || m.H % m.G || m.raw_ld % 8 || n_chunks > 65535 || n_parts > 65535 ||
       m.H > 65535 || (reinterpret_cast<uintptr_t>(m.raw) | reinterpret_cast<uintptr_t>(m.dt_bias) | reinterpret_cast<uintptr_t>(act)) % 16)
@@ -628,7 +831,18 @@ extern "C" int mb_delta_chunk(const void* proj, long long ld, const void* act, M
   }
   Args a{reinterpret_cast<const bf16*>(proj), ld, reinterpret_cast<const bf16*>(act), m, chunks, parts, reinterpret_cast<uint8_t*>(scratch), unit_of(m.K, m.V),
          reinterpret_cast<bf16*>(out), error_flag};
-  cudaError_t e = launch_pdl(delta_prepare_kernel, dim3(m.H, n_chunks), dim3(kThreads), sizeof(Shared), s, a);
-  if (e == cudaSuccess) e = warps >= 8 ? scan<8>(a, n_parts, s) : warps >= 4 ? scan<4>(a, n_parts, s) : scan<2>(a, n_parts, s);
+  CUtensorMap tm_act, tm_raw;
+  const long long CH = 2ll * m.G * m.K + static_cast<long long>(m.H) * m.V;
+  int rc = make_tmap_bf16_2d(&tm_act, act, T, CH, CH, C, 64);
+  if (rc) return 1000 + rc;
+  rc = make_tmap_bf16_2d(&tm_raw, m.raw, T, static_cast<long long>(m.H) * m.K, m.raw_ld, C, 64);
+  if (rc) return 2000 + rc;
+  const int n_units = n_chunks * m.H;
+  cudaError_t e = launch_pdl(delta_prepare_kernel, dim3(n_units < 148 ? n_units : 148), dim3(kThreads), sizeof(Shared), s, tm_act, tm_raw, a, n_units);
+  // with few slices per CTA two warps share one, unless the channels of a second one are all padding
+  const bool two = m.K > 64;
+  if (e == cudaSuccess)
+    e = warps >= 8 ? scan<8, 1>(a, n_parts, s) : warps >= 4 ? (two ? scan<4, 2>(a, n_parts, s) : scan<4, 1>(a, n_parts, s))
+                                               : (two ? scan<2, 2>(a, n_parts, s) : scan<2, 1>(a, n_parts, s));
   return static_cast<int>(e);
 }

@@ -133,7 +133,7 @@ __global__ void __launch_bounds__(128) delta_seq_kernel(const T* __restrict__ pr
 static constexpr int kStep = 256;
 // grid (heads, rows), 256 threads; V % 4 == 0.  A thread owns four columns of U state rows, 256 / (V / 4) rows apart.
 template <typename T, int U>
-__global__ void __launch_bounds__(kStep) delta_step_kernel(const T* __restrict__ proj, long long ld, MbDelta m, const T* __restrict__ norm_w,
+__global__ void __launch_bounds__(kStep, U <= 4 ? 4 : U <= 8 ? 3 : 2) delta_step_kernel(const T* __restrict__ proj, long long ld, MbDelta m, const T* __restrict__ norm_w,
                                                            const T* __restrict__ gate, long long gate_ld, float eps, T* __restrict__ out) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float sh[kStep / 32];

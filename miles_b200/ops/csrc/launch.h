@@ -372,7 +372,7 @@ int mb_delta_step_max(void);
 // mb_delta_chunk_bytes(K, V) per chunk and head.  warps (2, 4 or 8): 16 value columns each that a CTA of the second kernel takes.
 long long mb_delta_chunk_bytes(int K, int V);
 int mb_delta_chunk(const void* proj, long long ld, const void* act, MbDelta m, const int* chunks, const int* parts, void* scratch, void* out,
-                   int n_chunks, int n_parts, int warps, int* error_flag, cudaStream_t s);
+                   int T, int n_chunks, int n_parts, int warps, int* error_flag, cudaStream_t s);
 // ---- ssm_*.cu (state-space mixer: S ← exp(−exp(A_log)·dt)·S + dt·B xᵀ, y = Sᵀ C + D·x) ----
 // A row of the projection is [z: H·V | x: H·V | B: G·N | C: G·N | dt: H]; x, B and C pass a causal convolution of `taps` columns and silu.
 typedef struct {
