@@ -71,7 +71,7 @@ void gemv(const at::Tensor& x, const c10::optional<at::Tensor>& residual, const 
           const c10::optional<at::Tensor>& xn_out, bool static_w) {
   c10::cuda::CUDAGuard g(x.device());
   const int64_t K = x.size(-1), M = x.numel() / K, N = W.size(0);
-  check(mb_gemv(x.data_ptr(), cptr(residual), cptr(norm_w), eps, W.data_ptr(), cptr(bias), y.data_ptr(), y.stride(0),
+  check(mb_gemv(x.data_ptr(), x.size(0) > 1 ? x.stride(0) : W.size(1), cptr(residual), cptr(norm_w), eps, W.data_ptr(), cptr(bias), y.data_ptr(), y.stride(0),
                 y.scalar_type() == at::kFloat, mptr(res_out), mptr(xn_out), M, N, K, static_w, cur_stream()),
         "mb_gemv");
 }

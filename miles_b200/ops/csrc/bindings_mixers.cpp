@@ -160,7 +160,7 @@ void sum_norm(const at::Tensor& x, const OptTensor& to, const OptTensor& y1, con
 void gemv_sum_norm(const OptTensor& x32, const OptTensor& y1, const OptTensor& s1, const OptTensor& y2, const OptTensor& s2, const OptTensor& extra,
                    const OptTensor& x, const OptTensor& norm_w, const OptTensor& norm_w2, double eps, double shift, const at::Tensor& W, at::Tensor& y,
                    const OptTensor& W2, const OptTensor& bias2, const OptTensor& y2out, const OptTensor& x_out, const OptTensor& xn_out, bool static_w,
-                   double mult) {
+                   double mult, const OptTensor& x2) {
   c10::cuda::CUDAGuard g(W.device());
   const bool two = W2.has_value() && W2->defined();
   MbGemvSum a{};
@@ -171,6 +171,9 @@ void gemv_sum_norm(const OptTensor& x32, const OptTensor& y1, const OptTensor& s
   a.s2 = cptr(s2);
   a.extra = fptr(extra);
   a.x = cptr(x);
+  a.x2 = cptr(x2);
+  a.ldx = a.x != nullptr && x->size(0) > 1 ? row_of(x) : W.size(1);
+  TORCH_CHECK(a.x2 == nullptr || x->size(0) == 1 || row_of(x2) == a.ldx, "gemv_sum_norm: both rows out of one matrix");
   a.norm_w = cptr(norm_w);
   a.norm_w2 = cptr(norm_w2);
   a.eps = eps;
@@ -595,7 +598,8 @@ void register_mixers(pybind11::module& m) {
   m.def("sum_norm", &sum_norm, arg("x"), arg("to"), arg("y1"), arg("s1"), arg("y2"), arg("s2"), arg("rows"), arg("weights"), arg("dst"), arg("extra"),
         arg("nw"), arg("h"), arg("nw2"), arg("h2"), arg("eps"), arg("shift"), arg("gain"), arg("mult") = 1.0);
   m.def("gemv_sum_norm", &gemv_sum_norm, arg("x32"), arg("y1"), arg("s1"), arg("y2"), arg("s2"), arg("extra"), arg("x"), arg("norm_w"), arg("norm_w2"),
-        arg("eps"), arg("shift"), arg("W"), arg("y"), arg("W2"), arg("bias2"), arg("y2out"), arg("x_out"), arg("xn_out"), arg("static_w"), arg("mult") = 1.0);
+        arg("eps"), arg("shift"), arg("W"), arg("y"), arg("W2"), arg("bias2"), arg("y2out"), arg("x_out"), arg("xn_out"), arg("static_w"), arg("mult") = 1.0,
+        arg("x2") = pybind11::none());
   m.def("gated_norm", &gated_norm);
   m.def("relu_square", &relu_square, pybind11::arg("x"), pybind11::arg("rows") = pybind11::none());
   m.def("part_norm", &part_norm);
@@ -621,7 +625,7 @@ void register_mixers(pybind11::module& m) {
   m.def("delta_conv", &delta_conv);
   m.def("delta_seq", &delta_seq);
   m.def("delta_step", &delta_step);
-  m.def("delta_step_max", &mb_delta_step_max);
+  m.def("delta_step_ok", &mb_delta_step_ok);
   m.def("delta_chunk", &delta_chunk);
   m.def("delta_chunk_bytes", &mb_delta_chunk_bytes);
 #endif

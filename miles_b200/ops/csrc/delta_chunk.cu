@@ -181,375 +181,375 @@ __global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(const __grid
   fetch(blockIdx.x);
   uint32_t phase = 0;
   for (int idx = blockIdx.x; idx < n_units; idx += gridDim.x) {
-  const int h = idx % H, gq = h / per, t0_now = ch.y, n_now = ch.z - ch.y, after_idx = idx + gridDim.x;
-  if (after_idx < n_units) ch = reinterpret_cast<const int4*>(p.chunks)[after_idx / H];
-  uint8_t* unit = p.scratch + static_cast<long long>(idx) * p.unit.bytes();
-  if (!mbar_wait(&s.full, phase)) {
-    atomicExch(p.error_flag, 92);
-    return;
-  }
-  phase ^= 1;
-  __syncthreads();
-  // ---- q and k with the factors that make unit vectors of them, v into its place, log decays, β
-  uint4 q_in[2], k_in[2];
-  const float rate = __expf(__bfloat162float(a_raw));
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int r = my_row + i * 32, at = r * P + my_c;
-    const int from = (my_c >> 6) * 8192 + r * 128 + ((((my_c >> 3) & 7) ^ (r & 7)) << 4);
-    const bool ok = r < n_now && my_c < K;
-    uint4 v = make_uint4(0, 0, 0, 0), x = make_uint4(0, 0, 0, 0);
-    q_in[i] = k_in[i] = v;
-    if (ok) {
-      q_in[i] = *reinterpret_cast<const uint4*>(in_q + from);
-      k_in[i] = *reinterpret_cast<const uint4*>(in_k + from);
-      x = *reinterpret_cast<const uint4*>(in_k + 16384 + from);
+    const int h = idx % H, gq = h / per, t0_now = ch.y, n_now = ch.z - ch.y, after_idx = idx + gridDim.x;
+    if (after_idx < n_units) ch = reinterpret_cast<const int4*>(p.chunks)[after_idx / H];
+    uint8_t* unit = p.scratch + static_cast<long long>(idx) * p.unit.bytes();
+    if (!mbar_wait(&s.full, phase)) {
+      atomicExch(p.error_flag, 92);
+      return;
     }
-    if (r < n_now && my_c < V) v = *reinterpret_cast<const uint4*>(in_q + 16384 + from);
-    *reinterpret_cast<uint4*>(s.v + at) = v;
-    const uint32_t qw[4] = {q_in[i].x, q_in[i].y, q_in[i].z, q_in[i].w}, kw[4] = {k_in[i].x, k_in[i].y, k_in[i].z, k_in[i].w};
-    float sq = 0.f, sk = 0.f;
+    phase ^= 1;
+    __syncthreads();
+    // ---- q and k with the factors that make unit vectors of them, v into its place, log decays, β
+    uint4 q_in[2], k_in[2];
+    const float rate = __expf(__bfloat162float(a_raw));
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      sq += lo16(qw[j]) * lo16(qw[j]) + hi16(qw[j]) * hi16(qw[j]);
-      sk += lo16(kw[j]) * lo16(kw[j]) + hi16(kw[j]) * hi16(kw[j]);
-    }
-#pragma unroll
-    for (int o = 8; o > 0; o >>= 1) {    // a row's 16 threads are half a warp
-      sq += __shfl_xor_sync(0xffffffffu, sq, o);
-      sk += __shfl_xor_sync(0xffffffffu, sk, o);
-    }
-    if (my_c == 0) {
-      s.fq[r] = inv_sqrt(sq + 1e-6f) * q_scale;
-      s.fk[r] = inv_sqrt(sk + 1e-6f);
-    }
-    const uint32_t xw[4] = {x.x, x.y, x.z, x.w}, bw[4] = {bias_raw.x, bias_raw.y, bias_raw.z, bias_raw.w};
-    float l[8];
-#pragma unroll
-    for (int j = 0; j < 8; ++j)
-      l[j] = ok ? -rate * softplus2((j & 1) ? hi16(xw[j / 2]) + hi16(bw[j / 2]) : lo16(xw[j / 2]) + lo16(bw[j / 2])) : 0.f;
-    mx::store_n<8>(s.L + r * LP + my_c, l);
-  }
-  if (tid < C) s.beta[tid] = tid < n_now ? mx::sigmoid_t<bf16>(__bfloat162float(beta_raw)) : 0.f;
-  if (tid < 4) s.direct[tid] = 0;
-  if (tid == 4) s.next = 0;
-  __syncthreads();
-  {                                      // running sums inside the blocks: a thread per (block, channel)
-    const int b = tid >> 7, c = tid & 127;
-    float* x = s.L + b * 16 * LP + c;
-    float sum = 0.f;
-#pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      sum += x[i * LP];
-      x[i * LP] = sum;
-    }
-    s.D[b][c] = sum;
-    if (sum < kFar) s.direct[b] = 1;
-  }
-  __syncthreads();
-  if (tid < 128) {
-    const float d0 = s.D[0][tid], d1 = s.D[1][tid], d2 = s.D[2][tid], d3 = s.D[3][tid];
-    s.before[0][tid] = 1.f;
-    s.before[1][tid] = e2(d0);
-    s.before[2][tid] = e2(d0 + d1);
-    s.before[3][tid] = e2(d0 + d1 + d2);
-    s.after[0][tid] = e2(d1 + d2 + d3);
-    s.after[1][tid] = e2(d2 + d3);
-    s.after[2][tid] = e2(d3);
-    s.after[3][tid] = 1.f;
-    s.between[0][tid] = e2(fminf(-d0, -kFar));           // blocks beyond are summed directly
-    s.between[1][tid] = e2(fminf(-d1, -kFar));
-    s.between[2][tid] = e2(fminf(-d2, -kFar));
-    s.between[3][tid] = e2(fminf(-d3, -kFar));
-    s.between[4][tid] = e2(d1);
-    s.between[5][tid] = e2(d1 + d2);
-    s.between[6][tid] = e2(d2);
-    reinterpret_cast<float*>(unit + p.unit.decay())[tid] = e2(d0 + d1 + d2 + d3);
-  } else if (tid < 128 + C) {
-    s.beta_k[tid - 128] = s.beta[tid - 128] * s.fk[tid - 128];
-  }
-  __syncthreads();
-  // ---- q and k decayed from the start of their block, k to its end; queries decayed from the chunk's start
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int r = my_row + i * 32, c = my_c, at = r * P + c;
-    float q[8], k[8], l[8], d[8], x[8];
-    uint4 hi, lo;
-    const uint32_t qw[4] = {q_in[i].x, q_in[i].y, q_in[i].z, q_in[i].w}, kw[4] = {k_in[i].x, k_in[i].y, k_in[i].z, k_in[i].w};
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      q[j] = (j & 1) ? hi16(qw[j / 2]) : lo16(qw[j / 2]);
-      k[j] = (j & 1) ? hi16(kw[j / 2]) : lo16(kw[j / 2]);
-    }
-    mx::load_n<8>(s.L + r * LP + c, l);
-    mx::load_n<8>(s.D[r >> 4] + c, d);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      d[j] = k[j] * e2(d[j] - l[j]);
-      l[j] = e2(l[j]);
-      x[j] = q[j] * l[j];
-    }
-    split8(x, hi, lo);
-    *reinterpret_cast<uint4*>(s.q_hi + at) = hi;
-    *reinterpret_cast<uint4*>(s.q_lo + at) = lo;
-    if (c < kdk * 16) {
-      float f[8];
-      mx::load_n<8>(s.before[r >> 4] + c, f);
-      const float scale = s.fq[r];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) x[j] *= f[j] * scale;
-      split8(x, hi, lo);
-      uint8_t* to = unit + p.unit.q() + r * KR * 2 + (((c >> 3) ^ (r & 7)) << 4);
-      *reinterpret_cast<uint4*>(to) = hi;
-      *reinterpret_cast<uint4*>(to + half) = lo;
-    }
-#pragma unroll
-    for (int j = 0; j < 8; ++j) x[j] = k[j] * l[j];
-    split8(x, hi, lo);
-    *reinterpret_cast<uint4*>(s.k_hi + at) = hi;
-    *reinterpret_cast<uint4*>(s.k_lo + at) = lo;
-    split8(d, hi, lo);
-    *reinterpret_cast<uint4*>(s.c_hi + at) = hi;
-    *reinterpret_cast<uint4*>(s.c_lo + at) = lo;
-  }
-  __syncthreads();
-  // ---- A and B, a warp per pair of blocks; the diagonal blocks of I + A are inverted by the warps that made them
-  if (warp < 10) {
-    int a, b;
-    pair_of(warp, a, b);
-    float kk[2][4] = {}, qk[2][4] = {}, kk1[2][4] = {}, qk1[2][4] = {};      // (the products with low parts have sums of their own)
-    if (a == b && s.direct[a]) {
-#pragma unroll 1
-      for (int x = 0; x < 8; ++x) {
-        const int i = a * 16 + g + (x & 2) * 4, j = a * 16 + (x >> 2) * 8 + t4 * 2 + (x & 1);
-        float sk = 0.f, sq = 0.f;
-        if (j <= i && i < n_now) {
-          const bf16* qi = p.act + static_cast<long long>(t0_now + i) * CH + gq * K;
-          const bf16* ki = qi + p.m.G * K;
-          const bf16* kj = p.act + static_cast<long long>(t0_now + j) * CH + p.m.G * K + gq * K;
-          for (int c = 0; c < K; ++c) {
-            const float w = __bfloat162float(kj[c]) * e2(s.L[i * LP + c] - s.L[j * LP + c]);
-            sk = fmaf(__bfloat162float(ki[c]), w, sk);
-            sq = fmaf(__bfloat162float(qi[c]), w, sq);
-          }
-        }
-#pragma unroll
-        for (int y = 0; y < 8; ++y)
-          if (y == x) { kk[y >> 2][y & 3] = sk; qk[y >> 2][y & 3] = sq; }
+    for (int i = 0; i < 2; ++i) {
+      const int r = my_row + i * 32, at = r * P + my_c;
+      const int from = (my_c >> 6) * 8192 + r * 128 + ((((my_c >> 3) & 7) ^ (r & 7)) << 4);
+      const bool ok = r < n_now && my_c < K;
+      uint4 v = make_uint4(0, 0, 0, 0), x = make_uint4(0, 0, 0, 0);
+      q_in[i] = k_in[i] = v;
+      if (ok) {
+        q_in[i] = *reinterpret_cast<const uint4*>(in_q + from);
+        k_in[i] = *reinterpret_cast<const uint4*>(in_k + from);
+        x = *reinterpret_cast<const uint4*>(in_k + 16384 + from);
       }
-      __syncwarp();
-    } else {
-      const int row_a = (a * 16 + (lane & 15)) * P + (lane >> 4) * 8;
-      const int row_b = (b * 16 + (lane & 7) + ((lane >> 4) << 3)) * P + ((lane >> 3) & 1) * 8;
-      const float* fac = s.between[min(warp, 6)];
-#pragma unroll 2
-      for (int ks = 0; ks < kdk; ++ks) {
-        uint32_t qh[4], ql[4], kh[4], kl[4], ch[4], cl[4];
-        ldsm4(smem_u32(s.c_hi + row_b + ks * 16), ch);
-        ldsm4(smem_u32(s.c_lo + row_b + ks * 16), cl);
-        ldsm4(smem_u32(s.k_hi + row_a + ks * 16), kh);
-        ldsm4(smem_u32(s.q_hi + row_a + ks * 16), qh);
-        ldsm4(smem_u32(s.k_lo + row_a + ks * 16), kl);
-        ldsm4(smem_u32(s.q_lo + row_a + ks * 16), ql);
-        if (warp < 7) {
+      if (r < n_now && my_c < V) v = *reinterpret_cast<const uint4*>(in_q + 16384 + from);
+      *reinterpret_cast<uint4*>(s.v + at) = v;
+      const uint32_t qw[4] = {q_in[i].x, q_in[i].y, q_in[i].z, q_in[i].w}, kw[4] = {k_in[i].x, k_in[i].y, k_in[i].z, k_in[i].w};
+      float sq = 0.f, sk = 0.f;
 #pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            const float2 f = *reinterpret_cast<const float2*>(fac + ks * 16 + i * 8 + t4 * 2);
-#pragma unroll
-            for (int n = 0; n < 4; n += 2) split2((lo16(ch[n + i]) + lo16(cl[n + i])) * f.x, (hi16(ch[n + i]) + hi16(cl[n + i])) * f.y, ch[n + i], cl[n + i]);
-          }
-        }
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          mma(kk[n], kh, ch[2 * n], ch[2 * n + 1]);
-          mma(qk[n], qh, ch[2 * n], ch[2 * n + 1]);
-        }
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          mma(kk1[n], kh, cl[2 * n], cl[2 * n + 1]);
-          mma(qk1[n], qh, cl[2 * n], cl[2 * n + 1]);
-        }
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          mma(kk1[n], kl, ch[2 * n], ch[2 * n + 1]);
-          mma(qk1[n], ql, ch[2 * n], ch[2 * n + 1]);
-        }
+      for (int j = 0; j < 4; ++j) {
+        sq += lo16(qw[j]) * lo16(qw[j]) + hi16(qw[j]) * hi16(qw[j]);
+        sk += lo16(kw[j]) * lo16(kw[j]) + hi16(kw[j]) * hi16(kw[j]);
       }
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) {    // a row's 16 threads are half a warp
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+      }
+      if (my_c == 0) {
+        s.fq[r] = inv_sqrt(sq + 1e-6f) * q_scale;
+        s.fk[r] = inv_sqrt(sk + 1e-6f);
+      }
+      const uint32_t xw[4] = {x.x, x.y, x.z, x.w}, bw[4] = {bias_raw.x, bias_raw.y, bias_raw.z, bias_raw.w};
+      float l[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        l[j] = ok ? -rate * softplus2((j & 1) ? hi16(xw[j / 2]) + hi16(bw[j / 2]) : lo16(xw[j / 2]) + lo16(bw[j / 2])) : 0.f;
+      mx::store_n<8>(s.L + r * LP + my_c, l);
     }
-#pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int i = a * 16 + g + e * 4, j = b * 16 + n * 8 + t4 * 2;
-        const float k0 = kk[n][e] + kk1[n][e], k1 = kk[n][e + 1] + kk1[n][e + 1], q0 = qk[n][e] + qk1[n][e], q1 = qk[n][e + 1] + qk1[n][e + 1];
-        const float f0 = s.fk[j], f1 = s.fk[j + 1], fi = s.beta_k[i], fo = s.fq[i];
-        uint32_t hi, lo;
-        if (a == b) {
-          *reinterpret_cast<float2*>(s.diagonal[a] + (i & 15) * DP + (j & 15)) = make_float2(k0 * fi * f0, k1 * fi * f1);      // (read below its diagonal)
-        } else {
-          split2(k0 * fi * f0, k1 * fi * f1, hi, lo);
-          *reinterpret_cast<uint32_t*>(s.a_hi + i * AP + j) = hi;
-          *reinterpret_cast<uint32_t*>(s.a_lo + i * AP + j) = lo;
-        }
-        split2(j <= i ? q0 * fo * f0 : 0.f, j + 1 <= i ? q1 * fo * f1 : 0.f, hi, lo);
-        uint8_t* at = unit + p.unit.b() + i * 128 + (((j >> 3) ^ (i & 7)) << 4) + (j & 7) * 2;
-        *reinterpret_cast<uint32_t*>(at) = hi;
-        *reinterpret_cast<uint32_t*>(at + 8192) = lo;
-      }
-  }
-  if (warp < 4) {                        // a lane per column of the inverse
-    __syncwarp();
-    const int c = lane & 15;
-    const float* blk = s.diagonal[warp];
-    float x[16];
-#pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      float r[4] = {i == c ? 1.f : 0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-      for (int j = 0; j < i; j += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(blk + i * DP + j);
-        r[0] = fmaf(-a.x, x[j], r[0]);
-        if (j + 1 < i) r[1] = fmaf(-a.y, x[j + 1], r[1]);
-        if (j + 2 < i) r[2] = fmaf(-a.z, x[j + 2], r[2]);
-        if (j + 3 < i) r[3] = fmaf(-a.w, x[j + 3], r[3]);
-      }
-      x[i] = (r[0] + r[1]) + (r[2] + r[3]);
-    }
-    if (lane < 16) {
-      const int at = warp * 16 * AP + warp * 16 + c;
+    if (tid < C) s.beta[tid] = tid < n_now ? mx::sigmoid_t<bf16>(__bfloat162float(beta_raw)) : 0.f;
+    if (tid < 4) s.direct[tid] = 0;
+    if (tid == 4) s.next = 0;
+    __syncthreads();
+    {                                      // running sums inside the blocks: a thread per (block, channel)
+      const int b = tid >> 7, c = tid & 127;
+      float* x = s.L + b * 16 * LP + c;
+      float sum = 0.f;
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
-        const bf16 hi = __float2bfloat16(x[i]);
-        s.a_hi[at + i * AP] = hi;
-        s.a_lo[at + i * AP] = __float2bfloat16(x[i] - __bfloat162float(hi));
+        sum += x[i * LP];
+        x[i * LP] = sum;
       }
+      s.D[b][c] = sum;
+      if (sum < kFar) s.direct[b] = 1;
     }
-  }
-  // ---- keys decayed to the chunk's end: two rows at a time by whichever warp has nothing else to do
-  for (;;) {
-    int turn = 0;
-    if (lane == 0) turn = atomicAdd(&s.next, 1);
-    turn = __shfl_sync(0xffffffffu, turn, 0);
-    if (turn >= C / 2) break;
-    const int r = turn * 2 + (lane >> 4), piece = lane & 15, c = piece * 8, at = r * P + c;
-    if (c < kdk * 16) {
-      float x[8], y[8], f[8];
-      mx::load_n<8>(s.c_hi + at, x);
-      mx::load_n<8>(s.c_lo + at, y);
-      mx::load_n<8>(s.after[r >> 4] + c, f);
-      const float scale = s.fk[r];
+    __syncthreads();
+    if (tid < 128) {
+      const float d0 = s.D[0][tid], d1 = s.D[1][tid], d2 = s.D[2][tid], d3 = s.D[3][tid];
+      s.before[0][tid] = 1.f;
+      s.before[1][tid] = e2(d0);
+      s.before[2][tid] = e2(d0 + d1);
+      s.before[3][tid] = e2(d0 + d1 + d2);
+      s.after[0][tid] = e2(d1 + d2 + d3);
+      s.after[1][tid] = e2(d2 + d3);
+      s.after[2][tid] = e2(d3);
+      s.after[3][tid] = 1.f;
+      s.between[0][tid] = e2(fminf(-d0, -kFar));           // blocks beyond are summed directly
+      s.between[1][tid] = e2(fminf(-d1, -kFar));
+      s.between[2][tid] = e2(fminf(-d2, -kFar));
+      s.between[3][tid] = e2(fminf(-d3, -kFar));
+      s.between[4][tid] = e2(d1);
+      s.between[5][tid] = e2(d1 + d2);
+      s.between[6][tid] = e2(d2);
+      reinterpret_cast<float*>(unit + p.unit.decay())[tid] = e2(d0 + d1 + d2 + d3);
+    } else if (tid < 128 + C) {
+      s.beta_k[tid - 128] = s.beta[tid - 128] * s.fk[tid - 128];
+    }
+    __syncthreads();
+    // ---- q and k decayed from the start of their block, k to its end; queries decayed from the chunk's start
 #pragma unroll
-      for (int j = 0; j < 8; ++j) x[j] = (x[j] + y[j]) * (f[j] * scale);
+    for (int i = 0; i < 2; ++i) {
+      const int r = my_row + i * 32, c = my_c, at = r * P + c;
+      float q[8], k[8], l[8], d[8], x[8];
       uint4 hi, lo;
+      const uint32_t qw[4] = {q_in[i].x, q_in[i].y, q_in[i].z, q_in[i].w}, kw[4] = {k_in[i].x, k_in[i].y, k_in[i].z, k_in[i].w};
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        q[j] = (j & 1) ? hi16(qw[j / 2]) : lo16(qw[j / 2]);
+        k[j] = (j & 1) ? hi16(kw[j / 2]) : lo16(kw[j / 2]);
+      }
+      mx::load_n<8>(s.L + r * LP + c, l);
+      mx::load_n<8>(s.D[r >> 4] + c, d);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        d[j] = k[j] * e2(d[j] - l[j]);
+        l[j] = e2(l[j]);
+        x[j] = q[j] * l[j];
+      }
       split8(x, hi, lo);
-      uint8_t* to = unit + p.unit.k() + r * KR * 2 + ((piece ^ (r & 7)) << 4);
-      *reinterpret_cast<uint4*>(to) = hi;
-      *reinterpret_cast<uint4*>(to + half) = lo;
+      *reinterpret_cast<uint4*>(s.q_hi + at) = hi;
+      *reinterpret_cast<uint4*>(s.q_lo + at) = lo;
+      if (c < kdk * 16) {
+        float f[8];
+        mx::load_n<8>(s.before[r >> 4] + c, f);
+        const float scale = s.fq[r];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] *= f[j] * scale;
+        split8(x, hi, lo);
+        uint8_t* to = unit + p.unit.q() + r * KR * 2 + (((c >> 3) ^ (r & 7)) << 4);
+        *reinterpret_cast<uint4*>(to) = hi;
+        *reinterpret_cast<uint4*>(to + half) = lo;
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[j] = k[j] * l[j];
+      split8(x, hi, lo);
+      *reinterpret_cast<uint4*>(s.k_hi + at) = hi;
+      *reinterpret_cast<uint4*>(s.k_lo + at) = lo;
+      split8(d, hi, lo);
+      *reinterpret_cast<uint4*>(s.c_hi + at) = hi;
+      *reinterpret_cast<uint4*>(s.c_lo + at) = lo;
     }
-  }
-  fence_proxy_async();                   // what was written to the tiles comes before the copies into them
-  __syncthreads();
-  if (after_idx < n_units) fetch(after_idx);
-  // ---- X = T·[β v | β k e^G] by blocks of tokens, transposed: a warp's 16 columns are the rows of its products
-  const int a_row = (lane & 7) + ((lane >> 4) << 3), a_col = ((lane >> 3) & 1) * 8;
-  const int r_row = (lane & 7) + ((lane >> 4) << 3), r_col = ((lane >> 3) & 1) * 8;
-  for (int mt = warp; mt < kdv + kdk; mt += kThreads / 32) {
-    const bool is_u = mt < kdv;
-    const int c0 = (is_u ? mt : mt - kdv) * 16;
-    uint8_t* w_rows = reinterpret_cast<uint8_t*>(s.L) + (mt - kdv) % 8 * 4096;      // 16 rows of W, hi and lo, on their way out (the decays are not needed any more)
-    uint32_t xh[4][4], xl[4][4];
-#pragma unroll
-    for (int a = 0; a < 4; ++a) {
-      float acc[2][4], acc1[2][4];
-      // rows of A (or T) are the columns of the second factor; the products with low parts have sums of their own
-      auto times = [&](const uint32_t (&yh)[4], const uint32_t (&yl)[4], int b) {
-        uint32_t bh[4], bl[4];
-        const int at = (a * 16 + a_row) * AP + b * 16 + a_col;
-        ldsm4(smem_u32(s.a_hi + at), bh);
-        ldsm4(smem_u32(s.a_lo + at), bl);
-        mma(acc[0], yh, bh[0], bh[1]);
-        mma(acc[1], yh, bh[2], bh[3]);
-        mma(acc1[0], yh, bl[0], bl[1]);
-        mma(acc1[1], yh, bl[2], bl[3]);
-        mma(acc1[0], yl, bh[0], bh[1]);
-        mma(acc1[1], yl, bh[2], bh[3]);
-      };
-      auto clear = [&]() {
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) acc[n][e] = acc1[n][e] = 0.f;
-      };
-      auto sum = [&]() {
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) acc[n][e] += acc1[n][e];
-      };
-      clear();
-#pragma unroll
-      for (int b = 0; b < a; ++b) times(xh[b], xl[b], b);
-      sum();
-      // the block's right-hand side, transposed on its way from shared memory: register 2n + e holds tokens 8n + 2·t4 and the next of column g + 8e
-      const int at = (a * 16 + r_row) * P + c0 + r_col;
-      if (is_u) {
-        uint32_t v[4];
-        ldsm4t(smem_u32(s.v + at), v);
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          const float2 f = *reinterpret_cast<const float2*>(s.beta + a * 16 + n * 8 + t4 * 2);
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            acc[n][e * 2] = fmaf(lo16(v[n * 2 + e]), f.x, -acc[n][e * 2]);
-            acc[n][e * 2 + 1] = fmaf(hi16(v[n * 2 + e]), f.y, -acc[n][e * 2 + 1]);
+    __syncthreads();
+    // ---- A and B, a warp per pair of blocks; the diagonal blocks of I + A are inverted by the warps that made them
+    if (warp < 10) {
+      int a, b;
+      pair_of(warp, a, b);
+      float kk[2][4] = {}, qk[2][4] = {}, kk1[2][4] = {}, qk1[2][4] = {};      // (the products with low parts have sums of their own)
+      if (a == b && s.direct[a]) {
+#pragma unroll 1
+        for (int x = 0; x < 8; ++x) {
+          const int i = a * 16 + g + (x & 2) * 4, j = a * 16 + (x >> 2) * 8 + t4 * 2 + (x & 1);
+          float sk = 0.f, sq = 0.f;
+          if (j <= i && i < n_now) {
+            const bf16* qi = p.act + static_cast<long long>(t0_now + i) * CH + gq * K;
+            const bf16* ki = qi + p.m.G * K;
+            const bf16* kj = p.act + static_cast<long long>(t0_now + j) * CH + p.m.G * K + gq * K;
+            for (int c = 0; c < K; ++c) {
+              const float w = __bfloat162float(kj[c]) * e2(s.L[i * LP + c] - s.L[j * LP + c]);
+              sk = fmaf(__bfloat162float(ki[c]), w, sk);
+              sq = fmaf(__bfloat162float(qi[c]), w, sq);
+            }
           }
+#pragma unroll
+          for (int y = 0; y < 8; ++y)
+            if (y == x) { kk[y >> 2][y & 3] = sk; qk[y >> 2][y & 3] = sq; }
         }
+        __syncwarp();
       } else {
-        uint32_t v[4], w[4];
-        ldsm4t(smem_u32(s.k_hi + at), v);
-        ldsm4t(smem_u32(s.k_lo + at), w);
-        const float from[2] = {s.before[a][c0 + g], s.before[a][c0 + g + 8]};
+        const int row_a = (a * 16 + (lane & 15)) * P + (lane >> 4) * 8;
+        const int row_b = (b * 16 + (lane & 7) + ((lane >> 4) << 3)) * P + ((lane >> 3) & 1) * 8;
+        const float* fac = s.between[min(warp, 6)];
+#pragma unroll 2
+        for (int ks = 0; ks < kdk; ++ks) {
+          uint32_t qh[4], ql[4], kh[4], kl[4], ch[4], cl[4];
+          ldsm4(smem_u32(s.c_hi + row_b + ks * 16), ch);
+          ldsm4(smem_u32(s.c_lo + row_b + ks * 16), cl);
+          ldsm4(smem_u32(s.k_hi + row_a + ks * 16), kh);
+          ldsm4(smem_u32(s.q_hi + row_a + ks * 16), qh);
+          ldsm4(smem_u32(s.k_lo + row_a + ks * 16), kl);
+          ldsm4(smem_u32(s.q_lo + row_a + ks * 16), ql);
+          if (warp < 7) {
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          const float2 f = *reinterpret_cast<const float2*>(s.beta_k + a * 16 + n * 8 + t4 * 2);
+            for (int i = 0; i < 2; ++i) {
+              const float2 f = *reinterpret_cast<const float2*>(fac + ks * 16 + i * 8 + t4 * 2);
 #pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            acc[n][e * 2] = fmaf(lo16(v[n * 2 + e]) + lo16(w[n * 2 + e]), f.x * from[e], -acc[n][e * 2]);
-            acc[n][e * 2 + 1] = fmaf(hi16(v[n * 2 + e]) + hi16(w[n * 2 + e]), f.y * from[e], -acc[n][e * 2 + 1]);
+              for (int n = 0; n < 4; n += 2) split2((lo16(ch[n + i]) + lo16(cl[n + i])) * f.x, (hi16(ch[n + i]) + hi16(cl[n + i])) * f.y, ch[n + i], cl[n + i]);
+            }
+          }
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            mma(kk[n], kh, ch[2 * n], ch[2 * n + 1]);
+            mma(qk[n], qh, ch[2 * n], ch[2 * n + 1]);
+          }
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            mma(kk1[n], kh, cl[2 * n], cl[2 * n + 1]);
+            mma(qk1[n], qh, cl[2 * n], cl[2 * n + 1]);
+          }
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            mma(kk1[n], kl, ch[2 * n], ch[2 * n + 1]);
+            mma(qk1[n], ql, ch[2 * n], ch[2 * n + 1]);
           }
         }
       }
-      uint32_t yh[4], yl[4];
-      operand(acc[0], acc[1], yh, yl);
-      clear();
-      times(yh, yl, a);
-      sum();
-      operand(acc[0], acc[1], xh[a], xl[a]);
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int c = c0 + g + e * 8, t = a * 16 + n * 8 + t4 * 2;
-          if (is_u) {
-            *reinterpret_cast<float2*>(unit + p.unit.u() + c * kUPitch + t * 4) = make_float2(acc[n][e * 2], acc[n][e * 2 + 1]);
-          } else {                       // −W: the second kernel adds
-            uint8_t* to = w_rows + (g + e * 8) * 128 + (((t >> 3) ^ (c & 7)) << 4) + (t & 7) * 2;
-            *reinterpret_cast<uint32_t*>(to) = xh[a][n * 2 + e] ^ 0x80008000u;
-            *reinterpret_cast<uint32_t*>(to + 2048) = xl[a][n * 2 + e] ^ 0x80008000u;
+        for (int e = 0; e < 4; e += 2) {
+          const int i = a * 16 + g + e * 4, j = b * 16 + n * 8 + t4 * 2;
+          const float k0 = kk[n][e] + kk1[n][e], k1 = kk[n][e + 1] + kk1[n][e + 1], q0 = qk[n][e] + qk1[n][e], q1 = qk[n][e + 1] + qk1[n][e + 1];
+          const float f0 = s.fk[j], f1 = s.fk[j + 1], fi = s.beta_k[i], fo = s.fq[i];
+          uint32_t hi, lo;
+          if (a == b) {
+            *reinterpret_cast<float2*>(s.diagonal[a] + (i & 15) * DP + (j & 15)) = make_float2(k0 * fi * f0, k1 * fi * f1);      // (read below its diagonal)
+          } else {
+            split2(k0 * fi * f0, k1 * fi * f1, hi, lo);
+            *reinterpret_cast<uint32_t*>(s.a_hi + i * AP + j) = hi;
+            *reinterpret_cast<uint32_t*>(s.a_lo + i * AP + j) = lo;
           }
+          split2(j <= i ? q0 * fo * f0 : 0.f, j + 1 <= i ? q1 * fo * f1 : 0.f, hi, lo);
+          uint8_t* at = unit + p.unit.b() + i * 128 + (((j >> 3) ^ (i & 7)) << 4) + (j & 7) * 2;
+          *reinterpret_cast<uint32_t*>(at) = hi;
+          *reinterpret_cast<uint32_t*>(at + 8192) = lo;
         }
     }
-    if (!is_u) {
+    if (warp < 4) {                        // a lane per column of the inverse
       __syncwarp();
+      const int c = lane & 15;
+      const float* blk = s.diagonal[warp];
+      float x[16];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int at = (i * 32 + lane) * 16;
-        *reinterpret_cast<uint4*>(unit + c0 * 128 + at) = *reinterpret_cast<const uint4*>(w_rows + at);
-        *reinterpret_cast<uint4*>(unit + half + c0 * 128 + at) = *reinterpret_cast<const uint4*>(w_rows + 2048 + at);
+      for (int i = 0; i < 16; ++i) {
+        float r[4] = {i == c ? 1.f : 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int j = 0; j < i; j += 4) {
+          const float4 a = *reinterpret_cast<const float4*>(blk + i * DP + j);
+          r[0] = fmaf(-a.x, x[j], r[0]);
+          if (j + 1 < i) r[1] = fmaf(-a.y, x[j + 1], r[1]);
+          if (j + 2 < i) r[2] = fmaf(-a.z, x[j + 2], r[2]);
+          if (j + 3 < i) r[3] = fmaf(-a.w, x[j + 3], r[3]);
+        }
+        x[i] = (r[0] + r[1]) + (r[2] + r[3]);
       }
-      __syncwarp();
+      if (lane < 16) {
+        const int at = warp * 16 * AP + warp * 16 + c;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const bf16 hi = __float2bfloat16(x[i]);
+          s.a_hi[at + i * AP] = hi;
+          s.a_lo[at + i * AP] = __float2bfloat16(x[i] - __bfloat162float(hi));
+        }
+      }
     }
-  }
+    // ---- keys decayed to the chunk's end: two rows at a time by whichever warp has nothing else to do
+    for (;;) {
+      int turn = 0;
+      if (lane == 0) turn = atomicAdd(&s.next, 1);
+      turn = __shfl_sync(0xffffffffu, turn, 0);
+      if (turn >= C / 2) break;
+      const int r = turn * 2 + (lane >> 4), piece = lane & 15, c = piece * 8, at = r * P + c;
+      if (c < kdk * 16) {
+        float x[8], y[8], f[8];
+        mx::load_n<8>(s.c_hi + at, x);
+        mx::load_n<8>(s.c_lo + at, y);
+        mx::load_n<8>(s.after[r >> 4] + c, f);
+        const float scale = s.fk[r];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] = (x[j] + y[j]) * (f[j] * scale);
+        uint4 hi, lo;
+        split8(x, hi, lo);
+        uint8_t* to = unit + p.unit.k() + r * KR * 2 + ((piece ^ (r & 7)) << 4);
+        *reinterpret_cast<uint4*>(to) = hi;
+        *reinterpret_cast<uint4*>(to + half) = lo;
+      }
+    }
+    fence_proxy_async();                   // what was written to the tiles comes before the copies into them
+    __syncthreads();
+    if (after_idx < n_units) fetch(after_idx);
+    // ---- X = T·[β v | β k e^G] by blocks of tokens, transposed: a warp's 16 columns are the rows of its products
+    const int a_row = (lane & 7) + ((lane >> 4) << 3), a_col = ((lane >> 3) & 1) * 8;
+    const int r_row = (lane & 7) + ((lane >> 4) << 3), r_col = ((lane >> 3) & 1) * 8;
+    for (int mt = warp; mt < kdv + kdk; mt += kThreads / 32) {
+      const bool is_u = mt < kdv;
+      const int c0 = (is_u ? mt : mt - kdv) * 16;
+      uint8_t* w_rows = reinterpret_cast<uint8_t*>(s.L) + (mt - kdv) % 8 * 4096;      // 16 rows of W, hi and lo, on their way out (the decays are not needed any more)
+      uint32_t xh[4][4], xl[4][4];
+#pragma unroll
+      for (int a = 0; a < 4; ++a) {
+        float acc[2][4], acc1[2][4];
+        // rows of A (or T) are the columns of the second factor; the products with low parts have sums of their own
+        auto times = [&](const uint32_t (&yh)[4], const uint32_t (&yl)[4], int b) {
+          uint32_t bh[4], bl[4];
+          const int at = (a * 16 + a_row) * AP + b * 16 + a_col;
+          ldsm4(smem_u32(s.a_hi + at), bh);
+          ldsm4(smem_u32(s.a_lo + at), bl);
+          mma(acc[0], yh, bh[0], bh[1]);
+          mma(acc[1], yh, bh[2], bh[3]);
+          mma(acc1[0], yh, bl[0], bl[1]);
+          mma(acc1[1], yh, bl[2], bl[3]);
+          mma(acc1[0], yl, bh[0], bh[1]);
+          mma(acc1[1], yl, bh[2], bh[3]);
+        };
+        auto clear = [&]() {
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[n][e] = acc1[n][e] = 0.f;
+        };
+        auto sum = [&]() {
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[n][e] += acc1[n][e];
+        };
+        clear();
+#pragma unroll
+        for (int b = 0; b < a; ++b) times(xh[b], xl[b], b);
+        sum();
+        // the block's right-hand side, transposed on its way from shared memory: register 2n + e holds tokens 8n + 2·t4 and the next of column g + 8e
+        const int at = (a * 16 + r_row) * P + c0 + r_col;
+        if (is_u) {
+          uint32_t v[4];
+          ldsm4t(smem_u32(s.v + at), v);
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const float2 f = *reinterpret_cast<const float2*>(s.beta + a * 16 + n * 8 + t4 * 2);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              acc[n][e * 2] = fmaf(lo16(v[n * 2 + e]), f.x, -acc[n][e * 2]);
+              acc[n][e * 2 + 1] = fmaf(hi16(v[n * 2 + e]), f.y, -acc[n][e * 2 + 1]);
+            }
+          }
+        } else {
+          uint32_t v[4], w[4];
+          ldsm4t(smem_u32(s.k_hi + at), v);
+          ldsm4t(smem_u32(s.k_lo + at), w);
+          const float from[2] = {s.before[a][c0 + g], s.before[a][c0 + g + 8]};
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const float2 f = *reinterpret_cast<const float2*>(s.beta_k + a * 16 + n * 8 + t4 * 2);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              acc[n][e * 2] = fmaf(lo16(v[n * 2 + e]) + lo16(w[n * 2 + e]), f.x * from[e], -acc[n][e * 2]);
+              acc[n][e * 2 + 1] = fmaf(hi16(v[n * 2 + e]) + hi16(w[n * 2 + e]), f.y * from[e], -acc[n][e * 2 + 1]);
+            }
+          }
+        }
+        uint32_t yh[4], yl[4];
+        operand(acc[0], acc[1], yh, yl);
+        clear();
+        times(yh, yl, a);
+        sum();
+        operand(acc[0], acc[1], xh[a], xl[a]);
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int c = c0 + g + e * 8, t = a * 16 + n * 8 + t4 * 2;
+            if (is_u) {
+              *reinterpret_cast<float2*>(unit + p.unit.u() + c * kUPitch + t * 4) = make_float2(acc[n][e * 2], acc[n][e * 2 + 1]);
+            } else {                       // −W: the second kernel adds
+              uint8_t* to = w_rows + (g + e * 8) * 128 + (((t >> 3) ^ (c & 7)) << 4) + (t & 7) * 2;
+              *reinterpret_cast<uint32_t*>(to) = xh[a][n * 2 + e] ^ 0x80008000u;
+              *reinterpret_cast<uint32_t*>(to + 2048) = xl[a][n * 2 + e] ^ 0x80008000u;
+            }
+          }
+      }
+      if (!is_u) {
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int at = (i * 32 + lane) * 16;
+          *reinterpret_cast<uint4*>(unit + c0 * 128 + at) = *reinterpret_cast<const uint4*>(w_rows + at);
+          *reinterpret_cast<uint4*>(unit + half + c0 * 128 + at) = *reinterpret_cast<const uint4*>(w_rows + 2048 + at);
+        }
+        __syncwarp();
+      }
+    }
   }
 }
 

@@ -130,69 +130,71 @@ __global__ void __launch_bounds__(128) delta_seq_kernel(const T* __restrict__ pr
     if (col < V) st[static_cast<long long>(d) * V + col] = S[d * kSlice + lane];
 }
 
-static constexpr int kStep = 256;
-// grid (heads, rows), 256 threads; V % 4 == 0.  A thread owns four columns of U state rows, 256 / (V / 4) rows apart.
-template <typename T, int U>
-__global__ void __launch_bounds__(kStep, U <= 4 ? 4 : U <= 8 ? 3 : 2) delta_step_kernel(const T* __restrict__ proj, long long ld, MbDelta m, const T* __restrict__ norm_w,
-                                                           const T* __restrict__ gate, long long gate_ld, float eps, T* __restrict__ out) {
+static constexpr int kStepRows = 16, kStepThreads = 512;      // state rows of a lane, threads of a CTA at most
+// grid (heads, rows of the batch), 32·⌈V/16⌉ threads; V % 4 == 0.  A warp owns 16 state columns: lane = (4 columns lane % 4, rows lane / 4 + 8·u), so
+// that both sums over rows are exchanges inside the warp.  THREADS: the most a launch has.
+template <typename T, int U, int THREADS>
+__global__ void __launch_bounds__(THREADS, 512 / THREADS) delta_step_kernel(const T* __restrict__ proj, long long ld, MbDelta m, const T* __restrict__ norm_w,
+                                                                            const T* __restrict__ gate, long long gate_ld, float eps, T* __restrict__ out) {
   extern __shared__ __align__(16) float sm[];
-  __shared__ float sh[kStep / 32];
-  __shared__ float unit[2];
+  __shared__ float part[kStepThreads / 32];
   pdl_trigger();
   pdl_wait();
   const int K = m.K, V = m.V, H = m.H, CH = channels_of(m), h = blockIdx.x, b = blockIdx.y, per = H / m.G, g = h / per;
-  const int slot = m.slots[b];
+  const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31;
+  const int slot = m.slots[b], pos = m.positions[b];
   T* o = out + (static_cast<long long>(b) * H + h) * V;
   if (slot < 0) {                        // padding row
-    for (int i = threadIdx.x; i < V; i += kStep) o[i] = from_f<T>(0.f);
+    for (int i = tid; i < V; i += threads) o[i] = from_f<T>(0.f);
     return;
   }
-  const int cg = V / 4, rpp = kStep / cg;                // column groups, state rows per pass
-  float* red = sm;                       // [rpp][V]
-  float* sx = red + rpp * V;             // [K | K | V]: q, k, v of this token
+  float* sx = sm;                        // [K | K | V]: q, k, v of this token
   float* sg = sx + 2 * K + V;            // [K] decays
-  const int row0 = threadIdx.x / cg, col = (threadIdx.x % cg) * 4;
-  const bool on = row0 < rpp;
+  const int row0 = lane >> 2, col = warp * 16 + (lane & 3) * 4;
+  const bool on = col < V;
   float* st = m.state + (static_cast<long long>(slot) * H + h) * K * V + col;
-  const int pos = m.positions[b];
   // the state is on its way while the projections of this token are read, convolved and activated
   float4 s[U];
 #pragma unroll
   for (int u = 0; u < U; ++u) {
-    const int d = row0 + u * rpp;
+    const int d = row0 + u * 8;
     s[u] = (on && pos > 0 && d < K) ? *reinterpret_cast<const float4*>(st + static_cast<long long>(d) * V) : make_float4(0, 0, 0, 0);
   }
   const T* p = proj + b * ld;
   const T* W = reinterpret_cast<const T*>(m.conv_w);
   float* ring = m.ring != nullptr ? m.ring + static_cast<long long>(slot) * m.taps * CH : nullptr;
-  const T* gt = gate + b * gate_ld + h * V;
-  const float gate0 = threadIdx.x < V ? to_f(gt[threadIdx.x]) : 0.f, norm0 = threadIdx.x < V ? to_f(norm_w[threadIdx.x]) : 0.f;
+  const T* gt = gate + b * gate_ld + h * V + col;
+  float gv[4], nv[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    gv[j] = on ? to_f(gt[j]) : 0.f;
+    nv[j] = on ? to_f(norm_w[col + j]) : 0.f;
+  }
   const float beta = sigmoid_t<T>(to_f(p[m.beta_at + h])), rate = exp_t<T>(to_f(reinterpret_cast<const T*>(m.A_log)[h]));
-  for (int i = threadIdx.x; i < K; i += kStep)
-    sg[i] = decay_of<T>(to_f(reinterpret_cast<const T*>(m.raw)[b * m.raw_ld + h * K + i]), to_f(reinterpret_cast<const T*>(m.dt_bias)[h * K + i]), rate);
-  constexpr int R = 2;                                   // channels of a thread that are on their way together
+  // everything that is read is on its way before anything is written
+  const T* raw = reinterpret_cast<const T*>(m.raw) + b * m.raw_ld + h * K;
+  const T* bias = reinterpret_cast<const T*>(m.dt_bias) + h * K;
+  const float raw0 = tid < K ? to_f(raw[tid]) : 0.f, bias0 = tid < K ? to_f(bias[tid]) : 0.f;
   const int n = 2 * K + V;
   auto channel = [&](int i) { return i < K ? g * K + i : i < 2 * K ? (m.G + g) * K + i - K : 2 * m.G * K + h * V + i - 2 * K; };
-  for (int i0 = threadIdx.x; i0 < n; i0 += R * kStep) {
+  constexpr int R = 3;                   // channels of a thread at a time
+  for (int i0 = tid; i0 < n; i0 += R * threads) {
     float x[R], y[R];
 #pragma unroll
     for (int u = 0; u < R; ++u) {
-      const int i = i0 + u * kStep;
-      x[u] = y[u] = 0.f;
-      if (i >= n) continue;
-      const int c = channel(i);
+      const int i = i0 + u * threads, c = channel(min(i, n - 1));
       x[u] = to_f(p[c]);
       y[u] = to_f(W[static_cast<long long>(c) * m.taps + m.taps - 1]) * x[u];
     }
-    for (int k0 = 1; k0 < m.taps; k0 += 3) {             // three inputs back at a time, all on their way together
+    for (int k0 = 1; k0 < m.taps; k0 += 3) {             // three inputs back at a time
       float f[R][3], w[R][3];
 #pragma unroll
       for (int u = 0; u < R; ++u) {
-        const int i = i0 + u * kStep, c = i < n ? channel(i) : 0;
+        const int c = channel(min(i0 + u * threads, n - 1));
 #pragma unroll
         for (int k = 0; k < 3; ++k) {
           const int q = pos - k0 - k;
-          const bool ok = i < n && k0 + k < m.taps && q >= 0;
+          const bool ok = k0 + k < m.taps && q >= 0;
           f[u][k] = ok ? ring[static_cast<long long>(q % m.taps) * CH + c] : 0.f;
           w[u][k] = ok ? to_f(W[static_cast<long long>(c) * m.taps + m.taps - 1 - k0 - k]) : 0.f;
         }
@@ -204,29 +206,35 @@ __global__ void __launch_bounds__(kStep, U <= 4 ? 4 : U <= 8 ? 3 : 2) delta_step
     }
 #pragma unroll
     for (int u = 0; u < R; ++u) {
-      const int i = i0 + u * kStep;
+      const int i = i0 + u * threads;
       if (i >= n) continue;
       sx[i] = to_f(from_f<T>(silu_t<T>(y[u])));          // as the general path stores it
       if (ring != nullptr && (i >= 2 * K || h % per == 0)) ring[static_cast<long long>(pos % m.taps) * CH + channel(i)] = x[u];
     }
   }
-  __syncthreads();
-  if (threadIdx.x < 64) {                // warp 0: length of q, warp 1: of k
-    const float* x = sx + (threadIdx.x >> 5) * K;
-    float ss = 0.f;
-    for (int d = threadIdx.x & 31; d < K; d += 32) ss = fmaf(x[d], x[d], ss);
-    ss = warp_sum(ss);
-    if ((threadIdx.x & 31) == 0)
-      unit[threadIdx.x >> 5] = rsqrt_exact(ss + kUnitEps) * (threadIdx.x < 32 ? __fdiv_rn(1.f, __fsqrt_rn(static_cast<float>(K))) : 1.f);
+  for (int i = tid; i < K; i += threads) {
+    const bool first = i == tid;
+    sg[i] = decay_of<T>(first ? raw0 : to_f(raw[i]), first ? bias0 : to_f(bias[i]), rate);
   }
   __syncthreads();
-  const float fq = unit[0], fk = unit[1];
-  if (on) {
-    float y[4] = {0.f, 0.f, 0.f, 0.f};
+  float fq = 0.f, fk = 0.f;              // every warp finds the lengths of q and k
+  for (int d = lane; d < K; d += 32) {
+    fq = fmaf(sx[d], sx[d], fq);
+    fk = fmaf(sx[K + d], sx[K + d], fk);
+  }
+  fq = rsqrt_exact(warp_sum(fq) + kUnitEps) * __fdiv_rn(1.f, __fsqrt_rn(static_cast<float>(K)));
+  fk = rsqrt_exact(warp_sum(fk) + kUnitEps);
+  auto over_rows = [&](float (&y)[4]) {
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int d = row0 + u * rpp;
-      if (d >= K) break;
+    for (int x = 4; x < 32; x <<= 1)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) y[j] += __shfl_xor_sync(0xffffffffu, y[j], x);
+  };
+  float y[4] = {0.f, 0.f, 0.f, 0.f}, a[4];
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int d = row0 + u * 8;
+    if (d < K) {
       const float dec = sg[d], k = sx[K + d] * fk;
       s[u].x *= dec; s[u].y *= dec; s[u].z *= dec; s[u].w *= dec;
       y[0] = fmaf(s[u].x, k, y[0]);
@@ -234,25 +242,17 @@ __global__ void __launch_bounds__(kStep, U <= 4 ? 4 : U <= 8 ? 3 : 2) delta_step
       y[2] = fmaf(s[u].z, k, y[2]);
       y[3] = fmaf(s[u].w, k, y[3]);
     }
-    *reinterpret_cast<float4*>(red + row0 * V + col) = make_float4(y[0], y[1], y[2], y[3]);
   }
-  __syncthreads();
-  float a[4] = {0.f, 0.f, 0.f, 0.f};
-  if (on) {
-    for (int w = 0; w < rpp; ++w) {
-      const float4 r = *reinterpret_cast<const float4*>(red + w * V + col);
-      a[0] += r.x; a[1] += r.y; a[2] += r.z; a[3] += r.w;
-    }
+  over_rows(y);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) a[j] = beta * (sx[2 * K + col + j] - a[j]);
+  for (int j = 0; j < 4; ++j) {
+    a[j] = on ? beta * (sx[2 * K + col + j] - y[j]) : 0.f;
+    y[j] = 0.f;
   }
-  __syncthreads();
-  if (on) {
-    float y[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int d = row0 + u * rpp;
-      if (d >= K) break;
+  for (int u = 0; u < U; ++u) {
+    const int d = row0 + u * 8;
+    if (d < K) {
       const float k = sx[K + d] * fk, q = sx[d] * fq;
       s[u].x = fmaf(k, a[0], s[u].x);
       s[u].y = fmaf(k, a[1], s[u].y);
@@ -262,24 +262,19 @@ __global__ void __launch_bounds__(kStep, U <= 4 ? 4 : U <= 8 ? 3 : 2) delta_step
       y[1] = fmaf(s[u].y, q, y[1]);
       y[2] = fmaf(s[u].z, q, y[2]);
       y[3] = fmaf(s[u].w, q, y[3]);
-      *reinterpret_cast<float4*>(st + static_cast<long long>(d) * V) = s[u];
+      if (on) *reinterpret_cast<float4*>(st + static_cast<long long>(d) * V) = s[u];
     }
-    *reinterpret_cast<float4*>(red + row0 * V + col) = make_float4(y[0], y[1], y[2], y[3]);
   }
+  over_rows(y);
+  const float ss = warp_sum(lane < 4 && on ? y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3] : 0.f);
+  if (lane == 0) part[warp] = ss;
   __syncthreads();
-  float ss = 0.f, r0 = 0.f;
-  for (int i = threadIdx.x; i < V; i += kStep) {
-    float r = 0.f;
-    for (int w = 0; w < rpp; ++w) r += red[w * V + i];
-    ss = fmaf(r, r, ss);
-    if (i == threadIdx.x) r0 = r;
-    else red[i] = r;                     // row 0 of a column that only this thread reads
-  }
-  const float rstd = rsqrt_exact(__fdiv_rn(block_sum<kStep>(ss, sh), static_cast<float>(V)) + eps);
-  for (int i = threadIdx.x; i < V; i += kStep) {
-    const bool mine = i == threadIdx.x;
-    o[i] = from_f<T>((mine ? r0 : red[i]) * rstd * (mine ? norm0 : to_f(norm_w[i])) * sigmoid_t<T>(mine ? gate0 : to_f(gt[i])));
-  }
+  if (lane >= 4 || !on) return;
+  float sum = 0.f;
+  for (int w = 0; w < threads / 32; ++w) sum += part[w];
+  const float rstd = rsqrt_exact(__fdiv_rn(sum, static_cast<float>(V)) + eps);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) o[col + j] = from_f<T>(y[j] * rstd * nv[j] * sigmoid_t<T>(gv[j]));
 }
 
 static bool sizes_ok(const MbDelta& m) {
@@ -330,21 +325,19 @@ extern "C" int mb_delta_seq(const void* proj, long long ld, const void* act, MbD
   return f32 ? run(float{}) : run(bf16{});
 }
 
-static constexpr int kMaxRows = 16;      // state rows of a thread
-extern "C" int mb_delta_step_max(void) { return kMaxRows * 4 * kStep; }
+extern "C" int mb_delta_step_ok(int K, int V) { return V % 4 == 0 && (V + 15) / 16 * 32 <= kStepThreads && K <= 8 * kStepRows; }
 
 extern "C" int mb_delta_step(const void* proj, long long ld, MbDelta m, const void* norm_w, const void* gate, long long gate_ld, float eps, void* out, int B,
                              int f32, cudaStream_t s) {
   if (B <= 0) return 0;
-  if (!sizes_ok(m) || m.V % 4 || m.V > 4 * kStep || B > 65535) return -3;
-  const int rpp = kStep / (m.V / 4), rows = (m.K + rpp - 1) / rpp;
-  const size_t bytes = (static_cast<size_t>(rpp) * m.V + m.V + 3 * m.K) * sizeof(float);
-  if (rows > kMaxRows || bytes > 48 * 1024) return -3;
+  if (!sizes_ok(m) || !mb_delta_step_ok(m.K, m.V) || B > 65535) return -3;
+  const int rows = (m.K + 7) / 8, threads = (m.V + 15) / 16 * 32;
   auto run = [&](auto ty) {
     using E = decltype(ty);
-    auto kern = rows <= 4 ? delta_step_kernel<E, 4> : rows <= 8 ? delta_step_kernel<E, 8> : delta_step_kernel<E, kMaxRows>;
-    return static_cast<int>(launch_pdl(kern, dim3(m.H, B), dim3(kStep), bytes, s, reinterpret_cast<const E*>(proj), ld, m, reinterpret_cast<const E*>(norm_w),
-                                       reinterpret_cast<const E*>(gate), gate_ld, eps, reinterpret_cast<E*>(out)));
+    auto kern = threads <= 256 ? (rows <= 4 ? delta_step_kernel<E, 4, 256> : rows <= 8 ? delta_step_kernel<E, 8, 256> : delta_step_kernel<E, kStepRows, 256>)
+                               : delta_step_kernel<E, kStepRows, kStepThreads>;
+    return static_cast<int>(launch_pdl(kern, dim3(m.H, B), dim3(threads), (3 * m.K + m.V) * sizeof(float), s, reinterpret_cast<const E*>(proj), ld, m,
+                                       reinterpret_cast<const E*>(norm_w), reinterpret_cast<const E*>(gate), gate_ld, eps, reinterpret_cast<E*>(out)));
   };
   return f32 ? run(float{}) : run(bf16{});
 }

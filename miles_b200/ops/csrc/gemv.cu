@@ -112,10 +112,10 @@ __device__ __forceinline__ float warp_sum(float v) {
 // (8 lanes × 16 bytes) fall on disjoint banks.
 __host__ __device__ inline int staged_stride(int K) { return K * 2 + 64; }
 
-// Stage rows [0, rows) of a [*, K] bf16 matrix into shared memory (rows ≥ valid are zero); warp w takes rows w, w+8, ….
+// Stage rows [0, rows) of a [*, K] bf16 matrix (rows ldx apart) into shared memory (rows ≥ valid are zero); warp w takes rows w, w+8, ….
 // NORM: h = bf16(x + residual) (block 0 also writes it to res_out), Σh² → rstd[row], the staged value is bf16(h · norm_w).
 template <bool NORM>
-__device__ __forceinline__ void stage_rows(uint8_t* xs, int rows, int valid, int K, const bf16* __restrict__ x,
+__device__ __forceinline__ void stage_rows(uint8_t* xs, int rows, int valid, int K, const bf16* __restrict__ x, long long ldx,
                                            const bf16* __restrict__ residual, const bf16* __restrict__ norm_w, float eps,
                                            bf16* res_out, float* rstd) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -125,7 +125,7 @@ __device__ __forceinline__ void stage_rows(uint8_t* xs, int rows, int valid, int
     uint8_t* row = xs + r * stride;
     float ss = 0.f;
     if (r < valid) {
-      const bf16* xr = x + static_cast<long long>(r) * K;
+      const bf16* xr = x + r * ldx;
       for (int v0 = lane; v0 < nv; v0 += 32 * B) {
         uint4 xb[B], rb[B], nb[B];
 #pragma unroll
@@ -282,13 +282,13 @@ __device__ __forceinline__ void stage_rows_sum_norm(uint8_t* xs, int rows, int v
   }
 }
 
-// Plain copy of rows [0, valid) of a [*, K] bf16 matrix into shared memory with cp.async (every piece in flight at once, no
+// Plain copy of rows [0, valid) of a [*, K] bf16 matrix (rows ldx apart) into shared memory with cp.async (every piece in flight at once, no
 // registers); rows [valid, rows) are zeroed.  The caller commits the group and waits for it before the CTA barrier.
-__device__ __forceinline__ void stage_rows_async(uint8_t* xs, int rows, int valid, int K, const bf16* __restrict__ x) {
+__device__ __forceinline__ void stage_rows_async(uint8_t* xs, int rows, int valid, int K, const bf16* __restrict__ x, long long ldx) {
   const int nv = K / 8, stride = staged_stride(K);
   for (int i = threadIdx.x; i < valid * nv; i += kThreads) {
     const int r = i / nv, v = i - r * nv;
-    cp16(smem_addr(xs + r * stride + v * 16), x + static_cast<long long>(r) * K + v * 8);
+    cp16(smem_addr(xs + r * stride + v * 16), x + r * ldx + v * 8);
   }
   for (int i = threadIdx.x; i < (rows - valid) * nv; i += kThreads) {
     const int r = valid + i / nv, v = i % nv;
@@ -297,7 +297,9 @@ __device__ __forceinline__ void stage_rows_async(uint8_t* xs, int rows, int vali
 }
 
 struct GemvParams {
-  const bf16* x;          // [M, K]
+  const bf16* x;          // [M, K], rows ldx apart
+  const bf16* x2;         // kPlain: rows of the second product (null: x)
+  long long ldx;
   const bf16* residual;   // [M, K] or null (NORM only)
   const bf16* norm_w;     // [K] (NORM only)
   float eps;
@@ -365,14 +367,14 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
   for (int i = 0; i < S; ++i) issue(i);
   if (p.static_w) pdl_wait();          // static weights: their first loads are already in flight
   if (NORM) {
-    stage_rows<true>(xs, NT * 8, p.M, p.K, p.x, p.residual, p.norm_w, p.eps, p.res_out, rstd_s);
+    stage_rows<true>(xs, NT * 8, p.M, p.K, p.x, p.ldx, p.residual, p.norm_w, p.eps, p.res_out, rstd_s);
   } else if (MODE == kOutputNorm || MODE == kOutputNormNext) {
     stage_rows_output_norm<MODE == kOutputNormNext>(xs, NT * 8, p.M, p.K, p.x, p.x32, p.norm_w, p.scale_w, p.mult, p.norm_w2, p.eps, p.x32_out, rstd_s);
   } else if (SUM) {
     stage_rows_sum_norm<MODE == kScaledSum>(xs, NT * 8, p.M, p.K, p.x32, p.y1, p.s1, p.y2, p.s2, p.extra, second && p.norm_w2 != nullptr ? p.norm_w2 : p.norm_w, p.eps,
                         p.shift, p.mult, p.x32_out, rstd_s);
   } else {
-    stage_rows_async(xs, NT * 8, p.M, p.K, p.x);
+    stage_rows_async(xs, NT * 8, p.M, p.K, second && p.x2 != nullptr ? p.x2 : p.x, p.ldx);
     cp_commit();
     cp_wait<0>();
   }
@@ -437,7 +439,7 @@ __global__ void __launch_bounds__(kThreads) gemv_kernel(GemvParams p) {
     // second pass over the (cache-resident) activations: xn = bf16(h · rstd · w)
     for (int i = threadIdx.x; i < p.M * (p.K / 8); i += kThreads) {
       const int tok = i / (p.K / 8), kv = (i % (p.K / 8)) * 8;
-      uint4 xv = *reinterpret_cast<const uint4*>(p.x + static_cast<long long>(tok) * p.K + kv);
+      uint4 xv = *reinterpret_cast<const uint4*>(p.x + tok * p.ldx + kv);
       if (p.residual != nullptr) {
         const uint4 rv = *reinterpret_cast<const uint4*>(p.residual + static_cast<long long>(tok) * p.K + kv);
         add_residual(xv, rv);
@@ -527,7 +529,7 @@ __global__ void __launch_bounds__(kThreads) moe_gemv_up_kernel(const bf16* __res
     }
     if (lane == 0) n_slots_s = cnt;
   }
-  stage_rows_async(xs, 8, T, H, x);
+  stage_rows_async(xs, 8, T, H, x, H);
   cp_commit();
   cp_wait<0>();
   __syncthreads();
@@ -625,7 +627,7 @@ __global__ void __launch_bounds__(kThreads) moe_gemv_down_kernel(const bf16* __r
   const int n_pairs = T * k;
   // all pair rows of the activations → shared memory, in flight while warp 0 builds the expert table (rows of other
   // ranks' experts are copied too and never read)
-  stage_rows_async(as, n_pairs, n_pairs, F, act);
+  stage_rows_async(as, n_pairs, n_pairs, F, act, F);
   cp_commit();
   if (warp == 0) {
     // the distinct experts of the step with, per token, the pair routed to them and its gate weight
@@ -747,14 +749,15 @@ using namespace mb::gv;
 // norm_w != null: RMSNorm over K with weight norm_w (after adding `residual` when given) is applied to x first; res_out / xn_out
 // (optional) receive bf16(x + residual) and the normalised activations.  static_w: W is a parameter (not produced by a kernel that
 // may still be running), so its loads may start before the previous kernel has finished.
-extern "C" int mb_gemv(const void* x, const void* residual, const void* norm_w, float eps, const void* W, const void* bias, void* y,
+extern "C" int mb_gemv(const void* x, long long ldx, const void* residual, const void* norm_w, float eps, const void* W, const void* bias, void* y,
                        long long ldy, int out_fp32, void* res_out, void* xn_out, int M, int N, int K, int static_w, cudaStream_t s) {
   if (M <= 0 || N <= 0) return 0;
-  if (M > 16 || K % 32 || K <= 0) return -1;
+  if (M > 16 || K % 32 || K <= 0 || ldx % 8 || reinterpret_cast<uintptr_t>(x) % 16) return -1;
   const int nt = M <= 8 ? 1 : 2;
   if (kDenseStages * 2 * kThreads * 16 + nt * 8 * staged_stride(K) > kMaxSmem) return -2;
   GemvParams p{};
   p.x = reinterpret_cast<const bf16*>(x);
+  p.ldx = ldx;
   p.residual = reinterpret_cast<const bf16*>(residual);
   p.norm_w = reinterpret_cast<const bf16*>(norm_w);
   p.eps = eps;
@@ -799,12 +802,14 @@ extern "C" int mb_gemv_output_norm(const float* x, const void* y, const void* no
 // See launch.h; same limits as mb_gemv.
 extern "C" int mb_gemv_sum_norm(MbGemvSum a, cudaStream_t s) {
   if (a.M <= 0 || a.N <= 0) return 0;
-  if (a.M > 16 || a.K % 32 || a.K <= 0) return -1;
+  if (a.M > 16 || a.K % 32 || a.K <= 0 || (a.x != nullptr && (a.ldx % 8 || (reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.x2)) % 16))) return -1;
   const int nt = a.M <= 8 ? 1 : 2;
   if (kDenseStages * 2 * kThreads * 16 + nt * 8 * staged_stride(a.K) > kMaxSmem) return -2;
   auto b = [](const void* p) { return reinterpret_cast<const bf16*>(p); };
   GemvParams p{};
   p.x = b(a.x);
+  p.x2 = b(a.x2);
+  p.ldx = a.ldx;
   p.x32 = a.x32;
   p.y1 = b(a.y1); p.s1 = b(a.s1);
   p.y2 = b(a.y2); p.s2 = b(a.s2);

@@ -28,7 +28,7 @@ int mb_gemm_small(const void* X, const void* W, void* C, int tokens, int N, int 
 int mb_gemm_small_grouped(const void* X, const void* W, void* C, int rows, int N, int K, int num_experts, const int* tile_expert,
                           const int* used_rows, int bt, int* error_flag, cudaStream_t stream);
 // ---- gemv.cu: ≤ 16 tokens (dense) / ≤ 8 tokens (MoE), no pipeline set-up ----
-int mb_gemv(const void* x, const void* residual, const void* norm_w, float eps, const void* W, const void* bias, void* y, long long ldy,
+int mb_gemv(const void* x, long long ldx, const void* residual, const void* norm_w, float eps, const void* W, const void* bias, void* y, long long ldy,
             int out_fp32, void* res_out, void* xn_out, int M, int N, int K, int static_w, cudaStream_t s);
 int mb_moe_gemv(const void* x, const void* w13, const void* w2, const int* topk_idx, const float* topk_w, void* act, void* out, int T, int k,
                 int E, int expert_offset, int H, int F, float limit, float alpha, float shift, int ungated, cudaStream_t s);
@@ -257,7 +257,8 @@ typedef struct {
   const float* x32;
   const void *y1, *s1, *y2, *s2;
   const float* extra;
-  const void* x;
+  const void *x, *x2;                        // plain rows, ldx elements apart; x2: those of the second product (null: x)
+  long long ldx;
   const void *norm_w, *norm_w2;
   float eps, shift, mult;                    // mult: factor on the addends; norm_w null: the sum as it is
   const void* W;
@@ -363,10 +364,10 @@ int mb_delta_conv(const void* proj, long long ld, MbDelta m, const int* tiles, c
 // Any pieces token by token from the convolution's outputs (cu_q null: one token per sequence); out [T, H·V] = o.
 int mb_delta_seq(const void* proj, long long ld, const void* act, MbDelta m, const int* cu_q, void* out, int B, int f32, cudaStream_t s);
 // One token per sequence in one launch: convolution, state, and o over its root mean square per head, times norm_w [V] and sigmoid(gate).
-// V % 4 == 0, V ≤ 1024, K·V ≤ mb_delta_step_max().
+// Sizes: mb_delta_step_ok(K, V).
 int mb_delta_step(const void* proj, long long ld, MbDelta m, const void* norm_w, const void* gate, long long gate_ld, float eps, void* out, int B,
                   int f32, cudaStream_t s);
-int mb_delta_step_max(void);
+int mb_delta_step_ok(int K, int V);
 // Long pieces in chunks of 64 tokens on tensor cores (bf16; K, V multiples of 8 up to 128).  chunks [n_chunks][4]: sequence, first token,
 // end; parts [n_parts][4]: first chunk, chunks, sequence (a part's chunks follow one another; a sequence has one part).  scratch:
 // mb_delta_chunk_bytes(K, V) per chunk and head.  warps (2, 4 or 8): 16 value columns each that a CTA of the second kernel takes.

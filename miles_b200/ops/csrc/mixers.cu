@@ -346,6 +346,13 @@ __global__ void __launch_bounds__(256) head_gated_norm_kernel(const T* __restric
   }
 }
 
+// exp(z) − 1 − z for z ≤ 0; in bf16 models by its series near zero, where the difference would lose what matters
+template <typename T> __device__ __forceinline__ float exp_rest(float z) {
+  if constexpr (is_exact<T>::value) return expm1f(z) - z;
+  const float series = z * z * fmaf(z, fmaf(z, fmaf(z, 8.3333333e-3f, 4.1666667e-2f), 0.16666667f), 0.5f);
+  return z > -0.25f ? series : __expf(z) - 1.f - z;
+}
+
 template <typename T, int V>
 __global__ void __launch_bounds__(256) xielu_kernel(const T* __restrict__ z, const T* __restrict__ act, T* __restrict__ out, long long n) {
   pdl_trigger();
@@ -355,7 +362,7 @@ __global__ void __launch_bounds__(256) xielu_kernel(const T* __restrict__ z, con
     float a[V];
     load_n<V>(z + i, a);
 #pragma unroll
-    for (int j = 0; j < V; ++j) a[j] = fmaf(0.5f, a[j], a[j] > 0.f ? pos * a[j] * a[j] : neg * (expm1f(a[j]) - a[j]));
+    for (int j = 0; j < V; ++j) a[j] = fmaf(0.5f, a[j], a[j] > 0.f ? pos * a[j] * a[j] : neg * exp_rest<T>(a[j]));
     store_n<V>(out + i, a);
   }
 }
@@ -381,18 +388,25 @@ __global__ void __launch_bounds__(256) gelu_rows_kernel(const T* __restrict__ z,
   }
 }
 
-template <bool EXACT>
+template <bool EXACT, int V>
 __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long long n, float cap) {
   pdl_trigger();
   pdl_wait();
   const float inv = __fdiv_rn(1.f, cap);
-  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
-    if (EXACT) {
-      x[i] = static_cast<float>(cap * tanh(static_cast<double>(x[i]) / cap));
-    } else {                           // tanh u = 1 − 2 / (exp(2u) + 1), odd: exponentials of −2|u| never overflow
-      const float u = x[i] * inv, e = __expf(-2.f * fabsf(u));
-      x[i] = copysignf(cap * __fdividef(1.f - e, 1.f + e), u);
+#pragma unroll 2
+  for (long long i = (blockIdx.x * 256ll + threadIdx.x) * V; i < n; i += gridDim.x * 256ll * V) {
+    float a[V];
+    load_n<V>(x + i, a);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      if (EXACT) {
+        a[j] = static_cast<float>(cap * tanh(static_cast<double>(a[j]) / cap));
+      } else {                         // tanh u = (1 − e) / (1 + e) with e = exp(−2|u|), odd: nothing overflows
+        const float u = a[j] * inv, e = __expf(-2.f * fabsf(u));
+        a[j] = copysignf(cap * __fdividef(1.f - e, 1.f + e), u);
+      }
     }
+    store_n<V>(x + i, a);
   }
 }
 
@@ -488,7 +502,9 @@ extern "C" int mb_gelu_rows(const void* z, long long ld, const int* tok, const v
 extern "C" int mb_softcap(float* x, long long n, float cap, int exact, cudaStream_t s) {
   if (n <= 0) return 0;
   if (!(cap > 0.f)) return -3;
-  return static_cast<int>(launch_pdl(exact ? softcap_kernel<true> : softcap_kernel<false>, dim3(elementwise_blocks(n)), dim3(256), 0, s, x, n, cap));
+  const bool vec = n % 4 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0;
+  auto kern = exact ? (vec ? softcap_kernel<true, 4> : softcap_kernel<true, 1>) : (vec ? softcap_kernel<false, 4> : softcap_kernel<false, 1>);
+  return static_cast<int>(launch_pdl(kern, dim3(elementwise_blocks(vec ? n / 4 : n)), dim3(256), 0, s, x, n, cap));
 }
 
 extern "C" int mb_head_gated_norm(const void* o, const void* w, const void* gate, long long gate_ld, void* out, long long T, int H, int V, float eps, int f32,

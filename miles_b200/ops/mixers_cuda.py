@@ -362,29 +362,42 @@ def differential_attention(proj, lay, kc, vc, meta, scale, diff, temperature, lv
 
 # ---- gated delta rule -------------------------------------------------------------------------------------------------
 
-def _low_rank(x, w):
-    """x·wᵀ for rows that are part of a wider projection."""
+def _low_rank(x, w, x2, w2):
+    """(x·wᵀ, x2·w2ᵀ) for rows that are part of a wider projection."""
     if x.dtype != BF16:
-        return torch.nn.functional.linear(x, w)
-    K_ = x.shape[1]
-    if x.shape[0] > K.GEMV_M and K_ % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
-        out = _rows(x.shape[0], w.shape[0], BF16, x.device)
-        C.gemm(x, w, out, x.shape[0], w.shape[0], K_, x.stride(0), K_, out.stride(0), False, False, False, None, 0)
+        return torch.nn.functional.linear(x, w), torch.nn.functional.linear(x2, w2)
+    T = x.shape[0]
+
+    def aligned(a):
+        return a.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0
+
+    if T <= K.GEMV_M and x.shape[1] == x2.shape[1] and aligned(x) and aligned(x2) and K._gemv_k_ok(T, x.shape[1]) and max(w.shape[0], w2.shape[0]) <= GEMV_MAX_N:
+        y, y2 = (torch.empty(T, m.shape[0], dtype=BF16, device=x.device) for m in (w, w2))
+        C.gemv_sum_norm(None, None, None, None, None, None, x, None, None, 0.0, 0.0, w, y, w2, None, y2, None, None, _static(w) and _static(w2), x2=x2)
+        return y, y2
+
+    def one(a, m):
+        n = a.shape[1]
+        if T <= K.GEMV_M or n % 8 or not aligned(a):
+            return K.gemm_nt(a, m)
+        out = _rows(T, m.shape[0], BF16, a.device)
+        C.gemm(a, m, out, T, m.shape[0], n, a.stride(0), n, out.stride(0), False, False, False, None, 0)
         return out
-    return K.gemm_nt(x, w)
+
+    return one(x, w), one(x2, w2)
 
 
 def delta_rule(proj, lay, conv, w_a, w_g, A_log, dt_bias, norm_w, state, ring, meta, eps):
     T, dt, dev, rg = proj.shape[0], proj.dtype, proj.device, meta.ragged
     sizes = [lay.heads, lay.kv_heads, lay.dim, lay.vdim, lay.taps, lay.beta_at]
-    raw, gate = _low_rank(proj[:, lay.channels: lay.gate_at], w_a), _low_rank(proj[:, lay.gate_at: lay.beta_at], w_g)
+    raw, gate = _low_rank(proj[:, lay.channels: lay.gate_at], w_a, proj[:, lay.gate_at: lay.beta_at], w_g)
     out = torch.empty(T, lay.heads * lay.vdim, dtype=dt, device=dev)
 
     def tensors(slots, positions, raw):
         return [conv, A_log, dt_bias, state, ring, slots, positions, raw]
 
     slots, cu_q = meta.state_slots, rg.cu_q
-    if cu_q is None and _step_ok(lay):
+    if cu_q is None and C.delta_step_ok(lay.dim, lay.vdim):
         C.delta_step(proj, sizes, tensors(slots, meta.positions, raw), norm_w, gate, float(eps), out)
         return out
     act = torch.empty(T, lay.channels, dtype=dt, device=dev)
@@ -438,13 +451,6 @@ def scan_warps(pairs: int, vdim: int, sms: int = 148) -> int:
     share the SM."""
     slices = -(-vdim // 16)
     return min((-(-pairs * -(-slices // w) // sms) * cost, w) for w, cost in ((8, 1.0), (4, 0.6), (2, 0.45)) if w == 2 or w <= slices)[1]
-
-
-def _step_ok(lay) -> bool:
-    if lay.vdim % 4 or lay.vdim > 1024:
-        return False
-    rows = 256 // (lay.vdim // 4)
-    return -(-lay.dim // rows) * rows * lay.vdim <= C.delta_step_max() and (rows * lay.vdim + lay.vdim + 3 * lay.dim) * 4 <= 48 * 1024
 
 
 # ---- state-space mixer ------------------------------------------------------------------------------------------------
@@ -535,8 +541,10 @@ def softcap_(logits, cap, exact):
 
 
 def part_norm_linear(x, nw, parts, eps, w):
-    if parts == 1 and w.shape[0] <= GEMV_MAX_N and gemv_ok(x, w):
-        return K.add_rmsnorm_linear(x, None, nw, eps, w)[0]        # a handful of rows: the norm inside the product
+    if parts == 1 and w.shape[0] <= GEMV_MAX_N and gemv_ok(x, w) and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
+        y = torch.empty(x.shape[0], w.shape[0], dtype=BF16, device=x.device)
+        C.gemv(x, None, nw, float(eps), w, None, y, None, None, _static(w))      # a handful of rows: the norm inside the product
+        return y
     h = torch.empty(x.shape, dtype=x.dtype, device=x.device)
     C.part_norm(x, nw, h, parts, float(eps))
     return K.linear(h, w)
