@@ -112,7 +112,7 @@ struct Shared {
   float diagonal[4][16 * DP];              // A inside them
   float D[4][128], before[4][128], after[4][128], between[7][128];
   float fq[C], fk[C], beta[C], beta_k[C];
-  int direct[4], next;
+  int direct[4];
   uint64_t full;             // the inputs of a unit have come
 };
 
@@ -232,7 +232,6 @@ __global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(const __grid
     }
     if (tid < C) s.beta[tid] = tid < n_now ? mx::sigmoid_t<bf16>(__bfloat162float(beta_raw)) : 0.f;
     if (tid < 4) s.direct[tid] = 0;
-    if (tid == 4) s.next = 0;
     __syncthreads();
     {                                      // running sums inside the blocks: a thread per (block, channel)
       const int b = tid >> 7, c = tid & 127;
@@ -269,7 +268,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(const __grid
       s.beta_k[tid - 128] = s.beta[tid - 128] * s.fk[tid - 128];
     }
     __syncthreads();
-    // ---- q and k decayed from the start of their block, k to its end; queries decayed from the chunk's start
+    // ---- q and k decayed from the start of their block, k to its end; queries decayed from the chunk's start, keys to its end
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int r = my_row + i * 32, c = my_c, at = r * P + c;
@@ -311,6 +310,17 @@ __global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(const __grid
       split8(d, hi, lo);
       *reinterpret_cast<uint4*>(s.c_hi + at) = hi;
       *reinterpret_cast<uint4*>(s.c_lo + at) = lo;
+      if (c < kdk * 16) {
+        float f[8];
+        mx::load_n<8>(s.after[r >> 4] + c, f);
+        const float scale = s.fk[r];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) d[j] *= f[j] * scale;
+        split8(d, hi, lo);
+        uint8_t* to = unit + p.unit.k() + r * KR * 2 + (((c >> 3) ^ (r & 7)) << 4);
+        *reinterpret_cast<uint4*>(to) = hi;
+        *reinterpret_cast<uint4*>(to + half) = lo;
+      }
     }
     __syncthreads();
     // ---- A and B, a warp per pair of blocks; the diagonal blocks of I + A are inverted by the warps that made them
@@ -423,28 +433,6 @@ __global__ void __launch_bounds__(kThreads, 1) delta_prepare_kernel(const __grid
           s.a_hi[at + i * AP] = hi;
           s.a_lo[at + i * AP] = __float2bfloat16(x[i] - __bfloat162float(hi));
         }
-      }
-    }
-    // ---- keys decayed to the chunk's end: two rows at a time by whichever warp has nothing else to do
-    for (;;) {
-      int turn = 0;
-      if (lane == 0) turn = atomicAdd(&s.next, 1);
-      turn = __shfl_sync(0xffffffffu, turn, 0);
-      if (turn >= C / 2) break;
-      const int r = turn * 2 + (lane >> 4), piece = lane & 15, c = piece * 8, at = r * P + c;
-      if (c < kdk * 16) {
-        float x[8], y[8], f[8];
-        mx::load_n<8>(s.c_hi + at, x);
-        mx::load_n<8>(s.c_lo + at, y);
-        mx::load_n<8>(s.after[r >> 4] + c, f);
-        const float scale = s.fk[r];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) x[j] = (x[j] + y[j]) * (f[j] * scale);
-        uint4 hi, lo;
-        split8(x, hi, lo);
-        uint8_t* to = unit + p.unit.k() + r * KR * 2 + ((piece ^ (r & 7)) << 4);
-        *reinterpret_cast<uint4*>(to) = hi;
-        *reinterpret_cast<uint4*>(to + half) = lo;
       }
     }
     fence_proxy_async();                   // what was written to the tiles comes before the copies into them

@@ -379,7 +379,7 @@ def _low_rank(x, w, x2, w2):
     def one(a, m):
         n = a.shape[1]
         if T <= K.GEMV_M or n % 8 or not aligned(a):
-            return K.gemm_nt(a, m)
+            return K.gemm_nt(a.clone(memory_format=torch.contiguous_format), m)      # (a single row counts as contiguous wherever it starts)
         out = _rows(T, m.shape[0], BF16, a.device)
         C.gemm(a, m, out, T, m.shape[0], n, a.stride(0), n, out.stride(0), False, False, False, None, 0)
         return out

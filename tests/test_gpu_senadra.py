@@ -117,6 +117,7 @@ DELTAS = {
     "large": delta(2, 1, 160, 144, 4, 8, 8),                  # token by token
     "odd": delta(3, 3, 9, 7, 6, 5, 3),
     "many_taps": delta(2, 2, 16, 16, 20, 8, 8),
+    "off_the_grid": delta(1, 1, 9, 7, 2, 32, 64),             # inner rows of whole steps that start between 16-byte boundaries
 }
 
 
